@@ -11,8 +11,8 @@ constexpr int ATT_SOFTMAX_THREADS = 256;
 constexpr int ATT_THREADS = 64 + ATT_SOFTMAX_THREADS;
 constexpr int ATT_HALF_BYTES = 128 * 128;  // a [128 rows x 64 bf16] swizzled half tile
 
-// 2^x in one MUFU instruction (ex2.approx with flush-to-zero; exp2f() without fast-math wraps the same
-// instruction in range fix-ups that cost four more issue slots per element). Inputs here are <= 8 or -inf.
+// 2^x with the PTX approximation ex2.approx.ftz.f32: inputs here are <= 8 or -inf, so neither exp2f()'s full range
+// nor subnormal results are needed.
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
