@@ -2,6 +2,7 @@
 
     serve   the OpenAI-compatible server (all flags of ``entrypoints/api_server.py``)
     build   compile the CUDA kernels into ``tokenweave_b200/_C.so``
+    trace   replay given steps through a model and write logits (also ``bin/trace_run``)
     info    versions, devices and the kernels library in use
 """
 import sys
@@ -15,6 +16,9 @@ def main(argv=None) -> int:
         sys.argv = ["tokenweave_b200 serve"] + argv
         api_server.main()
         return 0
+    if cmd == "trace":
+        from .entrypoints import trace_run
+        return trace_run.main(argv)
     if cmd == "build":
         from . import build
         print(build.build())

@@ -21,11 +21,24 @@ _DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float32": torch.
            "float16": torch.float16, "half": torch.float16, "auto": None}
 
 
+# mixers of hybrid decoders that keep a state slot per sequence (layers/mixers.py)
+RECURRENT_MIXERS = ("mamba2",)
+# config.json's "architecture" -> reader(dict, name, path) -> ModelConfig, for designs not in the Hugging Face layout
+CONFIG_READERS: dict = {}
+
+
+def register_config_reader(architecture: str):
+    def wrap(fn):
+        CONFIG_READERS[architecture] = fn
+        return fn
+    return wrap
+
+
 @dataclass
 class ModelConfig:
     """Architecture of a decoder-only transformer (Llama-3.x, Qwen2.5, Mixtral layouts)."""
     name: str = "tiny-llama"
-    architecture: str = "llama"          # "llama" | "qwen2" | "mixtral" | "qwen3" | "mistral" | "phi3"
+    architecture: str = "llama"          # "llama" | "qwen2" | "mixtral" | "qwen3" | "mistral" | "phi3" | "sidisun"
     hidden_size: int = 256
     num_layers: int = 2
     num_q_heads: int = 4
@@ -53,12 +66,22 @@ class ModelConfig:
     # weight-only integer checkpoints (AWQ, GPTQ): {"method", "bits", "group_size", "zeros_plus_one"}; their packed
     # tensors are expanded to the model's dtype while loading (models/loader.py)
     checkpoint_packing: Optional[dict] = None
+    # hybrid decoders (models/hybrid.py): one {"type", "mixer", "mlp"} per layer; None for the uniform families above
+    layers: Optional[list] = None
+    logit_scale: float = 1.0             # factor on the logits (hybrid decoders)
+
+    @property
+    def has_state(self) -> bool:
+        """Some layer keeps recurrent state: a request holds a state slot besides its cache blocks."""
+        return any(l["type"] in RECURRENT_MIXERS for l in self.layers or ())
 
     @property
     def is_moe(self) -> bool:
         return self.num_experts > 0
 
     def num_params(self) -> int:
+        if self.layers:
+            raise NotImplementedError("num_params counts the uniform families")
         h, l = self.hidden_size, self.num_layers
         attn = h * (self.num_q_heads + 2 * self.num_kv_heads) * self.head_dim + self.num_q_heads * self.head_dim * h
         mlp = 3 * h * self.intermediate_size * max(1, self.num_experts)
@@ -67,6 +90,13 @@ class ModelConfig:
 
     @staticmethod
     def from_hf_dict(cfg: dict, name: str = "", path: Optional[str] = None) -> "ModelConfig":
+        if "architecture" in cfg:            # configurations of designs with a reader of their own
+            from .models import registry     # noqa: F401  (its import registers the readers)
+            registry.load_config_readers()
+            reader = CONFIG_READERS.get(cfg["architecture"])
+            if reader is None:
+                raise ValueError(f"unsupported architecture {cfg['architecture']!r} (readers: {sorted(CONFIG_READERS)})")
+            return reader(cfg, name, path)
         archs = cfg.get("architectures") or [cfg.get("model_type", "llama")]
         a = archs[0].lower()
         if any(k in a for k in ("moe", "vl", "omni", "audio")) and "mixtral" not in a:
@@ -155,6 +185,19 @@ def _preset(**kw) -> ModelConfig:
     return ModelConfig(**kw)
 
 
+def _latent_layer(heads, dim, rot, vdim, kv_rank, q_rank, ff, base=10000.0, scaling=None) -> dict:
+    return {"type": "latent_attention",
+            "mixer": dict(heads=heads, dim=dim, rot_dim=rot, vdim=vdim, kv_rank=kv_rank, q_rank=q_rank,
+                          scale=(dim + rot) ** -0.5, rot=dict(base=base, dims=rot, scaling=scaling)),
+            "mlp": None if ff is None else dict(kind="dense", ff=ff)}
+
+
+def _mamba2_layer(heads, vdim, state, groups, ff, conv=4, norm_groups=1) -> dict:
+    return {"type": "mamba2", "mixer": dict(heads=heads, vdim=vdim, state=state, groups=groups, conv=conv,
+                                            norm_groups=norm_groups),
+            "mlp": None if ff is None else dict(kind="dense", ff=ff)}
+
+
 MODEL_PRESETS: dict[str, dict[str, Any]] = {
     # correctness configuration: fp32 on CPU, split path must equal the unsplit path
     "tiny-llama": dict(architecture="llama", hidden_size=256, num_layers=2, num_q_heads=4, num_kv_heads=2,
@@ -185,6 +228,14 @@ MODEL_PRESETS: dict[str, dict[str, Any]] = {
     "phi-3-medium-4k": dict(architecture="phi3", hidden_size=5120, num_layers=40, num_q_heads=40, num_kv_heads=10,
                             head_dim=128, intermediate_size=17920, vocab_size=32064, rms_norm_eps=1e-5,
                             rope_theta=10000.0, max_model_len=4096),
+    "tiny-sidisun": dict(architecture="sidisun", hidden_size=160, num_layers=3, num_q_heads=6, num_kv_heads=1, head_dim=56,
+                         intermediate_size=256, vocab_size=512, rms_norm_eps=1e-5, max_model_len=4096, logit_scale=0.5,
+                         layers=[_mamba2_layer(8, 40, 48, 2, 256, norm_groups=2), _latent_layer(6, 40, 16, 32, 96, 64, 256),
+                                 _mamba2_layer(8, 40, 48, 2, None, norm_groups=2)]),
+    "sidisun-8b": dict(architecture="sidisun", hidden_size=4096, num_layers=32, num_q_heads=32, num_kv_heads=1,
+                       head_dim=192, intermediate_size=16384, vocab_size=128256, rms_norm_eps=1e-5, max_model_len=131072,
+                       layers=[_latent_layer(32, 128, 64, 128, 512, 1536, 16384, base=500000.0) if i % 4 == 3
+                               else _mamba2_layer(128, 64, 128, 8, 16384, norm_groups=8) for i in range(32)]),
     "llama-3.3-70b": dict(architecture="llama", hidden_size=8192, num_layers=80, num_q_heads=64, num_kv_heads=8,
                           head_dim=128, intermediate_size=28672, vocab_size=128256, rms_norm_eps=1e-5,
                           rope_theta=500000.0, max_model_len=131072,
@@ -225,6 +276,9 @@ def resolve_model_config(model: "str | ModelConfig", dtype: Optional[str] = None
         cfg.max_model_len = max_model_len
     if num_layers:
         cfg.num_layers = num_layers
+        if cfg.layers:
+            cfg.layers = cfg.layers[:num_layers]
+            cfg.num_layers = len(cfg.layers)
     return cfg
 
 
@@ -390,6 +444,7 @@ class EngineArgs:
             if model.num_experts % self.tensor_parallel_size:
                 raise ValueError("enable_expert_parallel needs num_experts divisible by tensor_parallel_size")
             model.expert_parallel = True
+        self._check_hybrid(model)
         max_len = model.max_model_len
         budget = self.max_num_batched_tokens or (8192 if self.enable_chunked_prefill else max(max_len, 8192))
         if self.quantization is None and model.checkpoint_quantization is not None:
@@ -426,6 +481,24 @@ class EngineArgs:
             disable_log_stats=self.disable_log_stats, enable_sleep_mode=self.enable_sleep_mode,
             speculative=self._speculative(), enable_lora=self._lora_checked(model), max_loras=self.max_loras,
             kv_transfer=self._kv_transfer(), engine_core_process=self.engine_core_process)
+
+    def _check_hybrid(self, model) -> None:
+        """Options a layer-list model cannot take are refused here, before any weight is read."""
+        if not model.layers:
+            return
+        refused = [("tensor_parallel_size > 1", self.tensor_parallel_size > 1),
+                   ("pipeline_parallel_size > 1", self.pipeline_parallel_size > 1),
+                   ("quantization", self.quantization is not None), ("enable_lora", self.enable_lora),
+                   ("tokenweave_force_overlap", self.tokenweave_force_overlap),
+                   ("kv_transfer_config", self.kv_transfer_config is not None)]
+        if model.has_state:
+            # a recurrent state exists for the end of a sequence only: it can neither be entered at a cached prefix
+            # nor taken back by rejected draft tokens
+            refused += [("enable_prefix_caching", self.enable_prefix_caching),
+                        ("speculative_config", self.speculative_config is not None)]
+        bad = [name for name, on in refused if on]
+        if bad:
+            raise ValueError(f"{model.architecture} does not support {', '.join(bad)}")
 
     def _kv_transfer(self):
         from .engine.kv_connector import KVTransferConfig

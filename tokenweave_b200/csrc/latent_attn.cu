@@ -1,0 +1,467 @@
+// Latent attention (keys and values are linear maps of one low-rank latent per token): the kernels around the paged
+// latent cache, for bf16 and fp32 storage and any sizes.
+//
+// A cache row holds [latent c (kv_rank) | zero pad | rotated key part (rot) | zero pad], both parts padded to eight
+// elements, `row` elements in all. In the absorbed form a head's query for such a row is
+// [W_uk^T q_unrotated | pad | q_rotated | pad] (W_uk: the head's key map), so a score is one dot product over a row,
+// the value is the latent part of the same row, and the head's output is W_uv applied to the weighted latent sum.
+//
+//   tw_latent_prep     per token: RMS norm of the query latent; RMS norm of the key/value latent and rotation of the
+//                      shared key part, both written straight into the cache slot
+//   tw_rope_tail       rotates the tail of every head of q in place (the un-absorbed prefill form)
+//   tw_latent_query    the rotated tail and the pads of absorbed query rows
+//   tw_head_gemm       out[t, h, :] = B[h] a[t, h, :] for every head, rows through optional index lists, optionally
+//                      times sigmoid(gate) element by element (tensor cores for bf16)
+//   tw_latent_attn     absorbed causal attention of single query rows over the paged cache, fp32 softmax
+//   tw_latent_gather   cache rows of some sequences, in order, into one contiguous buffer
+#include "tw_host.h"
+#include "tw_kernels.h"
+#include "tw_typed.cuh"
+
+namespace tw {
+
+__device__ __forceinline__ int round8(int x) { return (x + 7) & ~7; }
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+latent_prep_kernel(const T* __restrict__ p, long long ldp, int q_off, int q_rank, const T* __restrict__ wq,
+                   T* __restrict__ cq, long long ldcq, int kv_off, int kv_rank, const T* __restrict__ wkv, int rot,
+                   int rot_dims, const float* __restrict__ cos_sin, const int* __restrict__ positions,
+                   const int* __restrict__ slots, T* __restrict__ cache, int row, float eps) {
+  __shared__ float scratch[64];
+  const int t = blockIdx.x;
+  const T* src = p + t * ldp;
+  float s[2] = {0.f, 0.f};
+  for (int i = threadIdx.x * 8; i < q_rank; i += blockDim.x * 8) {
+    float v[8];
+    ld8n<VEC>(src + q_off + i, q_rank - i, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s[0] += v[j] * v[j];
+  }
+  for (int i = threadIdx.x * 8; i < kv_rank; i += blockDim.x * 8) {
+    float v[8];
+    ld8n<VEC>(src + kv_off + i, kv_rank - i, v);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) s[1] += v[j] * v[j];
+  }
+  block_sum<2>(s, scratch);
+  const float rq = 1.f / sqrtf(s[0] / static_cast<float>(q_rank) + eps);
+  const float rk = 1.f / sqrtf(s[1] / static_cast<float>(kv_rank) + eps);
+  for (int i = threadIdx.x * 8; i < q_rank; i += blockDim.x * 8) {
+    float v[8], g[8];
+    ld8n<VEC>(src + q_off + i, q_rank - i, v);
+    ld8n<VEC>(wq + i, q_rank - i, g);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = v[j] * rq * g[j];
+    st8n<VEC>(cq + t * ldcq + i, q_rank - i, v);
+  }
+  const int slot = slots[t];
+  if (slot < 0) return;
+  T* dst = cache + static_cast<long long>(slot) * row;
+  const int rp = round8(kv_rank);
+  for (int i = threadIdx.x * 8; i < rp; i += blockDim.x * 8) {
+    float v[8], g[8];
+    ld8n<VEC>(src + kv_off + i, kv_rank - i, v);
+    ld8n<VEC>(wkv + i, kv_rank - i, g);
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = v[j] * rk * g[j];
+    st8(dst + i, v);                       // the pad behind the latent is written as zeros
+  }
+  const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot_dims;
+  const int half = rot_dims >> 1;
+  for (int i = threadIdx.x; i < row - rp; i += blockDim.x) {
+    float v = 0.f;
+    if (i < half) {
+      v = ld1(src + kv_off + kv_rank + i) * cs[i] - ld1(src + kv_off + kv_rank + half + i) * cs[half + i];
+    } else if (i < rot_dims) {
+      v = ld1(src + kv_off + kv_rank + i) * cs[i - half] + ld1(src + kv_off + kv_rank + i - half) * cs[i];
+    } else if (i < rot) {
+      v = ld1(src + kv_off + kv_rank + i);
+    }
+    st1(dst + rp + i, v);
+  }
+}
+
+// Rotates elements [off, off + rot_dims) of every head of the listed rows in place.
+template <typename T>
+__global__ void __launch_bounds__(256)
+rope_tail_kernel(T* __restrict__ q, long long ldq, int heads, int head_stride, int off, int rot_dims,
+                 const float* __restrict__ cos_sin, const int* __restrict__ positions) {
+  const int t = blockIdx.x;
+  const int half = rot_dims >> 1;
+  const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot_dims;
+  for (int i = threadIdx.x; i < heads * half; i += blockDim.x) {
+    const int h = i / half, j = i - h * half;
+    T* u = q + t * ldq + h * head_stride + off + j;
+    const float a = ld1(u), b = ld1(u + half), c = cs[j], s = cs[half + j];
+    st1(u, a * c - b * s);
+    st1(u + half, b * c + a * s);
+  }
+}
+
+// qa: [n, heads, row] absorbed queries; fills everything behind the kv_rank columns the head GEMM writes.
+template <typename T>
+__global__ void __launch_bounds__(256)
+latent_query_kernel(const T* __restrict__ q, long long ldq, const int* __restrict__ rows, T* __restrict__ qa, int heads,
+                    int head_stride, int off, int rot, int rot_dims, int kv_rank, int row,
+                    const float* __restrict__ cos_sin, const int* __restrict__ positions) {
+  const int i = blockIdx.x;
+  const int t = rows[i];
+  const int half = rot_dims >> 1;
+  const int rp = round8(kv_rank), tail = row - kv_rank;
+  const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot_dims;
+  for (int e = threadIdx.x; e < heads * tail; e += blockDim.x) {
+    const int h = e / tail, c = kv_rank + e - h * tail, j = c - rp;
+    const T* src = q + t * ldq + h * head_stride + off;
+    float v = 0.f;
+    if (j >= 0 && j < half) v = ld1(src + j) * cs[j] - ld1(src + half + j) * cs[half + j];
+    else if (j >= half && j < rot_dims) v = ld1(src + j) * cs[j - half] + ld1(src + j - half) * cs[j];
+    else if (j >= rot_dims && j < rot) v = ld1(src + j);
+    st1(qa + (static_cast<long long>(i) * heads + h) * row + c, v);
+  }
+}
+
+// ---- per-head matrix product -------------------------------------------------------------------------
+struct HeadGemm {
+  const void* A; long long lda; int a_hs; const int* a_rows;     // A[row, h * a_hs + k]
+  const void* B; long long b_hs; int ldb;                        // B[h * b_hs + n * ldb + k]
+  void* C; long long ldc; int c_hs; const int* c_rows;           // C[row, h * c_hs + n]
+  const void* gate; long long ldg; int g_hs;                     // gate[c row, h * g_hs + n] or null
+  int M, N, K;
+};
+
+constexpr int HG_M = 64, HG_N = 64, HG_K = 64;
+constexpr int HG_LD = HG_K + 8;        // padded rows: conflict-free ldmatrix
+
+__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// VEC: K, the strides and the bases keep 16-byte groups aligned.
+template <bool VEC>
+__device__ __forceinline__ void hg_load(__nv_bfloat16* dst, const __nv_bfloat16* src, bool row_ok, int k_left) {
+  // eight elements of one row; beyond the row's end or for rows outside the problem they are zero
+  uint4 u = make_uint4(0, 0, 0, 0);
+  if (row_ok) {
+    if (VEC && k_left >= 8) {
+      u = *reinterpret_cast<const uint4*>(src);
+    } else {
+      __nv_bfloat16* e = reinterpret_cast<__nv_bfloat16*>(&u);
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        if (j < k_left) e[j] = src[j];
+    }
+  }
+  *reinterpret_cast<uint4*>(dst) = u;
+}
+
+template <bool VEC>
+__global__ void __launch_bounds__(128)
+head_gemm_bf16_kernel(const HeadGemm g) {
+  __shared__ __align__(16) __nv_bfloat16 sa[HG_M * HG_LD], sb[HG_N * HG_LD];
+  const int h = blockIdx.z, m0 = blockIdx.y * HG_M, n0 = blockIdx.x * HG_N;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int wm = (warp & 1) * 32, wn = (warp >> 1) * 32;
+  const __nv_bfloat16* A = reinterpret_cast<const __nv_bfloat16*>(g.A) + static_cast<long long>(h) * g.a_hs;
+  const __nv_bfloat16* B = reinterpret_cast<const __nv_bfloat16*>(g.B) + h * g.b_hs;
+  float acc[2][4][4] = {};
+  const int lr = threadIdx.x >> 3, lc = (threadIdx.x & 7) * 8;      // 16 rows x 8 groups per pass
+  const __nv_bfloat16* arow[4];
+  const __nv_bfloat16* brow[4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + lr + 16 * i, n = n0 + lr + 16 * i;
+    arow[i] = m < g.M ? A + (g.a_rows != nullptr ? g.a_rows[m] : m) * g.lda : nullptr;
+    brow[i] = n < g.N ? B + static_cast<long long>(n) * g.ldb : nullptr;
+  }
+  for (int k0 = 0; k0 < g.K; k0 += HG_K) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int off = (lr + 16 * i) * HG_LD + lc;
+      hg_load<VEC>(sa + off, arow[i] + k0 + lc, arow[i] != nullptr && k0 + lc < g.K, g.K - k0 - lc);
+      hg_load<VEC>(sb + off, brow[i] + k0 + lc, brow[i] != nullptr && k0 + lc < g.K, g.K - k0 - lc);
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < HG_K; k += 16) {
+      uint32_t a[2][4], b[2][4];
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        ldmatrix_x4(a[i], smem_u32(sa + (wm + i * 16 + (lane & 15)) * HG_LD + k + (lane >> 4) * 8));
+        // two 8-column blocks of B: registers 0, 1 belong to the first, 2, 3 to the second
+        ldmatrix_x4(b[i], smem_u32(sb + (wn + i * 16 + (lane >> 4) * 8 + (lane & 7)) * HG_LD + k + ((lane >> 3) & 1) * 8));
+      }
+#pragma unroll
+      for (int i = 0; i < 2; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) mma_bf16(acc[i][j], a[i], b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
+    }
+    __syncthreads();
+  }
+  __nv_bfloat16* C = reinterpret_cast<__nv_bfloat16*>(g.C) + static_cast<long long>(h) * g.c_hs;
+  const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(g.gate);
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int m = m0 + wm + i * 16 + half * 8 + (lane >> 2);
+      if (m >= g.M) continue;
+      const long long r = g.c_rows != nullptr ? g.c_rows[m] : m;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int n = n0 + wn + j * 8 + (lane & 3) * 2 + e;
+          if (n >= g.N) continue;
+          float v = acc[i][j][half * 2 + e];
+          if (gate != nullptr) v *= sigmoid_f(ld1(gate + r * g.ldg + static_cast<long long>(h) * g.g_hs + n));
+          C[r * g.ldc + n] = __float2bfloat16_rn(v);
+        }
+      }
+    }
+}
+
+__global__ void __launch_bounds__(256)
+head_gemm_f32_kernel(const HeadGemm g) {
+  __shared__ float sa[16][64 + 4], sb[16][64 + 4];
+  const int h = blockIdx.z, m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
+  const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
+  const float* A = reinterpret_cast<const float*>(g.A) + static_cast<long long>(h) * g.a_hs;
+  const float* B = reinterpret_cast<const float*>(g.B) + h * g.b_hs;
+  float acc[4][4] = {};
+  for (int k0 = 0; k0 < g.K; k0 += 16) {
+    for (int i = threadIdx.x; i < 64 * 16; i += 256) {
+      const int r = i >> 4, k = i & 15, m = m0 + r, n = n0 + r;
+      const bool kin = k0 + k < g.K;
+      sa[k][r] = (kin && m < g.M) ? A[(g.a_rows != nullptr ? g.a_rows[m] : m) * g.lda + k0 + k] : 0.f;
+      sb[k][r] = (kin && n < g.N) ? B[static_cast<long long>(n) * g.ldb + k0 + k] : 0.f;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < 16; ++k)
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(sa[k][ty * 4 + i], sb[k][tx * 4 + j], acc[i][j]);
+    __syncthreads();
+  }
+  float* C = reinterpret_cast<float*>(g.C) + static_cast<long long>(h) * g.c_hs;
+  const float* gate = reinterpret_cast<const float*>(g.gate);
+  for (int i = 0; i < 4; ++i) {
+    const int m = m0 + ty * 4 + i;
+    if (m >= g.M) continue;
+    const long long r = g.c_rows != nullptr ? g.c_rows[m] : m;
+    for (int j = 0; j < 4; ++j) {
+      const int n = n0 + tx * 4 + j;
+      if (n >= g.N) continue;
+      float v = acc[i][j];
+      if (gate != nullptr) v *= sigmoid_f(gate[r * g.ldg + static_cast<long long>(h) * g.g_hs + n]);
+      C[r * g.ldc + n] = v;
+    }
+  }
+}
+
+// ---- absorbed attention, any sizes ---------------------------------------------------------------------
+// One warp per (query row, head): lane l holds elements l, l + 32, ... of the query and of the output latent. A key
+// costs one pass over its cache row: dot product, shuffle reduction, and the same registers feed the weighted sum.
+template <typename T, int NK>
+__global__ void __launch_bounds__(128)
+latent_attn_kernel(const T* __restrict__ qa, const T* __restrict__ cache, const int* __restrict__ tok_seq,
+                   const int* __restrict__ tok_kvlen, const int* __restrict__ block_table, int max_blocks, int page,
+                   T* __restrict__ out, int heads, int row, int kv_rank, float scale) {
+  const int i = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (h >= heads) return;
+  const long long item = static_cast<long long>(i) * heads + h;
+  float q[NK], o[NK];
+#pragma unroll
+  for (int k = 0; k < NK; ++k) {
+    const int c = lane + 32 * k;
+    q[k] = c < row ? ld1(qa + item * row + c) * scale : 0.f;
+    o[k] = 0.f;
+  }
+  const int* table = block_table + static_cast<long long>(tok_seq[i]) * max_blocks;
+  const int n_keys = tok_kvlen[i];
+  float m = -INFINITY, l = 0.f;
+  for (int j0 = 0; j0 < n_keys; j0 += 2) {
+    float x[2][NK], s[2];
+#pragma unroll
+    for (int u = 0; u < 2; ++u) {
+      const int j = min(j0 + u, n_keys - 1);
+      const T* src = cache + (static_cast<long long>(table[j / page]) * page + j % page) * row;
+      s[u] = 0.f;
+#pragma unroll
+      for (int k = 0; k < NK; ++k) {
+        const int c = lane + 32 * k;
+        x[u][k] = c < row ? ld1(src + c) : 0.f;
+        s[u] = fmaf(q[k], x[u][k], s[u]);
+      }
+    }
+#pragma unroll
+    for (int u = 0; u < 2; ++u) s[u] = warp_sum(s[u]);
+    if (j0 + 1 >= n_keys) s[1] = -INFINITY;
+    const float mn = fmaxf(m, fmaxf(s[0], s[1]));
+    const float a = expf(m - mn), p0 = expf(s[0] - mn), p1 = expf(s[1] - mn);
+    m = mn;
+    l = l * a + p0 + p1;
+#pragma unroll
+    for (int k = 0; k < NK; ++k) o[k] = fmaf(o[k], a, fmaf(p0, x[0][k], p1 * x[1][k]));
+  }
+  const float inv = 1.f / l;
+#pragma unroll
+  for (int k = 0; k < NK; ++k) {
+    const int c = lane + 32 * k;
+    if (c < kv_rank) st1(out + item * kv_rank + c, o[k] * inv);
+  }
+}
+
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint4* __restrict__ cache, uint4* __restrict__ dst, const int* __restrict__ seqs,
+                     const int* __restrict__ cu, const int* __restrict__ block_table, int max_blocks, int page,
+                     int row_vec) {
+  const int b = blockIdx.y;
+  const int n = cu[b + 1] - cu[b], first = blockIdx.x * page;
+  if (first >= n) return;
+  const int rows = min(page, n - first);
+  const long long src = static_cast<long long>(block_table[static_cast<long long>(seqs[b]) * max_blocks + blockIdx.x]) * page * row_vec;
+  const long long to = (static_cast<long long>(cu[b]) + first) * row_vec;
+  for (int i = threadIdx.x; i < rows * row_vec; i += blockDim.x) dst[to + i] = cache[src + i];
+}
+
+static int check_launch(const char* what) {
+  const cudaError_t e = cudaGetLastError();
+  if (e == cudaSuccess) return 0;
+  set_last_error("%s launch failed: %s", what, cudaGetErrorString(e));
+  return 1;
+}
+static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+}  // namespace tw
+
+using namespace tw;
+
+extern "C" int tw_latent_prep(const void* p, long long ldp, int q_off, int q_rank, const void* wq, void* cq,
+                              long long ldcq, int kv_off, int kv_rank, const void* wkv, int rot, int rot_dims,
+                              const float* cos_sin, const int* positions, const int* slots, void* cache, int row, int T,
+                              float eps, int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (row % 8 != 0 || rot_dims % 2 != 0 || rot_dims > rot || row < ((kv_rank + 7) & ~7) + rot) {
+    set_last_error("latent_prep: bad row layout (row=%d, kv_rank=%d, rot=%d, rotated=%d)", row, kv_rank, rot, rot_dims);
+    return 1;
+  }
+  const bool vec = ldp % 8 == 0 && q_off % 8 == 0 && kv_off % 8 == 0 && ldcq % 8 == 0 && aligned16(p) && aligned16(cq) &&
+                   aligned16(wq) && aligned16(wkv);
+  const int n = q_rank > kv_rank ? q_rank : kv_rank;
+  int threads = ((n + 7) / 8 + 31) / 32 * 32;
+  if (threads > 256) threads = 256;
+#define TW_GO(TT, V)                                                                                                   \
+  latent_prep_kernel<TT, V><<<T, threads, 0, stream>>>(                                                                \
+      reinterpret_cast<const TT*>(p), ldp, q_off, q_rank, reinterpret_cast<const TT*>(wq), reinterpret_cast<TT*>(cq), \
+      ldcq, kv_off, kv_rank, reinterpret_cast<const TT*>(wkv), rot, rot_dims, cos_sin, positions, slots,               \
+      reinterpret_cast<TT*>(cache), row, eps)
+  if (dtype == TW_BF16) {
+    if (vec) TW_GO(__nv_bfloat16, true); else TW_GO(__nv_bfloat16, false);
+  } else {
+    if (vec) TW_GO(float, true); else TW_GO(float, false);
+  }
+#undef TW_GO
+  return check_launch("latent_prep");
+}
+
+extern "C" int tw_rope_tail(void* q, long long ldq, int T, int heads, int head_stride, int off, int rot_dims,
+                            const float* cos_sin, const int* positions, int dtype, cudaStream_t stream) {
+  if (T <= 0 || rot_dims <= 0) return 0;
+  if (dtype == TW_BF16)
+    rope_tail_kernel<__nv_bfloat16><<<T, 256, 0, stream>>>(reinterpret_cast<__nv_bfloat16*>(q), ldq, heads, head_stride,
+                                                           off, rot_dims, cos_sin, positions);
+  else
+    rope_tail_kernel<float><<<T, 256, 0, stream>>>(reinterpret_cast<float*>(q), ldq, heads, head_stride, off, rot_dims,
+                                                   cos_sin, positions);
+  return check_launch("rope_tail");
+}
+
+extern "C" int tw_latent_query(const void* q, long long ldq, const int* rows, int n, void* qa, int heads,
+                               int head_stride, int off, int rot, int rot_dims, int kv_rank, int row,
+                               const float* cos_sin, const int* positions, int dtype, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (dtype == TW_BF16)
+    latent_query_kernel<__nv_bfloat16><<<n, 256, 0, stream>>>(
+        reinterpret_cast<const __nv_bfloat16*>(q), ldq, rows, reinterpret_cast<__nv_bfloat16*>(qa), heads, head_stride,
+        off, rot, rot_dims, kv_rank, row, cos_sin, positions);
+  else
+    latent_query_kernel<float><<<n, 256, 0, stream>>>(reinterpret_cast<const float*>(q), ldq, rows,
+                                                      reinterpret_cast<float*>(qa), heads, head_stride, off, rot,
+                                                      rot_dims, kv_rank, row, cos_sin, positions);
+  return check_launch("latent_query");
+}
+
+extern "C" int tw_head_gemm(const void* A, long long lda, int a_hs, const int* a_rows, const void* B, long long b_hs,
+                            int ldb, void* C, long long ldc, int c_hs, const int* c_rows, const void* gate,
+                            long long ldg, int g_hs, int heads, int M, int N, int K, int dtype, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || heads <= 0) return 0;
+  const HeadGemm g{A, lda, a_hs, a_rows, B, b_hs, ldb, C, ldc, c_hs, c_rows, gate, ldg, g_hs, M, N, K};
+  const dim3 grid((N + 63) / 64, (M + 63) / 64, heads);
+  if (grid.y > 65535 || grid.z > 65535) {
+    set_last_error("head_gemm: too many rows (%d) or heads (%d)", M, heads);
+    return 1;
+  }
+  if (dtype == TW_BF16) {
+    const bool vec = K % 8 == 0 && lda % 8 == 0 && a_hs % 8 == 0 && b_hs % 8 == 0 && ldb % 8 == 0 && aligned16(A) &&
+                     aligned16(B);
+    if (vec) head_gemm_bf16_kernel<true><<<grid, 128, 0, stream>>>(g);
+    else head_gemm_bf16_kernel<false><<<grid, 128, 0, stream>>>(g);
+  } else {
+    head_gemm_f32_kernel<<<grid, 256, 0, stream>>>(g);
+  }
+  return check_launch("head_gemm");
+}
+
+extern "C" int tw_latent_attn(const void* qa, const void* cache, const int* tok_seq, const int* tok_kvlen, int n,
+                              const int* block_table, int max_blocks, int page, void* out, int heads, int row,
+                              int kv_rank, float scale, int dtype, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  const dim3 grid(n, (heads + 3) / 4);
+#define TW_GO(NK)                                                                                                      \
+  do {                                                                                                                 \
+    if (dtype == TW_BF16)                                                                                              \
+      latent_attn_kernel<__nv_bfloat16, NK><<<grid, 128, 0, stream>>>(                                                 \
+          reinterpret_cast<const __nv_bfloat16*>(qa), reinterpret_cast<const __nv_bfloat16*>(cache), tok_seq, tok_kvlen, \
+          block_table, max_blocks, page, reinterpret_cast<__nv_bfloat16*>(out), heads, row, kv_rank, scale);           \
+    else                                                                                                               \
+      latent_attn_kernel<float, NK><<<grid, 128, 0, stream>>>(                                                         \
+          reinterpret_cast<const float*>(qa), reinterpret_cast<const float*>(cache), tok_seq, tok_kvlen, block_table,  \
+          max_blocks, page, reinterpret_cast<float*>(out), heads, row, kv_rank, scale);                                \
+  } while (0)
+  if (row <= 64) TW_GO(2);
+  else if (row <= 128) TW_GO(4);
+  else if (row <= 192) TW_GO(6);
+  else if (row <= 320) TW_GO(10);
+  else if (row <= 576) TW_GO(18);
+  else if (row <= 1152) TW_GO(36);
+  else {
+    set_last_error("latent_attn: cache rows of up to 1152 elements are supported (got %d)", row);
+    return 1;
+  }
+#undef TW_GO
+  return check_launch("latent_attn");
+}
+
+extern "C" int tw_latent_gather(const void* cache, void* dst, const int* seqs, const int* cu, int n_seqs,
+                                int max_rows, const int* block_table, int max_blocks, int page, int row_bytes,
+                                cudaStream_t stream) {
+  if (n_seqs <= 0 || max_rows <= 0) return 0;
+  if (row_bytes % 16 != 0) {
+    set_last_error("latent_gather: rows of %d bytes are not a multiple of 16", row_bytes);
+    return 1;
+  }
+  const dim3 grid((max_rows + page - 1) / page, n_seqs);
+  latent_gather_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<const uint4*>(cache), reinterpret_cast<uint4*>(dst),
+                                                 seqs, cu, block_table, max_blocks, page, row_bytes / 16);
+  return check_launch("latent_gather");
+}

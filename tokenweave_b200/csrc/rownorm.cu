@@ -1,0 +1,288 @@
+// Row-wise kernels around the residual stream and the feed-forward of models that norm a sublayer's OUTPUT.
+// The residual stream is fp32; activations are bf16 or fp32 (template argument), all arithmetic is fp32.
+//
+//   tw_embed_residual   x32 = table[id] (the residual stream), xa = the same in the activation type
+//   tw_postnorm_add     x32 += rmsnorm(y) * w ; xa = x32, or rmsnorm(x32) * w_final behind the last layer
+//   tw_polynorm         out = a N(z) + b N(z^2) + c N(z^3) + e with N(v) = v / rms(v) over the row, powers
+//                       element by element (the activation between the two matrices of a feed-forward)
+//   tw_gated_group_norm out = groupnorm_rms(y * silu(z)) * w, the row cut in equal groups, each with its own
+//                       root mean square (what follows a state-space recurrence)
+//
+// One CTA per row (per row and group), the row kept in registers between the passes when it fits.
+#include "tw_host.h"
+#include "tw_kernels.h"
+#include "tw_typed.cuh"
+
+namespace tw {
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+embed_residual_kernel(const int* __restrict__ ids, const T* __restrict__ table, long long ldt, float* __restrict__ x32,
+                      long long ldx, T* __restrict__ xa, long long lda, int H, int vocab) {
+  const int t = blockIdx.x;
+  const int id = ids[t];
+  const bool ok = id >= 0 && id < vocab;
+  const T* src = table + (ok ? id : 0) * ldt;
+  for (int i = threadIdx.x * 8; i < H; i += blockDim.x * 8) {
+    float v[8];
+    ld8n<VEC>(src + i, H - i, v);
+    if (!ok) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] = 0.f;
+    }
+    st8n<VEC>(x32 + t * ldx + i, H - i, v);
+    st8n<VEC>(xa + t * lda + i, H - i, v);
+  }
+}
+
+// VPT groups of eight elements per thread stay in registers.
+template <typename T, bool VEC, int VPT>
+__global__ void __launch_bounds__(1024)
+postnorm_add_kernel(const T* __restrict__ y, long long ldy, float* __restrict__ x32, long long ldx,
+                    const T* __restrict__ w, T* __restrict__ xa, long long lda, const T* __restrict__ w_final, int rows,
+                    int H, float eps) {
+  __shared__ float scratch[32];
+  for (int t = blockIdx.x; t < rows; t += gridDim.x) {
+    float v[VPT][8];
+    float ss[1] = {0.f};
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      ld8n<VEC>(y + t * ldy + i, H - i, v[k]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss[0] += v[k][j] * v[k][j];
+    }
+    block_sum<1>(ss, scratch);
+    const float r = 1.f / sqrtf(ss[0] / static_cast<float>(H) + eps);
+    ss[0] = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      if (i >= H) continue;
+      float x[8], g[8];
+      ld8n<VEC>(x32 + t * ldx + i, H - i, x);
+      ld8n<VEC>(w + i, H - i, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        x[j] += v[k][j] * r * g[j];
+        v[k][j] = x[j];
+        ss[0] += x[j] * x[j];
+      }
+      st8n<VEC>(x32 + t * ldx + i, H - i, x);
+      if (w_final == nullptr) st8n<VEC>(xa + t * lda + i, H - i, x);
+    }
+    if (w_final != nullptr) {
+      block_sum<1>(ss, scratch);
+      const float rf = 1.f / sqrtf(ss[0] / static_cast<float>(H) + eps);
+#pragma unroll
+      for (int k = 0; k < VPT; ++k) {
+        const int i = (threadIdx.x + k * blockDim.x) * 8;
+        if (i >= H) continue;
+        float g[8], o[8];
+        ld8n<VEC>(w_final + i, H - i, g);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) o[j] = v[k][j] * rf * g[j];
+        st8n<VEC>(xa + t * lda + i, H - i, o);
+      }
+    }
+  }
+}
+
+template <typename T, bool VEC, int VPT>
+__global__ void __launch_bounds__(1024)
+polynorm_kernel(const T* __restrict__ z, long long ldz, const T* __restrict__ coef, T* __restrict__ out, long long ldo,
+                int rows, int F, float eps) {
+  __shared__ float scratch[96];
+  const float ca = ld1(coef), cb = ld1(coef + 1), cc = ld1(coef + 2), ce = ld1(coef + 3);
+  for (int t = blockIdx.x; t < rows; t += gridDim.x) {
+    float v[VPT][8];
+    float s[3] = {0.f, 0.f, 0.f};
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      ld8n<VEC>(z + t * ldz + i, F - i, v[k]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float q = v[k][j] * v[k][j];
+        s[0] += q;
+        s[1] += q * q;
+        s[2] += q * q * q;
+      }
+    }
+    block_sum<3>(s, scratch);
+    const float n = static_cast<float>(F);
+    const float ra = ca / sqrtf(s[0] / n + eps), rb = cb / sqrtf(s[1] / n + eps), rc = cc / sqrtf(s[2] / n + eps);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      if (i >= F) continue;
+      float o[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        const float a = v[k][j];
+        o[j] = ((rc * a + rb) * a + ra) * a + ce;
+      }
+      st8n<VEC>(out + t * ldo + i, F - i, o);
+    }
+  }
+}
+
+template <typename T, bool VEC, int VPT>
+__global__ void __launch_bounds__(1024)
+gated_group_norm_kernel(const T* __restrict__ y, long long ldy, const T* __restrict__ z, long long ldz,
+                        const T* __restrict__ w, T* __restrict__ out, long long ldo, int items, int groups, int part,
+                        float eps) {
+  __shared__ float scratch[32];
+  for (int it = blockIdx.x; it < items; it += gridDim.x) {
+    const int t = it / groups, c0 = (it - t * groups) * part;
+    float v[VPT][8];
+    float ss[1] = {0.f};
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      float g[8];
+      ld8n<VEC>(y + t * ldy + c0 + i, part - i, v[k]);
+      ld8n<VEC>(z + t * ldz + c0 + i, part - i, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        v[k][j] *= silu_f(g[j]);
+        ss[0] += v[k][j] * v[k][j];
+      }
+    }
+    block_sum<1>(ss, scratch);
+    const float r = 1.f / sqrtf(ss[0] / static_cast<float>(part) + eps);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      if (i >= part) continue;
+      float g[8];
+      ld8n<VEC>(w + c0 + i, part - i, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) g[j] = v[k][j] * r * g[j];
+      st8n<VEC>(out + t * ldo + c0 + i, part - i, g);
+    }
+  }
+}
+
+static int check_launch(const char* what) {
+  const cudaError_t e = cudaGetLastError();
+  if (e == cudaSuccess) return 0;
+  set_last_error("%s launch failed: %s", what, cudaGetErrorString(e));
+  return 1;
+}
+
+// Threads and register groups for a row of n elements.
+static bool row_shape(int n, int* threads, int* vpt, const char* what) {
+  const int nvec = (n + 7) / 8;
+  for (int v = 1; v <= 8; v *= 2) {
+    const int th = ((nvec + v - 1) / v + 31) / 32 * 32;
+    if (th <= 512 || (v == 8 && th <= 1024)) {
+      *threads = th;
+      *vpt = v;
+      return true;
+    }
+  }
+  set_last_error("%s: a row of %d elements is too long", what, n);
+  return false;
+}
+static int row_grid(int items, int threads) {
+  const int cap = device_sm_count() * (threads <= 128 ? 16 : threads <= 256 ? 8 : threads <= 512 ? 4 : 2);
+  return items < cap ? items : cap;
+}
+static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+}  // namespace tw
+
+using namespace tw;
+
+#define TW_ROW_VPT(KERNEL, T, VEC, ...)                                          \
+  switch (vpt) {                                                                 \
+    case 1: KERNEL<T, VEC, 1><<<grid, threads, 0, stream>>>(__VA_ARGS__); break; \
+    case 2: KERNEL<T, VEC, 2><<<grid, threads, 0, stream>>>(__VA_ARGS__); break; \
+    case 4: KERNEL<T, VEC, 4><<<grid, threads, 0, stream>>>(__VA_ARGS__); break; \
+    default: KERNEL<T, VEC, 8><<<grid, threads, 0, stream>>>(__VA_ARGS__); break; \
+  }
+
+extern "C" int tw_embed_residual(const int* ids, const void* table, long long ldt, float* x32, long long ldx, void* xa,
+                                 long long lda, int T, int H, int vocab, int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  const bool vec = ldt % 8 == 0 && ldx % 8 == 0 && lda % 8 == 0 && aligned16(table) && aligned16(x32) && aligned16(xa);
+  int threads = ((H + 7) / 8 + 31) / 32 * 32;
+  if (threads > 256) threads = 256;
+#define TW_GO(TT, V)                                                                                       \
+  embed_residual_kernel<TT, V><<<T, threads, 0, stream>>>(ids, reinterpret_cast<const TT*>(table), ldt, x32, ldx, \
+                                                          reinterpret_cast<TT*>(xa), lda, H, vocab)
+  if (dtype == TW_BF16) {
+    if (vec) TW_GO(__nv_bfloat16, true); else TW_GO(__nv_bfloat16, false);
+  } else {
+    if (vec) TW_GO(float, true); else TW_GO(float, false);
+  }
+#undef TW_GO
+  return check_launch("embed_residual");
+}
+
+extern "C" int tw_postnorm_add(const void* y, long long ldy, float* x32, long long ldx, const void* w, void* xa,
+                               long long lda, const void* w_final, int T, int H, float eps, int dtype,
+                               cudaStream_t stream) {
+  if (T <= 0) return 0;
+  int threads, vpt;
+  if (!row_shape(H, &threads, &vpt, "postnorm_add")) return 1;
+  const int grid = row_grid(T, threads);
+  const bool vec = ldy % 8 == 0 && ldx % 8 == 0 && lda % 8 == 0 && aligned16(y) && aligned16(x32) && aligned16(xa) &&
+                   aligned16(w) && aligned16(w_final);
+#define TW_GO(TT, V)                                                                                              \
+  TW_ROW_VPT(postnorm_add_kernel, TT, V, reinterpret_cast<const TT*>(y), ldy, x32, ldx,                           \
+             reinterpret_cast<const TT*>(w), reinterpret_cast<TT*>(xa), lda, reinterpret_cast<const TT*>(w_final), \
+             T, H, eps)
+  if (dtype == TW_BF16) {
+    if (vec) TW_GO(__nv_bfloat16, true) else TW_GO(__nv_bfloat16, false)
+  } else {
+    if (vec) TW_GO(float, true) else TW_GO(float, false)
+  }
+#undef TW_GO
+  return check_launch("postnorm_add");
+}
+
+extern "C" int tw_polynorm(const void* z, long long ldz, const void* coef, void* out, long long ldo, int T, int F,
+                           float eps, int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  int threads, vpt;
+  if (!row_shape(F, &threads, &vpt, "polynorm")) return 1;
+  const int grid = row_grid(T, threads);
+  const bool vec = ldz % 8 == 0 && ldo % 8 == 0 && aligned16(z) && aligned16(out);
+#define TW_GO(TT, V)                                                                                        \
+  TW_ROW_VPT(polynorm_kernel, TT, V, reinterpret_cast<const TT*>(z), ldz, reinterpret_cast<const TT*>(coef), \
+             reinterpret_cast<TT*>(out), ldo, T, F, eps)
+  if (dtype == TW_BF16) {
+    if (vec) TW_GO(__nv_bfloat16, true) else TW_GO(__nv_bfloat16, false)
+  } else {
+    if (vec) TW_GO(float, true) else TW_GO(float, false)
+  }
+#undef TW_GO
+  return check_launch("polynorm");
+}
+
+extern "C" int tw_gated_group_norm(const void* y, long long ldy, const void* z, long long ldz, const void* w, void* out,
+                                   long long ldo, int T, int C, int groups, float eps, int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (groups <= 0 || C % groups != 0) {
+    set_last_error("gated_group_norm: %d channels do not divide into %d groups", C, groups);
+    return 1;
+  }
+  const int part = C / groups;
+  int threads, vpt;
+  if (!row_shape(part, &threads, &vpt, "gated_group_norm")) return 1;
+  const int grid = row_grid(T * groups, threads);
+  const bool vec = ldy % 8 == 0 && ldz % 8 == 0 && ldo % 8 == 0 && (groups == 1 || part % 8 == 0) && aligned16(y) &&
+                   aligned16(z) && aligned16(w) && aligned16(out);
+#define TW_GO(TT, V)                                                                                                \
+  TW_ROW_VPT(gated_group_norm_kernel, TT, V, reinterpret_cast<const TT*>(y), ldy, reinterpret_cast<const TT*>(z), ldz, \
+             reinterpret_cast<const TT*>(w), reinterpret_cast<TT*>(out), ldo, T * groups, groups, part, eps)
+  if (dtype == TW_BF16) {
+    if (vec) TW_GO(__nv_bfloat16, true) else TW_GO(__nv_bfloat16, false)
+  } else {
+    if (vec) TW_GO(float, true) else TW_GO(float, false)
+  }
+#undef TW_GO
+  return check_launch("gated_group_norm");
+}

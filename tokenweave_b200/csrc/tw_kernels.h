@@ -141,6 +141,49 @@ int tw_oneshot_allreduce(void* const* peer_bases, uint32_t* const* signal_pads, 
                          long long n_bytes, void* out, int max_ctas, cudaStream_t stream);
 int tw_wait_probe(uint32_t* flag, unsigned long long budget_ns, uint32_t* status, cudaStream_t stream);
 
+// ---- fp32 matrix product (gemm_f32.cu) ----
+int tw_gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc,
+                const float* bias, int M, int N, int K, cudaStream_t stream);
+
+// In the launchers below dtype is 0 for bf16 and 1 for fp32 activations and weights.
+// ---- fp32 residual stream, norm of a sublayer's output, feed-forward activation (rownorm.cu) ----
+int tw_embed_residual(const int* ids, const void* table, long long ldt, float* x32, long long ldx, void* xa,
+                      long long lda, int T, int H, int vocab, int dtype, cudaStream_t stream);
+int tw_postnorm_add(const void* y, long long ldy, float* x32, long long ldx, const void* w, void* xa, long long lda,
+                    const void* w_final, int T, int H, float eps, int dtype, cudaStream_t stream);
+int tw_polynorm(const void* z, long long ldz, const void* coef, void* out, long long ldo, int T, int F, float eps,
+                int dtype, cudaStream_t stream);
+int tw_gated_group_norm(const void* y, long long ldy, const void* z, long long ldz, const void* w, void* out,
+                        long long ldo, int T, int C, int groups, float eps, int dtype, cudaStream_t stream);
+
+// ---- latent attention (latent_attn.cu) ----
+int tw_latent_prep(const void* p, long long ldp, int q_off, int q_rank, const void* wq, void* cq, long long ldcq,
+                   int kv_off, int kv_rank, const void* wkv, int rot, int rot_dims, const float* cos_sin,
+                   const int* positions, const int* slots, void* cache, int row, int T, float eps, int dtype,
+                   cudaStream_t stream);
+int tw_rope_tail(void* q, long long ldq, int T, int heads, int head_stride, int off, int rot_dims,
+                 const float* cos_sin, const int* positions, int dtype, cudaStream_t stream);
+int tw_latent_query(const void* q, long long ldq, const int* rows, int n, void* qa, int heads, int head_stride, int off,
+                    int rot, int rot_dims, int kv_rank, int row, const float* cos_sin, const int* positions, int dtype,
+                    cudaStream_t stream);
+int tw_head_gemm(const void* A, long long lda, int a_hs, const int* a_rows, const void* B, long long b_hs, int ldb,
+                 void* C, long long ldc, int c_hs, const int* c_rows, const void* gate, long long ldg, int g_hs,
+                 int heads, int M, int N, int K, int dtype, cudaStream_t stream);
+int tw_latent_attn(const void* qa, const void* cache, const int* tok_seq, const int* tok_kvlen, int n,
+                   const int* block_table, int max_blocks, int page, void* out, int heads, int row, int kv_rank,
+                   float scale, int dtype, cudaStream_t stream);
+int tw_latent_gather(const void* cache, void* dst, const int* seqs, const int* cu, int n_seqs, int max_rows,
+                     const int* block_table, int max_blocks, int page, int row_bytes, cudaStream_t stream);
+
+// ---- state-space recurrence (ssm.cu) ----
+int tw_causal_conv(const void* x, long long ldx, const void* w, const void* bias, void* state, void* out, long long ldo,
+                   const int* row_seq, const int* cu_q, const int* kv_lens, const int* slots, int T, int n_seqs,
+                   int channels, int taps, int single, int dtype, cudaStream_t stream);
+int tw_ssd_scan(const void* xbc, long long ldx, const void* dt, long long ldt, const void* dt_bias, const void* A_log,
+                const void* D, float* state, void* y, long long ldy, const int* seqs, int n_seqs, const int* cu_q,
+                const int* kv_lens, const int* slots, int heads, int vdim, int N, int groups, int dtype,
+                cudaStream_t stream);
+
 #ifdef __cplusplus
 }
 #endif

@@ -35,7 +35,8 @@ class EngineCore:
         num_blocks = self.executor.determine_num_blocks()
         self.executor.init_kv_cache(num_blocks)
         self.num_blocks = num_blocks
-        self.kv = KVCacheManager(num_blocks, config.cache.block_size, config.cache.enable_prefix_caching)
+        self.kv = KVCacheManager(num_blocks, config.cache.block_size, config.cache.enable_prefix_caching,
+                                 config.scheduler.max_num_seqs if config.model.has_state else 0)
         self.scheduler = Scheduler(config.scheduler, self.kv, config.speculative)
         self._sent_blocks: dict[str, int] = {}     # blocks of each request already known to the workers
         # KV connector: the scheduler side only asks which blocks the store can supply; the workers move the data
@@ -72,7 +73,8 @@ class EngineCore:
             r = s.request
             if s.is_new:
                 step.new_requests.append(NewRequestData(r.request_id, r.all_token_ids, r.num_prompt_tokens,
-                                                        r.sampling_params, list(r.block_ids), r.lora_request))
+                                                        r.sampling_params, list(r.block_ids), r.lora_request,
+                                                        r.state_slot))
                 new_blocks: list[int] = []
             else:
                 new_blocks = r.block_ids[self._sent_blocks.get(r.request_id, 0):]

@@ -90,11 +90,34 @@ def block_hashes(token_ids: list[int], block_size: int, salt: bytes = b"") -> li
     return out
 
 
+class StateSlotPool:
+    """Slots of recurrent state (convolution inputs, state matrices): one per live request, none shared. A slot is not
+    cleared when it changes hands: a sequence without tokens behind it starts from zeros whatever its slot holds."""
+
+    def __init__(self, num_slots: int):
+        self.num_slots = num_slots
+        self._free = list(range(num_slots - 1, -1, -1))
+
+    @property
+    def num_free(self) -> int:
+        return len(self._free)
+
+    def allocate(self) -> int:
+        return self._free.pop()
+
+    def release(self, slot: int) -> None:
+        assert slot not in self._free, "state slot released twice"
+        self._free.append(slot)
+
+
 class KVCacheManager:
-    def __init__(self, num_blocks: int, block_size: int, enable_caching: bool = False):
+    """Cache blocks and, for models with recurrent layers (``num_state_slots`` > 0), a state slot per request."""
+
+    def __init__(self, num_blocks: int, block_size: int, enable_caching: bool = False, num_state_slots: int = 0):
         self.block_size = block_size
         self.pool = BlockPool(num_blocks, enable_caching)
         self.enable_caching = enable_caching
+        self.states = StateSlotPool(num_state_slots) if num_state_slots > 0 else None
         self.prefix_queries = 0        # blocks looked up / found in the prefix cache since start
         self.prefix_hits = 0
         self.track_published = False   # a KV connector wants to know which blocks became full
@@ -128,6 +151,10 @@ class KVCacheManager:
         evictable_cached = sum(1 for b in cached_blocks if self.pool.ref[b] == 0)
         if need > self.pool.num_free - evictable_cached:
             return False
+        if self.states is not None and req.state_slot is None:
+            if self.states.num_free == 0:
+                return False
+            req.state_slot = self.states.allocate()
         for b in cached_blocks:
             self.pool.touch(b)
         req.block_ids.extend(cached_blocks)
@@ -169,6 +196,9 @@ class KVCacheManager:
     def free(self, req: Request) -> None:
         self.pool.release(req.block_ids)
         req.block_ids = []
+        if req.state_slot is not None:
+            self.states.release(req.state_slot)
+            req.state_slot = None
         req.num_published_blocks = 0       # the next owner of these block ids starts over; the hash chain stays
 
     def usage(self) -> float:

@@ -39,6 +39,7 @@ class Request:
     output_token_ids: list[int] = field(default_factory=list)
     num_computed_tokens: int = 0       # tokens whose KV is in the cache
     block_ids: list[int] = field(default_factory=list)
+    state_slot: Optional[int] = None   # slot of the recurrent state (models that keep one)
     spec_token_ids: list[int] = field(default_factory=list)   # drafts to verify in the next step
     lora_request: Optional[object] = None                     # tokenweave_b200.lora.LoRARequest
     prompt_logprobs: dict = field(default_factory=dict)       # prompt position -> {token id: log-probability}

@@ -19,8 +19,6 @@ from .. import ops
 from ..ops import reference
 
 PREFILL_MIN_Q = 16
-_I32_FIELDS = ("positions", "slot_mapping", "cu_q", "kv_lens", "tile_seq", "tile_q0", "tok_row", "tok_seq",
-               "tok_kvlen")
 
 
 @dataclass
@@ -43,6 +41,10 @@ class AttentionMetadata:
     max_kv_len: int
     cu_q_cpu: list = field(default_factory=list)
     kv_lens_cpu: list = field(default_factory=list)
+    all_single: bool = False         # every sequence has exactly one token in this step
+    # further int32 arrays of the step a model asks for (``plan_step`` of models/hybrid.py), and host values with them
+    extra: dict = field(default_factory=dict)
+    extra_cpu: dict = field(default_factory=dict)
 
 
 def plan_attention(q_lens: Sequence[int], kv_lens: Sequence[int]):
@@ -75,14 +77,16 @@ def plan_attention(q_lens: Sequence[int], kv_lens: Sequence[int]):
 def build_attention_metadata(q_lens: Sequence[int], kv_lens: Sequence[int], positions: np.ndarray,
                              slot_mapping: np.ndarray, block_table: np.ndarray, device: torch.device,
                              pinned: Optional[torch.Tensor] = None,
-                             device_buffer: Optional[torch.Tensor] = None) -> AttentionMetadata:
-    """Pack every int32 array into one staging buffer, copy it to the device once, slice views."""
+                             device_buffer: Optional[torch.Tensor] = None, plan: Optional[tuple] = None,
+                             extra: Optional[dict] = None, extra_cpu: Optional[dict] = None) -> AttentionMetadata:
+    """Pack every int32 array into one staging buffer, copy it to the device once, slice views. ``plan``: the routing
+    of the query rows (default: :func:`plan_attention`); ``extra``: further int32 arrays to carry along."""
     q_lens = [int(x) for x in q_lens]
     kv_lens = [int(x) for x in kv_lens]
     B = len(q_lens)
     cu = np.zeros(B + 1, dtype=np.int32)
     np.cumsum(q_lens, out=cu[1:])
-    tile_seq, tile_q0, tok_row, tok_seq, tok_kv = plan_attention(q_lens, kv_lens)
+    tile_seq, tile_q0, tok_row, tok_seq, tok_kv = plan if plan is not None else plan_attention(q_lens, kv_lens)
     arrays = {
         "positions": np.asarray(positions, dtype=np.int32), "slot_mapping": np.asarray(slot_mapping, dtype=np.int32),
         "cu_q": cu, "kv_lens": np.asarray(kv_lens, dtype=np.int32),
@@ -90,8 +94,10 @@ def build_attention_metadata(q_lens: Sequence[int], kv_lens: Sequence[int], posi
         "tok_row": np.asarray(tok_row, dtype=np.int32), "tok_seq": np.asarray(tok_seq, dtype=np.int32),
         "tok_kvlen": np.asarray(tok_kv, dtype=np.int32),
     }
+    extra = extra or {}
+    arrays.update({"extra." + k: np.asarray(v, dtype=np.int32) for k, v in extra.items()})
     bt = np.ascontiguousarray(block_table, dtype=np.int32).reshape(B, -1)
-    sizes = [(k, (arrays[k].size + 3) // 4 * 4) for k in _I32_FIELDS] + [("block_table", (bt.size + 3) // 4 * 4)]
+    sizes = [(k, (v.size + 3) // 4 * 4) for k, v in arrays.items()] + [("block_table", (bt.size + 3) // 4 * 4)]
     total = sum(s for _, s in sizes)
     if pinned is not None and pinned.numel() >= total:
         host = pinned[:total]
@@ -120,7 +126,9 @@ def build_attention_metadata(q_lens: Sequence[int], kv_lens: Sequence[int], posi
         cu_q=view["cu_q"], kv_lens=view["kv_lens"], block_table=view["block_table"].view(B, -1) if B else view["block_table"].view(0, 1),
         tile_seq=view["tile_seq"], tile_q0=view["tile_q0"], num_tiles=len(tile_seq), tok_row=view["tok_row"],
         tok_seq=view["tok_seq"], tok_kvlen=view["tok_kvlen"], num_single=len(tok_row),
-        max_kv_len=max(kv_lens) if kv_lens else 0, cu_q_cpu=cu.tolist(), kv_lens_cpu=kv_lens)
+        max_kv_len=max(kv_lens) if kv_lens else 0, cu_q_cpu=cu.tolist(), kv_lens_cpu=kv_lens,
+        all_single=bool(q_lens) and max(q_lens) == 1, extra={k: view["extra." + k] for k in extra},
+        extra_cpu=extra_cpu or {})
 
 
 class Attention(nn.Module):

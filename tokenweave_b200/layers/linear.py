@@ -186,3 +186,26 @@ class RowParallelLinear(_QuantizableLinear):
             param.data.copy_(loaded)
         else:
             param.data.copy_(loaded.narrow(1, r * self.in_per_rank, self.in_per_rank))
+
+
+def pad8(n: int) -> int:
+    return (n + 7) // 8 * 8
+
+
+class PaddedLinear(_QuantizableLinear):
+    """A replicated linear of any sizes: both dimensions are stored padded to eight elements (16-byte rows, what the
+    TMA-fed GEMM needs) with zeros, so ``x`` has ``in_padded`` columns whose pad is finite and the output's pad columns
+    come out as zeros. Several projections of one input can share it, each written with :meth:`load_rows`."""
+
+    def __init__(self, in_features: int, out_features: int, *, dtype, device):
+        super().__init__()
+        self.in_features, self.out_features = in_features, out_features
+        self.in_padded, self.out_padded = pad8(in_features), pad8(out_features)
+        self.weight = nn.Parameter(torch.zeros(self.out_padded, self.in_padded, dtype=dtype, device=device),
+                                   requires_grad=False)
+
+    def load_rows(self, t: torch.Tensor, row: int) -> None:
+        self.weight.data[row:row + t.shape[0], :t.shape[1]].copy_(t)
+
+    def forward(self, x: torch.Tensor, out: Optional[torch.Tensor] = None, max_ctas: int = 0) -> torch.Tensor:
+        return self._gemm(x, out, max_ctas=max_ctas)

@@ -226,6 +226,24 @@ class DecoderModel(nn.Module):
             v = torch.zeros_like(k)
             a.bind_kv_cache(k, v)
 
+    def cache_tensors(self) -> list[torch.Tensor]:
+        """Every tensor kept between steps."""
+        return [t for l in self.layers if l.attn.k_cache is not None for t in (l.attn.k_cache, l.attn.v_cache)]
+
+    def drop_caches(self) -> None:
+        for layer in self.layers:
+            layer.attn.bind_kv_cache(None, None)
+
+    def state_bytes_per_slot(self) -> int:
+        return 0
+
+    def launch_key(self, meta: AttentionMetadata, block_size: int):
+        """What shapes a step's launches besides its token and sequence counts (part of a graph's signature)."""
+        a = self.layers[0].attn
+        return ops.decode_plan(meta.num_single, a.hq, a.hkv, a.head_dim, block_size,
+                               min(meta.max_kv_len, a.window) if a.window > 0 else meta.max_kv_len, self.rt.sm_count,
+                               a.window <= 0 and a.softcap <= 0)
+
     # ---- forward -------------------------------------------------------------------------
     @torch.inference_mode()
     def forward(self, step: StepInput) -> torch.Tensor:

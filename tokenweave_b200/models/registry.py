@@ -13,11 +13,18 @@ def get_model_class(architecture: str):
     from .phi3 import Phi3ForCausalLM
     from .qwen2 import Qwen2ForCausalLM
     from .qwen3 import Qwen3ForCausalLM
+    from .sidisun import SidisunForCausalLM
     table = {"llama": LlamaForCausalLM, "qwen2": Qwen2ForCausalLM, "mixtral": MixtralForCausalLM,
-             "qwen3": Qwen3ForCausalLM, "mistral": MistralForCausalLM, "phi3": Phi3ForCausalLM}
+             "qwen3": Qwen3ForCausalLM, "mistral": MistralForCausalLM, "phi3": Phi3ForCausalLM,
+             "sidisun": SidisunForCausalLM}
     if architecture not in table:
         raise ValueError(f"unsupported architecture {architecture!r} (supported: {sorted(table)})")
     return table[architecture]
+
+
+def load_config_readers() -> None:
+    """Imports the modules that register a reader for their own ``config.json`` layout."""
+    from . import sidisun  # noqa: F401
 
 
 def build_model(config: EngineConfig, device: torch.device, embedding_parallel: bool = False):

@@ -101,6 +101,14 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
         res = reference.gemm_swiglu(a, w, row_scale) if swiglu else reference.gemm(a, w, bias, row_scale)
         out.copy_(res)
         return out
+    if a.dtype == torch.float32:
+        if swiglu or row_scale is not None or tile_expert is not None:
+            raise NotImplementedError("the fp32 matrix product is plain: no SwiGLU, row scales or groups")
+        if w.dtype != torch.float32 or out.dtype != torch.float32:
+            raise TypeError("the fp32 matrix product takes fp32 operands")
+        _native.call("tw_gemm_f32", a.data_ptr(), _row_stride(a), w.data_ptr(), _row_stride(w), out.data_ptr(),
+                     _row_stride(out), _p(bias), M, N, K, _stream())
+        return out
     _check_bf16(a, w, out, bias)
     if tile_expert is not None and tile_rows == 256:
         if bias is not None:

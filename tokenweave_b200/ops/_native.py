@@ -62,6 +62,19 @@ _SIGNATURES = {
                         i32, i32, vp],
     "tw_ag_gemm": [vp, vp, ll, ll, vp, ll, vp, i32, i32, i32, i32, i32, vp, vp, vp, vp, i32, i32, u64, vp, ll, i32, i32,
                    i32, vp],
+    "tw_gemm_f32": [vp, ll, vp, ll, vp, ll, vp, i32, i32, i32, vp],
+    "tw_embed_residual": [vp, vp, ll, vp, ll, vp, ll, i32, i32, i32, i32, vp],
+    "tw_postnorm_add": [vp, ll, vp, ll, vp, vp, ll, vp, i32, i32, f32, i32, vp],
+    "tw_polynorm": [vp, ll, vp, vp, ll, i32, i32, f32, i32, vp],
+    "tw_gated_group_norm": [vp, ll, vp, ll, vp, vp, ll, i32, i32, i32, f32, i32, vp],
+    "tw_latent_prep": [vp, ll, i32, i32, vp, vp, ll, i32, i32, vp, i32, i32, vp, vp, vp, vp, i32, i32, f32, i32, vp],
+    "tw_rope_tail": [vp, ll, i32, i32, i32, i32, i32, vp, vp, i32, vp],
+    "tw_latent_query": [vp, ll, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, vp],
+    "tw_head_gemm": [vp, ll, i32, vp, vp, ll, i32, vp, ll, i32, vp, vp, ll, i32, i32, i32, i32, i32, i32, vp],
+    "tw_latent_attn": [vp, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, f32, i32, vp],
+    "tw_latent_gather": [vp, vp, vp, vp, i32, i32, vp, i32, i32, i32, vp],
+    "tw_causal_conv": [vp, ll, vp, vp, vp, vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
+    "tw_ssd_scan": [vp, ll, vp, ll, vp, vp, vp, vp, vp, ll, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, vp],
 }
 
 

@@ -1,0 +1,185 @@
+"""Operators of models whose layers mix attention and recurrences and whose residual stream is fp32: latent attention
+over a paged latent cache, the state-space (Mamba-2) recurrence with its convolution, the norm of a sublayer's output
+added to the residual, and the polynomial-norm activation.
+
+Like the other operators, CUDA tensors (bf16 or fp32) go to the kernels of ``_C.so`` and CPU tensors to plain PyTorch
+(:mod:`.reference_hybrid`). ``meta`` below is the step's :class:`~tokenweave_b200.layers.attention.AttentionMetadata`.
+"""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+from . import _native, reference_hybrid as ref
+from . import _p, _row_stride, _stream
+
+
+def _dt(*ts: Optional[torch.Tensor]) -> int:
+    """The launchers' dtype code; every tensor must be stored in the same type."""
+    kinds = {t.dtype for t in ts if t is not None}
+    if len(kinds) != 1 or next(iter(kinds)) not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"expected tensors of one type, bfloat16 or float32, got {sorted(map(str, kinds))}")
+    return 0 if next(iter(kinds)) == torch.bfloat16 else 1
+
+
+# ---- residual stream and row-wise kernels ------------------------------------------------------------------
+def embed_residual(ids: torch.Tensor, table: torch.Tensor, x32: torch.Tensor, xa: torch.Tensor, width: int) -> None:
+    """``x32 = table[ids]`` (fp32 residual stream) and ``xa`` the same rows in the activation type."""
+    if not table.is_cuda:
+        ref.embed_residual(ids, table, x32, xa, width)
+        return
+    assert ids.dtype == torch.int32 and x32.dtype == torch.float32
+    _native.call("tw_embed_residual", ids.data_ptr(), table.data_ptr(), _row_stride(table), x32.data_ptr(),
+                 _row_stride(x32), xa.data_ptr(), _row_stride(xa), ids.shape[0], width, table.shape[0], _dt(table, xa),
+                 _stream())
+
+
+def postnorm_add_(y: torch.Tensor, x32: torch.Tensor, weight: torch.Tensor, eps: float, xa: torch.Tensor,
+                  final_weight: Optional[torch.Tensor] = None) -> None:
+    """``x32 += rmsnorm(y) * weight`` and ``xa = x32`` (in the activation type); behind the last layer, with
+    ``final_weight``, ``xa = rmsnorm(x32) * final_weight``. The row width is the weight's length."""
+    if not y.is_cuda:
+        ref.postnorm_add_(y, x32, weight, eps, xa, final_weight)
+        return
+    assert x32.dtype == torch.float32
+    _native.call("tw_postnorm_add", y.data_ptr(), _row_stride(y), x32.data_ptr(), _row_stride(x32), weight.data_ptr(),
+                 xa.data_ptr(), _row_stride(xa), _p(final_weight), y.shape[0], weight.numel(), float(eps),
+                 _dt(y, weight, xa, final_weight), _stream())
+
+
+def polynorm(z: torch.Tensor, coef: torch.Tensor, eps: float, out: torch.Tensor, width: int) -> torch.Tensor:
+    """``a N(z) + b N(z^2) + c N(z^3) + e`` with ``coef = (a, b, c, e)`` and N dividing a row by its root mean square."""
+    if not z.is_cuda:
+        out[:, :width] = ref.polynorm(z[:, :width], coef, eps)
+        return out
+    _native.call("tw_polynorm", z.data_ptr(), _row_stride(z), coef.data_ptr(), out.data_ptr(), _row_stride(out),
+                 z.shape[0], width, float(eps), _dt(z, coef, out), _stream())
+    return out
+
+
+def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float,
+                     out: torch.Tensor) -> torch.Tensor:
+    """RMS norm of ``y * silu(z)`` in ``groups`` equal parts of the row, times ``weight`` (the gate comes first)."""
+    c = weight.numel()
+    if not y.is_cuda:
+        out[:, :c] = ref.gated_group_norm(y[:, :c], z[:, :c], weight, groups, eps)
+        return out
+    _native.call("tw_gated_group_norm", y.data_ptr(), _row_stride(y), z.data_ptr(), _row_stride(z), weight.data_ptr(),
+                 out.data_ptr(), _row_stride(out), y.shape[0], c, groups, float(eps), _dt(y, z, weight, out), _stream())
+    return out
+
+
+# ---- latent attention -----------------------------------------------------------------------------------------
+def latent_row(kv_rank: int, rot: int) -> int:
+    """Elements of a latent cache row: the latent and the rotated key part, each padded to eight."""
+    return (kv_rank + 7) // 8 * 8 + (rot + 7) // 8 * 8
+
+
+def latent_prep(p: torch.Tensor, q_off: int, q_rank: int, wq: torch.Tensor, cq: torch.Tensor, kv_off: int, kv_rank: int,
+                wkv: torch.Tensor, rot: int, rot_dims: int, cos_sin: torch.Tensor, positions: torch.Tensor,
+                slots: torch.Tensor, cache: torch.Tensor, eps: float) -> None:
+    """Norms of the two latents in the packed projection rows ``p``, rotation of the shared key part, cache write.
+    ``cache``: [blocks, page, row]."""
+    if not p.is_cuda:
+        ref.latent_prep(p, q_off, q_rank, wq, cq, kv_off, kv_rank, wkv, rot, rot_dims, cos_sin, positions, slots, cache,
+                        eps)
+        return
+    _native.call("tw_latent_prep", p.data_ptr(), _row_stride(p), q_off, q_rank, wq.data_ptr(), cq.data_ptr(),
+                 _row_stride(cq), kv_off, kv_rank, wkv.data_ptr(), rot, rot_dims, cos_sin.data_ptr(),
+                 positions.data_ptr(), slots.data_ptr(), cache.data_ptr(), cache.shape[-1], p.shape[0], float(eps),
+                 _dt(p, wq, cq, wkv, cache), _stream())
+
+
+def rope_tail_(q: torch.Tensor, heads: int, head_stride: int, off: int, rot_dims: int, cos_sin: torch.Tensor,
+               positions: torch.Tensor) -> None:
+    """Rotates elements ``[off, off + rot_dims)`` of every head of every row in place (CUDA; the un-absorbed form)."""
+    _native.call("tw_rope_tail", q.data_ptr(), _row_stride(q), q.shape[0], heads, head_stride, off, rot_dims,
+                 cos_sin.data_ptr(), positions.data_ptr(), _dt(q), _stream())
+
+
+def latent_absorb(q: torch.Tensor, rows: torch.Tensor, w_ukt: torch.Tensor, heads: int, dim: int, rot: int,
+                  rot_dims: int, kv_rank: int, cos_sin: torch.Tensor, positions: torch.Tensor, qa: torch.Tensor) -> None:
+    """Absorbed queries ``qa`` [n, heads, row] of the listed rows of ``q`` ([T, heads * (dim + rot)]): the key map
+    ``w_ukt`` [heads, kv_rank, >= dim] applied to the unrotated part, the rotated part, zero pads."""
+    n = rows.shape[0]
+    if not q.is_cuda:
+        qa[:n] = ref.latent_absorb(q, rows, w_ukt, heads, dim, rot, rot_dims, kv_rank, cos_sin, positions, qa.shape[-1])
+        return
+    dt = _dt(q, w_ukt, qa)
+    row = qa.shape[-1]
+    _native.call("tw_head_gemm", q.data_ptr(), _row_stride(q), dim + rot, rows.data_ptr(), w_ukt.data_ptr(),
+                 w_ukt.stride(0), w_ukt.stride(1), qa.data_ptr(), heads * row, row, None, None, 0, 0, heads, n, kv_rank,
+                 dim, dt, _stream())
+    _native.call("tw_latent_query", q.data_ptr(), _row_stride(q), rows.data_ptr(), n, qa.data_ptr(), heads, dim + rot,
+                 dim, rot, rot_dims, kv_rank, row, cos_sin.data_ptr(), positions.data_ptr(), dt, _stream())
+
+
+def latent_attention(qa: torch.Tensor, cache: torch.Tensor, tok_seq: torch.Tensor, tok_kvlen: torch.Tensor, n: int,
+                     block_table: torch.Tensor, kv_rank: int, scale: float, out: torch.Tensor) -> None:
+    """Causal attention of ``n`` absorbed query rows over the paged latent cache; ``out`` [n, heads, kv_rank]."""
+    if n == 0:
+        return
+    heads, row, page = qa.shape[1], qa.shape[2], cache.shape[1]
+    if not qa.is_cuda:
+        out[:n] = ref.latent_attention(qa[:n], cache, tok_seq, tok_kvlen, block_table, kv_rank, scale)
+        return
+    _native.call("tw_latent_attn", qa.data_ptr(), cache.data_ptr(), tok_seq.data_ptr(), tok_kvlen.data_ptr(), n,
+                 block_table.data_ptr(), block_table.shape[1], page, out.data_ptr(), heads, row, kv_rank, float(scale),
+                 _dt(qa, cache, out), _stream())
+
+
+def latent_values(o: torch.Tensor, rows: torch.Tensor, w_uv: torch.Tensor, heads: int, vdim: int, kv_rank: int,
+                  gate: Optional[torch.Tensor], out: torch.Tensor) -> None:
+    """``out[rows, h * vdim : ] = (w_uv[h] o[:, h]) * sigmoid(gate)``: head values of the weighted latents. ``w_uv``:
+    [heads, vdim, >= kv_rank]; ``gate`` (or None) and ``out`` are rows of all tokens of the step."""
+    n = rows.shape[0]
+    if not o.is_cuda:
+        ref.latent_values(o[:n], rows, w_uv, heads, vdim, kv_rank, gate, out)
+        return
+    _native.call("tw_head_gemm", o.data_ptr(), heads * kv_rank, kv_rank, None, w_uv.data_ptr(), w_uv.stride(0),
+                 w_uv.stride(1), out.data_ptr(), _row_stride(out), vdim, rows.data_ptr(), _p(gate),
+                 _row_stride(gate) if gate is not None else 0, vdim, heads, n, vdim, kv_rank, _dt(o, w_uv, out, gate),
+                 _stream())
+
+
+def latent_gather(cache: torch.Tensor, seqs: torch.Tensor, cu: torch.Tensor, max_rows: int, block_table: torch.Tensor,
+                  out: torch.Tensor) -> None:
+    """The first ``cu[i + 1] - cu[i]`` cache rows of sequence ``seqs[i]``, in order, into ``out[cu[i]:]`` (CUDA)."""
+    _native.call("tw_latent_gather", cache.data_ptr(), out.data_ptr(), seqs.data_ptr(), cu.data_ptr(), seqs.shape[0],
+                 max_rows, block_table.data_ptr(), block_table.shape[1], cache.shape[1],
+                 cache.shape[2] * cache.element_size(), _stream())
+
+
+# ---- state-space recurrence -------------------------------------------------------------------------------------
+def causal_conv(x: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+                row_seq: torch.Tensor, cu_q: torch.Tensor, kv_lens: torch.Tensor, slots: torch.Tensor,
+                single: bool) -> None:
+    """Per-channel causal convolution + bias + silu of the step's rows; ``weight`` [taps, channels] (last tap = current
+    token), ``state`` [slots, taps - 1, channels] is read for the inputs before a sequence's rows and moved on.
+    ``single``: every sequence has exactly one row."""
+    taps, channels = weight.shape
+    if not x.is_cuda:
+        ref.causal_conv(x, weight, bias, state, out, cu_q, kv_lens, slots)
+        return
+    _native.call("tw_causal_conv", x.data_ptr(), _row_stride(x), weight.data_ptr(), bias.data_ptr(), state.data_ptr(),
+                 out.data_ptr(), _row_stride(out), row_seq.data_ptr(), cu_q.data_ptr(), kv_lens.data_ptr(),
+                 slots.data_ptr(), x.shape[0], cu_q.shape[0] - 1, channels, taps, int(single),
+                 _dt(x, weight, bias, state, out), _stream())
+
+
+def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor,
+             state: torch.Tensor, y: torch.Tensor, seqs: torch.Tensor, cu_q: torch.Tensor, kv_lens: torch.Tensor,
+             slots: torch.Tensor, groups: int) -> None:
+    """Token-by-token state-space recurrence of the listed sequences. ``state``: fp32 [slots, heads, vdim, state]."""
+    if seqs.shape[0] == 0:
+        return
+    _, heads, vdim, N = state.shape
+    if not xbc.is_cuda:
+        ref.ssd_scan(xbc, dt, dt_bias, A_log, D, state, y, seqs, cu_q, kv_lens, slots, groups)
+        return
+    assert state.dtype == torch.float32
+    _native.call("tw_ssd_scan", xbc.data_ptr(), _row_stride(xbc), dt.data_ptr(), _row_stride(dt), dt_bias.data_ptr(),
+                 A_log.data_ptr(), D.data_ptr(), state.data_ptr(), y.data_ptr(), _row_stride(y), seqs.data_ptr(),
+                 seqs.shape[0], cu_q.data_ptr(), kv_lens.data_ptr(), slots.data_ptr(), heads, vdim, N, groups,
+                 _dt(xbc, dt, dt_bias, A_log, D, y), _stream())

@@ -223,9 +223,7 @@ def build_cos_sin_cache(head_dim: int, max_pos: int, theta: float,
             hi = min(math.ceil(corr_dim(beta_slow)), head_dim - 1)
             if rope_scaling.get("truncate", True) is False:
                 lo, hi = max(corr_dim(beta_fast), 0), min(corr_dim(beta_slow), head_dim - 1)
-            if lo == hi:
-                hi += 0.001
-            ramp = ((torch.arange(half, dtype=torch.float64) - lo) / (hi - lo)).clamp(0, 1)
+            ramp = ((torch.arange(half, dtype=torch.float64) - lo) / max(hi - lo, 0.001)).clamp(0, 1)
             extrap = 1.0 - ramp                                   # 1 where the frequency is kept as is
             inv_freq = inv_freq / factor * (1 - extrap) + inv_freq * extrap
             att = rope_scaling.get("attention_factor")

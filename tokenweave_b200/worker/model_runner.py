@@ -38,6 +38,7 @@ class NewRequestData:
     sampling_params: SamplingParams
     block_ids: list[int]
     lora_request: Optional[object] = None        # tokenweave_b200.lora.LoRARequest
+    state_slot: Optional[int] = None             # slot of the recurrent state (models that keep one)
 
 
 @dataclass
@@ -50,6 +51,10 @@ class StepData:
     finished_req_ids: list[str] = field(default_factory=list)
     preempted_req_ids: list[str] = field(default_factory=list)
     total_num_tokens: int = 0
+    # replayed steps (engine/replay.py): the tokens a request brings to this step, and the places among them whose
+    # logits come back in ``StepResult.logits``; nothing is sampled
+    given_tokens: Optional[dict] = None
+    want_logits: Optional[dict] = None
 
 
 @dataclass
@@ -60,6 +65,7 @@ class StepResult:
     device_time_ms: Optional[float] = None
     # request id -> [(prompt position, {token id: log-probability})] for the prompt positions of this step
     prompt_logprobs: Optional[dict] = None
+    logits: Optional[torch.Tensor] = None     # replayed steps: fp32 rows on the host, in order of entries and places
     pooled: Optional[dict] = None        # request id -> final-norm hidden state (host fp32) of pooling requests
 
 
@@ -71,6 +77,7 @@ class _CachedRequest:
     block_ids: list[int]
     generator: Optional[torch.Generator] = None
     lora_id: int = 0
+    state_slot: Optional[int] = None
     # fixed for the life of a request (its sampling parameters do not change once it is with the workers); read
     # for every request on every step, so not recomputed from the dozen fields behind them each time
     needs_penalties: bool = False
@@ -103,6 +110,7 @@ class ModelRunner:
         self.device = device
         self.tp = get_tp()
         self.model: Optional[DecoderModel] = None
+        self.plan_step = None                # set from the model: routing of a step's rows, extra metadata
         self.requests: dict[str, _CachedRequest] = {}
         self.sampler = Sampler(seed=config.seed)
         self.sampler.vocab_provider = self._token_bytes       # structured output: built on first use
@@ -155,6 +163,7 @@ class ModelRunner:
         t0 = time.monotonic()
         with (weights_pool if weights_pool is not None else contextlib.nullcontext()):
             self.model = build_model(self.config, self.device, embedding_parallel)
+        self.plan_step = getattr(self.model, "plan_step", None)     # models that route a step's rows themselves
         self.model.setup_runtime(self.max_tokens, self.config.tokenweave,
                                  disable_custom_all_reduce=self.config.parallel.disable_custom_all_reduce)
         if self.config.enable_lora:
@@ -167,6 +176,8 @@ class ModelRunner:
 
     def init_kv_cache(self, num_blocks: int) -> None:
         self.model.init_kv_cache(num_blocks, self.block_size)
+        if self.config.model.has_state:
+            self.model.init_state(self.config.scheduler.max_num_seqs)
 
     def release_graphs(self) -> None:
         """Drop every captured CUDA graph and the pool they allocate from."""
@@ -190,6 +201,10 @@ class ModelRunner:
             self.requests.pop(rid, None)
         for rid in step.preempted_req_ids:
             self.requests.pop(rid, None)
+        if step.given_tokens:
+            for rid, toks in step.given_tokens.items():
+                if rid in self.requests:
+                    self.requests[rid].token_ids.extend(toks)
         for nr in step.new_requests:
             gen = None
             sp = nr.sampling_params
@@ -203,10 +218,10 @@ class ModelRunner:
                 self.lora.ensure_loaded(nr.lora_request)
                 lora_id = nr.lora_request.lora_int_id
             self.requests[nr.req_id] = _CachedRequest(list(nr.token_ids), nr.num_prompt_tokens, sp, list(nr.block_ids), gen,
-                                                      lora_id)
+                                                      lora_id, nr.state_slot)
 
     def _build_metadata(self, entries, tokens_base: int, positions: np.ndarray, slots: np.ndarray,
-                        tables: dict[int, list[int]], which: int) -> AttentionMetadata:
+                        tables: dict[int, list[int]], which: int, state_slots: list) -> AttentionMetadata:
         """entries: list of (seq_index, q_len, kv_len) laid out back to back starting at row tokens_base."""
         q_lens = [e[1] for e in entries]
         kv_lens = [e[2] for e in entries]
@@ -218,9 +233,12 @@ class ModelRunner:
         for i, e in enumerate(entries):
             t = tables[e[0]]
             bt[i, : len(t)] = t
+        plan = extra = extra_cpu = None
+        if self.plan_step is not None:
+            plan, extra, extra_cpu = self.plan_step(q_lens, kv_lens, [state_slots[e[0]] for e in entries])
         return build_attention_metadata(q_lens, kv_lens, positions[tokens_base:tokens_base + n],
                                         slots[tokens_base:tokens_base + n], bt, self.device, self._meta_host[which],
-                                        self._meta_dev[which])
+                                        self._meta_dev[which], plan=plan, extra=extra, extra_cpu=extra_cpu)
 
     def _signature(self, step_in: StepInput, n_logits: int, greedy: bool):
         parts = [step_in.plan, n_logits, greedy]
@@ -228,11 +246,8 @@ class ModelRunner:
             if m is None:
                 parts.append(None)
                 continue
-            a = self.model.layers[0].attn
-            splits = ops.decode_plan(m.num_single, a.hq, a.hkv, a.head_dim, self.block_size,
-                                     min(m.max_kv_len, a.window) if a.window > 0 else m.max_kv_len,
-                                     self.model.rt.sm_count, a.window <= 0 and a.softcap <= 0)
-            parts.append((m.num_actual_tokens, m.num_seqs, m.num_tiles, m.num_single, m.block_table.shape[1], splits))
+            parts.append((m.num_actual_tokens, m.num_seqs, m.num_tiles, m.num_single, m.block_table.shape[1],
+                          self.model.launch_key(m, self.block_size)))
         return tuple(parts)
 
     def _forward_and_logits(self, step_in: StepInput, n_logits: int, greedy: bool):
@@ -284,7 +299,8 @@ class ModelRunner:
         ids = self._ids_host.numpy()
         positions = np.empty(T, dtype=np.int32)
         slots = np.empty(T, dtype=np.int32)
-        q_lens, kv_lens, tables = [], [], {}
+        q_lens, kv_lens, tables, state_slots = [], [], {}, []
+        want = step.want_logits
         logits_rows, sample_reqs = [], []
         row = 0
         bs = self.block_size
@@ -294,6 +310,7 @@ class ModelRunner:
         for b, (rid, computed, n_new, new_blocks, *rest) in enumerate(step.scheduled):
             req = self.requests[rid]
             req.block_ids.extend(new_blocks)
+            state_slots.append(req.state_slot)
             drafts = list(rest[0]) if rest and rest[0] else []
             if n_new == 1 and not drafts and req.sampling_params.prompt_logprobs is None:
                 # decode fast path (most rows of a serving step): scalars only, no array temporaries
@@ -303,7 +320,9 @@ class ModelRunner:
                 q_lens.append(1)
                 kv_lens.append(computed + 1)
                 tables[b] = req.block_array()
-                if computed + 1 >= len(req.token_ids):
+                if want is not None:
+                    logits_rows.extend(row + w for w in want.get(rid, ()))
+                elif computed + 1 >= len(req.token_ids):
                     logits_rows.append(row)
                     sample_reqs.append(rid)
                 if self.lora is not None:
@@ -322,7 +341,9 @@ class ModelRunner:
             q_lens.append(n_new)
             kv_lens.append(computed + n_new)
             tables[b] = blocks
-            if computed + n_base >= len(req.token_ids):
+            if want is not None:
+                logits_rows.extend(row + w for w in want.get(rid, ()))
+            elif computed + n_base >= len(req.token_ids):
                 # one logits row at the request's last own token, and one after every draft
                 for k in range(len(drafts) + 1):
                     logits_rows.append(row + n_base - 1 + k)
@@ -347,12 +368,12 @@ class ModelRunner:
         h2d = T * 4
         if plan.overlap:
             first, second = split_batch(q_lens, kv_lens, plan.split)
-            meta0 = self._build_metadata(first, 0, positions, slots, tables, 0)
-            meta1 = self._build_metadata(second, plan.split, positions, slots, tables, 1)
+            meta0 = self._build_metadata(first, 0, positions, slots, tables, 0, state_slots)
+            meta1 = self._build_metadata(second, plan.split, positions, slots, tables, 1, state_slots)
             step_in = StepInput(ids_dev, plan, meta0=meta0, meta1=meta1)
         else:
             entries = [(b, q_lens[b], kv_lens[b]) for b in range(len(q_lens))]
-            step_in = StepInput(ids_dev, plan, meta=self._build_metadata(entries, 0, positions, slots, tables, 0))
+            step_in = StepInput(ids_dev, plan, meta=self._build_metadata(entries, 0, positions, slots, tables, 0, state_slots))
         for m in (step_in.meta, step_in.meta0, step_in.meta1):
             if m is not None:
                 h2d += 4 * (2 * m.num_actual_tokens + 2 * m.num_seqs + 1 + m.block_table.numel() + 2 * m.num_tiles + 3 * m.num_single)
@@ -377,6 +398,8 @@ class ModelRunner:
                     self.requests[rid].token_ids.extend(list(tok) if isinstance(tok, (list, tuple)) else [int(tok)])
             return result
         n_logits = len(logits_rows)
+        if want is not None:
+            return self._replayed(step, step_in, logits_rows, h2d)
         reqs = [self.requests[r] for r in sample_reqs]
         greedy = bool(reqs) and all(r.plain_greedy for r in reqs)
         if n_logits:
@@ -462,6 +485,23 @@ class ModelRunner:
         if self.tp.pp_size > 1:
             result = broadcast_from_last_stage(result)       # every stage's scheduler sees the same result
         return result
+
+    def _replayed(self, step: StepData, step_in: StepInput, rows: list[int], h2d: int) -> StepResult:
+        """A step with given tokens: the forward pass of every other step, logits at the wanted rows, no sampling."""
+        hidden = self.model(step_in)
+        logits = None
+        if rows:
+            idx = torch.as_tensor(rows, dtype=torch.long, device=hidden.device)
+            # blocks of rows bound the size of the device logits (a whole prompt may be asked for)
+            parts = [self.model.compute_logits(hidden.index_select(0, idx[i:i + 512])).float().cpu()
+                     for i in range(0, len(rows), 512)]
+            logits = torch.cat(parts)
+        if self._status_src is not None:
+            self._status_host.copy_(self._status_src())
+            self._raise_on_device_status()
+        self.h2d_bytes_last_step, self.d2h_bytes_last_step = h2d, 0 if logits is None else logits.numel() * 4
+        req_ids = [s[0] for s in step.scheduled]
+        return StepResult(req_ids, [None] * len(req_ids), logits=logits)
 
     def _raise_on_device_status(self) -> None:
         """Called right after the step's device -> host synchronisation: a kernel that gave up on a bounded

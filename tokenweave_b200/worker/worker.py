@@ -73,6 +73,7 @@ class Worker:
         free, total = torch.cuda.mem_get_info(self.device)
         used_by_others = total - free - torch.cuda.memory_reserved(self.device)
         budget = total * cache.gpu_memory_utilization - torch.cuda.memory_reserved(self.device) - max(0, used_by_others)
+        budget -= self.runner.model.state_bytes_per_slot() * self.config.scheduler.max_num_seqs
         budget -= 2 << 30     # logits, sampler temporaries, NCCL buffers
         n = int(budget // per_block)
         if n < 4:
@@ -85,6 +86,7 @@ class Worker:
         from ..utils.sleep_allocator import TAG_KV_CACHE
         with self._sleep_pool(TAG_KV_CACHE):
             self.runner.init_kv_cache(num_blocks)
+        self._num_blocks = num_blocks
         logger.info("KV cache: %d blocks of %d tokens", num_blocks, self.config.cache.block_size)
 
     def execute_model(self, step: StepData) -> StepResult:
@@ -142,11 +144,8 @@ class Worker:
                 host.copy_(p.data)
                 self._sleeping[name] = host
             p.data = torch.empty(0, dtype=p.dtype, device=self.device)
-        self._kv_shape = None
-        for layer in model.layers:
-            if layer.attn.k_cache is not None:
-                self._kv_shape = tuple(layer.attn.k_cache.shape)
-            layer.attn.bind_kv_cache(None, None)
+        self._had_caches = bool(model.cache_tensors())
+        model.drop_caches()
         if self.device.type == "cuda":
             torch.cuda.synchronize()
             torch.cuda.empty_cache()
@@ -162,10 +161,8 @@ class Worker:
                 if self.config.quantization:
                     raise RuntimeError("sleep level 2 with online quantisation needs a fresh engine")
                 load_model_weights(model, self.config)
-            for layer in model.layers:      # the KV cache came back uninitialised
-                if layer.attn.k_cache is not None:
-                    layer.attn.k_cache.zero_()
-                    layer.attn.v_cache.zero_()
+            for t in model.cache_tensors():      # the caches came back uninitialised
+                t.zero_()
             torch.cuda.synchronize()
             self._vmm_sleep_level = None
             return
@@ -181,8 +178,8 @@ class Worker:
             for name, p in model.named_parameters():
                 p.data = torch.empty(self._param_shapes[name], dtype=p.dtype, device=self.device)
             load_model_weights(model, self.config)
-        if self._kv_shape is not None:
-            self.runner.init_kv_cache(self._kv_shape[0])
+        if self._had_caches:
+            self.runner.init_kv_cache(self._num_blocks)
         self._sleeping = None
         if self.device.type == "cuda":
             torch.cuda.synchronize()
