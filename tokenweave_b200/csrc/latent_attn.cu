@@ -16,6 +16,7 @@
 //   tw_latent_gather   cache rows of some sequences, in order, into one contiguous buffer
 #include "tw_host.h"
 #include "tw_kernels.h"
+#include "tw_mma.cuh"
 #include "tw_typed.cuh"
 
 namespace tw {
@@ -132,17 +133,6 @@ struct HeadGemm {
 
 constexpr int HG_M = 64, HG_N = 64, HG_K = 64;
 constexpr int HG_LD = HG_K + 8;        // padded rows: conflict-free ldmatrix
-
-__device__ __forceinline__ void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
 
 // VEC: K, the strides and the bases keep 16-byte groups aligned.
 template <bool VEC>

@@ -1,0 +1,451 @@
+// Absorbed latent attention of single query rows on the tensor cores (tcgen05): every head of a row attends to the same
+// cache rows, [latent | rotated key part], and the values are the latent part of the rows themselves.
+//
+// A tile of 128 cache rows is fetched once and used twice:
+//     S^T [128 keys x heads]   = K Q^T      A = the tile, K-major; B = the absorbed queries, 16 or 32 heads
+//     O^T [latent x heads]    += C^T P^T    A = the same tile read MN-major, 128 latent columns per MMA block
+// so M is always full although a token has few query rows, and the kernel is bound by the cache bytes: the tile's
+// columns travel as pairs of 64-column chunks with a barrier each, the score product starts with the first pair and a
+// pair is refilled as soon as its part of O^T is done. Rows of up to 640 elements, latents of up to 512. The keys of a
+// row can be cut into splits, whose fp32 partial results a second kernel merges.
+//
+// Roles (192 threads): warp 0 TMA producer, warp 1 MMA issuer, warps 2..5 softmax (one thread per key of the tile),
+// rescaling and epilogue (one thread per latent column). Waits are bounded; after a timeout the roles keep their trip
+// counts, report TW_ERR_MBAR_TIMEOUT and leave through the tear-down.
+#include "tw_common.cuh"
+#include "tw_host.h"
+#include "tw_kernels.h"
+
+namespace tw {
+
+constexpr int LD_BN = 128;                    // keys per tile
+constexpr int LD_THREADS = 192;
+constexpr int LD_CHUNK = LD_BN * 128;         // 64 columns of a tile
+constexpr int LD_MAX_PAIRS = 5, LD_MAX_STAGES = 4;
+constexpr int LD_SMEM_LIMIT = 227 * 1024;
+
+struct LatentDecodeParams {
+  const __nv_bfloat16* q;        // [n, heads, row]
+  __nv_bfloat16* out;            // [n, heads, kv_rank]
+  const int *tok_seq, *tok_kvlen, *block_table;
+  int max_blocks, page, heads, row, kv_rank, splits, chunks, stages;
+  float scale_log2;
+  float *part_o, *part_ml;
+  uint32_t* status;
+};
+
+__device__ __forceinline__ float ld_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ void ld_softmax_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void tmem_ld_cols(uint32_t addr, uint32_t (&r)[16]) { tmem_ld_32x16(addr, r); }
+__device__ __forceinline__ void tmem_ld_cols(uint32_t addr, uint32_t (&r)[32]) { tmem_ld_32x32(addr, r); }
+__device__ __forceinline__ void tmem_st_cols(uint32_t addr, const uint32_t (&r)[16]) { tmem_st_32x16(addr, r); }
+__device__ __forceinline__ void tmem_st_cols(uint32_t addr, const uint32_t (&r)[32]) { tmem_st_32x32(addr, r); }
+
+// Shared memory behind the tiles: Q, P, barriers, exchange.
+template <int NC>
+__host__ __device__ constexpr int ld_fixed_bytes(int chunks) {
+  return chunks * NC * 128 + 2 * NC * 128 + 512 + 2 * 4 * NC * 4 + 1024;
+}
+
+template <int NC>
+__global__ void __launch_bounds__(LD_THREADS, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecodeParams p) {
+  constexpr uint32_t IDESC_S = make_idesc_bf16(LD_BN, NC, 0, 0);     // A = rows (K-major), B = Q (K-major)
+  constexpr uint32_t IDESC_O = make_idesc_bf16(128, NC, 1, 0);       // A = latent columns (MN-major), B = P (K-major)
+  constexpr uint32_t TMEM_COLS = NC == 16 ? 128 : 256;               // 2 NC for S, 4 NC for O
+  constexpr uint32_t COL_O = 2 * NC;
+
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
+                                             ~static_cast<uintptr_t>(1023));
+  const int pairs = (p.chunks + 1) >> 1;
+  const int v_chunks = (p.kv_rank + 63) >> 6, v_pairs = (v_chunks + 1) >> 1;
+  const int tile_bytes = pairs * 2 * LD_CHUNK;
+  uint8_t* s_q = smem + p.stages * tile_bytes;
+  uint8_t* s_p = s_q + p.chunks * NC * 128;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(s_p + 2 * NC * 128);
+  uint64_t* full = bars;                                      // [stages][LD_MAX_PAIRS]
+  uint64_t* empty = bars + LD_MAX_STAGES * LD_MAX_PAIRS;
+  uint64_t* s_full = bars + 2 * LD_MAX_STAGES * LD_MAX_PAIRS;  // [2]
+  uint64_t* p_ready = s_full + 2;
+  uint64_t* o_done = s_full + 3;
+  uint64_t* q_ready = s_full + 4;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(s_full + 5);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+  float* xchg = reinterpret_cast<float*>(reinterpret_cast<uint8_t*>(bars) + 512);    // [2][4 warps][NC]
+
+  const int warp = threadIdx.x >> 5;
+  const int lane = threadIdx.x & 31;
+  const int tok = blockIdx.x, h0 = blockIdx.y * NC, split = blockIdx.z;
+  const int G = min(NC, p.heads - h0);
+  const int seq = p.tok_seq[tok];
+  const int kv_len = p.tok_kvlen[tok];
+  const int tiles_total = (kv_len + LD_BN - 1) / LD_BN;
+  const int per_split = (tiles_total + p.splits - 1) / p.splits;
+  const int t_begin = split * per_split;
+  const int n_tiles = max(0, min(tiles_total, t_begin + per_split) - t_begin);
+
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < p.stages * LD_MAX_PAIRS; ++i) {
+      mbar_init(&full[i], 1);
+      mbar_init(&empty[i], 1);
+    }
+    mbar_init(&s_full[0], 1);
+    mbar_init(&s_full[1], 1);
+    mbar_init(p_ready, 128);
+    mbar_init(o_done, 1);
+    mbar_init(q_ready, 128);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, TMEM_COLS);
+    tmem_relinquish();
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem_base = *tmem_slot;
+
+  if (warp == 0) {
+    // ---------------- TMA producer ----------------
+    if (lane == 0 && n_tiles > 0) {
+      tma_prefetch_desc(&tmC);
+      const int pages_per_tile = LD_BN / p.page;
+      const int last_page = (kv_len - 1) / p.page;
+      const int* table = p.block_table + static_cast<long long>(seq) * p.max_blocks;
+      bool ok = true;
+      for (int j = 0; ok && j < n_tiles; ++j) {
+        const int st = j % p.stages;
+        const uint32_t ph = (j / p.stages) & 1;
+        uint8_t* tile = smem + st * tile_bytes;
+        for (int pr = 0; pr < pairs; ++pr) {
+          if (!mbar_wait(&empty[st * LD_MAX_PAIRS + pr], ph ^ 1)) { ok = false; break; }
+          uint64_t* bar = &full[st * LD_MAX_PAIRS + pr];
+          const int c_end = min(p.chunks, 2 * pr + 2);
+          mbar_expect_tx(bar, (c_end - 2 * pr) * LD_CHUNK);
+          for (int pg = 0; pg < pages_per_tile; ++pg) {
+            const int block = table[min((t_begin + j) * pages_per_tile + pg, last_page)];
+            for (int c = 2 * pr; c < c_end; ++c)
+              tma_load_3d(tile + c * LD_CHUNK + pg * p.page * 128, &tmC, bar, c * 64, 0, block);
+          }
+        }
+      }
+      if (!ok) {
+        report_error(p.status, TW_ERR_MBAR_TIMEOUT);
+        *abort_flag = 1;
+      }
+    }
+  } else if (warp == 1) {
+    // ---------------- MMA issuer ----------------
+    if (lane == 0 && n_tiles > 0) {
+      const uint32_t q_addr = smem_u32(s_q), p_addr = smem_u32(s_p);
+      bool ok = mbar_wait(q_ready, 0);
+      auto issue_s = [&](int j) {
+        const int st = j % p.stages;
+        const uint32_t ph = (j / p.stages) & 1;
+        const uint32_t tile = smem_u32(smem + st * tile_bytes);
+        for (int pr = 0; pr < pairs; ++pr) {
+          if (!mbar_wait(&full[st * LD_MAX_PAIRS + pr], ph)) return false;
+          tc_fence_after_sync();
+          const int c_end = min(p.chunks, 2 * pr + 2);
+          for (int c = 2 * pr; c < c_end; ++c) {
+#pragma unroll
+            for (int k = 0; k < 4; ++k)
+              umma_ss(tmem_base + (j & 1) * NC, make_smem_desc_sw128(tile + c * LD_CHUNK + k * 32, 16, 1024),
+                      make_smem_desc_sw128(q_addr + c * (NC * 128) + k * 32, 16, 1024), IDESC_S, (c | k) != 0 ? 1u : 0u);
+          }
+          if (pr >= v_pairs) umma_commit(&empty[st * LD_MAX_PAIRS + pr]);     // no latent column in this pair
+        }
+        umma_commit(&s_full[j & 1]);
+        return true;
+      };
+      if (ok) ok = issue_s(0);
+      for (int j = 0; ok && j < n_tiles; ++j) {
+        // with one tile buffer the next score product has to follow this tile's last use
+        if (p.stages > 1 && j + 1 < n_tiles) {
+          ok = issue_s(j + 1);
+          if (!ok) break;
+        }
+        if (!mbar_wait(p_ready, j & 1)) { ok = false; break; }
+        tc_fence_after_sync();
+        const int st = j % p.stages;
+        const uint32_t tile = smem_u32(smem + st * tile_bytes);
+        for (int m = 0; m < v_pairs; ++m) {
+#pragma unroll
+          for (int k = 0; k < LD_BN / 16; ++k)
+            umma_ss(tmem_base + COL_O + m * NC, make_smem_desc_sw128(tile + m * 2 * LD_CHUNK + k * 16 * 128, LD_CHUNK, 1024),
+                    make_smem_desc_sw128(p_addr + (k >> 2) * (NC * 128) + (k & 3) * 32, 16, 1024), IDESC_O,
+                    (j | k) != 0 ? 1u : 0u);
+          umma_commit(&empty[st * LD_MAX_PAIRS + m]);
+        }
+        umma_commit(o_done);
+        if (p.stages == 1 && j + 1 < n_tiles) ok = issue_s(j + 1);
+      }
+      if (!ok) {
+        report_error(p.status, TW_ERR_MBAR_TIMEOUT);
+        *abort_flag = 1;
+      }
+    }
+  } else {
+    // ---------------- softmax + epilogue (warps 2..5) ----------------
+    const int qr = warp & 3;                 // TMEM lane quarter this warp may touch
+    const int r = qr * 32 + lane;            // key within the tile / latent column within a block in the epilogue
+    const int sw = warp - 2;
+    const int t = threadIdx.x - 64;          // 0..127
+    const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(qr * 32) << 16);
+
+    // queries into the swizzled K-major operand layout, zeros behind the row's end and behind the last head
+    for (int i = t; i < NC * p.chunks * 8; i += 128) {
+      const int g = i / (p.chunks * 8), cidx = i - g * (p.chunks * 8);
+      uint4 v = make_uint4(0u, 0u, 0u, 0u);
+      if (g < G && cidx * 8 < p.row)
+        v = *reinterpret_cast<const uint4*>(p.q + (static_cast<long long>(tok) * p.heads + h0 + g) * p.row + cidx * 8);
+      *reinterpret_cast<uint4*>(s_q + (cidx >> 3) * (NC * 128) + g * 128 + (((cidx & 7) ^ (g & 7)) * 16)) = v;
+    }
+    fence_proxy_async_smem();
+    mbar_arrive(q_ready);
+
+    float m_ref[NC], l_part[NC];
+#pragma unroll
+    for (int g = 0; g < NC; ++g) {
+      m_ref[g] = -INFINITY;
+      l_part[g] = 0.f;
+    }
+    bool ok = true;
+    for (int j = 0; j < n_tiles; ++j) {
+      // fixed trip count for all 128 threads: after a failed wait the remaining waits are skipped, not the iterations
+      if (ok) ok = mbar_wait(&s_full[j & 1], (j >> 1) & 1);
+      tc_fence_after_sync();
+      uint32_t sv[NC];
+      tmem_ld_cols(t_lane + (j & 1) * NC, sv);
+      tmem_wait_ld();
+      float* xm = xchg + (j & 1) * 4 * NC;
+      if ((t_begin + j + 1) * LD_BN > kv_len && (t_begin + j) * LD_BN + r >= kv_len) {
+#pragma unroll
+        for (int g = 0; g < NC; ++g) sv[g] = __float_as_uint(-INFINITY);
+      }
+#pragma unroll
+      for (int g4 = 0; g4 < NC; g4 += 4) {
+        float4 mx;
+        mx.x = warp_max_redux(__uint_as_float(sv[g4]));
+        mx.y = warp_max_redux(__uint_as_float(sv[g4 + 1]));
+        mx.z = warp_max_redux(__uint_as_float(sv[g4 + 2]));
+        mx.w = warp_max_redux(__uint_as_float(sv[g4 + 3]));
+        if (lane == 0) *reinterpret_cast<float4*>(xm + sw * NC + g4) = mx;
+      }
+      ld_softmax_sync();
+      // a head's reference maximum moves when its maximum grew by more than 2^8 (rare after the first tiles); all 128
+      // threads see the same maxima and decide alike
+      float over = -1.f, mt[NC];
+#pragma unroll
+      for (int g4 = 0; g4 < NC; g4 += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(xm + g4);
+        const float4 b = *reinterpret_cast<const float4*>(xm + NC + g4);
+        const float4 c = *reinterpret_cast<const float4*>(xm + 2 * NC + g4);
+        const float4 d = *reinterpret_cast<const float4*>(xm + 3 * NC + g4);
+        mt[g4] = fmaxf(fmaxf(a.x, b.x), fmaxf(c.x, d.x)) * p.scale_log2;
+        mt[g4 + 1] = fmaxf(fmaxf(a.y, b.y), fmaxf(c.y, d.y)) * p.scale_log2;
+        mt[g4 + 2] = fmaxf(fmaxf(a.z, b.z), fmaxf(c.z, d.z)) * p.scale_log2;
+        mt[g4 + 3] = fmaxf(fmaxf(a.w, b.w), fmaxf(c.w, d.w)) * p.scale_log2;
+      }
+      bool rescale = false;
+      if (j == 0) {
+#pragma unroll
+        for (int g = 0; g < NC; ++g) m_ref[g] = mt[g];
+      } else {
+#pragma unroll
+        for (int g = 0; g < NC; ++g) over = fmaxf(over, mt[g] - m_ref[g]);
+        if (over > 8.f) {
+          rescale = true;
+#pragma unroll
+          for (int g = 0; g < NC; ++g) {
+            // mt becomes the factor of column g
+            const float a = mt[g] > m_ref[g] + 8.f ? ld_exp2(m_ref[g] - mt[g]) : 1.f;
+            if (mt[g] > m_ref[g] + 8.f) m_ref[g] = mt[g];
+            l_part[g] *= a;
+            mt[g] = a;
+          }
+        }
+      }
+      // P and O belong to the previous tile until its products are done. Every tile waits, needed or not: a parity
+      // wait only tells that the phase before the current one has completed
+      if (j > 0) {
+        if (ok) ok = mbar_wait(o_done, (j - 1) & 1);
+        tc_fence_after_sync();
+      }
+      uint8_t* p_buf = s_p + (r >> 6) * (NC * 128);
+      const int kc = (r & 63) >> 3, ke = r & 7;
+#pragma unroll
+      for (int g = 0; g < NC; ++g) {
+        const float pv = ld_exp2(fmaf(__uint_as_float(sv[g]), p.scale_log2, -m_ref[g]));
+        l_part[g] += pv;
+        *reinterpret_cast<__nv_bfloat16*>(p_buf + g * 128 + ((kc ^ (g & 7)) * 16) + ke * 2) = __float2bfloat16(pv);
+      }
+      if (rescale) {
+#pragma unroll 1
+        for (int m = 0; m < v_pairs; ++m) {
+          uint32_t ov[NC];
+          tmem_ld_cols(t_lane + COL_O + m * NC, ov);
+          tmem_wait_ld();
+#pragma unroll
+          for (int g = 0; g < NC; ++g) ov[g] = __float_as_uint(__uint_as_float(ov[g]) * mt[g]);
+          tmem_st_cols(t_lane + COL_O + m * NC, ov);
+        }
+        tmem_wait_st();
+      }
+      tc_fence_before_sync();
+      fence_proxy_async_smem();
+      mbar_arrive(p_ready);       // arrive even after a failed wait so that the issuer is not left hanging
+    }
+
+    // row sums over the owners of the keys
+    float* xs = xchg + (n_tiles & 1) * 4 * NC;
+#pragma unroll
+    for (int g = 0; g < NC; ++g) {
+      const float l = warp_sum(l_part[g]);
+      if (lane == 0) xs[sw * NC + g] = l;
+    }
+    ld_softmax_sync();
+    if (n_tiles > 0 && ok) ok = mbar_wait(o_done, (n_tiles - 1) & 1);
+    if (ok) {
+      tc_fence_after_sync();
+#pragma unroll 1
+      for (int m = 0; m < v_pairs; ++m) {
+        uint32_t ov[NC];
+        if (n_tiles > 0) {
+          tmem_ld_cols(t_lane + COL_O + m * NC, ov);
+          tmem_wait_ld();
+        }
+        const int d = m * 128 + r;
+#pragma unroll
+        for (int g = 0; g < NC; ++g) {
+          if (g < G && d < p.kv_rank) {
+            const float o = n_tiles > 0 ? __uint_as_float(ov[g]) : 0.f;
+            const float l = (xs[g] + xs[NC + g]) + (xs[2 * NC + g] + xs[3 * NC + g]);
+            const long long item = static_cast<long long>(tok) * p.heads + h0 + g;
+            if (p.splits == 1) {
+              p.out[item * p.kv_rank + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
+            } else {
+              const long long pi = item * p.splits + split;
+              p.part_o[pi * p.kv_rank + d] = o;
+              if (d == 0) {
+                p.part_ml[pi * 2] = m_ref[g];
+                p.part_ml[pi * 2 + 1] = l;
+              }
+            }
+          }
+        }
+      }
+    } else {
+      report_error(p.status, TW_ERR_MBAR_TIMEOUT);
+      *abort_flag = 1;
+    }
+  }
+
+  if (*abort_flag) {
+    // let copies and MMAs in flight land before shared memory and TMEM are given back
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after_sync();
+    tmem_dealloc(tmem_base, TMEM_COLS);
+  }
+}
+
+__global__ void __launch_bounds__(128)
+latent_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits, int kv_rank,
+                           __nv_bfloat16* __restrict__ out) {
+  const long long item = blockIdx.x;
+  float mm = -INFINITY, ll = 0.f;
+  for (int s = 0; s < splits; ++s) mm = fmaxf(mm, part_ml[(item * splits + s) * 2]);
+  for (int s = 0; s < splits; ++s) {
+    const float m = part_ml[(item * splits + s) * 2];
+    ll += m == -INFINITY ? 0.f : part_ml[(item * splits + s) * 2 + 1] * exp2f(m - mm);
+  }
+  const float inv = ll > 0.f ? 1.f / ll : 0.f;
+  for (int d = threadIdx.x; d < kv_rank; d += blockDim.x) {
+    float acc = 0.f;
+    for (int s = 0; s < splits; ++s) {
+      const float m = part_ml[(item * splits + s) * 2];
+      if (m != -INFINITY) acc = fmaf(part_o[(item * splits + s) * kv_rank + d], exp2f(m - mm), acc);
+    }
+    out[item * kv_rank + d] = __float2bfloat16(acc * inv);
+  }
+}
+
+template <int NC>
+static int launch_latent_decode(const CUtensorMap& tm, LatentDecodeParams& p, int n, cudaStream_t stream) {
+  const int pairs = (p.chunks + 1) / 2;
+  const int fixed = ld_fixed_bytes<NC>(p.chunks);
+  int stages = (LD_SMEM_LIMIT - fixed) / (pairs * 2 * LD_CHUNK);
+  if (stages > LD_MAX_STAGES) stages = LD_MAX_STAGES;
+  if (stages < 1) {
+    set_last_error("latent_decode: rows of %d elements do not fit shared memory", p.row);
+    return 1;
+  }
+  p.stages = stages;
+  const int bytes = fixed + stages * pairs * 2 * LD_CHUNK;
+  static thread_local int configured_dev = -1;
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (configured_dev != dev) {
+    const cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, LD_SMEM_LIMIT);
+    if (e != cudaSuccess) {
+      set_last_error("latent_decode: cudaFuncSetAttribute failed: %s", cudaGetErrorString(e));
+      return 1;
+    }
+    configured_dev = dev;
+  }
+  latent_decode_kernel<NC><<<dim3(n, (p.heads + NC - 1) / NC, p.splits), LD_THREADS, bytes, stream>>>(tm, p);
+  cudaError_t e = cudaGetLastError();
+  if (e == cudaSuccess && p.splits > 1) {
+    latent_decode_merge_kernel<<<n * p.heads, 128, 0, stream>>>(p.part_o, p.part_ml, p.splits, p.kv_rank, p.out);
+    e = cudaGetLastError();
+  }
+  if (e != cudaSuccess) {
+    set_last_error("latent_decode launch failed: %s", cudaGetErrorString(e));
+    return 1;
+  }
+  return 0;
+}
+
+}  // namespace tw
+
+using namespace tw;
+
+// qa [n, heads, row] absorbed queries, cache [num_blocks, page, row] (page a power of two, 8...128), out
+// [n, heads, kv_rank]; part_o [n, heads, splits, kv_rank] and part_ml [n, heads, splits, 2] when splits > 1.
+extern "C" int tw_latent_decode(const void* qa, const void* cache, int num_blocks, int page, const int* tok_seq,
+                                const int* tok_kvlen, int n, const int* block_table, int max_blocks, void* out, int heads,
+                                int row, int kv_rank, float scale, int splits, float* part_o, float* part_ml,
+                                uint32_t* status, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (row % 8 != 0 || row > 64 * 2 * LD_MAX_PAIRS || kv_rank > 512 || kv_rank > row || page < 8 || page > 128 || 128 % page != 0) {
+    set_last_error("latent_decode: unsupported cache rows (row=%d, kv_rank=%d, page=%d)", row, kv_rank, page);
+    return 1;
+  }
+  if (splits < 1) splits = 1;
+  if (splits > 1 && (part_o == nullptr || part_ml == nullptr)) {
+    set_last_error("latent_decode: splits need the partial-result workspace");
+    return 1;
+  }
+  CUtensorMap tm;
+  {
+    uint64_t dims[3] = {(uint64_t)row, (uint64_t)page, (uint64_t)num_blocks};
+    uint64_t strides[2] = {(uint64_t)row * 2, (uint64_t)page * row * 2};
+    uint32_t box[3] = {64, (uint32_t)page, 1};
+    if (!make_tensor_map_bf16(&tm, cache, 3, dims, strides, box)) return 1;
+  }
+  LatentDecodeParams p{reinterpret_cast<const __nv_bfloat16*>(qa), reinterpret_cast<__nv_bfloat16*>(out), tok_seq, tok_kvlen,
+                       block_table, max_blocks, page, heads, row, kv_rank, splits, (row + 63) / 64, 1,
+                       scale * 1.4426950408889634f, part_o, part_ml, status};
+  return heads <= 16 ? launch_latent_decode<16>(tm, p, n, stream) : launch_latent_decode<32>(tm, p, n, stream);
+}

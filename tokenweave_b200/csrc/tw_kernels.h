@@ -172,10 +172,19 @@ int tw_head_gemm(const void* A, long long lda, int a_hs, const int* a_rows, cons
 int tw_latent_attn(const void* qa, const void* cache, const int* tok_seq, const int* tok_kvlen, int n,
                    const int* block_table, int max_blocks, int page, void* out, int heads, int row, int kv_rank,
                    float scale, int dtype, cudaStream_t stream);
+// tensor-core forms (latent_attn_decode.cu, latent_attn_prefill.cu), bf16
+int tw_latent_decode(const void* qa, const void* cache, int num_blocks, int page, const int* tok_seq,
+                     const int* tok_kvlen, int n, const int* block_table, int max_blocks, void* out, int heads, int row,
+                     int kv_rank, float scale, int splits, float* part_o, float* part_ml, uint32_t* status,
+                     cudaStream_t stream);
+int tw_latent_prefill(const void* q, long long ldq, int T, const void* kv, long long ldkv, const void* kr, long long ldr,
+                      int ctx_rows, const int* ctx_begin, void* out, long long ldo, const void* gate, long long ldg,
+                      const int* cu_q, const int* kv_lens, const int* tile_seq, const int* tile_q0, int num_tiles,
+                      int heads, int dim, int rot, int vdim, float scale, uint32_t* status, cudaStream_t stream);
 int tw_latent_gather(const void* cache, void* dst, const int* seqs, const int* cu, int n_seqs, int max_rows,
                      const int* block_table, int max_blocks, int page, int row_bytes, cudaStream_t stream);
 
-// ---- state-space recurrence (ssm.cu) ----
+// ---- state-space recurrence (ssm.cu, ssd_chunk.cu) ----
 int tw_causal_conv(const void* x, long long ldx, const void* w, const void* bias, void* state, void* out, long long ldo,
                    const int* row_seq, const int* cu_q, const int* kv_lens, const int* slots, int T, int n_seqs,
                    int channels, int taps, int single, int dtype, cudaStream_t stream);
@@ -183,6 +192,9 @@ int tw_ssd_scan(const void* xbc, long long ldx, const void* dt, long long ldt, c
                 const void* D, float* state, void* y, long long ldy, const int* seqs, int n_seqs, const int* cu_q,
                 const int* kv_lens, const int* slots, int heads, int vdim, int N, int groups, int dtype,
                 cudaStream_t stream);
+int tw_ssd_chunk(const void* xbc, long long ldx, const void* dt, long long ldt, const void* dt_bias, const void* A_log,
+                 const void* D, float* state, void* y, long long ldy, const int* seqs, int n_seqs, const int* cu_q,
+                 const int* kv_lens, const int* slots, int heads, int vdim, int N, int groups, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

@@ -100,6 +100,19 @@ class LatentAttention(Mixer):
                 ("query", self.uq_proj.out_padded), ("mixed", self.o_proj.in_padded),
                 ("absorbed", self.heads * self.row), ("latent_out", self.heads * self.kv_rank)]
 
+    def context_workspaces(self) -> list[tuple[str, int]]:
+        """Buffers with one row per context token of the expanded form."""
+        return [("ctx_latent", self.row), ("ctx_kv", self.ukv_proj.out_padded)]
+
+    @property
+    def expandable(self) -> bool:
+        w = self.o_proj.weight
+        return w.is_cuda and hops.latent_expandable(w.dtype, self.dim, self.rot_dim, self.vdim)
+
+    def launch_key(self, meta: AttentionMetadata, block_size: int, sm_count: int) -> tuple:
+        return hops.latent_decode_plan(meta.num_single, self.heads, self.row, self.kv_rank, block_size,
+                                       self.o_proj.weight.dtype, meta.max_kv_len, sm_count)
+
     # ---- cache -----------------------------------------------------------------------------------------
     def cache_bytes_per_block(self, block_size: int) -> int:
         return block_size * self.row * self.o_proj.weight.element_size()
@@ -169,8 +182,19 @@ class LatentAttention(Mixer):
                                self.cos_sin, meta.positions, qa)
             o = rt.buffer("latent_out", m, H * self.kv_rank).view(m, H, self.kv_rank)
             hops.latent_attention(qa, self.cache, meta.tok_seq, meta.tok_kvlen, m, meta.block_table, self.kv_rank,
-                                  self.scale, o)
+                                  self.scale, o, meta.max_kv_len, rt.sm_count)
             hops.latent_values(o, meta.tok_row, w_uv, H, self.vdim, self.kv_rank, gate, attn)
+        if meta.num_tiles:
+            # keys and values of the tiles' contexts (the step's own tokens are in the cache already)
+            rows = meta.extra_cpu["ctx_rows"]
+            lat = rt.buffer("ctx_latent", rows, self.row)
+            hops.latent_gather(self.cache, meta.extra["ctx_seqs"], meta.extra["ctx_cu"], meta.extra_cpu["ctx_max"],
+                               meta.block_table, lat)
+            kv = self.ukv_proj(lat[:, :self.ukv_proj.in_padded], out=rt.buffer("ctx_kv", rows, self.ukv_proj.out_padded))
+            hops.rope_tail_(q, H, self.dim + self.rot_dim, self.dim, self.rot_dims, self.cos_sin, meta.positions)
+            hops.latent_prefill(q, kv, lat, pad8(self.kv_rank), rows, meta.extra["ctx_begin"], attn, gate, meta.cu_q,
+                                meta.kv_lens, meta.tile_seq, meta.tile_q0, meta.num_tiles, H, self.dim, self.rot_dim,
+                                self.vdim, self.scale)
         self.o_proj(attn, out=out)
 
 
@@ -207,6 +231,10 @@ class Mamba2Mixer(Mixer):
     def workspaces(self) -> list[tuple[str, int]]:
         return [("proj", self.in_proj.out_padded), ("conv", pad8(self.channels)), ("mixed", self.o_proj.in_padded),
                 ("gated", self.o_proj.in_padded)]
+
+    @property
+    def chunkable(self) -> bool:
+        return self.conv_w.is_cuda and hops.ssd_chunkable(self.conv_w.dtype, self.vdim, self.N)
 
     # ---- state -----------------------------------------------------------------------------------------
     def state_bytes_per_slot(self) -> int:
@@ -252,8 +280,11 @@ class Mamba2Mixer(Mixer):
         hops.causal_conv(p[:, self.x_off:], self.conv_w, self.conv_b, self.conv_state, xbc, e["row_seq"], meta.cu_q,
                          meta.kv_lens, e["state_slots"], meta.all_single)
         y = rt.buffer("mixed", n, self.o_proj.in_padded)
-        hops.ssd_scan(xbc, p[:, self.dt_off:], self.dt_bias, self.A_log, self.D, self.state, y, e["scan_seqs"],
-                      meta.cu_q, meta.kv_lens, e["state_slots"], self.groups)
+        # long runs in chunks on the tensor cores (sizes permitting), everything else token by token
+        for run, seqs in ((hops.ssd_scan, e["scan_seqs"]),
+                          (hops.ssd_chunk if self.chunkable else hops.ssd_scan, e["chunk_seqs"])):
+            run(xbc, p[:, self.dt_off:], self.dt_bias, self.A_log, self.D, self.state, y, seqs, meta.cu_q, meta.kv_lens,
+                e["state_slots"], self.groups)
         g = rt.buffer("gated", n, self.o_proj.in_padded)
         hops.gated_group_norm(y, p, self.norm_w, self.norm_groups, self.eps, g)
         self.o_proj(g, out=out)

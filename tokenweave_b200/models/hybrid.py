@@ -20,9 +20,9 @@ import torch
 from torch import nn
 
 from ..config import ModelConfig
-from ..layers.attention import AttentionMetadata
+from ..layers.attention import PREFILL_MIN_Q, AttentionMetadata
 from ..layers.linear import PaddedLinear, pad8
-from ..layers.mixers import FEED_FORWARDS, MIXERS, LatentAttention, Mamba2Mixer
+from ..layers.mixers import FEED_FORWARDS, MIXERS, LatentAttention
 from ..ops import hybrid as hops
 from ..parallel.comm import TPCommunicator
 from ..parallel.state import get_tp
@@ -47,6 +47,8 @@ class HybridRuntime:
         self.comm = TPCommunicator(self.staging, tp, tw_cfg.wait_budget_ms, tw_cfg.transport)
         self.dtype = cfg.dtype
         self.sm_count = torch.cuda.get_device_properties(device).multi_processor_count if device.type == "cuda" else 0
+        # context tokens whose keys and values a step may expand
+        self.context_rows = max(max_tokens, min(cfg.max_model_len, 32768))
         self.rope_tables: dict = {}
         self._buffers: dict[tuple, torch.Tensor] = {}
 
@@ -104,6 +106,8 @@ class HybridDecoder(nn.Module):
         self.final_norm_w = nn.Parameter(torch.ones(W, dtype=dt, device=device), requires_grad=False)
         self.head = PaddedLinear(W, cfg.vocab_size, dtype=dt, device=device)
         self.rt: Optional[HybridRuntime] = None
+        latent = [l.mixer for l in self.layers if isinstance(l.mixer, LatentAttention)]
+        self.expand = bool(latent) and all(m.expandable for m in latent)      # long runs may use the expanded form
         self.recurrent = any(l.mixer.recurrent for l in self.layers)
 
     # ---- runtime ---------------------------------------------------------------------------------------
@@ -115,6 +119,9 @@ class HybridDecoder(nn.Module):
             for part in (m, layer.mlp):
                 for name, cols in part.workspaces() if part is not None else ():
                     self.rt.buffer(name, max_tokens, cols)
+                if self.expand and part is m and isinstance(m, LatentAttention):
+                    for name, cols in m.context_workspaces():
+                        self.rt.buffer(name, self.rt.context_rows, cols)
             if isinstance(m, LatentAttention):
                 key = m.rope_key()
                 if key not in self.rt.rope_tables:
@@ -145,26 +152,56 @@ class HybridDecoder(nn.Module):
 
     # ---- a step's layout -------------------------------------------------------------------------------
     def plan_step(self, q_lens, kv_lens, state_slots):
-        """Routing of a step's rows: (attention plan as of ``plan_attention``, extra int32 arrays,
-        host values)."""
-        rows, seqs, lens = [], [], []
-        row = 0
-        for b, (n, kv) in enumerate(zip(q_lens, kv_lens)):
-            rows.append(np.arange(row, row + n, dtype=np.int32))
-            seqs.append(np.full(n, b, dtype=np.int32))
-            lens.append(np.arange(kv - n + 1, kv + 1, dtype=np.int32))
-            row += n
-        cat = lambda parts: np.concatenate(parts) if parts else np.empty(0, np.int32)
-        row_seq = cat(seqs)
-        extra = {"row_seq": row_seq}
+        """Routing of a step's rows: (attention plan as of ``plan_attention``, extra int32 arrays, host values).
+
+        Attention: a run of a prompt goes to 128-query tiles over expanded keys and values when it is long enough to
+        pay for expanding its context (a product over the whole context, whatever the run's length), and when the
+        context fits the workspace; every other row is attended alone in the absorbed form. Recurrences: long runs in
+        chunks, short ones token by token."""
+        B = len(q_lens)
+        if max(q_lens) == 1:
+            rows = np.arange(B, dtype=np.int32)
+            plan = ([], [], rows, rows, np.asarray(kv_lens, dtype=np.int32))
+            extra = {"row_seq": rows}
+            if self.recurrent:
+                extra.update(state_slots=np.asarray(state_slots, dtype=np.int32), scan_seqs=rows, chunk_seqs=rows[:0])
+            return plan, extra, {}
+        n = np.asarray(q_lens)
+        tiled, ctx_rows = [], 0
+        if self.expand:
+            for b, (ql, kv) in enumerate(zip(q_lens, kv_lens)):
+                if (ql >= 64 or (ql >= PREFILL_MIN_Q and kv <= 2 * ql)) and ctx_rows + kv <= self.rt.context_rows:
+                    tiled.append(b)
+                    ctx_rows += kv
+        row_seq = np.repeat(np.arange(B, dtype=np.int32), n)
+        start = np.cumsum(n) - n
+        tok_row = np.flatnonzero(~np.isin(row_seq, tiled)).astype(np.int32)
+        tok_seq = row_seq[tok_row]
+        tok_kv = (np.asarray(kv_lens) - n)[tok_seq] + (tok_row - start[tok_seq]) + 1
+        tile_seq = [b for b in tiled for _ in range(0, q_lens[b], 128)]
+        tile_q0 = [q0 for b in tiled for q0 in range(0, q_lens[b], 128)]
+        order = np.argsort([-(kv_lens[b] - q_lens[b] + q0) for b, q0 in zip(tile_seq, tile_q0)], kind="stable")
+        plan = ([tile_seq[i] for i in order], [tile_q0[i] for i in order], tok_row, tok_seq, tok_kv.astype(np.int32))
+        extra, host = {"row_seq": row_seq}, {}
+        if tiled:
+            cu = np.zeros(len(tiled) + 1, dtype=np.int32)
+            np.cumsum([kv_lens[b] for b in tiled], out=cu[1:])
+            begin = np.full(B, -1, dtype=np.int32)
+            begin[tiled] = cu[:-1]
+            extra.update(ctx_seqs=np.asarray(tiled, dtype=np.int32), ctx_cu=cu, ctx_begin=begin)
+            host = {"ctx_rows": int(cu[-1]), "ctx_max": max(kv_lens[b] for b in tiled)}
         if self.recurrent:
-            extra["state_slots"] = np.asarray(state_slots, dtype=np.int32)
-            extra["scan_seqs"] = np.arange(len(q_lens), dtype=np.int32)
-        return ([], [], cat(rows), row_seq, cat(lens)), extra, {}
+            long = n >= hops.CHUNK_MIN_TOKENS
+            extra.update(state_slots=np.asarray(state_slots, dtype=np.int32),
+                         scan_seqs=np.flatnonzero(~long).astype(np.int32), chunk_seqs=np.flatnonzero(long).astype(np.int32))
+        return plan, extra, host
 
     def launch_key(self, meta: AttentionMetadata, block_size: int) -> tuple:
         """What shapes a step's launches besides its token and sequence counts (part of a graph's signature)."""
-        return (meta.all_single,) + tuple(sorted((k, v.shape[0]) for k, v in meta.extra.items()))
+        return (meta.all_single, tuple(sorted(meta.extra_cpu.items())),
+                tuple(sorted((k, v.shape[0]) for k, v in meta.extra.items())),
+                tuple(sorted({l.mixer.launch_key(meta, block_size, self.rt.sm_count) for l in self.layers
+                              if isinstance(l.mixer, LatentAttention)})))
 
     # ---- forward ---------------------------------------------------------------------------------------
     @torch.inference_mode()

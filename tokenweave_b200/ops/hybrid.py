@@ -12,7 +12,7 @@ from typing import Optional
 import torch
 
 from . import _native, reference_hybrid as ref
-from . import _p, _row_stride, _stream
+from . import _p, _row_stride, _stream, decode_splits_tc, status_word
 
 
 def _dt(*ts: Optional[torch.Tensor]) -> int:
@@ -115,18 +115,77 @@ def latent_absorb(q: torch.Tensor, rows: torch.Tensor, w_ukt: torch.Tensor, head
                  dim, rot, rot_dims, kv_rank, row, cos_sin.data_ptr(), positions.data_ptr(), dt, _stream())
 
 
+def latent_decode_plan(n: int, heads: int, row: int, kv_rank: int, page: int, dtype: torch.dtype, max_kv_len: int,
+                       sm_count: int = 148) -> tuple[str, int]:
+    """(kernel, key splits) of an absorbed attention launch: "tc" (tensor cores: bf16, cache rows of up to 640 elements
+    with a latent of up to 512) or "simt" (fp32 and every other size)."""
+    if dtype != torch.bfloat16 or row > 640 or kv_rank > 512 or page < 8 or page > 128 or 128 % page:
+        return "simt", 1
+    blocks = (heads + 15) // 16 if heads <= 16 else (heads + 31) // 32
+    return "tc", decode_splits_tc(n * blocks, (max_kv_len + 127) // 128, sm_count)
+
+
+_partials: dict[tuple, tuple[torch.Tensor, torch.Tensor]] = {}
+
+
+def _partial_buffers(device, count: int, width: int) -> tuple[torch.Tensor, torch.Tensor]:
+    """Workspace of split launches; sizes are powers of two and buffers are never freed (captured graphs keep their
+    addresses)."""
+    count = 1 << max(0, (count - 1).bit_length())
+    key = (device.index, count, width)
+    ws = _partials.get(key)
+    if ws is None:
+        ws = _partials[key] = (torch.empty(count * width, dtype=torch.float32, device=device),
+                               torch.empty(count * 2, dtype=torch.float32, device=device))
+    return ws
+
+
 def latent_attention(qa: torch.Tensor, cache: torch.Tensor, tok_seq: torch.Tensor, tok_kvlen: torch.Tensor, n: int,
-                     block_table: torch.Tensor, kv_rank: int, scale: float, out: torch.Tensor) -> None:
-    """Causal attention of ``n`` absorbed query rows over the paged latent cache; ``out`` [n, heads, kv_rank]."""
+                     block_table: torch.Tensor, kv_rank: int, scale: float, out: torch.Tensor, max_kv_len: int,
+                     sm_count: int = 148, kernel: Optional[str] = None) -> None:
+    """Causal attention of ``n`` absorbed query rows over the paged latent cache; ``out`` [n, heads, kv_rank].
+    ``kernel``: force one of :func:`latent_decode_plan`'s kernels (tests)."""
     if n == 0:
         return
     heads, row, page = qa.shape[1], qa.shape[2], cache.shape[1]
     if not qa.is_cuda:
         out[:n] = ref.latent_attention(qa[:n], cache, tok_seq, tok_kvlen, block_table, kv_rank, scale)
         return
+    dt = _dt(qa, cache, out)
+    plan, splits = latent_decode_plan(n, heads, row, kv_rank, page, qa.dtype, max_kv_len, sm_count)
+    if (kernel or plan) == "tc":
+        po = pm = None
+        if splits > 1:
+            po, pm = _partial_buffers(qa.device, n * heads * splits, kv_rank)
+        _native.call("tw_latent_decode", qa.data_ptr(), cache.data_ptr(), cache.shape[0], page, tok_seq.data_ptr(),
+                     tok_kvlen.data_ptr(), n, block_table.data_ptr(), block_table.shape[1], out.data_ptr(), heads, row,
+                     kv_rank, float(scale), splits, _p(po), _p(pm), status_word(qa.device).data_ptr(), _stream())
+        return
     _native.call("tw_latent_attn", qa.data_ptr(), cache.data_ptr(), tok_seq.data_ptr(), tok_kvlen.data_ptr(), n,
                  block_table.data_ptr(), block_table.shape[1], page, out.data_ptr(), heads, row, kv_rank, float(scale),
-                 _dt(qa, cache, out), _stream())
+                 dt, _stream())
+
+
+def latent_expandable(dtype: torch.dtype, dim: int, rot: int, vdim: int) -> bool:
+    """Head sizes the expanded tensor-core prefill takes (bf16)."""
+    kc, vc = (dim + 63) // 64 + (rot + 63) // 64, (vdim + 63) // 64
+    return dtype == torch.bfloat16 and dim % 8 == rot % 8 == vdim % 8 == 0 and vc <= 2 and kc + vc <= 5
+
+
+def latent_prefill(q: torch.Tensor, kv: torch.Tensor, latents: torch.Tensor, rot_off: int, ctx_rows: int,
+                   ctx_begin: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor], cu_q: torch.Tensor,
+                   kv_lens: torch.Tensor, tile_seq: torch.Tensor, tile_q0: torch.Tensor, num_tiles: int, heads: int,
+                   dim: int, rot: int, vdim: int, scale: float) -> None:
+    """Expanded causal attention of the listed 128-query tiles (CUDA, bf16). ``q`` [T, heads * (dim + rot)] with rotated
+    tails; ``kv`` [ctx_rows, heads * dim | heads * vdim] and the rotated part ``latents[:, rot_off:]`` of every
+    context row; sequence b's context starts at workspace row ``ctx_begin[b]``."""
+    _dt(q, kv, latents, out, gate)
+    kr = latents[:, rot_off:]
+    _native.call("tw_latent_prefill", q.data_ptr(), _row_stride(q), q.shape[0], kv.data_ptr(), _row_stride(kv),
+                 kr.data_ptr(), _row_stride(kr), ctx_rows, ctx_begin.data_ptr(), out.data_ptr(), _row_stride(out),
+                 _p(gate), _row_stride(gate) if gate is not None else 0, cu_q.data_ptr(), kv_lens.data_ptr(),
+                 tile_seq.data_ptr(), tile_q0.data_ptr(), num_tiles, heads, dim, rot, vdim, float(scale),
+                 status_word(q.device).data_ptr(), _stream())
 
 
 def latent_values(o: torch.Tensor, rows: torch.Tensor, w_uv: torch.Tensor, heads: int, vdim: int, kv_rank: int,
@@ -183,3 +242,24 @@ def ssd_scan(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, A_log: 
                  A_log.data_ptr(), D.data_ptr(), state.data_ptr(), y.data_ptr(), _row_stride(y), seqs.data_ptr(),
                  seqs.shape[0], cu_q.data_ptr(), kv_lens.data_ptr(), slots.data_ptr(), heads, vdim, N, groups,
                  _dt(xbc, dt, dt_bias, A_log, D, y), _stream())
+
+
+CHUNK_MIN_TOKENS = 16        # runs of at least this many tokens take the chunked form
+
+
+def ssd_chunkable(dtype: torch.dtype, vdim: int, N: int) -> bool:
+    """Sizes the chunked tensor-core form of the recurrence takes (bf16 activations)."""
+    return dtype == torch.bfloat16 and vdim % 8 == 0 and N % 8 == 0 and N <= 256
+
+
+def ssd_chunk(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor,
+              state: torch.Tensor, y: torch.Tensor, seqs: torch.Tensor, cu_q: torch.Tensor, kv_lens: torch.Tensor,
+              slots: torch.Tensor, groups: int) -> None:
+    """:func:`ssd_scan` for long runs: 64 tokens at a time on the tensor cores (CUDA, bf16)."""
+    if seqs.shape[0] == 0:
+        return
+    _, heads, vdim, N = state.shape
+    assert state.dtype == torch.float32 and _dt(xbc, dt, dt_bias, A_log, D, y) == 0
+    _native.call("tw_ssd_chunk", xbc.data_ptr(), _row_stride(xbc), dt.data_ptr(), _row_stride(dt), dt_bias.data_ptr(),
+                 A_log.data_ptr(), D.data_ptr(), state.data_ptr(), y.data_ptr(), _row_stride(y), seqs.data_ptr(),
+                 seqs.shape[0], cu_q.data_ptr(), kv_lens.data_ptr(), slots.data_ptr(), heads, vdim, N, groups, _stream())
