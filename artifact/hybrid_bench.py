@@ -181,13 +181,18 @@ def kernels(width: int, T: int = 8192, batch: int = 128, context: int = 2048) ->
               m * (chan + inner) * 2 + mh * P * N * 8, 2.0 * m * mh * (64 * N / (mh / groups) / 2 + 64 * P / 2 + 2 * N * P))
         del pr, qkv, xbc, xo, st, ys
         # matrix products, both models' shapes go through the same kernel
-        for name, n, k in (("in_proj (latent)", q8 + kv8 + heads * VDIM, width), ("in_proj (mamba)", inner + chan + mh, width),
-                           ("up_proj", ff, width), ("down_proj", width, ff)):
+        for name, n, k, like in (("in_proj (latent)", q8 + kv8 + heads * VDIM, width, "qkv"),
+                                 ("in_proj (mamba)", inner + chan + mh, width, "gate_up"),
+                                 ("up_proj", ff, width, "gate_up"), ("down_proj", width, ff, "down")):
             a, b = _r(m, k), _r(n + (-n) % 8, k, scale=0.02)
             c = torch.empty(m, b.shape[0], dtype=torch.bfloat16, device="cuda")
-            t(f"gemm {name} [{tag}]", f"gemm llama gate_up [{tag}]", lambda: ops.gemm(a, b, out=c), (m * k + n * k + m * n) * 2,
+            t(f"gemm {name} [{tag}]", f"gemm llama {like} [{tag}]", lambda: ops.gemm(a, b, out=c), (m * k + n * k + m * n) * 2,
               2.0 * m * n * k)
         lf = ff * 2 // 3 // 64 * 64
+        for name, n, k in (("qkv", (heads + 2 * hkv) * 128, width), ("down", width, lf)):
+            a, b = _r(m, k), _r(n, k, scale=0.02)
+            c = torch.empty(m, n, dtype=torch.bfloat16, device="cuda")
+            t(f"gemm llama {name} [{tag}]", "", lambda: ops.gemm(a, b, out=c), (m * k + n * k + m * n) * 2, 2.0 * m * n * k)
         a, b = _r(m, width), _r(2 * lf, width, scale=0.02)
         t(f"gemm llama gate_up [{tag}]", "", lambda: ops.gemm(a, b, swiglu=True), (m * width + 2 * lf * width + m * lf) * 2,
           4.0 * m * lf * width)

@@ -23,7 +23,9 @@ namespace tw {
 
 __device__ __forceinline__ int round8(int x) { return (x + 7) & ~7; }
 
-template <typename T, bool VEC>
+// One CTA per token. The groups of eight of the query latent and of the key/value latent are dealt to the threads in one
+// sequence and stay in registers between the sums and the writes.
+template <typename T, bool VEC, int VPT>
 __global__ void __launch_bounds__(256)
 latent_prep_kernel(const T* __restrict__ p, long long ldp, int q_off, int q_rank, const T* __restrict__ wq,
                    T* __restrict__ cq, long long ldcq, int kv_off, int kv_rank, const T* __restrict__ wkv, int rot,
@@ -32,42 +34,39 @@ latent_prep_kernel(const T* __restrict__ p, long long ldp, int q_off, int q_rank
   __shared__ float scratch[64];
   const int t = blockIdx.x;
   const T* src = p + t * ldp;
+  const int nq = (q_rank + 7) >> 3, n_all = nq + ((kv_rank + 7) >> 3);
+  float v[VPT][8], g[VPT][8];
   float s[2] = {0.f, 0.f};
-  for (int i = threadIdx.x * 8; i < q_rank; i += blockDim.x * 8) {
-    float v[8];
-    ld8n<VEC>(src + q_off + i, q_rank - i, v);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) s[0] += v[j] * v[j];
-  }
-  for (int i = threadIdx.x * 8; i < kv_rank; i += blockDim.x * 8) {
-    float v[8];
-    ld8n<VEC>(src + kv_off + i, kv_rank - i, v);
+  for (int k = 0; k < VPT; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    const bool is_q = i < nq;
+    const int c = (is_q ? i : i - nq) * 8, n = i < n_all ? (is_q ? q_rank : kv_rank) - c : 0;
+    ld8n<VEC>(src + (is_q ? q_off : kv_off) + c, n, v[k]);
+    ld8n<VEC>((is_q ? wq : wkv) + c, n, g[k]);
+    float ss = 0.f;
 #pragma unroll
-    for (int j = 0; j < 8; ++j) s[1] += v[j] * v[j];
+    for (int j = 0; j < 8; ++j) ss += v[k][j] * v[k][j];
+    if (is_q) s[0] += ss; else s[1] += ss;
   }
   block_sum<2>(s, scratch);
   const float rq = 1.f / sqrtf(s[0] / static_cast<float>(q_rank) + eps);
   const float rk = 1.f / sqrtf(s[1] / static_cast<float>(kv_rank) + eps);
-  for (int i = threadIdx.x * 8; i < q_rank; i += blockDim.x * 8) {
-    float v[8], g[8];
-    ld8n<VEC>(src + q_off + i, q_rank - i, v);
-    ld8n<VEC>(wq + i, q_rank - i, g);
-#pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] = v[j] * rq * g[j];
-    st8n<VEC>(cq + t * ldcq + i, q_rank - i, v);
-  }
   const int slot = slots[t];
-  if (slot < 0) return;
-  T* dst = cache + static_cast<long long>(slot) * row;
+  T* dst = cache + static_cast<long long>(slot < 0 ? 0 : slot) * row;
   const int rp = round8(kv_rank);
-  for (int i = threadIdx.x * 8; i < rp; i += blockDim.x * 8) {
-    float v[8], g[8];
-    ld8n<VEC>(src + kv_off + i, kv_rank - i, v);
-    ld8n<VEC>(wkv + i, kv_rank - i, g);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] = v[j] * rk * g[j];
-    st8(dst + i, v);                       // the pad behind the latent is written as zeros
+  for (int k = 0; k < VPT; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    if (i >= n_all) continue;
+    const bool is_q = i < nq;
+    const int c = (is_q ? i : i - nq) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[k][j] = v[k][j] * (is_q ? rq : rk) * g[k][j];
+    if (is_q) st8n<VEC>(cq + t * ldcq + c, q_rank - c, v[k]);
+    else if (slot >= 0) st8(dst + c, v[k]);          // the pad behind the latent is written as zeros
   }
+  if (slot < 0) return;
   const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot_dims;
   const int half = rot_dims >> 1;
   for (int i = threadIdx.x; i < row - rp; i += blockDim.x) {
@@ -83,20 +82,38 @@ latent_prep_kernel(const T* __restrict__ p, long long ldp, int q_off, int q_rank
   }
 }
 
-// Rotates elements [off, off + rot_dims) of every head of the listed rows in place.
-template <typename T>
+// Rotates elements [off, off + rot_dims) of every head of every row in place; VEC: eight pairs per thread.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 rope_tail_kernel(T* __restrict__ q, long long ldq, int heads, int head_stride, int off, int rot_dims,
                  const float* __restrict__ cos_sin, const int* __restrict__ positions) {
   const int t = blockIdx.x;
   const int half = rot_dims >> 1;
   const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot_dims;
-  for (int i = threadIdx.x; i < heads * half; i += blockDim.x) {
-    const int h = i / half, j = i - h * half;
+  constexpr int W = VEC ? 8 : 1;
+  const int per = half / W;
+  for (int i = threadIdx.x; i < heads * per; i += blockDim.x) {
+    const int h = i / per, j = (i - h * per) * W;
     T* u = q + t * ldq + h * head_stride + off + j;
-    const float a = ld1(u), b = ld1(u + half), c = cs[j], s = cs[half + j];
-    st1(u, a * c - b * s);
-    st1(u + half, b * c + a * s);
+    if (VEC) {
+      float a[8], b[8], c[8], s[8];
+      ld8(u, a);
+      ld8(u + half, b);
+      ld8(cs + j, c);
+      ld8(cs + half + j, s);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        const float x = a[e] * c[e] - b[e] * s[e];
+        b[e] = b[e] * c[e] + a[e] * s[e];
+        a[e] = x;
+      }
+      st8(u, a);
+      st8(u + half, b);
+    } else {
+      const float a = ld1(u), b = ld1(u + half), c = cs[j], s = cs[half + j];
+      st1(u, a * c - b * s);
+      st1(u + half, b * c + a * s);
+    }
   }
 }
 
@@ -134,28 +151,30 @@ struct HeadGemm {
 constexpr int HG_M = 64, HG_N = 64, HG_K = 64;
 constexpr int HG_LD = HG_K + 8;        // padded rows: conflict-free ldmatrix
 
-// VEC: K, the strides and the bases keep 16-byte groups aligned.
+constexpr int HG_STAGES = 4;
+constexpr int HG_SMEM = HG_STAGES * (HG_M + HG_N) * HG_LD * 2;
+
+// Eight elements of one row into shared memory, zeros behind the row's end and for rows outside the problem. VEC: K, the
+// strides and the bases keep 16-byte groups aligned, the copy is asynchronous.
 template <bool VEC>
-__device__ __forceinline__ void hg_load(__nv_bfloat16* dst, const __nv_bfloat16* src, bool row_ok, int k_left) {
-  // eight elements of one row; beyond the row's end or for rows outside the problem they are zero
-  uint4 u = make_uint4(0, 0, 0, 0);
-  if (row_ok) {
-    if (VEC && k_left >= 8) {
-      u = *reinterpret_cast<const uint4*>(src);
-    } else {
-      __nv_bfloat16* e = reinterpret_cast<__nv_bfloat16*>(&u);
+__device__ __forceinline__ void hg_load(__nv_bfloat16* dst, const __nv_bfloat16* row, int k, int K, const void* base) {
+  const bool ok = row != nullptr && k < K;
+  if (VEC) {
+    cp_async16(dst, ok ? static_cast<const void*>(row + k) : base, ok ? 16 : 0);    // zero bytes: base is not read
+  } else {
+    uint4 u = make_uint4(0, 0, 0, 0);
+    __nv_bfloat16* e = reinterpret_cast<__nv_bfloat16*>(&u);
 #pragma unroll
-      for (int j = 0; j < 8; ++j)
-        if (j < k_left) e[j] = src[j];
-    }
+    for (int j = 0; j < 8; ++j)
+      if (ok && k + j < K) e[j] = row[k + j];
+    *reinterpret_cast<uint4*>(dst) = u;
   }
-  *reinterpret_cast<uint4*>(dst) = u;
 }
 
 template <bool VEC>
 __global__ void __launch_bounds__(128)
 head_gemm_bf16_kernel(const HeadGemm g) {
-  __shared__ __align__(16) __nv_bfloat16 sa[HG_M * HG_LD], sb[HG_N * HG_LD];
+  extern __shared__ __align__(16) __nv_bfloat16 hg_smem[];
   const int h = blockIdx.z, m0 = blockIdx.y * HG_M, n0 = blockIdx.x * HG_N;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int wm = (warp & 1) * 32, wn = (warp >> 1) * 32;
@@ -171,32 +190,46 @@ head_gemm_bf16_kernel(const HeadGemm g) {
     arow[i] = m < g.M ? A + (g.a_rows != nullptr ? g.a_rows[m] : m) * g.lda : nullptr;
     brow[i] = n < g.N ? B + static_cast<long long>(n) * g.ldb : nullptr;
   }
-  for (int k0 = 0; k0 < g.K; k0 += HG_K) {
+  const int steps = (g.K + HG_K - 1) / HG_K;
+  auto load = [&](int step) {
+    __nv_bfloat16* sa = hg_smem + (step % HG_STAGES) * (HG_M + HG_N) * HG_LD;
+    if (step < steps) {
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      const int off = (lr + 16 * i) * HG_LD + lc;
-      hg_load<VEC>(sa + off, arow[i] + k0 + lc, arow[i] != nullptr && k0 + lc < g.K, g.K - k0 - lc);
-      hg_load<VEC>(sb + off, brow[i] + k0 + lc, brow[i] != nullptr && k0 + lc < g.K, g.K - k0 - lc);
+      for (int i = 0; i < 4; ++i) {
+        const int off = (lr + 16 * i) * HG_LD + lc;
+        hg_load<VEC>(sa + off, arow[i], step * HG_K + lc, g.K, g.A);
+        hg_load<VEC>(sa + HG_M * HG_LD + off, brow[i], step * HG_K + lc, g.K, g.A);
+      }
     }
-    __syncthreads();
+    cp_async_commit();           // one group per step, empty behind the last
+  };
+#pragma unroll
+  for (int i = 0; i < HG_STAGES - 1; ++i) load(i);
+  for (int step = 0; step < steps; ++step) {
+    cp_async_wait<HG_STAGES - 2>();
+    __syncthreads();             // this step's tiles have landed, and everyone is done with the previous step's
+    load(step + HG_STAGES - 1);
+    const __nv_bfloat16* sa = hg_smem + (step % HG_STAGES) * (HG_M + HG_N) * HG_LD;
+    const __nv_bfloat16* sb = sa + HG_M * HG_LD;
 #pragma unroll
     for (int k = 0; k < HG_K; k += 16) {
       uint32_t a[2][4], b[2][4];
 #pragma unroll
       for (int i = 0; i < 2; ++i) {
-        ldmatrix_x4(a[i], smem_u32(sa + (wm + i * 16 + (lane & 15)) * HG_LD + k + (lane >> 4) * 8));
-        // two 8-column blocks of B: registers 0, 1 belong to the first, 2, 3 to the second
-        ldmatrix_x4(b[i], smem_u32(sb + (wn + i * 16 + (lane >> 4) * 8 + (lane & 7)) * HG_LD + k + ((lane >> 3) & 1) * 8));
+        ldmatrix_x4(a[i], smem_u32(sa + (wm + i * 16) * HG_LD + k + frag_a(lane, HG_LD)));
+        ldmatrix_x4(b[i], smem_u32(sb + (wn + i * 16) * HG_LD + k + frag_b(lane, HG_LD)));
       }
 #pragma unroll
       for (int i = 0; i < 2; ++i)
 #pragma unroll
         for (int j = 0; j < 4; ++j) mma_bf16(acc[i][j], a[i], b[j >> 1][(j & 1) * 2], b[j >> 1][(j & 1) * 2 + 1]);
     }
-    __syncthreads();
   }
   __nv_bfloat16* C = reinterpret_cast<__nv_bfloat16*>(g.C) + static_cast<long long>(h) * g.c_hs;
   const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(g.gate);
+  // column pairs as one 4-byte access when every row starts on one
+  const bool pairs = ((g.N | g.ldc | g.c_hs | g.ldg | g.g_hs) & 1) == 0 &&
+                     ((reinterpret_cast<uintptr_t>(g.C) | reinterpret_cast<uintptr_t>(g.gate)) & 3) == 0;
 #pragma unroll
   for (int i = 0; i < 2; ++i)
 #pragma unroll
@@ -204,15 +237,26 @@ head_gemm_bf16_kernel(const HeadGemm g) {
       const int m = m0 + wm + i * 16 + half * 8 + (lane >> 2);
       if (m >= g.M) continue;
       const long long r = g.c_rows != nullptr ? g.c_rows[m] : m;
+      const __nv_bfloat16* grow = gate + r * g.ldg + static_cast<long long>(h) * g.g_hs;
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int n = n0 + wn + j * 8 + (lane & 3) * 2 + e;
-          if (n >= g.N) continue;
-          float v = acc[i][j][half * 2 + e];
-          if (gate != nullptr) v *= sigmoid_f(ld1(gate + r * g.ldg + static_cast<long long>(h) * g.g_hs + n));
-          C[r * g.ldc + n] = __float2bfloat16_rn(v);
+        const int n = n0 + wn + j * 8 + (lane & 3) * 2;
+        if (n >= g.N) continue;
+        float2 v = make_float2(acc[i][j][half * 2], acc[i][j][half * 2 + 1]);
+        if (pairs) {
+          if (gate != nullptr) {
+            const float2 s = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(grow + n));
+            v.x *= sigmoid_t<__nv_bfloat16>(s.x);
+            v.y *= sigmoid_t<__nv_bfloat16>(s.y);
+          }
+          *reinterpret_cast<uint32_t*>(C + r * g.ldc + n) = pack_bf16x2(v.x, v.y);
+        } else {
+          if (gate != nullptr) {
+            v.x *= sigmoid_t<__nv_bfloat16>(ld1(grow + n));
+            if (n + 1 < g.N) v.y *= sigmoid_t<__nv_bfloat16>(ld1(grow + n + 1));
+          }
+          st1(C + r * g.ldc + n, v.x);
+          if (n + 1 < g.N) st1(C + r * g.ldc + n + 1, v.y);
         }
       }
     }
@@ -311,17 +355,22 @@ latent_attn_kernel(const T* __restrict__ qa, const T* __restrict__ cache, const 
   }
 }
 
+constexpr int LG_ROWS = 16;      // rows per CTA
+
 __global__ void __launch_bounds__(256)
 latent_gather_kernel(const uint4* __restrict__ cache, uint4* __restrict__ dst, const int* __restrict__ seqs,
                      const int* __restrict__ cu, const int* __restrict__ block_table, int max_blocks, int page,
                      int row_vec) {
   const int b = blockIdx.y;
-  const int n = cu[b + 1] - cu[b], first = blockIdx.x * page;
+  const int n = cu[b + 1] - cu[b], first = blockIdx.x * LG_ROWS;
   if (first >= n) return;
-  const int rows = min(page, n - first);
-  const long long src = static_cast<long long>(block_table[static_cast<long long>(seqs[b]) * max_blocks + blockIdx.x]) * page * row_vec;
-  const long long to = (static_cast<long long>(cu[b]) + first) * row_vec;
-  for (int i = threadIdx.x; i < rows * row_vec; i += blockDim.x) dst[to + i] = cache[src + i];
+  const int* table = block_table + static_cast<long long>(seqs[b]) * max_blocks;
+  const int items = min(LG_ROWS, n - first) * row_vec;
+  for (int i = threadIdx.x; i < items; i += blockDim.x) {
+    const int r = i / row_vec, v = i - r * row_vec, j = first + r;
+    dst[(static_cast<long long>(cu[b]) + j) * row_vec + v] =
+        cache[(static_cast<long long>(table[j / page]) * page + j % page) * row_vec + v];
+  }
 }
 
 static int check_launch(const char* what) {
@@ -347,32 +396,50 @@ extern "C" int tw_latent_prep(const void* p, long long ldp, int q_off, int q_ran
   }
   const bool vec = ldp % 8 == 0 && q_off % 8 == 0 && kv_off % 8 == 0 && ldcq % 8 == 0 && aligned16(p) && aligned16(cq) &&
                    aligned16(wq) && aligned16(wkv);
-  const int n = q_rank > kv_rank ? q_rank : kv_rank;
-  int threads = ((n + 7) / 8 + 31) / 32 * 32;
-  if (threads > 256) threads = 256;
-#define TW_GO(TT, V)                                                                                                   \
-  latent_prep_kernel<TT, V><<<T, threads, 0, stream>>>(                                                                \
+  const int groups = (q_rank + 7) / 8 + (kv_rank + 7) / 8;
+  const int threads = groups >= 256 ? 256 : (groups + 31) / 32 * 32;
+  const int vpt = (groups + threads - 1) / threads;
+#define TW_PREP(TT, V, N)                                                                                              \
+  latent_prep_kernel<TT, V, N><<<T, threads, 0, stream>>>(                                                             \
       reinterpret_cast<const TT*>(p), ldp, q_off, q_rank, reinterpret_cast<const TT*>(wq), reinterpret_cast<TT*>(cq), \
       ldcq, kv_off, kv_rank, reinterpret_cast<const TT*>(wkv), rot, rot_dims, cos_sin, positions, slots,               \
       reinterpret_cast<TT*>(cache), row, eps)
+#define TW_GO(TT, V)                       \
+  do {                                     \
+    if (vpt <= 1) TW_PREP(TT, V, 1);       \
+    else if (vpt <= 2) TW_PREP(TT, V, 2);  \
+    else if (vpt <= 4) TW_PREP(TT, V, 4);  \
+    else TW_PREP(TT, V, 8);                \
+  } while (0)
+  if (vpt > 8) {
+    set_last_error("latent_prep: latents of %d and %d elements are too long", q_rank, kv_rank);
+    return 1;
+  }
   if (dtype == TW_BF16) {
     if (vec) TW_GO(__nv_bfloat16, true); else TW_GO(__nv_bfloat16, false);
   } else {
     if (vec) TW_GO(float, true); else TW_GO(float, false);
   }
 #undef TW_GO
+#undef TW_PREP
   return check_launch("latent_prep");
 }
 
 extern "C" int tw_rope_tail(void* q, long long ldq, int T, int heads, int head_stride, int off, int rot_dims,
                             const float* cos_sin, const int* positions, int dtype, cudaStream_t stream) {
   if (T <= 0 || rot_dims <= 0) return 0;
-  if (dtype == TW_BF16)
-    rope_tail_kernel<__nv_bfloat16><<<T, 256, 0, stream>>>(reinterpret_cast<__nv_bfloat16*>(q), ldq, heads, head_stride,
-                                                           off, rot_dims, cos_sin, positions);
-  else
-    rope_tail_kernel<float><<<T, 256, 0, stream>>>(reinterpret_cast<float*>(q), ldq, heads, head_stride, off, rot_dims,
-                                                   cos_sin, positions);
+  const bool vec = rot_dims % 16 == 0 && head_stride % 8 == 0 && off % 8 == 0 && ldq % 8 == 0 && aligned16(q) && aligned16(cos_sin);
+  const int items = heads * (rot_dims / 2) / (vec ? 8 : 1);
+  const int threads = items >= 256 ? 256 : (items + 31) / 32 * 32;
+#define TW_GO(TT, V)                                                                                               \
+  rope_tail_kernel<TT, V><<<T, threads, 0, stream>>>(reinterpret_cast<TT*>(q), ldq, heads, head_stride, off, rot_dims, \
+                                                     cos_sin, positions)
+  if (dtype == TW_BF16) {
+    if (vec) TW_GO(__nv_bfloat16, true); else TW_GO(__nv_bfloat16, false);
+  } else {
+    if (vec) TW_GO(float, true); else TW_GO(float, false);
+  }
+#undef TW_GO
   return check_launch("rope_tail");
 }
 
@@ -404,8 +471,21 @@ extern "C" int tw_head_gemm(const void* A, long long lda, int a_hs, const int* a
   if (dtype == TW_BF16) {
     const bool vec = K % 8 == 0 && lda % 8 == 0 && a_hs % 8 == 0 && b_hs % 8 == 0 && ldb % 8 == 0 && aligned16(A) &&
                      aligned16(B);
-    if (vec) head_gemm_bf16_kernel<true><<<grid, 128, 0, stream>>>(g);
-    else head_gemm_bf16_kernel<false><<<grid, 128, 0, stream>>>(g);
+    static thread_local int configured_dev = -1;
+    int dev = 0;
+    cudaGetDevice(&dev);
+    if (configured_dev != dev) {
+      cudaError_t e = cudaFuncSetAttribute(head_gemm_bf16_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, HG_SMEM);
+      if (e == cudaSuccess)
+        e = cudaFuncSetAttribute(head_gemm_bf16_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, HG_SMEM);
+      if (e != cudaSuccess) {
+        set_last_error("head_gemm: cudaFuncSetAttribute failed: %s", cudaGetErrorString(e));
+        return 1;
+      }
+      configured_dev = dev;
+    }
+    if (vec) head_gemm_bf16_kernel<true><<<grid, 128, HG_SMEM, stream>>>(g);
+    else head_gemm_bf16_kernel<false><<<grid, 128, HG_SMEM, stream>>>(g);
   } else {
     head_gemm_f32_kernel<<<grid, 256, 0, stream>>>(g);
   }
@@ -450,7 +530,7 @@ extern "C" int tw_latent_gather(const void* cache, void* dst, const int* seqs, c
     set_last_error("latent_gather: rows of %d bytes are not a multiple of 16", row_bytes);
     return 1;
   }
-  const dim3 grid((max_rows + page - 1) / page, n_seqs);
+  const dim3 grid((max_rows + LG_ROWS - 1) / LG_ROWS, n_seqs);
   latent_gather_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<const uint4*>(cache), reinterpret_cast<uint4*>(dst),
                                                  seqs, cu, block_table, max_blocks, page, row_bytes / 16);
   return check_launch("latent_gather");

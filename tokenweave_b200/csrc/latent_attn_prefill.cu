@@ -414,7 +414,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                 float s[8];
                 ld8(grow + col0 + q8 * 8, s);
 #pragma unroll
-                for (int i = 0; i < 8; ++i) v[i] *= sigmoid_f(s[i]);
+                for (int i = 0; i < 8; ++i) v[i] *= sigmoid_t<__nv_bfloat16>(s[i]);
               }
               st8(orow + col0 + q8 * 8, v);
             }

@@ -145,7 +145,7 @@ gated_group_norm_kernel(const T* __restrict__ y, long long ldy, const T* __restr
       ld8n<VEC>(z + t * ldz + c0 + i, part - i, g);
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        v[k][j] *= silu_f(g[j]);
+        v[k][j] *= silu_t<T>(g[j]);
         ss[0] += v[k][j] * v[k][j];
       }
     }

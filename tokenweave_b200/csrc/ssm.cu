@@ -62,25 +62,35 @@ causal_conv_kernel(const ConvArgs a) {
     ld8n<VEC>(reinterpret_cast<const T*>(a.w) + static_cast<long long>(k) * a.channels + c, a.channels - c, w[k]);
   ld8n<VEC>(reinterpret_cast<const T*>(a.bias) + c, a.channels - c, bias);
   float hist[TAPS > 1 ? TAPS - 1 : 1][8];        // hist[k]: the input k + 1 tokens back
-  int seq = -1;
-  const int t_end = min(a.T, static_cast<int>(blockIdx.y + 1) * CONV_STRIP);
-  for (int t = blockIdx.y * CONV_STRIP; t < t_end; ++t) {
-    const int b = a.row_seq[t];
-    if (b != seq) {
-      seq = b;
+  const int t0 = blockIdx.y * CONV_STRIP, t_end = min(a.T, t0 + CONV_STRIP);
+  // all rows of the strip are requested before the first is used
+  float x[CONV_STRIP][8];
+  int seqs[CONV_STRIP];
 #pragma unroll
-      for (int k = 0; k < TAPS - 1; ++k) conv_input<T, VEC>(a, b, t, k + 1, c, hist[k]);
+  for (int i = 0; i < CONV_STRIP; ++i) {
+    const int t = min(t0 + i, t_end - 1);
+    ld8n<VEC>(reinterpret_cast<const T*>(a.x) + t * a.ldx + c, a.channels - c, x[i]);
+    seqs[i] = a.row_seq[t];
+  }
+#pragma unroll
+  for (int k = 0; k < TAPS - 1; ++k) conv_input<T, VEC>(a, seqs[0], t0, k + 1, c, hist[k]);
+#pragma unroll
+  for (int i = 0; i < CONV_STRIP; ++i) {
+    const int t = t0 + i;
+    if (t >= t_end) break;
+    if (i > 0 && seqs[i] != seqs[i - 1]) {
+#pragma unroll
+      for (int k = 0; k < TAPS - 1; ++k) conv_input<T, VEC>(a, seqs[i], t, k + 1, c, hist[k]);
     }
-    float x[8], y[8];
-    ld8n<VEC>(reinterpret_cast<const T*>(a.x) + t * a.ldx + c, a.channels - c, x);
+    float y[8];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) y[j] = fmaf(x[j], w[TAPS - 1][j], bias[j]);
+    for (int j = 0; j < 8; ++j) y[j] = fmaf(x[i][j], w[TAPS - 1][j], bias[j]);
 #pragma unroll
     for (int k = 0; k < TAPS - 1; ++k)
 #pragma unroll
       for (int j = 0; j < 8; ++j) y[j] = fmaf(hist[k][j], w[TAPS - 2 - k][j], y[j]);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) y[j] = silu_f(y[j]);
+    for (int j = 0; j < 8; ++j) y[j] = silu_t<T>(y[j]);
     st8n<VEC>(reinterpret_cast<T*>(a.out) + t * a.ldo + c, a.channels - c, y);
 #pragma unroll
     for (int k = TAPS - 2; k > 0; --k)
@@ -88,7 +98,7 @@ causal_conv_kernel(const ConvArgs a) {
       for (int j = 0; j < 8; ++j) hist[k][j] = hist[k - 1][j];
     if (TAPS > 1) {
 #pragma unroll
-      for (int j = 0; j < 8; ++j) hist[0][j] = x[j];
+      for (int j = 0; j < 8; ++j) hist[0][j] = x[i][j];
     }
   }
 }
@@ -129,7 +139,7 @@ causal_conv_step_kernel(const ConvArgs a) {
     for (int j = 0; j < 8; ++j) y[j] = fmaf(h[k][j], w[j], y[j]);
   }
 #pragma unroll
-  for (int j = 0; j < 8; ++j) y[j] = silu_f(y[j]);
+  for (int j = 0; j < 8; ++j) y[j] = silu_t<T>(y[j]);
   st8n<VEC>(reinterpret_cast<T*>(a.out) + t * a.ldo + c, a.channels - c, y);
   T* st = reinterpret_cast<T*>(a.state) + static_cast<long long>(a.slots[b]) * (TAPS - 1) * a.channels + c;
 #pragma unroll

@@ -63,6 +63,18 @@ __device__ __forceinline__ void st8n(T* p, int n, const float (&v)[8]) {
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// Activations of bf16 tensors: the result is rounded to 8 bits of mantissa, the hardware exponential and division
+// (__expf, __fdividef) are exact enough; fp32 tensors take the functions above.
+template <typename T>
+__device__ __forceinline__ float silu_t(float x) {
+  if (sizeof(T) == 2) return __fdividef(x, 1.f + __expf(-x));
+  return silu_f(x);
+}
+template <typename T>
+__device__ __forceinline__ float sigmoid_t(float x) {
+  if (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-x));
+  return sigmoid_f(x);
+}
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 }  // namespace tw
