@@ -125,6 +125,7 @@ def test_latent_prep_and_absorb(dtype, q_rank, kv_rank, rot, rot_dims):
 
 @pytest.mark.parametrize("kernel,dtype", [("simt", torch.float32), ("simt", torch.bfloat16), ("tc", torch.bfloat16)])
 @pytest.mark.parametrize("heads,kv_rank,rot,page", [(3, 40, 16, 8), (16, 128, 32, 64), (20, 200, 24, 32), (40, 512, 64, 128),
+                                                    (12, 512, 64, 32), (32, 448, 40, 64),
                                                     (5, 64, 64, 128)])
 def test_latent_attention(kernel, dtype, heads, kv_rank, rot, page):
     lens = [1, 7, page, page + 1, 127, 128, 129, 400, 1500]

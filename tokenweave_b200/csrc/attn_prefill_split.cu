@@ -352,7 +352,7 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         auto exp_chunk = [&](const uint32_t (&buf)[32]) {
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
-            const float2 x = ffma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc2, nm2);
+            const float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc2, nm2);
             const float2 e = make_float2(fast_exp2(x.x), fast_exp2(x.y));
             sum2[i & 1] = fadd2(sum2[i & 1], e);
             pk[i] = pack_bf16x2(e.x, e.y);

@@ -2,31 +2,33 @@
 // cache rows, [latent | rotated key part], and the values are the latent part of the rows themselves.
 //
 // A tile of 128 cache rows is fetched once and used twice:
-//     S^T [128 keys x heads]   = K Q^T      A = the tile, K-major; B = the absorbed queries, 16 or 32 heads
+//     S^T [keys x heads]       = K Q^T      A = the tile, K-major; B = the absorbed queries, 16 or 32 heads
 //     O^T [latent x heads]    += C^T P^T    A = the same tile read MN-major, 128 latent columns per MMA block
 // so M is always full although a token has few query rows, and the kernel is bound by the cache bytes: the tile's
 // columns travel as pairs of 64-column chunks with a barrier each, the score product starts with the first pair and a
-// pair is refilled as soon as its part of O^T is done. Rows of up to 640 elements, latents of up to 512. The keys of a
+// pair is refilled as soon as its part of O^T is done; the next tile travels to L2 meanwhile, since wide rows leave
+// room for one tile in shared memory (two tiles of 64 keys were 40 % slower: an MMA of this shape takes about 60 cycles
+// whether it has 64 or 128 rows). Rows of up to 640 elements, latents of up to 512. The keys of a
 // row can be cut into splits, whose fp32 partial results a second kernel merges.
 //
 // Roles (192 threads): warp 0 TMA producer, warp 1 MMA issuer, warps 2..5 softmax (one thread per key of the tile),
 // rescaling and epilogue (one thread per latent column). Waits are bounded; after a timeout the roles keep their trip
 // counts, report TW_ERR_MBAR_TIMEOUT and leave through the tear-down.
-#include "tw_common.cuh"
+#include "tw_elect.cuh"
 #include "tw_host.h"
 #include "tw_kernels.h"
 
 namespace tw {
 
-constexpr int LD_BN = 128;                    // keys per tile
+constexpr int LD_BN = 128;                       // keys per tile
 constexpr int LD_THREADS = 192;
-constexpr int LD_CHUNK = LD_BN * 128;         // 64 columns of a tile
 constexpr int LD_MAX_PAIRS = 5, LD_MAX_STAGES = 4;
 constexpr int LD_SMEM_LIMIT = 227 * 1024;
 
 struct LatentDecodeParams {
   const __nv_bfloat16* q;        // [n, heads, row]
   __nv_bfloat16* out;            // [n, heads, kv_rank]
+  const __nv_bfloat16* cache;    // [blocks, page, row]
   const int *tok_seq, *tok_kvlen, *block_table;
   int max_blocks, page, heads, row, kv_rank, splits, chunks, stages;
   float scale_log2;
@@ -53,18 +55,21 @@ __host__ __device__ constexpr int ld_fixed_bytes(int chunks) {
 
 template <int NC>
 __global__ void __launch_bounds__(LD_THREADS, 1)
-latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecodeParams p) {
+latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmQ,
+                     const LatentDecodeParams p) {
   constexpr uint32_t IDESC_S = make_idesc_bf16(LD_BN, NC, 0, 0);     // A = rows (K-major), B = Q (K-major)
   constexpr uint32_t IDESC_O = make_idesc_bf16(128, NC, 1, 0);       // A = latent columns (MN-major), B = P (K-major)
   constexpr uint32_t TMEM_COLS = NC == 16 ? 128 : 256;               // 2 NC for S, 4 NC for O
   constexpr uint32_t COL_O = 2 * NC;
+
+  constexpr int CHUNK = LD_BN * 128;                                    // 64 columns of a tile
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
   const int pairs = (p.chunks + 1) >> 1;
   const int v_chunks = (p.kv_rank + 63) >> 6, v_pairs = (v_chunks + 1) >> 1;
-  const int tile_bytes = pairs * 2 * LD_CHUNK;
+  const int tile_bytes = pairs * 2 * CHUNK;
   uint8_t* s_q = smem + p.stages * tile_bytes;
   uint8_t* s_p = s_q + p.chunks * NC * 128;
   uint64_t* bars = reinterpret_cast<uint64_t*>(s_p + 2 * NC * 128);
@@ -98,7 +103,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     mbar_init(&s_full[1], 1);
     mbar_init(p_ready, 128);
     mbar_init(o_done, 1);
-    mbar_init(q_ready, 128);
+    mbar_init(q_ready, 1);
     *abort_flag = 0;
     mbar_fence_init();
   }
@@ -112,81 +117,127 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
   const uint32_t tmem_base = *tmem_slot;
 
   if (warp == 0) {
-    // ---------------- TMA producer ----------------
-    if (lane == 0 && n_tiles > 0) {
-      tma_prefetch_desc(&tmC);
-      const int pages_per_tile = LD_BN / p.page;
+    // ---------------- TMA producer (uniform over the warp, see the issuer) ----------------
+    if (n_tiles > 0) {
+      // The queries: NC rows from the token's first head on. Rows behind the block's last head are another token's or
+      // zeros; their columns of S and O are not used.
+      mbar_expect_tx_e(q_ready, p.chunks * NC * 128);
+      for (int c = 0; c < p.chunks; ++c) tma_load_2d_e(s_q + c * NC * 128, &tmQ, q_ready, c * 64, tok * p.heads + h0);
+      // a tile is several pages, or a page several tiles; a piece (rows of one page) is contiguous in memory
+      const int piece = min(p.page, LD_BN), pieces = LD_BN / piece;
       const int last_page = (kv_len - 1) / p.page;
       const int* table = p.block_table + static_cast<long long>(seq) * p.max_blocks;
+      const uint32_t piece_bytes = piece * p.row * 2;
+      // A tile's copies are issued when its buffer is free; by then its bytes should not be in DRAM any more.
+      auto prefetch = [&](int j) {
+        if (j >= n_tiles || lane >= pieces) return;
+        const int key = (t_begin + j) * LD_BN + lane * piece;
+        if (key >= kv_len) return;
+        const __nv_bfloat16* src =
+            p.cache + (static_cast<long long>(table[key / p.page]) * p.page + key % p.page) * p.row;
+        asm volatile("cp.async.bulk.prefetch.L2.global [%0], %1;" ::"l"(src), "r"(piece_bytes) : "memory");
+      };
+      for (int j = 0; j < p.stages; ++j) prefetch(j);
       bool ok = true;
       for (int j = 0; ok && j < n_tiles; ++j) {
         const int st = j % p.stages;
         const uint32_t ph = (j / p.stages) & 1;
+        const int key0 = (t_begin + j) * LD_BN;
+        // page ids of the tile's pieces, one per lane
+        const int block = table[min((key0 + (lane & (pieces - 1)) * piece) / p.page, last_page)];
         uint8_t* tile = smem + st * tile_bytes;
         for (int pr = 0; pr < pairs; ++pr) {
           if (!mbar_wait(&empty[st * LD_MAX_PAIRS + pr], ph ^ 1)) { ok = false; break; }
           uint64_t* bar = &full[st * LD_MAX_PAIRS + pr];
-          const int c_end = min(p.chunks, 2 * pr + 2);
-          mbar_expect_tx(bar, (c_end - 2 * pr) * LD_CHUNK);
-          for (int pg = 0; pg < pages_per_tile; ++pg) {
-            const int block = table[min((t_begin + j) * pages_per_tile + pg, last_page)];
-            for (int c = 2 * pr; c < c_end; ++c)
-              tma_load_3d(tile + c * LD_CHUNK + pg * p.page * 128, &tmC, bar, c * 64, 0, block);
+          const bool two = 2 * pr + 1 < p.chunks;
+          mbar_expect_tx_e(bar, (two ? 2 : 1) * CHUNK);
+          for (int pc = 0; pc < pieces; ++pc) {
+            const int blk = __shfl_sync(0xffffffffu, block, pc), y = (key0 + pc * piece) % p.page;
+            uint8_t* dst = tile + pr * 2 * CHUNK + pc * piece * 128;
+            tma_load_3d_e(dst, &tmC, bar, pr * 128, y, blk);
+            if (two) tma_load_3d_e(dst + CHUNK, &tmC, bar, pr * 128 + 64, y, blk);
           }
         }
+        prefetch(j + p.stages);
       }
-      if (!ok) {
+      if (!ok && lane == 0) {
         report_error(p.status, TW_ERR_MBAR_TIMEOUT);
         *abort_flag = 1;
       }
     }
   } else if (warp == 1) {
     // ---------------- MMA issuer ----------------
-    if (lane == 0 && n_tiles > 0) {
-      const uint32_t q_addr = smem_u32(s_q), p_addr = smem_u32(s_p);
+    // The whole warp walks through the loops and one elected lane issues: everything a descriptor is made of stays
+    // uniform over the warp.
+    if (n_tiles > 0) {
+      const uint64_t desc_tile = make_smem_desc_sw128(smem_u32(smem), 16, 1024);          // K-major: scores
+      const uint64_t desc_v = make_smem_desc_sw128(smem_u32(smem), CHUNK, 1024);          // MN-major: latent columns
+      const uint64_t desc_q = make_smem_desc_sw128(smem_u32(s_q), 16, 1024);
+      const uint64_t desc_p = make_smem_desc_sw128(smem_u32(s_p), 16, 1024);
       bool ok = mbar_wait(q_ready, 0);
       auto issue_s = [&](int j) {
         const int st = j % p.stages;
         const uint32_t ph = (j / p.stages) & 1;
-        const uint32_t tile = smem_u32(smem + st * tile_bytes);
+        const uint32_t tile_off = st * tile_bytes;
+        const uint32_t d = tmem_base + (j & 1) * NC;
         for (int pr = 0; pr < pairs; ++pr) {
           if (!mbar_wait(&full[st * LD_MAX_PAIRS + pr], ph)) return false;
           tc_fence_after_sync();
-          const int c_end = min(p.chunks, 2 * pr + 2);
-          for (int c = 2 * pr; c < c_end; ++c) {
+          // descriptors hold addresses in units of 16 bytes in their low bits: one addition each per instruction
+          const uint64_t da = desc_tile + (tile_off + pr * 2 * CHUNK) / 16, db = desc_q + pr * (2 * NC * 128 / 16);
+#pragma unroll
+          for (int k = 0; k < 4; ++k) umma_ss_e(d, da + k * 2, db + k * 2, IDESC_S, (pr | k) != 0 ? 1u : 0u);
+          if (2 * pr + 1 < p.chunks) {
 #pragma unroll
             for (int k = 0; k < 4; ++k)
-              umma_ss(tmem_base + (j & 1) * NC, make_smem_desc_sw128(tile + c * LD_CHUNK + k * 32, 16, 1024),
-                      make_smem_desc_sw128(q_addr + c * (NC * 128) + k * 32, 16, 1024), IDESC_S, (c | k) != 0 ? 1u : 0u);
+              umma_ss_e(d, da + CHUNK / 16 + k * 2, db + NC * 128 / 16 + k * 2, IDESC_S, 1u);
           }
-          if (pr >= v_pairs) umma_commit(&empty[st * LD_MAX_PAIRS + pr]);     // no latent column in this pair
+          if (pr >= v_pairs) umma_commit_e(&empty[st * LD_MAX_PAIRS + pr]);     // no latent column in this pair
         }
-        umma_commit(&s_full[j & 1]);
+        umma_commit_e(&s_full[j & 1]);
+        return true;
+      };
+      auto tile_here = [&](int j) {
+        const uint32_t ph = (j / p.stages) & 1;
+        for (int pr = 0; pr < pairs; ++pr)
+          if (!mbar_test(&full[(j % p.stages) * LD_MAX_PAIRS + pr], ph)) return false;
         return true;
       };
       if (ok) ok = issue_s(0);
       for (int j = 0; ok && j < n_tiles; ++j) {
-        // with one tile buffer the next score product has to follow this tile's last use
-        if (p.stages > 1 && j + 1 < n_tiles) {
-          ok = issue_s(j + 1);
-          if (!ok) break;
+        // The next tile's score product goes first if its rows have landed before this tile's probabilities are there;
+        // otherwise this tile's products go first, because they free the buffer that the load after the next waits for.
+        bool ahead = j + 1 >= n_tiles;
+        bool have_p = false;
+        const uint64_t t_start = globaltimer_ns();
+        while (!have_p) {
+#pragma unroll 1
+          for (int i = 0; i < 64 && !have_p; ++i) {
+            if (!ahead && p.stages > 1 && tile_here(j + 1)) {
+              ok = issue_s(j + 1);
+              if (!ok) break;
+              ahead = true;
+            }
+            have_p = ahead || p.stages == 1 ? mbar_try_wait(p_ready, j & 1) : mbar_test(p_ready, j & 1);
+          }
+          if (!ok || (!have_p && globaltimer_ns() - t_start > TW_WAIT_BUDGET_NS)) { ok = false; break; }
         }
-        if (!mbar_wait(p_ready, j & 1)) { ok = false; break; }
+        if (!ok) break;
         tc_fence_after_sync();
         const int st = j % p.stages;
-        const uint32_t tile = smem_u32(smem + st * tile_bytes);
         for (int m = 0; m < v_pairs; ++m) {
+          const uint64_t da = desc_v + (st * tile_bytes + m * 2 * CHUNK) / 16;
+          const uint32_t d = tmem_base + COL_O + m * NC;
 #pragma unroll
           for (int k = 0; k < LD_BN / 16; ++k)
-            umma_ss(tmem_base + COL_O + m * NC, make_smem_desc_sw128(tile + m * 2 * LD_CHUNK + k * 16 * 128, LD_CHUNK, 1024),
-                    make_smem_desc_sw128(p_addr + (k >> 2) * (NC * 128) + (k & 3) * 32, 16, 1024), IDESC_O,
+            umma_ss_e(d, da + k * (16 * 128 / 16), desc_p + ((k >> 2) * (NC * 128) + (k & 3) * 32) / 16, IDESC_O,
                     (j | k) != 0 ? 1u : 0u);
-          umma_commit(&empty[st * LD_MAX_PAIRS + m]);
+          umma_commit_e(&empty[st * LD_MAX_PAIRS + m]);
         }
-        umma_commit(o_done);
-        if (p.stages == 1 && j + 1 < n_tiles) ok = issue_s(j + 1);
+        umma_commit_e(o_done);
+        if (!ahead) ok = issue_s(j + 1);
       }
-      if (!ok) {
+      if (!ok && lane == 0) {
         report_error(p.status, TW_ERR_MBAR_TIMEOUT);
         *abort_flag = 1;
       }
@@ -198,17 +249,6 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     const int sw = warp - 2;
     const int t = threadIdx.x - 64;          // 0..127
     const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(qr * 32) << 16);
-
-    // queries into the swizzled K-major operand layout, zeros behind the row's end and behind the last head
-    for (int i = t; i < NC * p.chunks * 8; i += 128) {
-      const int g = i / (p.chunks * 8), cidx = i - g * (p.chunks * 8);
-      uint4 v = make_uint4(0u, 0u, 0u, 0u);
-      if (g < G && cidx * 8 < p.row)
-        v = *reinterpret_cast<const uint4*>(p.q + (static_cast<long long>(tok) * p.heads + h0 + g) * p.row + cidx * 8);
-      *reinterpret_cast<uint4*>(s_q + (cidx >> 3) * (NC * 128) + g * 128 + (((cidx & 7) ^ (g & 7)) * 16)) = v;
-    }
-    fence_proxy_async_smem();
-    mbar_arrive(q_ready);
 
     float m_ref[NC], l_part[NC];
 #pragma unroll
@@ -225,7 +265,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
       tmem_ld_cols(t_lane + (j & 1) * NC, sv);
       tmem_wait_ld();
       float* xm = xchg + (j & 1) * 4 * NC;
-      if ((t_begin + j + 1) * LD_BN > kv_len && (t_begin + j) * LD_BN + r >= kv_len) {
+      if ((t_begin + j) * LD_BN + r >= kv_len) {
 #pragma unroll
         for (int g = 0; g < NC; ++g) sv[g] = __float_as_uint(-INFINITY);
       }
@@ -312,36 +352,64 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const LatentDecode
     }
     ld_softmax_sync();
     if (n_tiles > 0 && ok) ok = mbar_wait(o_done, (n_tiles - 1) & 1);
-    if (ok) {
-      tc_fence_after_sync();
+    tc_fence_after_sync();
+    if (p.splits == 1) {
+      // O^T to [head][latent] through the tile buffers (nothing is in flight any more), then whole rows to memory
+      __nv_bfloat16* s_o = reinterpret_cast<__nv_bfloat16*>(smem);
+      const int ld_o = v_pairs * 128 + 8;
+      float inv[NC];
+#pragma unroll
+      for (int g = 0; g < NC; ++g) {
+        const float l = (xs[g] + xs[NC + g]) + (xs[2 * NC + g] + xs[3 * NC + g]);
+        inv[g] = l > 0.f ? __fdividef(1.f, l) : 0.f;
+      }
 #pragma unroll 1
       for (int m = 0; m < v_pairs; ++m) {
         uint32_t ov[NC];
-        if (n_tiles > 0) {
-          tmem_ld_cols(t_lane + COL_O + m * NC, ov);
-          tmem_wait_ld();
+        tmem_ld_cols(t_lane + COL_O + m * NC, ov);
+        tmem_wait_ld();
+#pragma unroll
+        for (int g = 0; g < NC; ++g)
+          s_o[g * ld_o + m * 128 + r] = __float2bfloat16(n_tiles > 0 ? __uint_as_float(ov[g]) * inv[g] : 0.f);
+      }
+      ld_softmax_sync();
+      if (ok) {
+        const long long first = (static_cast<long long>(tok) * p.heads + h0) * p.kv_rank;
+        if (p.kv_rank % 8 == 0) {
+          const int per = p.kv_rank >> 3;
+          for (int i = t; i < G * per; i += 128) {
+            const int g = i / per, v = i - g * per;
+            *reinterpret_cast<uint4*>(p.out + first + static_cast<long long>(i) * 8) =
+                *reinterpret_cast<const uint4*>(s_o + g * ld_o + v * 8);
+          }
+        } else {
+          for (int i = t; i < G * p.kv_rank; i += 128) {
+            const int g = i / p.kv_rank;
+            p.out[first + i] = s_o[g * ld_o + i - g * p.kv_rank];
+          }
         }
+      }
+    } else if (ok) {
+#pragma unroll 1
+      for (int m = 0; m < v_pairs; ++m) {
+        uint32_t ov[NC];
+        tmem_ld_cols(t_lane + COL_O + m * NC, ov);
+        tmem_wait_ld();
         const int d = m * 128 + r;
 #pragma unroll
         for (int g = 0; g < NC; ++g) {
           if (g < G && d < p.kv_rank) {
-            const float o = n_tiles > 0 ? __uint_as_float(ov[g]) : 0.f;
-            const float l = (xs[g] + xs[NC + g]) + (xs[2 * NC + g] + xs[3 * NC + g]);
-            const long long item = static_cast<long long>(tok) * p.heads + h0 + g;
-            if (p.splits == 1) {
-              p.out[item * p.kv_rank + d] = __float2bfloat16(l > 0.f ? o / l : 0.f);
-            } else {
-              const long long pi = item * p.splits + split;
-              p.part_o[pi * p.kv_rank + d] = o;
-              if (d == 0) {
-                p.part_ml[pi * 2] = m_ref[g];
-                p.part_ml[pi * 2 + 1] = l;
-              }
+            const long long pi = (static_cast<long long>(tok) * p.heads + h0 + g) * p.splits + split;
+            p.part_o[pi * p.kv_rank + d] = n_tiles > 0 ? __uint_as_float(ov[g]) : 0.f;
+            if (d == 0) {
+              p.part_ml[pi * 2] = m_ref[g];
+              p.part_ml[pi * 2 + 1] = (xs[g] + xs[NC + g]) + (xs[2 * NC + g] + xs[3 * NC + g]);
             }
           }
         }
       }
-    } else {
+    }
+    if (!ok) {
       report_error(p.status, TW_ERR_MBAR_TIMEOUT);
       *abort_flag = 1;
     }
@@ -382,29 +450,42 @@ latent_decode_merge_kernel(const float* __restrict__ part_o, const float* __rest
 }
 
 template <int NC>
-static int launch_latent_decode(const CUtensorMap& tm, LatentDecodeParams& p, int n, cudaStream_t stream) {
-  const int pairs = (p.chunks + 1) / 2;
-  const int fixed = ld_fixed_bytes<NC>(p.chunks);
-  int stages = (LD_SMEM_LIMIT - fixed) / (pairs * 2 * LD_CHUNK);
-  if (stages > LD_MAX_STAGES) stages = LD_MAX_STAGES;
-  if (stages < 1) {
+static int launch_latent_decode(const void* cache, int num_blocks, LatentDecodeParams& p, int n, cudaStream_t stream) {
+  CUtensorMap tm;
+  {
+    uint64_t dims[3] = {(uint64_t)p.row, (uint64_t)p.page, (uint64_t)num_blocks};
+    uint64_t strides[2] = {(uint64_t)p.row * 2, (uint64_t)p.page * p.row * 2};
+    uint32_t box[3] = {64, (uint32_t)(p.page < LD_BN ? p.page : LD_BN), 1};
+    if (!make_tensor_map_bf16(&tm, cache, 3, dims, strides, box)) return 1;
+  }
+  CUtensorMap tmQ;
+  {
+    uint64_t dims[2] = {(uint64_t)p.row, (uint64_t)n * p.heads};
+    uint64_t strides[1] = {(uint64_t)p.row * 2};
+    uint32_t box[2] = {64, NC};
+    if (!make_tensor_map_bf16(&tmQ, p.q, 2, dims, strides, box)) return 1;
+  }
+  const int tile_bytes = (p.chunks + 1) / 2 * 2 * LD_BN * 128, fixed = ld_fixed_bytes<NC>(p.chunks);
+  p.stages = (LD_SMEM_LIMIT - fixed) / tile_bytes;
+  if (p.stages > LD_MAX_STAGES) p.stages = LD_MAX_STAGES;
+  if (p.stages < 1) {
     set_last_error("latent_decode: rows of %d elements do not fit shared memory", p.row);
     return 1;
   }
-  p.stages = stages;
-  const int bytes = fixed + stages * pairs * 2 * LD_CHUNK;
+  const int bytes = fixed + p.stages * tile_bytes;
   static thread_local int configured_dev = -1;
   int dev = 0;
   cudaGetDevice(&dev);
   if (configured_dev != dev) {
-    const cudaError_t e = cudaFuncSetAttribute(latent_decode_kernel<NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, LD_SMEM_LIMIT);
+    const cudaError_t e =
+        cudaFuncSetAttribute(latent_decode_kernel<NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, LD_SMEM_LIMIT);
     if (e != cudaSuccess) {
       set_last_error("latent_decode: cudaFuncSetAttribute failed: %s", cudaGetErrorString(e));
       return 1;
     }
     configured_dev = dev;
   }
-  latent_decode_kernel<NC><<<dim3(n, (p.heads + NC - 1) / NC, p.splits), LD_THREADS, bytes, stream>>>(tm, p);
+  latent_decode_kernel<NC><<<dim3(n, (p.heads + NC - 1) / NC, p.splits), LD_THREADS, bytes, stream>>>(tm, tmQ, p);
   cudaError_t e = cudaGetLastError();
   if (e == cudaSuccess && p.splits > 1) {
     latent_decode_merge_kernel<<<n * p.heads, 128, 0, stream>>>(p.part_o, p.part_ml, p.splits, p.kv_rank, p.out);
@@ -437,15 +518,10 @@ extern "C" int tw_latent_decode(const void* qa, const void* cache, int num_block
     set_last_error("latent_decode: splits need the partial-result workspace");
     return 1;
   }
-  CUtensorMap tm;
-  {
-    uint64_t dims[3] = {(uint64_t)row, (uint64_t)page, (uint64_t)num_blocks};
-    uint64_t strides[2] = {(uint64_t)row * 2, (uint64_t)page * row * 2};
-    uint32_t box[3] = {64, (uint32_t)page, 1};
-    if (!make_tensor_map_bf16(&tm, cache, 3, dims, strides, box)) return 1;
-  }
-  LatentDecodeParams p{reinterpret_cast<const __nv_bfloat16*>(qa), reinterpret_cast<__nv_bfloat16*>(out), tok_seq, tok_kvlen,
+  LatentDecodeParams p{reinterpret_cast<const __nv_bfloat16*>(qa), reinterpret_cast<__nv_bfloat16*>(out),
+                       reinterpret_cast<const __nv_bfloat16*>(cache), tok_seq, tok_kvlen,
                        block_table, max_blocks, page, heads, row, kv_rank, splits, (row + 63) / 64, 1,
                        scale * 1.4426950408889634f, part_o, part_ml, status};
-  return heads <= 16 ? launch_latent_decode<16>(tm, p, n, stream) : launch_latent_decode<32>(tm, p, n, stream);
+  return heads <= 16 ? launch_latent_decode<16>(cache, num_blocks, p, n, stream)
+                     : launch_latent_decode<32>(cache, num_blocks, p, n, stream);
 }

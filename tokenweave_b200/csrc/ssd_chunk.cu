@@ -9,9 +9,12 @@
 // the three fp32 operands of products - the state, the weighted scores, the weighted inputs - are split into two
 // bf16 terms each.
 //
-// One CTA (eight warps) per sequence, head and 64 rows of vdim. The state lives in accumulator registers for the
-// whole sequence and passes through shared memory once per chunk as the operand of C S; the next chunk's B, C and x
-// arrive by cp.async meanwhile.
+// One CTA (16 warps) per sequence, head and 64 rows of vdim. The state lives in accumulator registers for the whole
+// sequence and passes through shared memory once per chunk as the operand of C S; the next chunk's B, C and x arrive by
+// cp.async meanwhile. A chunk has two phases between barriers: the weighted scores (ten warps own one 16 x 16 tile of
+// the lower triangle each), the weighted inputs and C S; then scores times x, the outputs, and the state. An earlier
+// form with eight warps, in which every warp made the weights of its own rows in registers, took 2.3 times the
+// instructions per scheduler slot (the weights were made twice) and was bound by latency.
 #include "tw_host.h"
 #include "tw_kernels.h"
 #include "tw_mma.cuh"
@@ -31,7 +34,7 @@ struct ChunkArgs {
 
 constexpr int CH_L = 64;          // tokens per chunk
 constexpr int CH_P = 64;          // rows of vdim per CTA
-constexpr int CH_THREADS = 256;
+constexpr int CH_THREADS = 512;
 
 template <int NP>
 struct ChunkSmem {
@@ -40,7 +43,8 @@ struct ChunkSmem {
   static constexpr int BC = CH_L * LDN, X = CH_L * LDP;        // elements
   static constexpr int STAGE = 2 * BC + X;
   static constexpr int S_ELEMS = CH_P * LDN;
-  static constexpr int BYTES = (BUFS * STAGE + 2 * S_ELEMS) * 2 + 2 * 4 * CH_L * 4;
+  static constexpr int W_ELEMS = CH_L * LDP;                                 // weighted scores, weighted inputs
+  static constexpr int BYTES = (BUFS * STAGE + 2 * S_ELEMS + 4 * W_ELEMS) * 2 + 2 * 4 * CH_L * 4;
 };
 
 // Running sums of one chunk by one warp: token 2 lane and 2 lane + 1 per lane.
@@ -50,14 +54,22 @@ struct ChunkSums {
   float last[CH_L];    // exp(l_last - l_j) dt_j
 };
 
-__device__ __forceinline__ void chunk_sums(const ChunkArgs& a, ChunkSums* s, int t0, int n, int h, float bias, float A,
-                                           int lane) {
+// The raw step sizes of a chunk: requested a chunk ahead of chunk_sums (a row of the projection per token: nothing of it
+// is in a cache).
+__device__ __forceinline__ float2 chunk_steps(const ChunkArgs& a, int t0, int t_end, int h, int lane) {
+  float2 r = make_float2(0.f, 0.f);
+  const int t = t0 + 2 * lane;
+  if (t < t_end) r.x = ld1(a.dt + t * a.ldt + h);
+  if (t + 1 < t_end) r.y = ld1(a.dt + (t + 1) * a.ldt + h);
+  return r;
+}
+
+__device__ __forceinline__ void chunk_sums(ChunkSums* s, float2 raw, int n, float bias, float A, int lane) {
   double l[2];
   float d[2];
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
-    const int j = 2 * lane + e;
-    d[e] = j < n ? softplus_f(ld1(a.dt + (t0 + j) * a.ldt + h) + bias) : 0.f;
+    d[e] = 2 * lane + e < n ? softplus_f((e ? raw.y : raw.x) + bias) : 0.f;
     l[e] = -static_cast<double>(A) * d[e];
   }
   double run = l[0] + l[1];
@@ -103,24 +115,30 @@ template <int NP>
 __global__ void __launch_bounds__(CH_THREADS, 1)
 ssd_chunk_kernel(const ChunkArgs a) {
   using SM = ChunkSmem<NP>;
-  constexpr int NT = NP / 16;                // 8-column tiles of this warp's half of the state dimension
+  constexpr int NT = NP / 32;                // 8-column tiles of this warp's quarter of the state dimension
   extern __shared__ __align__(16) uint8_t smem_raw[];
   __nv_bfloat16* stage = reinterpret_cast<__nv_bfloat16*>(smem_raw);
-  __nv_bfloat16* s_hi = stage + SM::BUFS * SM::STAGE;
+  __nv_bfloat16* s_hi = stage + SM::BUFS * SM::STAGE;        // state [vdim][N]
   __nv_bfloat16* s_lo = s_hi + SM::S_ELEMS;
-  ChunkSums* sums = reinterpret_cast<ChunkSums*>(s_lo + SM::S_ELEMS);     // [2]
+  __nv_bfloat16* m_hi = s_lo + SM::S_ELEMS;                  // weighted scores [token][token]
+  __nv_bfloat16* m_lo = m_hi + SM::W_ELEMS;
+  __nv_bfloat16* w_hi = m_lo + SM::W_ELEMS;                  // weighted inputs [token][vdim]
+  __nv_bfloat16* w_lo = w_hi + SM::W_ELEMS;
+  ChunkSums* sums = reinterpret_cast<ChunkSums*>(w_lo + SM::W_ELEMS);     // [2]
 
   const int b = a.seqs[blockIdx.x], h = blockIdx.y, p0 = blockIdx.z * CH_P;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int wr = warp & 3, wh = warp >> 2;   // row group (tokens for y, vdim for the state) and half of the columns
+  const int wr = warp & 3, wq = warp >> 2;   // row group (tokens for y, vdim for the state) and quarter of the columns
   const int q4 = lane >> 2, q2 = (lane & 3) * 2;
   const int t_begin = a.cu_q[b], t_end = a.cu_q[b + 1];
   const int p_valid = min(CH_P, a.vdim - p0);
   const int g = h / (a.heads / a.groups);
   const int off_x = h * a.vdim + p0, off_b = a.heads * a.vdim + g * a.N, off_c = off_b + a.groups * a.N;
   const float bias = ld1(a.dt_bias + h), A = expf(ld1(a.A_log + h)), D = ld1(a.D + h);
+  // tile of the lower triangle this warp makes (warps 0..9)
+  const int ti = warp < 1 ? 0 : warp < 3 ? 1 : warp < 6 ? 2 : 3, tj = warp - ti * (ti + 1) / 2;
 
-  // state rows p = 16 wr + q4 (+ 8), columns n = wh NP/2 + 8 k + q2 (+ 1)
+  // state rows p = 16 wr + q4 (+ 8), columns n = wq NP/4 + 8 k + q2 (+ 1)
   float S[NT][4];
   float* st = a.state + ((static_cast<long long>(a.slots[b]) * a.heads + h) * a.vdim + p0) * a.N;
   const bool past = a.kv_lens[b] > t_end - t_begin;
@@ -128,12 +146,17 @@ ssd_chunk_kernel(const ChunkArgs a) {
   for (int k = 0; k < NT; ++k)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int p = 16 * wr + q4 + (e >> 1) * 8, n = wh * (NP / 2) + 8 * k + q2 + (e & 1);
+      const int p = 16 * wr + q4 + (e >> 1) * 8, n = wq * (NP / 4) + 8 * k + q2 + (e & 1);
       S[k][e] = (past && p < p_valid && n < a.N) ? st[static_cast<long long>(p) * a.N + n] : 0.f;
     }
 
   chunk_load<NP>(a, stage, t_begin, min(CH_L, t_end - t_begin), off_x, p_valid, off_b, off_c);
-  if (warp == 0) chunk_sums(a, &sums[0], t_begin, min(CH_L, t_end - t_begin), h, bias, A, lane);
+  float2 steps = make_float2(0.f, 0.f);      // warp 15: raw step sizes of the next chunk
+  if (warp == 15) {
+    steps = chunk_steps(a, t_begin, t_end, h, lane);
+    chunk_sums(&sums[0], steps, t_end - t_begin, bias, A, lane);
+    steps = chunk_steps(a, t_begin + CH_L, t_end, h, lane);
+  }
 
   int c = 0;
   for (int t0 = t_begin; t0 < t_end; t0 += CH_L, ++c) {
@@ -144,12 +167,11 @@ ssd_chunk_kernel(const ChunkArgs a) {
     // the state as the operand of C S
 #pragma unroll
     for (int k = 0; k < NT; ++k) {
-      const int n = wh * (NP / 2) + 8 * k + q2;
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         uint32_t hi, lo;
         split_bf16x2(S[k][2 * e], S[k][2 * e + 1], hi, lo);
-        const int o = (16 * wr + q4 + 8 * e) * SM::LDN + n;
+        const int o = (16 * wr + q4 + 8 * e) * SM::LDN + wq * (NP / 4) + 8 * k + q2;
         *reinterpret_cast<uint32_t*>(s_hi + o) = hi;
         *reinterpret_cast<uint32_t*>(s_lo + o) = lo;
       }
@@ -161,80 +183,100 @@ ssd_chunk_kernel(const ChunkArgs a) {
       chunk_load<NP>(a, stage + ((c + 1) & 1) * SM::STAGE, t0 + CH_L, min(CH_L, t_end - t0 - CH_L), off_x, p_valid, off_b,
                      off_c);
 
-    // ---- C S and C B^T: tokens 16 wr.. of the chunk, vdim half wh ----
-    float Y[4][4] = {}, G[8][4] = {};
+    // ---- phase 1: one tile of weighted scores per warp ----
+    if (warp < 10) {
+      float G[2][4] = {};
 #pragma unroll
-    for (int k = 0; k < NP; k += 16) {
-      uint32_t fc[4];
-      ldmatrix_x4(fc, smem_u32(sc + 16 * wr * SM::LDN + k + frag_a(lane, SM::LDN)));
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        uint32_t fh[4], fl[4];
-        const int o = (32 * wh + 16 * i) * SM::LDN + k + frag_b(lane, SM::LDN);
-        ldmatrix_x4(fh, smem_u32(s_hi + o));
-        ldmatrix_x4(fl, smem_u32(s_lo + o));
-        mma_bf16(Y[2 * i], fc, fh[0], fh[1]);
-        mma_bf16(Y[2 * i + 1], fc, fh[2], fh[3]);
-        mma_bf16(Y[2 * i], fc, fl[0], fl[1]);
-        mma_bf16(Y[2 * i + 1], fc, fl[2], fl[3]);
+      for (int k = 0; k < NP; k += 16) {
+        uint32_t fc[4], fb[4];
+        ldmatrix_x4(fc, smem_u32(sc + 16 * ti * SM::LDN + k + frag_a(lane, SM::LDN)));
+        ldmatrix_x4(fb, smem_u32(sb + 16 * tj * SM::LDN + k + frag_b(lane, SM::LDN)));
+        mma_bf16(G[0], fc, fb[0], fb[1]);
+        mma_bf16(G[1], fc, fb[2], fb[3]);
       }
 #pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        if (i <= wr) {                        // keys behind the row group's last token are masked anyway
-          uint32_t fb[4];
-          ldmatrix_x4(fb, smem_u32(sb + 16 * i * SM::LDN + k + frag_b(lane, SM::LDN)));
-          mma_bf16(G[2 * i], fc, fb[0], fb[1]);
-          mma_bf16(G[2 * i + 1], fc, fb[2], fb[3]);
+      for (int e = 0; e < 2; ++e) {
+        const int i = 16 * ti + q4 + 8 * e;
+        const float hi_i = sm.hi[i], lo_i = sm.lo[i];
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+          const int j = 16 * tj + 8 * half + q2;
+          const float2 hj = *reinterpret_cast<const float2*>(sm.hi + j), lj = *reinterpret_cast<const float2*>(sm.lo + j);
+          const float2 d = *reinterpret_cast<const float2*>(sm.dt + j);
+          const float w0 = j <= i ? G[half][2 * e] * expf((hi_i - hj.x) + (lo_i - lj.x)) * d.x : 0.f;
+          const float w1 = j + 1 <= i ? G[half][2 * e + 1] * expf((hi_i - hj.y) + (lo_i - lj.y)) * d.y : 0.f;
+          uint32_t hi, lo;
+          split_bf16x2(w0, w1, hi, lo);
+          *reinterpret_cast<uint32_t*>(m_hi + i * SM::LDP + j) = hi;
+          *reinterpret_cast<uint32_t*>(m_lo + i * SM::LDP + j) = lo;
         }
       }
+    } else if (warp == 15 && more) {
+      const float2 now = steps;
+      steps = chunk_steps(a, t0 + 2 * CH_L, t_end, h, lane);
+      chunk_sums(&sums[(c + 1) & 1], now, t_end - t0 - CH_L, bias, A, lane);
+    }
+    // weighted inputs: eight values per thread
+    {
+      const int j = threadIdx.x >> 3, p = (threadIdx.x & 7) * 8;
+      float v[8];
+      ld8(sx + j * SM::LDP + p, v);
+      const float w = sm.last[j];
+      uint4 hi, lo;
+      split_bf16x2(v[0] * w, v[1] * w, hi.x, lo.x);
+      split_bf16x2(v[2] * w, v[3] * w, hi.y, lo.y);
+      split_bf16x2(v[4] * w, v[5] * w, hi.z, lo.z);
+      split_bf16x2(v[6] * w, v[7] * w, hi.w, lo.w);
+      *reinterpret_cast<uint4*>(w_hi + j * SM::LDP + p) = hi;
+      *reinterpret_cast<uint4*>(w_lo + j * SM::LDP + p) = lo;
+    }
+    // C S: tokens 16 wr.. of the chunk, vdim quarter wq; the two terms of the state in chains of their own
+    float Y[2][4] = {}, Z[2][4] = {};
+#pragma unroll
+    for (int k = 0; k < NP; k += 16) {
+      uint32_t fc[4], fh[4], fl[4];
+      const int o = 16 * wq * SM::LDN + k + frag_b(lane, SM::LDN);
+      ldmatrix_x4(fc, smem_u32(sc + 16 * wr * SM::LDN + k + frag_a(lane, SM::LDN)));
+      ldmatrix_x4(fh, smem_u32(s_hi + o));
+      ldmatrix_x4(fl, smem_u32(s_lo + o));
+      mma_bf16(Y[0], fc, fh[0], fh[1]);
+      mma_bf16(Y[1], fc, fh[2], fh[3]);
+      mma_bf16(Z[0], fc, fl[0], fl[1]);
+      mma_bf16(Z[1], fc, fl[2], fl[3]);
     }
     const int i0 = 16 * wr + q4, i1 = i0 + 8;
-    const float h0 = sm.hi[i0], l0 = sm.lo[i0], h1 = sm.hi[i1], l1 = sm.lo[i1];
-    const float e0 = expf(h0 + l0), e1 = expf(h1 + l1);
+    const float e0 = expf(sm.hi[i0] + sm.lo[i0]), e1 = expf(sm.hi[i1] + sm.lo[i1]);
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      Y[i][0] *= e0;
-      Y[i][1] *= e0;
-      Y[i][2] *= e1;
-      Y[i][3] *= e1;
+    for (int k = 0; k < 2; ++k) {
+      Y[k][0] = (Y[k][0] + Z[k][0]) * e0;
+      Y[k][1] = (Y[k][1] + Z[k][1]) * e0;
+      Y[k][2] = (Y[k][2] + Z[k][2]) * e1;
+      Y[k][3] = (Y[k][3] + Z[k][3]) * e1;
     }
-    // ---- weighted scores times x ----
+    __syncthreads();
+
+    // ---- phase 2: weighted scores times x, skip, store ----
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
       if (kt > wr) continue;
-      uint32_t ah[4], al[4];
-#pragma unroll
-      for (int half = 0; half < 2; ++half) {
-        float w[4];
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-          const int j = 16 * kt + 8 * half + q2 + e;
-          const float hj = sm.hi[j], lj = sm.lo[j], d = sm.dt[j];
-          w[e] = j <= i0 ? G[2 * kt + half][e] * expf((h0 - hj) + (l0 - lj)) * d : 0.f;
-          w[2 + e] = j <= i1 ? G[2 * kt + half][2 + e] * expf((h1 - hj) + (l1 - lj)) * d : 0.f;
-        }
-        split_bf16x2(w[0], w[1], ah[2 * half], al[2 * half]);
-        split_bf16x2(w[2], w[3], ah[2 * half + 1], al[2 * half + 1]);
-      }
-#pragma unroll
-      for (int i = 0; i < 2; ++i) {
-        uint32_t fx[4];
-        ldmatrix_x4_trans(fx, smem_u32(sx + 16 * kt * SM::LDP + 32 * wh + 16 * i + frag_b_t(lane, SM::LDP)));
-        mma_bf16(Y[2 * i], ah, fx[0], fx[1]);
-        mma_bf16(Y[2 * i + 1], ah, fx[2], fx[3]);
-        mma_bf16(Y[2 * i], al, fx[0], fx[1]);
-        mma_bf16(Y[2 * i + 1], al, fx[2], fx[3]);
-      }
+      uint32_t ah[4], al[4], fx[4];
+      const int o = 16 * wr * SM::LDP + 16 * kt + frag_a(lane, SM::LDP);
+      ldmatrix_x4(ah, smem_u32(m_hi + o));
+      ldmatrix_x4(al, smem_u32(m_lo + o));
+      ldmatrix_x4_trans(fx, smem_u32(sx + 16 * kt * SM::LDP + 16 * wq + frag_b_t(lane, SM::LDP)));
+      mma_bf16(Y[0], ah, fx[0], fx[1]);
+      mma_bf16(Y[1], ah, fx[2], fx[3]);
+      mma_bf16(Y[0], al, fx[0], fx[1]);
+      mma_bf16(Y[1], al, fx[2], fx[3]);
     }
-    // ---- skip and store ----
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const int i = e ? i1 : i0;
       if (i < n_tok) {
         __nv_bfloat16* yr = a.y + static_cast<long long>(t0 + i) * a.ldy + off_x;
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const int p = 32 * wh + 8 * k + q2;
+        for (int k = 0; k < 2; ++k) {
+          const int p = 16 * wq + 8 * k + q2;
           if (p < p_valid) {
             const float2 x = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(sx + i * SM::LDP + p));
             *reinterpret_cast<uint32_t*>(yr + p) = pack_bf16x2(fmaf(D, x.x, Y[k][2 * e]), fmaf(D, x.y, Y[k][2 * e + 1]));
@@ -242,7 +284,7 @@ ssd_chunk_kernel(const ChunkArgs a) {
         }
       }
     }
-    // ---- state: rows 16 wr.. of vdim, state half wh ----
+    // ---- state: rows 16 wr.. of vdim, state quarter wq ----
     const float keep = expf(sm.hi[CH_L - 1] + sm.lo[CH_L - 1]);
 #pragma unroll
     for (int k = 0; k < NT; ++k)
@@ -250,35 +292,30 @@ ssd_chunk_kernel(const ChunkArgs a) {
       for (int e = 0; e < 4; ++e) S[k][e] *= keep;
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
-      uint32_t fx[4], ah[4], al[4];
-      ldmatrix_x4_trans(fx, smem_u32(sx + 16 * kt * SM::LDP + 16 * wr + frag_a_t(lane, SM::LDP)));
-#pragma unroll
-      for (int r = 0; r < 4; ++r) {
-        const float2 x = unpack_bf16x2(fx[r]);
-        const int j = 16 * kt + (r >> 1) * 8 + q2;
-        split_bf16x2(x.x * sm.last[j], x.y * sm.last[j + 1], ah[r], al[r]);
-      }
+      uint32_t ah[4], al[4];
+      const int o = 16 * kt * SM::LDP + 16 * wr + frag_a_t(lane, SM::LDP);
+      ldmatrix_x4_trans(ah, smem_u32(w_hi + o));
+      ldmatrix_x4_trans(al, smem_u32(w_lo + o));
 #pragma unroll
       for (int k = 0; k < NT; k += 2) {
         uint32_t fb[4];
-        ldmatrix_x4_trans(fb, smem_u32(sb + 16 * kt * SM::LDN + wh * (NP / 2) + 8 * k + frag_b_t(lane, SM::LDN)));
+        ldmatrix_x4_trans(fb, smem_u32(sb + 16 * kt * SM::LDN + wq * (NP / 4) + 8 * k + frag_b_t(lane, SM::LDN)));
         mma_bf16(S[k], ah, fb[0], fb[1]);
         mma_bf16(S[k + 1], ah, fb[2], fb[3]);
         mma_bf16(S[k], al, fb[0], fb[1]);
         mma_bf16(S[k + 1], al, fb[2], fb[3]);
       }
     }
-    if (warp == 0 && more)
-      chunk_sums(a, &sums[(c + 1) & 1], t0 + CH_L, min(CH_L, t_end - t0 - CH_L), h, bias, A, lane);
-    __syncthreads();
-    if (SM::BUFS == 1 && more)
+    if (SM::BUFS == 1 && more) {
+      __syncthreads();
       chunk_load<NP>(a, stage, t0 + CH_L, min(CH_L, t_end - t0 - CH_L), off_x, p_valid, off_b, off_c);
+    }
   }
 #pragma unroll
   for (int k = 0; k < NT; ++k)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int p = 16 * wr + q4 + (e >> 1) * 8, n = wh * (NP / 2) + 8 * k + q2 + (e & 1);
+      const int p = 16 * wr + q4 + (e >> 1) * 8, n = wq * (NP / 4) + 8 * k + q2 + (e & 1);
       if (p < p_valid && n < a.N) st[static_cast<long long>(p) * a.N + n] = S[k][e];
     }
 }
@@ -327,7 +364,6 @@ extern "C" int tw_ssd_chunk(const void* xbc, long long ldx, const void* dt, long
                     reinterpret_cast<const bf*>(dt_bias), reinterpret_cast<const bf*>(A_log),
                     reinterpret_cast<const bf*>(D), state, reinterpret_cast<bf*>(y), ldy, seqs, cu_q, kv_lens, slots,
                     heads, vdim, N, groups};
-  if (N <= 32) return launch_chunk<32>(a, n_seqs, stream);
   if (N <= 64) return launch_chunk<64>(a, n_seqs, stream);
   if (N <= 128) return launch_chunk<128>(a, n_seqs, stream);
   return launch_chunk<256>(a, n_seqs, stream);

@@ -17,7 +17,7 @@
 namespace tw {
 
 constexpr int CONV_MAX_TAPS = 8;
-constexpr int CONV_STRIP = 8;
+constexpr int CONV_ROWS = 8;       // rows per thread
 
 struct ConvArgs {
   const void* x; long long ldx;       // inputs [T, channels]
@@ -51,55 +51,67 @@ __device__ __forceinline__ void conv_input(const ConvArgs& a, int b, int t, int 
   }
 }
 
+// A thread owns eight channels of CONV_ROWS consecutive rows. Where they and the rows before them belong to one sequence
+// (nearly everywhere) all rows are requested at once and a window of converted inputs slides over them; the rest takes
+// the general path row by row.
 template <typename T, bool VEC, int TAPS>
 __global__ void __launch_bounds__(128)
 causal_conv_kernel(const ConvArgs a) {
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
   if (c >= a.channels) return;
-  float w[TAPS][8], bias[8];
+  const int n_ch = a.channels - c;
+  const int t0 = blockIdx.y * CONV_ROWS;
+  const T* xp = reinterpret_cast<const T*>(a.x) + c;
+  T* op = reinterpret_cast<T*>(a.out) + c;
+  const T* wp = reinterpret_cast<const T*>(a.w) + c;
+  if (t0 >= TAPS - 1 && t0 + CONV_ROWS <= a.T && a.row_seq[t0 - (TAPS - 1)] == a.row_seq[t0 + CONV_ROWS - 1]) {
+    Raw8<T> raw[TAPS - 1 + CONV_ROWS];
 #pragma unroll
-  for (int k = 0; k < TAPS; ++k)
-    ld8n<VEC>(reinterpret_cast<const T*>(a.w) + static_cast<long long>(k) * a.channels + c, a.channels - c, w[k]);
-  ld8n<VEC>(reinterpret_cast<const T*>(a.bias) + c, a.channels - c, bias);
-  float hist[TAPS > 1 ? TAPS - 1 : 1][8];        // hist[k]: the input k + 1 tokens back
-  const int t0 = blockIdx.y * CONV_STRIP, t_end = min(a.T, t0 + CONV_STRIP);
-  // all rows of the strip are requested before the first is used
-  float x[CONV_STRIP][8];
-  int seqs[CONV_STRIP];
+    for (int i = 0; i < TAPS - 1 + CONV_ROWS; ++i) raw[i] = ld8raw<VEC>(xp + (t0 - (TAPS - 1) + i) * a.ldx, n_ch);
+    float2 w[TAPS][4], bias[4], win[TAPS][4];        // win[i % TAPS]: input of row i of the strip
+    float v[8];
 #pragma unroll
-  for (int i = 0; i < CONV_STRIP; ++i) {
-    const int t = min(t0 + i, t_end - 1);
-    ld8n<VEC>(reinterpret_cast<const T*>(a.x) + t * a.ldx + c, a.channels - c, x[i]);
-    seqs[i] = a.row_seq[t];
-  }
+    for (int k = 0; k < TAPS; ++k) {
+      ld8n<VEC>(wp + static_cast<long long>(k) * a.channels, n_ch, v);
 #pragma unroll
-  for (int k = 0; k < TAPS - 1; ++k) conv_input<T, VEC>(a, seqs[0], t0, k + 1, c, hist[k]);
-#pragma unroll
-  for (int i = 0; i < CONV_STRIP; ++i) {
-    const int t = t0 + i;
-    if (t >= t_end) break;
-    if (i > 0 && seqs[i] != seqs[i - 1]) {
-#pragma unroll
-      for (int k = 0; k < TAPS - 1; ++k) conv_input<T, VEC>(a, seqs[i], t, k + 1, c, hist[k]);
+      for (int j = 0; j < 4; ++j) w[k][j] = make_float2(v[2 * j], v[2 * j + 1]);
     }
+    ld8n<VEC>(reinterpret_cast<const T*>(a.bias) + c, n_ch, v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) bias[j] = make_float2(v[2 * j], v[2 * j + 1]);
+#pragma unroll
+    for (int i = 0; i < TAPS - 1 + CONV_ROWS; ++i) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) win[i % TAPS][j] = make_float2(ld1(&raw[i].v[2 * j]), ld1(&raw[i].v[2 * j + 1]));
+      if (i < TAPS - 1) continue;
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        float2 y = bias[j];
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) y = fma2(win[(i - (TAPS - 1) + k) % TAPS][j], w[k][j], y);
+        v[2 * j] = silu_t<T>(y.x);
+        v[2 * j + 1] = silu_t<T>(y.y);
+      }
+      st8n<VEC>(op + (t0 + i - (TAPS - 1)) * a.ldo, n_ch, v);
+    }
+    return;
+  }
+  const int t_end = min(a.T, t0 + CONV_ROWS);
+#pragma unroll 1
+  for (int t = t0; t < t_end; ++t) {
     float y[8];
+    ld8n<VEC>(reinterpret_cast<const T*>(a.bias) + c, n_ch, y);
+#pragma unroll 1
+    for (int k = 0; k < TAPS; ++k) {
+      float v[8], w[8];
+      conv_input<T, VEC>(a, a.row_seq[t], t, TAPS - 1 - k, c, v);
+      ld8n<VEC>(wp + static_cast<long long>(k) * a.channels, n_ch, w);
 #pragma unroll
-    for (int j = 0; j < 8; ++j) y[j] = fmaf(x[i][j], w[TAPS - 1][j], bias[j]);
-#pragma unroll
-    for (int k = 0; k < TAPS - 1; ++k)
-#pragma unroll
-      for (int j = 0; j < 8; ++j) y[j] = fmaf(hist[k][j], w[TAPS - 2 - k][j], y[j]);
+      for (int j = 0; j < 8; ++j) y[j] = fmaf(v[j], w[j], y[j]);
+    }
 #pragma unroll
     for (int j = 0; j < 8; ++j) y[j] = silu_t<T>(y[j]);
-    st8n<VEC>(reinterpret_cast<T*>(a.out) + t * a.ldo + c, a.channels - c, y);
-#pragma unroll
-    for (int k = TAPS - 2; k > 0; --k)
-#pragma unroll
-      for (int j = 0; j < 8; ++j) hist[k][j] = hist[k - 1][j];
-    if (TAPS > 1) {
-#pragma unroll
-      for (int j = 0; j < 8; ++j) hist[0][j] = x[i][j];
-    }
+    st8n<VEC>(op + t * a.ldo, n_ch, y);
   }
 }
 
@@ -244,7 +256,7 @@ static int launch_conv(const ConvArgs& a, int single, cudaStream_t stream) {
 #undef TW_CASE
     return check_launch("causal_conv (single tokens)");
   }
-  const dim3 grid(gx, (a.T + CONV_STRIP - 1) / CONV_STRIP);
+  const dim3 grid(gx, (a.T + CONV_ROWS - 1) / CONV_ROWS);
 #define TW_CASE(K) case K: causal_conv_kernel<T, VEC, K><<<grid, threads, 0, stream>>>(a); break;
   switch (a.taps) { TW_CASE(1) TW_CASE(2) TW_CASE(3) TW_CASE(4) TW_CASE(5) TW_CASE(6) TW_CASE(7) TW_CASE(8) }
 #undef TW_CASE

@@ -61,6 +61,28 @@ __device__ __forceinline__ void st8n(T* p, int n, const float (&v)[8]) {
   }
 }
 
+// Eight elements as they are stored (a request whose conversion can wait).
+template <typename T>
+struct __align__(16) Raw8 {
+  T v[8];
+};
+template <bool VEC, typename T>
+__device__ __forceinline__ Raw8<T> ld8raw(const T* p, int n) {
+  Raw8<T> r;
+  if (VEC && n >= 8) {
+    if constexpr (sizeof(T) == 2) {
+      *reinterpret_cast<uint4*>(&r) = *reinterpret_cast<const uint4*>(p);
+    } else {
+      reinterpret_cast<uint4*>(&r)[0] = reinterpret_cast<const uint4*>(p)[0];
+      reinterpret_cast<uint4*>(&r)[1] = reinterpret_cast<const uint4*>(p)[1];
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < 8; ++j) st1(&r.v[j], j < n ? ld1(p + j) : 0.f);
+  }
+  return r;
+}
+
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
 // Activations of bf16 tensors: the result is rounded to 8 bits of mantissa, the hardware exponential and division
