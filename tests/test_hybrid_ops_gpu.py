@@ -1,5 +1,6 @@
 """Kernels of the hybrid operators (``ops/hybrid.py``) against plain fp32 PyTorch on the CPU: bf16 and fp32 storage, sizes
 that are not multiples of anything, and the tensor-core forms against the same references."""
+import functools
 import math
 
 import pytest
@@ -208,10 +209,11 @@ def test_causal_conv(dtype, channels, taps, q_lens, kv_lens):
     assert torch.equal(gs.cpu(), state)
 
 
-@pytest.mark.parametrize("form,dtype", [("scan", torch.float32), ("scan", torch.bfloat16), ("chunk", torch.bfloat16)])
+@pytest.mark.parametrize("form,dtype", [("scan", torch.float32), ("scan", torch.bfloat16), ("chunk", torch.bfloat16),
+                                        ("chunk64", torch.bfloat16)])
 @pytest.mark.parametrize("heads,vdim,N,groups", [(4, 40, 48, 2), (6, 64, 128, 1), (3, 72, 16, 3), (2, 24, 200, 1), (8, 8, 64, 8)])
 def test_ssd(form, dtype, heads, vdim, N, groups):
-    q_lens, kv_lens = [70, 1, 200, 64, 3], [70, 9, 201, 500, 3]
+    q_lens, kv_lens = [70, 1, 400, 64, 3, 128], [70, 9, 401, 500, 3, 129]
     T, B, inner = sum(q_lens), len(q_lens), heads * vdim
     xbc = rnd(T, inner + 2 * groups * N, dtype=dtype, scale=0.5)
     dt, bias = rnd(T, heads, dtype=dtype), rnd(heads, dtype=dtype, scale=0.5)
@@ -225,7 +227,7 @@ def test_ssd(form, dtype, heads, vdim, N, groups):
     y, gy, gs = torch.zeros(T, inner, dtype=dtype), torch.zeros(T, inner, dtype=dtype, device=DEV), state.to(DEV)
     seqs = i32(range(B))
     ref.ssd_scan(xbc, dt, bias, A, D, state, y, seqs, cu, i32(kv_lens), slots, groups)
-    fn = hops.ssd_scan if form == "scan" else hops.ssd_chunk
+    fn = {"scan": hops.ssd_scan, "chunk": hops.ssd_chunk, "chunk64": functools.partial(hops.ssd_chunk, form=1)}[form]
     fn(xbc.to(DEV), dt.to(DEV), bias.to(DEV), A.to(DEV), D.to(DEV), gs, gy, seqs.to(DEV), cu.to(DEV), i32(kv_lens).to(DEV),
        slots.to(DEV), groups)
     # the state is fp32 in every form: what the two-term products of the chunked form leave is far below bf16

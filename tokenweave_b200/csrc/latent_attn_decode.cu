@@ -147,7 +147,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
         const int block = table[min((key0 + (lane & (pieces - 1)) * piece) / p.page, last_page)];
         uint8_t* tile = smem + st * tile_bytes;
         for (int pr = 0; pr < pairs; ++pr) {
-          if (!mbar_wait(&empty[st * LD_MAX_PAIRS + pr], ph ^ 1)) { ok = false; break; }
+          if (!mbar_wait_warp(&empty[st * LD_MAX_PAIRS + pr], ph ^ 1)) { ok = false; break; }
           uint64_t* bar = &full[st * LD_MAX_PAIRS + pr];
           const bool two = 2 * pr + 1 < p.chunks;
           mbar_expect_tx_e(bar, (two ? 2 : 1) * CHUNK);
@@ -174,14 +174,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       const uint64_t desc_v = make_smem_desc_sw128(smem_u32(smem), CHUNK, 1024);          // MN-major: latent columns
       const uint64_t desc_q = make_smem_desc_sw128(smem_u32(s_q), 16, 1024);
       const uint64_t desc_p = make_smem_desc_sw128(smem_u32(s_p), 16, 1024);
-      bool ok = mbar_wait(q_ready, 0);
+      bool ok = mbar_wait_warp(q_ready, 0);
       auto issue_s = [&](int j) {
         const int st = j % p.stages;
         const uint32_t ph = (j / p.stages) & 1;
         const uint32_t tile_off = st * tile_bytes;
         const uint32_t d = tmem_base + (j & 1) * NC;
         for (int pr = 0; pr < pairs; ++pr) {
-          if (!mbar_wait(&full[st * LD_MAX_PAIRS + pr], ph)) return false;
+          if (!mbar_wait_warp(&full[st * LD_MAX_PAIRS + pr], ph)) return false;
           tc_fence_after_sync();
           // descriptors hold addresses in units of 16 bytes in their low bits: one addition each per instruction
           const uint64_t da = desc_tile + (tile_off + pr * 2 * CHUNK) / 16, db = desc_q + pr * (2 * NC * 128 / 16);
@@ -200,7 +200,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       auto tile_here = [&](int j) {
         const uint32_t ph = (j / p.stages) & 1;
         for (int pr = 0; pr < pairs; ++pr)
-          if (!mbar_test(&full[(j % p.stages) * LD_MAX_PAIRS + pr], ph)) return false;
+          if (!mbar_test_warp(&full[(j % p.stages) * LD_MAX_PAIRS + pr], ph)) return false;
         return true;
       };
       if (ok) ok = issue_s(0);
@@ -218,9 +218,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
               if (!ok) break;
               ahead = true;
             }
-            have_p = ahead || p.stages == 1 ? mbar_try_wait(p_ready, j & 1) : mbar_test(p_ready, j & 1);
+            have_p = ahead || p.stages == 1 ? mbar_try_wait_warp(p_ready, j & 1) : mbar_test_warp(p_ready, j & 1);
           }
-          if (!ok || (!have_p && globaltimer_ns() - t_start > TW_WAIT_BUDGET_NS)) { ok = false; break; }
+          if (!ok || (!have_p && __any_sync(0xffffffffu, globaltimer_ns() - t_start > TW_WAIT_BUDGET_NS))) { ok = false; break; }
         }
         if (!ok) break;
         tc_fence_after_sync();

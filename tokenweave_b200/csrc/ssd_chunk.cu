@@ -344,14 +344,21 @@ static int launch_chunk(const ChunkArgs& a, int n_seqs, cudaStream_t stream) {
   return 0;
 }
 
+int launch_ssd_chunk_tc(const void* xbc, long long ldx, int T, const void* dt, long long ldt, const void* dt_bias,
+                        const void* A_log, const void* D, float* state, void* y, long long ldy, const int* seqs,
+                        int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads, int vdim, int N,
+                        int groups, uint32_t* status, cudaStream_t stream);
+
 }  // namespace tw
 
 using namespace tw;
 
-extern "C" int tw_ssd_chunk(const void* xbc, long long ldx, const void* dt, long long ldt, const void* dt_bias,
+// xbc [T, ...]; form 0: tcgen05 (ssd_chunk_tc.cu) for states of up to 128 dimensions, this file's kernel otherwise;
+// form 1: this file's kernel.
+extern "C" int tw_ssd_chunk(const void* xbc, long long ldx, int T, const void* dt, long long ldt, const void* dt_bias,
                             const void* A_log, const void* D, float* state, void* y, long long ldy, const int* seqs,
                             int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads, int vdim, int N,
-                            int groups, cudaStream_t stream) {
+                            int groups, int form, uint32_t* status, cudaStream_t stream) {
   if (n_seqs <= 0) return 0;
   if (groups <= 0 || heads % groups != 0 || vdim % 8 != 0 || N % 8 != 0 || ldx % 8 != 0 || ldy % 2 != 0 || N > 256 ||
       (reinterpret_cast<uintptr_t>(xbc) & 15) != 0) {
@@ -359,6 +366,9 @@ extern "C" int tw_ssd_chunk(const void* xbc, long long ldx, const void* dt, long
                    N, ldx);
     return 1;
   }
+  if (form == 0 && N <= 128 && ldy % 8 == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0)
+    return launch_ssd_chunk_tc(xbc, ldx, T, dt, ldt, dt_bias, A_log, D, state, y, ldy, seqs, n_seqs, cu_q, kv_lens, slots,
+                               heads, vdim, N, groups, status, stream);
   using bf = __nv_bfloat16;
   const ChunkArgs a{reinterpret_cast<const bf*>(xbc), ldx, reinterpret_cast<const bf*>(dt), ldt,
                     reinterpret_cast<const bf*>(dt_bias), reinterpret_cast<const bf*>(A_log),

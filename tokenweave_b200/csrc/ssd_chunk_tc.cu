@@ -1,0 +1,464 @@
+// State-space (Mamba-2) recurrence of long runs on tcgen05: 128 tokens at a time in the quadratic form, for states of up
+// to 128 dimensions (ssd_chunk.cu has the form for wider states and the arithmetic in words).
+//
+// Per chunk and head, with tokens as the 128 rows of an MMA:
+//     G  = C B^T                      [128 x 128]      A = C, B operand = B
+//     Y2 = C (S_hi + S_lo)            [128 x 64]       the state, read out; rows scaled by exp(l_i) in the epilogue
+//     Y1 = (M_hi + M_lo) X            [128 x 64]       M = weighted scores, the A operand from tensor memory
+//     dS = B^T (W_hi + W_lo)          [N x 64]         W = inputs weighted with exp(l_last - l_j) dt_j
+// B, C, X are the bf16 activations as TMA brings them; S, M, W are fp32 values in two bf16 terms. The state itself is in
+// the registers of the state warps (one row of 64 per thread): S = exp(l_last) S + dS, so only its read-out passes
+// through shared memory and nothing but that small update is serial from chunk to chunk.
+//
+// Roles (480 threads): warp 0 TMA producer, warp 1 MMA issuer, warps 2..5 and 6..9 scores (thread = token, each group half
+// of the keys) and epilogue (each group half of vdim), warps 10..13 state (thread = state row) and W (thread = token),
+// warp 14 running sums. G is double-buffered in tensor memory, so that the scores of a chunk are made while the products of
+// the one before run. All waits are bounded; after a timeout the roles keep their trip counts (the named barriers of the
+// score warps are not bounded), skip further waits, report TW_ERR_MBAR_TIMEOUT and leave through the tear-down.
+#include "attn_prefill_common.cuh"
+#include "tw_elect.cuh"
+#include "tw_host.h"
+#include "tw_kernels.h"
+#include "tw_mma.cuh"
+#include "tw_typed.cuh"
+
+namespace tw {
+
+constexpr int SC_L = 128;                          // tokens per chunk
+constexpr int SC_P = 64;                           // rows of vdim per CTA
+constexpr int SC_THREADS = 480;
+constexpr int SC_CHUNK = SC_L * 128;               // 128 rows x 64 bf16, swizzled
+
+struct ScanTcParams {
+  const __nv_bfloat16* dt; long long ldt;
+  const __nv_bfloat16 *dt_bias, *A_log, *D;
+  float* state;
+  __nv_bfloat16* y; long long ldy;
+  const int *seqs, *cu_q, *kv_lens, *slots;
+  int heads, vdim, N, groups, n_chunks;            // n_chunks: 64-column chunks of the state dimension (1 or 2)
+  uint32_t* status;
+};
+
+// Running sums of a chunk in base 2: hi + lo = l log2(e) to two floats.
+struct ScanSums {
+  float dt[SC_L], hi[SC_L], lo[SC_L], last[SC_L], grow[SC_L];      // last: exp(l_last - l) dt, grow: exp(l)
+  float keep, pad[3];                                              // exp(l_last)
+};
+
+constexpr int SC_OFF_C = 0;                                  // [2 chunks]
+constexpr int SC_OFF_B = SC_OFF_C + 2 * SC_CHUNK;            // [2 buffers][2 chunks]
+constexpr int SC_OFF_X = SC_OFF_B + 4 * SC_CHUNK;            // [2 buffers]
+constexpr int SC_OFF_S = SC_OFF_X + 2 * SC_CHUNK;            // hi, lo: [state][vdim]
+constexpr int SC_OFF_W = SC_OFF_S + 2 * SC_CHUNK;            // hi, lo: [token][vdim]
+constexpr int SC_OFF_SUMS = SC_OFF_W + 2 * SC_CHUNK;
+constexpr int SC_OFF_BAR = SC_OFF_SUMS + 2 * static_cast<int>(sizeof(ScanSums));
+constexpr int SC_SMEM = SC_OFF_BAR + 256 + 1024;
+
+// Column c (of 64) of row r of a swizzled tile with 128-byte rows: byte offset of its 16-byte group.
+__device__ __forceinline__ uint32_t sw_off(int r, int group) { return r * 128 + ((group ^ (r & 7)) * 16); }
+
+__global__ void __launch_bounds__(SC_THREADS, 1)
+ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_constant__ CUtensorMap tmBC,
+                    const ScanTcParams p) {
+  constexpr uint32_t IDESC_G = make_idesc_bf16(128, 128, 0, 0);     // A = C, B = B: both K-major
+  constexpr uint32_t IDESC_Y = make_idesc_bf16(128, 64, 0, 1);      // A = C or M, B operand = S or X (MN-major)
+  constexpr uint32_t IDESC_S = make_idesc_bf16(128, 64, 1, 1);      // A = B^T (MN-major), B operand = W (MN-major)
+  constexpr uint32_t TMEM_COLS = 512;
+  constexpr uint32_t COL_G = 0, COL_Y1 = 256, COL_Y2 = 320, COL_DS = 384;      // G: two buffers of 128
+
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
+                                             ~static_cast<uintptr_t>(1023));
+  ScanSums* sums = reinterpret_cast<ScanSums*>(smem + SC_OFF_SUMS);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + SC_OFF_BAR);
+  uint64_t *c_full = bars, *c_empty = bars + 1, *bx_full = bars + 2, *bx_empty = bars + 4;
+  uint64_t *sums_full = bars + 6, *sums_empty = bars + 8;
+  uint64_t *g_full = bars + 10, *m_ready = bars + 11;
+  uint64_t *s_ready = bars + 12, *s_free = bars + 13, *w_ready = bars + 14, *ds_full = bars + 15, *ds_read = bars + 16;
+  uint64_t *y_full = bars + 17, *y_free = bars + 18;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 19);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int b = p.seqs[blockIdx.x], h = blockIdx.y, p0 = blockIdx.z * SC_P;
+  const int t_begin = p.cu_q[b], t_end = p.cu_q[b + 1];
+  const int n_ch = (t_end - t_begin + SC_L - 1) / SC_L;
+  const int p_valid = min(SC_P, p.vdim - p0);
+  const int g = h / (p.heads / p.groups);
+
+  if (threadIdx.x == 0) {
+    mbar_init(c_full, 1);
+    mbar_init(c_empty, 1);
+    for (int i = 0; i < 2; ++i) {
+      mbar_init(&bx_full[i], 1);
+      mbar_init(&bx_empty[i], 1 + 128 + 256);
+      mbar_init(&sums_full[i], 32);
+      mbar_init(&sums_empty[i], 128 + 256);
+    }
+    mbar_init(g_full, 1);
+    mbar_init(m_ready, 256);
+    mbar_init(s_ready, 128);
+    mbar_init(s_free, 1);
+    mbar_init(w_ready, 128);
+    mbar_init(ds_full, 1);
+    mbar_init(ds_read, 128);
+    mbar_init(y_full, 1);
+    mbar_init(y_free, 256);
+    *abort_flag = 0;
+    mbar_fence_init();
+  }
+  if (warp == 1) {
+    tmem_alloc(tmem_slot, TMEM_COLS);
+    tmem_relinquish();
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem_base = *tmem_slot;
+  bool ok = true;
+
+  if (warp == 0) {
+    // ---------------- TMA producer (uniform over the warp) ----------------
+    for (int c = 0; ok && c < n_ch; ++c) {
+      const int st = c & 1, t0 = t_begin + c * SC_L;
+      if (!mbar_wait_warp(&bx_empty[st], ((c >> 1) & 1) ^ 1)) { ok = false; break; }
+      mbar_expect_tx_e(&bx_full[st], (p.n_chunks + 1) * SC_CHUNK);
+      for (int k = 0; k < p.n_chunks; ++k)
+        tma_load_3d_e(smem + SC_OFF_B + (2 * st + k) * SC_CHUNK, &tmBC, &bx_full[st], k * 64, g, t0);
+      tma_load_3d_e(smem + SC_OFF_X + st * SC_CHUNK, &tmX, &bx_full[st], p0, h, t0);
+      if (!mbar_wait_warp(c_empty, (c & 1) ^ 1)) { ok = false; break; }
+      mbar_expect_tx_e(c_full, p.n_chunks * SC_CHUNK);
+      for (int k = 0; k < p.n_chunks; ++k)
+        tma_load_3d_e(smem + SC_OFF_C + k * SC_CHUNK, &tmBC, c_full, k * 64, p.groups + g, t0);
+    }
+  } else if (warp == 1) {
+    // ---------------- MMA issuer (uniform over the warp) ----------------
+    const uint64_t d_c = make_smem_desc_sw128(smem_u32(smem + SC_OFF_C), 16, 1024);
+    const uint64_t d_b = make_smem_desc_sw128(smem_u32(smem + SC_OFF_B), 16, 1024);
+    const uint64_t d_bt = make_smem_desc_sw128(smem_u32(smem + SC_OFF_B), SC_CHUNK, 1024);
+    const uint64_t d_x = make_smem_desc_sw128(smem_u32(smem + SC_OFF_X), SC_CHUNK, 1024);
+    const uint64_t d_s = make_smem_desc_sw128(smem_u32(smem + SC_OFF_S), SC_CHUNK, 1024);
+    const uint64_t d_w = make_smem_desc_sw128(smem_u32(smem + SC_OFF_W), SC_CHUNK, 1024);
+    constexpr int K_ROWS = 16 * 128 / 16;        // 16 rows of an MN-major tile, in descriptor units
+    auto issue_g = [&](int c) {
+      if (!mbar_wait_warp(c_full, c & 1) || !mbar_wait_warp(&bx_full[c & 1], (c >> 1) & 1)) return false;
+      tc_fence_after_sync();
+      const uint64_t db = d_b + (c & 1) * (2 * SC_CHUNK / 16);
+      for (int q = 0; q < p.n_chunks; ++q) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k)
+          umma_ss_e(tmem_base + COL_G + (c & 1) * 128, d_c + q * (SC_CHUNK / 16) + k * 2, db + q * (SC_CHUNK / 16) + k * 2,
+                    IDESC_G, (q | k) != 0 ? 1u : 0u);
+      }
+      umma_commit_e(g_full);
+      return true;
+    };
+    if (n_ch > 0) ok = issue_g(0);
+    for (int c = 0; ok && c < n_ch; ++c) {
+      const int st = c & 1;
+      // Y2: the state before the chunk
+      if (!mbar_wait_warp(s_ready, c & 1) || !mbar_wait_warp(y_free, (c & 1) ^ 1)) { ok = false; break; }
+      tc_fence_after_sync();
+      for (int q = 0; q < p.n_chunks; ++q) {
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+          const uint64_t da = d_c + q * (SC_CHUNK / 16) + k * 2, db = d_s + (q * 4 + k) * K_ROWS;
+          umma_ss_e(tmem_base + COL_Y2, da, db, IDESC_Y, (q | k) != 0 ? 1u : 0u);
+          umma_ss_e(tmem_base + COL_Y2, da, db + SC_CHUNK / 16, IDESC_Y, 1u);
+        }
+      }
+      umma_commit_e(c_empty);
+      umma_commit_e(s_free);
+      // dS
+      if (!mbar_wait_warp(w_ready, c & 1) || !mbar_wait_warp(ds_read, (c & 1) ^ 1)) { ok = false; break; }
+      tc_fence_after_sync();
+      {
+        const uint64_t da = d_bt + st * (2 * SC_CHUNK / 16);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          umma_ss_e(tmem_base + COL_DS, da + k * K_ROWS, d_w + k * K_ROWS, IDESC_S, k != 0 ? 1u : 0u);
+          umma_ss_e(tmem_base + COL_DS, da + k * K_ROWS, d_w + SC_CHUNK / 16 + k * K_ROWS, IDESC_S, 1u);
+        }
+      }
+      umma_commit_e(ds_full);
+      // the next chunk's scores, then this chunk's weighted scores times X
+      if (c + 1 < n_ch) {
+        ok = issue_g(c + 1);
+        if (!ok) break;
+      }
+      if (!mbar_wait_warp(m_ready, c & 1)) { ok = false; break; }
+      tc_fence_after_sync();
+      {
+        const uint32_t m = tmem_base + COL_G + st * 128;
+        const uint64_t dx = d_x + st * (SC_CHUNK / 16);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) {
+          umma_ts_e(tmem_base + COL_Y1, m + k * 8, dx + k * K_ROWS, IDESC_Y, k != 0 ? 1u : 0u);
+          umma_ts_e(tmem_base + COL_Y1, m + 64 + k * 8, dx + k * K_ROWS, IDESC_Y, 1u);
+        }
+      }
+      umma_commit_e(y_full);
+      umma_commit_e(&bx_empty[st]);
+    }
+  } else if (warp < 10) {
+    // ---------------- scores and epilogue ----------------
+    const int grp = (warp - 2) >> 2, qr = warp & 3;
+    const int r = qr * 32 + lane;                               // token of the chunk
+    const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(qr * 32) << 16);
+    const float D = ld1(p.D + h);
+    auto epilogue = [&](int c) {
+      const int st = c & 1;
+      if (ok) ok = mbar_wait(y_full, c & 1);
+      tc_fence_after_sync();
+      const float e = sums[st].grow[r];
+      const int t = t_begin + c * SC_L + r;
+      uint32_t a[32], s[32];
+      tmem_ld_32x32(t_lane + COL_Y1 + grp * 32, a);
+      tmem_ld_32x32(t_lane + COL_Y2 + grp * 32, s);
+      tmem_wait_ld();
+      tc_fence_before_sync();
+      mbar_arrive(y_free);
+      const uint8_t* xr = smem + SC_OFF_X + st * SC_CHUNK;
+#pragma unroll
+      for (int v = 0; v < 4; ++v) {
+        const int p8 = grp * 4 + v;
+        float x[8];
+        ld8(reinterpret_cast<const __nv_bfloat16*>(xr + sw_off(r, p8)), x);
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+          x[i] = fmaf(D, x[i], fmaf(e, __uint_as_float(s[8 * v + i]), __uint_as_float(a[8 * v + i])));
+        if (ok && t < t_end && p8 * 8 < p_valid) st8(p.y + t * p.ldy + h * p.vdim + p0 + p8 * 8, x);
+      }
+      mbar_arrive(&bx_empty[st]);
+      mbar_arrive(&sums_empty[st]);
+    };
+    for (int c = 0; c < n_ch; ++c) {
+      const int st = c & 1;
+      if (ok) ok = mbar_wait(&sums_full[st], (c >> 1) & 1);
+      if (ok) ok = mbar_wait(g_full, c & 1);
+      tc_fence_after_sync();
+      const uint32_t t_g = t_lane + COL_G + st * 128;
+      uint32_t s0[32], s1[32];
+      tmem_ld_32x32(t_g + grp * 64, s0);
+      tmem_ld_32x32(t_g + grp * 64 + 32, s1);
+      tmem_wait_ld();
+      // the other group's half is overwritten below: both have to be in registers first
+      tc_fence_before_sync();
+      split_pair_sync(qr);
+      tc_fence_after_sync();
+      const ScanSums& sm = sums[st];
+      const float hi_i = sm.hi[r], lo_i = sm.lo[r];
+      auto half = [&](const uint32_t (&sc)[32], int j0, uint32_t col) {
+        uint32_t mh[16], ml[16];
+        if (j0 > qr * 32 + 31) {                                // warp-uniform: every key is behind every token
+#pragma unroll
+          for (int i = 0; i < 16; ++i) mh[i] = ml[i] = 0u;
+        } else {
+#pragma unroll
+          for (int i = 0; i < 16; i += 2) {
+            const float4 hj = *reinterpret_cast<const float4*>(sm.hi + j0 + 2 * i);
+            const float4 lj = *reinterpret_cast<const float4*>(sm.lo + j0 + 2 * i);
+            const float4 d = *reinterpret_cast<const float4*>(sm.dt + j0 + 2 * i);
+            float w[4];
+            w[0] = __uint_as_float(sc[2 * i]) * (fast_exp2((hi_i - hj.x) + (lo_i - lj.x)) * d.x);
+            w[1] = __uint_as_float(sc[2 * i + 1]) * (fast_exp2((hi_i - hj.y) + (lo_i - lj.y)) * d.y);
+            w[2] = __uint_as_float(sc[2 * i + 2]) * (fast_exp2((hi_i - hj.z) + (lo_i - lj.z)) * d.z);
+            w[3] = __uint_as_float(sc[2 * i + 3]) * (fast_exp2((hi_i - hj.w) + (lo_i - lj.w)) * d.w);
+#pragma unroll
+            for (int e = 0; e < 4; ++e)
+              if (j0 + 2 * i + e > r) w[e] = 0.f;
+            split_bf16x2(w[0], w[1], mh[i], ml[i]);
+            split_bf16x2(w[2], w[3], mh[i + 1], ml[i + 1]);
+          }
+        }
+        tmem_st_32x16(t_g + col, mh);
+        tmem_st_32x16(t_g + 64 + col, ml);
+      };
+      half(s0, grp * 64, grp * 32);
+      half(s1, grp * 64 + 32, grp * 32 + 16);
+      tmem_wait_st();
+      tc_fence_before_sync();
+      mbar_arrive(m_ready);          // arrive even after a failed wait so that the issuer is not left waiting
+      if (c > 0) epilogue(c - 1);
+    }
+    if (n_ch > 0) epilogue(n_ch - 1);
+  } else if (warp < 14) {
+    // ---------------- state and weighted inputs ----------------
+    const int qr = warp & 3;
+    const int r = qr * 32 + lane;                               // state row, token of the chunk
+    const uint32_t t_ds = tmem_base + (static_cast<uint32_t>(qr * 32) << 16) + COL_DS;
+    float* st_g = p.state + ((static_cast<long long>(p.slots[b]) * p.heads + h) * p.vdim + p0) * p.N + r;
+    const bool past = p.kv_lens[b] > t_end - t_begin && r < p.N;
+    float S[SC_P];
+#pragma unroll
+    for (int i = 0; i < SC_P; ++i) S[i] = past && i < p_valid ? st_g[static_cast<long long>(i) * p.N] : 0.f;
+    for (int c = 0; c < n_ch; ++c) {
+      const int st = c & 1;
+      // S is read by the read-out of this chunk once the previous one's is done
+      if (ok && c > 0) ok = mbar_wait(s_free, (c - 1) & 1);
+      uint8_t* s_hi = smem + SC_OFF_S;
+#pragma unroll
+      for (int v = 0; v < 8; ++v) {
+        uint4 hi, lo;
+        split_bf16x2(S[8 * v], S[8 * v + 1], hi.x, lo.x);
+        split_bf16x2(S[8 * v + 2], S[8 * v + 3], hi.y, lo.y);
+        split_bf16x2(S[8 * v + 4], S[8 * v + 5], hi.z, lo.z);
+        split_bf16x2(S[8 * v + 6], S[8 * v + 7], hi.w, lo.w);
+        *reinterpret_cast<uint4*>(s_hi + sw_off(r, v)) = hi;
+        *reinterpret_cast<uint4*>(s_hi + SC_CHUNK + sw_off(r, v)) = lo;
+      }
+      fence_proxy_async_smem();
+      mbar_arrive(s_ready);
+      // W (free: the products of the previous chunk were waited for below)
+      if (ok) ok = mbar_wait(&sums_full[st], (c >> 1) & 1);
+      if (ok) ok = mbar_wait(&bx_full[st], (c >> 1) & 1);
+      const float w = sums[st].last[r], keep = sums[st].keep;
+      const uint8_t* xr = smem + SC_OFF_X + st * SC_CHUNK;
+      uint8_t* w_hi = smem + SC_OFF_W;
+#pragma unroll
+      for (int v = 0; v < 8; ++v) {
+        float x[8];
+        ld8(reinterpret_cast<const __nv_bfloat16*>(xr + sw_off(r, v)), x);
+        uint4 hi, lo;
+        split_bf16x2(x[0] * w, x[1] * w, hi.x, lo.x);
+        split_bf16x2(x[2] * w, x[3] * w, hi.y, lo.y);
+        split_bf16x2(x[4] * w, x[5] * w, hi.z, lo.z);
+        split_bf16x2(x[6] * w, x[7] * w, hi.w, lo.w);
+        *reinterpret_cast<uint4*>(w_hi + sw_off(r, v)) = hi;
+        *reinterpret_cast<uint4*>(w_hi + SC_CHUNK + sw_off(r, v)) = lo;
+      }
+      fence_proxy_async_smem();
+      mbar_arrive(w_ready);
+      mbar_arrive(&bx_empty[st]);
+      mbar_arrive(&sums_empty[st]);
+      if (ok) ok = mbar_wait(ds_full, c & 1);
+      tc_fence_after_sync();
+      uint32_t d[32];
+      tmem_ld_32x32(t_ds, d);
+      tmem_wait_ld();
+#pragma unroll
+      for (int i = 0; i < 32; ++i) S[i] = fmaf(S[i], keep, __uint_as_float(d[i]));
+      tmem_ld_32x32(t_ds + 32, d);
+      tmem_wait_ld();
+#pragma unroll
+      for (int i = 0; i < 32; ++i) S[32 + i] = fmaf(S[32 + i], keep, __uint_as_float(d[i]));
+      tc_fence_before_sync();
+      mbar_arrive(ds_read);
+    }
+    if (ok && r < p.N) {
+#pragma unroll
+      for (int i = 0; i < SC_P; ++i)
+        if (i < p_valid) st_g[static_cast<long long>(i) * p.N] = S[i];
+    }
+  } else {
+    // ---------------- running sums: four tokens per lane ----------------
+    const float bias = ld1(p.dt_bias + h), A = expf(ld1(p.A_log + h));
+    auto request = [&](int c, float (&raw)[4]) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int t = t_begin + c * SC_L + 4 * lane + e;
+        raw[e] = t < t_end ? ld1(p.dt + t * p.ldt + h) : 0.f;
+      }
+    };
+    float next[4];
+    request(0, next);
+    for (int c = 0; c < n_ch; ++c) {
+      const int st = c & 1, n = t_end - t_begin - c * SC_L;
+      float raw[4], d[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) raw[e] = next[e];
+      request(c + 1, next);                     // a chunk ahead: nothing of a projection row is in a cache
+      double l[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        d[e] = 4 * lane + e < n ? softplus_f(raw[e] + bias) : 0.f;
+        l[e] = -static_cast<double>(A) * d[e] * 1.4426950408889634 + (e > 0 ? l[e - 1] : 0.0);
+      }
+      double run = l[3];
+#pragma unroll
+      for (int o = 1; o < 32; o <<= 1) {
+        const double up = __shfl_up_sync(0xffffffffu, run, o);
+        if (lane >= o) run += up;
+      }
+      const double total = __shfl_sync(0xffffffffu, run, 31), before = run - l[3];
+      if (ok) ok = mbar_wait_warp(&sums_empty[st], ((c >> 1) & 1) ^ 1);
+      ScanSums& s = sums[st];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int j = 4 * lane + e;
+        const double v = before + l[e];
+        const float hi = static_cast<float>(v);
+        s.dt[j] = d[e];
+        s.hi[j] = hi;
+        s.lo[j] = static_cast<float>(v - static_cast<double>(hi));
+        s.last[j] = exp2f(static_cast<float>(total - v)) * d[e];
+        s.grow[j] = exp2f(hi);
+      }
+      if (lane == 0) s.keep = exp2f(static_cast<float>(total));
+      mbar_arrive(&sums_full[st]);
+    }
+  }
+  if (!ok) {
+    report_error(p.status, TW_ERR_MBAR_TIMEOUT);
+    *abort_flag = 1;
+  }
+
+  if (*abort_flag) {
+    // let copies and MMAs in flight land before shared memory and TMEM are given back
+    const uint64_t t0 = globaltimer_ns();
+    while (globaltimer_ns() - t0 < 200000ull) __nanosleep(1000);
+  }
+  tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after_sync();
+    tmem_dealloc(tmem_base, TMEM_COLS);
+  }
+}
+
+// Called by tw_ssd_chunk for states of up to 128 dimensions. BC: base of [B groups | C groups] in the rows.
+int launch_ssd_chunk_tc(const void* xbc, long long ldx, int T, const void* dt, long long ldt, const void* dt_bias,
+                        const void* A_log, const void* D, float* state, void* y, long long ldy, const int* seqs,
+                        int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads, int vdim, int N,
+                        int groups, uint32_t* status, cudaStream_t stream) {
+  using bf = __nv_bfloat16;
+  CUtensorMap tmX, tmBC;
+  {
+    uint64_t dims[3] = {(uint64_t)vdim, (uint64_t)heads, (uint64_t)T};
+    uint64_t strides[2] = {(uint64_t)vdim * 2, (uint64_t)ldx * 2};
+    uint32_t box[3] = {64, 1, SC_L};
+    if (!make_tensor_map_bf16(&tmX, xbc, 3, dims, strides, box)) return 1;
+  }
+  {
+    uint64_t dims[3] = {(uint64_t)N, (uint64_t)groups * 2, (uint64_t)T};
+    uint64_t strides[2] = {(uint64_t)N * 2, (uint64_t)ldx * 2};
+    uint32_t box[3] = {64, 1, SC_L};
+    if (!make_tensor_map_bf16(&tmBC, reinterpret_cast<const bf*>(xbc) + static_cast<long long>(heads) * vdim, 3, dims,
+                              strides, box))
+      return 1;
+  }
+  static thread_local int configured_dev = -1;
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (configured_dev != dev) {
+    const cudaError_t e = cudaFuncSetAttribute(ssd_chunk_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SC_SMEM);
+    if (e != cudaSuccess) {
+      set_last_error("ssd_chunk (tcgen05): cudaFuncSetAttribute(smem=%d) failed: %s", SC_SMEM, cudaGetErrorString(e));
+      return 1;
+    }
+    configured_dev = dev;
+  }
+  const ScanTcParams p{reinterpret_cast<const bf*>(dt), ldt, reinterpret_cast<const bf*>(dt_bias),
+                       reinterpret_cast<const bf*>(A_log), reinterpret_cast<const bf*>(D), state,
+                       reinterpret_cast<bf*>(y), ldy, seqs, cu_q, kv_lens, slots, heads, vdim, N, groups, (N + 63) / 64,
+                       status};
+  ssd_chunk_tc_kernel<<<dim3(n_seqs, heads, (vdim + SC_P - 1) / SC_P), SC_THREADS, SC_SMEM, stream>>>(tmX, tmBC, p);
+  const cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) {
+    set_last_error("ssd_chunk (tcgen05) launch failed: %s", cudaGetErrorString(e));
+    return 1;
+  }
+  return 0;
+}
+
+}  // namespace tw

@@ -9,6 +9,17 @@
 
 namespace tw {
 
+// Waits of such a warp: every lane gets the same answer, so the warp stays converged whatever the outcome.
+__device__ __forceinline__ bool mbar_wait_warp(uint64_t* bar, uint32_t parity) {
+  return __all_sync(0xffffffffu, mbar_wait(bar, parity));
+}
+__device__ __forceinline__ bool mbar_try_wait_warp(uint64_t* bar, uint32_t parity) {
+  return __all_sync(0xffffffffu, mbar_try_wait(bar, parity));
+}
+__device__ __forceinline__ bool mbar_test_warp(uint64_t* bar, uint32_t parity) {
+  return __all_sync(0xffffffffu, mbar_test(bar, parity));
+}
+
 __device__ __forceinline__ void umma_ss_e(uint32_t d_tmem, uint64_t a_desc, uint64_t b_desc, uint32_t idesc,
                                         uint32_t accumulate) {
   asm volatile(

@@ -184,7 +184,7 @@ int tw_latent_prefill(const void* q, long long ldq, int T, const void* kv, long 
 int tw_latent_gather(const void* cache, void* dst, const int* seqs, const int* cu, int n_seqs, int max_rows,
                      const int* block_table, int max_blocks, int page, int row_bytes, cudaStream_t stream);
 
-// ---- state-space recurrence (ssm.cu, ssd_chunk.cu) ----
+// ---- state-space recurrence (ssm.cu, ssd_chunk.cu, ssd_chunk_tc.cu) ----
 int tw_causal_conv(const void* x, long long ldx, const void* w, const void* bias, void* state, void* out, long long ldo,
                    const int* row_seq, const int* cu_q, const int* kv_lens, const int* slots, int T, int n_seqs,
                    int channels, int taps, int single, int dtype, cudaStream_t stream);
@@ -192,9 +192,10 @@ int tw_ssd_scan(const void* xbc, long long ldx, const void* dt, long long ldt, c
                 const void* D, float* state, void* y, long long ldy, const int* seqs, int n_seqs, const int* cu_q,
                 const int* kv_lens, const int* slots, int heads, int vdim, int N, int groups, int dtype,
                 cudaStream_t stream);
-int tw_ssd_chunk(const void* xbc, long long ldx, const void* dt, long long ldt, const void* dt_bias, const void* A_log,
-                 const void* D, float* state, void* y, long long ldy, const int* seqs, int n_seqs, const int* cu_q,
-                 const int* kv_lens, const int* slots, int heads, int vdim, int N, int groups, cudaStream_t stream);
+int tw_ssd_chunk(const void* xbc, long long ldx, int T, const void* dt, long long ldt, const void* dt_bias,
+                 const void* A_log, const void* D, float* state, void* y, long long ldy, const int* seqs, int n_seqs,
+                 const int* cu_q, const int* kv_lens, const int* slots, int heads, int vdim, int N, int groups, int form,
+                 uint32_t* status, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

@@ -78,7 +78,7 @@ _SIGNATURES = {
     "tw_latent_gather": [vp, vp, vp, vp, i32, i32, vp, i32, i32, i32, vp],
     "tw_causal_conv": [vp, ll, vp, vp, vp, vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
     "tw_ssd_scan": [vp, ll, vp, ll, vp, vp, vp, vp, vp, ll, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, vp],
-    "tw_ssd_chunk": [vp, ll, vp, ll, vp, vp, vp, vp, vp, ll, vp, i32, vp, vp, vp, i32, i32, i32, i32, vp],
+    "tw_ssd_chunk": [vp, ll, i32, vp, ll, vp, vp, vp, vp, vp, ll, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
 }
 
 

@@ -254,12 +254,14 @@ def ssd_chunkable(dtype: torch.dtype, vdim: int, N: int) -> bool:
 
 def ssd_chunk(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor,
               state: torch.Tensor, y: torch.Tensor, seqs: torch.Tensor, cu_q: torch.Tensor, kv_lens: torch.Tensor,
-              slots: torch.Tensor, groups: int) -> None:
-    """:func:`ssd_scan` for long runs: 64 tokens at a time on the tensor cores (CUDA, bf16)."""
+              slots: torch.Tensor, groups: int, form: int = 0) -> None:
+    """:func:`ssd_scan` for long runs, many tokens at a time on the tensor cores (CUDA, bf16). ``form`` 0: tcgen05 in
+    chunks of 128 for states of up to 128 dimensions, warp-level products in chunks of 64 beyond; 1: always the latter."""
     if seqs.shape[0] == 0:
         return
     _, heads, vdim, N = state.shape
     assert state.dtype == torch.float32 and _dt(xbc, dt, dt_bias, A_log, D, y) == 0
-    _native.call("tw_ssd_chunk", xbc.data_ptr(), _row_stride(xbc), dt.data_ptr(), _row_stride(dt), dt_bias.data_ptr(),
+    _native.call("tw_ssd_chunk", xbc.data_ptr(), _row_stride(xbc), xbc.shape[0], dt.data_ptr(), _row_stride(dt), dt_bias.data_ptr(),
                  A_log.data_ptr(), D.data_ptr(), state.data_ptr(), y.data_ptr(), _row_stride(y), seqs.data_ptr(),
-                 seqs.shape[0], cu_q.data_ptr(), kv_lens.data_ptr(), slots.data_ptr(), heads, vdim, N, groups, _stream())
+                 seqs.shape[0], cu_q.data_ptr(), kv_lens.data_ptr(), slots.data_ptr(), heads, vdim, N, groups, form,
+                 status_word(xbc.device).data_ptr(), _stream())
