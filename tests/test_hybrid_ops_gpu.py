@@ -88,7 +88,7 @@ def paged(lens, page, row, dtype, spare=3, scale=1.0):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("q_rank,kv_rank,rot,rot_dims", [(24, 40, 16, 16), (50, 37, 12, 8), (1536, 512, 64, 64)])
+@pytest.mark.parametrize("q_rank,kv_rank,rot,rot_dims", [(24, 40, 16, 16), (50, 37, 12, 8), (1536, 512, 64, 64), (3001, 600, 20, 20)])
 def test_latent_prep_and_absorb(dtype, q_rank, kv_rank, rot, rot_dims):
     T, heads, dim, page = 9, 3, 20, 8
     p8 = lambda n: (n + 7) // 8 * 8

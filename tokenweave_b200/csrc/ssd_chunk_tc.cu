@@ -12,9 +12,12 @@
 //
 // Roles (480 threads): warp 0 TMA producer, warp 1 MMA issuer, warps 2..5 and 6..9 scores (thread = token, each group half
 // of the keys) and epilogue (each group half of vdim), warps 10..13 state (thread = state row) and W (thread = token),
-// warp 14 running sums. G is double-buffered in tensor memory, so that the scores of a chunk are made while the products of
-// the one before run. All waits are bounded; after a timeout the roles keep their trip counts (the named barriers of the
-// score warps are not bounded), skip further waits, report TW_ERR_MBAR_TIMEOUT and leave through the tear-down.
+// warp 14 running sums. G and Y2 are double-buffered in tensor memory, so that the scores of a chunk are made while the
+// products of the one before run. All waits are bounded; after a timeout a role skips further waits, and the CTA reports
+// TW_ERR_MBAR_TIMEOUT and leaves through its tear-down.
+//
+// Five kinds of warps run at the same time, so the loops are kept rolled where registers allow: with everything unrolled
+// the roles' code did not fit the instruction caches, and 128 CTAs took 1.5 times as long as 64 of them.
 #include "attn_prefill_common.cuh"
 #include "tw_elect.cuh"
 #include "tw_host.h"
@@ -26,6 +29,7 @@ namespace tw {
 
 constexpr int SC_L = 128;                          // tokens per chunk
 constexpr int SC_P = 64;                           // rows of vdim per CTA
+constexpr int SC_AHEAD = 3;                        // chunks on their way to L2
 constexpr int SC_THREADS = 480;
 constexpr int SC_CHUNK = SC_L * 128;               // 128 rows x 64 bf16, swizzled
 
@@ -39,9 +43,9 @@ struct ScanTcParams {
   uint32_t* status;
 };
 
-// Running sums of a chunk in base 2: hi + lo = l log2(e) to two floats.
+// Running sums of a chunk in base 2, negated: nhi + nlo = -l log2(e) to two floats.
 struct ScanSums {
-  float dt[SC_L], hi[SC_L], lo[SC_L], last[SC_L], grow[SC_L];      // last: exp(l_last - l) dt, grow: exp(l)
+  float dt[SC_L], nhi[SC_L], nlo[SC_L], last[SC_L], grow[SC_L];      // last: exp(l_last - l) dt, grow: exp(l)
   float keep, pad[3];                                              // exp(l_last)
 };
 
@@ -54,6 +58,9 @@ constexpr int SC_OFF_SUMS = SC_OFF_W + 2 * SC_CHUNK;
 constexpr int SC_OFF_BAR = SC_OFF_SUMS + 2 * static_cast<int>(sizeof(ScanSums));
 constexpr int SC_SMEM = SC_OFF_BAR + 256 + 1024;
 
+// (a call: one copy of it in the kernel)
+__device__ __noinline__ float softplus_call(float x) { return softplus_f(x); }
+
 // Column c (of 64) of row r of a swizzled tile with 128-byte rows: byte offset of its 16-byte group.
 __device__ __forceinline__ uint32_t sw_off(int r, int group) { return r * 128 + ((group ^ (r & 7)) * 16); }
 
@@ -64,19 +71,20 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
   constexpr uint32_t IDESC_Y = make_idesc_bf16(128, 64, 0, 1);      // A = C or M, B operand = S or X (MN-major)
   constexpr uint32_t IDESC_S = make_idesc_bf16(128, 64, 1, 1);      // A = B^T (MN-major), B operand = W (MN-major)
   constexpr uint32_t TMEM_COLS = 512;
-  constexpr uint32_t COL_G = 0, COL_Y1 = 256, COL_Y2 = 320, COL_DS = 384;      // G: two buffers of 128
+  constexpr uint32_t COL_G = 0, COL_Y1 = 256, COL_DS = 320, COL_Y2 = 384;      // two buffers of G (128 columns) and Y2
 
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) &
                                              ~static_cast<uintptr_t>(1023));
   ScanSums* sums = reinterpret_cast<ScanSums*>(smem + SC_OFF_SUMS);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + SC_OFF_BAR);
-  uint64_t *c_full = bars, *c_empty = bars + 1, *bx_full = bars + 2, *bx_empty = bars + 4;
+  uint64_t *c_full = bars, *c_empty = bars + 1, *b_full = bars + 2, *b_empty = bars + 4;
   uint64_t *sums_full = bars + 6, *sums_empty = bars + 8;
   uint64_t *g_full = bars + 10, *m_ready = bars + 11;
   uint64_t *s_ready = bars + 12, *s_free = bars + 13, *w_ready = bars + 14, *ds_full = bars + 15, *ds_read = bars + 16;
   uint64_t *y_full = bars + 17, *y_free = bars + 18;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 19);
+  uint64_t *x_full = bars + 19, *x_empty = bars + 21;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 23);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -90,8 +98,10 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
     mbar_init(c_full, 1);
     mbar_init(c_empty, 1);
     for (int i = 0; i < 2; ++i) {
-      mbar_init(&bx_full[i], 1);
-      mbar_init(&bx_empty[i], 1 + 128 + 256);
+      mbar_init(&b_full[i], 1);
+      mbar_init(&b_empty[i], 1);
+      mbar_init(&x_full[i], 1);
+      mbar_init(&x_empty[i], 1 + 128 + 256);
       mbar_init(&sums_full[i], 32);
       mbar_init(&sums_empty[i], 128 + 256);
     }
@@ -119,17 +129,32 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
 
   if (warp == 0) {
     // ---------------- TMA producer (uniform over the warp) ----------------
+    // Chunks travel to L2 ahead of the buffers: a copy is issued when its buffer is free, by then its bytes should not be
+    // in DRAM any more.
+    auto prefetch = [&](int c) {
+      if (c >= n_ch) return;
+      const int t0 = t_begin + c * SC_L;
+      tma_prefetch_3d_e(&tmX, p0, h, t0);
+      for (int k = 0; k < p.n_chunks; ++k) {
+        tma_prefetch_3d_e(&tmBC, k * 64, g, t0);
+        tma_prefetch_3d_e(&tmBC, k * 64, p.groups + g, t0);
+      }
+    };
+    for (int c = 1; c < SC_AHEAD; ++c) prefetch(c);
     for (int c = 0; ok && c < n_ch; ++c) {
       const int st = c & 1, t0 = t_begin + c * SC_L;
-      if (!mbar_wait_warp(&bx_empty[st], ((c >> 1) & 1) ^ 1)) { ok = false; break; }
-      mbar_expect_tx_e(&bx_full[st], (p.n_chunks + 1) * SC_CHUNK);
+      prefetch(c + SC_AHEAD);
+      if (!mbar_wait_warp(&b_empty[st], ((c >> 1) & 1) ^ 1)) { ok = false; break; }
+      mbar_expect_tx_e(&b_full[st], p.n_chunks * SC_CHUNK);
       for (int k = 0; k < p.n_chunks; ++k)
-        tma_load_3d_e(smem + SC_OFF_B + (2 * st + k) * SC_CHUNK, &tmBC, &bx_full[st], k * 64, g, t0);
-      tma_load_3d_e(smem + SC_OFF_X + st * SC_CHUNK, &tmX, &bx_full[st], p0, h, t0);
+        tma_load_3d_e(smem + SC_OFF_B + (2 * st + k) * SC_CHUNK, &tmBC, &b_full[st], k * 64, g, t0);
       if (!mbar_wait_warp(c_empty, (c & 1) ^ 1)) { ok = false; break; }
       mbar_expect_tx_e(c_full, p.n_chunks * SC_CHUNK);
       for (int k = 0; k < p.n_chunks; ++k)
         tma_load_3d_e(smem + SC_OFF_C + k * SC_CHUNK, &tmBC, c_full, k * 64, p.groups + g, t0);
+      if (!mbar_wait_warp(&x_empty[st], ((c >> 1) & 1) ^ 1)) { ok = false; break; }
+      mbar_expect_tx_e(&x_full[st], SC_CHUNK);
+      tma_load_3d_e(smem + SC_OFF_X + st * SC_CHUNK, &tmX, &x_full[st], p0, h, t0);
     }
   } else if (warp == 1) {
     // ---------------- MMA issuer (uniform over the warp) ----------------
@@ -141,7 +166,7 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
     const uint64_t d_w = make_smem_desc_sw128(smem_u32(smem + SC_OFF_W), SC_CHUNK, 1024);
     constexpr int K_ROWS = 16 * 128 / 16;        // 16 rows of an MN-major tile, in descriptor units
     auto issue_g = [&](int c) {
-      if (!mbar_wait_warp(c_full, c & 1) || !mbar_wait_warp(&bx_full[c & 1], (c >> 1) & 1)) return false;
+      if (!mbar_wait_warp(c_full, c & 1) || !mbar_wait_warp(&b_full[c & 1], (c >> 1) & 1)) return false;
       tc_fence_after_sync();
       const uint64_t db = d_b + (c & 1) * (2 * SC_CHUNK / 16);
       for (int q = 0; q < p.n_chunks; ++q) {
@@ -157,14 +182,14 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
     for (int c = 0; ok && c < n_ch; ++c) {
       const int st = c & 1;
       // Y2: the state before the chunk
-      if (!mbar_wait_warp(s_ready, c & 1) || !mbar_wait_warp(y_free, (c & 1) ^ 1)) { ok = false; break; }
+      if (!mbar_wait_warp(s_ready, c & 1)) { ok = false; break; }
       tc_fence_after_sync();
       for (int q = 0; q < p.n_chunks; ++q) {
 #pragma unroll
         for (int k = 0; k < 4; ++k) {
           const uint64_t da = d_c + q * (SC_CHUNK / 16) + k * 2, db = d_s + (q * 4 + k) * K_ROWS;
-          umma_ss_e(tmem_base + COL_Y2, da, db, IDESC_Y, (q | k) != 0 ? 1u : 0u);
-          umma_ss_e(tmem_base + COL_Y2, da, db + SC_CHUNK / 16, IDESC_Y, 1u);
+          umma_ss_e(tmem_base + COL_Y2 + st * 64, da, db, IDESC_Y, (q | k) != 0 ? 1u : 0u);
+          umma_ss_e(tmem_base + COL_Y2 + st * 64, da, db + SC_CHUNK / 16, IDESC_Y, 1u);
         }
       }
       umma_commit_e(c_empty);
@@ -174,31 +199,38 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
       tc_fence_after_sync();
       {
         const uint64_t da = d_bt + st * (2 * SC_CHUNK / 16);
-#pragma unroll
+#pragma unroll 2
         for (int k = 0; k < 8; ++k) {
           umma_ss_e(tmem_base + COL_DS, da + k * K_ROWS, d_w + k * K_ROWS, IDESC_S, k != 0 ? 1u : 0u);
           umma_ss_e(tmem_base + COL_DS, da + k * K_ROWS, d_w + SC_CHUNK / 16 + k * K_ROWS, IDESC_S, 1u);
         }
       }
       umma_commit_e(ds_full);
+      umma_commit_e(&b_empty[st]);
       // the next chunk's scores, then this chunk's weighted scores times X
       if (c + 1 < n_ch) {
         ok = issue_g(c + 1);
         if (!ok) break;
       }
-      if (!mbar_wait_warp(m_ready, c & 1)) { ok = false; break; }
+      // (y_free also says that Y2 of the chunk before is read: the next Y2 but one may overwrite it)
+      if (!mbar_wait_warp(m_ready, c & 1) || !mbar_wait_warp(y_free, (c & 1) ^ 1) ||
+          !mbar_wait_warp(&x_full[st], (c >> 1) & 1)) {
+        ok = false;
+        break;
+      }
       tc_fence_after_sync();
       {
         const uint32_t m = tmem_base + COL_G + st * 128;
         const uint64_t dx = d_x + st * (SC_CHUNK / 16);
-#pragma unroll
+#pragma unroll 2
         for (int k = 0; k < 8; ++k) {
-          umma_ts_e(tmem_base + COL_Y1, m + k * 8, dx + k * K_ROWS, IDESC_Y, k != 0 ? 1u : 0u);
-          umma_ts_e(tmem_base + COL_Y1, m + 64 + k * 8, dx + k * K_ROWS, IDESC_Y, 1u);
+          const uint32_t mk = m + k * 16;
+          umma_ts_e(tmem_base + COL_Y1, mk, dx + k * K_ROWS, IDESC_Y, k != 0 ? 1u : 0u);
+          umma_ts_e(tmem_base + COL_Y1, mk + 8, dx + k * K_ROWS, IDESC_Y, 1u);
         }
       }
       umma_commit_e(y_full);
-      umma_commit_e(&bx_empty[st]);
+      umma_commit_e(&x_empty[st]);
     }
   } else if (warp < 10) {
     // ---------------- scores and epilogue ----------------
@@ -212,76 +244,78 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
       tc_fence_after_sync();
       const float e = sums[st].grow[r];
       const int t = t_begin + c * SC_L + r;
-      uint32_t a[32], s[32];
-      tmem_ld_32x32(t_lane + COL_Y1 + grp * 32, a);
-      tmem_ld_32x32(t_lane + COL_Y2 + grp * 32, s);
-      tmem_wait_ld();
+      const uint8_t* xr = smem + SC_OFF_X + st * SC_CHUNK;
+#pragma unroll 1
+      for (int v = 0; v < 2; ++v) {
+        uint32_t a[16], s[16];
+        tmem_ld_32x16(t_lane + COL_Y1 + grp * 32 + v * 16, a);
+        tmem_ld_32x16(t_lane + COL_Y2 + st * 64 + grp * 32 + v * 16, s);
+        tmem_wait_ld();
+#pragma unroll
+        for (int w = 0; w < 2; ++w) {
+          const int p8 = grp * 4 + v * 2 + w;
+          float x[8];
+          ld8(reinterpret_cast<const __nv_bfloat16*>(xr + sw_off(r, p8)), x);
+#pragma unroll
+          for (int i = 0; i < 8; ++i)
+            x[i] = fmaf(D, x[i], fmaf(e, __uint_as_float(s[8 * w + i]), __uint_as_float(a[8 * w + i])));
+          if (ok && t < t_end && p8 * 8 < p_valid) st8(p.y + t * p.ldy + h * p.vdim + p0 + p8 * 8, x);
+        }
+      }
       tc_fence_before_sync();
       mbar_arrive(y_free);
-      const uint8_t* xr = smem + SC_OFF_X + st * SC_CHUNK;
-#pragma unroll
-      for (int v = 0; v < 4; ++v) {
-        const int p8 = grp * 4 + v;
-        float x[8];
-        ld8(reinterpret_cast<const __nv_bfloat16*>(xr + sw_off(r, p8)), x);
-#pragma unroll
-        for (int i = 0; i < 8; ++i)
-          x[i] = fmaf(D, x[i], fmaf(e, __uint_as_float(s[8 * v + i]), __uint_as_float(a[8 * v + i])));
-        if (ok && t < t_end && p8 * 8 < p_valid) st8(p.y + t * p.ldy + h * p.vdim + p0 + p8 * 8, x);
-      }
-      mbar_arrive(&bx_empty[st]);
+      mbar_arrive(&x_empty[st]);
       mbar_arrive(&sums_empty[st]);
     };
-    for (int c = 0; c < n_ch; ++c) {
-      const int st = c & 1;
-      if (ok) ok = mbar_wait(&sums_full[st], (c >> 1) & 1);
-      if (ok) ok = mbar_wait(g_full, c & 1);
-      tc_fence_after_sync();
-      const uint32_t t_g = t_lane + COL_G + st * 128;
-      uint32_t s0[32], s1[32];
-      tmem_ld_32x32(t_g + grp * 64, s0);
-      tmem_ld_32x32(t_g + grp * 64 + 32, s1);
-      tmem_wait_ld();
-      // the other group's half is overwritten below: both have to be in registers first
-      tc_fence_before_sync();
-      split_pair_sync(qr);
-      tc_fence_after_sync();
-      const ScanSums& sm = sums[st];
-      const float hi_i = sm.hi[r], lo_i = sm.lo[r];
-      auto half = [&](const uint32_t (&sc)[32], int j0, uint32_t col) {
-        uint32_t mh[16], ml[16];
-        if (j0 > qr * 32 + 31) {                                // warp-uniform: every key is behind every token
+    for (int c = 0; c <= n_ch; ++c) {           // one place for each part: the code of all roles has to stay small
+      if (c < n_ch) {
+        const int st = c & 1;
+        if (ok) ok = mbar_wait(&sums_full[st], (c >> 1) & 1);
+        if (ok) ok = mbar_wait(g_full, c & 1);
+        tc_fence_after_sync();
+        // 16 keys at a time; their M (eight columns of hi terms, eight of lo terms) takes the place of their scores
+        const ScanSums& sm = sums[st];
+        const float2 hi_i = make_float2(-sm.nhi[r], -sm.nhi[r]), lo_i = make_float2(-sm.nlo[r], -sm.nlo[r]);
+#pragma unroll 1
+        for (int q = 0; q < 4; ++q) {
+          const int j0 = grp * 64 + q * 16;
+          const uint32_t t_g = t_lane + COL_G + st * 128 + j0;
+          uint32_t m[16];
+          if (j0 > qr * 32 + 31) {                              // warp-uniform: every key is behind every token
 #pragma unroll
-          for (int i = 0; i < 16; ++i) mh[i] = ml[i] = 0u;
-        } else {
+            for (int i = 0; i < 16; ++i) m[i] = 0u;
+          } else {
+            const int lim = r - j0;                             // keys behind the token get no weight
+            uint32_t sc[16];
+            tmem_ld_32x16(t_g, sc);
+            tmem_wait_ld();
 #pragma unroll
-          for (int i = 0; i < 16; i += 2) {
-            const float4 hj = *reinterpret_cast<const float4*>(sm.hi + j0 + 2 * i);
-            const float4 lj = *reinterpret_cast<const float4*>(sm.lo + j0 + 2 * i);
-            const float4 d = *reinterpret_cast<const float4*>(sm.dt + j0 + 2 * i);
-            float w[4];
-            w[0] = __uint_as_float(sc[2 * i]) * (fast_exp2((hi_i - hj.x) + (lo_i - lj.x)) * d.x);
-            w[1] = __uint_as_float(sc[2 * i + 1]) * (fast_exp2((hi_i - hj.y) + (lo_i - lj.y)) * d.y);
-            w[2] = __uint_as_float(sc[2 * i + 2]) * (fast_exp2((hi_i - hj.z) + (lo_i - lj.z)) * d.z);
-            w[3] = __uint_as_float(sc[2 * i + 3]) * (fast_exp2((hi_i - hj.w) + (lo_i - lj.w)) * d.w);
-#pragma unroll
-            for (int e = 0; e < 4; ++e)
-              if (j0 + 2 * i + e > r) w[e] = 0.f;
-            split_bf16x2(w[0], w[1], mh[i], ml[i]);
-            split_bf16x2(w[2], w[3], mh[i + 1], ml[i + 1]);
+            for (int i = 0; i < 8; i += 2) {
+              const float4 hj = *reinterpret_cast<const float4*>(sm.nhi + j0 + 2 * i);
+              const float4 lj = *reinterpret_cast<const float4*>(sm.nlo + j0 + 2 * i);
+              const float4 d = *reinterpret_cast<const float4*>(sm.dt + j0 + 2 * i);
+              float2 u = fadd2(fadd2(hi_i, make_float2(hj.x, hj.y)), fadd2(lo_i, make_float2(lj.x, lj.y)));
+              float2 v = fadd2(fadd2(hi_i, make_float2(hj.z, hj.w)), fadd2(lo_i, make_float2(lj.z, lj.w)));
+              u = mul2(make_float2(fast_exp2(u.x), fast_exp2(u.y)), make_float2(d.x, d.y));
+              v = mul2(make_float2(fast_exp2(v.x), fast_exp2(v.y)), make_float2(d.z, d.w));
+              u = mul2(u, make_float2(__uint_as_float(sc[2 * i]), __uint_as_float(sc[2 * i + 1])));
+              v = mul2(v, make_float2(__uint_as_float(sc[2 * i + 2]), __uint_as_float(sc[2 * i + 3])));
+              if (2 * i > lim) u.x = 0.f;
+              if (2 * i + 1 > lim) u.y = 0.f;
+              if (2 * i + 2 > lim) v.x = 0.f;
+              if (2 * i + 3 > lim) v.y = 0.f;
+              split_bf16x2(u.x, u.y, m[i], m[8 + i]);
+              split_bf16x2(v.x, v.y, m[i + 1], m[9 + i]);
+            }
           }
+          tmem_st_32x16(t_g, m);
         }
-        tmem_st_32x16(t_g + col, mh);
-        tmem_st_32x16(t_g + 64 + col, ml);
-      };
-      half(s0, grp * 64, grp * 32);
-      half(s1, grp * 64 + 32, grp * 32 + 16);
-      tmem_wait_st();
-      tc_fence_before_sync();
-      mbar_arrive(m_ready);          // arrive even after a failed wait so that the issuer is not left waiting
+        tmem_wait_st();
+        tc_fence_before_sync();
+        mbar_arrive(m_ready);        // arrive even after a failed wait so that the issuer is not left waiting
+      }
       if (c > 0) epilogue(c - 1);
     }
-    if (n_ch > 0) epilogue(n_ch - 1);
   } else if (warp < 14) {
     // ---------------- state and weighted inputs ----------------
     const int qr = warp & 3;
@@ -311,11 +345,11 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
       mbar_arrive(s_ready);
       // W (free: the products of the previous chunk were waited for below)
       if (ok) ok = mbar_wait(&sums_full[st], (c >> 1) & 1);
-      if (ok) ok = mbar_wait(&bx_full[st], (c >> 1) & 1);
+      if (ok) ok = mbar_wait(&x_full[st], (c >> 1) & 1);
       const float w = sums[st].last[r], keep = sums[st].keep;
       const uint8_t* xr = smem + SC_OFF_X + st * SC_CHUNK;
       uint8_t* w_hi = smem + SC_OFF_W;
-#pragma unroll
+#pragma unroll 2
       for (int v = 0; v < 8; ++v) {
         float x[8];
         ld8(reinterpret_cast<const __nv_bfloat16*>(xr + sw_off(r, v)), x);
@@ -329,7 +363,7 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
       }
       fence_proxy_async_smem();
       mbar_arrive(w_ready);
-      mbar_arrive(&bx_empty[st]);
+      mbar_arrive(&x_empty[st]);
       mbar_arrive(&sums_empty[st]);
       if (ok) ok = mbar_wait(ds_full, c & 1);
       tc_fence_after_sync();
@@ -360,6 +394,7 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
         raw[e] = t < t_end ? ld1(p.dt + t * p.ldt + h) : 0.f;
       }
     };
+    const double rate = -static_cast<double>(A) * 1.4426950408889634;
     float next[4];
     request(0, next);
     for (int c = 0; c < n_ch; ++c) {
@@ -371,30 +406,35 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
       double l[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        d[e] = 4 * lane + e < n ? softplus_f(raw[e] + bias) : 0.f;
-        l[e] = -static_cast<double>(A) * d[e] * 1.4426950408889634 + (e > 0 ? l[e - 1] : 0.0);
+        d[e] = 4 * lane + e < n ? softplus_call(raw[e] + bias) : 0.f;
+        l[e] = rate * d[e] + (e > 0 ? l[e - 1] : 0.0);
       }
       double run = l[3];
-#pragma unroll
+#pragma unroll 1
       for (int o = 1; o < 32; o <<= 1) {
         const double up = __shfl_up_sync(0xffffffffu, run, o);
         if (lane >= o) run += up;
       }
       const double total = __shfl_sync(0xffffffffu, run, 31), before = run - l[3];
-      if (ok) ok = mbar_wait_warp(&sums_empty[st], ((c >> 1) & 1) ^ 1);
-      ScanSums& s = sums[st];
+      float4 nhi, nlo, last, grow;
+      float *ph = &nhi.x, *pl = &nlo.x, *pt = &last.x, *pg = &grow.x;
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int j = 4 * lane + e;
         const double v = before + l[e];
         const float hi = static_cast<float>(v);
-        s.dt[j] = d[e];
-        s.hi[j] = hi;
-        s.lo[j] = static_cast<float>(v - static_cast<double>(hi));
-        s.last[j] = exp2f(static_cast<float>(total - v)) * d[e];
-        s.grow[j] = exp2f(hi);
+        ph[e] = -hi;
+        pl[e] = static_cast<float>(static_cast<double>(hi) - v);
+        pt[e] = fast_exp2(static_cast<float>(total - v)) * d[e];
+        pg[e] = fast_exp2(hi);
       }
-      if (lane == 0) s.keep = exp2f(static_cast<float>(total));
+      if (ok) ok = mbar_wait_warp(&sums_empty[st], ((c >> 1) & 1) ^ 1);
+      ScanSums& s = sums[st];
+      *reinterpret_cast<float4*>(s.dt + 4 * lane) = make_float4(d[0], d[1], d[2], d[3]);
+      *reinterpret_cast<float4*>(s.nhi + 4 * lane) = nhi;
+      *reinterpret_cast<float4*>(s.nlo + 4 * lane) = nlo;
+      *reinterpret_cast<float4*>(s.last + 4 * lane) = last;
+      *reinterpret_cast<float4*>(s.grow + 4 * lane) = grow;
+      if (lane == 0) s.keep = fast_exp2(static_cast<float>(total));
       mbar_arrive(&sums_full[st]);
     }
   }

@@ -24,8 +24,8 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
 // hi + lo = (x, y) to 16 bits of mantissa
 __device__ __forceinline__ void split_bf16x2(float x, float y, uint32_t& hi, uint32_t& lo) {
   hi = pack_bf16x2(x, y);
-  const float2 h = unpack_bf16x2(hi);
-  lo = pack_bf16x2(x - h.x, y - h.y);
+  const float2 l = fma2(unpack_bf16x2(hi), make_float2(-1.f, -1.f), make_float2(x, y));
+  lo = pack_bf16x2(l.x, l.y);
 }
 
 // Element offsets of a lane's row for ldmatrix.x4 out of a row-major tile with row stride `ld`:
