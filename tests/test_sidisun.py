@@ -4,7 +4,6 @@ GPU, in true fp32 and in bf16."""
 import json
 import os
 import subprocess
-import sys
 
 import numpy as np
 import pytest

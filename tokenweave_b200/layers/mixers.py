@@ -12,12 +12,11 @@ decays and recurrent state are fp32 in both.
 """
 from __future__ import annotations
 
-from typing import Iterable, Optional
+from typing import Optional
 
 import torch
 from torch import nn
 
-from .. import ops
 from ..ops import hybrid as hops
 from ..ops import reference
 from .attention import AttentionMetadata
