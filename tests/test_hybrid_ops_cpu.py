@@ -110,10 +110,10 @@ def test_row_routing():
                      max_model_len=512).create_engine_config()
     model = HybridDecoder(cfg.model, device="cpu")
     model.setup_runtime(512, cfg.tokenweave)
-    model.expand, model.rt.context_rows = True, 600
+    model.tiles, model.rt.context_rows = True, 600
     q = [1, 64, 16, 40, 200, 20]
     kv = [300, 64, 30, 500, 400, 200]
-    (tile_seq, tile_q0, tok_row, tok_seq, tok_kv), extra, host = model.plan_step(q, kv, list(range(6)))
+    (tile_seq, tile_q0, tok_row, tok_seq, tok_kv), extra, host = model.plan_step(q, kv, list(range(6)), [-1] * 6)
     tiled = sorted(set(tile_seq))
     assert tiled == [1, 2, 4] and host == {"ctx_rows": 494, "ctx_max": 400}
     assert list(extra["ctx_begin"]) == [-1, 0, 64, -1, 94, -1] and list(extra["ctx_cu"]) == [0, 64, 94, 494]
@@ -124,6 +124,6 @@ def test_row_routing():
     assert list(tok_kv) == [kv[b] - q[b] + i + 1 for b, i in rows]
     assert list(extra["scan_seqs"]) == [0] and list(extra["chunk_seqs"]) == [1, 2, 3, 4, 5]
     model.rt.context_rows = 100                                      # the long context no longer fits
-    assert sorted(set(model.plan_step(q, kv, list(range(6)))[0][0])) == [1, 2]
-    plan, extra, _ = model.plan_step([1, 1], [5, 9], [1, 0])
+    assert sorted(set(model.plan_step(q, kv, list(range(6)), [-1] * 6)[0][0])) == [1, 2]
+    plan, extra, _ = model.plan_step([1, 1], [5, 9], [1, 0], [-1] * 2)
     assert list(plan[2]) == [0, 1] and list(plan[4]) == [5, 9] and list(extra["state_slots"]) == [1, 0]

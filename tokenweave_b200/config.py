@@ -21,8 +21,17 @@ _DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float32": torch.
            "float16": torch.float16, "half": torch.float16, "auto": None}
 
 
-# mixers of hybrid decoders that keep a state slot per sequence (layers/mixers.py)
-RECURRENT_MIXERS = ("mamba2",)
+# mixers, and parts of summed mixers, of hybrid decoders that keep a state slot per sequence (layers/mixers.py); a
+# short convolution in front of an attention keeps one too
+RECURRENT_MIXERS = ("mamba2", "lightning_attention")
+
+
+def _keeps_state(layer: dict) -> bool:
+    parts = layer["mixer"].get("parts", {}).values()
+    return layer["type"] in RECURRENT_MIXERS or any(
+        p["kind"] in RECURRENT_MIXERS or (p.get("options", {}).get("conv") or 1) > 1 for p in parts)
+
+
 # config.json's "architecture" -> reader(dict, name, path) -> ModelConfig, for designs not in the Hugging Face layout
 CONFIG_READERS: dict = {}
 
@@ -38,7 +47,7 @@ def register_config_reader(architecture: str):
 class ModelConfig:
     """Architecture of a decoder-only transformer (Llama-3.x, Qwen2.5, Mixtral layouts)."""
     name: str = "tiny-llama"
-    architecture: str = "llama"          # "llama" | "qwen2" | "mixtral" | "qwen3" | "mistral" | "phi3" | "sidisun"
+    architecture: str = "llama"          # "llama" | "qwen2" | "mixtral" | "qwen3" | "mistral" | "phi3" | "sidisun" | "kebopel"
     hidden_size: int = 256
     num_layers: int = 2
     num_q_heads: int = 4
@@ -69,11 +78,16 @@ class ModelConfig:
     # hybrid decoders (models/hybrid.py): one {"type", "mixer", "mlp"} per layer; None for the uniform families above
     layers: Optional[list] = None
     logit_scale: float = 1.0             # factor on the logits (hybrid decoders)
+    # hybrid decoders: how a layer adds to the residual stream ("output_norm" or "parallel"); layers start .. stop - 1
+    # run ``times`` times in a row ({"start", "stop", "times"}); pair embeddings ({"buckets", "mul_prev", "mul_cur"})
+    block: str = "output_norm"
+    loop: Optional[dict] = None
+    bigram: Optional[dict] = None
 
     @property
     def has_state(self) -> bool:
         """Some layer keeps recurrent state: a request holds a state slot besides its cache blocks."""
-        return any(l["type"] in RECURRENT_MIXERS for l in self.layers or ())
+        return any(_keeps_state(l) for l in self.layers or ())
 
     @property
     def is_moe(self) -> bool:
@@ -279,6 +293,9 @@ def resolve_model_config(model: "str | ModelConfig", dtype: Optional[str] = None
         if cfg.layers:
             cfg.layers = cfg.layers[:num_layers]
             cfg.num_layers = len(cfg.layers)
+            if cfg.loop:
+                stop = min(cfg.loop["stop"], cfg.num_layers)
+                cfg.loop = {**cfg.loop, "stop": stop} if cfg.loop["start"] < stop else None
     return cfg
 
 

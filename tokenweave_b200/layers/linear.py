@@ -197,15 +197,21 @@ class PaddedLinear(_QuantizableLinear):
     TMA-fed GEMM needs) with zeros, so ``x`` has ``in_padded`` columns whose pad is finite and the output's pad columns
     come out as zeros. Several projections of one input can share it, each written with :meth:`load_rows`."""
 
-    def __init__(self, in_features: int, out_features: int, *, dtype, device):
+    def __init__(self, in_features: int, out_features: int, bias: bool = False, *, dtype, device):
         super().__init__()
         self.in_features, self.out_features = in_features, out_features
         self.in_padded, self.out_padded = pad8(in_features), pad8(out_features)
         self.weight = nn.Parameter(torch.zeros(self.out_padded, self.in_padded, dtype=dtype, device=device),
                                    requires_grad=False)
+        self.bias = (nn.Parameter(torch.zeros(self.out_padded, dtype=dtype, device=device), requires_grad=False)
+                     if bias else None)
 
     def load_rows(self, t: torch.Tensor, row: int) -> None:
         self.weight.data[row:row + t.shape[0], :t.shape[1]].copy_(t)
 
+    def load_cols(self, t: torch.Tensor, col: int) -> None:
+        """Columns of the weight (projections of several inputs that lie side by side share it)."""
+        self.weight.data[:t.shape[0], col:col + t.shape[1]].copy_(t)
+
     def forward(self, x: torch.Tensor, out: Optional[torch.Tensor] = None, max_ctas: int = 0) -> torch.Tensor:
-        return self._gemm(x, out, max_ctas=max_ctas)
+        return self._gemm(x, out, bias=self.bias, max_ctas=max_ctas)

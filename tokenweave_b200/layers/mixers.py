@@ -1,11 +1,15 @@
 """Token mixers and feed-forwards of hybrid decoders: layers that a model's configuration lists one by one, each with
 its own kind and sizes (``models/hybrid.py``).
 
-A mixer owns its weights and whatever it keeps between steps - pages of a cache (``cache_bytes_per_block`` /
-``init_cache``) or a slot of recurrent state per sequence (``state_bytes_per_slot`` / ``init_state``) - and maps
-activation rows to sublayer outputs: ``forward(x, meta, rt, out)``. All sizes and constants are parameters, so
-another design can list the same mixers with other values. :data:`MIXERS` and :data:`FEED_FORWARDS` are the names a
-configuration may use.
+A mixer owns its weights and maps activation rows to sublayer outputs: ``forward(x, meta, rt, out, kept)``. What it
+keeps between steps - pages of a cache (``cache_bytes_per_block`` / ``init_cache``), a slot of recurrent state per
+sequence (``state_bytes_per_slot`` / ``init_state``) - is in ``kept``, which the model makes once per RUN of the layer: a
+layer that runs several times in a row has one set of weights and one ``kept`` per pass. All sizes and constants are
+parameters, so another design can list the same mixers with other values. :data:`MIXERS` and :data:`FEED_FORWARDS` are
+the names a configuration may use.
+
+A :class:`SumMixer` adds up several :class:`Part` s that read the same input (and, where a layer's feed-forward reads
+that input too, the feed-forward): their input projections are one matrix product, and so are their output projections.
 
 Activations and weights are bf16 or fp32 (the engine's dtype); norms, rotary angles, attention scores and softmax,
 decays and recurrent state are fp32 in both.
@@ -36,18 +40,22 @@ class Mixer(nn.Module):
     def state_bytes_per_slot(self) -> int:
         return 0
 
-    def init_cache(self, num_blocks: int, block_size: int) -> None:
+    def new_kept(self) -> dict:
+        """What one run of the layer keeps between steps, empty; a tree of dicts of tensors."""
+        return {}
+
+    def init_cache(self, kept: dict, num_blocks: int, block_size: int) -> None:
         pass
 
-    def init_state(self, num_slots: int) -> None:
+    def init_state(self, kept: dict, num_slots: int) -> None:
         pass
 
-    def state_tensors(self) -> list[torch.Tensor]:
-        """Every tensor kept between steps."""
-        return []
+    def bind_runtime(self, rt) -> None:
+        """Called once when the runtime exists: constants on the device."""
 
-    def drop_state(self) -> None:
-        pass
+    def launch_key(self, meta: AttentionMetadata, block_size: int, sm_count: int) -> tuple:
+        """What shapes this mixer's launches besides the step's counts."""
+        return ()
 
     def workspaces(self) -> list[tuple[str, int]]:
         """(name, columns) of the runtime buffers a forward pass uses."""
@@ -91,7 +99,6 @@ class LatentAttention(Mixer):
         self.ukt_w = nn.Parameter(torch.zeros(H, self.kv_rank, pad8(self.dim), dtype=dtype, device=device), requires_grad=False)
         self.o_proj = PaddedLinear(H * self.vdim, width, dtype=dtype, device=device)
         self.row = hops.latent_row(self.kv_rank, self.rot_dim)
-        self.cache: Optional[torch.Tensor] = None
         self.cos_sin: Optional[torch.Tensor] = None
 
     def workspaces(self) -> list[tuple[str, int]]:
@@ -116,15 +123,15 @@ class LatentAttention(Mixer):
     def cache_bytes_per_block(self, block_size: int) -> int:
         return block_size * self.row * self.o_proj.weight.element_size()
 
-    def init_cache(self, num_blocks: int, block_size: int) -> None:
+    def init_cache(self, kept: dict, num_blocks: int, block_size: int) -> None:
         w = self.o_proj.weight
-        self.cache = torch.zeros(num_blocks, block_size, self.row, dtype=w.dtype, device=w.device)
+        kept["latents"] = torch.zeros(num_blocks, block_size, self.row, dtype=w.dtype, device=w.device)
 
-    def state_tensors(self) -> list[torch.Tensor]:
-        return [] if self.cache is None else [self.cache]
-
-    def drop_state(self) -> None:
-        self.cache = None
+    def bind_runtime(self, rt) -> None:
+        key = self.rope_key()
+        if key not in rt.rope_tables:
+            rt.rope_tables[key] = self.make_rope_table()
+        self.cos_sin = rt.rope_tables[key]
 
     def rope_key(self) -> tuple:
         s = self.rot.get("scaling")
@@ -164,12 +171,12 @@ class LatentAttention(Mixer):
         return out
 
     # ---- forward ---------------------------------------------------------------------------------------
-    def forward(self, x: torch.Tensor, meta: AttentionMetadata, rt, out: torch.Tensor) -> None:
-        n, H = x.shape[0], self.heads
+    def forward(self, x: torch.Tensor, meta: AttentionMetadata, rt, out: torch.Tensor, kept: dict) -> None:
+        n, H, cache = x.shape[0], self.heads, kept["latents"]
         p = self.in_proj(x, out=rt.buffer("proj", n, self.in_proj.out_padded))
         cq = rt.buffer("latent_q", n, self.uq_proj.in_padded)
         hops.latent_prep(p, 0, self.q_rank, self.q_norm_w, cq, self.kv_off, self.kv_rank, self.kv_norm_w, self.rot_dim,
-                         self.rot_dims, self.cos_sin, meta.positions, meta.slot_mapping, self.cache, self.eps)
+                         self.rot_dims, self.cos_sin, meta.positions, meta.slot_mapping, cache, self.eps)
         q = self.uq_proj(cq, out=rt.buffer("query", n, self.uq_proj.out_padded))
         gate = p[:, self.gate_off:] if self.gated else None
         attn = rt.buffer("mixed", n, self.o_proj.in_padded)
@@ -180,14 +187,14 @@ class LatentAttention(Mixer):
             hops.latent_absorb(q, meta.tok_row, self.ukt_w, H, self.dim, self.rot_dim, self.rot_dims, self.kv_rank,
                                self.cos_sin, meta.positions, qa)
             o = rt.buffer("latent_out", m, H * self.kv_rank).view(m, H, self.kv_rank)
-            hops.latent_attention(qa, self.cache, meta.tok_seq, meta.tok_kvlen, m, meta.block_table, self.kv_rank,
+            hops.latent_attention(qa, cache, meta.tok_seq, meta.tok_kvlen, m, meta.block_table, self.kv_rank,
                                   self.scale, o, meta.max_kv_len, rt.sm_count)
             hops.latent_values(o, meta.tok_row, w_uv, H, self.vdim, self.kv_rank, gate, attn)
         if meta.num_tiles:
             # keys and values of the tiles' contexts (the step's own tokens are in the cache already)
             rows = meta.extra_cpu["ctx_rows"]
             lat = rt.buffer("ctx_latent", rows, self.row)
-            hops.latent_gather(self.cache, meta.extra["ctx_seqs"], meta.extra["ctx_cu"], meta.extra_cpu["ctx_max"],
+            hops.latent_gather(cache, meta.extra["ctx_seqs"], meta.extra["ctx_cu"], meta.extra_cpu["ctx_max"],
                                meta.block_table, lat)
             kv = self.ukv_proj(lat[:, :self.ukv_proj.in_padded], out=rt.buffer("ctx_kv", rows, self.ukv_proj.out_padded))
             hops.rope_tail_(q, H, self.dim + self.rot_dim, self.dim, self.rot_dims, self.cos_sin, meta.positions)
@@ -224,8 +231,6 @@ class Mamba2Mixer(Mixer):
         self.D = _vec(self.heads, dtype, device)
         self.norm_w = _vec(self.inner, dtype, device)
         self.o_proj = PaddedLinear(self.inner, width, dtype=dtype, device=device)
-        self.state: Optional[torch.Tensor] = None        # [slots, heads, vdim, N] fp32
-        self.conv_state: Optional[torch.Tensor] = None   # [slots, taps - 1, channels]
 
     def workspaces(self) -> list[tuple[str, int]]:
         return [("proj", self.in_proj.out_padded), ("conv", pad8(self.channels)), ("mixed", self.o_proj.in_padded),
@@ -239,16 +244,10 @@ class Mamba2Mixer(Mixer):
     def state_bytes_per_slot(self) -> int:
         return 4 * self.inner * self.N + (self.taps - 1) * self.channels * self.conv_w.element_size()
 
-    def init_state(self, num_slots: int) -> None:
+    def init_state(self, kept: dict, num_slots: int) -> None:
         dev = self.conv_w.device
-        self.state = torch.zeros(num_slots, self.heads, self.vdim, self.N, dtype=torch.float32, device=dev)
-        self.conv_state = torch.zeros(num_slots, self.taps - 1, self.channels, dtype=self.conv_w.dtype, device=dev)
-
-    def state_tensors(self) -> list[torch.Tensor]:
-        return [] if self.state is None else [self.state, self.conv_state]
-
-    def drop_state(self) -> None:
-        self.state = self.conv_state = None
+        kept["state"] = torch.zeros(num_slots, self.heads, self.vdim, self.N, dtype=torch.float32, device=dev)
+        kept["conv"] = torch.zeros(num_slots, self.taps - 1, self.channels, dtype=self.conv_w.dtype, device=dev)
 
     # ---- weights ---------------------------------------------------------------------------------------
     def tensor_targets(self) -> dict:
@@ -271,18 +270,18 @@ class Mamba2Mixer(Mixer):
         }
 
     # ---- forward ---------------------------------------------------------------------------------------
-    def forward(self, x: torch.Tensor, meta: AttentionMetadata, rt, out: torch.Tensor) -> None:
+    def forward(self, x: torch.Tensor, meta: AttentionMetadata, rt, out: torch.Tensor, kept: dict) -> None:
         n = x.shape[0]
         p = self.in_proj(x, out=rt.buffer("proj", n, self.in_proj.out_padded))
         xbc = rt.buffer("conv", n, pad8(self.channels))
         e = meta.extra
-        hops.causal_conv(p[:, self.x_off:], self.conv_w, self.conv_b, self.conv_state, xbc, e["row_seq"], meta.cu_q,
+        hops.causal_conv(p[:, self.x_off:], self.conv_w, self.conv_b, kept["conv"], xbc, e["row_seq"], meta.cu_q,
                          meta.kv_lens, e["state_slots"], meta.all_single)
         y = rt.buffer("mixed", n, self.o_proj.in_padded)
         # long runs in chunks on the tensor cores (sizes permitting), everything else token by token
         for run, seqs in ((hops.ssd_scan, e["scan_seqs"]),
                           (hops.ssd_chunk if self.chunkable else hops.ssd_scan, e["chunk_seqs"])):
-            run(xbc, p[:, self.dt_off:], self.dt_bias, self.A_log, self.D, self.state, y, seqs, meta.cu_q, meta.kv_lens,
+            run(xbc, p[:, self.dt_off:], self.dt_bias, self.A_log, self.D, kept["state"], y, seqs, meta.cu_q, meta.kv_lens,
                 e["state_slots"], self.groups)
         g = rt.buffer("gated", n, self.o_proj.in_padded)
         hops.gated_group_norm(y, p, self.norm_w, self.norm_groups, self.eps, g)
@@ -314,5 +313,329 @@ class PolyNormMLP(nn.Module):
         self.down_proj(a, out=out)
 
 
-MIXERS = {"latent_attention": LatentAttention, "mamba2": Mamba2Mixer}
+# ---- several parts side by side --------------------------------------------------------------------------------------
+class Part(nn.Module):
+    """One summand of a :class:`SumMixer`. It reads its ``in_cols`` columns of the shared input projection and writes its
+    ``out_cols`` columns of the row that the shared output projection takes (both multiples of eight; heads are stored
+    padded to eight elements, pads are zero). ``silu_cols``: the projection applies silu to that many of its first
+    columns. What it keeps between steps: as for a :class:`Mixer`."""
+    in_cols = out_cols = silu_cols = 0
+    biased = False               # its projections have biases
+    recurrent = False
+    attends = False              # attention over cached keys: rows are routed to query tiles or single rows
+
+    cache_bytes_per_block = Mixer.cache_bytes_per_block
+    state_bytes_per_slot = Mixer.state_bytes_per_slot
+    init_cache, init_state, bind_runtime, launch_key = (Mixer.init_cache, Mixer.init_state, Mixer.bind_runtime,
+                                                        Mixer.launch_key)
+    tileable = False             # long runs may go to 128-query tiles
+
+    def workspaces(self) -> list[tuple[str, int]]:
+        return []
+
+    def tensor_targets(self, width: int, load_in, load_bias, load_out) -> dict:
+        """checkpoint name -> (shape, callable). ``load_in(t, row)`` / ``load_bias(t, row)`` / ``load_out(t, col)`` write
+        into the shared projections, counted from this part's first row or column."""
+        raise NotImplementedError
+
+    def mix(self, p: torch.Tensor, meta: AttentionMetadata, rt, out: torch.Tensor, kept: dict) -> None:
+        raise NotImplementedError
+
+
+def _by_head(load, dim: int, padded: int, base: int):
+    """Spreads the rows of ``t`` (heads of ``dim``) over heads of ``padded`` rows from ``base`` on."""
+    def put(t: torch.Tensor) -> None:
+        for h in range(t.shape[0] // dim):
+            load(t[h * dim:(h + 1) * dim], base + h * padded)
+    return put
+
+
+def _pad_heads(dst: torch.Tensor, heads: int, dim: int, padded: int):
+    """Writes a vector of ``heads * dim`` elements into ``dst`` [..., heads * padded] (last axis)."""
+    def put(t: torch.Tensor) -> None:
+        dst.data.view(*dst.shape[:-1], heads, padded)[..., :dim].copy_(t.reshape(*dst.shape[:-1], heads, dim))
+    return put
+
+
+class GroupedAttention(Part):
+    """Grouped-query attention with its own sizes of queries / keys (``dim``) and values (``vdim``) over a paged cache.
+    Options, each a parameter:
+
+    * ``bias``: biases of the three projections;
+    * ``conv``: a causal convolution of that many taps over time on every channel of q, k and v, right behind the
+      projection (no bias, no activation); the last ``conv - 1`` projected rows of a sequence are part of its state;
+    * ``qk_norm``: "head" (RMS norm of every query and key head, one weight for all), "whole" (RMS norm of all queries,
+      and of all keys, of a token at once) or None;
+    * ``q_temp`` = {"coef", "every"}: queries times ``1 + coef * ln(floor((p + 1) / every) + 1)`` at position p;
+    * ``distance_bias``: ``2^(-8 (h + 1) / heads) * (i - j)`` is taken off the score of head h;
+    * ``sink``: one is added to the softmax's denominator (a key of score 0 without a value);
+    * ``out_scale``: factor on the result.
+    """
+    attends = True
+
+    def __init__(self, sizes: dict, eps: float, *, dtype, device, bias: bool = False, conv: Optional[int] = None,
+                 qk_norm: Optional[str] = None, q_temp: Optional[dict] = None, distance_bias: bool = False,
+                 sink: bool = False, out_scale: float = 1.0):
+        super().__init__()
+        self.heads, self.kv_heads, self.dim, self.vdim = (int(sizes[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
+        if self.heads % self.kv_heads:
+            raise ValueError(f"{self.heads} query heads do not divide into {self.kv_heads} groups")
+        if qk_norm not in (None, "head", "whole"):
+            raise ValueError(f"unknown query and key norm {qk_norm!r}")
+        self.scale, self.eps, self.dtype, self.taps = float(sizes["scale"]), eps, dtype, int(conv or 0)
+        self.qk_norm, self.distance_bias, self.sink, self.out_scale = qk_norm, distance_bias, sink, float(out_scale)
+        self.temp_coef, self.temp_every = (float(q_temp["coef"]), int(q_temp["every"])) if q_temp else (0.0, 1)
+        self.biased, self.recurrent = bias, self.taps > 1
+        self.dp, self.vp = pad8(self.dim), pad8(self.vdim)
+        self.k_off = self.heads * self.dp
+        self.v_off = self.k_off + self.kv_heads * self.dp
+        self.in_cols, self.out_cols = self.v_off + self.kv_heads * self.vp, self.heads * self.vp
+        self.conv_w = self.q_norm_w = self.k_norm_w = None
+        if self.taps:
+            self.conv_w = nn.Parameter(torch.zeros(self.taps, self.in_cols, dtype=dtype, device=device), requires_grad=False)
+        if qk_norm:
+            n = (1, 1) if qk_norm == "head" else (self.heads, self.kv_heads)
+            self.q_norm_w, self.k_norm_w = (_vec(i * self.dp, dtype, device, 0.0) for i in n)
+        self.device = torch.device(device)
+        self.slopes: Optional[torch.Tensor] = None
+
+    def bind_runtime(self, rt) -> None:
+        if self.distance_bias:
+            h = torch.arange(1, self.heads + 1, dtype=torch.float64)
+            self.slopes = torch.exp2(-8.0 * h / self.heads).float().to(self.device)
+
+    def workspaces(self) -> list[tuple[str, int]]:
+        return [("query", self.k_off)]
+
+    # ---- cache and state ---------------------------------------------------------------------------------
+    def cache_bytes_per_block(self, block_size: int) -> int:
+        return block_size * self.kv_heads * (self.dp + self.vp) * self.dtype.itemsize
+
+    def init_cache(self, kept: dict, num_blocks: int, block_size: int) -> None:
+        for name, n in (("k", self.dp), ("v", self.vp)):
+            kept[name] = torch.zeros(num_blocks, block_size, self.kv_heads, n, dtype=self.dtype, device=self.device)
+
+    def state_bytes_per_slot(self) -> int:
+        return max(0, self.taps - 1) * self.in_cols * self.dtype.itemsize
+
+    def init_state(self, kept: dict, num_slots: int) -> None:
+        if self.taps > 1:
+            kept["conv"] = torch.zeros(num_slots, self.taps - 1, self.in_cols, dtype=self.dtype, device=self.device)
+
+    # ---- launches ------------------------------------------------------------------------------------------
+    @property
+    def tileable(self) -> bool:
+        return self.device.type == "cuda" and hops.attention_tileable(self.dtype, self.dp, self.vp)
+
+    def launch_key(self, meta: AttentionMetadata, block_size: int, sm_count: int) -> tuple:
+        return hops.attention_rows_plan(meta.num_single, self.heads, self.kv_heads, self.dp, self.vp, block_size, self.dtype,
+                                        meta.max_kv_len, sm_count)
+
+    # ---- weights -------------------------------------------------------------------------------------------
+    def tensor_targets(self, width: int, load_in, load_bias, load_out) -> dict:
+        H, G, D, V = self.heads, self.kv_heads, self.dim, self.vdim
+        spans = {"q": (H, D, self.dp, 0), "k": (G, D, self.dp, self.k_off), "v": (G, V, self.vp, self.v_off)}
+        out = {"o": ((width, H * V), lambda t: _by_head(lambda r, i: load_out(r.t(), i), V, self.vp, 0)(t.t()))}
+        for name, (n, d, padded, base) in spans.items():
+            out[name] = ((n * d, width), _by_head(load_in, d, padded, base))
+            if self.biased:
+                out[name + ".b"] = ((n * d,), _by_head(load_bias, d, padded, base))
+            if self.taps:
+                put = _pad_heads(self.conv_w[:, base:base + n * padded], n, d, padded)
+                out[name + ".conv"] = ((n * d, self.taps), lambda t, put=put: put(t.t()))
+        if self.qk_norm:
+            for name, w, n in (("q", self.q_norm_w, H), ("k", self.k_norm_w, G)):
+                n = n if self.qk_norm == "whole" else 1
+                out[name + ".norm"] = ((n * D,), _pad_heads(w, n, D, self.dp))
+        return out
+
+    # ---- forward -------------------------------------------------------------------------------------------
+    def mix(self, p: torch.Tensor, meta: AttentionMetadata, rt, out: torch.Tensor, kept: dict) -> None:
+        q = rt.buffer("query", p.shape[0], self.k_off)
+        hops.qkv_prep(p, self.heads, self.kv_heads, self.dim, self.vdim, q, kept["k"], kept["v"], meta, self.conv_w,
+                      kept.get("conv"), self.qk_norm, self.q_norm_w, self.k_norm_w, self.eps, self.temp_coef,
+                      self.temp_every)
+        hops.grouped_attention(q, kept["k"], kept["v"], out, meta, self.heads, self.kv_heads, self.scale, self.slopes,
+                               self.sink, self.out_scale, rt.sm_count)
+
+
+class LightningAttention(Part):
+    """Linear attention with a fixed decay per head: ``S <- decay S + k v^T``, ``o = S^T q`` on ``silu`` of the projected
+    queries, keys and values (fp32 state), then one RMS norm over the concatenated heads with a weight, times
+    ``sigmoid(W_g x)`` and ``out_scale``. It is the state-space recurrence with unit steps, one group per head and no
+    skip, and runs on the same kernels."""
+    recurrent = True
+
+    def __init__(self, sizes: dict, eps: float, *, dtype, device, out_scale: float = 1.0):
+        super().__init__()
+        self.heads, self.dim, self.vdim = (int(sizes[k]) for k in ("heads", "dim", "vdim"))
+        self.decays = [float(d) for d in sizes["decay"]]
+        if len(self.decays) != self.heads or not all(0.0 <= d <= 1.0 for d in self.decays):
+            raise ValueError(f"{self.heads} decays between 0 and 1 are needed, got {self.decays}")
+        self.eps, self.dtype, self.device, self.out_scale = eps, dtype, torch.device(device), float(out_scale)
+        self.dp, self.vp = pad8(self.dim), pad8(self.vdim)
+        H = self.heads
+        # [values | keys | queries | gate]: the first three in the order of the recurrence's kernels
+        self.k_off, self.q_off, self.g_off = H * self.vp, H * (self.vp + self.dp), H * (self.vp + 2 * self.dp)
+        self.in_cols, self.out_cols, self.silu_cols = self.g_off + H * self.vp, H * self.vp, self.g_off
+        self.norm_w = _vec(H * self.vp, dtype, device, 0.0)
+        self.decay: Optional[torch.Tensor] = None
+
+    def bind_runtime(self, rt) -> None:
+        self.decay = torch.tensor(self.decays, dtype=torch.float32, device=self.device)
+
+    def workspaces(self) -> list[tuple[str, int]]:
+        return [("recurrent", self.out_cols)]
+
+    def state_bytes_per_slot(self) -> int:
+        return 4 * self.heads * self.vp * self.dp
+
+    def init_state(self, kept: dict, num_slots: int) -> None:
+        kept["state"] = torch.zeros(num_slots, self.heads, self.vp, self.dp, dtype=torch.float32, device=self.device)
+
+    def tensor_targets(self, width: int, load_in, load_bias, load_out) -> dict:
+        H, D, V = self.heads, self.dim, self.vdim
+        return {
+            "q": ((H * D, width), _by_head(load_in, D, self.dp, self.q_off)),
+            "k": ((H * D, width), _by_head(load_in, D, self.dp, self.k_off)),
+            "v": ((H * V, width), _by_head(load_in, V, self.vp, 0)),
+            "g": ((H * V, width), _by_head(load_in, V, self.vp, self.g_off)),
+            "norm": ((H * V,), _pad_heads(self.norm_w, H, V, self.vp)),
+            "o": ((width, H * V), lambda t: _by_head(lambda r, i: load_out(r.t(), i), V, self.vp, 0)(t.t())),
+        }
+
+    @property
+    def chunkable(self) -> bool:
+        return self.device.type == "cuda" and hops.ssd_chunkable(self.dtype, self.vp, self.dp)
+
+    def mix(self, p: torch.Tensor, meta: AttentionMetadata, rt, out: torch.Tensor, kept: dict) -> None:
+        y, e = rt.buffer("recurrent", p.shape[0], self.out_cols), meta.extra
+        for run, seqs in ((hops.decay_scan, e["scan_seqs"]),
+                          (hops.decay_chunk if self.chunkable else hops.decay_scan, e["chunk_seqs"])):
+            run(p, self.decay, kept["state"], y, seqs, meta.cu_q, meta.kv_lens, e["state_slots"])
+        hops.norm_gate(y, p[:, self.g_off:], self.norm_w, self.heads * self.vdim, self.eps, self.out_scale, out)
+
+
+class GatedMLP(nn.Module):
+    """The first half of a gated feed-forward, ``act(W_gate x) * (W_up x)``, as a part of a :class:`SumMixer` (whose output
+    projection holds ``W_down``). ``act``: "silu" or "gelu_tanh"."""
+
+    def __init__(self, sizes: dict, width: int, *, dtype, device):
+        super().__init__()
+        self.ff, self.width, self.act = int(sizes["ff"]), width, str(sizes["act"])
+        self.out_cols = pad8(self.ff)
+        self.gate_up = PaddedLinear(width, 2 * self.out_cols, dtype=dtype, device=device)
+
+    def workspaces(self) -> list[tuple[str, int]]:
+        # the fp32 product has no gated form: its two halves go through a buffer
+        return [("gate_up", 2 * self.out_cols)] if self.gate_up.weight.dtype == torch.float32 else []
+
+    def tensor_targets(self, load_out) -> dict:
+        return {"gate": ((self.ff, self.width), lambda t: self.gate_up.load_rows(t, 0)),
+                "up": ((self.ff, self.width), lambda t: self.gate_up.load_rows(t, self.out_cols)),
+                "down": ((self.width, self.ff), lambda t: load_out(t, 0))}
+
+    def forward(self, x: torch.Tensor, rt, out: torch.Tensor) -> None:
+        w = self.gate_up.weight
+        tmp = rt.buffer("gate_up", x.shape[0], w.shape[0]) if w.dtype == torch.float32 else None
+        hops.gated_product(x, w, self.act, out, tmp)
+
+
+PARTS = {"grouped_attention": GroupedAttention, "lightning_attention": LightningAttention}
+
+
+class SumMixer(Mixer):
+    """The sum of its parts (and of a gated feed-forward), all of the same input. ``sizes`` = {"parts": {name: {"kind",
+    "sizes", "options"}}}; the checkpoint names of a part's tensors have ``<name>.`` in front, or nothing for the name
+    "". One matrix product makes every part's projected input, one more the feed-forward's, and the last one takes the
+    parts' results side by side, so that their sum is its accumulation."""
+
+    def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device, max_positions: int = 0,
+                 mlp: Optional[dict] = None):
+        super().__init__()
+        self.width = width
+        self.parts = nn.ModuleDict()
+        for name, spec in sizes["parts"].items():
+            self.parts[name or "only"] = PARTS[spec["kind"]](spec["sizes"], eps, dtype=dtype, device=device,
+                                                             **spec.get("options", {}))
+        self.prefix = {name or "only": name + "." if name else "" for name in sizes["parts"]}
+        self.glu = GatedMLP(mlp, width, dtype=dtype, device=device) if mlp is not None else None
+        self.in_at, self.out_at, i, o = {}, {}, 0, 0
+        for name, part in self.parts.items():
+            self.in_at[name], self.out_at[name] = (i, i + part.in_cols), (o, o + part.out_cols)
+            i, o = i + part.in_cols, o + part.out_cols
+        self.glu_at = (o, o + self.glu.out_cols) if self.glu is not None else (o, o)
+        self.in_proj = PaddedLinear(width, i, bias=any(p.biased for p in self.parts.values()), dtype=dtype, device=device)
+        self.out_proj = PaddedLinear(self.glu_at[1], width, dtype=dtype, device=device)
+        silu = [(self.in_at[n][0], self.in_at[n][0] + p.silu_cols) for n, p in self.parts.items() if p.silu_cols]
+        if len(silu) > 1:
+            raise ValueError("one part per mixer may ask for silu on its projection")
+        self.silu = silu[0] if silu else None
+        self.recurrent = any(p.recurrent for p in self.parts.values())
+        self.attends = any(p.attends for p in self.parts.values())
+
+    @property
+    def tileable(self) -> bool:
+        return all(p.tileable for p in self.parts.values() if p.attends)
+
+    def workspaces(self) -> list[tuple[str, int]]:
+        out = [("proj", self.in_proj.out_padded), ("mixed", self.out_proj.in_padded)]
+        for part in list(self.parts.values()) + ([self.glu] if self.glu is not None else []):
+            out += part.workspaces()
+        return out
+
+    def cache_bytes_per_block(self, block_size: int) -> int:
+        return sum(p.cache_bytes_per_block(block_size) for p in self.parts.values())
+
+    def state_bytes_per_slot(self) -> int:
+        return sum(p.state_bytes_per_slot() for p in self.parts.values())
+
+    def new_kept(self) -> dict:
+        return {name: {} for name in self.parts}
+
+    def init_cache(self, kept: dict, num_blocks: int, block_size: int) -> None:
+        for name, part in self.parts.items():
+            part.init_cache(kept[name], num_blocks, block_size)
+
+    def init_state(self, kept: dict, num_slots: int) -> None:
+        for name, part in self.parts.items():
+            part.init_state(kept[name], num_slots)
+
+    def bind_runtime(self, rt) -> None:
+        for part in self.parts.values():
+            part.bind_runtime(rt)
+
+    def launch_key(self, meta: AttentionMetadata, block_size: int, sm_count: int) -> tuple:
+        return tuple(p.launch_key(meta, block_size, sm_count) for p in self.parts.values())
+
+    def tensor_targets(self) -> dict:
+        out = {}
+        for name, part in self.parts.items():
+            i, o = self.in_at[name][0], self.out_at[name][0]
+
+            def load_bias(t, row, i=i):
+                self.in_proj.bias.data[i + row:i + row + t.shape[0]].copy_(t)
+            targets = part.tensor_targets(self.width, lambda t, row, i=i: self.in_proj.load_rows(t, i + row), load_bias,
+                                          lambda t, col, o=o: self.out_proj.load_cols(t, o + col))
+            out.update({self.prefix[name] + k: v for k, v in targets.items()})
+        return out
+
+    def mlp_targets(self) -> dict:
+        """Tensors of the feed-forward (behind ``<layer>.mlp.``)."""
+        return self.glu.tensor_targets(lambda t, col: self.out_proj.load_cols(t, self.glu_at[0] + col))
+
+    def forward(self, x: torch.Tensor, meta: AttentionMetadata, rt, out: torch.Tensor, kept: dict) -> None:
+        n = x.shape[0]
+        mixed = rt.buffer("mixed", n, self.out_proj.in_padded)
+        if self.glu is not None:
+            self.glu(x, rt, mixed[:, self.glu_at[0]:self.glu_at[1]])
+        p = hops.projection(x, self.in_proj.weight, self.in_proj.bias, self.silu,
+                            rt.buffer("proj", n, self.in_proj.out_padded))
+        for name, part in self.parts.items():
+            (i0, i1), (o0, o1) = self.in_at[name], self.out_at[name]
+            part.mix(p[:, i0:i1], meta, rt, mixed[:, o0:o1], kept[name])
+        self.out_proj(mixed, out=out)
+
+
+MIXERS = {"latent_attention": LatentAttention, "mamba2": Mamba2Mixer, "sum": SumMixer}
 FEED_FORWARDS = {"dense": PolyNormMLP}

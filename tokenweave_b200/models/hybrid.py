@@ -4,12 +4,18 @@ or a recurrence with a state slot per sequence) and an optional feed-forward (``
 Differences from :class:`~tokenweave_b200.models.decoder.DecoderModel`, whose interface towards the worker and the model
 runner this class shares:
 
-* the residual stream is fp32 and the sublayers read it directly (in the activation type); the RMS norm is applied to
-  a sublayer's OUTPUT before the sum: ``x += norm(f(x))``. Sum, norm, and the cast of the next input (or the model's
-  final norm) are one kernel;
+* the residual stream is fp32. ``ModelConfig.block`` says how a layer adds to it:
+  "output_norm": the sublayers read the stream directly (in the activation type) and the RMS norm is applied to a
+  sublayer's OUTPUT, ``x += norm1(mixer(x))``, ``x += norm2(ff(x))``; sum, norm, and the cast of the next input (or the
+  model's final norm) are one kernel;
+  "parallel": both sublayers read one norm of the stream, ``x += mixer(norm1(x)) + ff(norm1(x))``; the two results come
+  out of one matrix product, and their addition and the next layer's norm (or the final one) are one kernel;
+* layers may be run several times in a row with the same weights (``ModelConfig.loop``); every pass keeps its own cache
+  and state, and before each pass but the first the embedding output is added to the stream;
+* a table of embeddings of token pairs may be added to the token embeddings (``ModelConfig.bigram``);
 * bf16 and fp32 both run on the GPU (the fp32 mode in true fp32);
-* one GPU: a norm on the sublayer's output needs the whole output, so the fused reduce-scatter + add + norm of the
-  pre-norm families does not apply, and tensor / pipeline parallelism are refused.
+* one GPU: tensor / pipeline parallelism are refused (the fused reduce-scatter + add + norm of the pre-norm families
+  works on a bf16 residual stream and neither on a norm of the sublayer's output nor on a sum with a stored row).
 """
 from __future__ import annotations
 
@@ -22,7 +28,7 @@ from torch import nn
 from ..config import ModelConfig
 from ..layers.attention import PREFILL_MIN_Q, AttentionMetadata
 from ..layers.linear import PaddedLinear, pad8
-from ..layers.mixers import FEED_FORWARDS, MIXERS, LatentAttention
+from ..layers.mixers import FEED_FORWARDS, MIXERS, LatentAttention, SumMixer
 from ..ops import hybrid as hops
 from ..parallel.comm import TPCommunicator
 from ..parallel.state import get_tp
@@ -44,6 +50,8 @@ class HybridRuntime:
         self.hidden.zero_()
         self.residual = torch.zeros(max_tokens, w8, dtype=torch.float32, device=device)
         self.sublayer = torch.zeros(max_tokens, w8, dtype=cfg.dtype, device=device)
+        # the embedding output, for layers that run again
+        self.first = torch.zeros(max_tokens, w8, dtype=torch.float32, device=device) if cfg.loop else None
         self.comm = TPCommunicator(self.staging, tp, tw_cfg.wait_budget_ms, tw_cfg.transport)
         self.dtype = cfg.dtype
         self.sm_count = torch.cuda.get_device_properties(device).multi_processor_count if device.type == "cuda" else 0
@@ -63,6 +71,8 @@ class HybridRuntime:
 
 
 class HybridLayer(nn.Module):
+    """``x += norm1(mixer(x))``, ``x += norm2(ff(x))``"""
+
     def __init__(self, spec: dict, cfg: ModelConfig, *, device):
         super().__init__()
         kind = spec["type"]
@@ -89,6 +99,53 @@ class HybridLayer(nn.Module):
         return out
 
 
+class ParallelLayer(nn.Module):
+    """``x += mixer(norm1(x)) + ff(norm1(x))``: the mixer is a :class:`SumMixer` with the feed-forward as one more summand."""
+
+    def __init__(self, spec: dict, cfg: ModelConfig, *, device):
+        super().__init__()
+        if spec["type"] != "sum":
+            raise ValueError(f"a parallel block takes a sum of parts, not {spec['type']!r}")
+        mlp = spec.get("mlp")
+        if mlp is not None and mlp["kind"] != "gated":
+            raise ValueError(f"unknown feed-forward {mlp['kind']!r} in a parallel block")
+        dt = cfg.dtype
+        self.mixer = SumMixer(spec["mixer"], cfg.hidden_size, cfg.rms_norm_eps, dtype=dt, device=device,
+                              max_positions=cfg.max_model_len, mlp=mlp)
+        self.norm1_w = nn.Parameter(torch.ones(cfg.hidden_size, dtype=dt, device=device), requires_grad=False)
+        self.mlp = None                     # part of the mixer
+
+    def tensor_targets(self) -> dict:
+        out = {"norm1": ((self.norm1_w.numel(),), self.norm1_w.data.copy_)}
+        out.update({f"mix.{k}": v for k, v in self.mixer.tensor_targets().items()})
+        if self.mixer.glu is not None:
+            out.update({f"mlp.{k}": v for k, v in self.mixer.mlp_targets().items()})
+        return out
+
+
+BLOCKS = {"output_norm": HybridLayer, "parallel": ParallelLayer}
+
+
+def layer_runs(num_layers: int, loop: Optional[dict]) -> list[tuple[int, bool]]:
+    """(layer, a pass other than the first begins here) in the order in which the layers run."""
+    if not loop:
+        return [(i, False) for i in range(num_layers)]
+    start, stop, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not 0 <= start < stop <= num_layers or times < 1:
+        raise ValueError(f"a loop over layers {start} .. {stop - 1} of {num_layers}, {times} times")
+    runs = [(i, False) for i in range(start)]
+    for n in range(times):
+        runs += [(i, n > 0 and i == start) for i in range(start, stop)]
+    return runs + [(i, False) for i in range(stop, num_layers)]
+
+
+def _tensors(kept: dict) -> list[torch.Tensor]:
+    out = []
+    for v in kept.values():
+        out += _tensors(v) if isinstance(v, dict) else [v]
+    return out
+
+
 class HybridDecoder(nn.Module):
     architecture = "hybrid"
 
@@ -102,13 +159,26 @@ class HybridDecoder(nn.Module):
         self.cfg = cfg
         dt, W = cfg.dtype, cfg.hidden_size
         self.embed_w = nn.Parameter(torch.zeros(cfg.vocab_size, pad8(W), dtype=dt, device=device), requires_grad=False)
-        self.layers = nn.ModuleList([HybridLayer(s, cfg, device=device) for s in cfg.layers])
+        self.bigram_w = None
+        if cfg.bigram:                      # one row per bucket, and one for tokens without a token before them
+            self.bigram_w = nn.Parameter(torch.zeros(int(cfg.bigram["buckets"]) + 1, pad8(W), dtype=dt, device=device),
+                                         requires_grad=False)
+        self.layers = nn.ModuleList([BLOCKS[cfg.block](s, cfg, device=device) for s in cfg.layers])
+        self.runs = layer_runs(len(self.layers), cfg.loop)
+        if cfg.block != "parallel" and (cfg.loop or cfg.bigram):
+            raise ValueError("loops and pair embeddings are built for parallel blocks")
+        self.kept = [self.layers[i].mixer.new_kept() for i, _ in self.runs]
         self.final_norm_w = nn.Parameter(torch.ones(W, dtype=dt, device=device), requires_grad=False)
         self.head = PaddedLinear(W, cfg.vocab_size, dtype=dt, device=device)
         self.rt: Optional[HybridRuntime] = None
-        latent = [l.mixer for l in self.layers if isinstance(l.mixer, LatentAttention)]
-        self.expand = bool(latent) and all(m.expandable for m in latent)      # long runs may use the expanded form
-        self.recurrent = any(l.mixer.recurrent for l in self.layers)
+        mixers = [l.mixer for l in self.layers]
+        latent = [m for m in mixers if isinstance(m, LatentAttention)]
+        grouped = [m for m in mixers if isinstance(m, SumMixer) and m.attends]
+        # long runs may go to query tiles: every attention of the model can take them; with latent attention their
+        # contexts are expanded into a workspace first
+        self.expand = bool(latent)
+        self.tiles = (bool(latent or grouped) and all(m.expandable for m in latent) and all(m.tileable for m in grouped))
+        self.recurrent = any(m.recurrent for m in mixers)
 
     # ---- runtime ---------------------------------------------------------------------------------------
     def setup_runtime(self, max_tokens: int, tw_cfg, provider: Optional[str] = None,
@@ -119,56 +189,55 @@ class HybridDecoder(nn.Module):
             for part in (m, layer.mlp):
                 for name, cols in part.workspaces() if part is not None else ():
                     self.rt.buffer(name, max_tokens, cols)
-                if self.expand and part is m and isinstance(m, LatentAttention):
+                if self.tiles and part is m and isinstance(m, LatentAttention):
                     for name, cols in m.context_workspaces():
                         self.rt.buffer(name, self.rt.context_rows, cols)
-            if isinstance(m, LatentAttention):
-                key = m.rope_key()
-                if key not in self.rt.rope_tables:
-                    self.rt.rope_tables[key] = m.make_rope_table()
-                m.cos_sin = self.rt.rope_tables[key]
+            m.bind_runtime(self.rt)
         return self.rt
 
     def kv_cache_bytes_per_block(self, block_size: int) -> int:
-        return max(1, sum(l.mixer.cache_bytes_per_block(block_size) for l in self.layers))
+        return max(1, sum(self.layers[i].mixer.cache_bytes_per_block(block_size) for i, _ in self.runs))
 
     def state_bytes_per_slot(self) -> int:
-        return sum(l.mixer.state_bytes_per_slot() for l in self.layers)
+        return sum(self.layers[i].mixer.state_bytes_per_slot() for i, _ in self.runs)
 
     def init_kv_cache(self, num_blocks: int, block_size: int) -> None:
-        for l in self.layers:
-            l.mixer.init_cache(num_blocks, block_size)
+        for (i, _), kept in zip(self.runs, self.kept):
+            self.layers[i].mixer.init_cache(kept, num_blocks, block_size)
 
     def init_state(self, num_slots: int) -> None:
-        for l in self.layers:
-            l.mixer.init_state(num_slots)
+        for (i, _), kept in zip(self.runs, self.kept):
+            self.layers[i].mixer.init_state(kept, num_slots)
 
     def cache_tensors(self) -> list[torch.Tensor]:
-        return [t for l in self.layers for t in l.mixer.state_tensors()]
+        return [t for kept in self.kept for t in _tensors(kept)]
 
     def drop_caches(self) -> None:
-        for l in self.layers:
-            l.mixer.drop_state()
+        self.kept = [self.layers[i].mixer.new_kept() for i, _ in self.runs]
 
     # ---- a step's layout -------------------------------------------------------------------------------
-    def plan_step(self, q_lens, kv_lens, state_slots):
+    def plan_step(self, q_lens, kv_lens, state_slots, prev_tokens):
         """Routing of a step's rows: (attention plan as of ``plan_attention``, extra int32 arrays, host values).
+        ``prev_tokens``: the token before each sequence's first row of the step, -1 where there is none.
 
-        Attention: a run of a prompt goes to 128-query tiles over expanded keys and values when it is long enough to
-        pay for expanding its context (a product over the whole context, whatever the run's length), and when the
-        context fits the workspace; every other row is attended alone in the absorbed form. Recurrences: long runs in
-        chunks, short ones token by token."""
+        Attention: a run of a prompt goes to 128-query tiles. In models with latent attention it does so when it is long
+        enough to pay for expanding its context (a product over the whole context, whatever the run's length), and when
+        the context fits the workspace. Every other row is attended alone (over latents: in the absorbed form).
+        Recurrences: long runs in chunks, short ones token by token."""
         B = len(q_lens)
+        extra = {"prev_token": np.asarray(prev_tokens, dtype=np.int32)} if self.bigram_w is not None else {}
         if max(q_lens) == 1:
             rows = np.arange(B, dtype=np.int32)
             plan = ([], [], rows, rows, np.asarray(kv_lens, dtype=np.int32))
-            extra = {"row_seq": rows}
+            extra["row_seq"] = rows
             if self.recurrent:
                 extra.update(state_slots=np.asarray(state_slots, dtype=np.int32), scan_seqs=rows, chunk_seqs=rows[:0])
             return plan, extra, {}
         n = np.asarray(q_lens)
         tiled, ctx_rows = [], 0
-        if self.expand:
+        if self.tiles and not self.expand:
+            tiled = [b for b, ql in enumerate(q_lens) if ql >= PREFILL_MIN_Q]
+        elif self.tiles:
             for b, (ql, kv) in enumerate(zip(q_lens, kv_lens)):
                 if (ql >= 64 or (ql >= PREFILL_MIN_Q and kv <= 2 * ql)) and ctx_rows + kv <= self.rt.context_rows:
                     tiled.append(b)
@@ -182,8 +251,9 @@ class HybridDecoder(nn.Module):
         tile_q0 = [q0 for b in tiled for q0 in range(0, q_lens[b], 128)]
         order = np.argsort([-(kv_lens[b] - q_lens[b] + q0) for b, q0 in zip(tile_seq, tile_q0)], kind="stable")
         plan = ([tile_seq[i] for i in order], [tile_q0[i] for i in order], tok_row, tok_seq, tok_kv.astype(np.int32))
-        extra, host = {"row_seq": row_seq}, {}
-        if tiled:
+        host = {}
+        extra["row_seq"] = row_seq
+        if tiled and self.expand:
             cu = np.zeros(len(tiled) + 1, dtype=np.int32)
             np.cumsum([kv_lens[b] for b in tiled], out=cu[1:])
             begin = np.full(B, -1, dtype=np.int32)
@@ -200,8 +270,7 @@ class HybridDecoder(nn.Module):
         """What shapes a step's launches besides its token and sequence counts (part of a graph's signature)."""
         return (meta.all_single, tuple(sorted(meta.extra_cpu.items())),
                 tuple(sorted((k, v.shape[0]) for k, v in meta.extra.items())),
-                tuple(sorted({l.mixer.launch_key(meta, block_size, self.rt.sm_count) for l in self.layers
-                              if isinstance(l.mixer, LatentAttention)})))
+                tuple(l.mixer.launch_key(meta, block_size, self.rt.sm_count) for l in self.layers))
 
     # ---- forward ---------------------------------------------------------------------------------------
     @torch.inference_mode()
@@ -210,10 +279,20 @@ class HybridDecoder(nn.Module):
         rt, cfg, meta = self.rt, self.cfg, step.meta
         T, eps = step.plan.num_tokens, cfg.rms_norm_eps
         x32, xa, y = rt.residual[:T], rt.hidden[:T], rt.sublayer[:T]
+        if cfg.block == "parallel":
+            first = rt.first[:T] if rt.first is not None else None
+            hops.embed_norm(step.input_ids, self.embed_w, self.bigram_w, cfg.bigram, meta, x32, first,
+                            self.layers[self.runs[0][0]].norm1_w, eps, xa)
+            for n, (i, _) in enumerate(self.runs):
+                self.layers[i].mixer(xa, meta, rt, y, self.kept[n])
+                nxt, again = self.runs[n + 1] if n + 1 < len(self.runs) else (None, False)
+                hops.add_prenorm_(y, x32, first if again else None,
+                                  self.final_norm_w if nxt is None else self.layers[nxt].norm1_w, eps, xa)
+            return xa
         hops.embed_residual(step.input_ids, self.embed_w, x32, xa, cfg.hidden_size)
         last = self.layers[-1]
-        for layer in self.layers:
-            layer.mixer(xa, meta, rt, y)
+        for layer, kept in zip(self.layers, self.kept):
+            layer.mixer(xa, meta, rt, y, kept)
             final = self.final_norm_w if layer is last and layer.mlp is None else None
             hops.postnorm_add_(y, x32, layer.norm1_w, eps, xa, final)
             if layer.mlp is not None:
@@ -232,6 +311,8 @@ class HybridDecoder(nn.Module):
         out = {"embed": ((V, W), lambda t: self.embed_w.data[:, :W].copy_(t)),
                "final.norm": ((W,), self.final_norm_w.data.copy_),
                "head": ((V, W), lambda t: self.head.load_rows(t, 0))}
+        if self.bigram_w is not None:
+            out["bigram"] = ((self.bigram_w.shape[0], W), lambda t: self.bigram_w.data[:, :W].copy_(t))
         for i, layer in enumerate(self.layers):
             out.update({f"l{i}.{k}": v for k, v in layer.tensor_targets().items()})
         return out
@@ -274,9 +355,9 @@ class HybridDecoder(nn.Module):
                 return t.uniform_(1.0, 16.0, generator=g).log_()
             if leaf == "dt_bias":
                 return t.uniform_(-6.9, -2.3, generator=g)
-            if leaf == "conv.b":
+            if name.endswith(".b"):
                 return t.zero_()
-            if leaf == "conv":
+            if leaf.endswith("conv"):
                 return t.normal_(0.0, shape[1] ** -0.5, generator=g)
             if name.endswith(".mlp.act"):
                 return torch.tensor([1 / 3, 1 / 3, 1 / 3, 0.0], device=dev)

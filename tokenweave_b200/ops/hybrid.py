@@ -1,6 +1,8 @@
 """Operators of models whose layers mix attention and recurrences and whose residual stream is fp32: latent attention
 over a paged latent cache, the state-space (Mamba-2) recurrence with its convolution, the norm of a sublayer's output
-added to the residual, and the polynomial-norm activation.
+added to the residual, and the polynomial-norm activation; for blocks whose sublayers read one norm of the stream,
+grouped attention with its options (query and key norms, short convolution, query temperature, distance bias, sink),
+lightning attention, embeddings with token pairs, and the fused projections.
 
 Like the other operators, CUDA tensors (bf16 or fp32) go to the kernels of ``_C.so`` and CPU tensors to plain PyTorch
 (:mod:`.reference_hybrid`). ``meta`` below is the step's :class:`~tokenweave_b200.layers.attention.AttentionMetadata`.
@@ -12,7 +14,7 @@ from typing import Optional
 import torch
 
 from . import _native, reference_hybrid as ref
-from . import _p, _row_stride, _stream, decode_splits_tc, status_word
+from . import _p, _row_stride, _stream, decode_splits_tc, gemm, status_word
 
 
 def _dt(*ts: Optional[torch.Tensor]) -> int:
@@ -265,3 +267,188 @@ def ssd_chunk(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, A_log:
                  A_log.data_ptr(), D.data_ptr(), state.data_ptr(), y.data_ptr(), _row_stride(y), seqs.data_ptr(),
                  seqs.shape[0], cu_q.data_ptr(), kv_lens.data_ptr(), slots.data_ptr(), heads, vdim, N, groups, form,
                  status_word(xbc.device).data_ptr(), _stream())
+
+
+# ---- lightning attention: the recurrence with unit steps and a fixed decay per head --------------------------------
+def decay_scan(p: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, y: torch.Tensor, seqs: torch.Tensor,
+               cu_q: torch.Tensor, kv_lens: torch.Tensor, slots: torch.Tensor) -> None:
+    """``S <- decay[h] S + v k^T``, ``y = S q`` token by token; ``p`` rows are [v of all heads | k | q | ...]."""
+    if seqs.shape[0] == 0:
+        return
+    _, heads, vdim, N = state.shape
+    if not p.is_cuda:
+        ref.decay_scan(p, decay, state, y, seqs, cu_q, kv_lens, slots)
+        return
+    assert state.dtype == decay.dtype == torch.float32
+    _native.call("tw_decay_scan", p.data_ptr(), _row_stride(p), decay.data_ptr(), state.data_ptr(), y.data_ptr(),
+                 _row_stride(y), seqs.data_ptr(), seqs.shape[0], cu_q.data_ptr(), kv_lens.data_ptr(), slots.data_ptr(),
+                 heads, vdim, N, _dt(p, y), _stream())
+
+
+def decay_chunk(p: torch.Tensor, decay: torch.Tensor, state: torch.Tensor, y: torch.Tensor, seqs: torch.Tensor,
+                cu_q: torch.Tensor, kv_lens: torch.Tensor, slots: torch.Tensor, form: int = 0) -> None:
+    """:func:`decay_scan` for long runs on the tensor cores (CUDA, bf16); ``form`` as for :func:`ssd_chunk`."""
+    if seqs.shape[0] == 0:
+        return
+    _, heads, vdim, N = state.shape
+    assert state.dtype == decay.dtype == torch.float32 and _dt(p, y) == 0
+    _native.call("tw_decay_chunk", p.data_ptr(), _row_stride(p), p.shape[0], decay.data_ptr(), state.data_ptr(),
+                 y.data_ptr(), _row_stride(y), seqs.data_ptr(), seqs.shape[0], cu_q.data_ptr(), kv_lens.data_ptr(),
+                 slots.data_ptr(), heads, vdim, N, form, status_word(p.device).data_ptr(), _stream())
+
+
+def norm_gate(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, count: int, eps: float, scale: float,
+              out: torch.Tensor) -> None:
+    """``out = rmsnorm(y) * weight * sigmoid(gate) * scale``; rows as wide as the weight, of which ``count`` elements are
+    not padding (zeros)."""
+    if not y.is_cuda:
+        ref.norm_gate(y, gate, weight, count, eps, scale, out)
+        return
+    _native.call("tw_norm_gate", y.data_ptr(), _row_stride(y), gate.data_ptr(), _row_stride(gate), weight.data_ptr(),
+                 out.data_ptr(), _row_stride(out), y.shape[0], weight.numel(), count, float(eps), float(scale),
+                 _dt(y, gate, weight, out), _stream())
+
+
+# ---- parallel blocks: embedding, sums and norms, projections ---------------------------------------------------------
+def embed_norm(ids: torch.Tensor, table: torch.Tensor, pairs: Optional[torch.Tensor], spec: Optional[dict], meta,
+               x32: torch.Tensor, first: Optional[torch.Tensor], weight: torch.Tensor, eps: float, xa: torch.Tensor) -> None:
+    """``x32 = table[ids]``, plus the token pair's row of ``pairs`` (``spec`` = {"buckets", "mul_prev", "mul_cur"}: row
+    ``(previous * mul_prev + token * mul_cur) mod buckets``, the last row for a sequence's first token); ``first``: a copy
+    of that; ``xa = rmsnorm(x32) * weight``."""
+    if not table.is_cuda:
+        ref.embed_norm(ids, table, pairs, spec, meta, x32, first, weight, eps, xa)
+        return
+    assert ids.dtype == torch.int32 and x32.dtype == torch.float32
+    row_seq = prev = None
+    mul = (1, 0, 0)
+    if pairs is not None:
+        row_seq, prev = meta.extra["row_seq"], meta.extra["prev_token"]
+        mul = tuple(int(spec[k]) for k in ("buckets", "mul_prev", "mul_cur"))
+        assert pairs.shape[0] == mul[0] + 1
+    _native.call("tw_embed_norm", ids.data_ptr(), table.data_ptr(), _row_stride(table), table.shape[0], _p(pairs),
+                 _row_stride(pairs) if pairs is not None else 0, *mul, _p(row_seq), meta.cu_q.data_ptr(), _p(prev),
+                 x32.data_ptr(), _row_stride(x32), _p(first), _row_stride(first) if first is not None else 0,
+                 weight.data_ptr(), xa.data_ptr(), _row_stride(xa), ids.shape[0], weight.numel(), float(eps),
+                 _dt(table, pairs, weight, xa), _stream())
+
+
+def add_prenorm_(y: torch.Tensor, x32: torch.Tensor, first: Optional[torch.Tensor], weight: torch.Tensor, eps: float,
+                 xa: torch.Tensor) -> None:
+    """``x32 += y (+ first)``, ``xa = rmsnorm(x32) * weight``."""
+    if not y.is_cuda:
+        ref.add_prenorm_(y, x32, first, weight, eps, xa)
+        return
+    assert x32.dtype == torch.float32 and (first is None or first.dtype == torch.float32)
+    _native.call("tw_add_prenorm", y.data_ptr(), _row_stride(y), x32.data_ptr(), _row_stride(x32), _p(first),
+                 _row_stride(first) if first is not None else 0, weight.data_ptr(), xa.data_ptr(), _row_stride(xa),
+                 y.shape[0], weight.numel(), float(eps), _dt(y, weight, xa), _stream())
+
+
+def projection(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], silu: Optional[tuple[int, int]],
+               out: torch.Tensor) -> torch.Tensor:
+    """``out = x w^T + bias``, then silu on the columns ``[silu[0], silu[1])`` (in the product's epilogue in bf16)."""
+    if not x.is_cuda:
+        gemm(x, w, out=out, bias=bias)
+        if silu is not None:
+            out[:, silu[0]:silu[1]] = torch.nn.functional.silu(out[:, silu[0]:silu[1]])
+        return out
+    if silu is None or x.dtype == torch.bfloat16:
+        return gemm(x, w, out=out, bias=bias, silu_cols=silu)
+    gemm(x, w, out=out, bias=bias)
+    part = out[:, silu[0]:silu[1]]
+    _native.call("tw_silu_cols", part.data_ptr(), _row_stride(part), part.shape[0], part.shape[1], _dt(part), _stream())
+    return out
+
+
+GLU_ACTS = {"silu": 1, "gelu_tanh": 2}
+
+
+def gated_product(x: torch.Tensor, w: torch.Tensor, act: str, out: torch.Tensor, tmp: Optional[torch.Tensor]) -> None:
+    """``out = act(x w_gate^T) * (x w_up^T)`` with ``w`` = [gate; up]: one product in bf16, in fp32 a product into ``tmp``
+    and the gate behind it."""
+    if not x.is_cuda:
+        ref.gated_product(x, w, act, out)
+        return
+    if x.dtype == torch.bfloat16:
+        gemm(x, w, out=out, swiglu=True, act=act)
+        return
+    gemm(x, w, out=tmp)
+    _native.call("tw_glu", tmp.data_ptr(), _row_stride(tmp), out.data_ptr(), _row_stride(out), x.shape[0], out.shape[1],
+                 GLU_ACTS[act], _dt(tmp, out), _stream())
+
+
+# ---- grouped attention ------------------------------------------------------------------------------------------------
+QK_NORMS = {None: 0, "head": 1, "whole": 2}
+
+
+def qkv_prep(p: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, q: torch.Tensor, k_cache: torch.Tensor,
+             v_cache: torch.Tensor, meta, conv_w: Optional[torch.Tensor], conv_state: Optional[torch.Tensor],
+             qk_norm: Optional[str], wq: Optional[torch.Tensor], wk: Optional[torch.Tensor], eps: float, temp_coef: float,
+             temp_every: int) -> None:
+    """Everything between the projection and the attention. ``p`` rows are [queries | keys | values], heads padded to
+    the caches' last dimension; ``conv_w`` [taps, columns] and ``conv_state`` [slots, taps - 1, columns]: causal
+    convolution over time, the state moved on; norm of queries and keys per head or whole; queries times
+    ``1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)``; ``q`` [T, heads * padded], keys and values into the
+    caches [blocks, page, kv_heads, padded]."""
+    if not p.is_cuda:
+        ref.qkv_prep(p, heads, kv_heads, dim, vdim, q, k_cache, v_cache, meta, conv_w, conv_state, qk_norm, wq, wk, eps,
+                     temp_coef, temp_every)
+        return
+    e = meta.extra
+    _native.call("tw_qkv_prep", p.data_ptr(), _row_stride(p), p.shape[0], heads, kv_heads, dim, k_cache.shape[-1],
+                 v_cache.shape[-1], q.data_ptr(), _row_stride(q), k_cache.data_ptr(), v_cache.data_ptr(),
+                 meta.positions.data_ptr(), meta.slot_mapping.data_ptr(), _p(conv_w), _p(conv_state),
+                 conv_w.shape[0] if conv_w is not None else 1, _p(e.get("row_seq")), meta.cu_q.data_ptr(),
+                 meta.kv_lens.data_ptr(), _p(e.get("state_slots")), meta.num_seqs, int(meta.all_single),
+                 QK_NORMS[qk_norm], _p(wq), _p(wk), float(eps), float(temp_coef), int(temp_every),
+                 _dt(p, q, k_cache, v_cache, conv_w, conv_state, wq, wk), _stream())
+
+
+def attention_tileable(dtype: torch.dtype, dp: int, vp: int) -> bool:
+    """Padded head sizes the query-tile kernel takes (bf16)."""
+    return dtype == torch.bfloat16 and dp <= 128 and vp <= 128
+
+
+def attention_rows_plan(n: int, heads: int, kv_heads: int, dp: int, vp: int, page: int, dtype: torch.dtype,
+                        max_kv_len: int, sm_count: int = 148) -> tuple[str, int]:
+    """(kernel, key splits) for rows attended alone: "tc" (tensor cores) or "simt" (fp32, heads beyond 128 elements)."""
+    if dtype != torch.bfloat16 or dp > 128 or vp > 128 or page < 8 or page > 128 or 128 % page:
+        return "simt", 1
+    blocks = kv_heads * ((heads // kv_heads + 15) // 16)
+    return "tc", decode_splits_tc(n * blocks, (max_kv_len + 127) // 128, sm_count)
+
+
+def grouped_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, meta, heads: int,
+                      kv_heads: int, scale: float, slopes: Optional[torch.Tensor], sink: bool, out_scale: float,
+                      sm_count: int = 148, kernel: Optional[str] = None) -> None:
+    """Causal attention of a step's rows over the paged caches; head h's score loses ``slopes[h] * (i - j)``; ``sink``
+    adds one to the denominator; the result is multiplied by ``out_scale``. ``kernel``: force "simt" (tests)."""
+    if not q.is_cuda:
+        ref.grouped_attention(q, k_cache, v_cache, out, meta, heads, kv_heads, scale, slopes, sink, out_scale)
+        return
+    dt = _dt(q, k_cache, v_cache, out)
+    page, dp, vp = k_cache.shape[1], k_cache.shape[-1], v_cache.shape[-1]
+    if meta.num_tiles:
+        _native.call("tw_attn_prefill_grouped", q.data_ptr(), _row_stride(q), q.shape[0], k_cache.data_ptr(),
+                     v_cache.data_ptr(), k_cache.shape[0], page, out.data_ptr(), _row_stride(out), meta.cu_q.data_ptr(),
+                     meta.kv_lens.data_ptr(), meta.block_table.data_ptr(), meta.block_table.shape[1],
+                     meta.tile_seq.data_ptr(), meta.tile_q0.data_ptr(), meta.num_tiles, heads, kv_heads, dp, vp,
+                     float(scale), _p(slopes), int(sink), float(out_scale), status_word(q.device).data_ptr(), _stream())
+    n = meta.num_single
+    if n == 0:
+        return
+    plan, splits = attention_rows_plan(n, heads, kv_heads, dp, vp, page, q.dtype, meta.max_kv_len, sm_count)
+    if (kernel or plan) == "simt":
+        _native.call("tw_attn_rows", q.data_ptr(), _row_stride(q), k_cache.data_ptr(), v_cache.data_ptr(), page,
+                     out.data_ptr(), _row_stride(out), meta.tok_row.data_ptr(), meta.tok_seq.data_ptr(),
+                     meta.tok_kvlen.data_ptr(), n, meta.block_table.data_ptr(), meta.block_table.shape[1], heads, kv_heads,
+                     dp, vp, float(scale), _p(slopes), int(sink), float(out_scale), dt, _stream())
+        return
+    po = pm = None
+    if splits > 1:
+        po, pm = _partial_buffers(q.device, n * heads * splits, vp)
+    _native.call("tw_attn_decode_grouped", q.data_ptr(), _row_stride(q), k_cache.data_ptr(), v_cache.data_ptr(),
+                 k_cache.shape[0], page, out.data_ptr(), _row_stride(out), meta.tok_row.data_ptr(), meta.tok_seq.data_ptr(),
+                 meta.tok_kvlen.data_ptr(), n, meta.block_table.data_ptr(), meta.block_table.shape[1], heads, kv_heads, dp,
+                 vp, float(scale), _p(slopes), int(sink), float(out_scale), splits, _p(po), _p(pm),
+                 status_word(q.device).data_ptr(), _stream())

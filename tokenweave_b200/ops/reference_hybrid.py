@@ -97,33 +97,156 @@ def latent_values(o, rows, w_uv, heads, vdim, kv_rank, gate, out) -> None:
     out[r, : heads * vdim] = v.to(out.dtype)
 
 
+def _with_past(rows, state, slot: int, past: bool, taps: int):
+    """``rows`` behind the taps - 1 inputs before them, and the inputs to keep."""
+    before = state[slot].float() if past and taps > 1 else torch.zeros(taps - 1, rows.shape[1])
+    full = torch.cat([before, rows], 0)
+    return full, full[full.shape[0] - (taps - 1):]
+
+
 def causal_conv(x, weight, bias, state, out, cu_q, kv_lens, slots) -> None:
     taps, channels = weight.shape
     cu, kv, sl = cu_q.tolist(), kv_lens.tolist(), slots.tolist()
     w = weight.float()
     for b in range(len(kv)):
         rows = x[cu[b]:cu[b + 1], :channels].float()
-        past = state[sl[b]].float() if kv[b] > rows.shape[0] else torch.zeros(taps - 1, channels)
-        full = torch.cat([past, rows], 0)
+        full, keep = _with_past(rows, state, sl[b], kv[b] > rows.shape[0], taps)
         y = bias.float() + sum(w[k] * full[k:k + rows.shape[0]] for k in range(taps))
         out[cu[b]:cu[b + 1], :channels] = F.silu(y).to(out.dtype)
         if taps > 1:
-            state[sl[b]] = full[full.shape[0] - (taps - 1):].to(state.dtype)
+            state[sl[b]] = keep.to(state.dtype)
+
+
+def _recurrence(x, B, C, decay, step, D, state, y, seqs, cu_q, kv_lens, slots) -> None:
+    """``S <- decay_t S + step_t x B^T``, ``y = S C + D x``; x [T, H, P], B and C [T, H, N], decay and step [T, H]."""
+    cu, kv, sl = cu_q.tolist(), kv_lens.tolist(), slots.tolist()
+    _, heads, vdim, N = state.shape
+    for b in seqs.tolist():
+        s = state[sl[b]].clone() if kv[b] > cu[b + 1] - cu[b] else torch.zeros(heads, vdim, N)
+        for t in range(cu[b], cu[b + 1]):
+            s = decay[t][:, None, None] * s + (step[t][:, None] * x[t])[:, :, None] * B[t][:, None, :]
+            o = torch.einsum("hpn,hn->hp", s, C[t])
+            y[t, :heads * vdim] = (o if D is None else o + D[:, None] * x[t]).reshape(-1).to(y.dtype)
+        state[sl[b]] = s
 
 
 def ssd_scan(xbc, dt, dt_bias, A_log, D, state, y, seqs, cu_q, kv_lens, slots, groups: int) -> None:
     _, heads, vdim, N = state.shape
-    cu, kv, sl = cu_q.tolist(), kv_lens.tolist(), slots.tolist()
-    inner, rep = heads * vdim, heads // groups
+    inner, rep, T = heads * vdim, heads // groups, xbc.shape[0]
     step = F.softplus(dt[:, :heads].float() + dt_bias.float(), threshold=1e9)
     decay = torch.exp(-torch.exp(A_log.float()) * step)
-    for b in seqs.tolist():
-        s = state[sl[b]].clone() if kv[b] > cu[b + 1] - cu[b] else torch.zeros(heads, vdim, N)
-        for t in range(cu[b], cu[b + 1]):
-            r = xbc[t].float()
-            x = r[:inner].reshape(heads, vdim)
-            B = r[inner:inner + groups * N].reshape(groups, N).repeat_interleave(rep, 0)
-            C = r[inner + groups * N:inner + 2 * groups * N].reshape(groups, N).repeat_interleave(rep, 0)
-            s = decay[t][:, None, None] * s + (step[t][:, None] * x)[:, :, None] * B[:, None, :]
-            y[t, :inner] = (torch.einsum("hpn,hn->hp", s, C) + D.float()[:, None] * x).reshape(-1).to(y.dtype)
-        state[sl[b]] = s
+    r = xbc.float()
+    B, C = (r[:, inner + i * groups * N:inner + (i + 1) * groups * N].reshape(T, groups, N).repeat_interleave(rep, 1)
+            for i in (0, 1))
+    _recurrence(r[:, :inner].reshape(T, heads, vdim), B, C, decay, step, D.float(), state, y, seqs, cu_q, kv_lens, slots)
+
+
+def decay_scan(p, decay, state, y, seqs, cu_q, kv_lens, slots) -> None:
+    _, heads, vdim, N = state.shape
+    inner, T, r = heads * vdim, p.shape[0], p.float()
+    k, q = (r[:, inner + i * heads * N:inner + (i + 1) * heads * N].reshape(T, heads, N) for i in (0, 1))
+    one = torch.ones(T, heads)
+    _recurrence(r[:, :inner].reshape(T, heads, vdim), k, q, one * decay, one, None, state, y, seqs, cu_q, kv_lens, slots)
+
+
+# ---- blocks whose sublayers read one norm of the stream ---------------------------------------------------------
+def pair_rows(ids, row_seq, cu_q, prev_token, spec):
+    """Row of the pair table for every token; its last row for a token without one before it."""
+    ids = ids.long()
+    prev = torch.cat([ids[:1], ids[:-1]])
+    first = cu_q.long()[row_seq.long()] == torch.arange(len(ids))
+    prev = torch.where(first, prev_token.long()[row_seq.long()], prev)
+    buckets = int(spec["buckets"])
+    rows = (prev * int(spec["mul_prev"]) + ids * int(spec["mul_cur"])) % buckets
+    return torch.where(prev < 0, torch.full_like(rows, buckets), rows)
+
+
+def embed_norm(ids, table, pairs, spec, meta, x32, first, weight, eps: float, xa) -> None:
+    h = weight.numel()
+    ok = (ids >= 0) & (ids < table.shape[0])
+    x = table.index_select(0, torch.where(ok, ids, torch.zeros_like(ids)).long())[:, :h].float()
+    x = x * ok.unsqueeze(-1)
+    if pairs is not None:
+        x = x + pairs.index_select(0, pair_rows(ids, meta.extra["row_seq"], meta.cu_q, meta.extra["prev_token"],
+                                                spec))[:, :h].float()
+    x32[:, :h] = x
+    if first is not None:
+        first[:, :h] = x
+    xa[:, :h] = _unit(x, eps) * weight.float()
+
+
+def add_prenorm_(y, x32, first, weight, eps: float, xa) -> None:
+    h = weight.numel()
+    x = x32[:, :h]
+    x += y[:, :h].float()
+    if first is not None:
+        x += first[:, :h]
+    xa[:, :h] = _unit(x, eps) * weight.float()
+
+
+def gated_product(x, w, act: str, out) -> None:
+    d = w.shape[0] // 2
+    z = x.float() @ w.float().t()
+    g = F.silu(z[:, :d]) if act == "silu" else F.gelu(z[:, :d], approximate="tanh")
+    out.copy_(g * z[:, d:])
+
+
+def norm_gate(y, gate, weight, count: int, eps: float, scale: float, out) -> None:
+    v = y.float()
+    r = torch.rsqrt(v.pow(2).sum(-1, keepdim=True) / count + eps)
+    out.copy_(v * r * weight.float() * torch.sigmoid(gate.float()) * scale)
+
+
+def qkv_prep(p, heads: int, kv_heads: int, dim: int, vdim: int, q, k_cache, v_cache, meta, conv_w, conv_state, qk_norm,
+             wq, wk, eps: float, temp_coef: float, temp_every: int) -> None:
+    dp, vp, T = k_cache.shape[-1], v_cache.shape[-1], p.shape[0]
+    x = p.float()
+    if conv_w is not None:
+        taps, w = conv_w.shape[0], conv_w.float()
+        cu, kv, sl = meta.cu_q.tolist(), meta.kv_lens.tolist(), meta.extra.get("state_slots", meta.cu_q).tolist()
+        mixed = torch.empty_like(x)
+        for b in range(len(kv)):
+            rows = x[cu[b]:cu[b + 1]]
+            full, keep = _with_past(rows, conv_state, sl[b], kv[b] > rows.shape[0], taps)
+            mixed[cu[b]:cu[b + 1]] = sum(w[k] * full[k:k + rows.shape[0]] for k in range(taps))
+            if taps > 1:
+                conv_state[sl[b]] = keep.to(conv_state.dtype)
+        x = mixed
+    nq, nk = heads * dp, kv_heads * dp
+    qs, ks, vs = x[:, :nq], x[:, nq:nq + nk], x[:, nq + nk:]
+
+    def normed(t, weight, n):
+        parts = n if qk_norm == "head" else 1
+        t = t.reshape(T, parts, -1)
+        count = dim * n // parts
+        t = t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / count + eps) * weight.float()
+        return t.reshape(T, -1)
+    if qk_norm:
+        qs, ks = normed(qs, wq, heads), normed(ks, wk, kv_heads)
+    if temp_coef:
+        turn = torch.div(meta.positions.long() + 1, temp_every, rounding_mode="floor")
+        qs = qs * (1 + temp_coef * torch.log(turn.float() + 1)).unsqueeze(-1)
+    q.copy_(qs)
+    slots = meta.slot_mapping.long()
+    ok = slots >= 0
+    k_cache.view(-1, nk)[slots[ok]] = ks[ok].to(k_cache.dtype)
+    v_cache.view(-1, kv_heads * vp)[slots[ok]] = vs[ok].to(v_cache.dtype)
+
+
+def grouped_attention(q, k_cache, v_cache, out, meta, heads: int, kv_heads: int, scale: float, slopes, sink: bool,
+                      out_scale: float) -> None:
+    page, dp, vp, rep = k_cache.shape[1], k_cache.shape[-1], v_cache.shape[-1], heads // kv_heads
+    for b, kv_len in enumerate(meta.kv_lens_cpu):
+        t0, t1 = meta.cu_q_cpu[b], meta.cu_q_cpu[b + 1]
+        blocks = meta.block_table[b, :(kv_len + page - 1) // page].long()
+        k = k_cache.index_select(0, blocks).reshape(-1, kv_heads, dp)[:kv_len].float().repeat_interleave(rep, 1)
+        v = v_cache.index_select(0, blocks).reshape(-1, kv_heads, vp)[:kv_len].float().repeat_interleave(rep, 1)
+        s = torch.einsum("qhd,khd->hqk", q[t0:t1].reshape(t1 - t0, heads, dp).float(), k) * scale
+        dist = torch.arange(kv_len - (t1 - t0), kv_len).unsqueeze(-1) - torch.arange(kv_len)
+        if slopes is not None:
+            s = s - slopes[:, None, None] * dist
+        s = s.masked_fill(dist < 0, float("-inf"))
+        if sink:
+            s = torch.cat([s, torch.zeros(heads, t1 - t0, 1)], -1)
+        w = torch.softmax(s, -1)[..., :kv_len]
+        out[t0:t1] = (torch.einsum("hqk,khd->qhd", w, v) * out_scale).reshape(t1 - t0, -1).to(out.dtype)

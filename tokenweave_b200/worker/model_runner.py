@@ -221,7 +221,7 @@ class ModelRunner:
                                                       lora_id, nr.state_slot)
 
     def _build_metadata(self, entries, tokens_base: int, positions: np.ndarray, slots: np.ndarray,
-                        tables: dict[int, list[int]], which: int, state_slots: list) -> AttentionMetadata:
+                        tables: dict[int, list[int]], which: int, reqs: list) -> AttentionMetadata:
         """entries: list of (seq_index, q_len, kv_len) laid out back to back starting at row tokens_base."""
         q_lens = [e[1] for e in entries]
         kv_lens = [e[2] for e in entries]
@@ -235,7 +235,11 @@ class ModelRunner:
             bt[i, : len(t)] = t
         plan = extra = extra_cpu = None
         if self.plan_step is not None:
-            plan, extra, extra_cpu = self.plan_step(q_lens, kv_lens, [state_slots[e[0]] for e in entries])
+            own = [reqs[e[0]] for e in entries]
+            starts = [kv - q for q, kv in zip(q_lens, kv_lens)]
+            plan, extra, extra_cpu = self.plan_step(
+                q_lens, kv_lens, [r.state_slot for r in own],
+                [r.token_ids[s - 1] if s > 0 else -1 for r, s in zip(own, starts)])
         return build_attention_metadata(q_lens, kv_lens, positions[tokens_base:tokens_base + n],
                                         slots[tokens_base:tokens_base + n], bt, self.device, self._meta_host[which],
                                         self._meta_dev[which], plan=plan, extra=extra, extra_cpu=extra_cpu)
@@ -299,7 +303,7 @@ class ModelRunner:
         ids = self._ids_host.numpy()
         positions = np.empty(T, dtype=np.int32)
         slots = np.empty(T, dtype=np.int32)
-        q_lens, kv_lens, tables, state_slots = [], [], {}, []
+        q_lens, kv_lens, tables, step_reqs = [], [], {}, []
         want = step.want_logits
         logits_rows, sample_reqs = [], []
         row = 0
@@ -310,7 +314,7 @@ class ModelRunner:
         for b, (rid, computed, n_new, new_blocks, *rest) in enumerate(step.scheduled):
             req = self.requests[rid]
             req.block_ids.extend(new_blocks)
-            state_slots.append(req.state_slot)
+            step_reqs.append(req)
             drafts = list(rest[0]) if rest and rest[0] else []
             if n_new == 1 and not drafts and req.sampling_params.prompt_logprobs is None:
                 # decode fast path (most rows of a serving step): scalars only, no array temporaries
@@ -368,12 +372,12 @@ class ModelRunner:
         h2d = T * 4
         if plan.overlap:
             first, second = split_batch(q_lens, kv_lens, plan.split)
-            meta0 = self._build_metadata(first, 0, positions, slots, tables, 0, state_slots)
-            meta1 = self._build_metadata(second, plan.split, positions, slots, tables, 1, state_slots)
+            meta0 = self._build_metadata(first, 0, positions, slots, tables, 0, step_reqs)
+            meta1 = self._build_metadata(second, plan.split, positions, slots, tables, 1, step_reqs)
             step_in = StepInput(ids_dev, plan, meta0=meta0, meta1=meta1)
         else:
             entries = [(b, q_lens[b], kv_lens[b]) for b in range(len(q_lens))]
-            step_in = StepInput(ids_dev, plan, meta=self._build_metadata(entries, 0, positions, slots, tables, 0, state_slots))
+            step_in = StepInput(ids_dev, plan, meta=self._build_metadata(entries, 0, positions, slots, tables, 0, step_reqs))
         for m in (step_in.meta, step_in.meta0, step_in.meta1):
             if m is not None:
                 h2d += 4 * (2 * m.num_actual_tokens + 2 * m.num_seqs + 1 + m.block_table.numel() + 2 * m.num_tiles + 3 * m.num_single)
