@@ -21,9 +21,14 @@
 // O is rescaled lazily (only when a head's running maximum grew by more than 2^8), as in the prefill
 // kernel. With splits > 1 the un-normalised O, the reference maximum and the sum go to the partial
 // buffers that attn_decode_merge_kernel reduces. Every wait is bounded.
+//
+// The grouped form (tw_attn_decode_grouped) takes head sizes of queries / keys and values of their own up to 128, any
+// number of query heads per KV head (in blocks of 16), slope times distance off the scores, a sink and a factor on the
+// result; its probabilities enter the product with V as two bf16 terms, which keeps 16 bits of them.
 #include "tw_common.cuh"
 #include "tw_host.h"
 #include "tw_kernels.h"
+#include "tw_typed.cuh"
 
 namespace tw {
 
@@ -40,7 +45,7 @@ constexpr int DTC_OFF_K = 0;
 constexpr int DTC_OFF_V = DTC_OFF_K + DTC_RING * DTC_KV_BYTES;
 constexpr int DTC_OFF_Q = DTC_OFF_V + DTC_RING * DTC_KV_BYTES;
 constexpr int DTC_OFF_P = DTC_OFF_Q + DTC_Q_BYTES;             // two buffers
-constexpr int DTC_OFF_BAR = DTC_OFF_P + 2 * DTC_P_BYTES;
+constexpr int DTC_OFF_BAR = DTC_OFF_P + 4 * DTC_P_BYTES;      // (the second terms of the grouped form behind the first)
 constexpr int DTC_OFF_XCHG = DTC_OFF_BAR + 256;               // float [2][4 warps][16]
 constexpr int DTC_SMEM = DTC_OFF_XCHG + 2 * 4 * 16 * 4 + 1024;
 
@@ -67,12 +72,18 @@ struct DecodeTcParams {
   float* part_o;
   float* part_ml;
   uint32_t* status;
+  // grouped form
+  int dp, vp;              // padded sizes of queries / keys and values
+  int blocks;              // blocks of 16 query heads per KV head
+  const float* slopes;     // [hq] or null
+  int sink;
+  float out_scale;
 };
 
 // GT: query heads per KV head as a compile-time constant (4, 8 or 16), or 0 to read it from the arguments. The
 // softmax costs a few instructions per head, key and tile, all in the 128 threads that own the keys; with the
 // group size known the loops over the 16 columns of S^T shrink to the heads that exist.
-template <int GT>
+template <int GT, bool GROUPED>
 __global__ void __launch_bounds__(DTC_THREADS, 1)
 attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                       const DecodeTcParams p) {
@@ -100,8 +111,13 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
-  const int tok = blockIdx.x, kvh = blockIdx.y, split = blockIdx.z;
-  const int G = GT > 0 ? GT : p.hq / p.hkv;
+  const int tok = blockIdx.x, split = blockIdx.z;
+  const int kvh = GROUPED ? blockIdx.y / p.blocks : blockIdx.y;
+  const int g0 = GROUPED ? (blockIdx.y - kvh * p.blocks) * DTC_NH : 0;      // first head of this block
+  const int G = GT > 0 ? GT : GROUPED ? min(DTC_NH, p.hq / p.hkv - g0) : p.hq / p.hkv;
+  const int head0 = kvh * (p.hq / p.hkv) + g0;
+  const int DK = GROUPED ? p.dp : DTC_D, DV = GROUPED ? p.vp : DTC_D;
+  const int k_halves = GROUPED ? (p.dp + 63) / 64 : 2, v_halves = GROUPED ? (p.vp + 63) / 64 : 2;
   const int row = p.tok_row[tok];
   const int seq = p.tok_seq[tok];
   const int kv_len = p.tok_kvlen[tok];
@@ -148,20 +164,20 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         const uint32_t ph = (j / DTC_RING) & 1;
         const int tile = t_begin + j;
         if (!mbar_wait(&k_empty[st], ph ^ 1)) { report_error(p.status, TW_ERR_MBAR_TIMEOUT); *abort_flag = 1; break; }
-        mbar_expect_tx(&k_full[st], DTC_KV_BYTES);
+        mbar_expect_tx(&k_full[st], k_halves * DTC_HALF_BYTES);
         for (int pg = 0; pg < pages_per_tile; ++pg) {
           const int block = table[min(tile * pages_per_tile + pg, last_page)];
 #pragma unroll
-          for (int h = 0; h < 2; ++h)
+          for (int h = 0; h < k_halves; ++h)
             tma_load_4d(smem + DTC_OFF_K + st * DTC_KV_BYTES + h * DTC_HALF_BYTES + pg * p.page * 128, &tmK,
                         &k_full[st], h * 64, kvh, 0, block);
         }
         if (!mbar_wait(&v_empty[st], ph ^ 1)) { report_error(p.status, TW_ERR_MBAR_TIMEOUT); *abort_flag = 1; break; }
-        mbar_expect_tx(&v_full[st], DTC_KV_BYTES);
+        mbar_expect_tx(&v_full[st], v_halves * DTC_HALF_BYTES);
         for (int pg = 0; pg < pages_per_tile; ++pg) {
           const int block = table[min(tile * pages_per_tile + pg, last_page)];
 #pragma unroll
-          for (int h = 0; h < 2; ++h)
+          for (int h = 0; h < v_halves; ++h)
             tma_load_4d(smem + DTC_OFF_V + st * DTC_KV_BYTES + h * DTC_HALF_BYTES + pg * p.page * 128, &tmV,
                         &v_full[st], h * 64, kvh, 0, block);
         }
@@ -179,6 +195,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
         const uint32_t k_addr = smem_u32(smem + DTC_OFF_K + st * DTC_KV_BYTES);
 #pragma unroll
         for (int k = 0; k < DTC_D / 16; ++k) {
+          if (GROUPED && k >= 4 * k_halves) break;
           // 16 elements of the head dimension per instruction: 32 bytes along the swizzled 128-byte row
           const uint32_t a_off = (k >> 2) * DTC_HALF_BYTES + (k & 3) * 32;
           const uint32_t b_off = (k >> 2) * (DTC_NH * 128) + (k & 3) * 32;
@@ -208,6 +225,15 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
           umma_ss(tmem_base + COL_O, make_smem_desc_sw128(v_addr + k * 16 * 128, DTC_HALF_BYTES, 1024),
                   make_smem_desc_sw128(p_addr + b_off, 16, 1024), IDESC_O, (j | k) != 0 ? 1u : 0u);
         }
+        if (GROUPED) {
+          // the second terms of the probabilities (rows of O^T beyond the value size are never read)
+#pragma unroll
+          for (int k = 0; k < DTC_BN / 16; ++k) {
+            const uint32_t b_off = 2 * DTC_P_BYTES + (k >> 2) * (DTC_NH * 128) + (k & 3) * 32;
+            umma_ss(tmem_base + COL_O, make_smem_desc_sw128(v_addr + k * 16 * 128, DTC_HALF_BYTES, 1024),
+                    make_smem_desc_sw128(p_addr + b_off, 16, 1024), IDESC_O, 1u);
+          }
+        }
         umma_commit(&v_empty[st]);
         umma_commit(o_done);
       }
@@ -231,12 +257,12 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       for (int u = 0; u < 2; ++u) {
         const int cidx = (t & 7) * 2 + u;    // 16-byte chunk of the 128-element row
         uint4 v = make_uint4(0u, 0u, 0u, 0u);
-        if (g < G)
-          v = *reinterpret_cast<const uint4*>(p.q + row * p.ldq + (static_cast<long long>(kvh) * G + g) * DTC_D + cidx * 8);
+        if (g < G && (!GROUPED || cidx * 8 < DK))
+          v = *reinterpret_cast<const uint4*>(p.q + row * p.ldq + static_cast<long long>(head0 + g) * DK + cidx * 8);
         const int half = cidx >> 3, c = cidx & 7;
         *reinterpret_cast<uint4*>(smem + DTC_OFF_Q + half * (DTC_NH * 128) + g * 128 + ((c ^ (g & 7)) * 16)) = v;
       }
-      for (int i = t; i < 2 * DTC_P_BYTES / 16; i += 128)
+      for (int i = t; i < (GROUPED ? 4 : 2) * DTC_P_BYTES / 16; i += 128)
         *reinterpret_cast<uint4*>(smem + DTC_OFF_P + i * 16) = make_uint4(0u, 0u, 0u, 0u);
       fence_proxy_async_smem();
       mbar_arrive(q_ready);
@@ -250,6 +276,11 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       m_ref[g] = -INFINITY;
       l_part[g] = 0.f;
     }
+    float slope[DTC_NH];
+#pragma unroll
+    for (int g = 0; g < DTC_NH; ++g)
+      slope[g] = GROUPED && g < G && p.slopes != nullptr ? p.slopes[head0 + g] * 1.4426950408889634f : 0.f;
+    const float to_log2 = GROUPED ? 1.f : p.scale_log2;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
       // fixed trip count for all 128 threads (the named barrier below is unbounded): after a failed wait
@@ -265,6 +296,13 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       float s[DTC_NH], mx[DTC_NH];
 #pragma unroll
       for (int g = 0; g < DTC_NH; ++g) s[g] = __uint_as_float(sv[g]);
+      if (GROUPED) {
+        // in base 2, slope times distance (the key before the query: negative) added
+        const float dist = static_cast<float>((t_begin + j) * DTC_BN + r - (kv_len - 1));
+#pragma unroll
+        for (int g = 0; g < DTC_NH; ++g)
+          if (g < G) s[g] = fmaf(s[g], p.scale_log2, slope[g] * dist);
+      }
       if ((t_begin + j + 1) * DTC_BN > kv_len) {            // the same for the whole CTA
         const bool valid = (t_begin + j) * DTC_BN + r < kv_len;
 #pragma unroll
@@ -291,10 +329,10 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
           c = *reinterpret_cast<const float4*>(xm + 32 + g4);
           d = *reinterpret_cast<const float4*>(xm + 48 + g4);
         }
-        mt_all[g4] = fmaxf(fmaxf(a.x, b.x), fmaxf(c.x, d.x)) * p.scale_log2;
-        mt_all[g4 + 1] = fmaxf(fmaxf(a.y, b.y), fmaxf(c.y, d.y)) * p.scale_log2;
-        mt_all[g4 + 2] = fmaxf(fmaxf(a.z, b.z), fmaxf(c.z, d.z)) * p.scale_log2;
-        mt_all[g4 + 3] = fmaxf(fmaxf(a.w, b.w), fmaxf(c.w, d.w)) * p.scale_log2;
+        mt_all[g4] = fmaxf(fmaxf(a.x, b.x), fmaxf(c.x, d.x)) * to_log2;
+        mt_all[g4 + 1] = fmaxf(fmaxf(a.y, b.y), fmaxf(c.y, d.y)) * to_log2;
+        mt_all[g4 + 2] = fmaxf(fmaxf(a.z, b.z), fmaxf(c.z, d.z)) * to_log2;
+        mt_all[g4 + 3] = fmaxf(fmaxf(a.w, b.w), fmaxf(c.w, d.w)) * to_log2;
       }
       // The reference maxima move only when a head's maximum grew by more than 2^8 (rare after the first tiles):
       // one combined test here, the per-head work in the branch. All 128 threads see the same maxima and decide alike.
@@ -327,9 +365,12 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 #pragma unroll
       for (int g = 0; g < DTC_NH; ++g) {
         if (g < G) {
-          const float pv = dtc_exp2(fmaf(s[g], p.scale_log2, -m_ref[g]));
+          const float pv = dtc_exp2(fmaf(s[g], to_log2, -m_ref[g]));
           l_part[g] += pv;
-          *reinterpret_cast<__nv_bfloat16*>(p_buf + g * 128 + ((kc ^ (g & 7)) * 16) + ke * 2) = __float2bfloat16(pv);
+          const __nv_bfloat16 hi = __float2bfloat16(pv);
+          uint8_t* at = p_buf + g * 128 + ((kc ^ (g & 7)) * 16) + ke * 2;
+          *reinterpret_cast<__nv_bfloat16*>(at) = hi;
+          if (GROUPED) *reinterpret_cast<__nv_bfloat16*>(at + 2 * DTC_P_BYTES) = __float2bfloat16(pv - __bfloat162float(hi));
         }
       }
       // Every tile waits for the previous tile's P.V, needed or not: the parity wait only tells "the phase
@@ -382,13 +423,17 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 #pragma unroll
       for (int g = 0; g < DTC_NH; ++g) {
         if (g < G) {
-          const int h = kvh * G + g;
+          const int h = head0 + g;
           const float o = __uint_as_float(ov[g]);
-          if (p.splits == 1) {
-            p.out[row * p.ldo + h * DTC_D + d] = __float2bfloat16(l_tot[g] > 0.f ? o / l_tot[g] : 0.f);
+          if (GROUPED && d >= DV) {
+            continue;
+          } else if (p.splits == 1) {
+            const float l = GROUPED && p.sink ? l_tot[g] + dtc_exp2(-m_ref[g]) : l_tot[g];
+            const float v = l > 0.f ? o / l : 0.f;
+            p.out[row * p.ldo + h * DV + d] = __float2bfloat16(GROUPED ? v * p.out_scale : v);
           } else {
             const long long pidx = (static_cast<long long>(tok) * p.hq + h) * p.splits + split;
-            p.part_o[pidx * DTC_D + d] = o;
+            p.part_o[pidx * DV + d] = o;
             if (d == 0) {
               p.part_ml[pidx * 2] = m_ref[g];
               p.part_ml[pidx * 2 + 1] = l_tot[g];
@@ -414,6 +459,25 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     tmem_dealloc(tmem_base, TMEM_COLS);
   }
 }
+
+// Sum of the splits of one (token, head), with the sink and the factor of the grouped form.
+__global__ void __launch_bounds__(128)
+attn_decode_grouped_merge_kernel(const DecodeTcParams p) {
+  const int tok = blockIdx.x, h = blockIdx.y, d = threadIdx.x;
+  const long long base = (static_cast<long long>(tok) * p.hq + h) * p.splits;
+  float mm = -INFINITY;
+  for (int s = 0; s < p.splits; ++s) mm = fmaxf(mm, p.part_ml[(base + s) * 2]);
+  float acc = 0.f, ll = p.sink ? dtc_exp2(-mm) : 0.f;
+  for (int s = 0; s < p.splits; ++s) {
+    const float ms = p.part_ml[(base + s) * 2];
+    const float a = ms == -INFINITY ? 0.f : dtc_exp2(ms - mm);
+    if (d < p.vp) acc += p.part_o[(base + s) * p.vp + d] * a;
+    ll += p.part_ml[(base + s) * 2 + 1] * a;
+  }
+  if (d < p.vp)
+    p.out[p.tok_row[tok] * p.ldo + h * p.vp + d] = __float2bfloat16(ll > 0.f ? acc / ll * p.out_scale : 0.f);
+}
+
 
 // ---------------------------------------------------------------------------------------------------
 // Persistent variant: one CTA per SM walks the list of (token, KV head, split) items. TMEM, the barriers
@@ -855,18 +919,18 @@ extern "C" int tw_attn_decode_tc(const void* q, long long ldq, const void* k_cac
   int dev = 0;
   cudaGetDevice(&dev);
   if (configured_dev != dev) {
-    cudaError_t e = cudaFuncSetAttribute(attn_decode_tc_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
+    cudaError_t e = cudaFuncSetAttribute(attn_decode_tc_kernel<0, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(attn_decode_tc_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
+      e = cudaFuncSetAttribute(attn_decode_tc_kernel<4, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
     if (e == cudaSuccess)
-      e = cudaFuncSetAttribute(attn_decode_tc_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
+      e = cudaFuncSetAttribute(attn_decode_tc_kernel<8, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
     if (e != cudaSuccess) {
       set_last_error("attn_decode_tc: cudaFuncSetAttribute(smem=%d) failed: %s", DTC_SMEM, cudaGetErrorString(e));
       return 1;
     }
     configured_dev = dev;
   }
-  DecodeTcParams p;
+  DecodeTcParams p{};
   p.q = reinterpret_cast<const __nv_bfloat16*>(q);
   p.ldq = ldq;
   p.out = reinterpret_cast<__nv_bfloat16*>(out);
@@ -886,15 +950,99 @@ extern "C" int tw_attn_decode_tc(const void* q, long long ldq, const void* k_cac
   p.status = status;
   const dim3 grid(n_tok, hkv, splits);
   const int group = hq / hkv;
-  if (group == 8) attn_decode_tc_kernel<8><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tmK, tmV, p);
-  else if (group == 4) attn_decode_tc_kernel<4><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tmK, tmV, p);
-  else attn_decode_tc_kernel<0><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tmK, tmV, p);
+  if (group == 8) attn_decode_tc_kernel<8, false><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tmK, tmV, p);
+  else if (group == 4) attn_decode_tc_kernel<4, false><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tmK, tmV, p);
+  else attn_decode_tc_kernel<0, false><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tmK, tmV, p);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {
     set_last_error("attn_decode_tc launch failed: %s", cudaGetErrorString(e));
     return 1;
   }
   if (splits > 1) return tw_attn_decode_merge(part_o, part_ml, tok_row, n_tok, hq, D, splits, out, ldo, stream);
+  return 0;
+}
+
+// Grouped form: queries [T, hq * dp], caches [num_blocks, page, hkv, dp] and [.., vp] with dp and vp multiples of 8 up to
+// 128, any hq / hkv; see the head of the file.
+extern "C" int tw_attn_decode_grouped(const void* q, long long ldq, const void* k_cache, const void* v_cache,
+                                      int num_blocks, int page, void* out, long long ldo, const int* tok_row,
+                                      const int* tok_seq, const int* tok_kvlen, int n_tok, const int* block_table,
+                                      int max_blocks, int hq, int hkv, int dp, int vp, float scale, const float* slopes,
+                                      int sink, float out_scale, int splits, float* part_o, float* part_ml,
+                                      uint32_t* status, cudaStream_t stream) {
+  if (n_tok <= 0) return 0;
+  if (dp % 8 != 0 || vp % 8 != 0 || dp < 8 || vp < 8 || dp > DTC_D || vp > DTC_D || hkv <= 0 || hq % hkv != 0) {
+    set_last_error("attn_decode_grouped: head sizes must be multiples of 8 up to 128 (dp=%d, vp=%d, hq=%d, hkv=%d)", dp, vp,
+                   hq, hkv);
+    return 1;
+  }
+  if (page < 8 || page > 128 || (128 % page) != 0 || ldq % 8 != 0 || (reinterpret_cast<uintptr_t>(q) & 15) != 0) {
+    set_last_error("attn_decode_grouped: page size must divide 128 and be >= 8 (got %d); q rows 16-byte aligned", page);
+    return 1;
+  }
+  if (splits < 1) splits = 1;
+  if (splits > 1 && (part_o == nullptr || part_ml == nullptr)) {
+    set_last_error("attn_decode_grouped: split-KV needs the partial-result workspace");
+    return 1;
+  }
+  CUtensorMap tm[2];
+  for (int i = 0; i < 2; ++i) {
+    const uint64_t d = i == 0 ? dp : vp;
+    uint64_t dims[4] = {d, (uint64_t)hkv, (uint64_t)page, (uint64_t)num_blocks};
+    uint64_t strides[3] = {d * 2, (uint64_t)hkv * d * 2, (uint64_t)page * hkv * d * 2};
+    uint32_t box[4] = {64, 1, (uint32_t)page, 1};
+    if (!make_tensor_map_bf16(&tm[i], i == 0 ? k_cache : v_cache, 4, dims, strides, box)) return 1;
+  }
+  static thread_local int configured_dev = -1;
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (configured_dev != dev) {
+    cudaError_t e = cudaFuncSetAttribute(attn_decode_tc_kernel<0, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
+    if (e == cudaSuccess)
+      e = cudaFuncSetAttribute(attn_decode_tc_kernel<4, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
+    if (e == cudaSuccess)
+      e = cudaFuncSetAttribute(attn_decode_tc_kernel<8, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
+    if (e != cudaSuccess) {
+      set_last_error("attn_decode_grouped: cudaFuncSetAttribute(smem=%d) failed: %s", DTC_SMEM, cudaGetErrorString(e));
+      return 1;
+    }
+    configured_dev = dev;
+  }
+  const int group = hq / hkv;
+  DecodeTcParams p{};
+  p.q = reinterpret_cast<const __nv_bfloat16*>(q);
+  p.ldq = ldq;
+  p.out = reinterpret_cast<__nv_bfloat16*>(out);
+  p.ldo = ldo;
+  p.tok_row = tok_row;
+  p.tok_seq = tok_seq;
+  p.tok_kvlen = tok_kvlen;
+  p.block_table = block_table;
+  p.max_blocks = max_blocks;
+  p.page = page;
+  p.hq = hq;
+  p.hkv = hkv;
+  p.splits = splits;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.part_o = part_o;
+  p.part_ml = part_ml;
+  p.status = status;
+  p.dp = dp;
+  p.vp = vp;
+  p.blocks = (group + DTC_NH - 1) / DTC_NH;
+  p.slopes = slopes;
+  p.sink = sink;
+  p.out_scale = out_scale;
+  const dim3 grid(n_tok, hkv * p.blocks, splits);
+  if (group == 8) attn_decode_tc_kernel<8, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
+  else if (group == 4) attn_decode_tc_kernel<4, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
+  else attn_decode_tc_kernel<0, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
+  if (splits > 1) attn_decode_grouped_merge_kernel<<<dim3(n_tok, hq), 128, 0, stream>>>(p);
+  cudaError_t e = cudaGetLastError();
+  if (e != cudaSuccess) {
+    set_last_error("attn_decode_grouped launch failed: %s", cudaGetErrorString(e));
+    return 1;
+  }
   return 0;
 }
 
@@ -948,7 +1096,7 @@ extern "C" int tw_attn_decode_tc_persistent(const void* q, long long ldq, const 
     }
     configured_dev = dev;
   }
-  DecodeTcParams p;
+  DecodeTcParams p{};
   p.q = reinterpret_cast<const __nv_bfloat16*>(q);
   p.ldq = ldq;
   p.out = reinterpret_cast<__nv_bfloat16*>(out);

@@ -794,6 +794,10 @@ extern "C" int tw_attn_prefill(const void* q, long long ldq, int T, const void* 
   p.window = window > 0 ? window : 0;
   p.softcap = softcap > 0.f ? softcap : 0.f;
   p.scale = scale;
+  p.vdim = D;
+  p.slopes = nullptr;
+  p.sink = 0;
+  p.out_scale = 1.f;
   p.status = status;
   // Persistent kernel with the key range of an item split between the softmax groups (variant 3): the
   // only one that honours an SM budget.
@@ -807,6 +811,69 @@ extern "C" int tw_attn_prefill(const void* q, long long ldq, int T, const void* 
                     : launch_prefill_pair<64>(tmQ, tmK, tmV, p, num_tiles, stream);
   return D == 128 ? launch_prefill<128>(tmQ, tmK, tmV, p, num_tiles, stream)
                   : launch_prefill<64>(tmQ, tmK, tmV, p, num_tiles, stream);
+}
+
+// Grouped attention with its own sizes of queries / keys (dp) and values (vp), each a multiple of 8 up to 128: queries
+// [T, hq * dp], caches [num_blocks, page, hkv, dp] and [.., vp], out [T, hq * vp]. `slopes` [hq] (or null): slope times
+// distance is taken off the scaled score; `sink`: one more key of score 0 without a value; `out_scale`: factor on the
+// result. The softmax weights enter the product with the values as two bf16 terms.
+extern "C" int tw_attn_prefill_grouped(const void* q, long long ldq, int T, const void* k_cache, const void* v_cache,
+                                       int num_blocks, int page, void* out, long long ldo, const int* cu_q,
+                                       const int* kv_lens, const int* block_table, int max_blocks, const int* tile_seq,
+                                       const int* tile_q0, int num_tiles, int hq, int hkv, int dp, int vp, float scale,
+                                       const float* slopes, int sink, float out_scale, uint32_t* status,
+                                       cudaStream_t stream) {
+  if (num_tiles <= 0 || T <= 0) return 0;
+  if (dp % 8 != 0 || vp % 8 != 0 || dp < 8 || vp < 8 || dp > 128 || vp > 128) {
+    set_last_error("attn_prefill_grouped: head sizes must be multiples of 8 up to 128 (got %d and %d)", dp, vp);
+    return 1;
+  }
+  if (page < 8 || page > 128 || (128 % page) != 0) {
+    set_last_error("attn_prefill_grouped: page size must divide 128 and be >= 8 (got %d)", page);
+    return 1;
+  }
+  if (hkv <= 0 || hq % hkv != 0 || ldq % 8 != 0 || ldo % 8 != 0 || (reinterpret_cast<uintptr_t>(out) & 15) != 0) {
+    set_last_error("attn_prefill_grouped: bad head counts or strides");
+    return 1;
+  }
+  CUtensorMap tmQ, tmK, tmV;
+  {
+    // (head, row) as two dimensions: a box of 64 columns never reaches into the next head
+    uint64_t dims[3] = {(uint64_t)dp, (uint64_t)hq, (uint64_t)T};
+    uint64_t strides[2] = {(uint64_t)dp * 2, (uint64_t)ldq * 2};
+    uint32_t box[3] = {64, 1, ATT_BM};
+    if (!make_tensor_map_bf16(&tmQ, q, 3, dims, strides, box)) return 1;
+  }
+  for (int i = 0; i < 2; ++i) {
+    const uint64_t d = i == 0 ? dp : vp;
+    uint64_t dims[4] = {d, (uint64_t)hkv, (uint64_t)page, (uint64_t)num_blocks};
+    uint64_t strides[3] = {d * 2, (uint64_t)hkv * d * 2, (uint64_t)page * hkv * d * 2};
+    uint32_t box[4] = {64, 1, (uint32_t)page, 1};
+    if (!make_tensor_map_bf16(i == 0 ? &tmK : &tmV, i == 0 ? k_cache : v_cache, 4, dims, strides, box)) return 1;
+  }
+  AttnParams p;
+  p.out = reinterpret_cast<__nv_bfloat16*>(out);
+  p.ldo = ldo;
+  p.cu_q = cu_q;
+  p.kv_lens = kv_lens;
+  p.block_table = block_table;
+  p.tile_seq = tile_seq;
+  p.tile_q0 = tile_q0;
+  p.max_blocks = max_blocks;
+  p.page = page;
+  p.hq = hq;
+  p.hkv = hkv;
+  p.ring = 3;
+  p.scale_log2 = scale * 1.4426950408889634f;
+  p.window = 0;
+  p.softcap = 0.f;
+  p.scale = scale;
+  p.vdim = vp;
+  p.slopes = slopes;
+  p.sink = sink;
+  p.out_scale = out_scale;
+  p.status = status;
+  return launch_prefill_grouped(dp, vp, tmQ, tmK, tmV, p, num_tiles, stream);
 }
 
 // Kernel choice for tuning runs and tests: 0 automatic, 1 one head per CTA, 2 head pairs where legal,

@@ -83,11 +83,18 @@ struct AttnParams {
   int window;              // sliding window: a query at position p sees keys (p - window, p]; 0 = unlimited
   float softcap;           // logits soft cap: s -> cap * tanh(s / cap) on the scaled scores; 0 = off
   float scale;             // softmax scale (needed with the soft cap)
+  // grouped attention with its own value size (attn_prefill_split.cu only)
+  int vdim;                // value columns that are stored (a multiple of 8)
+  const float* slopes;     // [hq]: slope * distance is taken off the scaled score; null: off
+  int sink;                // one is added to the softmax's denominator
+  float out_scale;         // factor on the result
   uint32_t* status;
 };
 
 // Kernel of attn_prefill_split.cu: persistent CTAs, one query head per work item, the item's key range
 // split between the two softmax groups. max_ctas bounds the grid (0 = every SM).
+int launch_prefill_grouped(int D, int DV, const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
+                           const AttnParams& p, int num_tiles, cudaStream_t stream);
 int launch_prefill_split(int D, const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
                          const AttnParams& p, int num_tiles, int max_ctas, cudaStream_t stream);
 

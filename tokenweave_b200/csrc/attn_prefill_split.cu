@@ -24,6 +24,9 @@
 // exponentials as a cubic on the FMA pipe instead of ex2.approx (correct to 8e-5, but 17 to 25 % slower at
 // every share: the softmax warps are bound by issue slots, and the polynomial costs six times the
 // instructions of the MUFU form).
+// Grouped forms (OPTS 2 and 3): values of their own width, a sink, a factor on the result; OPTS 3 also takes slope times
+// distance off the scores. Their softmax weights reach the product with V as two bf16 terms (hi in the upper half of the
+// S columns, lo in the lower one: every score is in registers by then), which keeps 16 bits of them.
 // Replaces the FlashAttention-2 varlen call the reference makes on Blackwell
 // (vllm/v1/attention/backends/flash_attn.py:713-733, vllm/attention/utils/fa_utils.py:29-34).
 //
@@ -35,16 +38,17 @@
 #include "attn_prefill_common.cuh"
 #include "tw_host.h"
 #include "tw_kernels.h"
+#include "tw_mma.cuh"
 
 namespace tw {
 
 constexpr int SPL_RING = 3;   // K/V tile slots per softmax group
 
-template <int D>
+template <int D, int DV>
 struct SplitSmem {
-  static constexpr int HALVES = D / 64;
+  static constexpr int HALVES = D / 64, V_HALVES = DV / 64;
   static constexpr int Q_BYTES = HALVES * ATT_HALF_BYTES;
-  static constexpr int KV_BYTES = HALVES * ATT_HALF_BYTES;      // one K or V tile of 128 keys
+  static constexpr int KV_BYTES = (D > DV ? HALVES : V_HALVES) * ATT_HALF_BYTES;   // slot of one K or V tile of 128 keys
   static constexpr int OFF_Q = 0;
   static constexpr int OFF_RING = OFF_Q + Q_BYTES;              // [2 groups][SPL_RING]
   static constexpr int OFF_BAR = OFF_RING + 2 * SPL_RING * KV_BYTES;
@@ -84,17 +88,18 @@ __device__ __forceinline__ SplitItem split_item(const AttnParams& p, int idx) {
   return it;
 }
 
-// OPTS: sliding window and logits soft cap compiled in (a separate instantiation, so that the plain causal
-// kernel keeps its register budget).
-template <int D, bool OPTS>
+// MODE 1: sliding window and logits soft cap compiled in (separate instantiations, so that the plain causal kernel, MODE 0,
+// keeps its register budget); 2: grouped attention; 3: grouped attention with distance bias.
+template <int D, int DV, int MODE>
 __global__ void __launch_bounds__(ATT_THREADS, 1)
 attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                           const __grid_constant__ CUtensorMap tmV, const AttnParams p, const int total_items) {
-  using S = SplitSmem<D>;
+  using S = SplitSmem<D, DV>;
+  constexpr bool OPTS = MODE == 1, GROUPED = MODE >= 2, BIAS = MODE == 3;
   constexpr int HALVES = S::HALVES;
   constexpr int R = SPL_RING;
   constexpr uint32_t IDESC_QK = make_idesc_bf16(ATT_BM, ATT_BN, 0, 0);
-  constexpr uint32_t IDESC_PV = make_idesc_bf16(ATT_BM, D, 0, 1);
+  constexpr uint32_t IDESC_PV = make_idesc_bf16(ATT_BM, DV, 0, 1);
   constexpr uint32_t TMEM_COLS = 512;
   constexpr uint32_t COL_S = 0;     // S_A at 0, S_B at 128; P_g lives in columns [64, 128) of S_g
   constexpr uint32_t COL_P = 64;
@@ -162,20 +167,22 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         if (items_done > 0 && !mbar_wait(q_empty, (items_done - 1) & 1)) { ok = false; break; }
         mbar_expect_tx(q_full, S::Q_BYTES);
 #pragma unroll
-        for (int h = 0; h < HALVES; ++h)
-          tma_load_2d(smem + S::OFF_Q + h * ATT_HALF_BYTES, &tmQ, q_full, it.head * D + h * 64, it.q_begin + it.q0);
+        for (int h = 0; h < HALVES; ++h) {
+          if (GROUPED) tma_load_3d(smem + S::OFF_Q + h * ATT_HALF_BYTES, &tmQ, q_full, h * 64, it.head, it.q_begin + it.q0);
+          else tma_load_2d(smem + S::OFF_Q + h * ATT_HALF_BYTES, &tmQ, q_full, it.head * D + h * 64, it.q_begin + it.q0);
+        }
         const int last_page = (it.kv_len - 1) / p.page;
         const int* table = p.block_table + static_cast<long long>(it.seq) * p.max_blocks;
-        auto load_tile = [&](int g, const CUtensorMap* tm, int j) {
+        auto load_tile = [&](int g, const CUtensorMap* tm, int halves, int j) {
           const int slot = e[g] % R;
           const uint32_t ph = (e[g] / R) & 1;
           if (!mbar_wait(&ring_empty[g * R + slot], ph ^ 1)) return false;
-          mbar_expect_tx(&ring_full[g * R + slot], S::KV_BYTES);
+          mbar_expect_tx(&ring_full[g * R + slot], halves * ATT_HALF_BYTES);
           uint8_t* dst = smem + S::OFF_RING + (g * R + slot) * S::KV_BYTES;
           for (int pg = 0; pg < pages_per_tile; ++pg) {
             const int block = table[min(j * pages_per_tile + pg, last_page)];
 #pragma unroll
-            for (int h = 0; h < HALVES; ++h)
+            for (int h = 0; h < halves; ++h)
               tma_load_4d(dst + h * ATT_HALF_BYTES + pg * p.page * 128, tm, &ring_full[g * R + slot], h * 64, it.kvh, 0,
                           block);
           }
@@ -184,10 +191,10 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         };
         const int n_b = it.n_tiles - it.n_a;
         for (int t = 0; t < it.n_a && ok; ++t) {
-          ok = load_tile(0, &tmK, it.j_lo + t);
-          if (ok && t < n_b) ok = load_tile(1, &tmK, it.j_lo + it.n_a + t);
-          if (ok) ok = load_tile(0, &tmV, it.j_lo + t);
-          if (ok && t < n_b) ok = load_tile(1, &tmV, it.j_lo + it.n_a + t);
+          ok = load_tile(0, &tmK, HALVES, it.j_lo + t);
+          if (ok && t < n_b) ok = load_tile(1, &tmK, HALVES, it.j_lo + it.n_a + t);
+          if (ok) ok = load_tile(0, &tmV, S::V_HALVES, it.j_lo + t);
+          if (ok && t < n_b) ok = load_tile(1, &tmV, S::V_HALVES, it.j_lo + it.n_a + t);
         }
         ++items_done;
       }
@@ -242,6 +249,12 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
             umma_ts(tmem_base + COL_O + g * 128, tmem_base + COL_S + g * 128 + COL_P + k * 8,
                     make_smem_desc_sw128(v_addr + k * 16 * 128, ATT_HALF_BYTES, 1024), IDESC_PV,
                     (first && k == 0) ? 0u : 1u);
+          if (GROUPED) {
+#pragma unroll
+            for (int k = 0; k < ATT_BN / 16; ++k)
+              umma_ts(tmem_base + COL_O + g * 128, tmem_base + COL_S + g * 128 + k * 8,
+                      make_smem_desc_sw128(v_addr + k * 16 * 128, ATT_HALF_BYTES, 1024), IDESC_PV, 1u);
+          }
           umma_commit(&ring_empty[g * R + slot]);
           umma_commit(&o_done[g]);
           ++e[g];
@@ -311,6 +324,26 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
             s3[i] = __float_as_uint(cap_mul * fast_tanh(__uint_as_float(s3[i]) * cap_in));
           }
         }
+        if (BIAS) {
+          // scores in base 2 with the bias: slope * (key - position) is at most zero for every key that is seen
+          const float sl = p.slopes[it.head] * 1.4426950408889634f;
+          const float2 sl2 = make_float2(sl, sl), sc = make_float2(p.scale_log2, p.scale_log2);
+          auto bias_chunk = [&](uint32_t (&buf)[32], int chunk) {
+            const float b0 = sl * static_cast<float>(k_base + chunk * 32 - pos);
+            const float2 b2 = make_float2(b0, b0);
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+              const float2 b = fma2(make_float2(2 * i, 2 * i + 1), sl2, b2);
+              const float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc, b);
+              buf[2 * i] = __float_as_uint(x.x);
+              buf[2 * i + 1] = __float_as_uint(x.y);
+            }
+          };
+          bias_chunk(s0, 0);
+          bias_chunk(s1, 1);
+          bias_chunk(s2, 2);
+          bias_chunk(s3, 3);
+        }
         if (need_mask) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
@@ -329,7 +362,8 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
           m4[2] = max3f(m4[2], __uint_as_float(s2[2 * i]), __uint_as_float(s2[2 * i + 1]));
           m4[3] = max3f(m4[3], __uint_as_float(s3[2 * i]), __uint_as_float(s3[2 * i + 1]));
         }
-        const float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * p.scale_log2;
+        const float to_log2 = BIAS ? 1.f : p.scale_log2;
+        const float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * to_log2;
         float alpha = 1.f;
         bool rescale = false;
         if (t == 0) {
@@ -345,30 +379,35 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         // exponentials, two scores per instruction where the ISA has a packed form (scale and subtract,
         // running sum, bf16 conversion); 32 keys become 16 columns of P, which overwrites S columns
         // 64..127 (every score is in registers by now)
-        const float2 sc2 = make_float2(p.scale_log2, p.scale_log2);
+        const float2 sc2 = make_float2(to_log2, to_log2);
         const float2 nm2 = make_float2(-m_use, -m_use);
         float2 sum2[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
-        uint32_t pk[16];
+        uint32_t pk[16], lo[16];
         auto exp_chunk = [&](const uint32_t (&buf)[32]) {
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
             const float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc2, nm2);
             const float2 e = make_float2(fast_exp2(x.x), fast_exp2(x.y));
             sum2[i & 1] = fadd2(sum2[i & 1], e);
-            pk[i] = pack_bf16x2(e.x, e.y);
+            if (GROUPED) split_bf16x2(e.x, e.y, pk[i], lo[i]);
+            else pk[i] = pack_bf16x2(e.x, e.y);
           }
         };
+        auto store_chunk = [&](int chunk) {
+          tmem_st_32x16(t_p + chunk * 16, pk);
+          if (GROUPED) tmem_st_32x16(t_s + chunk * 16, lo);
+        };
         exp_chunk(s0);
-        tmem_st_32x16(t_p, pk);
+        store_chunk(0);
         exp_chunk(s1);
-        tmem_st_32x16(t_p + 16, pk);
+        store_chunk(1);
         if (t > 0 && __any_sync(0xffffffffu, rescale)) {
           // O_g may be touched once P V of the previous tile has completed
           if (ok) ok = mbar_wait(&o_done[g], (cnt - 1) & 1);
           tc_fence_after_sync();
           const uint32_t t_o = t_lane + COL_O + g * 128;
 #pragma unroll 1
-          for (int c = 0; c < D / 32; ++c) {
+          for (int c = 0; c < DV / 32; ++c) {
             uint32_t v[32];
             tmem_ld_32x32(t_o + c * 32, v);
             tmem_wait_ld();
@@ -378,9 +417,9 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
           }
         }
         exp_chunk(s2);
-        tmem_st_32x16(t_p + 32, pk);
+        store_chunk(2);
         exp_chunk(s3);
-        tmem_st_32x16(t_p + 48, pk);
+        store_chunk(3);
         l_sum = l_sum * alpha + ((sum2[0].x + sum2[0].y) + (sum2[1].x + sum2[1].y));
         tmem_wait_st();
         tc_fence_before_sync();
@@ -389,7 +428,7 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       }
       if (n_mine > 0 && ok) ok = mbar_wait(&o_done[g], (cnt - 1) & 1);
       tc_fence_after_sync();
-      // ---- epilogue: merge the two halves of the key range; group g writes output columns [g D/2, (g+1) D/2) ----
+      // ---- epilogue: merge the two halves of the key range; group g writes output columns [g DV/2, (g+1) DV/2) ----
       tmem_st_32x2(t_s, __float_as_uint(m_ref), __float_as_uint(l_sum));
       tmem_wait_st();
       tc_fence_before_sync();
@@ -403,14 +442,17 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       const float o_m = __uint_as_float(om_u), o_l = __uint_as_float(ol_u);
       const float m_all = fmaxf(m_ref, o_m);
       const float f_me = fast_exp2(m_ref - m_all), f_ot = fast_exp2(o_m - m_all);
-      const float inv = 1.f / (l_sum * f_me + o_l * f_ot);
+      float l_all = l_sum * f_me + o_l * f_ot;
+      if (GROUPED && p.sink) l_all += fast_exp2(-m_all);        // a key of score 0 (infinite: every key is negligible)
+      const float inv = (GROUPED ? p.out_scale : 1.f) / l_all;
       const float f_a = (g == 0 ? f_me : f_ot) * inv, f_b = (g == 0 ? f_ot : f_me) * inv;
       __nv_bfloat16* orow =
-          p.out + static_cast<long long>(it.q_begin + it.q0 + r) * p.ldo + it.head * D + g * (D / 2);
+          p.out + static_cast<long long>(it.q_begin + it.q0 + r) * p.ldo + it.head * p.vdim + g * (DV / 2);
+      const int v_left = p.vdim - g * (DV / 2);                  // columns from this group's first one on
 #pragma unroll 1
-      for (int c = 0; c < D / 64; ++c) {
+      for (int c = 0; c < DV / 64; ++c) {
         uint32_t a[32], b[32];
-        const uint32_t col = COL_O + g * (D / 2) + c * 32;
+        const uint32_t col = COL_O + g * (DV / 2) + c * 32;
         tmem_ld_32x32(t_lane + col, a);
         if (n_b > 0) tmem_ld_32x32(t_lane + col + 128, b);
         tmem_wait_ld();
@@ -430,7 +472,7 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
             o.y = pack_bf16x2(__uint_as_float(a[8 * q4 + 2]), __uint_as_float(a[8 * q4 + 3]));
             o.z = pack_bf16x2(__uint_as_float(a[8 * q4 + 4]), __uint_as_float(a[8 * q4 + 5]));
             o.w = pack_bf16x2(__uint_as_float(a[8 * q4 + 6]), __uint_as_float(a[8 * q4 + 7]));
-            *reinterpret_cast<uint4*>(orow + c * 32 + q4 * 8) = o;
+            if (!GROUPED || c * 32 + q4 * 8 < v_left) *reinterpret_cast<uint4*>(orow + c * 32 + q4 * 8) = o;
           }
         }
       }
@@ -459,11 +501,11 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
   }
 }
 
-template <int D, bool OPTS>
+template <int D, int DV, int MODE>
 static int launch_split_t(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnParams& p,
                           int num_tiles, int max_ctas, cudaStream_t stream) {
-  using S = SplitSmem<D>;
-  auto kern = attn_prefill_split_kernel<D, OPTS>;
+  using S = SplitSmem<D, DV>;
+  auto kern = attn_prefill_split_kernel<D, DV, MODE>;
   static thread_local int configured_dev = -1;
   int dev = 0;
   cudaGetDevice(&dev);
@@ -491,10 +533,25 @@ static int launch_split_t(const CUtensorMap& tmQ, const CUtensorMap& tmK, const 
 int launch_prefill_split(int D, const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
                          const AttnParams& p, int num_tiles, int max_ctas, cudaStream_t stream) {
   if (p.window > 0 || p.softcap > 0.f)
-    return D == 128 ? launch_split_t<128, true>(tmQ, tmK, tmV, p, num_tiles, max_ctas, stream)
-                    : launch_split_t<64, true>(tmQ, tmK, tmV, p, num_tiles, max_ctas, stream);
-  return D == 128 ? launch_split_t<128, false>(tmQ, tmK, tmV, p, num_tiles, max_ctas, stream)
-                  : launch_split_t<64, false>(tmQ, tmK, tmV, p, num_tiles, max_ctas, stream);
+    return D == 128 ? launch_split_t<128, 128, 1>(tmQ, tmK, tmV, p, num_tiles, max_ctas, stream)
+                    : launch_split_t<64, 64, 1>(tmQ, tmK, tmV, p, num_tiles, max_ctas, stream);
+  return D == 128 ? launch_split_t<128, 128, 0>(tmQ, tmK, tmV, p, num_tiles, max_ctas, stream)
+                  : launch_split_t<64, 64, 0>(tmQ, tmK, tmV, p, num_tiles, max_ctas, stream);
+}
+
+// D, DV: sizes of queries / keys and values, up to 128; tmQ is (column, head, row).
+int launch_prefill_grouped(int D, int DV, const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
+                           const AttnParams& p, int num_tiles, cudaStream_t stream) {
+#define TW_GO(A, B)                                                                                    \
+  return p.slopes != nullptr ? launch_split_t<A, B, 3>(tmQ, tmK, tmV, p, num_tiles, 0, stream)         \
+                             : launch_split_t<A, B, 2>(tmQ, tmK, tmV, p, num_tiles, 0, stream)
+  if (D > 64) {
+    if (DV > 64) TW_GO(128, 128);
+    TW_GO(128, 64);
+  }
+  if (DV > 64) TW_GO(64, 128);
+  TW_GO(64, 64);
+#undef TW_GO
 }
 
 }  // namespace tw

@@ -14,8 +14,8 @@
 // The tile width BN is a run-time value (a multiple of 32 up to 256; the instruction descriptor and
 // the pipeline depth are computed from it), chosen per problem by a wave-quantisation cost model:
 // skinny tensor-parallel shapes such as N = 1280 waste a third of the machine with 256-wide tiles.
-// Epilogues: plain, +bias[n], *row_scale[m], and SwiGLU (the B tile holds BN/2 "gate" rows and
-// BN/2 "up" rows; the stored value is silu(gate)*up, BN/2 output columns per tile).
+// Epilogues: plain, +bias[n], silu on a range of columns, *row_scale[m], and gated (the B tile holds BN/2 "gate" rows and
+// BN/2 "up" rows; the stored value is silu(gate)*up - SwiGLU - or gelu(gate)*up, BN/2 output columns per tile).
 // Grouped mode: each 128-row tile of A belongs to one expert (tile_expert[m_tile]); the B rows
 // are offset by expert * n_per_expert; the number of valid tiles is read from device memory.
 //
@@ -51,6 +51,8 @@ struct GemmParams {
   int bn;        // accumulator columns per tile
   int stages;    // pipeline depth
   int kb_per_stage;  // 64-wide k-blocks per stage: 2 halves the barrier round trips per FLOP
+  int glu;           // gated epilogue: GLU_SILU or GLU_GELU_TANH (bf16)
+  int silu_begin, silu_end;   // plain bf16 epilogue: silu on these columns (none: begin = end)
   uint32_t* status;
 };
 
@@ -235,6 +237,12 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           uint32_t u[32];
           tmem_ld_32x32(taddr + BN / 2 + c * 32, u);
           tmem_wait_ld();
+          if (!FP8 && p.glu == GLU_GELU_TANH) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              packed[j] = pack_bf16x2(epi_gelu_tanh(__uint_as_float(v[2 * j])) * __uint_as_float(u[2 * j]) * rs,
+                                      epi_gelu_tanh(__uint_as_float(v[2 * j + 1])) * __uint_as_float(u[2 * j + 1]) * rs);
+          } else
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
             float g0 = __uint_as_float(v[2 * j]), g1 = __uint_as_float(v[2 * j + 1]);
@@ -314,6 +322,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
             }
           }
           if (!FP8) {
+            epi_silu_cols(v, n0 + c * 32, p.silu_begin, p.silu_end);
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               packed[j] = pack_bf16x2(__uint_as_float(v[2 * j]) * rs, __uint_as_float(v[2 * j + 1]) * rs);
@@ -472,8 +481,8 @@ extern "C" int tw_gemm_set_kernel_override(int kind) {
 extern "C" int tw_gemm_pair(int fp8, const void* A, long long lda, const void* B, long long ldb, long long rows_b,
                             void* C, long long ldc, const void* bias, const float* row_scale, const float* col_scale,
                             int M, int N, int K, int swiglu, int up_row_offset, int bn, int max_ctas,
-                            const int* tile_expert, const int* num_m_tiles_dev, int n_per_expert, uint32_t* status,
-                            cudaStream_t stream);
+                            const int* tile_expert, const int* num_m_tiles_dev, int n_per_expert, int silu_begin,
+                            int silu_end, uint32_t* status, cudaStream_t stream);
 
 // Shared launcher body. A is [M,K] with row stride lda, B is [rows_b, K] with row stride ldb
 // (rows_b = N, 2*N for SwiGLU, or experts * n_per_expert); strides count elements (2 bytes, or 1 for fp8).
@@ -481,7 +490,8 @@ static int gemm_dispatch(bool fp8, const void* A, long long lda, const void* B, 
                          void* C, long long ldc, const void* bias, const float* row_scale, const float* col_scale,
                          int M, int N, int K, int swiglu, int up_row_offset, const int* tile_expert,
                          const int* num_m_tiles_dev, int n_per_expert, int max_ctas, int plan_hint,
-                         uint32_t* status, cudaStream_t stream, int group_tile_rows = 128) {
+                         uint32_t* status, cudaStream_t stream, int group_tile_rows = 128, int silu_begin = 0,
+                         int silu_end = 0) {
   // group_tile_rows: rows per entry of tile_expert (grouped mode). 256: the caller padded every expert to 256
   // rows, so the CTA-pair kernel can take the groups; 128: single-CTA tiles.
   // plan_hint: 0 = cost model; otherwise kernel * 1000 + tile width (kernel 1 = single-CTA tiles,
@@ -500,7 +510,7 @@ static int gemm_dispatch(bool fp8, const void* A, long long lda, const void* B, 
   const int num_m = (M + GEMM_BM - 1) / GEMM_BM;
   if (tile_expert != nullptr && group_tile_rows == 256 && sms >= 2)
     return tw_gemm_pair(fp8, A, lda, B, ldb, rows_b, C, ldc, bias, row_scale, col_scale, M, N, K, swiglu,
-                        up_row_offset, 256, sms, tile_expert, num_m_tiles_dev, n_per_expert, status, stream);
+                        up_row_offset, 256, sms, tile_expert, num_m_tiles_dev, n_per_expert, 0, 0, status, stream);
   // the cost model sees k-blocks: an fp8 problem has K / 128 of them
   GemmPlan plan = choose_plan(M, N, fp8 ? K / 2 : K, sms, swiglu != 0, tile_expert != nullptr);
   if (plan_hint > 0) {
@@ -512,7 +522,7 @@ static int gemm_dispatch(bool fp8, const void* A, long long lda, const void* B, 
   }
   if (plan.pair)
     return tw_gemm_pair(fp8, A, lda, B, ldb, rows_b, C, ldc, bias, row_scale, col_scale, M, N, K, swiglu, up_row_offset,
-                        plan.bn, sms, nullptr, nullptr, 0, status, stream);
+                        plan.bn, sms, nullptr, nullptr, 0, silu_begin, silu_end, status, stream);
   const int BN = plan.bn;
   const int out_cols = swiglu ? BN / 2 : BN;
   const int num_n = (N + out_cols - 1) / out_cols;
@@ -558,6 +568,9 @@ static int gemm_dispatch(bool fp8, const void* A, long long lda, const void* B, 
   p.bn = BN;
   p.stages = stages;
   p.kb_per_stage = kbps;
+  p.glu = swiglu;
+  p.silu_begin = silu_begin;
+  p.silu_end = silu_end;
   p.status = status;
   int grid = num_m * num_n;
   if (grid > sms) grid = sms;
@@ -576,6 +589,14 @@ extern "C" int tw_gemm_bf16(const void* A, long long lda, const void* B, long lo
   return gemm_dispatch(false, A, lda, B, ldb, rows_b, C, ldc, bias, row_scale, nullptr, M, N, K, swiglu,
                        up_row_offset, tile_expert, num_m_tiles_dev, n_per_expert, max_ctas, plan_hint, status,
                        stream);
+}
+
+// The same with silu on the columns [silu_begin, silu_end) of the result.
+extern "C" int tw_gemm_bf16_silu(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc,
+                                 const void* bias, int M, int N, int K, int silu_begin, int silu_end, int max_ctas,
+                                 int plan_hint, uint32_t* status, cudaStream_t stream) {
+  return gemm_dispatch(false, A, lda, B, ldb, N, C, ldc, bias, nullptr, nullptr, M, N, K, 0, 0, nullptr, nullptr, N,
+                       max_ctas, plan_hint, status, stream, 128, silu_begin, silu_end);
 }
 
 // Grouped GEMM over experts padded to 256 rows each: tile_expert has one entry per 256-row tile and the groups
@@ -623,5 +644,5 @@ extern "C" int tw_gemm_int8(const void* A, long long lda, const void* B, long lo
     bn = plan.pair ? plan.bn : (N > 128 || swiglu ? 256 : 128);
   }
   return tw_gemm_pair(2, A, lda, B, ldb, swiglu ? 2LL * N : N, C, ldc, bias, row_scale, col_scale, M, N, K, swiglu,
-                      swiglu ? N : 0, bn, sms, nullptr, nullptr, 0, status, stream);
+                      swiglu ? N : 0, bn, sms, nullptr, nullptr, 0, 0, 0, status, stream);
 }

@@ -1,4 +1,4 @@
-// Row-wise kernels around the residual stream and the feed-forward of models that norm a sublayer's OUTPUT.
+// Row-wise kernels around the fp32 residual stream and the feed-forward of hybrid decoders.
 // The residual stream is fp32; activations are bf16 or fp32 (template argument), all arithmetic is fp32.
 //
 //   tw_embed_residual   x32 = table[id] (the residual stream), xa = the same in the activation type
@@ -7,6 +7,11 @@
 //                       element by element (the activation between the two matrices of a feed-forward)
 //   tw_gated_group_norm out = groupnorm_rms(y * silu(z)) * w, the row cut in equal groups, each with its own
 //                       root mean square (what follows a state-space recurrence)
+//   tw_embed_norm       x32 = table[id] + pairs[row(previous id, id)] ; first = x32 ; xa = rmsnorm(x32) * w
+//   tw_add_prenorm      x32 += y (+ first) ; xa = rmsnorm(x32) * w (the next layer's norm, or the final one)
+//   tw_norm_gate        out = rmsnorm(y) * w * sigmoid(gate) * scale, the mean over `count` of the row's elements
+//   tw_silu_cols, tw_glu  activations behind a projection, for the fp32 products (the bf16 product has them in its
+//                       epilogue): silu in place, act(z_gate) * z_up
 //
 // One CTA per row (per row and group), the row kept in registers between the passes when it fits.
 #include "tw_host.h"
@@ -164,6 +169,170 @@ gated_group_norm_kernel(const T* __restrict__ y, long long ldy, const T* __restr
   }
 }
 
+struct EmbedArgs {
+  const int* ids;
+  const void* table; long long ldt; int vocab;
+  const void* pairs; long long ldp;                  // [buckets + 1, H]; null: no pair embeddings
+  long long buckets, mul_prev, mul_cur;
+  const int *row_seq, *cu_q, *prev_token;            // the token before a sequence's first row of the step, -1: none
+  float* x32; long long ldx;
+  float* first; long long ldf;                       // null: not kept
+  const void* w;
+  void* xa; long long lda;
+  int rows, H;
+  float eps;
+};
+
+template <typename T, bool VEC, int VPT>
+__global__ void __launch_bounds__(1024)
+embed_norm_kernel(const EmbedArgs a) {
+  __shared__ float scratch[32];
+  for (int t = blockIdx.x; t < a.rows; t += gridDim.x) {
+    const int id = a.ids[t];
+    const bool ok = id >= 0 && id < a.vocab;
+    const T* src = reinterpret_cast<const T*>(a.table) + (ok ? id : 0) * a.ldt;
+    const T* pair = nullptr;
+    if (a.pairs != nullptr) {
+      const int b = a.row_seq[t];
+      const int prev = t == a.cu_q[b] ? a.prev_token[b] : a.ids[t - 1];
+      long long row = a.buckets;
+      if (prev >= 0) {
+        row = (prev * a.mul_prev + id * a.mul_cur) % a.buckets;
+        if (row < 0) row += a.buckets;
+      }
+      pair = reinterpret_cast<const T*>(a.pairs) + row * a.ldp;
+    }
+    float v[VPT][8];
+    float ss[1] = {0.f};
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      ld8n<VEC>(src + i, a.H - i, v[k]);
+      if (!ok) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[k][j] = 0.f;
+      }
+      if (pair != nullptr) {
+        float u[8];
+        ld8n<VEC>(pair + i, a.H - i, u);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[k][j] += u[j];
+      }
+      if (i < a.H) {
+        st8n<VEC>(a.x32 + t * a.ldx + i, a.H - i, v[k]);
+        if (a.first != nullptr) st8n<VEC>(a.first + t * a.ldf + i, a.H - i, v[k]);
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss[0] += v[k][j] * v[k][j];
+    }
+    block_sum<1>(ss, scratch);
+    const float r = 1.f / sqrtf(ss[0] / static_cast<float>(a.H) + a.eps);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      if (i >= a.H) continue;
+      float g[8];
+      ld8n<VEC>(reinterpret_cast<const T*>(a.w) + i, a.H - i, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) g[j] = v[k][j] * r * g[j];
+      st8n<VEC>(reinterpret_cast<T*>(a.xa) + t * a.lda + i, a.H - i, g);
+    }
+  }
+}
+
+template <typename T, bool VEC, int VPT>
+__global__ void __launch_bounds__(1024)
+add_prenorm_kernel(const T* __restrict__ y, long long ldy, float* __restrict__ x32, long long ldx,
+                   const float* __restrict__ first, long long ldf, const T* __restrict__ w, T* __restrict__ xa,
+                   long long lda, int rows, int H, float eps) {
+  __shared__ float scratch[32];
+  for (int t = blockIdx.x; t < rows; t += gridDim.x) {
+    float v[VPT][8];
+    float ss[1] = {0.f};
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      float u[8];
+      ld8n<VEC>(x32 + t * ldx + i, H - i, v[k]);
+      ld8n<VEC>(y + t * ldy + i, H - i, u);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[k][j] += u[j];
+      if (first != nullptr) {
+        ld8n<VEC>(first + t * ldf + i, H - i, u);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[k][j] += u[j];
+      }
+      if (i < H) st8n<VEC>(x32 + t * ldx + i, H - i, v[k]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss[0] += v[k][j] * v[k][j];
+    }
+    block_sum<1>(ss, scratch);
+    const float r = 1.f / sqrtf(ss[0] / static_cast<float>(H) + eps);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      if (i >= H) continue;
+      float g[8];
+      ld8n<VEC>(w + i, H - i, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) g[j] = v[k][j] * r * g[j];
+      st8n<VEC>(xa + t * lda + i, H - i, g);
+    }
+  }
+}
+
+template <typename T, bool VEC, int VPT>
+__global__ void __launch_bounds__(1024)
+norm_gate_kernel(const T* __restrict__ y, long long ldy, const T* __restrict__ gate, long long ldg,
+                 const T* __restrict__ w, T* __restrict__ out, long long ldo, int rows, int C, float count, float eps,
+                 float scale) {
+  __shared__ float scratch[32];
+  for (int t = blockIdx.x; t < rows; t += gridDim.x) {
+    float v[VPT][8];
+    Raw8<T> graw[VPT];
+    float ss[1] = {0.f};
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      ld8n<VEC>(y + t * ldy + i, C - i, v[k]);
+      graw[k] = ld8raw<VEC>(gate + t * ldg + i, C - i);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) ss[0] += v[k][j] * v[k][j];
+    }
+    block_sum<1>(ss, scratch);
+    const float r = scale / sqrtf(ss[0] / count + eps);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8;
+      if (i >= C) continue;
+      float g[8];
+      ld8n<VEC>(w + i, C - i, g);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) g[j] *= v[k][j] * r * sigmoid_t<T>(ld1(&graw[k].v[j]));
+      st8n<VEC>(out + t * ldo + i, C - i, g);
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+silu_cols_kernel(T* __restrict__ x, long long ldx, int n) {
+  T* row = x + blockIdx.y * ldx;
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x)
+    st1(row + i, silu_t<T>(ld1(row + i)));
+}
+
+// z rows are [gate | up], d elements each; act 1: silu, 2: the tanh form of gelu
+template <typename T>
+__global__ void __launch_bounds__(256)
+glu_kernel(const T* __restrict__ z, long long ldz, T* __restrict__ out, long long ldo, int d, int act) {
+  const T* row = z + blockIdx.y * ldz;
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < d; i += gridDim.x * blockDim.x) {
+    const float g = ld1(row + i), u = ld1(row + d + i);
+    st1(out + blockIdx.y * ldo + i, (act == 2 ? gelu_tanh_f(g) : silu_t<T>(g)) * u);
+  }
+}
+
 static int check_launch(const char* what) {
   const cudaError_t e = cudaGetLastError();
   if (e == cudaSuccess) return 0;
@@ -285,4 +454,107 @@ extern "C" int tw_gated_group_norm(const void* y, long long ldy, const void* z, 
   }
 #undef TW_GO
   return check_launch("gated_group_norm");
+}
+
+extern "C" int tw_embed_norm(const int* ids, const void* table, long long ldt, int vocab, const void* pairs, long long ldp,
+                             long long buckets, long long mul_prev, long long mul_cur, const int* row_seq,
+                             const int* cu_q, const int* prev_token, float* x32, long long ldx, float* first,
+                             long long ldf, const void* w, void* xa, long long lda, int T, int H, float eps, int dtype,
+                             cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (pairs != nullptr && (buckets <= 0 || row_seq == nullptr || prev_token == nullptr)) {
+    set_last_error("embed_norm: token pairs need buckets and the tokens before the rows");
+    return 1;
+  }
+  int threads, vpt;
+  if (!row_shape(H, &threads, &vpt, "embed_norm")) return 1;
+  const int grid = row_grid(T, threads);
+  const bool vec = ldt % 8 == 0 && ldp % 8 == 0 && ldx % 8 == 0 && ldf % 8 == 0 && lda % 8 == 0 && aligned16(table) &&
+                   aligned16(pairs) && aligned16(x32) && aligned16(first) && aligned16(w) && aligned16(xa);
+  const EmbedArgs a{ids, table, ldt, vocab, pairs, ldp, buckets, mul_prev, mul_cur, row_seq, cu_q, prev_token,
+                    x32, ldx, first, ldf, w, xa, lda, T, H, eps};
+  if (dtype == TW_BF16) {
+    if (vec) { TW_ROW_VPT(embed_norm_kernel, __nv_bfloat16, true, a) } else { TW_ROW_VPT(embed_norm_kernel, __nv_bfloat16, false, a) }
+  } else {
+    if (vec) { TW_ROW_VPT(embed_norm_kernel, float, true, a) } else { TW_ROW_VPT(embed_norm_kernel, float, false, a) }
+  }
+  return check_launch("embed_norm");
+}
+
+extern "C" int tw_add_prenorm(const void* y, long long ldy, float* x32, long long ldx, const float* first, long long ldf,
+                              const void* w, void* xa, long long lda, int T, int H, float eps, int dtype,
+                              cudaStream_t stream) {
+  if (T <= 0) return 0;
+  int threads, vpt;
+  if (!row_shape(H, &threads, &vpt, "add_prenorm")) return 1;
+  const int grid = row_grid(T, threads);
+  const bool vec = ldy % 8 == 0 && ldx % 8 == 0 && ldf % 8 == 0 && lda % 8 == 0 && aligned16(y) && aligned16(x32) &&
+                   aligned16(first) && aligned16(w) && aligned16(xa);
+#define TW_GO(TT, V)                                                                                             \
+  TW_ROW_VPT(add_prenorm_kernel, TT, V, reinterpret_cast<const TT*>(y), ldy, x32, ldx, first, ldf,               \
+             reinterpret_cast<const TT*>(w), reinterpret_cast<TT*>(xa), lda, T, H, eps)
+  if (dtype == TW_BF16) {
+    if (vec) TW_GO(__nv_bfloat16, true) else TW_GO(__nv_bfloat16, false)
+  } else {
+    if (vec) TW_GO(float, true) else TW_GO(float, false)
+  }
+#undef TW_GO
+  return check_launch("add_prenorm");
+}
+
+extern "C" int tw_norm_gate(const void* y, long long ldy, const void* gate, long long ldg, const void* w, void* out,
+                            long long ldo, int T, int C, int count, float eps, float scale, int dtype,
+                            cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (count <= 0 || count > C) {
+    set_last_error("norm_gate: %d elements of a row of %d", count, C);
+    return 1;
+  }
+  int threads, vpt;
+  if (!row_shape(C, &threads, &vpt, "norm_gate")) return 1;
+  const int grid = row_grid(T, threads);
+  const bool vec = ldy % 8 == 0 && ldg % 8 == 0 && ldo % 8 == 0 && aligned16(y) && aligned16(gate) && aligned16(w) &&
+                   aligned16(out);
+#define TW_GO(TT, V)                                                                                                 \
+  TW_ROW_VPT(norm_gate_kernel, TT, V, reinterpret_cast<const TT*>(y), ldy, reinterpret_cast<const TT*>(gate), ldg,   \
+             reinterpret_cast<const TT*>(w), reinterpret_cast<TT*>(out), ldo, T, C, static_cast<float>(count), eps, scale)
+  if (dtype == TW_BF16) {
+    if (vec) TW_GO(__nv_bfloat16, true) else TW_GO(__nv_bfloat16, false)
+  } else {
+    if (vec) TW_GO(float, true) else TW_GO(float, false)
+  }
+#undef TW_GO
+  return check_launch("norm_gate");
+}
+
+// Grid of the two elementwise kernels; the row is the second grid dimension, launched in blocks of 65535 rows.
+extern "C" int tw_silu_cols(void* x, long long ldx, int T, int n, int dtype, cudaStream_t stream) {
+  if (T <= 0 || n <= 0) return 0;
+  const int gx = (n + 1023) / 1024;
+  for (int t = 0; t < T; t += 65535) {
+    const dim3 grid(gx, T - t < 65535 ? T - t : 65535);
+    if (dtype == TW_BF16) silu_cols_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<__nv_bfloat16*>(x) + t * ldx, ldx, n);
+    else silu_cols_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<float*>(x) + t * ldx, ldx, n);
+  }
+  return check_launch("silu_cols");
+}
+
+extern "C" int tw_glu(const void* z, long long ldz, void* out, long long ldo, int T, int d, int act, int dtype,
+                      cudaStream_t stream) {
+  if (T <= 0 || d <= 0) return 0;
+  if (act != 1 && act != 2) {
+    set_last_error("glu: unknown activation %d", act);
+    return 1;
+  }
+  const int gx = (d + 1023) / 1024;
+  for (int t = 0; t < T; t += 65535) {
+    const dim3 grid(gx, T - t < 65535 ? T - t : 65535);
+    if (dtype == TW_BF16)
+      glu_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<const __nv_bfloat16*>(z) + t * ldz, ldz,
+                                           reinterpret_cast<__nv_bfloat16*>(out) + t * ldo, ldo, d, act);
+    else
+      glu_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<const float*>(z) + t * ldz, ldz,
+                                           reinterpret_cast<float*>(out) + t * ldo, ldo, d, act);
+  }
+  return check_launch("glu");
 }

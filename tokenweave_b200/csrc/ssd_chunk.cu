@@ -25,7 +25,8 @@ namespace tw {
 struct ChunkArgs {
   const __nv_bfloat16* xbc; long long ldx;       // [T, heads * vdim | groups * N | groups * N]
   const __nv_bfloat16* dt; long long ldt;        // [T, heads]
-  const __nv_bfloat16 *dt_bias, *A_log, *D;      // [heads]
+  const __nv_bfloat16 *dt_bias, *A_log, *D;      // [heads]; unused with `decay`
+  const float* decay;                            // [heads]: fixed decays, unit steps, no skip
   float* state;                                  // [slots, heads, vdim, N]
   __nv_bfloat16* y; long long ldy;
   const int *seqs, *cu_q, *kv_lens, *slots;
@@ -59,18 +60,19 @@ struct ChunkSums {
 __device__ __forceinline__ float2 chunk_steps(const ChunkArgs& a, int t0, int t_end, int h, int lane) {
   float2 r = make_float2(0.f, 0.f);
   const int t = t0 + 2 * lane;
+  if (a.decay != nullptr) return r;
   if (t < t_end) r.x = ld1(a.dt + t * a.ldt + h);
   if (t + 1 < t_end) r.y = ld1(a.dt + (t + 1) * a.ldt + h);
   return r;
 }
 
-__device__ __forceinline__ void chunk_sums(ChunkSums* s, float2 raw, int n, float bias, float A, int lane) {
+__device__ __forceinline__ void chunk_sums(ChunkSums* s, float2 raw, int n, float bias, double A, bool fixed, int lane) {
   double l[2];
   float d[2];
 #pragma unroll
   for (int e = 0; e < 2; ++e) {
-    d[e] = 2 * lane + e < n ? softplus_f((e ? raw.y : raw.x) + bias) : 0.f;
-    l[e] = -static_cast<double>(A) * d[e];
+    d[e] = 2 * lane + e >= n ? 0.f : fixed ? 1.f : softplus_f((e ? raw.y : raw.x) + bias);
+    l[e] = -A * d[e];
   }
   double run = l[0] + l[1];
 #pragma unroll
@@ -134,7 +136,9 @@ ssd_chunk_kernel(const ChunkArgs a) {
   const int p_valid = min(CH_P, a.vdim - p0);
   const int g = h / (a.heads / a.groups);
   const int off_x = h * a.vdim + p0, off_b = a.heads * a.vdim + g * a.N, off_c = off_b + a.groups * a.N;
-  const float bias = ld1(a.dt_bias + h), A = expf(ld1(a.A_log + h)), D = ld1(a.D + h);
+  const bool fixed = a.decay != nullptr;
+  const float bias = fixed ? 0.f : ld1(a.dt_bias + h), D = fixed ? 0.f : ld1(a.D + h);
+  const double A = fixed ? decay_rate(a.decay[h]) : static_cast<double>(expf(ld1(a.A_log + h)));
   // tile of the lower triangle this warp makes (warps 0..9)
   const int ti = warp < 1 ? 0 : warp < 3 ? 1 : warp < 6 ? 2 : 3, tj = warp - ti * (ti + 1) / 2;
 
@@ -154,7 +158,7 @@ ssd_chunk_kernel(const ChunkArgs a) {
   float2 steps = make_float2(0.f, 0.f);      // warp 15: raw step sizes of the next chunk
   if (warp == 15) {
     steps = chunk_steps(a, t_begin, t_end, h, lane);
-    chunk_sums(&sums[0], steps, t_end - t_begin, bias, A, lane);
+    chunk_sums(&sums[0], steps, t_end - t_begin, bias, A, fixed, lane);
     steps = chunk_steps(a, t_begin + CH_L, t_end, h, lane);
   }
 
@@ -214,7 +218,7 @@ ssd_chunk_kernel(const ChunkArgs a) {
     } else if (warp == 15 && more) {
       const float2 now = steps;
       steps = chunk_steps(a, t0 + 2 * CH_L, t_end, h, lane);
-      chunk_sums(&sums[(c + 1) & 1], now, t_end - t0 - CH_L, bias, A, lane);
+      chunk_sums(&sums[(c + 1) & 1], now, t_end - t0 - CH_L, bias, A, fixed, lane);
     }
     // weighted inputs: eight values per thread
     {
@@ -345,9 +349,26 @@ static int launch_chunk(const ChunkArgs& a, int n_seqs, cudaStream_t stream) {
 }
 
 int launch_ssd_chunk_tc(const void* xbc, long long ldx, int T, const void* dt, long long ldt, const void* dt_bias,
-                        const void* A_log, const void* D, float* state, void* y, long long ldy, const int* seqs,
-                        int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads, int vdim, int N,
-                        int groups, uint32_t* status, cudaStream_t stream);
+                        const void* A_log, const void* D, const float* decay, float* state, void* y, long long ldy,
+                        const int* seqs, int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads,
+                        int vdim, int N, int groups, uint32_t* status, cudaStream_t stream);
+
+static int chunk_dispatch(const char* what, const ChunkArgs& a, int T, int n_seqs, int form, uint32_t* status,
+                          cudaStream_t stream) {
+  if (n_seqs <= 0) return 0;
+  if (a.groups <= 0 || a.heads % a.groups != 0 || a.vdim % 8 != 0 || a.N % 8 != 0 || a.ldx % 8 != 0 || a.ldy % 2 != 0 ||
+      a.N > 256 || (reinterpret_cast<uintptr_t>(a.xbc) & 15) != 0) {
+    set_last_error("%s: vdim and N (<= 256) must be multiples of 8 in 16-byte rows (vdim=%d, N=%d, ldx=%lld)", what, a.vdim,
+                   a.N, a.ldx);
+    return 1;
+  }
+  if (form == 0 && a.N <= 128 && a.ldy % 8 == 0 && (reinterpret_cast<uintptr_t>(a.y) & 15) == 0)
+    return launch_ssd_chunk_tc(a.xbc, a.ldx, T, a.dt, a.ldt, a.dt_bias, a.A_log, a.D, a.decay, a.state, a.y, a.ldy, a.seqs,
+                               n_seqs, a.cu_q, a.kv_lens, a.slots, a.heads, a.vdim, a.N, a.groups, status, stream);
+  if (a.N <= 64) return launch_chunk<64>(a, n_seqs, stream);
+  if (a.N <= 128) return launch_chunk<128>(a, n_seqs, stream);
+  return launch_chunk<256>(a, n_seqs, stream);
+}
 
 }  // namespace tw
 
@@ -359,22 +380,21 @@ extern "C" int tw_ssd_chunk(const void* xbc, long long ldx, int T, const void* d
                             const void* A_log, const void* D, float* state, void* y, long long ldy, const int* seqs,
                             int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads, int vdim, int N,
                             int groups, int form, uint32_t* status, cudaStream_t stream) {
-  if (n_seqs <= 0) return 0;
-  if (groups <= 0 || heads % groups != 0 || vdim % 8 != 0 || N % 8 != 0 || ldx % 8 != 0 || ldy % 2 != 0 || N > 256 ||
-      (reinterpret_cast<uintptr_t>(xbc) & 15) != 0) {
-    set_last_error("ssd_chunk: vdim and N (<= 256) must be multiples of 8 in 16-byte rows (vdim=%d, N=%d, ldx=%lld)", vdim,
-                   N, ldx);
-    return 1;
-  }
-  if (form == 0 && N <= 128 && ldy % 8 == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0)
-    return launch_ssd_chunk_tc(xbc, ldx, T, dt, ldt, dt_bias, A_log, D, state, y, ldy, seqs, n_seqs, cu_q, kv_lens, slots,
-                               heads, vdim, N, groups, status, stream);
   using bf = __nv_bfloat16;
   const ChunkArgs a{reinterpret_cast<const bf*>(xbc), ldx, reinterpret_cast<const bf*>(dt), ldt,
                     reinterpret_cast<const bf*>(dt_bias), reinterpret_cast<const bf*>(A_log),
-                    reinterpret_cast<const bf*>(D), state, reinterpret_cast<bf*>(y), ldy, seqs, cu_q, kv_lens, slots,
-                    heads, vdim, N, groups};
-  if (N <= 64) return launch_chunk<64>(a, n_seqs, stream);
-  if (N <= 128) return launch_chunk<128>(a, n_seqs, stream);
-  return launch_chunk<256>(a, n_seqs, stream);
+                    reinterpret_cast<const bf*>(D), nullptr, state, reinterpret_cast<bf*>(y), ldy, seqs, cu_q, kv_lens,
+                    slots, heads, vdim, N, groups};
+  return chunk_dispatch("ssd_chunk", a, T, n_seqs, form, status, stream);
+}
+
+// The same with unit steps, a given decay per head and no skip; vkq rows are [values | keys | queries] of all heads.
+extern "C" int tw_decay_chunk(const void* vkq, long long ldx, int T, const float* decay, float* state, void* y,
+                              long long ldy, const int* seqs, int n_seqs, const int* cu_q, const int* kv_lens,
+                              const int* slots, int heads, int vdim, int N, int form, uint32_t* status,
+                              cudaStream_t stream) {
+  using bf = __nv_bfloat16;
+  const ChunkArgs a{reinterpret_cast<const bf*>(vkq), ldx, nullptr, 0, nullptr, nullptr, nullptr, decay, state,
+                    reinterpret_cast<bf*>(y), ldy, seqs, cu_q, kv_lens, slots, heads, vdim, N, heads};
+  return chunk_dispatch("decay_chunk", a, T, n_seqs, form, status, stream);
 }

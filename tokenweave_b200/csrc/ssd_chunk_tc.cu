@@ -36,6 +36,7 @@ constexpr int SC_CHUNK = SC_L * 128;               // 128 rows x 64 bf16, swizzl
 struct ScanTcParams {
   const __nv_bfloat16* dt; long long ldt;
   const __nv_bfloat16 *dt_bias, *A_log, *D;
+  const float* decay;                              // [heads]: fixed decays, unit steps, no skip (the four above unused)
   float* state;
   __nv_bfloat16* y; long long ldy;
   const int *seqs, *cu_q, *kv_lens, *slots;
@@ -237,7 +238,7 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
     const int grp = (warp - 2) >> 2, qr = warp & 3;
     const int r = qr * 32 + lane;                               // token of the chunk
     const uint32_t t_lane = tmem_base + (static_cast<uint32_t>(qr * 32) << 16);
-    const float D = ld1(p.D + h);
+    const float D = p.decay != nullptr ? 0.f : ld1(p.D + h);
     auto epilogue = [&](int c) {
       const int st = c & 1;
       if (ok) ok = mbar_wait(y_full, c & 1);
@@ -386,15 +387,17 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
     }
   } else {
     // ---------------- running sums: four tokens per lane ----------------
-    const float bias = ld1(p.dt_bias + h), A = expf(ld1(p.A_log + h));
+    const bool fixed = p.decay != nullptr;
+    const float bias = fixed ? 0.f : ld1(p.dt_bias + h);
     auto request = [&](int c, float (&raw)[4]) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int t = t_begin + c * SC_L + 4 * lane + e;
-        raw[e] = t < t_end ? ld1(p.dt + t * p.ldt + h) : 0.f;
+        raw[e] = t < t_end && !fixed ? ld1(p.dt + t * p.ldt + h) : 0.f;
       }
     };
-    const double rate = -static_cast<double>(A) * 1.4426950408889634;
+    const double A = fixed ? decay_rate(p.decay[h]) : static_cast<double>(expf(ld1(p.A_log + h)));
+    const double rate = -A * 1.4426950408889634;
     float next[4];
     request(0, next);
     for (int c = 0; c < n_ch; ++c) {
@@ -406,7 +409,7 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
       double l[4];
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        d[e] = 4 * lane + e < n ? softplus_call(raw[e] + bias) : 0.f;
+        d[e] = 4 * lane + e >= n ? 0.f : fixed ? 1.f : softplus_call(raw[e] + bias);
         l[e] = rate * d[e] + (e > 0 ? l[e - 1] : 0.0);
       }
       double run = l[3];
@@ -456,11 +459,11 @@ ssd_chunk_tc_kernel(const __grid_constant__ CUtensorMap tmX, const __grid_consta
   }
 }
 
-// Called by tw_ssd_chunk for states of up to 128 dimensions. BC: base of [B groups | C groups] in the rows.
+// Called by tw_ssd_chunk and tw_decay_chunk for states of up to 128 dimensions. BC: base of [B groups | C groups] in the rows.
 int launch_ssd_chunk_tc(const void* xbc, long long ldx, int T, const void* dt, long long ldt, const void* dt_bias,
-                        const void* A_log, const void* D, float* state, void* y, long long ldy, const int* seqs,
-                        int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads, int vdim, int N,
-                        int groups, uint32_t* status, cudaStream_t stream) {
+                        const void* A_log, const void* D, const float* decay, float* state, void* y, long long ldy,
+                        const int* seqs, int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads,
+                        int vdim, int N, int groups, uint32_t* status, cudaStream_t stream) {
   using bf = __nv_bfloat16;
   CUtensorMap tmX, tmBC;
   {
@@ -489,7 +492,7 @@ int launch_ssd_chunk_tc(const void* xbc, long long ldx, int T, const void* dt, l
     configured_dev = dev;
   }
   const ScanTcParams p{reinterpret_cast<const bf*>(dt), ldt, reinterpret_cast<const bf*>(dt_bias),
-                       reinterpret_cast<const bf*>(A_log), reinterpret_cast<const bf*>(D), state,
+                       reinterpret_cast<const bf*>(A_log), reinterpret_cast<const bf*>(D), decay, state,
                        reinterpret_cast<bf*>(y), ldy, seqs, cu_q, kv_lens, slots, heads, vdim, N, groups, (N + 63) / 64,
                        status};
   ssd_chunk_tc_kernel<<<dim3(n_seqs, heads, (vdim + SC_P - 1) / SC_P), SC_THREADS, SC_SMEM, stream>>>(tmX, tmBC, p);

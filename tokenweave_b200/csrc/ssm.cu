@@ -6,8 +6,11 @@
 //   tw_causal_conv       per-channel causal convolution with bias and silu. The taps - 1 inputs before a sequence's
 //                        first row come from its convolution state [slot, taps - 1, channels] (oldest first), which
 //                        is moved on by the second launch; a step of single-token sequences does both in one launch
+//   tw_conv_state        the second launch alone, for kernels that convolve on their own
 //   tw_ssd_scan          token-by-token recurrence S <- exp(-exp(A) dt) S + dt B x^T, y = S^T C + D x, dt =
 //                        softplus(raw + bias): decoding, short portions, fp32
+//   tw_decay_scan        the same with unit steps, a given decay per head and no skip (lightning attention: x = values,
+//                        B = keys, C = queries, every head a group of its own)
 //
 // State layout [slot, head, vdim, state]: a warp owns rows of vdim, its lanes the state dimension.
 #include "tw_host.h"
@@ -162,7 +165,8 @@ causal_conv_step_kernel(const ConvArgs a) {
 struct ScanArgs {
   const void* xbc; long long ldx;              // [T, heads * vdim | groups * state | groups * state]
   const void* dt; long long ldt;               // [T, heads] raw step sizes
-  const void* dt_bias; const void* A_log; const void* D;    // [heads]
+  const void* dt_bias; const void* A_log; const void* D;    // [heads]; unused with `decay`
+  const float* decay;                          // [heads]: fixed decays, unit steps and no skip (dt may be null)
   float* state;                                // [slots, heads, vdim, state]
   void* y; long long ldy;                      // [T, heads * vdim]
   const int* seqs;                             // sequences of this launch
@@ -190,9 +194,10 @@ ssd_scan_kernel(const ScanArgs a) {
       const int n = lane + 32 * k;
       S[p][k] = (past && p0 + p < a.vdim && n < a.N) ? st[static_cast<long long>(p) * a.N + n] : 0.f;
     }
-  const float bias = ld1(reinterpret_cast<const T*>(a.dt_bias) + h);
-  const float A = expf(ld1(reinterpret_cast<const T*>(a.A_log) + h));
-  const float D = ld1(reinterpret_cast<const T*>(a.D) + h);
+  const bool fixed = a.decay != nullptr;
+  const float bias = fixed ? 0.f : ld1(reinterpret_cast<const T*>(a.dt_bias) + h);
+  const float A = fixed ? 0.f : expf(ld1(reinterpret_cast<const T*>(a.A_log) + h));
+  const float D = fixed ? 0.f : ld1(reinterpret_cast<const T*>(a.D) + h);
   const int g = h / (a.heads / a.groups);
   const int off_b = a.heads * a.vdim + g * a.N, off_c = off_b + a.groups * a.N;
   for (int t = t0; t < t1; ++t) {
@@ -206,8 +211,8 @@ ssd_scan_kernel(const ScanArgs a) {
     }
 #pragma unroll
     for (int p = 0; p < PW; ++p) x[p] = p0 + p < a.vdim ? ld1(xr + h * a.vdim + p0 + p) : 0.f;
-    const float dt = softplus_f(ld1(reinterpret_cast<const T*>(a.dt) + t * a.ldt + h) + bias);
-    const float decay = expf(-A * dt);
+    const float dt = fixed ? 1.f : softplus_f(ld1(reinterpret_cast<const T*>(a.dt) + t * a.ldt + h) + bias);
+    const float decay = fixed ? a.decay[h] : expf(-A * dt);
 #pragma unroll
     for (int p = 0; p < PW; ++p) {
       const float dx = dt * x[p];
@@ -317,6 +322,33 @@ extern "C" int tw_ssd_scan(const void* xbc, long long ldx, const void* dt, long 
     set_last_error("ssd_scan: %d heads do not divide into %d groups", heads, groups);
     return 1;
   }
-  const ScanArgs a{xbc, ldx, dt, ldt, dt_bias, A_log, D, state, y, ldy, seqs, cu_q, kv_lens, slots, heads, vdim, N, groups};
+  const ScanArgs a{xbc, ldx, dt, ldt, dt_bias, A_log, D, nullptr, state, y, ldy, seqs, cu_q, kv_lens, slots, heads, vdim, N, groups};
   return dtype == TW_BF16 ? launch_scan<__nv_bfloat16>(a, n_seqs, stream) : launch_scan<float>(a, n_seqs, stream);
+}
+
+extern "C" int tw_decay_scan(const void* vkq, long long ldx, const float* decay, float* state, void* y, long long ldy,
+                             const int* seqs, int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads,
+                             int vdim, int N, int dtype, cudaStream_t stream) {
+  if (n_seqs <= 0) return 0;
+  const ScanArgs a{vkq, ldx, nullptr, 0, nullptr, nullptr, nullptr, decay, state, y, ldy, seqs, cu_q, kv_lens, slots,
+                   heads, vdim, N, heads};
+  return dtype == TW_BF16 ? launch_scan<__nv_bfloat16>(a, n_seqs, stream) : launch_scan<float>(a, n_seqs, stream);
+}
+
+extern "C" int tw_conv_state(const void* x, long long ldx, void* state, const int* cu_q, const int* kv_lens,
+                             const int* slots, int n_seqs, int channels, int taps, int dtype, cudaStream_t stream) {
+  if (n_seqs <= 0 || taps <= 1) return 0;
+  const ConvArgs a{x, ldx, nullptr, nullptr, state, nullptr, 0, nullptr, cu_q, kv_lens, slots, 0, n_seqs, channels, taps};
+  const bool vec = ldx % 8 == 0 && channels % 8 == 0 && aligned16(x) && aligned16(state);
+  const int groups = (channels + 7) / 8;
+  const int threads = groups >= 128 ? 128 : (groups + 31) / 32 * 32;
+  const dim3 grid((groups + threads - 1) / threads, n_seqs);
+  if (dtype == TW_BF16) {
+    if (vec) conv_state_kernel<__nv_bfloat16, true><<<grid, threads, 0, stream>>>(a);
+    else conv_state_kernel<__nv_bfloat16, false><<<grid, threads, 0, stream>>>(a);
+  } else {
+    if (vec) conv_state_kernel<float, true><<<grid, threads, 0, stream>>>(a);
+    else conv_state_kernel<float, false><<<grid, threads, 0, stream>>>(a);
+  }
+  return check_launch("conv_state");
 }

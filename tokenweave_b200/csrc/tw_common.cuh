@@ -416,4 +416,21 @@ __device__ __forceinline__ void block_sum(float (&v)[R], float* scratch) {
   }
 }
 
+// ---- activations of the bf16 products' epilogues ---------------------------------------------
+// act(gate) * up: the kinds of the gated products (what the launchers call `swiglu`).
+constexpr int GLU_SILU = 1, GLU_GELU_TANH = 2;
+__device__ __forceinline__ float epi_silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }
+// z / 2 (1 + tanh(u)) = z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float epi_gelu_tanh(float z) {
+  const float u2 = -1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+  return __fdividef(z, 1.f + __expf(u2));
+}
+// silu on the columns [begin, end) of a chunk of 32 columns that starts at n
+__device__ __forceinline__ void epi_silu_cols(uint32_t (&v)[32], int n, int begin, int end) {
+  if (n + 32 <= begin || n >= end) return;
+#pragma unroll
+  for (int j = 0; j < 32; ++j)
+    if (n + j >= begin && n + j < end) v[j] = __float_as_uint(epi_silu(__uint_as_float(v[j])));
+}
+
 }  // namespace tw

@@ -156,6 +156,41 @@ int tw_polynorm(const void* z, long long ldz, const void* coef, void* out, long 
 int tw_gated_group_norm(const void* y, long long ldy, const void* z, long long ldz, const void* w, void* out,
                         long long ldo, int T, int C, int groups, float eps, int dtype, cudaStream_t stream);
 
+int tw_embed_norm(const int* ids, const void* table, long long ldt, int vocab, const void* pairs, long long ldp,
+                  long long buckets, long long mul_prev, long long mul_cur, const int* row_seq, const int* cu_q,
+                  const int* prev_token, float* x32, long long ldx, float* first, long long ldf, const void* w, void* xa,
+                  long long lda, int T, int H, float eps, int dtype, cudaStream_t stream);
+int tw_add_prenorm(const void* y, long long ldy, float* x32, long long ldx, const float* first, long long ldf,
+                   const void* w, void* xa, long long lda, int T, int H, float eps, int dtype, cudaStream_t stream);
+int tw_norm_gate(const void* y, long long ldy, const void* gate, long long ldg, const void* w, void* out, long long ldo,
+                 int T, int C, int count, float eps, float scale, int dtype, cudaStream_t stream);
+int tw_silu_cols(void* x, long long ldx, int T, int n, int dtype, cudaStream_t stream);
+int tw_glu(const void* z, long long ldz, void* out, long long ldo, int T, int d, int act, int dtype, cudaStream_t stream);
+
+// ---- grouped attention (grouped_attn.cu; tensor cores: attn_prefill_split.cu, attn_decode_tc.cu, bf16) ----
+int tw_qkv_prep(const void* p, long long ldp, int T, int heads, int kv_heads, int dim, int dp, int vp, void* q,
+                long long ldq, void* k_cache, void* v_cache, const int* positions, const int* cache_slots,
+                const void* conv_w, void* conv_state, int taps, const int* row_seq, const int* cu_q, const int* kv_lens,
+                const int* slots, int n_seqs, int single, int norm, const void* wq, const void* wk, float eps,
+                float temp_coef, int temp_every, int dtype, cudaStream_t stream);
+int tw_attn_rows(const void* q, long long ldq, const void* k_cache, const void* v_cache, int page, void* out,
+                 long long ldo, const int* tok_row, const int* tok_seq, const int* tok_kvlen, int n,
+                 const int* block_table, int max_blocks, int heads, int kv_heads, int dp, int vp, float scale,
+                 const float* slopes, int sink, float out_scale, int dtype, cudaStream_t stream);
+int tw_attn_prefill_grouped(const void* q, long long ldq, int T, const void* k_cache, const void* v_cache,
+                            int num_blocks, int page, void* out, long long ldo, const int* cu_q, const int* kv_lens,
+                            const int* block_table, int max_blocks, const int* tile_seq, const int* tile_q0,
+                            int num_tiles, int hq, int hkv, int dp, int vp, float scale, const float* slopes, int sink,
+                            float out_scale, uint32_t* status, cudaStream_t stream);
+int tw_attn_decode_grouped(const void* q, long long ldq, const void* k_cache, const void* v_cache, int num_blocks,
+                           int page, void* out, long long ldo, const int* tok_row, const int* tok_seq,
+                           const int* tok_kvlen, int n_tok, const int* block_table, int max_blocks, int hq, int hkv,
+                           int dp, int vp, float scale, const float* slopes, int sink, float out_scale, int splits,
+                           float* part_o, float* part_ml, uint32_t* status, cudaStream_t stream);
+int tw_gemm_bf16_silu(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc,
+                      const void* bias, int M, int N, int K, int silu_begin, int silu_end, int max_ctas, int plan_hint,
+                      uint32_t* status, cudaStream_t stream);
+
 // ---- latent attention (latent_attn.cu) ----
 int tw_latent_prep(const void* p, long long ldp, int q_off, int q_rank, const void* wq, void* cq, long long ldcq,
                    int kv_off, int kv_rank, const void* wkv, int rot, int rot_dims, const float* cos_sin,
@@ -192,6 +227,14 @@ int tw_ssd_scan(const void* xbc, long long ldx, const void* dt, long long ldt, c
                 const void* D, float* state, void* y, long long ldy, const int* seqs, int n_seqs, const int* cu_q,
                 const int* kv_lens, const int* slots, int heads, int vdim, int N, int groups, int dtype,
                 cudaStream_t stream);
+int tw_conv_state(const void* x, long long ldx, void* state, const int* cu_q, const int* kv_lens, const int* slots,
+                  int n_seqs, int channels, int taps, int dtype, cudaStream_t stream);
+int tw_decay_scan(const void* vkq, long long ldx, const float* decay, float* state, void* y, long long ldy,
+                  const int* seqs, int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads, int vdim,
+                  int N, int dtype, cudaStream_t stream);
+int tw_decay_chunk(const void* vkq, long long ldx, int T, const float* decay, float* state, void* y, long long ldy,
+                   const int* seqs, int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int heads,
+                   int vdim, int N, int form, uint32_t* status, cudaStream_t stream);
 int tw_ssd_chunk(const void* xbc, long long ldx, int T, const void* dt, long long ldt, const void* dt_bias,
                  const void* A_log, const void* D, float* state, void* y, long long ldy, const int* seqs, int n_seqs,
                  const int* cu_q, const int* kv_lens, const int* slots, int heads, int vdim, int N, int groups, int form,

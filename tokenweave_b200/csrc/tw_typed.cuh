@@ -97,6 +97,14 @@ __device__ __forceinline__ float sigmoid_t(float x) {
   if (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-x));
   return sigmoid_f(x);
 }
+// the tanh form of gelu, z / 2 (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+
+// -ln(decay) of a fixed decay per token; a decay of (nearly) nothing is kept finite, since differences of its multiples
+// are formed (1e-30 wipes a state out in one token).
+__device__ __forceinline__ double decay_rate(float decay) { return -log(static_cast<double>(fmaxf(decay, 1e-30f))); }
 
 }  // namespace tw

@@ -83,10 +83,12 @@ def _row_stride(t: torch.Tensor) -> int:
 # ---------------------------------------------------------------------------------------------
 def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *,
          bias: Optional[torch.Tensor] = None, row_scale: Optional[torch.Tensor] = None, swiglu: bool = False,
-         max_ctas: int = 0, tile_expert: Optional[torch.Tensor] = None,
+         act: str = "silu", silu_cols: Optional[tuple[int, int]] = None, max_ctas: int = 0,
+         tile_expert: Optional[torch.Tensor] = None,
          num_m_tiles: Optional[torch.Tensor] = None, n_per_expert: int = 0, tile_rows: int = 128) -> torch.Tensor:
     """``out = a @ w.T`` (+bias, *row_scale); with ``swiglu`` the weight is ``[gate; up]`` and the
-    output is ``silu(a@gate.T) * (a@up.T)``. Grouped mode (``tile_expert`` given): every ``tile_rows``-row
+    output is ``act(a@gate.T) * (a@up.T)``, ``act`` "silu" or "gelu_tanh". ``silu_cols`` = (begin, end): silu on these
+    columns of a plain product (behind the bias). Grouped mode (``tile_expert`` given): every ``tile_rows``-row
     tile of ``a`` multiplies the weight block of its expert, ``w`` being ``[E * n_per_expert, K]``;
     ``tile_rows`` is 128 (single-CTA tiles) or 256 (experts padded to 256 rows: the groups run on CTA pairs)."""
     M, K = a.shape
@@ -96,6 +98,8 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
     if out is None:
         out = torch.empty(M, N, dtype=a.dtype, device=a.device)
     if not a.is_cuda:
+        if act != "silu" or silu_cols is not None:
+            raise NotImplementedError("these epilogues on CPU go through ops.reference_hybrid")
         if tile_expert is not None:
             raise NotImplementedError("grouped GEMM on CPU goes through reference.moe_experts")
         res = reference.gemm_swiglu(a, w, row_scale) if swiglu else reference.gemm(a, w, bias, row_scale)
@@ -110,6 +114,14 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
                      _row_stride(out), _p(bias), M, N, K, _stream())
         return out
     _check_bf16(a, w, out, bias)
+    if silu_cols is not None:
+        if swiglu or row_scale is not None or tile_expert is not None:
+            raise ValueError("silu on a range of columns goes with a plain product")
+        _native.call("tw_gemm_bf16_silu", a.data_ptr(), _row_stride(a), w.data_ptr(), _row_stride(w), out.data_ptr(),
+                     _row_stride(out), _p(bias), M, N, K, int(silu_cols[0]), int(silu_cols[1]), max_ctas,
+                     gemm_table.lookup(M, N, K, False, max_ctas), status_word(a.device).data_ptr(), _stream(),
+                     tag=f"[{M}x{N}x{K}+silu]" if _native._timing is not None else "")
+        return out
     if tile_expert is not None and tile_rows == 256:
         if bias is not None:
             raise ValueError("the grouped GEMM has no bias")
@@ -120,7 +132,8 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
                      tag=f"[grouped {M}x{N}x{K}{'+swiglu' if swiglu else ''}]" if _native._timing is not None else "")
         return out
     _native.call("tw_gemm_bf16", a.data_ptr(), _row_stride(a), w.data_ptr(), _row_stride(w), rows_b,
-                 out.data_ptr(), _row_stride(out), _p(bias), _p(row_scale), M, N, K, int(swiglu),
+                 out.data_ptr(), _row_stride(out), _p(bias), _p(row_scale), M, N, K,
+                 {"silu": 1, "gelu_tanh": 2}[act] if swiglu else 0,
                  per_expert // 2 if swiglu else 0, _p(tile_expert), _p(num_m_tiles), per_expert, max_ctas,
                  0 if tile_expert is not None else gemm_table.lookup(M, N, K, swiglu, max_ctas),
                  status_word(a.device).data_ptr(), _stream(),

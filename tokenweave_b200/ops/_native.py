@@ -67,6 +67,19 @@ _SIGNATURES = {
     "tw_postnorm_add": [vp, ll, vp, ll, vp, vp, ll, vp, i32, i32, f32, i32, vp],
     "tw_polynorm": [vp, ll, vp, vp, ll, i32, i32, f32, i32, vp],
     "tw_gated_group_norm": [vp, ll, vp, ll, vp, vp, ll, i32, i32, i32, f32, i32, vp],
+    "tw_embed_norm": [vp, vp, ll, i32, vp, ll, ll, ll, ll, vp, vp, vp, vp, ll, vp, ll, vp, vp, ll, i32, i32, f32, i32, vp],
+    "tw_add_prenorm": [vp, ll, vp, ll, vp, ll, vp, vp, ll, i32, i32, f32, i32, vp],
+    "tw_norm_gate": [vp, ll, vp, ll, vp, vp, ll, i32, i32, i32, f32, f32, i32, vp],
+    "tw_silu_cols": [vp, ll, i32, i32, i32, vp],
+    "tw_glu": [vp, ll, vp, ll, i32, i32, i32, i32, vp],
+    "tw_qkv_prep": [vp, ll, i32, i32, i32, i32, i32, i32, vp, ll, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, i32, i32,
+                    i32, vp, vp, f32, f32, i32, i32, vp],
+    "tw_attn_rows": [vp, ll, vp, vp, i32, vp, ll, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, f32, vp, i32, f32, i32, vp],
+    "tw_attn_prefill_grouped": [vp, ll, i32, vp, vp, i32, i32, vp, ll, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32,
+                                f32, vp, i32, f32, vp, vp],
+    "tw_attn_decode_grouped": [vp, ll, vp, vp, i32, i32, vp, ll, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, f32, vp, i32,
+                               f32, i32, vp, vp, vp, vp],
+    "tw_gemm_bf16_silu": [vp, ll, vp, ll, vp, ll, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp],
     "tw_latent_prep": [vp, ll, i32, i32, vp, vp, ll, i32, i32, vp, i32, i32, vp, vp, vp, vp, i32, i32, f32, i32, vp],
     "tw_rope_tail": [vp, ll, i32, i32, i32, i32, i32, vp, vp, i32, vp],
     "tw_latent_query": [vp, ll, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, vp],
@@ -77,6 +90,9 @@ _SIGNATURES = {
                           f32, vp, vp],
     "tw_latent_gather": [vp, vp, vp, vp, i32, i32, vp, i32, i32, i32, vp],
     "tw_causal_conv": [vp, ll, vp, vp, vp, vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
+    "tw_conv_state": [vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, vp],
+    "tw_decay_scan": [vp, ll, vp, vp, vp, ll, vp, i32, vp, vp, vp, i32, i32, i32, i32, vp],
+    "tw_decay_chunk": [vp, ll, i32, vp, vp, vp, ll, vp, i32, vp, vp, vp, i32, i32, i32, i32, vp, vp],
     "tw_ssd_scan": [vp, ll, vp, ll, vp, vp, vp, vp, vp, ll, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, vp],
     "tw_ssd_chunk": [vp, ll, i32, vp, ll, vp, vp, vp, vp, vp, ll, vp, i32, vp, vp, vp, i32, i32, i32, i32, i32, vp, vp],
 }
