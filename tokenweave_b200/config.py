@@ -212,6 +212,25 @@ def _mamba2_layer(heads, vdim, state, groups, ff, conv=4, norm_groups=1) -> dict
             "mlp": None if ff is None else dict(kind="dense", ff=ff)}
 
 
+def _kebopel(vocab, width, ff, layers, attn, left, right, decay, loop, bigram) -> dict:
+    """``config.json`` of a Kebopel model: every third layer (from the second on) is an attention, the others the pair."""
+    sizes = lambda names, v: dict(zip(names.split(), v))
+    pair = {"left": {**sizes("heads kv_heads dim vdim", left), "scale": left[2] ** -0.5},
+            "right": {**sizes("heads dim vdim", right), "decay": decay}, "left_scale": 0.7, "right_scale": 0.7}
+    conv = {**sizes("heads kv_heads dim vdim", attn), "scale": attn[2] ** -0.5, "conv": 4,
+            "q_temp": {"coef": 0.1, "every": 8192}}
+    return {"architecture": "Kebopel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "loop": loop,
+            "embedding": {"bigram": dict(buckets=bigram, mul_prev=8191, mul_cur=31)},
+            "layers": [{"type": "attention" if i % 3 == 1 else "parallel", "mixer": conv if i % 3 == 1 else pair,
+                        "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
+
+
+def _decays(n: int) -> list:
+    """Memories from a few tokens to a few thousand, evenly spaced in the logarithm."""
+    return [1.0 - 2.0 ** (-2.0 - 9.0 * i / max(1, n - 1)) for i in range(n)]
+
+
+# fields of ModelConfig, or {"config": a config.json} for designs with a reader of their own
 MODEL_PRESETS: dict[str, dict[str, Any]] = {
     # correctness configuration: fp32 on CPU, split path must equal the unsplit path
     "tiny-llama": dict(architecture="llama", hidden_size=256, num_layers=2, num_q_heads=4, num_kv_heads=2,
@@ -250,6 +269,10 @@ MODEL_PRESETS: dict[str, dict[str, Any]] = {
                        head_dim=192, intermediate_size=16384, vocab_size=128256, rms_norm_eps=1e-5, max_model_len=131072,
                        layers=[_latent_layer(32, 128, 64, 128, 512, 1536, 16384, base=500000.0) if i % 4 == 3
                                else _mamba2_layer(128, 64, 128, 8, 16384, norm_groups=8) for i in range(32)]),
+    "tiny-kebopel": dict(config=_kebopel(512, 160, 256, 4, (6, 2, 40, 32), (8, 2, 48, 40), (4, 32, 56), _decays(4),
+                                         dict(start=1, stop=3, times=2), 1000)),
+    "kebopel-9b": dict(config=_kebopel(128256, 4096, 14336, 27, (32, 8, 128, 128), (32, 8, 128, 128), (32, 128, 128),
+                                       _decays(32), dict(start=9, stop=18, times=2), 262144)),
     "llama-3.3-70b": dict(architecture="llama", hidden_size=8192, num_layers=80, num_q_heads=64, num_kv_heads=8,
                           head_dim=128, intermediate_size=28672, vocab_size=128256, rms_norm_eps=1e-5,
                           rope_theta=500000.0, max_model_len=131072,
@@ -279,7 +302,9 @@ def resolve_model_config(model: "str | ModelConfig", dtype: Optional[str] = None
     else:
         key = _ALIASES.get(model.lower(), model.lower())
         if key in MODEL_PRESETS:
-            cfg = ModelConfig(name=key, **MODEL_PRESETS[key])
+            preset = MODEL_PRESETS[key]
+            cfg = (ModelConfig.from_hf_dict(preset["config"], name=key) if "config" in preset
+                   else ModelConfig(name=key, **preset))
         elif Path(model).is_dir() and (Path(model) / "config.json").exists():
             cfg = ModelConfig.from_pretrained(model)
         else:
