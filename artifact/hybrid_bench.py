@@ -251,29 +251,34 @@ def _attention(t, heads, hkv, R, row, T, batch, context, page, nb, cs_rot) -> No
       2.0 * n * heads * VDIM * R)
 
 
+def with_ratios(rows: list[dict]) -> list[dict]:
+    """Adds to every row how much further it is from its roofline than the like kernel."""
+    frac = {r["kernel"]: r["fraction"] for r in rows}
+    for r in rows:
+        if r["like"]:
+            r["like_fraction"] = frac[r["like"]]
+            r["distance_ratio"] = round(frac[r["like"]] / r["fraction"], 2)
+    return rows
+
+
 def run(sizes=None, steps: int = 20) -> dict:
     out = {}
     for width in sizes or SIZES:
         hybrid, llama = models(width)
-        rows = kernels(width)
-        frac = {r["kernel"]: r["fraction"] for r in rows}
-        for r in rows:
-            if r["like"]:
-                r["like_fraction"] = frac[r["like"]]
-                r["distance_ratio"] = round(frac[r["like"]] / r["fraction"], 2)
+        rows = with_ratios(kernels(width))
         out[str(width)] = {"hybrid": throughput(hybrid, steps=steps), "llama": throughput(llama, steps=steps), "kernels": rows}
     return out
 
 
-def main() -> None:
-    for width, res in run().items():
+def print_tables(result: dict, names: tuple) -> None:
+    for width, res in result.items():
         print(f"== width {width}")
-        for name in ("hybrid", "llama"):
+        for name in names:
             print(f"{name:8s}" + "  ".join(f"{k} {v:.1f}" for k, v in res[name].items()))
         for r in res["kernels"]:
-            print(f"{r['kernel']:44s} {r['us']:9.1f} us  roofline {r['roofline_us']:8.1f}  {r['fraction']:.2f}"
+            print(f"{r['kernel']:52s} {r['us']:9.1f} us  roofline {r['roofline_us']:8.1f}  {r['fraction']:.2f}"
                   + (f"   like {r['like']} {r['like_fraction']:.2f}  x{r['distance_ratio']:.2f}" if r["like"] else ""))
 
 
 if __name__ == "__main__":
-    main()
+    print_tables(run(), ("hybrid", "llama"))

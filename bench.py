@@ -51,9 +51,10 @@ def parse_args():
                     choices=["overlap", "fuse_only", "fused_gemm", "baseline_nccl", "baseline_custom_ar", "baseline_multimem",
                              "no_ar"])
     ap.add_argument("--layers", type=int, default=None, help="debug only: fewer layers (marks the result invalid)")
-    ap.add_argument("--workload", default="prefill", choices=["prefill", "hybrid"],
+    ap.add_argument("--workload", default="prefill", choices=["prefill", "hybrid", "kebopel"],
                     help="hybrid: the hybrid decoder (latent attention + Mamba-2) beside the Llama layout at equal size, "
-                         "prefill, decode and every kernel (artifact/hybrid_bench.py); one GPU")
+                         "prefill, decode and every kernel (artifact/hybrid_bench.py); kebopel: the same for Kebopel "
+                         "(artifact/kebopel_bench.py); one GPU")
     ap.add_argument("--cuda-graphs", dest="cuda_graphs", action="store_true", default=None,
                     help="replay the step from a CUDA graph (captured during warm-up; the default when --warmup >= 3)")
     ap.add_argument("--no-cuda-graphs", dest="cuda_graphs", action="store_false",
@@ -184,29 +185,31 @@ def run_reference(args) -> None:
         "clocks": clocks, "e2e": {"value": value, "unit": "tokens/s"}, "impl": "reference"}), flush=True)
 
 
-def run_hybrid(args) -> None:
-    """Throughput of the hybrid decoder and of the Llama layout at the same widths, one JSON line; ``value`` is the
-    hybrid model's prefill at the largest width."""
+def run_beside_llama(args) -> None:
+    """Throughput of a hybrid decoder (``--workload``) and of the Llama layout at the same widths, one JSON line; ``value``
+    is the hybrid model's prefill at the largest width."""
+    import importlib
+    name, model = args.workload, {"hybrid": "sidisun", "kebopel": "kebopel"}[args.workload]
     if args.gpus != 1:
-        raise SystemExit("--workload hybrid runs on one GPU")
-    from artifact.hybrid_bench import run
+        raise SystemExit(f"--workload {name} runs on one GPU")
+    run = importlib.import_module(f"artifact.{name}_bench").run
     sampler = ClockSampler(True)
     sizes = run(steps=max(args.steps, 5))
     clocks = sampler.stop({0})
     top = max(sizes, key=int)
     print(json.dumps({
-        "metric": "hybrid_prefill_tokens_per_s", "value": sizes[top]["hybrid"]["prefill_tokens_per_s"], "unit": "tokens/s",
+        "metric": f"{name}_prefill_tokens_per_s", "value": sizes[top][name]["prefill_tokens_per_s"], "unit": "tokens/s",
         "n_gpus": 1, "higher_is_better": True, "vs_baseline": None, "dtype": "bf16",
         "data": "synthetic random token ids, random weights",
-        "config": {"model": f"sidisun-{top}", "layers": 4, "seq_len": 8192, "l2": "a 256 MB buffer is zeroed before "
+        "config": {"model": f"{model}-{top}", "layers": 4, "seq_len": 8192, "l2": "a 256 MB buffer is zeroed before "
                    "every prefill and every timed kernel; decode steps read more than the 126 MB L2"},
         "sizes": sizes, "clocks": clocks, "impl": "ours"}), flush=True)
 
 
 def main() -> None:
     args = parse_args()
-    if args.workload == "hybrid":
-        run_hybrid(args)
+    if args.workload != "prefill":
+        run_beside_llama(args)
         return
     if args.cuda_graphs is None:
         # eager on the first sight of a step shape, capture on the second, replay from the third on
