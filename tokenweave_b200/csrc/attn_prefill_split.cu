@@ -26,7 +26,8 @@
 // instructions of the MUFU form).
 // Grouped forms (OPTS 2 and 3): values of their own width, a sink, a factor on the result; OPTS 3 also takes slope times
 // distance off the scores. Their softmax weights reach the product with V as two bf16 terms (hi in the upper half of the
-// S columns, lo in the lower one: every score is in registers by then), which keeps 16 bits of them.
+// S columns, lo in the lower one: every score is in registers by then), which keeps 16 bits of them. That product starts
+// when the weights of the tile's first 64 keys are there.
 // Replaces the FlashAttention-2 varlen call the reference makes on Blackwell
 // (vllm/v1/attention/backends/flash_attn.py:713-733, vllm/attention/utils/fa_utils.py:29-34).
 //
@@ -38,20 +39,22 @@
 #include "attn_prefill_common.cuh"
 #include "tw_host.h"
 #include "tw_kernels.h"
-#include "tw_mma.cuh"
 
 namespace tw {
 
-constexpr int SPL_RING = 3;   // K/V tile slots per softmax group
+// K/V tile slots per softmax group. The grouped forms spill registers in the softmax, and beside three slots per group there
+// is hardly an L1 cache left for them (head size 128: 776 us with two slots, 808 with three; with bias 928 and 1143).
+template <int MODE>
+constexpr int split_ring() { return MODE >= 2 ? 2 : 3; }
 
-template <int D, int DV>
+template <int D, int DV, int RING>
 struct SplitSmem {
   static constexpr int HALVES = D / 64, V_HALVES = DV / 64;
   static constexpr int Q_BYTES = HALVES * ATT_HALF_BYTES;
   static constexpr int KV_BYTES = (D > DV ? HALVES : V_HALVES) * ATT_HALF_BYTES;   // slot of one K or V tile of 128 keys
   static constexpr int OFF_Q = 0;
-  static constexpr int OFF_RING = OFF_Q + Q_BYTES;              // [2 groups][SPL_RING]
-  static constexpr int OFF_BAR = OFF_RING + 2 * SPL_RING * KV_BYTES;
+  static constexpr int OFF_RING = OFF_Q + Q_BYTES;              // [2 groups][RING]
+  static constexpr int OFF_BAR = OFF_RING + 2 * RING * KV_BYTES;
   static constexpr int TOTAL = OFF_BAR + 256 + 1024;            // barriers, then slack for the 1024-byte alignment
 };
 
@@ -59,6 +62,15 @@ __device__ __forceinline__ float fast_tanh(float x) {
   float y;
   asm("tanh.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
+}
+
+// e to 16 bits of mantissa in two bf16 terms: the leading one cut off (no conversion), the rest rounded
+__device__ __forceinline__ void split_weights(float2 e, uint32_t& hi, uint32_t& lo) {
+  const uint32_t x = __float_as_uint(e.x), y = __float_as_uint(e.y);
+  hi = __byte_perm(x, y, 0x7632);
+  const float2 l = fma2(make_float2(__uint_as_float(x & 0xffff0000u), __uint_as_float(y & 0xffff0000u)),
+                        make_float2(-1.f, -1.f), e);
+  lo = pack_bf16x2(l.x, l.y);
 }
 
 // One work item: a 128-query tile of one head.
@@ -94,10 +106,10 @@ template <int D, int DV, int MODE>
 __global__ void __launch_bounds__(ATT_THREADS, 1)
 attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                           const __grid_constant__ CUtensorMap tmV, const AttnParams p, const int total_items) {
-  using S = SplitSmem<D, DV>;
+  constexpr int R = split_ring<MODE>();
+  using S = SplitSmem<D, DV, R>;
   constexpr bool OPTS = MODE == 1, GROUPED = MODE >= 2, BIAS = MODE == 3;
   constexpr int HALVES = S::HALVES;
-  constexpr int R = SPL_RING;
   constexpr uint32_t IDESC_QK = make_idesc_bf16(ATT_BM, ATT_BN, 0, 0);
   constexpr uint32_t IDESC_PV = make_idesc_bf16(ATT_BM, DV, 0, 1);
   constexpr uint32_t TMEM_COLS = 512;
@@ -117,7 +129,8 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
   uint64_t* p_ready = bars + 16;      // [2]
   uint64_t* o_done = bars + 18;       // [2]
   uint64_t* epi_done = bars + 20;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 21);
+  uint64_t* p_half = bars + 21;       // [2], grouped forms: weights of the first 64 keys
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 23);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5;
@@ -135,6 +148,7 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
     for (int g = 0; g < 2; ++g) {
       mbar_init(&s_full[g], 1);
       mbar_init(&p_ready[g], 128);
+      mbar_init(&p_half[g], 128);
       mbar_init(&o_done[g], 1);
     }
     mbar_init(epi_done, ATT_SOFTMAX_THREADS);
@@ -239,21 +253,23 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
           return true;
         };
         auto issue_pv = [&](int g, bool first) {
-          if (!mbar_wait(&p_ready[g], cnt[g] & 1)) return false;
+          if (!mbar_wait(GROUPED ? &p_half[g] : &p_ready[g], cnt[g] & 1)) return false;
           const int slot = e[g] % R;
           if (!mbar_wait(&ring_full[g * R + slot], (e[g] / R) & 1)) return false;
           tc_fence_after_sync();
           const uint32_t v_addr = smem_u32(smem + S::OFF_RING + (g * R + slot) * S::KV_BYTES);
+          auto pv = [&](int k, uint32_t col, bool init) {
+            umma_ts(tmem_base + COL_O + g * 128, tmem_base + COL_S + g * 128 + col + k * 8,
+                    make_smem_desc_sw128(v_addr + k * 16 * 128, ATT_HALF_BYTES, 1024), IDESC_PV, init ? 0u : 1u);
+          };
 #pragma unroll
-          for (int k = 0; k < ATT_BN / 16; ++k)
-            umma_ts(tmem_base + COL_O + g * 128, tmem_base + COL_S + g * 128 + COL_P + k * 8,
-                    make_smem_desc_sw128(v_addr + k * 16 * 128, ATT_HALF_BYTES, 1024), IDESC_PV,
-                    (first && k == 0) ? 0u : 1u);
-          if (GROUPED) {
-#pragma unroll
-            for (int k = 0; k < ATT_BN / 16; ++k)
-              umma_ts(tmem_base + COL_O + g * 128, tmem_base + COL_S + g * 128 + k * 8,
-                      make_smem_desc_sw128(v_addr + k * 16 * 128, ATT_HALF_BYTES, 1024), IDESC_PV, 1u);
+          for (int k = 0; k < ATT_BN / 16; ++k) {
+            if (GROUPED && k == 4) {
+              if (!mbar_wait(&p_ready[g], cnt[g] & 1)) return false;
+              tc_fence_after_sync();
+            }
+            pv(k, COL_P, first && k == 0);
+            if (GROUPED) pv(k, 0, false);
           }
           umma_commit(&ring_empty[g * R + slot]);
           umma_commit(&o_done[g]);
@@ -297,6 +313,11 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       const float cap_in = (OPTS && p.softcap > 0.f) ? p.scale / p.softcap : 0.f;
       const int pos = it.pos0 + min(r, it.rows_valid - 1);   // padding rows copy the last valid row's mask
       const int pos_w = (OPTS && p.window > 0) ? pos - p.window + 1 : 0;    // first key this row sees
+      // slope in base 2, and slope times the key's place in a block of eight
+      const float slope = BIAS ? p.slopes[it.head] * 1.4426950408889634f : 0.f;
+      float2 in_block[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) in_block[i] = make_float2(slope * (2 * i), slope * (2 * i + 1));
       float m_ref = -INFINITY;   // softmax reference (a stale running maximum), log2 domain
       float l_sum = 0.f;
       for (int t = 0; t < n_mine; ++t) {
@@ -325,24 +346,20 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
           }
         }
         if (BIAS) {
-          // scores in base 2 with the bias: slope * (key - position) is at most zero for every key that is seen
-          const float sl = p.slopes[it.head] * 1.4426950408889634f;
-          const float2 sl2 = make_float2(sl, sl), sc = make_float2(p.scale_log2, p.scale_log2);
-          auto bias_chunk = [&](uint32_t (&buf)[32], int chunk) {
-            const float b0 = sl * static_cast<float>(k_base + chunk * 32 - pos);
-            const float2 b2 = make_float2(b0, b0);
+          // scores in base 2 with the part of the bias inside a block of eight keys (the block's part comes below)
+          const float2 sc = make_float2(p.scale_log2, p.scale_log2);
+          auto bias_chunk = [&](uint32_t (&buf)[32]) {
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
-              const float2 b = fma2(make_float2(2 * i, 2 * i + 1), sl2, b2);
-              const float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc, b);
+              const float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc, in_block[i & 3]);
               buf[2 * i] = __float_as_uint(x.x);
               buf[2 * i + 1] = __float_as_uint(x.y);
             }
           };
-          bias_chunk(s0, 0);
-          bias_chunk(s1, 1);
-          bias_chunk(s2, 2);
-          bias_chunk(s3, 3);
+          bias_chunk(s0);
+          bias_chunk(s1);
+          bias_chunk(s2);
+          bias_chunk(s3);
         }
         if (need_mask) {
 #pragma unroll
@@ -354,16 +371,32 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
           }
         }
         // row maximum: three-input max, one chain per chunk
+        const float row_bias = BIAS ? slope * static_cast<float>(k_base - pos) : 0.f;
         float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+        if (BIAS) {
+          auto max_chunk = [&](const uint32_t (&buf)[32], int chunk) {
 #pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          m4[0] = max3f(m4[0], __uint_as_float(s0[2 * i]), __uint_as_float(s0[2 * i + 1]));
-          m4[1] = max3f(m4[1], __uint_as_float(s1[2 * i]), __uint_as_float(s1[2 * i + 1]));
-          m4[2] = max3f(m4[2], __uint_as_float(s2[2 * i]), __uint_as_float(s2[2 * i + 1]));
-          m4[3] = max3f(m4[3], __uint_as_float(s3[2 * i]), __uint_as_float(s3[2 * i + 1]));
+            for (int q = 0; q < 4; ++q) {
+              float m = fmaxf(__uint_as_float(buf[8 * q]), __uint_as_float(buf[8 * q + 1]));
+#pragma unroll
+              for (int i = 1; i < 4; ++i) m = max3f(m, __uint_as_float(buf[8 * q + 2 * i]), __uint_as_float(buf[8 * q + 2 * i + 1]));
+              m4[chunk] = fmaxf(m4[chunk], m + fmaf(slope, static_cast<float>(chunk * 32 + q * 8), row_bias));
+            }
+          };
+          max_chunk(s0, 0);
+          max_chunk(s1, 1);
+          max_chunk(s2, 2);
+          max_chunk(s3, 3);
+        } else {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            m4[0] = max3f(m4[0], __uint_as_float(s0[2 * i]), __uint_as_float(s0[2 * i + 1]));
+            m4[1] = max3f(m4[1], __uint_as_float(s1[2 * i]), __uint_as_float(s1[2 * i + 1]));
+            m4[2] = max3f(m4[2], __uint_as_float(s2[2 * i]), __uint_as_float(s2[2 * i + 1]));
+            m4[3] = max3f(m4[3], __uint_as_float(s3[2 * i]), __uint_as_float(s3[2 * i + 1]));
+          }
         }
-        const float to_log2 = BIAS ? 1.f : p.scale_log2;
-        const float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * to_log2;
+        const float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * (BIAS ? 1.f : p.scale_log2);
         float alpha = 1.f;
         bool rescale = false;
         if (t == 0) {
@@ -379,17 +412,24 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         // exponentials, two scores per instruction where the ISA has a packed form (scale and subtract,
         // running sum, bf16 conversion); 32 keys become 16 columns of P, which overwrites S columns
         // 64..127 (every score is in registers by now)
-        const float2 sc2 = make_float2(to_log2, to_log2);
+        const float2 sc2 = make_float2(p.scale_log2, p.scale_log2);
         const float2 nm2 = make_float2(-m_use, -m_use);
         float2 sum2[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
         uint32_t pk[16], lo[16];
-        auto exp_chunk = [&](const uint32_t (&buf)[32]) {
+        auto exp_chunk = [&](const uint32_t (&buf)[32], int chunk) {
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
-            const float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc2, nm2);
+            const float2 v = make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1]));
+            float2 x;
+            if (BIAS) {
+              const float nb = fmaf(slope, static_cast<float>(chunk * 32 + (i >> 2) * 8), row_bias - m_use);
+              x = fadd2(v, make_float2(nb, nb));
+            } else {
+              x = fma2(v, sc2, nm2);
+            }
             const float2 e = make_float2(fast_exp2(x.x), fast_exp2(x.y));
             sum2[i & 1] = fadd2(sum2[i & 1], e);
-            if (GROUPED) split_bf16x2(e.x, e.y, pk[i], lo[i]);
+            if (GROUPED) split_weights(e, pk[i], lo[i]);
             else pk[i] = pack_bf16x2(e.x, e.y);
           }
         };
@@ -397,9 +437,9 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
           tmem_st_32x16(t_p + chunk * 16, pk);
           if (GROUPED) tmem_st_32x16(t_s + chunk * 16, lo);
         };
-        exp_chunk(s0);
+        exp_chunk(s0, 0);
         store_chunk(0);
-        exp_chunk(s1);
+        exp_chunk(s1, 1);
         store_chunk(1);
         if (t > 0 && __any_sync(0xffffffffu, rescale)) {
           // O_g may be touched once P V of the previous tile has completed
@@ -416,9 +456,14 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
             tmem_st_32x32(t_o + c * 32, v);
           }
         }
-        exp_chunk(s2);
+        if (GROUPED) {
+          tmem_wait_st();
+          tc_fence_before_sync();
+          mbar_arrive(&p_half[g]);      // (O_g is scaled by then: the product may go on)
+        }
+        exp_chunk(s2, 2);
         store_chunk(2);
-        exp_chunk(s3);
+        exp_chunk(s3, 3);
         store_chunk(3);
         l_sum = l_sum * alpha + ((sum2[0].x + sum2[0].y) + (sum2[1].x + sum2[1].y));
         tmem_wait_st();
@@ -504,7 +549,7 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
 template <int D, int DV, int MODE>
 static int launch_split_t(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const AttnParams& p,
                           int num_tiles, int max_ctas, cudaStream_t stream) {
-  using S = SplitSmem<D, DV>;
+  using S = SplitSmem<D, DV, split_ring<MODE>()>;
   auto kern = attn_prefill_split_kernel<D, DV, MODE>;
   static thread_local int configured_dev = -1;
   int dev = 0;
