@@ -28,10 +28,13 @@ def i32(x):
                                      dict(factor=16.0, original=10 ** 6, fast=32.0, slow=2.0)])
 def test_rotary_table(scaling):
     """Including a configuration whose blend range is empty (the slow end before the fast one)."""
-    from tokenweave_b200.layers.mixers import LatentAttention
+    from types import SimpleNamespace
+
+    from tokenweave_b200.layers.mixers import rope_table
     sizes = oracle.attn_layer(2, 8, 24, 8, 16, 16, None, base=300.0, scaling=scaling)["mixer"]
-    m = LatentAttention(sizes, 16, EPS, dtype=torch.float32, device="cpu", max_positions=200)
-    table, x = m.make_rope_table(), torch.randn(24)
+    rt = SimpleNamespace(rope_tables={}, max_positions=200, device="cpu")
+    table, x = rope_table(rt, sizes["rot"]), torch.randn(24)
+    assert rope_table(rt, dict(sizes["rot"])) is table and table.shape == (200, 24)
     for pos in (0, 1, 63, 199):
         cache = torch.zeros(1, 1, hops.latent_row(8, 24))
         p = torch.cat([torch.zeros(8), torch.ones(8), x]).view(1, -1)
@@ -123,6 +126,16 @@ def test_row_routing():
     assert list(tok_row) == [start[b] + i for b, i in rows] and list(tok_seq) == [b for b, _ in rows]
     assert list(tok_kv) == [kv[b] - q[b] + i + 1 for b, i in rows]
     assert list(extra["scan_seqs"]) == [0] and list(extra["chunk_seqs"]) == [1, 2, 3, 4, 5]
+    # under a window of 150 only the visible keys' tiles travel: the contexts of all long runs are short then
+    model.expand_window = 150
+    plan, extra, host = model.plan_step(q, kv, list(range(6)), [-1] * 6)
+    assert sorted(set(plan[0])) == [1, 2, 4] and list(extra["ctx_first"]) == [0, 0, 0]      # (200 - 150 + 1 is in tile 0)
+    model.expand_window = 60
+    plan, extra, host = model.plan_step(q, kv, list(range(6)), [-1] * 6)
+    assert sorted(set(plan[0])) == [1, 2, 4] and list(extra["ctx_first"]) == [0, 0, 128]    # (200 - 60 + 1 in tile 1)
+    assert list(extra["ctx_cu"]) == [0, 64, 94, 366] and list(extra["ctx_begin"]) == [-1, 0, 64, -1, -34, -1]
+    assert host == {"ctx_rows": 366, "ctx_max": 272}
+    model.expand_window = 0
     model.rt.context_rows = 100                                      # the long context no longer fits
     assert sorted(set(model.plan_step(q, kv, list(range(6)), [-1] * 6)[0][0])) == [1, 2]
     plan, extra, _ = model.plan_step([1, 1], [5, 9], [1, 0], [-1] * 2)

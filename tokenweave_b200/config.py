@@ -47,7 +47,7 @@ def register_config_reader(architecture: str):
 class ModelConfig:
     """Architecture of a decoder-only transformer (Llama-3.x, Qwen2.5, Mixtral layouts)."""
     name: str = "tiny-llama"
-    architecture: str = "llama"          # "llama" | "qwen2" | "mixtral" | "qwen3" | "mistral" | "phi3" | "sidisun" | "kebopel"
+    architecture: str = "llama"          # "llama" | "qwen2" | "mixtral" | "qwen3" | "mistral" | "phi3" | "sidisun" | "kebopel" | "netezen"
     hidden_size: int = 256
     num_layers: int = 2
     num_q_heads: int = 4
@@ -78,9 +78,12 @@ class ModelConfig:
     # hybrid decoders (models/hybrid.py): one {"type", "mixer", "mlp"} per layer; None for the uniform families above
     layers: Optional[list] = None
     logit_scale: float = 1.0             # factor on the logits (hybrid decoders)
-    # hybrid decoders: how a layer adds to the residual stream ("output_norm" or "parallel"); layers start .. stop - 1
+    # hybrid decoders: how a layer adds to the residual stream ("output_norm", "parallel" or "streams"); layers start .. stop - 1
     # run ``times`` times in a row ({"start", "stop", "times"}); pair embeddings ({"buckets", "mul_prev", "mul_cur"})
     block: str = "output_norm"
+    streams: int = 0                     # block "streams": residual streams of the hyper-connections (0: one, not learned)
+    residual_mult: float = 1.0           # block "streams": factor on every sublayer's output
+    norm_offset: float = 0.0             # block "streams": the norms' weights are stored around zero and add to this
     loop: Optional[dict] = None
     bigram: Optional[dict] = None
 

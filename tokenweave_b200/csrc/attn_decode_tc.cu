@@ -23,8 +23,8 @@
 // buffers that attn_decode_merge_kernel reduces. Every wait is bounded.
 //
 // The grouped form (tw_attn_decode_grouped) takes head sizes of queries / keys and values of their own up to 128, any
-// number of query heads per KV head (in blocks of 16), slope times distance off the scores, a sink and a factor on the
-// result; its probabilities enter the product with V as two bf16 terms, which keeps 16 bits of them.
+// number of query heads per KV head (in blocks of 16), slope times distance off the scores, a sink, a factor on the
+// result and a sliding window with kept first keys (only the tiles that hold visible keys are visited); its probabilities enter the product with V as two bf16 terms, which keeps 16 bits of them.
 #include "tw_common.cuh"
 #include "tw_host.h"
 #include "tw_kernels.h"
@@ -78,6 +78,7 @@ struct DecodeTcParams {
   const float* slopes;     // [hq] or null
   int sink;
   float out_scale;
+  int window, keep;        // window > 0: a query sees the last `window` keys (itself among them) and the first `keep`
 };
 
 // GT: query heads per KV head as a compile-time constant (4, 8 or 16), or 0 to read it from the arguments. The
@@ -121,11 +122,15 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
   const int row = p.tok_row[tok];
   const int seq = p.tok_seq[tok];
   const int kv_len = p.tok_kvlen[tok];
-  const int tiles_total = (kv_len + DTC_BN - 1) / DTC_BN;
+  // first key of the window, its tile, and the tiles before that one that hold kept keys
+  const int win_lo = GROUPED && p.window > 0 ? max(0, kv_len - p.window) : 0;
+  const int j_lo = win_lo / DTC_BN, n_pre = GROUPED ? min((p.keep + DTC_BN - 1) / DTC_BN, j_lo) : 0;
+  const int tiles_total = (kv_len + DTC_BN - 1) / DTC_BN - j_lo + n_pre;
   const int tiles_per_split = (tiles_total + p.splits - 1) / p.splits;
   const int t_begin = split * tiles_per_split;
   const int t_end = min(tiles_total, t_begin + tiles_per_split);
   const int n_tiles = max(0, t_end - t_begin);
+  auto tile_at = [&](int j) { return GROUPED && t_begin + j >= n_pre ? t_begin + j - n_pre + j_lo : t_begin + j; };
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < DTC_RING; ++i) {
@@ -162,7 +167,7 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       for (int j = 0; j < n_tiles; ++j) {
         const int st = j % DTC_RING;
         const uint32_t ph = (j / DTC_RING) & 1;
-        const int tile = t_begin + j;
+        const int tile = tile_at(j);
         if (!mbar_wait(&k_empty[st], ph ^ 1)) { report_error(p.status, TW_ERR_MBAR_TIMEOUT); *abort_flag = 1; break; }
         mbar_expect_tx(&k_full[st], k_halves * DTC_HALF_BYTES);
         for (int pg = 0; pg < pages_per_tile; ++pg) {
@@ -298,13 +303,14 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
       for (int g = 0; g < DTC_NH; ++g) s[g] = __uint_as_float(sv[g]);
       if (GROUPED) {
         // in base 2, slope times distance (the key before the query: negative) added
-        const float dist = static_cast<float>((t_begin + j) * DTC_BN + r - (kv_len - 1));
+        const float dist = static_cast<float>(tile_at(j) * DTC_BN + r - (kv_len - 1));
 #pragma unroll
         for (int g = 0; g < DTC_NH; ++g)
           if (g < G) s[g] = fmaf(s[g], p.scale_log2, slope[g] * dist);
       }
-      if ((t_begin + j + 1) * DTC_BN > kv_len) {            // the same for the whole CTA
-        const bool valid = (t_begin + j) * DTC_BN + r < kv_len;
+      const int key0 = tile_at(j) * DTC_BN;
+      if (key0 + DTC_BN > kv_len || (GROUPED && key0 < win_lo)) {            // the same for the whole CTA
+        const bool valid = key0 + r < kv_len && (!GROUPED || key0 + r >= win_lo || key0 + r < p.keep);
 #pragma unroll
         for (int g = 0; g < DTC_NH; ++g) s[g] = valid ? s[g] : -INFINITY;
       }
@@ -968,8 +974,8 @@ extern "C" int tw_attn_decode_grouped(const void* q, long long ldq, const void* 
                                       int num_blocks, int page, void* out, long long ldo, const int* tok_row,
                                       const int* tok_seq, const int* tok_kvlen, int n_tok, const int* block_table,
                                       int max_blocks, int hq, int hkv, int dp, int vp, float scale, const float* slopes,
-                                      int sink, float out_scale, int splits, float* part_o, float* part_ml,
-                                      uint32_t* status, cudaStream_t stream) {
+                                      int sink, float out_scale, int window, int keep, int splits, float* part_o,
+                                      float* part_ml, uint32_t* status, cudaStream_t stream) {
   if (n_tok <= 0) return 0;
   if (dp % 8 != 0 || vp % 8 != 0 || dp < 8 || vp < 8 || dp > DTC_D || vp > DTC_D || hkv <= 0 || hq % hkv != 0) {
     set_last_error("attn_decode_grouped: head sizes must be multiples of 8 up to 128 (dp=%d, vp=%d, hq=%d, hkv=%d)", dp, vp,
@@ -1033,6 +1039,8 @@ extern "C" int tw_attn_decode_grouped(const void* q, long long ldq, const void* 
   p.slopes = slopes;
   p.sink = sink;
   p.out_scale = out_scale;
+  p.window = window;
+  p.keep = keep;
   const dim3 grid(n_tok, hkv * p.blocks, splits);
   if (group == 8) attn_decode_tc_kernel<8, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
   else if (group == 4) attn_decode_tc_kernel<4, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);

@@ -821,8 +821,8 @@ extern "C" int tw_attn_prefill_grouped(const void* q, long long ldq, int T, cons
                                        int num_blocks, int page, void* out, long long ldo, const int* cu_q,
                                        const int* kv_lens, const int* block_table, int max_blocks, const int* tile_seq,
                                        const int* tile_q0, int num_tiles, int hq, int hkv, int dp, int vp, float scale,
-                                       const float* slopes, int sink, float out_scale, uint32_t* status,
-                                       cudaStream_t stream) {
+                                       const float* slopes, int sink, float out_scale, int window, int keep,
+                                       uint32_t* status, cudaStream_t stream) {
   if (num_tiles <= 0 || T <= 0) return 0;
   if (dp % 8 != 0 || vp % 8 != 0 || dp < 8 || vp < 8 || dp > 128 || vp > 128) {
     set_last_error("attn_prefill_grouped: head sizes must be multiples of 8 up to 128 (got %d and %d)", dp, vp);
@@ -865,7 +865,12 @@ extern "C" int tw_attn_prefill_grouped(const void* q, long long ldq, int T, cons
   p.hkv = hkv;
   p.ring = 3;
   p.scale_log2 = scale * 1.4426950408889634f;
-  p.window = 0;
+  if (window > 0 && slopes != nullptr) {
+    set_last_error("attn_prefill_grouped: a sliding window together with a distance bias is not built");
+    return 1;
+  }
+  p.window = window;
+  p.keep = window > 0 ? keep : 0;
   p.softcap = 0.f;
   p.scale = scale;
   p.vdim = vp;

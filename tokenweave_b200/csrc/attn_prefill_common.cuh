@@ -88,6 +88,7 @@ struct AttnParams {
   const float* slopes;     // [hq]: slope * distance is taken off the scaled score; null: off
   int sink;                // one is added to the softmax's denominator
   float out_scale;         // factor on the result
+  int keep;                // keys that stay visible before a sliding window: the first `keep`
   uint32_t* status;
 };
 

@@ -24,8 +24,8 @@
 // exponentials as a cubic on the FMA pipe instead of ex2.approx (correct to 8e-5, but 17 to 25 % slower at
 // every share: the softmax warps are bound by issue slots, and the polynomial costs six times the
 // instructions of the MUFU form).
-// Grouped forms (OPTS 2 and 3): values of their own width, a sink, a factor on the result; OPTS 3 also takes slope times
-// distance off the scores. Their softmax weights reach the product with V as two bf16 terms (hi in the upper half of the
+// Grouped forms (MODE 2, 3 and 4): values of their own width, a sink, a factor on the result; MODE 3 also takes slope times
+// distance off the scores, MODE 4 has a sliding window whose first keys of the sequence may stay visible. Their softmax weights reach the product with V as two bf16 terms (hi in the upper half of the
 // S columns, lo in the lower one: every score is in registers by then), which keeps 16 bits of them. That product starts
 // when the weights of the tile's first 64 keys are there.
 // Replaces the FlashAttention-2 varlen call the reference makes on Blackwell
@@ -75,11 +75,13 @@ __device__ __forceinline__ void split_weights(float2 e, uint32_t& hi, uint32_t& 
 
 // One work item: a 128-query tile of one head.
 struct SplitItem {
-  // key tiles [j_lo, j_lo + n_tiles) are needed (j_lo > 0 only under a sliding window);
-  // group A takes the first n_a of them, group B the rest
-  int head, kvh, seq, q_begin, q0, rows_valid, pos0, kv_len, j_lo, n_tiles, n_a;
+  // key tiles [0, n_pre) and [j_lo, j_lo + n_tiles - n_pre) are needed (j_lo > 0 only under a sliding window, n_pre > 0 only
+  // when it keeps the first keys); group A takes the first n_a of them, group B the rest
+  int head, kvh, seq, q_begin, q0, rows_valid, pos0, kv_len, j_lo, n_pre, n_tiles, n_a;
+  __device__ __forceinline__ int tile(int t) const { return t < n_pre ? t : j_lo + t - n_pre; }
 };
 
+template <bool KEEP>
 __device__ __forceinline__ SplitItem split_item(const AttnParams& p, int idx) {
   SplitItem it;
   const int tile = idx / p.hq;
@@ -95,20 +97,22 @@ __device__ __forceinline__ SplitItem split_item(const AttnParams& p, int idx) {
   const int kv_end = min(it.kv_len, it.pos0 + it.rows_valid);  // keys [0, kv_end) are needed
   // under a sliding window the tile's first query sees nothing before key pos0 - window + 1
   it.j_lo = p.window > 0 ? max(0, it.pos0 - p.window + 1) / ATT_BN : 0;
-  it.n_tiles = (kv_end + ATT_BN - 1) / ATT_BN - it.j_lo;
+  it.n_pre = KEEP ? min((p.keep + ATT_BN - 1) / ATT_BN, it.j_lo) : 0;
+  it.n_tiles = (kv_end + ATT_BN - 1) / ATT_BN - it.j_lo + it.n_pre;
   it.n_a = (it.n_tiles + 1) / 2;
   return it;
 }
 
 // MODE 1: sliding window and logits soft cap compiled in (separate instantiations, so that the plain causal kernel, MODE 0,
-// keeps its register budget); 2: grouped attention; 3: grouped attention with distance bias.
+// keeps its register budget); 2: grouped attention; 3: grouped attention with distance bias; 4: grouped attention with a
+// sliding window.
 template <int D, int DV, int MODE>
 __global__ void __launch_bounds__(ATT_THREADS, 1)
 attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                           const __grid_constant__ CUtensorMap tmV, const AttnParams p, const int total_items) {
   constexpr int R = split_ring<MODE>();
   using S = SplitSmem<D, DV, R>;
-  constexpr bool OPTS = MODE == 1, GROUPED = MODE >= 2, BIAS = MODE == 3;
+  constexpr bool OPTS = MODE == 1, GROUPED = MODE >= 2, BIAS = MODE == 3, KEEP = MODE == 4, WINDOW = OPTS || KEEP;
   constexpr int HALVES = S::HALVES;
   constexpr uint32_t IDESC_QK = make_idesc_bf16(ATT_BM, ATT_BN, 0, 0);
   constexpr uint32_t IDESC_PV = make_idesc_bf16(ATT_BM, DV, 0, 1);
@@ -177,7 +181,7 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       for (int round = 0; ok; ++round) {
         const int idx = split_item_index(round, cta, G);
         if (idx >= total_items) break;
-        const SplitItem it = split_item(p, idx);
+        const SplitItem it = split_item<KEEP>(p, idx);
         if (items_done > 0 && !mbar_wait(q_empty, (items_done - 1) & 1)) { ok = false; break; }
         mbar_expect_tx(q_full, S::Q_BYTES);
 #pragma unroll
@@ -205,10 +209,10 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         };
         const int n_b = it.n_tiles - it.n_a;
         for (int t = 0; t < it.n_a && ok; ++t) {
-          ok = load_tile(0, &tmK, HALVES, it.j_lo + t);
-          if (ok && t < n_b) ok = load_tile(1, &tmK, HALVES, it.j_lo + it.n_a + t);
-          if (ok) ok = load_tile(0, &tmV, S::V_HALVES, it.j_lo + t);
-          if (ok && t < n_b) ok = load_tile(1, &tmV, S::V_HALVES, it.j_lo + it.n_a + t);
+          ok = load_tile(0, &tmK, HALVES, it.tile(t));
+          if (ok && t < n_b) ok = load_tile(1, &tmK, HALVES, it.tile(it.n_a + t));
+          if (ok) ok = load_tile(0, &tmV, S::V_HALVES, it.tile(t));
+          if (ok && t < n_b) ok = load_tile(1, &tmV, S::V_HALVES, it.tile(it.n_a + t));
         }
         ++items_done;
       }
@@ -228,7 +232,7 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       for (int round = 0; ok; ++round) {
         const int idx = split_item_index(round, cta, G);
         if (idx >= total_items) break;
-        const SplitItem it = split_item(p, idx);
+        const SplitItem it = split_item<KEEP>(p, idx);
         const int n_b = it.n_tiles - it.n_a;
         if (!mbar_wait(q_full, items_done & 1)) { ok = false; break; }
         // S_g carried the (m, l) exchange of the previous item's epilogue
@@ -305,14 +309,14 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
     for (int round = 0;; ++round) {
       const int idx = split_item_index(round, cta, G);
       if (idx >= total_items) break;
-      const SplitItem it = split_item(p, idx);
+      const SplitItem it = split_item<KEEP>(p, idx);
       const int n_b = it.n_tiles - it.n_a;
       const int n_mine = g == 0 ? it.n_a : n_b;
-      const int j0 = it.j_lo + (g == 0 ? 0 : it.n_a);
+      const int j0 = g == 0 ? 0 : it.n_a;
       const float cap_mul = (OPTS && p.softcap > 0.f) ? p.softcap / p.scale : 0.f;
       const float cap_in = (OPTS && p.softcap > 0.f) ? p.scale / p.softcap : 0.f;
       const int pos = it.pos0 + min(r, it.rows_valid - 1);   // padding rows copy the last valid row's mask
-      const int pos_w = (OPTS && p.window > 0) ? pos - p.window + 1 : 0;    // first key this row sees
+      const int pos_w = (WINDOW && p.window > 0) ? pos - p.window + 1 : 0;    // first key of this row's window
       // slope in base 2, and slope times the key's place in a block of eight
       const float slope = BIAS ? p.slopes[it.head] * 1.4426950408889634f : 0.f;
       float2 in_block[4];
@@ -323,10 +327,10 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       for (int t = 0; t < n_mine; ++t) {
         if (ok) ok = mbar_wait(&s_full[g], cnt & 1);
         tc_fence_after_sync();
-        const int k_base = (j0 + t) * ATT_BN;
+        const int k_base = it.tile(j0 + t) * ATT_BN;
         // warp-uniform: lane 0 holds the warp's smallest position, lane 31 its largest
         bool need_mask = (k_base + ATT_BN - 1) > __shfl_sync(0xffffffffu, pos, 0);
-        if (OPTS) need_mask = need_mask || k_base < __shfl_sync(0xffffffffu, pos_w, 31);
+        if (WINDOW) need_mask = need_mask || k_base < __shfl_sync(0xffffffffu, pos_w, 31);
         // The row's 128 scores come to registers in one go (four loads in flight, one wait): the latency of
         // tensor-memory loads is paid once per tile, and everything below runs from registers.
         uint32_t s0[32], s1[32], s2[32], s3[32];
@@ -364,10 +368,11 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         if (need_mask) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
-            if (k_base + i > pos || (OPTS && k_base + i < pos_w)) s0[i] = __float_as_uint(-INFINITY);
-            if (k_base + 32 + i > pos || (OPTS && k_base + 32 + i < pos_w)) s1[i] = __float_as_uint(-INFINITY);
-            if (k_base + 64 + i > pos || (OPTS && k_base + 64 + i < pos_w)) s2[i] = __float_as_uint(-INFINITY);
-            if (k_base + 96 + i > pos || (OPTS && k_base + 96 + i < pos_w)) s3[i] = __float_as_uint(-INFINITY);
+            auto hidden = [&](int k) { return k > pos || (WINDOW && k < pos_w && (!KEEP || k >= p.keep)); };
+            if (hidden(k_base + i)) s0[i] = __float_as_uint(-INFINITY);
+            if (hidden(k_base + 32 + i)) s1[i] = __float_as_uint(-INFINITY);
+            if (hidden(k_base + 64 + i)) s2[i] = __float_as_uint(-INFINITY);
+            if (hidden(k_base + 96 + i)) s3[i] = __float_as_uint(-INFINITY);
           }
         }
         // row maximum: three-input max, one chain per chunk
@@ -588,8 +593,9 @@ int launch_prefill_split(int D, const CUtensorMap& tmQ, const CUtensorMap& tmK, 
 int launch_prefill_grouped(int D, int DV, const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
                            const AttnParams& p, int num_tiles, cudaStream_t stream) {
 #define TW_GO(A, B)                                                                                    \
-  return p.slopes != nullptr ? launch_split_t<A, B, 3>(tmQ, tmK, tmV, p, num_tiles, 0, stream)         \
-                             : launch_split_t<A, B, 2>(tmQ, tmK, tmV, p, num_tiles, 0, stream)
+  return p.window > 0          ? launch_split_t<A, B, 4>(tmQ, tmK, tmV, p, num_tiles, 0, stream)       \
+         : p.slopes != nullptr ? launch_split_t<A, B, 3>(tmQ, tmK, tmV, p, num_tiles, 0, stream)       \
+                               : launch_split_t<A, B, 2>(tmQ, tmK, tmV, p, num_tiles, 0, stream)
   if (D > 64) {
     if (DV > 64) TW_GO(128, 128);
     TW_GO(128, 64);

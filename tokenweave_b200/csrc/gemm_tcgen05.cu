@@ -14,8 +14,8 @@
 // The tile width BN is a run-time value (a multiple of 32 up to 256; the instruction descriptor and
 // the pipeline depth are computed from it), chosen per problem by a wave-quantisation cost model:
 // skinny tensor-parallel shapes such as N = 1280 waste a third of the machine with 256-wide tiles.
-// Epilogues: plain, +bias[n], silu on a range of columns, *row_scale[m], and gated (the B tile holds BN/2 "gate" rows and
-// BN/2 "up" rows; the stored value is silu(gate)*up - SwiGLU - or gelu(gate)*up, BN/2 output columns per tile).
+// Epilogues: plain, +bias[n], silu or relu^2 on a range of columns, *row_scale[m], and gated (the B tile holds BN/2 "gate" rows and
+// BN/2 "up" rows; the stored value is silu(gate)*up - SwiGLU -, gelu(gate)*up or the clamped form, BN/2 output columns).
 // Grouped mode: each 128-row tile of A belongs to one expert (tile_expert[m_tile]); the B rows
 // are offset by expert * n_per_expert; the number of valid tiles is read from device memory.
 //
@@ -51,8 +51,7 @@ struct GemmParams {
   int bn;        // accumulator columns per tile
   int stages;    // pipeline depth
   int kb_per_stage;  // 64-wide k-blocks per stage: 2 halves the barrier round trips per FLOP
-  int glu;           // gated epilogue: GLU_SILU or GLU_GELU_TANH (bf16)
-  int silu_begin, silu_end;   // plain bf16 epilogue: silu on these columns (none: begin = end)
+  GemmActs acts;     // bf16 epilogues
   uint32_t* status;
 };
 
@@ -237,11 +236,18 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
           uint32_t u[32];
           tmem_ld_32x32(taddr + BN / 2 + c * 32, u);
           tmem_wait_ld();
-          if (!FP8 && p.glu == GLU_GELU_TANH) {
+          if (!FP8 && p.acts.glu == GLU_GELU_TANH) {
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               packed[j] = pack_bf16x2(epi_gelu_tanh(__uint_as_float(v[2 * j])) * __uint_as_float(u[2 * j]) * rs,
                                       epi_gelu_tanh(__uint_as_float(v[2 * j + 1])) * __uint_as_float(u[2 * j + 1]) * rs);
+          } else if (!FP8 && p.acts.glu == GLU_CLAMPED) {
+            const float lim = p.acts.limit, al = p.acts.alpha;
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              packed[j] = pack_bf16x2(
+                  epi_clamped(__uint_as_float(v[2 * j]), __uint_as_float(u[2 * j]), lim, al) * rs,
+                  epi_clamped(__uint_as_float(v[2 * j + 1]), __uint_as_float(u[2 * j + 1]), lim, al) * rs);
           } else
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
@@ -322,7 +328,7 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
             }
           }
           if (!FP8) {
-            epi_silu_cols(v, n0 + c * 32, p.silu_begin, p.silu_end);
+            epi_col_act(v, n0 + c * 32, p.acts);
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               packed[j] = pack_bf16x2(__uint_as_float(v[2 * j]) * rs, __uint_as_float(v[2 * j + 1]) * rs);
@@ -481,8 +487,8 @@ extern "C" int tw_gemm_set_kernel_override(int kind) {
 extern "C" int tw_gemm_pair(int fp8, const void* A, long long lda, const void* B, long long ldb, long long rows_b,
                             void* C, long long ldc, const void* bias, const float* row_scale, const float* col_scale,
                             int M, int N, int K, int swiglu, int up_row_offset, int bn, int max_ctas,
-                            const int* tile_expert, const int* num_m_tiles_dev, int n_per_expert, int silu_begin,
-                            int silu_end, uint32_t* status, cudaStream_t stream);
+                            const int* tile_expert, const int* num_m_tiles_dev, int n_per_expert, const GemmActs* acts,
+                            uint32_t* status, cudaStream_t stream);
 
 // Shared launcher body. A is [M,K] with row stride lda, B is [rows_b, K] with row stride ldb
 // (rows_b = N, 2*N for SwiGLU, or experts * n_per_expert); strides count elements (2 bytes, or 1 for fp8).
@@ -490,8 +496,8 @@ static int gemm_dispatch(bool fp8, const void* A, long long lda, const void* B, 
                          void* C, long long ldc, const void* bias, const float* row_scale, const float* col_scale,
                          int M, int N, int K, int swiglu, int up_row_offset, const int* tile_expert,
                          const int* num_m_tiles_dev, int n_per_expert, int max_ctas, int plan_hint,
-                         uint32_t* status, cudaStream_t stream, int group_tile_rows = 128, int silu_begin = 0,
-                         int silu_end = 0) {
+                         uint32_t* status, cudaStream_t stream, int group_tile_rows = 128, GemmActs acts = {}) {
+  if (swiglu && acts.glu == 0) acts.glu = swiglu;
   // group_tile_rows: rows per entry of tile_expert (grouped mode). 256: the caller padded every expert to 256
   // rows, so the CTA-pair kernel can take the groups; 128: single-CTA tiles.
   // plan_hint: 0 = cost model; otherwise kernel * 1000 + tile width (kernel 1 = single-CTA tiles,
@@ -510,7 +516,7 @@ static int gemm_dispatch(bool fp8, const void* A, long long lda, const void* B, 
   const int num_m = (M + GEMM_BM - 1) / GEMM_BM;
   if (tile_expert != nullptr && group_tile_rows == 256 && sms >= 2)
     return tw_gemm_pair(fp8, A, lda, B, ldb, rows_b, C, ldc, bias, row_scale, col_scale, M, N, K, swiglu,
-                        up_row_offset, 256, sms, tile_expert, num_m_tiles_dev, n_per_expert, 0, 0, status, stream);
+                        up_row_offset, 256, sms, tile_expert, num_m_tiles_dev, n_per_expert, &acts, status, stream);
   // the cost model sees k-blocks: an fp8 problem has K / 128 of them
   GemmPlan plan = choose_plan(M, N, fp8 ? K / 2 : K, sms, swiglu != 0, tile_expert != nullptr);
   if (plan_hint > 0) {
@@ -522,7 +528,7 @@ static int gemm_dispatch(bool fp8, const void* A, long long lda, const void* B, 
   }
   if (plan.pair)
     return tw_gemm_pair(fp8, A, lda, B, ldb, rows_b, C, ldc, bias, row_scale, col_scale, M, N, K, swiglu, up_row_offset,
-                        plan.bn, sms, nullptr, nullptr, 0, silu_begin, silu_end, status, stream);
+                        plan.bn, sms, nullptr, nullptr, 0, &acts, status, stream);
   const int BN = plan.bn;
   const int out_cols = swiglu ? BN / 2 : BN;
   const int num_n = (N + out_cols - 1) / out_cols;
@@ -568,9 +574,7 @@ static int gemm_dispatch(bool fp8, const void* A, long long lda, const void* B, 
   p.bn = BN;
   p.stages = stages;
   p.kb_per_stage = kbps;
-  p.glu = swiglu;
-  p.silu_begin = silu_begin;
-  p.silu_end = silu_end;
+  p.acts = acts;
   p.status = status;
   int grid = num_m * num_n;
   if (grid > sms) grid = sms;
@@ -591,12 +595,38 @@ extern "C" int tw_gemm_bf16(const void* A, long long lda, const void* B, long lo
                        stream);
 }
 
-// The same with silu on the columns [silu_begin, silu_end) of the result.
-extern "C" int tw_gemm_bf16_silu(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc,
-                                 const void* bias, int M, int N, int K, int silu_begin, int silu_end, int max_ctas,
-                                 int plan_hint, uint32_t* status, cudaStream_t stream) {
+// The same with an activation (act 1: silu, 2: the square of relu) on the columns [act_begin, act_end) of the result.
+extern "C" int tw_gemm_bf16_act(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc,
+                                const void* bias, int M, int N, int K, int act, int act_begin, int act_end, int max_ctas,
+                                int plan_hint, uint32_t* status, cudaStream_t stream) {
+  if (act != COL_SILU && act != COL_RELU2) {
+    set_last_error("tw_gemm_bf16_act: unknown activation %d", act);
+    return 1;
+  }
+  GemmActs acts;
+  acts.col_act = act;
+  acts.col_begin = act_begin;
+  acts.col_end = act_end;
   return gemm_dispatch(false, A, lda, B, ldb, N, C, ldc, bias, nullptr, nullptr, M, N, K, 0, 0, nullptr, nullptr, N,
-                       max_ctas, plan_hint, status, stream, 128, silu_begin, silu_end);
+                       max_ctas, plan_hint, status, stream, 128, acts);
+}
+
+// The gated product with clamped halves: B = [gate; up], C = g sigmoid(alpha g) (u + 1) with g = min(gate, limit) and u = up
+// inside [-limit, limit]; over all rows, or grouped over experts padded to tile_rows (128 or 256) rows each.
+extern "C" int tw_gemm_bf16_clamped(const void* A, long long lda, const void* B, long long ldb, long long rows_b, void* C,
+                                    long long ldc, int M, int N, int K, float limit, float alpha, int up_row_offset,
+                                    const int* tile_expert, const int* num_m_tiles_dev, int n_per_expert, int tile_rows,
+                                    int max_ctas, int plan_hint, uint32_t* status, cudaStream_t stream) {
+  if (!(limit > 0.f) || (tile_rows != 128 && tile_rows != 256)) {
+    set_last_error("tw_gemm_bf16_clamped: limit %f, tiles of %d rows", limit, tile_rows);
+    return 1;
+  }
+  GemmActs acts;
+  acts.glu = GLU_CLAMPED;
+  acts.limit = limit;
+  acts.alpha = alpha;
+  return gemm_dispatch(false, A, lda, B, ldb, rows_b, C, ldc, nullptr, nullptr, nullptr, M, N, K, 1, up_row_offset,
+                       tile_expert, num_m_tiles_dev, n_per_expert, max_ctas, plan_hint, status, stream, tile_rows, acts);
 }
 
 // Grouped GEMM over experts padded to 256 rows each: tile_expert has one entry per 256-row tile and the groups
@@ -644,5 +674,5 @@ extern "C" int tw_gemm_int8(const void* A, long long lda, const void* B, long lo
     bn = plan.pair ? plan.bn : (N > 128 || swiglu ? 256 : 128);
   }
   return tw_gemm_pair(2, A, lda, B, ldb, swiglu ? 2LL * N : N, C, ldc, bias, row_scale, col_scale, M, N, K, swiglu,
-                      swiglu ? N : 0, bn, sms, nullptr, nullptr, 0, 0, 0, status, stream);
+                      swiglu ? N : 0, bn, sms, nullptr, nullptr, 0, nullptr, status, stream);
 }

@@ -66,8 +66,7 @@ struct Gemm2Params {
   int up_row_offset;
   int bn, stages;
   int kb_per_stage;
-  int glu;                        // gated epilogue: GLU_SILU or GLU_GELU_TANH (bf16)
-  int silu_begin, silu_end;       // plain bf16 epilogue: silu on these columns (none: begin = end)
+  GemmActs acts;                  // bf16 epilogues
   uint32_t* status;
 };
 
@@ -373,11 +372,18 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
           uint32_t u[32];
           tmem_ld_32x32(taddr + BN / 2 + c * 32, u);
           tmem_wait_ld();
-          if (KIND == KIND_BF16 && p.glu == GLU_GELU_TANH) {
+          if (KIND == KIND_BF16 && p.acts.glu == GLU_GELU_TANH) {
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               packed[j] = pack_bf16x2(epi_gelu_tanh(__uint_as_float(v[2 * j])) * __uint_as_float(u[2 * j]) * rs,
                                       epi_gelu_tanh(__uint_as_float(v[2 * j + 1])) * __uint_as_float(u[2 * j + 1]) * rs);
+          } else if (KIND == KIND_BF16 && p.acts.glu == GLU_CLAMPED) {
+            const float lim = p.acts.limit, al = p.acts.alpha;
+#pragma unroll
+            for (int j = 0; j < 16; ++j)
+              packed[j] = pack_bf16x2(
+                  epi_clamped(__uint_as_float(v[2 * j]), __uint_as_float(u[2 * j]), lim, al) * rs,
+                  epi_clamped(__uint_as_float(v[2 * j + 1]), __uint_as_float(u[2 * j + 1]), lim, al) * rs);
           } else
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
@@ -463,7 +469,7 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
               v[j] = __float_as_uint(__uint_as_float(v[j]) + bb);
             }
           }
-          epi_silu_cols(v, nc, p.silu_begin, p.silu_end);
+          epi_col_act(v, nc, p.acts);
 #pragma unroll
           for (int j = 0; j < 16; ++j)
             packed[j] = pack_bf16x2(__uint_as_float(v[2 * j]) * rs, __uint_as_float(v[2 * j + 1]) * rs);
@@ -582,8 +588,8 @@ extern "C" int tw_gemm_set_pair_kbps(int kbps) {
 extern "C" int tw_gemm_pair(int fp8, const void* A, long long lda, const void* B, long long ldb, long long rows_b,
                             void* C, long long ldc, const void* bias, const float* row_scale, const float* col_scale,
                             int M, int N, int K, int swiglu, int up_row_offset, int bn, int max_ctas,
-                            const int* tile_expert, const int* num_m_tiles_dev, int n_per_expert, int silu_begin,
-                            int silu_end, uint32_t* status, cudaStream_t stream) {
+                            const int* tile_expert, const int* num_m_tiles_dev, int n_per_expert, const GemmActs* acts,
+                            uint32_t* status, cudaStream_t stream) {
   if (M <= 0 || N <= 0 || K <= 0) return 0;
   const int in_align = fp8 ? 16 : 8;     // 16 bytes of operand elements
   if ((K % in_align) != 0 || (lda % in_align) != 0 || (ldb % in_align) != 0 || (ldc % 8) != 0 || bn % 64 != 0 ||
@@ -650,9 +656,8 @@ extern "C" int tw_gemm_pair(int fp8, const void* A, long long lda, const void* B
   p.bn = bn;
   p.stages = stages;
   p.kb_per_stage = kbps;
-  p.glu = swiglu;
-  p.silu_begin = silu_begin;
-  p.silu_end = silu_end;
+  if (acts != nullptr) p.acts = *acts;
+  if (swiglu && p.acts.glu == 0) p.acts.glu = swiglu;
   p.status = status;
   int pairs = num_m * num_n;
   if (pairs > pairs_avail) pairs = pairs_avail;
@@ -677,5 +682,5 @@ extern "C" int tw_gemm_bf16_pair(const void* A, long long lda, const void* B, lo
                                  const int* num_m_tiles_dev, int n_per_expert, uint32_t* status,
                                  cudaStream_t stream) {
   return tw_gemm_pair(0, A, lda, B, ldb, rows_b, C, ldc, bias, row_scale, nullptr, M, N, K, swiglu, up_row_offset, bn,
-                      max_ctas, tile_expert, num_m_tiles_dev, n_per_expert, 0, 0, status, stream);
+                      max_ctas, tile_expert, num_m_tiles_dev, n_per_expert, nullptr, status, stream);
 }

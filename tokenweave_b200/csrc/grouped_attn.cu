@@ -2,10 +2,12 @@
 //
 //   tw_qkv_prep    everything between the projection and the attention in one pass over the projection's rows: causal
 //                  convolution over time (with the sequence's kept inputs), RMS norm of queries and keys per head or over
-//                  the whole projection, query temperature, queries to a buffer, keys and values into the paged caches.
+//                  the whole projection, rotation of the leading dimensions of queries and keys (neighbouring dimensions
+//                  are a pair), query temperature, queries to a buffer, keys and values into the paged caches.
 //                  A step of single-token sequences moves the convolution's state on in the same launch
 //   tw_attn_rows   softmax attention of single query rows on SIMT: fp32, and heads beyond what the tensor-core kernels
-//                  take (attn_prefill_split.cu, attn_decode_tc.cu); distance bias, sink, factor on the result
+//                  take (attn_prefill_split.cu, attn_decode_tc.cu); distance bias, sink, factor on the result, sliding
+//                  window with kept first keys
 //
 // Heads are padded to eight elements in the projection's rows, the query buffer and the caches; pads are zeros. All
 // arithmetic is fp32.
@@ -28,6 +30,7 @@ struct PrepArgs {
   const void *wq, *wk;                      // norm weights: [dp] each, or [heads * dp] and [kv_heads * dp]
   float eps, temp_coef;
   int temp_every;
+  const float* cos_sin; int rot_dims;       // [positions, rot_dims]: cosines, then sines, of the pairs; null: no rotation
 };
 
 // Eight channels from column c on of row t behind the convolution. UPDATE: also writes the state that follows the row
@@ -67,6 +70,30 @@ __device__ __forceinline__ float query_temperature(const PrepArgs& a, int t) {
   return 1.f + a.temp_coef * logf(static_cast<float>((a.positions[t] + 1) / a.temp_every) + 1.f);
 }
 
+// Rotates the pairs among dimensions d .. d + 7 of a head whose first `dims` dimensions turn.
+__device__ __forceinline__ void rotate_pairs(float (&v)[8], int d, int dims, const float* cs) {
+  const int half = dims >> 1;
+  float c[4], s[4];
+  if ((half & 3) == 0) {
+    if (d >= dims) return;
+    *reinterpret_cast<float4*>(c) = *reinterpret_cast<const float4*>(cs + (d >> 1));
+    *reinterpret_cast<float4*>(s) = *reinterpret_cast<const float4*>(cs + half + (d >> 1));
+  } else {
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const bool in = d + 2 * j < dims;
+      c[j] = in ? cs[(d >> 1) + j] : 1.f;
+      s[j] = in ? cs[half + (d >> 1) + j] : 0.f;
+    }
+  }
+#pragma unroll
+  for (int j = 0; j < 4; ++j) {
+    const float x = v[2 * j], y = v[2 * j + 1];
+    v[2 * j] = x * c[j] - y * s[j];
+    v[2 * j + 1] = y * c[j] + x * s[j];
+  }
+}
+
 // One CTA per row; a group of S lanes (a power of two) takes one head at a time. NORM: 0 none, 1 per head, 2 whole.
 template <typename T, int NORM, bool CONV, int S>
 __global__ void __launch_bounds__(256)
@@ -98,6 +125,7 @@ qkv_prep_kernel(const PrepArgs a) {
     whole[1] = 1.f / sqrtf(whole[1] / static_cast<float>(G * a.dim) + a.eps);
   }
   const float temp = a.temp_coef != 0.f ? query_temperature(a, t) : 1.f;
+  const float* cs = a.cos_sin != nullptr ? a.cos_sin + static_cast<long long>(a.positions[t]) * a.rot_dims : nullptr;
   const int slot = a.cache_slots[t];
   T* q = reinterpret_cast<T*>(a.q) + t * a.ldq;
   T* kc = reinterpret_cast<T*>(a.k_cache) + static_cast<long long>(slot) * nk;
@@ -144,6 +172,7 @@ qkv_prep_kernel(const PrepArgs a) {
 #pragma unroll
         for (int j = 0; j < 8; ++j) v[j] *= temp;
       }
+      if (cs != nullptr && !is_v) rotate_pairs(v, d, a.rot_dims, cs);
       if (h < H) st8(q + h * a.dp + d, v);
       else if (slot >= 0) st8(is_v ? vc + (h - H - G) * a.vp + d : kc + (h - H) * a.dp + d, v);
     }
@@ -252,7 +281,7 @@ static void launch_prep(const PrepArgs& a, int norm, cudaStream_t stream) {
   const int heads = a.heads + 2 * a.kv_heads;
   int threads = (heads * S + 31) / 32 * 32;
   if (threads > 256) threads = 256;
-  if (a.conv_w != nullptr && !a.single && norm != 2 && a.taps <= 6 && a.dp <= S * 8 && a.vp <= S * 8) {
+  if (a.conv_w != nullptr && !a.single && norm != 2 && a.cos_sin == nullptr && a.taps <= 6 && a.dp <= S * 8 && a.vp <= S * 8) {
     const dim3 grid((a.T + PREP_ROWS - 1) / PREP_ROWS, (heads * S + threads - 1) / threads);
     if (norm == 1) launch_strip<T, true, S>(a, threads, grid, stream);
     else launch_strip<T, false, S>(a, threads, grid, stream);
@@ -283,6 +312,7 @@ struct RowsArgs {
   const float* slopes;
   int sink;
   float out_scale;
+  int window, keep;          // window > 0: a query sees the last `window` keys (itself among them) and the first `keep`
 };
 
 template <typename T>
@@ -304,11 +334,15 @@ attn_rows_kernel(const RowsArgs a) {
   float m = -INFINITY, l = 0.f, acc[ROWS_VPT];
 #pragma unroll
   for (int c = 0; c < ROWS_VPT; ++c) acc[c] = 0.f;
+  // the visible keys: `kept` first ones, then those from `from` on
+  const int from = a.window > 0 ? max(0, kv_len - a.window) : 0, kept = min(a.keep, from);
+  const int visible = kept + kv_len - from;
   __syncthreads();
-  for (int j0 = 0; j0 < kv_len; j0 += ROWS_THREADS) {
-    const int j = j0 + threadIdx.x, n = min(ROWS_THREADS, kv_len - j0);
+  for (int j0 = 0; j0 < visible; j0 += ROWS_THREADS) {
+    const int i0 = j0 + threadIdx.x, n = min(ROWS_THREADS, visible - j0);
     float s = -INFINITY;
-    if (j < kv_len) {
+    if (i0 < visible) {
+      const int j = i0 < kept ? i0 : i0 - kept + from;
       const int slot = table[j / a.page] * a.page + j % a.page;
       slot_s[threadIdx.x] = slot;
       const T* k = kc + (static_cast<long long>(slot) * a.kv_heads + g) * a.dp;
@@ -327,7 +361,7 @@ attn_rows_kernel(const RowsArgs a) {
     mx = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
     const float m_new = fmaxf(m, mx), alpha = expf(m - m_new);        // 0 in the first round
     m = m_new;
-    const float p = j < kv_len ? expf(s - m_new) : 0.f;
+    const float p = i0 < visible ? expf(s - m_new) : 0.f;
     l = l * alpha + p;
     p_s[threadIdx.x] = p;
     __syncthreads();
@@ -370,12 +404,17 @@ extern "C" int tw_qkv_prep(const void* p, long long ldp, int T, int heads, int k
                            long long ldq, void* k_cache, void* v_cache, const int* positions, const int* cache_slots,
                            const void* conv_w, void* conv_state, int taps, const int* row_seq, const int* cu_q,
                            const int* kv_lens, const int* slots, int n_seqs, int single, int norm, const void* wq,
-                           const void* wk, float eps, float temp_coef, int temp_every, int dtype, cudaStream_t stream) {
+                           const void* wk, float eps, float temp_coef, int temp_every, const float* cos_sin, int rot_dims,
+                           int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (dp % 8 != 0 || vp % 8 != 0 || ldp % 8 != 0 || ldq % 8 != 0 || !aligned16(p) || !aligned16(q) || !aligned16(k_cache) ||
       !aligned16(v_cache) || !aligned16(conv_w) || !aligned16(conv_state) || !aligned16(wq) || !aligned16(wk)) {
     set_last_error("qkv_prep: heads of %d and %d elements in rows of %lld: multiples of eight on 16-byte boundaries are needed",
                    dp, vp, ldp);
+    return 1;
+  }
+  if (cos_sin != nullptr && (rot_dims % 2 != 0 || rot_dims <= 0 || rot_dims > dim || !aligned16(cos_sin))) {
+    set_last_error("qkv_prep: %d rotated dimensions of %d", rot_dims, dim);
     return 1;
   }
   if (heads <= 0 || kv_heads <= 0 || norm < 0 || norm > 2 || (norm != 0 && (wq == nullptr || wk == nullptr)) ||
@@ -385,7 +424,7 @@ extern "C" int tw_qkv_prep(const void* p, long long ldp, int T, int heads, int k
     return 1;
   }
   const PrepArgs a{p, ldp, T, heads, kv_heads, dim, dp, vp, q, ldq, k_cache, v_cache, positions, cache_slots, conv_w,
-                   conv_state, taps, row_seq, cu_q, kv_lens, slots, single, wq, wk, eps, temp_coef, temp_every};
+                   conv_state, taps, row_seq, cu_q, kv_lens, slots, single, wq, wk, eps, temp_coef, temp_every, cos_sin, rot_dims};
   const int wide = dp > vp ? dp : vp;
 #define TW_GO(T)                                          \
   do {                                                    \
@@ -407,7 +446,8 @@ extern "C" int tw_qkv_prep(const void* p, long long ldp, int T, int heads, int k
 extern "C" int tw_attn_rows(const void* q, long long ldq, const void* k_cache, const void* v_cache, int page, void* out,
                             long long ldo, const int* tok_row, const int* tok_seq, const int* tok_kvlen, int n,
                             const int* block_table, int max_blocks, int heads, int kv_heads, int dp, int vp, float scale,
-                            const float* slopes, int sink, float out_scale, int dtype, cudaStream_t stream) {
+                            const float* slopes, int sink, float out_scale, int window, int keep, int dtype,
+                            cudaStream_t stream) {
   if (n <= 0) return 0;
   if (dp % 8 != 0 || dp > 4096 || vp > ROWS_VPT * ROWS_THREADS || kv_heads <= 0 || heads % kv_heads != 0 ||
       !aligned16(k_cache)) {
@@ -416,7 +456,7 @@ extern "C" int tw_attn_rows(const void* q, long long ldq, const void* k_cache, c
     return 1;
   }
   const RowsArgs a{q, ldq, k_cache, v_cache, page, out, ldo, tok_row, tok_seq, tok_kvlen, block_table, max_blocks, heads,
-                   kv_heads, dp, vp, scale, slopes, sink, out_scale};
+                   kv_heads, dp, vp, scale, slopes, sink, out_scale, window, keep};
   const dim3 grid(n, heads);
   if (dtype == TW_BF16) attn_rows_kernel<__nv_bfloat16><<<grid, ROWS_THREADS, dp * 4, stream>>>(a);
   else attn_rows_kernel<float><<<grid, ROWS_THREADS, dp * 4, stream>>>(a);

@@ -12,8 +12,9 @@
 //   tw_latent_query    the rotated tail and the pads of absorbed query rows
 //   tw_head_gemm       out[t, h, :] = B[h] a[t, h, :] for every head, rows through optional index lists, optionally
 //                      times sigmoid(gate) element by element (tensor cores for bf16)
-//   tw_latent_attn     absorbed causal attention of single query rows over the paged cache, fp32 softmax
-//   tw_latent_gather   cache rows of some sequences, in order, into one contiguous buffer
+//   tw_latent_attn     absorbed causal attention of single query rows over the paged cache, fp32 softmax; sliding window,
+//                      sink per head
+//   tw_latent_gather   cache rows of some sequences, in order and from a given key on, into one contiguous buffer
 #include "tw_host.h"
 #include "tw_kernels.h"
 #include "tw_mma.cuh"
@@ -309,7 +310,8 @@ template <typename T, int NK>
 __global__ void __launch_bounds__(128)
 latent_attn_kernel(const T* __restrict__ qa, const T* __restrict__ cache, const int* __restrict__ tok_seq,
                    const int* __restrict__ tok_kvlen, const int* __restrict__ block_table, int max_blocks, int page,
-                   T* __restrict__ out, int heads, int row, int kv_rank, float scale) {
+                   T* __restrict__ out, int heads, int row, int kv_rank, float scale, int window,
+                   const float* __restrict__ sink) {
   const int i = blockIdx.x, h = blockIdx.y * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (h >= heads) return;
   const long long item = static_cast<long long>(i) * heads + h;
@@ -323,7 +325,7 @@ latent_attn_kernel(const T* __restrict__ qa, const T* __restrict__ cache, const 
   const int* table = block_table + static_cast<long long>(tok_seq[i]) * max_blocks;
   const int n_keys = tok_kvlen[i];
   float m = -INFINITY, l = 0.f;
-  for (int j0 = 0; j0 < n_keys; j0 += 2) {
+  for (int j0 = window > 0 ? max(0, n_keys - window) : 0; j0 < n_keys; j0 += 2) {
     float x[2][NK], s[2];
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
@@ -347,6 +349,7 @@ latent_attn_kernel(const T* __restrict__ qa, const T* __restrict__ cache, const 
 #pragma unroll
     for (int k = 0; k < NK; ++k) o[k] = fmaf(o[k], a, fmaf(p0, x[0][k], p1 * x[1][k]));
   }
+  if (sink != nullptr) l += expf(sink[h] - m);
   const float inv = 1.f / l;
 #pragma unroll
   for (int k = 0; k < NK; ++k) {
@@ -359,16 +362,17 @@ constexpr int LG_ROWS = 16;      // rows per CTA
 
 __global__ void __launch_bounds__(256)
 latent_gather_kernel(const uint4* __restrict__ cache, uint4* __restrict__ dst, const int* __restrict__ seqs,
-                     const int* __restrict__ cu, const int* __restrict__ block_table, int max_blocks, int page,
-                     int row_vec) {
+                     const int* __restrict__ cu, const int* __restrict__ from, const int* __restrict__ block_table,
+                     int max_blocks, int page, int row_vec) {
   const int b = blockIdx.y;
+  const int key0 = from != nullptr ? from[b] : 0;
   const int n = cu[b + 1] - cu[b], first = blockIdx.x * LG_ROWS;
   if (first >= n) return;
   const int* table = block_table + static_cast<long long>(seqs[b]) * max_blocks;
   const int items = min(LG_ROWS, n - first) * row_vec;
   for (int i = threadIdx.x; i < items; i += blockDim.x) {
-    const int r = i / row_vec, v = i - r * row_vec, j = first + r;
-    dst[(static_cast<long long>(cu[b]) + j) * row_vec + v] =
+    const int r = i / row_vec, v = i - r * row_vec, j = key0 + first + r;
+    dst[(static_cast<long long>(cu[b]) + first + r) * row_vec + v] =
         cache[(static_cast<long long>(table[j / page]) * page + j % page) * row_vec + v];
   }
 }
@@ -494,7 +498,7 @@ extern "C" int tw_head_gemm(const void* A, long long lda, int a_hs, const int* a
 
 extern "C" int tw_latent_attn(const void* qa, const void* cache, const int* tok_seq, const int* tok_kvlen, int n,
                               const int* block_table, int max_blocks, int page, void* out, int heads, int row,
-                              int kv_rank, float scale, int dtype, cudaStream_t stream) {
+                              int kv_rank, float scale, int window, const float* sink, int dtype, cudaStream_t stream) {
   if (n <= 0) return 0;
   const dim3 grid(n, (heads + 3) / 4);
 #define TW_GO(NK)                                                                                                      \
@@ -502,11 +506,12 @@ extern "C" int tw_latent_attn(const void* qa, const void* cache, const int* tok_
     if (dtype == TW_BF16)                                                                                              \
       latent_attn_kernel<__nv_bfloat16, NK><<<grid, 128, 0, stream>>>(                                                 \
           reinterpret_cast<const __nv_bfloat16*>(qa), reinterpret_cast<const __nv_bfloat16*>(cache), tok_seq, tok_kvlen, \
-          block_table, max_blocks, page, reinterpret_cast<__nv_bfloat16*>(out), heads, row, kv_rank, scale);           \
+          block_table, max_blocks, page, reinterpret_cast<__nv_bfloat16*>(out), heads, row, kv_rank, scale, window,    \
+          sink);                                                                                                       \
     else                                                                                                               \
       latent_attn_kernel<float, NK><<<grid, 128, 0, stream>>>(                                                         \
           reinterpret_cast<const float*>(qa), reinterpret_cast<const float*>(cache), tok_seq, tok_kvlen, block_table,  \
-          max_blocks, page, reinterpret_cast<float*>(out), heads, row, kv_rank, scale);                                \
+          max_blocks, page, reinterpret_cast<float*>(out), heads, row, kv_rank, scale, window, sink);                  \
   } while (0)
   if (row <= 64) TW_GO(2);
   else if (row <= 128) TW_GO(4);
@@ -522,7 +527,7 @@ extern "C" int tw_latent_attn(const void* qa, const void* cache, const int* tok_
   return check_launch("latent_attn");
 }
 
-extern "C" int tw_latent_gather(const void* cache, void* dst, const int* seqs, const int* cu, int n_seqs,
+extern "C" int tw_latent_gather(const void* cache, void* dst, const int* seqs, const int* cu, const int* from, int n_seqs,
                                 int max_rows, const int* block_table, int max_blocks, int page, int row_bytes,
                                 cudaStream_t stream) {
   if (n_seqs <= 0 || max_rows <= 0) return 0;
@@ -532,6 +537,6 @@ extern "C" int tw_latent_gather(const void* cache, void* dst, const int* seqs, c
   }
   const dim3 grid((max_rows + LG_ROWS - 1) / LG_ROWS, n_seqs);
   latent_gather_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<const uint4*>(cache), reinterpret_cast<uint4*>(dst),
-                                                 seqs, cu, block_table, max_blocks, page, row_bytes / 16);
+                                                 seqs, cu, from, block_table, max_blocks, page, row_bytes / 16);
   return check_launch("latent_gather");
 }

@@ -9,7 +9,8 @@
 // pair is refilled as soon as its part of O^T is done; the next tile travels to L2 meanwhile, since wide rows leave
 // room for one tile in shared memory (two tiles of 64 keys were 40 % slower: an MMA of this shape takes about 60 cycles
 // whether it has 64 or 128 rows). Rows of up to 640 elements, latents of up to 512. The keys of a
-// row can be cut into splits, whose fp32 partial results a second kernel merges.
+// row can be cut into splits, whose fp32 partial results a second kernel merges. Under a sliding window only the tiles that
+// hold visible keys are visited; a sink per head joins the denominator at the end.
 //
 // Roles (192 threads): warp 0 TMA producer, warp 1 MMA issuer, warps 2..5 softmax (one thread per key of the tile),
 // rescaling and epilogue (one thread per latent column). Waits are bounded; after a timeout the roles keep their trip
@@ -34,6 +35,8 @@ struct LatentDecodeParams {
   float scale_log2;
   float *part_o, *part_ml;
   uint32_t* status;
+  int window;                    // > 0: the last `window` keys are visible
+  const float* sink;             // [heads] or null: exp(sink) joins the denominator
 };
 
 __device__ __forceinline__ float ld_exp2(float x) {
@@ -89,10 +92,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
   const int G = min(NC, p.heads - h0);
   const int seq = p.tok_seq[tok];
   const int kv_len = p.tok_kvlen[tok];
-  const int tiles_total = (kv_len + LD_BN - 1) / LD_BN;
+  const int win_lo = p.window > 0 ? max(0, kv_len - p.window) : 0, j_lo = win_lo / LD_BN;
+  const int tiles_total = (kv_len + LD_BN - 1) / LD_BN - j_lo;
   const int per_split = (tiles_total + p.splits - 1) / p.splits;
-  const int t_begin = split * per_split;
-  const int n_tiles = max(0, min(tiles_total, t_begin + per_split) - t_begin);
+  const int n_tiles = max(0, min(tiles_total - split * per_split, per_split));
+  const int t_begin = j_lo + split * per_split;
 
   if (threadIdx.x == 0) {
     for (int i = 0; i < p.stages * LD_MAX_PAIRS; ++i) {
@@ -265,7 +269,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       tmem_ld_cols(t_lane + (j & 1) * NC, sv);
       tmem_wait_ld();
       float* xm = xchg + (j & 1) * 4 * NC;
-      if ((t_begin + j) * LD_BN + r >= kv_len) {
+      const int key = (t_begin + j) * LD_BN + r;
+      if (key >= kv_len || key < win_lo) {
 #pragma unroll
         for (int g = 0; g < NC; ++g) sv[g] = __float_as_uint(-INFINITY);
       }
@@ -360,7 +365,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       float inv[NC];
 #pragma unroll
       for (int g = 0; g < NC; ++g) {
-        const float l = (xs[g] + xs[NC + g]) + (xs[2 * NC + g] + xs[3 * NC + g]);
+        float l = (xs[g] + xs[NC + g]) + (xs[2 * NC + g] + xs[3 * NC + g]);
+        if (p.sink != nullptr && g < G) l += ld_exp2(fmaf(p.sink[h0 + g], 1.4426950408889634f, -m_ref[g]));
         inv[g] = l > 0.f ? __fdividef(1.f, l) : 0.f;
       }
 #pragma unroll 1
@@ -430,10 +436,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
 
 __global__ void __launch_bounds__(128)
 latent_decode_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml, int splits, int kv_rank,
-                           __nv_bfloat16* __restrict__ out) {
+                           const float* __restrict__ sink, int heads, __nv_bfloat16* __restrict__ out) {
   const long long item = blockIdx.x;
   float mm = -INFINITY, ll = 0.f;
   for (int s = 0; s < splits; ++s) mm = fmaxf(mm, part_ml[(item * splits + s) * 2]);
+  if (sink != nullptr) ll = exp2f(fmaf(sink[item % heads], 1.4426950408889634f, -mm));
   for (int s = 0; s < splits; ++s) {
     const float m = part_ml[(item * splits + s) * 2];
     ll += m == -INFINITY ? 0.f : part_ml[(item * splits + s) * 2 + 1] * exp2f(m - mm);
@@ -488,7 +495,8 @@ static int launch_latent_decode(const void* cache, int num_blocks, LatentDecodeP
   latent_decode_kernel<NC><<<dim3(n, (p.heads + NC - 1) / NC, p.splits), LD_THREADS, bytes, stream>>>(tm, tmQ, p);
   cudaError_t e = cudaGetLastError();
   if (e == cudaSuccess && p.splits > 1) {
-    latent_decode_merge_kernel<<<n * p.heads, 128, 0, stream>>>(p.part_o, p.part_ml, p.splits, p.kv_rank, p.out);
+    latent_decode_merge_kernel<<<n * p.heads, 128, 0, stream>>>(p.part_o, p.part_ml, p.splits, p.kv_rank, p.sink,
+                                                                 p.heads, p.out);
     e = cudaGetLastError();
   }
   if (e != cudaSuccess) {
@@ -506,8 +514,8 @@ using namespace tw;
 // [n, heads, kv_rank]; part_o [n, heads, splits, kv_rank] and part_ml [n, heads, splits, 2] when splits > 1.
 extern "C" int tw_latent_decode(const void* qa, const void* cache, int num_blocks, int page, const int* tok_seq,
                                 const int* tok_kvlen, int n, const int* block_table, int max_blocks, void* out, int heads,
-                                int row, int kv_rank, float scale, int splits, float* part_o, float* part_ml,
-                                uint32_t* status, cudaStream_t stream) {
+                                int row, int kv_rank, float scale, int window, const float* sink, int splits,
+                                float* part_o, float* part_ml, uint32_t* status, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (row % 8 != 0 || row > 64 * 2 * LD_MAX_PAIRS || kv_rank > 512 || kv_rank > row || page < 8 || page > 128 || 128 % page != 0) {
     set_last_error("latent_decode: unsupported cache rows (row=%d, kv_rank=%d, page=%d)", row, kv_rank, page);
@@ -521,7 +529,7 @@ extern "C" int tw_latent_decode(const void* qa, const void* cache, int num_block
   LatentDecodeParams p{reinterpret_cast<const __nv_bfloat16*>(qa), reinterpret_cast<__nv_bfloat16*>(out),
                        reinterpret_cast<const __nv_bfloat16*>(cache), tok_seq, tok_kvlen,
                        block_table, max_blocks, page, heads, row, kv_rank, splits, (row + 63) / 64, 1,
-                       scale * 1.4426950408889634f, part_o, part_ml, status};
+                       scale * 1.4426950408889634f, part_o, part_ml, status, window, sink};
   return heads <= 16 ? launch_latent_decode<16>(cache, num_blocks, p, n, stream)
                      : launch_latent_decode<32>(cache, num_blocks, p, n, stream);
 }

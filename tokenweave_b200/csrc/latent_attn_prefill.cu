@@ -7,8 +7,9 @@
 // V buffers in shared memory) and merge in the epilogue straight from tensor memory; P is the tensor-memory A operand
 // of P V. What differs: a key tile is KC chunks of 64 columns, the first ones from the head's unrotated keys and the
 // others from the shared rotated part (chunks are zero-filled behind each part's end by the tensor maps, so widths need
-// not be multiples of 64); values are VC chunks; K and V have separate buffers because their sizes differ; and the
-// epilogue multiplies the output by sigmoid(gate), the output gate of the layer.
+// not be multiples of 64); values are VC chunks; K and V have separate buffers because their sizes differ; the epilogue
+// multiplies the output by sigmoid(gate), the output gate of the layer; a sink per head may join the denominator; and with a
+// sliding window (an instantiation of its own) an item visits the tiles that hold visible keys only.
 //
 // Roles (320 threads): warp 0 TMA producer, warp 1 MMA issuer, warps 2..5 softmax group A (one thread per query row),
 // warps 6..9 group B. Every mbarrier wait is bounded; after a timeout the roles keep their trip counts, report
@@ -41,16 +42,20 @@ struct LatentPrefillParams {
   __nv_bfloat16* out; long long ldo;
   const __nv_bfloat16* gate; long long ldg;     // null: no output gate
   const int *cu_q, *kv_lens, *tile_seq, *tile_q0;
-  const int* ctx_begin;                         // [B] first workspace row of a sequence's context
+  const int* ctx_begin;                         // [B] workspace row of a sequence's key 0 (may lie before the first row
+                                                // when a window leaves the first keys out)
   int heads, dim, vdim, k_chunks;               // k_chunks: chunks of the unrotated part
   float scale_log2;
   uint32_t* status;
+  int window;                                   // > 0: a query sees the last `window` keys, itself among them
+  const float* sink;                            // [heads] or null: exp(sink) joins the denominator
 };
 
 struct LatentPrefillItem {
-  int head, q_begin, q0, rows_valid, pos0, ctx, n_tiles, n_a;
+  int head, q_begin, q0, rows_valid, pos0, ctx, j_lo, n_tiles, n_a;
 };
 
+template <bool WINDOW>
 __device__ __forceinline__ LatentPrefillItem latent_item(const LatentPrefillParams& p, int idx) {
   LatentPrefillItem it;
   const int tile = idx / p.heads;
@@ -63,12 +68,13 @@ __device__ __forceinline__ LatentPrefillItem latent_item(const LatentPrefillPara
   it.ctx = p.ctx_begin[seq];
   it.rows_valid = min(ATT_BM, q_len - it.q0);
   it.pos0 = kv_len - q_len + it.q0;
-  it.n_tiles = (min(kv_len, it.pos0 + it.rows_valid) + ATT_BN - 1) / ATT_BN;
+  it.j_lo = WINDOW ? max(0, it.pos0 - p.window + 1) / ATT_BN : 0;
+  it.n_tiles = (min(kv_len, it.pos0 + it.rows_valid) + ATT_BN - 1) / ATT_BN - it.j_lo;
   it.n_a = (it.n_tiles + 1) / 2;
   return it;
 }
 
-template <int KC, int VC>
+template <int KC, int VC, bool WINDOW>
 __global__ void __launch_bounds__(ATT_THREADS, 1)
 latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                       const __grid_constant__ CUtensorMap tmR, const __grid_constant__ CUtensorMap tmV,
@@ -144,7 +150,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       for (int round = 0; ok; ++round) {
         const int idx = split_item_index(round, cta, G);
         if (idx >= total_items) break;
-        const LatentPrefillItem it = latent_item(p, idx);
+        const LatentPrefillItem it = latent_item<WINDOW>(p, idx);
         if (items_done > 0 && !mbar_wait(q_empty, (items_done - 1) & 1)) { ok = false; break; }
         mbar_expect_tx(q_full, S::K_BYTES);
 #pragma unroll
@@ -179,10 +185,10 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         };
         const int n_b = it.n_tiles - it.n_a;
         for (int t = 0; t < it.n_a && ok; ++t) {
-          ok = load_k(0, t);
-          if (ok && t < n_b) ok = load_k(1, it.n_a + t);
-          if (ok) ok = load_v(0, t);
-          if (ok && t < n_b) ok = load_v(1, it.n_a + t);
+          ok = load_k(0, it.j_lo + t);
+          if (ok && t < n_b) ok = load_k(1, it.j_lo + it.n_a + t);
+          if (ok) ok = load_v(0, it.j_lo + t);
+          if (ok && t < n_b) ok = load_v(1, it.j_lo + it.n_a + t);
         }
         ++items_done;
       }
@@ -202,7 +208,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       for (int round = 0; ok; ++round) {
         const int idx = split_item_index(round, cta, G);
         if (idx >= total_items) break;
-        const LatentPrefillItem it = latent_item(p, idx);
+        const LatentPrefillItem it = latent_item<WINDOW>(p, idx);
         const int n_b = it.n_tiles - it.n_a;
         if (!mbar_wait(q_full, items_done & 1)) { ok = false; break; }
         // S_g carried the (m, l) exchange of the previous item's epilogue
@@ -270,19 +276,21 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     for (int round = 0;; ++round) {
       const int idx = split_item_index(round, cta, G);
       if (idx >= total_items) break;
-      const LatentPrefillItem it = latent_item(p, idx);
+      const LatentPrefillItem it = latent_item<WINDOW>(p, idx);
       const int n_b = it.n_tiles - it.n_a;
       const int n_mine = g == 0 ? it.n_a : n_b;
-      const int j0 = (g == 0 ? 0 : it.n_a);
+      const int j0 = it.j_lo + (g == 0 ? 0 : it.n_a);
       const int pos = it.pos0 + min(r, it.rows_valid - 1);   // padding rows copy the last valid row's mask
+      const int pos_w = WINDOW ? pos - p.window + 1 : 0;     // first key this row sees
       float m_ref = -INFINITY;   // softmax reference (a stale running maximum), log2 domain
       float l_sum = 0.f;
       for (int t = 0; t < n_mine; ++t) {
         if (ok) ok = mbar_wait(&s_full[g], cnt & 1);
         tc_fence_after_sync();
         const int k_base = (j0 + t) * ATT_BN;
-        // warp-uniform: lane 0 holds the warp's smallest position
-        const bool need_mask = (k_base + ATT_BN - 1) > __shfl_sync(0xffffffffu, pos, 0);
+        // warp-uniform: lane 0 holds the warp's smallest position, lane 31 its largest
+        bool need_mask = (k_base + ATT_BN - 1) > __shfl_sync(0xffffffffu, pos, 0);
+        if (WINDOW) need_mask = need_mask || k_base < __shfl_sync(0xffffffffu, pos_w, 31);
         // The row's 128 scores come to registers in one go (four loads in flight, one wait): the latency of
         // tensor-memory loads is paid once per tile, and everything below runs from registers.
         uint32_t s0[32], s1[32], s2[32], s3[32];
@@ -294,10 +302,11 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         if (need_mask) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
-            if (k_base + i > pos) s0[i] = __float_as_uint(-INFINITY);
-            if (k_base + 32 + i > pos) s1[i] = __float_as_uint(-INFINITY);
-            if (k_base + 64 + i > pos) s2[i] = __float_as_uint(-INFINITY);
-            if (k_base + 96 + i > pos) s3[i] = __float_as_uint(-INFINITY);
+            auto hidden = [&](int k) { return k > pos || (WINDOW && k < pos_w); };
+            if (hidden(k_base + i)) s0[i] = __float_as_uint(-INFINITY);
+            if (hidden(k_base + 32 + i)) s1[i] = __float_as_uint(-INFINITY);
+            if (hidden(k_base + 64 + i)) s2[i] = __float_as_uint(-INFINITY);
+            if (hidden(k_base + 96 + i)) s3[i] = __float_as_uint(-INFINITY);
           }
         }
         // row maximum: three-input max, one chain per chunk
@@ -383,7 +392,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       const float o_m = __uint_as_float(om_u), o_l = __uint_as_float(ol_u);
       const float m_all = fmaxf(m_ref, o_m);
       const float f_me = fast_exp2(m_ref - m_all), f_ot = fast_exp2(o_m - m_all);
-      const float inv = 1.f / (l_sum * f_me + o_l * f_ot);
+      float l_all = l_sum * f_me + o_l * f_ot;
+      if (p.sink != nullptr) l_all += fast_exp2(fmaf(p.sink[it.head], 1.4426950408889634f, -m_all));
+      const float inv = 1.f / l_all;
       const float f_a = (g == 0 ? f_me : f_ot) * inv, f_b = (g == 0 ? f_ot : f_me) * inv;
       const long long out_row = it.q_begin + it.q0 + r;
       __nv_bfloat16* orow = p.out + out_row * p.ldo + it.head * p.vdim;
@@ -446,12 +457,12 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   }
 }
 
-template <int KC, int VC>
+template <int KC, int VC, bool WINDOW>
 static int launch_latent_prefill(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmR,
                                  const CUtensorMap& tmV, const LatentPrefillParams& p, int num_tiles,
                                  cudaStream_t stream) {
   using S = LatentPrefillSmem<KC, VC>;
-  auto kern = latent_prefill_kernel<KC, VC>;
+  auto kern = latent_prefill_kernel<KC, VC, WINDOW>;
   static thread_local int configured_dev = -1;
   int dev = 0;
   cudaGetDevice(&dev);
@@ -480,12 +491,14 @@ static int launch_latent_prefill(const CUtensorMap& tmQ, const CUtensorMap& tmK,
 using namespace tw;
 
 // q [T, heads * (dim + rot)] with the rotated tails, kv [ctx_rows, heads * dim | heads * vdim] (row stride ldkv),
-// kr [ctx_rows, rot] (row stride ldr); sequence b's context starts at workspace row ctx_begin[b].
+// kr [ctx_rows, rot] (row stride ldr); key k of sequence b is workspace row ctx_begin[b] + k, for every key from the first
+// visible one's tile of 128 on.
 extern "C" int tw_latent_prefill(const void* q, long long ldq, int T, const void* kv, long long ldkv, const void* kr,
                                  long long ldr, int ctx_rows, const int* ctx_begin, void* out, long long ldo,
                                  const void* gate, long long ldg, const int* cu_q, const int* kv_lens,
                                  const int* tile_seq, const int* tile_q0, int num_tiles, int heads, int dim, int rot,
-                                 int vdim, float scale, uint32_t* status, cudaStream_t stream) {
+                                 int vdim, float scale, int window, const float* sink, uint32_t* status,
+                                 cudaStream_t stream) {
   if (num_tiles <= 0) return 0;
   const int kc = (dim + 63) / 64 + (rot + 63) / 64, vc = (vdim + 63) / 64;
   if (dim % 8 != 0 || rot % 8 != 0 || vdim % 8 != 0 || ldq % 8 != 0 || ldkv % 8 != 0 || ldr % 8 != 0 || ldo % 8 != 0 ||
@@ -520,9 +533,11 @@ extern "C" int tw_latent_prefill(const void* q, long long ldq, int T, const void
   using bf = __nv_bfloat16;
   const LatentPrefillParams p{reinterpret_cast<bf*>(out), ldo, reinterpret_cast<const bf*>(gate), ldg, cu_q, kv_lens,
                               tile_seq, tile_q0, ctx_begin, heads, dim, vdim, (dim + 63) / 64,
-                              scale * 1.4426950408889634f, status};
+                              scale * 1.4426950408889634f, status, window, sink};
 #define TW_CASE(K, V) \
-  if (kc == K && vc == V) return launch_latent_prefill<K, V>(tmQ, tmK, tmR, tmV, p, num_tiles, stream);
+  if (kc == K && vc == V)                                                                               \
+    return window > 0 ? launch_latent_prefill<K, V, true>(tmQ, tmK, tmR, tmV, p, num_tiles, stream)      \
+                      : launch_latent_prefill<K, V, false>(tmQ, tmK, tmR, tmV, p, num_tiles, stream);
   TW_CASE(2, 1) TW_CASE(2, 2) TW_CASE(3, 1) TW_CASE(3, 2) TW_CASE(4, 1)
 #undef TW_CASE
   set_last_error("latent_prefill: unsupported head sizes (dim=%d, rot=%d, vdim=%d)", dim, rot, vdim);

@@ -10,8 +10,8 @@
 //   tw_embed_norm       x32 = table[id] + pairs[row(previous id, id)] ; first = x32 ; xa = rmsnorm(x32) * w
 //   tw_add_prenorm      x32 += y (+ first) ; xa = rmsnorm(x32) * w (the next layer's norm, or the final one)
 //   tw_norm_gate        out = rmsnorm(y) * w * sigmoid(gate) * scale, the mean over `count` of the row's elements
-//   tw_silu_cols, tw_glu  activations behind a projection, for the fp32 products (the bf16 product has them in its
-//                       epilogue): silu in place, act(z_gate) * z_up
+//   tw_act_cols, tw_glu  activations behind a projection, for the fp32 products (the bf16 product has them in its
+//                       epilogue): silu or relu^2 in place, act(z_gate) * z_up
 //
 // One CTA per row (per row and group), the row kept in registers between the passes when it fits.
 #include "tw_host.h"
@@ -316,20 +316,30 @@ norm_gate_kernel(const T* __restrict__ y, long long ldy, const T* __restrict__ g
 
 template <typename T>
 __global__ void __launch_bounds__(256)
-silu_cols_kernel(T* __restrict__ x, long long ldx, int n) {
+act_cols_kernel(T* __restrict__ x, long long ldx, int n, int act) {
   T* row = x + blockIdx.y * ldx;
-  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x)
-    st1(row + i, silu_t<T>(ld1(row + i)));
+  for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < n; i += gridDim.x * blockDim.x) {
+    const float v = ld1(row + i), r = fmaxf(v, 0.f);
+    st1(row + i, act == COL_RELU2 ? r * r : silu_t<T>(v));
+  }
 }
 
-// z rows are [gate | up], d elements each; act 1: silu, 2: the tanh form of gelu
+// z rows are [gate | up], d elements each; act: the kinds of the gated products
 template <typename T>
 __global__ void __launch_bounds__(256)
-glu_kernel(const T* __restrict__ z, long long ldz, T* __restrict__ out, long long ldo, int d, int act) {
+glu_kernel(const T* __restrict__ z, long long ldz, T* __restrict__ out, long long ldo, int d, int act, float limit,
+           float alpha) {
   const T* row = z + blockIdx.y * ldz;
   for (int i = blockIdx.x * blockDim.x + threadIdx.x; i < d; i += gridDim.x * blockDim.x) {
-    const float g = ld1(row + i), u = ld1(row + d + i);
-    st1(out + blockIdx.y * ldo + i, (act == 2 ? gelu_tanh_f(g) : silu_t<T>(g)) * u);
+    float g = ld1(row + i), u = ld1(row + d + i);
+    if (act == GLU_CLAMPED) {
+      g = fminf(g, limit);
+      u = fminf(fmaxf(u, -limit), limit) + 1.f;
+      g *= sigmoid_t<T>(alpha * g);
+    } else {
+      g = act == GLU_GELU_TANH ? gelu_tanh_f(g) : silu_t<T>(g);
+    }
+    st1(out + blockIdx.y * ldo + i, g * u);
   }
 }
 
@@ -528,21 +538,25 @@ extern "C" int tw_norm_gate(const void* y, long long ldy, const void* gate, long
 }
 
 // Grid of the two elementwise kernels; the row is the second grid dimension, launched in blocks of 65535 rows.
-extern "C" int tw_silu_cols(void* x, long long ldx, int T, int n, int dtype, cudaStream_t stream) {
+extern "C" int tw_act_cols(void* x, long long ldx, int T, int n, int act, int dtype, cudaStream_t stream) {
   if (T <= 0 || n <= 0) return 0;
+  if (act != COL_SILU && act != COL_RELU2) {
+    set_last_error("act_cols: unknown activation %d", act);
+    return 1;
+  }
   const int gx = (n + 1023) / 1024;
   for (int t = 0; t < T; t += 65535) {
     const dim3 grid(gx, T - t < 65535 ? T - t : 65535);
-    if (dtype == TW_BF16) silu_cols_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<__nv_bfloat16*>(x) + t * ldx, ldx, n);
-    else silu_cols_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<float*>(x) + t * ldx, ldx, n);
+    if (dtype == TW_BF16) act_cols_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<__nv_bfloat16*>(x) + t * ldx, ldx, n, act);
+    else act_cols_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<float*>(x) + t * ldx, ldx, n, act);
   }
-  return check_launch("silu_cols");
+  return check_launch("act_cols");
 }
 
-extern "C" int tw_glu(const void* z, long long ldz, void* out, long long ldo, int T, int d, int act, int dtype,
-                      cudaStream_t stream) {
+extern "C" int tw_glu(const void* z, long long ldz, void* out, long long ldo, int T, int d, int act, float limit,
+                      float alpha, int dtype, cudaStream_t stream) {
   if (T <= 0 || d <= 0) return 0;
-  if (act != 1 && act != 2) {
+  if (act < GLU_SILU || act > GLU_CLAMPED) {
     set_last_error("glu: unknown activation %d", act);
     return 1;
   }
@@ -551,10 +565,10 @@ extern "C" int tw_glu(const void* z, long long ldz, void* out, long long ldo, in
     const dim3 grid(gx, T - t < 65535 ? T - t : 65535);
     if (dtype == TW_BF16)
       glu_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<const __nv_bfloat16*>(z) + t * ldz, ldz,
-                                           reinterpret_cast<__nv_bfloat16*>(out) + t * ldo, ldo, d, act);
+                                           reinterpret_cast<__nv_bfloat16*>(out) + t * ldo, ldo, d, act, limit, alpha);
     else
       glu_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<const float*>(z) + t * ldz, ldz,
-                                           reinterpret_cast<float*>(out) + t * ldo, ldo, d, act);
+                                           reinterpret_cast<float*>(out) + t * ldo, ldo, d, act, limit, alpha);
   }
   return check_launch("glu");
 }

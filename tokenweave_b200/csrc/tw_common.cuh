@@ -418,19 +418,39 @@ __device__ __forceinline__ void block_sum(float (&v)[R], float* scratch) {
 
 // ---- activations of the bf16 products' epilogues ---------------------------------------------
 // act(gate) * up: the kinds of the gated products (what the launchers call `swiglu`).
-constexpr int GLU_SILU = 1, GLU_GELU_TANH = 2;
+constexpr int GLU_SILU = 1, GLU_GELU_TANH = 2, GLU_CLAMPED = 3;
+// activations of a range of columns of a plain product
+constexpr int COL_SILU = 1, COL_RELU2 = 2;
+
+// What a bf16 product does to its result besides bias and row scale: `glu` a gated kind (0: plain product) with the
+// constants of the clamped one, `col_act` an activation on the columns [col_begin, col_end) of a plain product.
+struct GemmActs {
+  int glu = 0;
+  float limit = 0.f, alpha = 0.f;
+  int col_act = 0, col_begin = 0, col_end = 0;
+};
+
 __device__ __forceinline__ float epi_silu(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 // z / 2 (1 + tanh(u)) = z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float epi_gelu_tanh(float z) {
   const float u2 = -1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
   return __fdividef(z, 1.f + __expf(u2));
 }
-// silu on the columns [begin, end) of a chunk of 32 columns that starts at n
-__device__ __forceinline__ void epi_silu_cols(uint32_t (&v)[32], int n, int begin, int end) {
-  if (n + 32 <= begin || n >= end) return;
+// g = min(gate, limit), u = up inside [-limit, limit]: g sigmoid(alpha g) (u + 1)
+__device__ __forceinline__ float epi_clamped(float g, float u, float limit, float alpha) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g, 1.f + __expf(-alpha * g)) * (u + 1.f);
+}
+// the activation on the columns [begin, end) of a chunk of 32 columns that starts at n
+__device__ __forceinline__ void epi_col_act(uint32_t (&v)[32], int n, const GemmActs& a) {
+  if (n + 32 <= a.col_begin || n >= a.col_end) return;
 #pragma unroll
-  for (int j = 0; j < 32; ++j)
-    if (n + j >= begin && n + j < end) v[j] = __float_as_uint(epi_silu(__uint_as_float(v[j])));
+  for (int j = 0; j < 32; ++j) {
+    if (n + j < a.col_begin || n + j >= a.col_end) continue;
+    const float x = __uint_as_float(v[j]), r = fmaxf(x, 0.f);
+    v[j] = __float_as_uint(a.col_act == COL_RELU2 ? r * r : epi_silu(x));
+  }
 }
 
 }  // namespace tw

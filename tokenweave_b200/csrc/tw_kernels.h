@@ -120,9 +120,12 @@ int tw_moe_align(const int* topk_ids, int n_pairs, int E, int tile_rows, int* ex
                  int* expert_cursor, int* tile_expert, int max_tiles, int* meta, cudaStream_t stream);
 int tw_moe_scatter(const void* x, long long ldx, const int* topk_ids, const float* topk_w,
                    const int* expert_offsets, int* expert_cursor, void* a_sorted, float* row_scale,
-                   int* sorted_pos, int n_pairs, int topk, int H, int E, cudaStream_t stream);
-int tw_moe_combine(const void* y, const int* sorted_pos, void* out, long long ldo, int T, int topk, int H,
-                   cudaStream_t stream);
+                   int* sorted_pos, int n_pairs, int topk, int H, int E, int dtype, cudaStream_t stream);
+int tw_moe_combine(const void* y, const int* sorted_pos, const void* shared_y, long long lds, const float* gate, void* out,
+                   long long ldo, int T, int topk, int H, int dtype, cudaStream_t stream);
+int tw_moe_route(const void* x, long long ldx, const void* w, long long ldw, const float* correction, float* topk_w,
+                 int* topk_ids, float* gate, int T, int H, int E, int gates, int topk, float sum_eps, int dtype,
+                 cudaStream_t stream);
 
 // ---- in-kernel collectives (comm_fused.cu) ----
 // mc_base: multicast address of the symmetric buffer or NULL (peer transport). peer_bases /
@@ -145,7 +148,11 @@ int tw_wait_probe(uint32_t* flag, unsigned long long budget_ns, uint32_t* status
 int tw_gemm_f32(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc,
                 const float* bias, int M, int N, int K, cudaStream_t stream);
 
-// In the launchers below dtype is 0 for bf16 and 1 for fp32 activations and weights.
+int tw_gemm_f32_grouped(const float* A, long long lda, const float* B, long long ldb, float* C, long long ldc, int M, int N,
+                        int K, const int* tile_expert, const int* num_tiles, int tile_rows, int n_per_expert,
+                        const float* row_scale, cudaStream_t stream);
+
+// In the launchers here dtype is 0 for bf16 and 1 for fp32 activations and weights.
 // ---- fp32 residual stream, norm of a sublayer's output, feed-forward activation (rownorm.cu) ----
 int tw_embed_residual(const int* ids, const void* table, long long ldt, float* x32, long long ldx, void* xa,
                       long long lda, int T, int H, int vocab, int dtype, cudaStream_t stream);
@@ -164,32 +171,45 @@ int tw_add_prenorm(const void* y, long long ldy, float* x32, long long ldx, cons
                    const void* w, void* xa, long long lda, int T, int H, float eps, int dtype, cudaStream_t stream);
 int tw_norm_gate(const void* y, long long ldy, const void* gate, long long ldg, const void* w, void* out, long long ldo,
                  int T, int C, int count, float eps, float scale, int dtype, cudaStream_t stream);
-int tw_silu_cols(void* x, long long ldx, int T, int n, int dtype, cudaStream_t stream);
-int tw_glu(const void* z, long long ldz, void* out, long long ldo, int T, int d, int act, int dtype, cudaStream_t stream);
+int tw_act_cols(void* x, long long ldx, int T, int n, int act, int dtype, cudaStream_t stream);
+int tw_glu(const void* z, long long ldz, void* out, long long ldo, int T, int d, int act, float limit, float alpha, int dtype,
+           cudaStream_t stream);
+
+// ---- hyper-connections (streams.cu) ----
+int tw_embed_streams(const int* ids, const void* table, long long ldt, int vocab, float* x, long long ldx, long long lds,
+                     int S, const float* in, const void* w, float offset, void* xa, long long lda, int T, int H, float eps,
+                     int dtype, cudaStream_t stream);
+int tw_streams_step(const void* y, long long ldy, float* x, long long ldx, long long lds, int S, const float* mix,
+                    const float* out, float mult, const float* in, int store, const void* w, float offset, void* xa,
+                    long long lda, int T, int H, float eps, int dtype, cudaStream_t stream);
 
 // ---- grouped attention (grouped_attn.cu; tensor cores: attn_prefill_split.cu, attn_decode_tc.cu, bf16) ----
 int tw_qkv_prep(const void* p, long long ldp, int T, int heads, int kv_heads, int dim, int dp, int vp, void* q,
                 long long ldq, void* k_cache, void* v_cache, const int* positions, const int* cache_slots,
                 const void* conv_w, void* conv_state, int taps, const int* row_seq, const int* cu_q, const int* kv_lens,
                 const int* slots, int n_seqs, int single, int norm, const void* wq, const void* wk, float eps,
-                float temp_coef, int temp_every, int dtype, cudaStream_t stream);
+                float temp_coef, int temp_every, const float* cos_sin, int rot_dims, int dtype, cudaStream_t stream);
 int tw_attn_rows(const void* q, long long ldq, const void* k_cache, const void* v_cache, int page, void* out,
                  long long ldo, const int* tok_row, const int* tok_seq, const int* tok_kvlen, int n,
                  const int* block_table, int max_blocks, int heads, int kv_heads, int dp, int vp, float scale,
-                 const float* slopes, int sink, float out_scale, int dtype, cudaStream_t stream);
+                 const float* slopes, int sink, float out_scale, int window, int keep, int dtype, cudaStream_t stream);
 int tw_attn_prefill_grouped(const void* q, long long ldq, int T, const void* k_cache, const void* v_cache,
                             int num_blocks, int page, void* out, long long ldo, const int* cu_q, const int* kv_lens,
                             const int* block_table, int max_blocks, const int* tile_seq, const int* tile_q0,
                             int num_tiles, int hq, int hkv, int dp, int vp, float scale, const float* slopes, int sink,
-                            float out_scale, uint32_t* status, cudaStream_t stream);
+                            float out_scale, int window, int keep, uint32_t* status, cudaStream_t stream);
 int tw_attn_decode_grouped(const void* q, long long ldq, const void* k_cache, const void* v_cache, int num_blocks,
                            int page, void* out, long long ldo, const int* tok_row, const int* tok_seq,
                            const int* tok_kvlen, int n_tok, const int* block_table, int max_blocks, int hq, int hkv,
-                           int dp, int vp, float scale, const float* slopes, int sink, float out_scale, int splits,
-                           float* part_o, float* part_ml, uint32_t* status, cudaStream_t stream);
-int tw_gemm_bf16_silu(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc,
-                      const void* bias, int M, int N, int K, int silu_begin, int silu_end, int max_ctas, int plan_hint,
-                      uint32_t* status, cudaStream_t stream);
+                           int dp, int vp, float scale, const float* slopes, int sink, float out_scale, int window,
+                           int keep, int splits, float* part_o, float* part_ml, uint32_t* status, cudaStream_t stream);
+int tw_gemm_bf16_act(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc,
+                     const void* bias, int M, int N, int K, int act, int act_begin, int act_end, int max_ctas, int plan_hint,
+                     uint32_t* status, cudaStream_t stream);
+int tw_gemm_bf16_clamped(const void* A, long long lda, const void* B, long long ldb, long long rows_b, void* C,
+                         long long ldc, int M, int N, int K, float limit, float alpha, int up_row_offset,
+                         const int* tile_expert, const int* num_m_tiles_dev, int n_per_expert, int tile_rows, int max_ctas,
+                         int plan_hint, uint32_t* status, cudaStream_t stream);
 
 // ---- latent attention (latent_attn.cu) ----
 int tw_latent_prep(const void* p, long long ldp, int q_off, int q_rank, const void* wq, void* cq, long long ldcq,
@@ -206,17 +226,18 @@ int tw_head_gemm(const void* A, long long lda, int a_hs, const int* a_rows, cons
                  int heads, int M, int N, int K, int dtype, cudaStream_t stream);
 int tw_latent_attn(const void* qa, const void* cache, const int* tok_seq, const int* tok_kvlen, int n,
                    const int* block_table, int max_blocks, int page, void* out, int heads, int row, int kv_rank,
-                   float scale, int dtype, cudaStream_t stream);
+                   float scale, int window, const float* sink, int dtype, cudaStream_t stream);
 // tensor-core forms (latent_attn_decode.cu, latent_attn_prefill.cu), bf16
 int tw_latent_decode(const void* qa, const void* cache, int num_blocks, int page, const int* tok_seq,
                      const int* tok_kvlen, int n, const int* block_table, int max_blocks, void* out, int heads, int row,
-                     int kv_rank, float scale, int splits, float* part_o, float* part_ml, uint32_t* status,
-                     cudaStream_t stream);
+                     int kv_rank, float scale, int window, const float* sink, int splits, float* part_o, float* part_ml,
+                     uint32_t* status, cudaStream_t stream);
 int tw_latent_prefill(const void* q, long long ldq, int T, const void* kv, long long ldkv, const void* kr, long long ldr,
                       int ctx_rows, const int* ctx_begin, void* out, long long ldo, const void* gate, long long ldg,
                       const int* cu_q, const int* kv_lens, const int* tile_seq, const int* tile_q0, int num_tiles,
-                      int heads, int dim, int rot, int vdim, float scale, uint32_t* status, cudaStream_t stream);
-int tw_latent_gather(const void* cache, void* dst, const int* seqs, const int* cu, int n_seqs, int max_rows,
+                      int heads, int dim, int rot, int vdim, float scale, int window, const float* sink, uint32_t* status,
+                      cudaStream_t stream);
+int tw_latent_gather(const void* cache, void* dst, const int* seqs, const int* cu, const int* from, int n_seqs, int max_rows,
                      const int* block_table, int max_blocks, int page, int row_bytes, cudaStream_t stream);
 
 // ---- state-space recurrence (ssm.cu, ssd_chunk.cu, ssd_chunk_tc.cu) ----

@@ -16,19 +16,55 @@ decays and recurrent state are fp32 in both.
 """
 from __future__ import annotations
 
+import math
 from typing import Optional
 
 import torch
 from torch import nn
 
+from .. import ops
 from ..ops import hybrid as hops
 from ..ops import reference
 from .attention import AttentionMetadata
 from .linear import PaddedLinear, pad8
+from .moe import expert_index, max_expert_rows, run_experts
 
 
 def _vec(n: int, dtype, device, fill: float = 1.0) -> nn.Parameter:
     return nn.Parameter(torch.full((n,), fill, dtype=dtype, device=device), requires_grad=False)
+
+
+# ---- rotation ---------------------------------------------------------------------------------------------------------
+# ``rot`` = {"base", "dims", "scaling": None or YaRN's {"factor", "original", "fast", "slow"}}
+def rope_table(rt, rot: dict) -> torch.Tensor:
+    """Cosines and sines by position ([positions, dims]: cosines, then sines), one table per kind of rotation in a model."""
+    s = rot.get("scaling")
+    key = (int(rot["dims"]), float(rot["base"]), tuple(sorted((s or {}).items())))
+    if key not in rt.rope_tables:
+        scaling = None
+        if s:
+            factor = float(s["factor"])
+            scaling = dict(rope_type="yarn", factor=factor, original_max_position_embeddings=float(s["original"]),
+                           beta_fast=float(s["fast"]), beta_slow=float(s["slow"]),
+                           attention_factor=0.1 * math.log(factor) + 1.0)
+        rt.rope_tables[key] = reference.build_cos_sin_cache(key[0], rt.max_positions, key[1], scaling, rt.device)
+    return rt.rope_tables[key]
+
+
+def check_rotation(rot: dict, size: int) -> int:
+    dims = int(rot["dims"])
+    if dims % 2 or not 0 < dims <= size:
+        raise ValueError(f"rotated dimensions {dims} do not fit a part of {size}")
+    return dims
+
+
+def pair_order(dims: int, size: int, to_halves: bool) -> torch.Tensor:
+    """Order of a head's ``size`` dimensions, of which the first ``dims`` turn, that changes neighbouring pairs (2i, 2i + 1)
+    into pairs of the two halves (i, i + dims / 2), or back. Queries and keys stored in one such order have the same
+    products, so a design's pairing is brought to the kernel's once, in the weights."""
+    i = torch.arange(dims)
+    order = torch.cat([i[0::2], i[1::2]]) if to_halves else i.view(2, -1).t().reshape(-1)
+    return torch.cat([order, torch.arange(dims, size)])
 
 
 class Mixer(nn.Module):
@@ -75,18 +111,25 @@ class LatentAttention(Mixer):
     weighted latent sum, so attention runs over cache rows directly (decoding, short runs). Expanded: the context's
     keys and values are made from the gathered latents with one matrix product and a tile kernel attends (long runs
     of a prompt).
+
+    Options: ``gated``; ``window`` > 0: a position sees the last ``window`` positions, itself among them; ``sink``: a learned
+    number per head whose exponential joins the softmax's denominator; ``neighbour_pairs``: dimensions 2i and 2i + 1 turn
+    together (else i and i + dims / 2).
     """
 
-    def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device, max_positions: int, gated: bool = True):
+    def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device, gated: bool = True, window: int = 0,
+                 sink: bool = False, neighbour_pairs: bool = False):
         super().__init__()
         self.heads, self.dim, self.rot_dim, self.vdim = (int(sizes[k]) for k in ("heads", "dim", "rot_dim", "vdim"))
         self.kv_rank, self.q_rank = int(sizes["kv_rank"]), int(sizes["q_rank"])
         self.scale, self.eps, self.width, self.gated = float(sizes["scale"]), eps, width, gated
         self.rot = dict(sizes["rot"])
-        self.rot_dims = int(self.rot["dims"])
-        if self.rot_dims % 2 or not 0 < self.rot_dims <= self.rot_dim:
-            raise ValueError(f"rotated dimensions {self.rot_dims} do not fit a part of {self.rot_dim}")
-        self.max_positions = max_positions
+        self.rot_dims = check_rotation(self.rot, self.rot_dim)
+        self.window = int(window)
+        # the kernels turn pairs of halves
+        self.rot_order = pair_order(self.rot_dims, self.rot_dim, True) if neighbour_pairs else None
+        self.sink = (nn.Parameter(torch.zeros(self.heads, dtype=torch.float32, device=device), requires_grad=False)
+                     if sink else None)
         H, q8, kv8 = self.heads, pad8(self.q_rank), pad8(self.kv_rank + self.rot_dim)
         # one projection for everything that reads the layer's input: [query latent | kv latent, rotated part | gate]
         self.kv_off, self.gate_off = q8, q8 + kv8
@@ -117,7 +160,7 @@ class LatentAttention(Mixer):
 
     def launch_key(self, meta: AttentionMetadata, block_size: int, sm_count: int) -> tuple:
         return hops.latent_decode_plan(meta.num_single, self.heads, self.row, self.kv_rank, block_size,
-                                       self.o_proj.weight.dtype, meta.max_kv_len, sm_count)
+                                       self.o_proj.weight.dtype, meta.max_kv_len, sm_count, self.window)
 
     # ---- cache -----------------------------------------------------------------------------------------
     def cache_bytes_per_block(self, block_size: int) -> int:
@@ -128,26 +171,7 @@ class LatentAttention(Mixer):
         kept["latents"] = torch.zeros(num_blocks, block_size, self.row, dtype=w.dtype, device=w.device)
 
     def bind_runtime(self, rt) -> None:
-        key = self.rope_key()
-        if key not in rt.rope_tables:
-            rt.rope_tables[key] = self.make_rope_table()
-        self.cos_sin = rt.rope_tables[key]
-
-    def rope_key(self) -> tuple:
-        s = self.rot.get("scaling")
-        return (self.rot_dims, float(self.rot["base"]), tuple(sorted((s or {}).items())))
-
-    def make_rope_table(self) -> torch.Tensor:
-        import math
-        s = self.rot.get("scaling")
-        scaling = None
-        if s:
-            factor = float(s["factor"])
-            scaling = dict(rope_type="yarn", factor=factor, original_max_position_embeddings=float(s["original"]),
-                           beta_fast=float(s["fast"]), beta_slow=float(s["slow"]),
-                           attention_factor=0.1 * math.log(factor) + 1.0)
-        return reference.build_cos_sin_cache(self.rot_dims, self.max_positions, float(self.rot["base"]), scaling,
-                                             self.o_proj.weight.device)
+        self.cos_sin = rope_table(rt, self.rot)
 
     # ---- weights ---------------------------------------------------------------------------------------
     def tensor_targets(self) -> dict:
@@ -156,11 +180,19 @@ class LatentAttention(Mixer):
         def uk(t):
             self.ukv_proj.load_rows(t, 0)
             self.ukt_w.data[:, :, :D].copy_(t.view(H, D, R).transpose(1, 2))
+
+        def reordered(t, heads, size):
+            """Rows of the rotated part, the last of every head's, in the kernels' order of pairs."""
+            if self.rot_order is None:
+                return t
+            order = torch.cat([torch.arange(size - self.rot_dim), size - self.rot_dim + self.rot_order])
+            return t.view(heads, size, -1)[:, order.to(t.device)].reshape(t.shape)
         out = {
             "dq": ((Q, W), lambda t: self.in_proj.load_rows(t, 0)),
             "dq.norm": ((Q,), self.q_norm_w.data.copy_),
-            "uq": ((H * (D + self.rot_dim), Q), lambda t: self.uq_proj.load_rows(t, 0)),
-            "dkv": ((R + self.rot_dim, W), lambda t: self.in_proj.load_rows(t, self.kv_off)),
+            "uq": ((H * (D + self.rot_dim), Q), lambda t: self.uq_proj.load_rows(reordered(t, H, D + self.rot_dim), 0)),
+            "dkv": ((R + self.rot_dim, W),
+                    lambda t: self.in_proj.load_rows(reordered(t, 1, R + self.rot_dim), self.kv_off)),
             "dkv.norm": ((R,), self.kv_norm_w.data.copy_),
             "uk": ((H * D, R), uk),
             "uv": ((H * V, R), lambda t: self.ukv_proj.load_rows(t, H * D)),
@@ -168,6 +200,8 @@ class LatentAttention(Mixer):
         }
         if self.gated:
             out["g"] = ((H * V, W), lambda t: self.in_proj.load_rows(t, self.gate_off))
+        if self.sink is not None:
+            out["sink"] = ((H,), self.sink.data.copy_)
         return out
 
     # ---- forward ---------------------------------------------------------------------------------------
@@ -188,19 +222,19 @@ class LatentAttention(Mixer):
                                self.cos_sin, meta.positions, qa)
             o = rt.buffer("latent_out", m, H * self.kv_rank).view(m, H, self.kv_rank)
             hops.latent_attention(qa, cache, meta.tok_seq, meta.tok_kvlen, m, meta.block_table, self.kv_rank,
-                                  self.scale, o, meta.max_kv_len, rt.sm_count)
+                                  self.scale, o, meta.max_kv_len, rt.sm_count, window=self.window, sink=self.sink)
             hops.latent_values(o, meta.tok_row, w_uv, H, self.vdim, self.kv_rank, gate, attn)
         if meta.num_tiles:
             # keys and values of the tiles' contexts (the step's own tokens are in the cache already)
             rows = meta.extra_cpu["ctx_rows"]
             lat = rt.buffer("ctx_latent", rows, self.row)
             hops.latent_gather(cache, meta.extra["ctx_seqs"], meta.extra["ctx_cu"], meta.extra_cpu["ctx_max"],
-                               meta.block_table, lat)
+                               meta.block_table, lat, meta.extra["ctx_first"])
             kv = self.ukv_proj(lat[:, :self.ukv_proj.in_padded], out=rt.buffer("ctx_kv", rows, self.ukv_proj.out_padded))
             hops.rope_tail_(q, H, self.dim + self.rot_dim, self.dim, self.rot_dims, self.cos_sin, meta.positions)
             hops.latent_prefill(q, kv, lat, pad8(self.kv_rank), rows, meta.extra["ctx_begin"], attn, gate, meta.cu_q,
                                 meta.kv_lens, meta.tile_seq, meta.tile_q0, meta.num_tiles, H, self.dim, self.rot_dim,
-                                self.vdim, self.scale)
+                                self.vdim, self.scale, self.window, self.sink)
         self.o_proj(attn, out=out)
 
 
@@ -209,7 +243,7 @@ class Mamba2Mixer(Mixer):
     recurrence per head with an fp32 state, skip ``D x``, gate, grouped RMS norm, output projection."""
     recurrent = True
 
-    def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device, max_positions: int = 0):
+    def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device):
         super().__init__()
         self.heads, self.vdim, self.N, self.groups = (int(sizes[k]) for k in ("heads", "vdim", "state", "groups"))
         self.taps, self.norm_groups = int(sizes["conv"]), int(sizes["norm_groups"])
@@ -288,7 +322,22 @@ class Mamba2Mixer(Mixer):
         self.o_proj(g, out=out)
 
 
-class PolyNormMLP(nn.Module):
+class FeedForward(nn.Module):
+    """A sublayer without state: ``forward(x, rt, out)``."""
+
+    def workspaces(self) -> list[tuple[str, int]]:
+        """(name, columns) of the runtime buffers with a row per token."""
+        raise NotImplementedError
+
+    def bind_runtime(self, rt) -> None:
+        """Called once when the runtime exists: buffers of other shapes."""
+
+    def tensor_targets(self) -> dict:
+        """checkpoint name (behind ``<layer>.mlp.``) -> (shape, callable taking the tensor)."""
+        raise NotImplementedError
+
+
+class PolyNormMLP(FeedForward):
     """``W_down act(W_up x)`` with the polynomial-norm activation ``a N(z) + b N(z^2) + c N(z^3) + e``."""
 
     def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device):
@@ -311,6 +360,118 @@ class PolyNormMLP(nn.Module):
         z = self.up_proj(x, out=rt.buffer("proj", n, self.up_proj.out_padded))
         a = hops.polynorm(z, self.coef, self.eps, rt.buffer("act", n, self.down_proj.in_padded), self.ff)
         self.down_proj(a, out=out)
+
+
+class ActMLP(FeedForward):
+    """``W_down act(W_up x)`` with an elementwise activation: "relu2" (the square of relu) or "silu"."""
+
+    def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device):
+        super().__init__()
+        self.ff, self.width, self.act = int(sizes["ff"]), width, str(sizes["act"])
+        if self.act not in ops.COL_ACTS:
+            raise ValueError(f"unknown activation {self.act!r} (known: {sorted(ops.COL_ACTS)})")
+        self.up_proj = PaddedLinear(width, self.ff, dtype=dtype, device=device)
+        self.down_proj = PaddedLinear(self.ff, width, dtype=dtype, device=device)
+
+    def workspaces(self) -> list[tuple[str, int]]:
+        return [("act", self.down_proj.in_padded)]
+
+    def tensor_targets(self) -> dict:
+        return {"up": ((self.ff, self.width), lambda t: self.up_proj.load_rows(t, 0)),
+                "down": ((self.width, self.ff), lambda t: self.down_proj.load_rows(t, 0))}
+
+    def forward(self, x: torch.Tensor, rt, out: torch.Tensor) -> None:
+        a = rt.buffer("act", x.shape[0], self.down_proj.in_padded)
+        hops.projection(x, self.up_proj.weight, None, (0, self.up_proj.out_padded), a, self.act)
+        self.down_proj(a, out=out)
+
+
+class RoutedMLP(FeedForward):
+    """Mixture of experts: every token takes ``top`` of ``experts`` gated feed-forwards, chosen by the softmax over all
+    experts plus a correction per expert; their outputs are weighted with the scores (without it) over the scores' sum +
+    ``sum_eps``. ``act``: as for ``ops.gemm``. ``shared`` = {"ff", "act"} or None: one more gated feed-forward that every
+    token takes, times the sigmoid of a projection to one number.
+
+    The router's rows and the shared feed-forward's gate are one product; the pipeline behind it is ``layers/moe.py``."""
+
+    def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device):
+        super().__init__()
+        self.experts, self.top, self.ff, self.width = (*(int(sizes[k]) for k in ("experts", "top", "ff")), width)
+        if not 0 < self.top <= self.experts:
+            raise ValueError(f"{self.top} of {self.experts} experts")
+        self.act, self.sum_eps = self._act(sizes["act"]), float(sizes.get("sum_eps", 0.0))
+        w8, self.f8 = pad8(width), pad8(self.ff)
+        par = lambda *s, dt=dtype: nn.Parameter(torch.zeros(*s, dtype=dt, device=device), requires_grad=False)
+        shared = sizes.get("shared")
+        self.router_w = par(self.experts + (1 if shared else 0), w8)
+        self.correction = par(self.experts, dt=torch.float32)
+        self.w13, self.w2 = par(self.experts, 2 * self.f8, w8), par(self.experts, w8, self.f8)
+        self.shared_up = self.shared_down = None
+        if shared:
+            self.shared_ff, self.shared_act = int(shared["ff"]), self._act(shared["act"])
+            self.shared_up = PaddedLinear(width, 2 * pad8(self.shared_ff), dtype=dtype, device=device)
+            self.shared_down = PaddedLinear(self.shared_ff, width, dtype=dtype, device=device)
+
+    @staticmethod
+    def _act(act):
+        return act if isinstance(act, str) else (act[0], float(act[1]), float(act[2]))
+
+    # ---- buffers -------------------------------------------------------------------------------------------
+    def workspaces(self) -> list[tuple[str, int]]:
+        if self.shared_up is None:
+            return []
+        out = [("shared_act", self.shared_down.in_padded), ("shared_out", self.shared_down.out_padded)]
+        return out + ([("shared_gate_up", self.shared_up.out_padded)] if self.w2.dtype == torch.float32 else [])
+
+    def _sorted_rows(self) -> list[tuple[str, int]]:
+        w8 = self.w2.shape[1]
+        out = [("a_sorted", w8), ("act", self.f8), ("y", w8)]
+        return out + ([("gate_up", 2 * self.f8)] if self.w2.dtype == torch.float32 else [])
+
+    def bind_runtime(self, rt) -> None:
+        if not self.w2.is_cuda:
+            return
+        key = ("experts", self.experts, self.top)
+        if key not in rt.tables:
+            rt.tables[key] = expert_index(rt.max_tokens, self.top, self.experts, self.w2.device)
+        for name, cols in self._sorted_rows():
+            rt.buffer("experts." + name, max_expert_rows(rt.max_tokens, self.top, self.experts), cols)
+
+    # ---- weights -------------------------------------------------------------------------------------------
+    def tensor_targets(self) -> dict:
+        W, F, f8 = self.width, self.ff, self.f8
+        out = {"router": ((self.experts, W), lambda t: self.router_w.data[:self.experts, :W].copy_(t)),
+               "correction": ((self.experts,), self.correction.data.copy_)}
+        for e in range(self.experts):
+            out[f"e{e}.gate"] = ((F, W), lambda t, e=e: self.w13.data[e, :F, :W].copy_(t))
+            out[f"e{e}.up"] = ((F, W), lambda t, e=e: self.w13.data[e, f8:f8 + F, :W].copy_(t))
+            out[f"e{e}.down"] = ((W, F), lambda t, e=e: self.w2.data[e, :W, :F].copy_(t))
+        if self.shared_up is not None:
+            S = self.shared_ff
+            out["shared.gate"] = ((S, W), lambda t: self.shared_up.load_rows(t, 0))
+            out["shared.up"] = ((S, W), lambda t: self.shared_up.load_rows(t, pad8(S)))
+            out["shared.down"] = ((W, S), lambda t: self.shared_down.load_rows(t, 0))
+            out["shared.sg"] = ((1, W), lambda t: self.router_w.data[self.experts:, :W].copy_(t))
+        return out
+
+    # ---- forward -------------------------------------------------------------------------------------------
+    def forward(self, x: torch.Tensor, rt, out: torch.Tensor) -> None:
+        n, shared, gate = x.shape[0], None, None
+        weights, ids, gates = ops.moe_route(x, self.router_w, self.experts, self.top, self.correction, self.sum_eps)
+        if self.shared_up is not None:
+            a = rt.buffer("shared_act", n, self.shared_down.in_padded)
+            tmp = rt.buffer("shared_gate_up", n, self.shared_up.out_padded) if x.dtype == torch.float32 else None
+            hops.gated_product(x, self.shared_up.weight, self.shared_act, a, tmp)
+            shared = self.shared_down(a, out=rt.buffer("shared_out", n, self.shared_down.out_padded))
+            gate = gates[:, 0]
+        if not x.is_cuda:
+            y = reference.moe_experts(x, self.w13, self.w2, weights, ids, self.act)
+            out.copy_(y if shared is None else y + gate[:, None] * shared)
+            return
+        ws = dict(rt.tables[("experts", self.experts, self.top)])
+        rows = max_expert_rows(n, self.top, self.experts)
+        ws.update((name, rt.buffer("experts." + name, rows, cols)) for name, cols in self._sorted_rows())
+        run_experts(x, weights, ids, self.w13, self.w2, ws, out, self.act, shared, gate)
 
 
 # ---- several parts side by side --------------------------------------------------------------------------------------
@@ -369,13 +530,18 @@ class GroupedAttention(Part):
     * ``q_temp`` = {"coef", "every"}: queries times ``1 + coef * ln(floor((p + 1) / every) + 1)`` at position p;
     * ``distance_bias``: ``2^(-8 (h + 1) / heads) * (i - j)`` is taken off the score of head h;
     * ``sink``: one is added to the softmax's denominator (a key of score 0 without a value);
-    * ``out_scale``: factor on the result.
+    * ``out_scale``: factor on the result;
+    * ``rot``: rotation of the first ``rot["dims"]`` dimensions of queries and keys, behind the norm;
+      ``neighbour_pairs``: dimensions 2i and 2i + 1 turn together (else i and i + dims / 2);
+    * ``window`` > 0: a position sees the last ``window`` positions, itself among them, and the sequence's first
+      ``keep_first``.
     """
     attends = True
 
     def __init__(self, sizes: dict, eps: float, *, dtype, device, bias: bool = False, conv: Optional[int] = None,
                  qk_norm: Optional[str] = None, q_temp: Optional[dict] = None, distance_bias: bool = False,
-                 sink: bool = False, out_scale: float = 1.0):
+                 sink: bool = False, out_scale: float = 1.0, rot: Optional[dict] = None, neighbour_pairs: bool = False,
+                 window: int = 0, keep_first: int = 0):
         super().__init__()
         self.heads, self.kv_heads, self.dim, self.vdim = (int(sizes[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
         if self.heads % self.kv_heads:
@@ -398,8 +564,17 @@ class GroupedAttention(Part):
             self.q_norm_w, self.k_norm_w = (_vec(i * self.dp, dtype, device, 0.0) for i in n)
         self.device = torch.device(device)
         self.slopes: Optional[torch.Tensor] = None
+        self.rot, self.window, self.keep = (dict(rot) if rot else None), int(window), int(keep_first)
+        # the kernels turn neighbouring pairs
+        self.rot_order = (pair_order(check_rotation(rot, self.dim), self.dim, False)
+                          if rot and not neighbour_pairs else None)
+        if rot:
+            check_rotation(rot, self.dim)
+        self.cos_sin: Optional[torch.Tensor] = None
 
     def bind_runtime(self, rt) -> None:
+        if self.rot:
+            self.cos_sin = rope_table(rt, self.rot)
         if self.distance_bias:
             h = torch.arange(1, self.heads + 1, dtype=torch.float64)
             self.slopes = torch.exp2(-8.0 * h / self.heads).float().to(self.device)
@@ -425,13 +600,20 @@ class GroupedAttention(Part):
     # ---- launches ------------------------------------------------------------------------------------------
     @property
     def tileable(self) -> bool:
-        return self.device.type == "cuda" and hops.attention_tileable(self.dtype, self.dp, self.vp)
+        return (self.device.type == "cuda" and hops.attention_tileable(self.dtype, self.dp, self.vp)
+                and not (self.window and self.distance_bias))
 
     def launch_key(self, meta: AttentionMetadata, block_size: int, sm_count: int) -> tuple:
         return hops.attention_rows_plan(meta.num_single, self.heads, self.kv_heads, self.dp, self.vp, block_size, self.dtype,
-                                        meta.max_kv_len, sm_count)
+                                        meta.max_kv_len, sm_count, self.window, self.keep)
 
     # ---- weights -------------------------------------------------------------------------------------------
+    def _reordered(self, t: torch.Tensor) -> torch.Tensor:
+        """Something with a leading axis of query or key dimensions, in the kernels' order of pairs."""
+        if self.rot_order is None:
+            return t
+        return t.reshape(-1, self.dim, *t.shape[1:])[:, self.rot_order.to(t.device)].reshape(t.shape)
+
     def tensor_targets(self, width: int, load_in, load_bias, load_out) -> dict:
         H, G, D, V = self.heads, self.kv_heads, self.dim, self.vdim
         spans = {"q": (H, D, self.dp, 0), "k": (G, D, self.dp, self.k_off), "v": (G, V, self.vp, self.v_off)}
@@ -447,6 +629,10 @@ class GroupedAttention(Part):
             for name, w, n in (("q", self.q_norm_w, H), ("k", self.k_norm_w, G)):
                 n = n if self.qk_norm == "whole" else 1
                 out[name + ".norm"] = ((n * D,), _pad_heads(w, n, D, self.dp))
+        if self.rot_order is not None:
+            for name, (shape, put) in list(out.items()):
+                if name[0] in "qk":
+                    out[name] = (shape, lambda t, put=put: put(self._reordered(t)))
         return out
 
     # ---- forward -------------------------------------------------------------------------------------------
@@ -454,9 +640,9 @@ class GroupedAttention(Part):
         q = rt.buffer("query", p.shape[0], self.k_off)
         hops.qkv_prep(p, self.heads, self.kv_heads, self.dim, self.vdim, q, kept["k"], kept["v"], meta, self.conv_w,
                       kept.get("conv"), self.qk_norm, self.q_norm_w, self.k_norm_w, self.eps, self.temp_coef,
-                      self.temp_every)
+                      self.temp_every, self.cos_sin)
         hops.grouped_attention(q, kept["k"], kept["v"], out, meta, self.heads, self.kv_heads, self.scale, self.slopes,
-                               self.sink, self.out_scale, rt.sm_count)
+                               self.sink, self.out_scale, rt.sm_count, window=self.window, keep=self.keep)
 
 
 class LightningAttention(Part):
@@ -550,8 +736,7 @@ class SumMixer(Mixer):
     "". One matrix product makes every part's projected input, one more the feed-forward's, and the last one takes the
     parts' results side by side, so that their sum is its accumulation."""
 
-    def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device, max_positions: int = 0,
-                 mlp: Optional[dict] = None):
+    def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device, mlp: Optional[dict] = None):
         super().__init__()
         self.width = width
         self.parts = nn.ModuleDict()
@@ -638,4 +823,4 @@ class SumMixer(Mixer):
 
 
 MIXERS = {"latent_attention": LatentAttention, "mamba2": Mamba2Mixer, "sum": SumMixer}
-FEED_FORWARDS = {"dense": PolyNormMLP}
+FEED_FORWARDS = {"dense": PolyNormMLP, "activated": ActMLP, "routed": RoutedMLP}

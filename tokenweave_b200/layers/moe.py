@@ -1,4 +1,5 @@
-"""Mixture-of-experts MLP with tensor-sharded experts (Mixtral).
+"""Mixture-of-experts MLPs: the grouped-experts pipeline that every routed feed-forward runs (:func:`run_experts`), and the
+layer with tensor-sharded experts (Mixtral). The routed feed-forward of hybrid decoders is ``layers/mixers.py::RoutedMLP``.
 
 Counterpart of vllm/model_executor/layers/fused_moe/layer.py:840-895 and fused_moe.py:1230-1426. Expert
 weights are ``w13 = [E, 2*I/tp, H]`` (w1 = gate rows first, w3 = up rows second) and
@@ -17,12 +18,51 @@ import torch
 from torch import nn
 
 from .. import ops
+from ..ops import hybrid as hops
 from ..ops import reference
 from ..parallel.state import get_tp
 
 TILE_ROWS = 128          # rows every expert's group is padded to ...
 TILE_ROWS_PAIR = 256     # ... or, once an expert gets 512 rows or more on average, this: the groups then run on
                          # CTA pairs (256-row tcgen05 tiles), which more than pays for the extra padding
+
+
+def max_expert_rows(tokens: int, top_k: int, experts: int) -> int:
+    """Rows of the expert-sorted buffers: every expert's group padded to the larger tile."""
+    n = tokens * top_k + experts * (TILE_ROWS_PAIR - 1)
+    return (n + TILE_ROWS_PAIR - 1) // TILE_ROWS_PAIR * TILE_ROWS_PAIR
+
+
+def expert_index(tokens: int, top_k: int, experts: int, device) -> dict:
+    """Bookkeeping buffers of :func:`run_experts` for up to ``tokens`` tokens."""
+    rows = max_expert_rows(tokens, top_k, experts)
+    i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=device)
+    return dict(offsets=i32(experts + 1), cursor=i32(experts), tile_expert=i32(rows // TILE_ROWS), meta=i32(2),
+                row_scale=torch.zeros(rows, dtype=torch.float32, device=device), sorted_pos=i32(tokens, top_k))
+
+
+def run_experts(x: torch.Tensor, topk_w: torch.Tensor, topk_ids: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, ws: dict,
+                out: torch.Tensor, act="silu", shared: Optional[torch.Tensor] = None,
+                gate: Optional[torch.Tensor] = None, pair_tiles: bool = True, max_ctas: int = 0) -> None:
+    """``out = sum_k w_k W2[e_k] act(W13[e_k] x) (+ gate * shared)`` (CUDA). ``ws``: the buffers of :func:`expert_index` and
+    the expert-sorted rows ``a_sorted``, ``act`` and ``y`` (in fp32 also ``gate_up``: that product has no gated form)."""
+    T, top_k = topk_ids.shape
+    E, I2, H = w13.shape
+    tile_rows = TILE_ROWS_PAIR if T * top_k >= 512 * E and pair_tiles else TILE_ROWS
+    n_rows = (T * top_k + E * (tile_rows - 1) + tile_rows - 1) // tile_rows * tile_rows
+    tile_expert = ws["tile_expert"][: n_rows // tile_rows]
+    ops.moe_align(topk_ids, E, tile_rows, ws["offsets"], ws["cursor"], tile_expert, ws["meta"])
+    sorted_pos = ws["sorted_pos"][:T]
+    ops.moe_scatter(x, topk_ids, topk_w, ws["offsets"], ws["cursor"], ws["a_sorted"], ws["row_scale"], sorted_pos, E)
+    a, mid = ws["a_sorted"][:n_rows], ws["act"][:n_rows]
+    groups = dict(tile_expert=tile_expert, num_m_tiles=ws["meta"][:1], max_ctas=max_ctas, tile_rows=tile_rows)
+    if x.dtype == torch.float32:
+        z = ops.gemm(a, w13.view(E * I2, H), out=ws["gate_up"][:n_rows], n_per_expert=I2, **groups)
+        hops.glu(z, act, mid)
+    else:
+        ops.gemm(a, w13.view(E * I2, H), out=mid, swiglu=True, act=act, n_per_expert=I2, **groups)
+    y = ops.gemm(mid, w2.view(E * H, I2 // 2), out=ws["y"][:n_rows], row_scale=ws["row_scale"], n_per_expert=H, **groups)
+    ops.moe_combine(y, sorted_pos, out, top_k, shared, gate)
 
 
 class FusedMoE(nn.Module):
@@ -77,18 +117,13 @@ class FusedMoE(nn.Module):
 
     def _workspace(self, T: int, device):
         if self._ws is None or self._ws_tokens < T:
-            n_pairs = T * self.top_k
-            max_rows = (n_pairs + self.E * (TILE_ROWS_PAIR - 1) + TILE_ROWS_PAIR - 1) // TILE_ROWS_PAIR * TILE_ROWS_PAIR
-            max_tiles = max_rows // TILE_ROWS
-            i32 = lambda *s: torch.zeros(*s, dtype=torch.int32, device=device)
+            max_rows = max_expert_rows(T, self.top_k, self.E)
             dt = self.w13.dtype
             self._ws = dict(
-                offsets=i32(self.E + 1), cursor=i32(self.E), tile_expert=i32(max_tiles), meta=i32(2),
+                expert_index(T, self.top_k, self.E, device),
                 a_sorted=torch.zeros(max_rows, self.hidden, dtype=dt, device=device),
                 act=torch.zeros(max_rows, self.inter_per_rank, dtype=dt, device=device),
-                y=torch.zeros(max_rows, self.hidden, dtype=dt, device=device),
-                row_scale=torch.zeros(max_rows, dtype=torch.float32, device=device),
-                sorted_pos=i32(T, self.top_k))
+                y=torch.zeros(max_rows, self.hidden, dtype=dt, device=device))
             self._ws_tokens = T
         return self._ws
 
@@ -106,20 +141,6 @@ class FusedMoE(nn.Module):
         if not x.is_cuda:
             out.copy_(reference.moe_experts(x, self.w13, self.w2, topk_w, topk_ids))
             return out
-        ws = self._workspace(T, x.device)
-        E, I = self.E, self.inter_per_rank
-        tile_rows = TILE_ROWS_PAIR if T * self.top_k >= 512 * E and self.pair_tiles else TILE_ROWS
-        n_rows = (T * self.top_k + E * (tile_rows - 1) + tile_rows - 1) // tile_rows * tile_rows
-        tile_expert = ws["tile_expert"][: n_rows // tile_rows]
-        ops.moe_align(topk_ids, E, tile_rows, ws["offsets"], ws["cursor"], tile_expert, ws["meta"])
-        sorted_pos = ws["sorted_pos"][:T]
-        ops.moe_scatter(x, topk_ids, topk_w, ws["offsets"], ws["cursor"], ws["a_sorted"], ws["row_scale"],
-                        sorted_pos, E)
-        a = ws["a_sorted"][:n_rows]
-        act = ops.gemm(a, self.w13.view(E * 2 * I, H), out=ws["act"][:n_rows], swiglu=True, tile_expert=tile_expert,
-                       num_m_tiles=ws["meta"][:1], n_per_expert=2 * I, max_ctas=max_ctas, tile_rows=tile_rows)
-        y = ops.gemm(act, self.w2.view(E * H, I), out=ws["y"][:n_rows], row_scale=ws["row_scale"],
-                     tile_expert=tile_expert, num_m_tiles=ws["meta"][:1], n_per_expert=H, max_ctas=max_ctas,
-                     tile_rows=tile_rows)
-        ops.moe_combine(y, sorted_pos, out, self.top_k)
+        run_experts(x, topk_w, topk_ids, self.w13, self.w2, self._workspace(T, x.device), out, pair_tiles=self.pair_tiles,
+                    max_ctas=max_ctas)
         return out

@@ -10,6 +10,9 @@ runner this class shares:
   model's final norm) are one kernel;
   "parallel": both sublayers read one norm of the stream, ``x += mixer(norm1(x)) + ff(norm1(x))``; the two results come
   out of one matrix product, and their addition and the next layer's norm (or the final one) are one kernel;
+  "streams": hyper-connections - several residual streams, every sublayer reads the norm of a weighted sum of them and all
+  streams are rebuilt from the old ones and the sublayer's output; that and the next sublayer's norm are one kernel (one
+  stream with weights of one is the usual pre-norm block);
 * layers may be run several times in a row with the same weights (``ModelConfig.loop``); every pass keeps its own cache
   and state, and before each pass but the first the embedding output is added to the stream;
 * a table of embeddings of token pairs may be added to the token embeddings (``ModelConfig.bigram``);
@@ -48,7 +51,7 @@ class HybridRuntime:
                                                tw_cfg.transport in ("auto", "multimem"))
         self.hidden = self.staging.tensor
         self.hidden.zero_()
-        self.residual = torch.zeros(max_tokens, w8, dtype=torch.float32, device=device)
+        self.residual = torch.zeros(max_tokens, max(1, cfg.streams) * w8, dtype=torch.float32, device=device)
         self.sublayer = torch.zeros(max_tokens, w8, dtype=cfg.dtype, device=device)
         # the embedding output, for layers that run again
         self.first = torch.zeros(max_tokens, w8, dtype=torch.float32, device=device) if cfg.loop else None
@@ -57,7 +60,9 @@ class HybridRuntime:
         self.sm_count = torch.cuda.get_device_properties(device).multi_processor_count if device.type == "cuda" else 0
         # context tokens whose keys and values a step may expand
         self.context_rows = max(max_tokens, min(cfg.max_model_len, 32768))
+        self.max_positions = cfg.max_model_len
         self.rope_tables: dict = {}
+        self.tables: dict = {}              # bookkeeping that layers share, by the layers' own keys
         self._buffers: dict[tuple, torch.Tensor] = {}
 
     def buffer(self, name: str, rows: int, cols: int) -> torch.Tensor:
@@ -79,7 +84,7 @@ class HybridLayer(nn.Module):
         if kind not in MIXERS:
             raise ValueError(f"unknown mixer {kind!r} (known: {sorted(MIXERS)})")
         W, eps, dt = cfg.hidden_size, cfg.rms_norm_eps, cfg.dtype
-        self.mixer = MIXERS[kind](spec["mixer"], W, eps, dtype=dt, device=device, max_positions=cfg.max_model_len)
+        self.mixer = MIXERS[kind](spec["mixer"], W, eps, dtype=dt, device=device, **spec.get("options", {}))
         self.norm1_w = nn.Parameter(torch.ones(W, dtype=dt, device=device), requires_grad=False)
         self.mlp = self.norm2_w = None
         mlp = spec.get("mlp")
@@ -110,8 +115,7 @@ class ParallelLayer(nn.Module):
         if mlp is not None and mlp["kind"] != "gated":
             raise ValueError(f"unknown feed-forward {mlp['kind']!r} in a parallel block")
         dt = cfg.dtype
-        self.mixer = SumMixer(spec["mixer"], cfg.hidden_size, cfg.rms_norm_eps, dtype=dt, device=device,
-                              max_positions=cfg.max_model_len, mlp=mlp)
+        self.mixer = SumMixer(spec["mixer"], cfg.hidden_size, cfg.rms_norm_eps, dtype=dt, device=device, mlp=mlp)
         self.norm1_w = nn.Parameter(torch.ones(cfg.hidden_size, dtype=dt, device=device), requires_grad=False)
         self.mlp = None                     # part of the mixer
 
@@ -123,7 +127,28 @@ class ParallelLayer(nn.Module):
         return out
 
 
-BLOCKS = {"output_norm": HybridLayer, "parallel": ParallelLayer}
+class StreamLayer(HybridLayer):
+    """Both sublayers of a layer read a norm of a weighted sum of the streams (``hops.streams_step``); ``hc[q]`` are the
+    coefficients around sublayer q."""
+
+    def __init__(self, spec: dict, cfg: ModelConfig, *, device):
+        super().__init__(spec, cfg, device=device)
+        S = max(1, cfg.streams)
+        self.learned = cfg.streams > 0
+        init = {"in": torch.ones(S), "out": torch.ones(S), "mix": torch.eye(S)}
+        self.hc = nn.ModuleList(
+            nn.ParameterDict({k: nn.Parameter(v.to(device=device, dtype=torch.float32, copy=True), requires_grad=False)
+                              for k, v in init.items()}) for _ in range(1 if self.mlp is None else 2))
+
+    def tensor_targets(self) -> dict:
+        out = super().tensor_targets()
+        if self.learned:
+            for q, hc in enumerate(self.hc):
+                out.update({f"hc{q + 1}.{k}": (tuple(v.shape), v.data.copy_) for k, v in hc.items()})
+        return out
+
+
+BLOCKS = {"output_norm": HybridLayer, "parallel": ParallelLayer, "streams": StreamLayer}
 
 
 def layer_runs(num_layers: int, loop: Optional[dict]) -> list[tuple[int, bool]]:
@@ -158,7 +183,10 @@ class HybridDecoder(nn.Module):
             raise ValueError("a hybrid decoder needs the list of its layers")
         self.cfg = cfg
         dt, W = cfg.dtype, cfg.hidden_size
-        self.embed_w = nn.Parameter(torch.zeros(cfg.vocab_size, pad8(W), dtype=dt, device=device), requires_grad=False)
+        self.head = PaddedLinear(W, cfg.vocab_size, dtype=dt, device=device)
+        table = (self.head.weight.data[:cfg.vocab_size] if cfg.tie_word_embeddings
+                 else torch.zeros(cfg.vocab_size, pad8(W), dtype=dt, device=device))
+        self.embed_w = nn.Parameter(table, requires_grad=False)
         self.bigram_w = None
         if cfg.bigram:                      # one row per bucket, and one for tokens without a token before them
             self.bigram_w = nn.Parameter(torch.zeros(int(cfg.bigram["buckets"]) + 1, pad8(W), dtype=dt, device=device),
@@ -169,7 +197,6 @@ class HybridDecoder(nn.Module):
             raise ValueError("loops and pair embeddings are built for parallel blocks")
         self.kept = [self.layers[i].mixer.new_kept() for i, _ in self.runs]
         self.final_norm_w = nn.Parameter(torch.ones(W, dtype=dt, device=device), requires_grad=False)
-        self.head = PaddedLinear(W, cfg.vocab_size, dtype=dt, device=device)
         self.rt: Optional[HybridRuntime] = None
         mixers = [l.mixer for l in self.layers]
         latent = [m for m in mixers if isinstance(m, LatentAttention)]
@@ -177,6 +204,8 @@ class HybridDecoder(nn.Module):
         # long runs may go to query tiles: every attention of the model can take them; with latent attention their
         # contexts are expanded into a workspace first
         self.expand = bool(latent)
+        # the keys an expanded run's first token sees: all of them, or the widest window's
+        self.expand_window = 0 if any(not m.window for m in latent) else max((m.window for m in latent), default=0)
         self.tiles = (bool(latent or grouped) and all(m.expandable for m in latent) and all(m.tileable for m in grouped))
         self.recurrent = any(m.recurrent for m in mixers)
 
@@ -193,6 +222,8 @@ class HybridDecoder(nn.Module):
                     for name, cols in m.context_workspaces():
                         self.rt.buffer(name, self.rt.context_rows, cols)
             m.bind_runtime(self.rt)
+            if layer.mlp is not None:
+                layer.mlp.bind_runtime(self.rt)
         return self.rt
 
     def kv_cache_bytes_per_block(self, block_size: int) -> int:
@@ -234,14 +265,18 @@ class HybridDecoder(nn.Module):
                 extra.update(state_slots=np.asarray(state_slots, dtype=np.int32), scan_seqs=rows, chunk_seqs=rows[:0])
             return plan, extra, {}
         n = np.asarray(q_lens)
-        tiled, ctx_rows = [], 0
+        tiled, ctx_rows, first = [], 0, {}
         if self.tiles and not self.expand:
             tiled = [b for b, ql in enumerate(q_lens) if ql >= PREFILL_MIN_Q]
         elif self.tiles:
             for b, (ql, kv) in enumerate(zip(q_lens, kv_lens)):
-                if (ql >= 64 or (ql >= PREFILL_MIN_Q and kv <= 2 * ql)) and ctx_rows + kv <= self.rt.context_rows:
+                # whole key tiles from the first visible key's on
+                lo = max(0, kv - ql - self.expand_window + 1) // 128 * 128 if self.expand_window else 0
+                rows = kv - lo
+                if (ql >= 64 or (ql >= PREFILL_MIN_Q and rows <= 2 * ql)) and ctx_rows + rows <= self.rt.context_rows:
                     tiled.append(b)
-                    ctx_rows += kv
+                    first[b] = lo
+                    ctx_rows += rows
         row_seq = np.repeat(np.arange(B, dtype=np.int32), n)
         start = np.cumsum(n) - n
         tok_row = np.flatnonzero(~np.isin(row_seq, tiled)).astype(np.int32)
@@ -255,11 +290,12 @@ class HybridDecoder(nn.Module):
         extra["row_seq"] = row_seq
         if tiled and self.expand:
             cu = np.zeros(len(tiled) + 1, dtype=np.int32)
-            np.cumsum([kv_lens[b] for b in tiled], out=cu[1:])
+            lo = np.asarray([first[b] for b in tiled], dtype=np.int32)
+            np.cumsum([kv_lens[b] - first[b] for b in tiled], out=cu[1:])
             begin = np.full(B, -1, dtype=np.int32)
-            begin[tiled] = cu[:-1]
-            extra.update(ctx_seqs=np.asarray(tiled, dtype=np.int32), ctx_cu=cu, ctx_begin=begin)
-            host = {"ctx_rows": int(cu[-1]), "ctx_max": max(kv_lens[b] for b in tiled)}
+            begin[tiled] = cu[:-1] - lo              # the workspace row of key 0, were it there
+            extra.update(ctx_seqs=np.asarray(tiled, dtype=np.int32), ctx_cu=cu, ctx_begin=begin, ctx_first=lo)
+            host = {"ctx_rows": int(cu[-1]), "ctx_max": max(kv_lens[b] - first[b] for b in tiled)}
         if self.recurrent:
             long = n >= hops.CHUNK_MIN_TOKENS
             extra.update(state_slots=np.asarray(state_slots, dtype=np.int32),
@@ -279,6 +315,9 @@ class HybridDecoder(nn.Module):
         rt, cfg, meta = self.rt, self.cfg, step.meta
         T, eps = step.plan.num_tokens, cfg.rms_norm_eps
         x32, xa, y = rt.residual[:T], rt.hidden[:T], rt.sublayer[:T]
+        if cfg.block == "streams":
+            self._forward_streams(step, x32.view(T, max(1, cfg.streams), -1), xa, y)
+            return xa
         if cfg.block == "parallel":
             first = rt.first[:T] if rt.first is not None else None
             hops.embed_norm(step.input_ids, self.embed_w, self.bigram_w, cfg.bigram, meta, x32, first,
@@ -300,6 +339,20 @@ class HybridDecoder(nn.Module):
                 hops.postnorm_add_(y, x32, layer.norm2_w, eps, xa, self.final_norm_w if layer is last else None)
         return xa
 
+    def _forward_streams(self, step, x: torch.Tensor, xa: torch.Tensor, y: torch.Tensor) -> None:
+        rt, cfg, meta = self.rt, self.cfg, step.meta
+        eps, off = cfg.rms_norm_eps, cfg.norm_offset
+        first = self.layers[0]
+        hops.embed_streams(step.input_ids, self.embed_w, x, first.hc[0]["in"], first.norm1_w, off, eps, xa)
+        for n, (layer, kept) in enumerate(zip(self.layers, self.kept)):
+            nxt = self.layers[n + 1] if n + 1 < len(self.layers) else None
+            behind = (None, self.final_norm_w) if nxt is None else (nxt.hc[0]["in"], nxt.norm1_w)
+            layer.mixer(xa, meta, rt, y, kept)
+            if layer.mlp is not None:
+                hops.streams_step(y, x, layer.hc[0], cfg.residual_mult, layer.hc[1]["in"], layer.norm2_w, off, eps, xa)
+                layer.mlp(xa, rt, y)
+            hops.streams_step(y, x, layer.hc[-1], cfg.residual_mult, *behind, off, eps, xa)
+
     @torch.inference_mode()
     def compute_logits(self, hidden_rows: torch.Tensor) -> torch.Tensor:
         """fp32 logits ``[rows, vocab]``."""
@@ -309,8 +362,9 @@ class HybridDecoder(nn.Module):
     def tensor_targets(self) -> dict:
         V, W = self.cfg.vocab_size, self.cfg.hidden_size
         out = {"embed": ((V, W), lambda t: self.embed_w.data[:, :W].copy_(t)),
-               "final.norm": ((W,), self.final_norm_w.data.copy_),
-               "head": ((V, W), lambda t: self.head.load_rows(t, 0))}
+               "final.norm": ((W,), self.final_norm_w.data.copy_)}
+        if not self.cfg.tie_word_embeddings:
+            out["head"] = ((V, W), lambda t: self.head.load_rows(t, 0))
         if self.bigram_w is not None:
             out["bigram"] = ((self.bigram_w.shape[0], W), lambda t: self.bigram_w.data[:, :W].copy_(t))
         for i, layer in enumerate(self.layers):
@@ -349,8 +403,14 @@ class HybridDecoder(nn.Module):
         def fill(name, shape):
             t = torch.empty(shape, dtype=torch.float32, device=dev)
             leaf = name.split(".mix.")[-1]
-            if name.endswith(("norm", "norm1", "norm2")) or leaf == "D":
+            if name.endswith(("norm1", "norm2", "final.norm")):
+                return t.fill_(1.0 - self.cfg.norm_offset)
+            if name.endswith("norm") or leaf == "D":
                 return t.fill_(1.0)
+            if ".hc" in name:
+                return t.copy_(torch.eye(shape[0]) if leaf.endswith("mix") else torch.full(shape, 1.0 / shape[0]))
+            if leaf == "sink" or name.endswith(".correction"):
+                return t.zero_()
             if leaf == "A_log":
                 return t.uniform_(1.0, 16.0, generator=g).log_()
             if leaf == "dt_bias":

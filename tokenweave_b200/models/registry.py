@@ -11,13 +11,14 @@ def get_model_class(architecture: str):
     from .llama import LlamaForCausalLM
     from .mistral import MistralForCausalLM
     from .mixtral import MixtralForCausalLM
+    from .netezen import NetezenForCausalLM
     from .phi3 import Phi3ForCausalLM
     from .qwen2 import Qwen2ForCausalLM
     from .qwen3 import Qwen3ForCausalLM
     from .sidisun import SidisunForCausalLM
     table = {"llama": LlamaForCausalLM, "qwen2": Qwen2ForCausalLM, "mixtral": MixtralForCausalLM,
              "qwen3": Qwen3ForCausalLM, "mistral": MistralForCausalLM, "phi3": Phi3ForCausalLM,
-             "sidisun": SidisunForCausalLM, "kebopel": KebopelForCausalLM}
+             "sidisun": SidisunForCausalLM, "kebopel": KebopelForCausalLM, "netezen": NetezenForCausalLM}
     if architecture not in table:
         raise ValueError(f"unsupported architecture {architecture!r} (supported: {sorted(table)})")
     return table[architecture]
@@ -25,7 +26,7 @@ def get_model_class(architecture: str):
 
 def load_config_readers() -> None:
     """Imports the modules that register a reader for their own ``config.json`` layout."""
-    from . import kebopel, sidisun  # noqa: F401
+    from . import kebopel, netezen, sidisun  # noqa: F401
 
 
 def build_model(config: EngineConfig, device: torch.device, embedding_parallel: bool = False):

@@ -81,14 +81,19 @@ def _row_stride(t: torch.Tensor) -> int:
 
 
 # ---------------------------------------------------------------------------------------------
+COL_ACTS = {"silu": 1, "relu2": 2}
+
+
 def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *,
          bias: Optional[torch.Tensor] = None, row_scale: Optional[torch.Tensor] = None, swiglu: bool = False,
-         act: str = "silu", silu_cols: Optional[tuple[int, int]] = None, max_ctas: int = 0,
+         act: "str | tuple" = "silu", col_act: Optional[tuple[str, int, int]] = None, max_ctas: int = 0,
          tile_expert: Optional[torch.Tensor] = None,
          num_m_tiles: Optional[torch.Tensor] = None, n_per_expert: int = 0, tile_rows: int = 128) -> torch.Tensor:
     """``out = a @ w.T`` (+bias, *row_scale); with ``swiglu`` the weight is ``[gate; up]`` and the
-    output is ``act(a@gate.T) * (a@up.T)``, ``act`` "silu" or "gelu_tanh". ``silu_cols`` = (begin, end): silu on these
-    columns of a plain product (behind the bias). Grouped mode (``tile_expert`` given): every ``tile_rows``-row
+    output is ``act(a@gate.T) * (a@up.T)``, ``act`` "silu", "gelu_tanh" or ("clamped", limit, alpha):
+    ``g sigmoid(alpha g) (u + 1)`` with ``g = min(a@gate.T, limit)`` and ``u = a@up.T`` inside ``[-limit, limit]``.
+    ``col_act`` = ("silu" or "relu2", begin, end): that activation on these columns of a plain product (behind the bias;
+    relu2: the square of relu). Grouped mode (``tile_expert`` given): every ``tile_rows``-row
     tile of ``a`` multiplies the weight block of its expert, ``w`` being ``[E * n_per_expert, K]``;
     ``tile_rows`` is 128 (single-CTA tiles) or 256 (experts padded to 256 rows: the groups run on CTA pairs)."""
     M, K = a.shape
@@ -98,7 +103,7 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
     if out is None:
         out = torch.empty(M, N, dtype=a.dtype, device=a.device)
     if not a.is_cuda:
-        if act != "silu" or silu_cols is not None:
+        if act != "silu" or col_act is not None:
             raise NotImplementedError("these epilogues on CPU go through ops.reference_hybrid")
         if tile_expert is not None:
             raise NotImplementedError("grouped GEMM on CPU goes through reference.moe_experts")
@@ -106,27 +111,43 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
         out.copy_(res)
         return out
     if a.dtype == torch.float32:
-        if swiglu or row_scale is not None or tile_expert is not None:
-            raise NotImplementedError("the fp32 matrix product is plain: no SwiGLU, row scales or groups")
+        if swiglu or col_act is not None or (tile_expert is None and row_scale is not None):
+            raise NotImplementedError("the fp32 matrix product has no activations, and row scales with groups only")
         if w.dtype != torch.float32 or out.dtype != torch.float32:
             raise TypeError("the fp32 matrix product takes fp32 operands")
+        if tile_expert is not None:
+            _native.call("tw_gemm_f32_grouped", a.data_ptr(), _row_stride(a), w.data_ptr(), _row_stride(w), out.data_ptr(),
+                         _row_stride(out), M, N, K, _p(tile_expert), _p(num_m_tiles), tile_rows, per_expert, _p(row_scale),
+                         _stream())
+            return out
         _native.call("tw_gemm_f32", a.data_ptr(), _row_stride(a), w.data_ptr(), _row_stride(w), out.data_ptr(),
                      _row_stride(out), _p(bias), M, N, K, _stream())
         return out
     _check_bf16(a, w, out, bias)
-    if silu_cols is not None:
+    if col_act is not None:
         if swiglu or row_scale is not None or tile_expert is not None:
-            raise ValueError("silu on a range of columns goes with a plain product")
-        _native.call("tw_gemm_bf16_silu", a.data_ptr(), _row_stride(a), w.data_ptr(), _row_stride(w), out.data_ptr(),
-                     _row_stride(out), _p(bias), M, N, K, int(silu_cols[0]), int(silu_cols[1]), max_ctas,
+            raise ValueError("an activation on a range of columns goes with a plain product")
+        _native.call("tw_gemm_bf16_act", a.data_ptr(), _row_stride(a), w.data_ptr(), _row_stride(w), out.data_ptr(),
+                     _row_stride(out), _p(bias), M, N, K, COL_ACTS[col_act[0]], int(col_act[1]), int(col_act[2]), max_ctas,
                      gemm_table.lookup(M, N, K, False, max_ctas), status_word(a.device).data_ptr(), _stream(),
-                     tag=f"[{M}x{N}x{K}+silu]" if _native._timing is not None else "")
+                     tag=f"[{M}x{N}x{K}+{col_act[0]}]" if _native._timing is not None else "")
+        return out
+    if swiglu and not isinstance(act, str):
+        kind, limit, alpha = act
+        if kind != "clamped" or bias is not None or row_scale is not None:
+            raise ValueError(f"unknown gated product {act!r}, or a bias or row scales with it")
+        grouped = tile_expert is not None
+        _native.call("tw_gemm_bf16_clamped", a.data_ptr(), _row_stride(a), w.data_ptr(), _row_stride(w), rows_b,
+                     out.data_ptr(), _row_stride(out), M, N, K, float(limit), float(alpha), per_expert // 2, _p(tile_expert),
+                     _p(num_m_tiles), per_expert, tile_rows, max_ctas,
+                     0 if grouped else gemm_table.lookup(M, N, K, True, max_ctas), status_word(a.device).data_ptr(),
+                     _stream(), tag=f"[{'grouped ' if grouped else ''}{M}x{N}x{K}+clamped]" if _native._timing is not None else "")
         return out
     if tile_expert is not None and tile_rows == 256:
         if bias is not None:
             raise ValueError("the grouped GEMM has no bias")
         _native.call("tw_gemm_bf16_grouped256", a.data_ptr(), _row_stride(a), w.data_ptr(), _row_stride(w), rows_b,
-                     out.data_ptr(), _row_stride(out), _p(row_scale), M, N, K, int(swiglu),
+                     out.data_ptr(), _row_stride(out), _p(row_scale), M, N, K, {"silu": 1, "gelu_tanh": 2}[act] if swiglu else 0,
                      per_expert // 2 if swiglu else 0, _p(tile_expert), _p(num_m_tiles), per_expert, max_ctas,
                      status_word(a.device).data_ptr(), _stream(),
                      tag=f"[grouped {M}x{N}x{K}{'+swiglu' if swiglu else ''}]" if _native._timing is not None else "")
@@ -681,6 +702,26 @@ def moe_router(x: torch.Tensor, gate_w: torch.Tensor, topk: int, renormalize: bo
     return w, ids, logits
 
 
+def moe_route(x: torch.Tensor, w: torch.Tensor, experts: int, topk: int, correction: Optional[torch.Tensor] = None,
+              sum_eps: float = 0.0):
+    """The general router, bf16 or fp32. ``w`` [experts + gates, >= width]: a row per expert, then a row per gate. Scores
+    are the softmax over all experts; the ``topk`` with the largest score + ``correction`` (fp32 [experts]) are chosen, their
+    weights are the scores without it over (their sum + ``sum_eps``). Returns (weights fp32 [T, k], ids int32 [T, k],
+    sigmoid of the gate rows fp32 [T, gates])."""
+    if not x.is_cuda:
+        return reference.moe_route(x, w, experts, topk, correction, sum_eps)
+    if x.dtype != w.dtype or x.dtype not in (torch.bfloat16, torch.float32):
+        raise TypeError(f"expected rows and router of one type, bfloat16 or float32, got {x.dtype} and {w.dtype}")
+    T, H = x.shape
+    gates = w.shape[0] - experts
+    ids = torch.empty(T, topk, dtype=torch.int32, device=x.device)
+    wts, gate = (torch.empty(T, n, dtype=torch.float32, device=x.device) for n in (topk, gates))
+    _native.call("tw_moe_route", x.data_ptr(), _row_stride(x), w.data_ptr(), _row_stride(w), _p(correction), wts.data_ptr(),
+                 ids.data_ptr(), gate.data_ptr() if gates else None, T, H, experts, gates, topk, float(sum_eps),
+                 0 if x.dtype == torch.bfloat16 else 1, _stream())
+    return wts, ids, gate
+
+
 def moe_align(topk_ids: torch.Tensor, num_experts: int, tile_rows: int, expert_offsets: torch.Tensor,
               expert_cursor: torch.Tensor, tile_expert: torch.Tensor, meta: torch.Tensor) -> None:
     """Counting sort bookkeeping: padded expert offsets, expert per row tile, meta = [tiles, padded rows]."""
@@ -696,10 +737,13 @@ def moe_scatter(x: torch.Tensor, topk_ids: torch.Tensor, topk_w: torch.Tensor, e
     topk = topk_ids.shape[1]
     _native.call("tw_moe_scatter", x.data_ptr(), _row_stride(x), topk_ids.data_ptr(), topk_w.data_ptr(),
                  expert_offsets.data_ptr(), expert_cursor.data_ptr(), a_sorted.data_ptr(), row_scale.data_ptr(),
-                 sorted_pos.data_ptr(), T * topk, topk, H, num_experts, _stream())
+                 sorted_pos.data_ptr(), T * topk, topk, H, num_experts, int(x.dtype == torch.float32), _stream())
 
 
-def moe_combine(y_sorted: torch.Tensor, sorted_pos: torch.Tensor, out: torch.Tensor, topk: int) -> None:
+def moe_combine(y_sorted: torch.Tensor, sorted_pos: torch.Tensor, out: torch.Tensor, topk: int,
+                shared: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+    """``out = sum over a token's experts`` of their weighted rows, ``+ gate * shared`` (one gate per token)."""
     T, H = out.shape
-    _native.call("tw_moe_combine", y_sorted.data_ptr(), sorted_pos.data_ptr(), out.data_ptr(), _row_stride(out),
-                 T, topk, H, _stream())
+    _native.call("tw_moe_combine", y_sorted.data_ptr(), sorted_pos.data_ptr(), _p(shared),
+                 _row_stride(shared) if shared is not None else 0, _p(gate), out.data_ptr(), _row_stride(out),
+                 T, topk, H, int(out.dtype == torch.float32), _stream())

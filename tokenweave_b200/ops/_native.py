@@ -51,8 +51,9 @@ _SIGNATURES = {
                                      i32, vp, vp, i32, vp, vp],
     "tw_moe_router": [vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp],
     "tw_moe_align": [vp, i32, i32, i32, vp, vp, vp, i32, vp, vp],
-    "tw_moe_scatter": [vp, ll, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, vp],
-    "tw_moe_combine": [vp, vp, vp, ll, i32, i32, i32, vp],
+    "tw_moe_scatter": [vp, ll, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp],
+    "tw_moe_combine": [vp, vp, vp, ll, vp, vp, ll, i32, i32, i32, i32, vp],
+    "tw_moe_route": [vp, ll, vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp],
     "tw_fused_rs_norm_ag": [vp, vp, vp, i32, i32, i32, u64, vp, ll, vp, ll, vp, i32, i32, f32, i32, i32, i32,
                             vp],
     "tw_collective": [vp, vp, vp, i32, i32, i32, u64, vp, ll, ll, i32, i32, vp],
@@ -63,6 +64,9 @@ _SIGNATURES = {
     "tw_ag_gemm": [vp, vp, ll, ll, vp, ll, vp, i32, i32, i32, i32, i32, vp, vp, vp, vp, i32, i32, u64, vp, ll, i32, i32,
                    i32, vp],
     "tw_gemm_f32": [vp, ll, vp, ll, vp, ll, vp, i32, i32, i32, vp],
+    "tw_gemm_f32_grouped": [vp, ll, vp, ll, vp, ll, i32, i32, i32, vp, vp, i32, i32, vp, vp],
+    "tw_embed_streams": [vp, vp, ll, i32, vp, ll, ll, i32, vp, vp, f32, vp, ll, i32, i32, f32, i32, vp],
+    "tw_streams_step": [vp, ll, vp, ll, ll, i32, vp, vp, f32, vp, i32, vp, f32, vp, ll, i32, i32, f32, i32, vp],
     "tw_embed_residual": [vp, vp, ll, vp, ll, vp, ll, i32, i32, i32, i32, vp],
     "tw_postnorm_add": [vp, ll, vp, ll, vp, vp, ll, vp, i32, i32, f32, i32, vp],
     "tw_polynorm": [vp, ll, vp, vp, ll, i32, i32, f32, i32, vp],
@@ -70,25 +74,27 @@ _SIGNATURES = {
     "tw_embed_norm": [vp, vp, ll, i32, vp, ll, ll, ll, ll, vp, vp, vp, vp, ll, vp, ll, vp, vp, ll, i32, i32, f32, i32, vp],
     "tw_add_prenorm": [vp, ll, vp, ll, vp, ll, vp, vp, ll, i32, i32, f32, i32, vp],
     "tw_norm_gate": [vp, ll, vp, ll, vp, vp, ll, i32, i32, i32, f32, f32, i32, vp],
-    "tw_silu_cols": [vp, ll, i32, i32, i32, vp],
-    "tw_glu": [vp, ll, vp, ll, i32, i32, i32, i32, vp],
+    "tw_act_cols": [vp, ll, i32, i32, i32, i32, vp],
+    "tw_glu": [vp, ll, vp, ll, i32, i32, i32, f32, f32, i32, vp],
     "tw_qkv_prep": [vp, ll, i32, i32, i32, i32, i32, i32, vp, ll, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, i32, i32,
-                    i32, vp, vp, f32, f32, i32, i32, vp],
-    "tw_attn_rows": [vp, ll, vp, vp, i32, vp, ll, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, f32, vp, i32, f32, i32, vp],
+                    i32, vp, vp, f32, f32, i32, vp, i32, i32, vp],
+    "tw_attn_rows": [vp, ll, vp, vp, i32, vp, ll, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, f32, vp, i32, f32, i32, i32,
+                     i32, vp],
     "tw_attn_prefill_grouped": [vp, ll, i32, vp, vp, i32, i32, vp, ll, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32,
-                                f32, vp, i32, f32, vp, vp],
+                                f32, vp, i32, f32, i32, i32, vp, vp],
     "tw_attn_decode_grouped": [vp, ll, vp, vp, i32, i32, vp, ll, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, f32, vp, i32,
-                               f32, i32, vp, vp, vp, vp],
-    "tw_gemm_bf16_silu": [vp, ll, vp, ll, vp, ll, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp],
+                               f32, i32, i32, i32, vp, vp, vp, vp],
+    "tw_gemm_bf16_act": [vp, ll, vp, ll, vp, ll, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
+    "tw_gemm_bf16_clamped": [vp, ll, vp, ll, ll, vp, ll, i32, i32, i32, f32, f32, i32, vp, vp, i32, i32, i32, i32, vp, vp],
     "tw_latent_prep": [vp, ll, i32, i32, vp, vp, ll, i32, i32, vp, i32, i32, vp, vp, vp, vp, i32, i32, f32, i32, vp],
     "tw_rope_tail": [vp, ll, i32, i32, i32, i32, i32, vp, vp, i32, vp],
     "tw_latent_query": [vp, ll, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, vp],
     "tw_head_gemm": [vp, ll, i32, vp, vp, ll, i32, vp, ll, i32, vp, vp, ll, i32, i32, i32, i32, i32, i32, vp],
-    "tw_latent_attn": [vp, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, f32, i32, vp],
-    "tw_latent_decode": [vp, vp, i32, i32, vp, vp, i32, vp, i32, vp, i32, i32, i32, f32, i32, vp, vp, vp, vp],
+    "tw_latent_attn": [vp, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, f32, i32, vp, i32, vp],
+    "tw_latent_decode": [vp, vp, i32, i32, vp, vp, i32, vp, i32, vp, i32, i32, i32, f32, i32, vp, i32, vp, vp, vp, vp],
     "tw_latent_prefill": [vp, ll, i32, vp, ll, vp, ll, i32, vp, vp, ll, vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, i32,
-                          f32, vp, vp],
-    "tw_latent_gather": [vp, vp, vp, vp, i32, i32, vp, i32, i32, i32, vp],
+                          f32, i32, vp, vp, vp],
+    "tw_latent_gather": [vp, vp, vp, vp, vp, i32, i32, vp, i32, i32, i32, vp],
     "tw_causal_conv": [vp, ll, vp, vp, vp, vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp],
     "tw_conv_state": [vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, vp],
     "tw_decay_scan": [vp, ll, vp, vp, vp, ll, vp, i32, vp, vp, vp, i32, i32, i32, i32, vp],

@@ -1,8 +1,8 @@
 """Operators of models whose layers mix attention and recurrences and whose residual stream is fp32: latent attention
 over a paged latent cache, the state-space (Mamba-2) recurrence with its convolution, the norm of a sublayer's output
 added to the residual, and the polynomial-norm activation; for blocks whose sublayers read one norm of the stream,
-grouped attention with its options (query and key norms, short convolution, query temperature, distance bias, sink),
-lightning attention, embeddings with token pairs, and the fused projections.
+grouped attention with its options (query and key norms, short convolution, rotation, query temperature, distance bias,
+sink, sliding window), lightning attention, embeddings with token pairs, and the fused projections; hyper-connections.
 
 Like the other operators, CUDA tensors (bf16 or fp32) go to the kernels of ``_C.so`` and CPU tensors to plain PyTorch
 (:mod:`.reference_hybrid`). ``meta`` below is the step's :class:`~tokenweave_b200.layers.attention.AttentionMetadata`.
@@ -14,7 +14,7 @@ from typing import Optional
 import torch
 
 from . import _native, reference_hybrid as ref
-from . import _p, _row_stride, _stream, decode_splits_tc, gemm, status_word
+from . import COL_ACTS, _p, _row_stride, _stream, decode_splits_tc, gemm, status_word
 
 
 def _dt(*ts: Optional[torch.Tensor]) -> int:
@@ -72,6 +72,37 @@ def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, gro
     return out
 
 
+# ---- hyper-connections: several residual streams ---------------------------------------------------------------
+# ``x``: fp32 [T, streams, padded width]; ``hc``: a sublayer's coefficients {"in" [S], "out" [S], "mix" [S, S] (from, to)}
+# in fp32; norm weights are stored around ``offset``.
+def embed_streams(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, hc_in: torch.Tensor, weight: torch.Tensor,
+                  offset: float, eps: float, xa: torch.Tensor) -> None:
+    """Every stream ``= table[ids]``; ``xa = rmsnorm(sum_s in[s] x_s) * (offset + weight)``."""
+    if not table.is_cuda:
+        ref.embed_streams(ids, table, x, hc_in, weight, offset, eps, xa)
+        return
+    assert ids.dtype == torch.int32 and x.dtype == hc_in.dtype == torch.float32 and x.stride(2) == 1
+    _native.call("tw_embed_streams", ids.data_ptr(), table.data_ptr(), _row_stride(table), table.shape[0], x.data_ptr(),
+                 x.stride(0), x.stride(1), x.shape[1], hc_in.data_ptr(), weight.data_ptr(), float(offset), xa.data_ptr(),
+                 _row_stride(xa), ids.shape[0], weight.numel(), float(eps), _dt(table, weight, xa), _stream())
+
+
+def streams_step(y: torch.Tensor, x: torch.Tensor, hc: dict, mult: float, next_in: Optional[torch.Tensor],
+                 weight: torch.Tensor, offset: float, eps: float, xa: torch.Tensor) -> None:
+    """``x_t <- sum_s mix[s, t] x_s + mult out[t] y`` (from the old streams), then the next sublayer's input
+    ``xa = rmsnorm(sum_s next_in[s] x_s) * (offset + weight)``. ``next_in`` None: behind the last sublayer - the norm of the
+    streams' sum, the streams themselves are not stored."""
+    if not y.is_cuda:
+        ref.streams_step(y, x, hc, mult, next_in, weight, offset, eps, xa)
+        return
+    assert x.dtype == hc["mix"].dtype == hc["out"].dtype == torch.float32 and x.stride(2) == 1
+    assert next_in is None or next_in.dtype == torch.float32
+    _native.call("tw_streams_step", y.data_ptr(), _row_stride(y), x.data_ptr(), x.stride(0), x.stride(1), x.shape[1],
+                 hc["mix"].data_ptr(), hc["out"].data_ptr(), float(mult), _p(next_in), int(next_in is not None),
+                 weight.data_ptr(), float(offset), xa.data_ptr(), _row_stride(xa), y.shape[0], weight.numel(), float(eps),
+                 _dt(y, weight, xa), _stream())
+
+
 # ---- latent attention -----------------------------------------------------------------------------------------
 def latent_row(kv_rank: int, rot: int) -> int:
     """Elements of a latent cache row: the latent and the rotated key part, each padded to eight."""
@@ -117,14 +148,20 @@ def latent_absorb(q: torch.Tensor, rows: torch.Tensor, w_ukt: torch.Tensor, head
                  dim, rot, rot_dims, kv_rank, row, cos_sin.data_ptr(), positions.data_ptr(), dt, _stream())
 
 
+def _key_tiles(max_kv_len: int, window: int = 0, keep: int = 0) -> int:
+    """Most 128-key tiles that hold visible keys of one row."""
+    tiles = (max_kv_len + 127) // 128
+    return min(tiles, (window + 126) // 128 + 1 + (keep + 127) // 128) if window else tiles
+
+
 def latent_decode_plan(n: int, heads: int, row: int, kv_rank: int, page: int, dtype: torch.dtype, max_kv_len: int,
-                       sm_count: int = 148) -> tuple[str, int]:
+                       sm_count: int = 148, window: int = 0) -> tuple[str, int]:
     """(kernel, key splits) of an absorbed attention launch: "tc" (tensor cores: bf16, cache rows of up to 640 elements
     with a latent of up to 512) or "simt" (fp32 and every other size)."""
     if dtype != torch.bfloat16 or row > 640 or kv_rank > 512 or page < 8 or page > 128 or 128 % page:
         return "simt", 1
     blocks = (heads + 15) // 16 if heads <= 16 else (heads + 31) // 32
-    return "tc", decode_splits_tc(n * blocks, (max_kv_len + 127) // 128, sm_count)
+    return "tc", decode_splits_tc(n * blocks, _key_tiles(max_kv_len, window), sm_count)
 
 
 _partials: dict[tuple, tuple[torch.Tensor, torch.Tensor]] = {}
@@ -144,28 +181,32 @@ def _partial_buffers(device, count: int, width: int) -> tuple[torch.Tensor, torc
 
 def latent_attention(qa: torch.Tensor, cache: torch.Tensor, tok_seq: torch.Tensor, tok_kvlen: torch.Tensor, n: int,
                      block_table: torch.Tensor, kv_rank: int, scale: float, out: torch.Tensor, max_kv_len: int,
-                     sm_count: int = 148, kernel: Optional[str] = None) -> None:
+                     sm_count: int = 148, kernel: Optional[str] = None, window: int = 0,
+                     sink: Optional[torch.Tensor] = None) -> None:
     """Causal attention of ``n`` absorbed query rows over the paged latent cache; ``out`` [n, heads, kv_rank].
-    ``kernel``: force one of :func:`latent_decode_plan`'s kernels (tests)."""
+    ``window`` > 0: a row sees the last ``window`` keys, itself among them; ``sink`` (fp32 [heads]): exp(sink) joins the
+    denominator. ``kernel``: force one of :func:`latent_decode_plan`'s kernels (tests)."""
     if n == 0:
         return
     heads, row, page = qa.shape[1], qa.shape[2], cache.shape[1]
     if not qa.is_cuda:
-        out[:n] = ref.latent_attention(qa[:n], cache, tok_seq, tok_kvlen, block_table, kv_rank, scale)
+        out[:n] = ref.latent_attention(qa[:n], cache, tok_seq, tok_kvlen, block_table, kv_rank, scale, window, sink)
         return
     dt = _dt(qa, cache, out)
-    plan, splits = latent_decode_plan(n, heads, row, kv_rank, page, qa.dtype, max_kv_len, sm_count)
+    assert sink is None or sink.dtype == torch.float32
+    plan, splits = latent_decode_plan(n, heads, row, kv_rank, page, qa.dtype, max_kv_len, sm_count, window)
     if (kernel or plan) == "tc":
         po = pm = None
         if splits > 1:
             po, pm = _partial_buffers(qa.device, n * heads * splits, kv_rank)
         _native.call("tw_latent_decode", qa.data_ptr(), cache.data_ptr(), cache.shape[0], page, tok_seq.data_ptr(),
                      tok_kvlen.data_ptr(), n, block_table.data_ptr(), block_table.shape[1], out.data_ptr(), heads, row,
-                     kv_rank, float(scale), splits, _p(po), _p(pm), status_word(qa.device).data_ptr(), _stream())
+                     kv_rank, float(scale), int(window), _p(sink), splits, _p(po), _p(pm),
+                     status_word(qa.device).data_ptr(), _stream())
         return
     _native.call("tw_latent_attn", qa.data_ptr(), cache.data_ptr(), tok_seq.data_ptr(), tok_kvlen.data_ptr(), n,
                  block_table.data_ptr(), block_table.shape[1], page, out.data_ptr(), heads, row, kv_rank, float(scale),
-                 dt, _stream())
+                 int(window), _p(sink), dt, _stream())
 
 
 def latent_expandable(dtype: torch.dtype, dim: int, rot: int, vdim: int) -> bool:
@@ -177,17 +218,19 @@ def latent_expandable(dtype: torch.dtype, dim: int, rot: int, vdim: int) -> bool
 def latent_prefill(q: torch.Tensor, kv: torch.Tensor, latents: torch.Tensor, rot_off: int, ctx_rows: int,
                    ctx_begin: torch.Tensor, out: torch.Tensor, gate: Optional[torch.Tensor], cu_q: torch.Tensor,
                    kv_lens: torch.Tensor, tile_seq: torch.Tensor, tile_q0: torch.Tensor, num_tiles: int, heads: int,
-                   dim: int, rot: int, vdim: int, scale: float) -> None:
+                   dim: int, rot: int, vdim: int, scale: float, window: int = 0,
+                   sink: Optional[torch.Tensor] = None) -> None:
     """Expanded causal attention of the listed 128-query tiles (CUDA, bf16). ``q`` [T, heads * (dim + rot)] with rotated
     tails; ``kv`` [ctx_rows, heads * dim | heads * vdim] and the rotated part ``latents[:, rot_off:]`` of every
-    context row; sequence b's context starts at workspace row ``ctx_begin[b]``."""
+    context row; key k of sequence b is workspace row ``ctx_begin[b] + k``. ``window`` and ``sink`` as for
+    :func:`latent_attention`."""
     _dt(q, kv, latents, out, gate)
     kr = latents[:, rot_off:]
     _native.call("tw_latent_prefill", q.data_ptr(), _row_stride(q), q.shape[0], kv.data_ptr(), _row_stride(kv),
                  kr.data_ptr(), _row_stride(kr), ctx_rows, ctx_begin.data_ptr(), out.data_ptr(), _row_stride(out),
                  _p(gate), _row_stride(gate) if gate is not None else 0, cu_q.data_ptr(), kv_lens.data_ptr(),
-                 tile_seq.data_ptr(), tile_q0.data_ptr(), num_tiles, heads, dim, rot, vdim, float(scale),
-                 status_word(q.device).data_ptr(), _stream())
+                 tile_seq.data_ptr(), tile_q0.data_ptr(), num_tiles, heads, dim, rot, vdim, float(scale), int(window),
+                 _p(sink), status_word(q.device).data_ptr(), _stream())
 
 
 def latent_values(o: torch.Tensor, rows: torch.Tensor, w_uv: torch.Tensor, heads: int, vdim: int, kv_rank: int,
@@ -205,10 +248,11 @@ def latent_values(o: torch.Tensor, rows: torch.Tensor, w_uv: torch.Tensor, heads
 
 
 def latent_gather(cache: torch.Tensor, seqs: torch.Tensor, cu: torch.Tensor, max_rows: int, block_table: torch.Tensor,
-                  out: torch.Tensor) -> None:
-    """The first ``cu[i + 1] - cu[i]`` cache rows of sequence ``seqs[i]``, in order, into ``out[cu[i]:]`` (CUDA)."""
-    _native.call("tw_latent_gather", cache.data_ptr(), out.data_ptr(), seqs.data_ptr(), cu.data_ptr(), seqs.shape[0],
-                 max_rows, block_table.data_ptr(), block_table.shape[1], cache.shape[1],
+                  out: torch.Tensor, first: Optional[torch.Tensor] = None) -> None:
+    """``cu[i + 1] - cu[i]`` cache rows of sequence ``seqs[i]``, in order from key ``first[i]`` (None: 0) on, into
+    ``out[cu[i]:]`` (CUDA)."""
+    _native.call("tw_latent_gather", cache.data_ptr(), out.data_ptr(), seqs.data_ptr(), cu.data_ptr(), _p(first),
+                 seqs.shape[0], max_rows, block_table.data_ptr(), block_table.shape[1], cache.shape[1],
                  cache.shape[2] * cache.element_size(), _stream())
 
 
@@ -344,28 +388,39 @@ def add_prenorm_(y: torch.Tensor, x32: torch.Tensor, first: Optional[torch.Tenso
                  y.shape[0], weight.numel(), float(eps), _dt(y, weight, xa), _stream())
 
 
-def projection(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], silu: Optional[tuple[int, int]],
-               out: torch.Tensor) -> torch.Tensor:
-    """``out = x w^T + bias``, then silu on the columns ``[silu[0], silu[1])`` (in the product's epilogue in bf16)."""
+def projection(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], cols: Optional[tuple[int, int]],
+               out: torch.Tensor, act: str = "silu") -> torch.Tensor:
+    """``out = x w^T + bias``, then ``act`` ("silu" or "relu2", the square of relu) on the columns ``[cols[0], cols[1])``
+    (in the product's epilogue in bf16)."""
     if not x.is_cuda:
         gemm(x, w, out=out, bias=bias)
-        if silu is not None:
-            out[:, silu[0]:silu[1]] = torch.nn.functional.silu(out[:, silu[0]:silu[1]])
+        if cols is not None:
+            part = out[:, cols[0]:cols[1]]
+            part.copy_(torch.relu(part) ** 2 if act == "relu2" else torch.nn.functional.silu(part))
         return out
-    if silu is None or x.dtype == torch.bfloat16:
-        return gemm(x, w, out=out, bias=bias, silu_cols=silu)
+    if cols is None or x.dtype == torch.bfloat16:
+        return gemm(x, w, out=out, bias=bias, col_act=None if cols is None else (act, *cols))
     gemm(x, w, out=out, bias=bias)
-    part = out[:, silu[0]:silu[1]]
-    _native.call("tw_silu_cols", part.data_ptr(), _row_stride(part), part.shape[0], part.shape[1], _dt(part), _stream())
+    part = out[:, cols[0]:cols[1]]
+    _native.call("tw_act_cols", part.data_ptr(), _row_stride(part), part.shape[0], part.shape[1], COL_ACTS[act], _dt(part),
+                 _stream())
     return out
 
 
-GLU_ACTS = {"silu": 1, "gelu_tanh": 2}
+GLU_ACTS = {"silu": 1, "gelu_tanh": 2, "clamped": 3}
 
 
-def gated_product(x: torch.Tensor, w: torch.Tensor, act: str, out: torch.Tensor, tmp: Optional[torch.Tensor]) -> None:
-    """``out = act(x w_gate^T) * (x w_up^T)`` with ``w`` = [gate; up]: one product in bf16, in fp32 a product into ``tmp``
-    and the gate behind it."""
+def glu(z: torch.Tensor, act: "str | tuple", out: torch.Tensor) -> None:
+    """``out = act(z_gate) * z_up`` of rows ``z`` = [gate | up] (CUDA); ``act`` as for :func:`ops.gemm`."""
+    kind, limit, alpha = (act, 0.0, 0.0) if isinstance(act, str) else act
+    _native.call("tw_glu", z.data_ptr(), _row_stride(z), out.data_ptr(), _row_stride(out), z.shape[0], out.shape[1],
+                 GLU_ACTS[kind], float(limit), float(alpha), _dt(z, out), _stream())
+
+
+def gated_product(x: torch.Tensor, w: torch.Tensor, act: "str | tuple", out: torch.Tensor,
+                  tmp: Optional[torch.Tensor]) -> None:
+    """``out = act(x w_gate^T) * (x w_up^T)`` with ``w`` = [gate; up] (``act`` as for :func:`ops.gemm`): one product in bf16,
+    in fp32 a product into ``tmp`` and the gate behind it."""
     if not x.is_cuda:
         ref.gated_product(x, w, act, out)
         return
@@ -373,8 +428,7 @@ def gated_product(x: torch.Tensor, w: torch.Tensor, act: str, out: torch.Tensor,
         gemm(x, w, out=out, swiglu=True, act=act)
         return
     gemm(x, w, out=tmp)
-    _native.call("tw_glu", tmp.data_ptr(), _row_stride(tmp), out.data_ptr(), _row_stride(out), x.shape[0], out.shape[1],
-                 GLU_ACTS[act], _dt(tmp, out), _stream())
+    glu(tmp, act, out)
 
 
 # ---- grouped attention ------------------------------------------------------------------------------------------------
@@ -384,23 +438,26 @@ QK_NORMS = {None: 0, "head": 1, "whole": 2}
 def qkv_prep(p: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, q: torch.Tensor, k_cache: torch.Tensor,
              v_cache: torch.Tensor, meta, conv_w: Optional[torch.Tensor], conv_state: Optional[torch.Tensor],
              qk_norm: Optional[str], wq: Optional[torch.Tensor], wk: Optional[torch.Tensor], eps: float, temp_coef: float,
-             temp_every: int) -> None:
+             temp_every: int, cos_sin: Optional[torch.Tensor] = None) -> None:
     """Everything between the projection and the attention. ``p`` rows are [queries | keys | values], heads padded to
     the caches' last dimension; ``conv_w`` [taps, columns] and ``conv_state`` [slots, taps - 1, columns]: causal
-    convolution over time, the state moved on; norm of queries and keys per head or whole; queries times
-    ``1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)``; ``q`` [T, heads * padded], keys and values into the
+    convolution over time, the state moved on; norm of queries and keys per head or whole; rotation of the first
+    ``cos_sin.shape[1]`` dimensions of every query and key head (dimensions 2i and 2i + 1 are a pair; the table's rows are
+    cosines, then sines, by position); queries times ``1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)``; ``q`` [T, heads * padded], keys and values into the
     caches [blocks, page, kv_heads, padded]."""
     if not p.is_cuda:
         ref.qkv_prep(p, heads, kv_heads, dim, vdim, q, k_cache, v_cache, meta, conv_w, conv_state, qk_norm, wq, wk, eps,
-                     temp_coef, temp_every)
+                     temp_coef, temp_every, cos_sin)
         return
     e = meta.extra
+    assert cos_sin is None or (cos_sin.dtype == torch.float32 and cos_sin.is_contiguous())
     _native.call("tw_qkv_prep", p.data_ptr(), _row_stride(p), p.shape[0], heads, kv_heads, dim, k_cache.shape[-1],
                  v_cache.shape[-1], q.data_ptr(), _row_stride(q), k_cache.data_ptr(), v_cache.data_ptr(),
                  meta.positions.data_ptr(), meta.slot_mapping.data_ptr(), _p(conv_w), _p(conv_state),
                  conv_w.shape[0] if conv_w is not None else 1, _p(e.get("row_seq")), meta.cu_q.data_ptr(),
                  meta.kv_lens.data_ptr(), _p(e.get("state_slots")), meta.num_seqs, int(meta.all_single),
-                 QK_NORMS[qk_norm], _p(wq), _p(wk), float(eps), float(temp_coef), int(temp_every),
+                 QK_NORMS[qk_norm], _p(wq), _p(wk), float(eps), float(temp_coef), int(temp_every), _p(cos_sin),
+                 cos_sin.shape[1] if cos_sin is not None else 0,
                  _dt(p, q, k_cache, v_cache, conv_w, conv_state, wq, wk), _stream())
 
 
@@ -410,21 +467,22 @@ def attention_tileable(dtype: torch.dtype, dp: int, vp: int) -> bool:
 
 
 def attention_rows_plan(n: int, heads: int, kv_heads: int, dp: int, vp: int, page: int, dtype: torch.dtype,
-                        max_kv_len: int, sm_count: int = 148) -> tuple[str, int]:
+                        max_kv_len: int, sm_count: int = 148, window: int = 0, keep: int = 0) -> tuple[str, int]:
     """(kernel, key splits) for rows attended alone: "tc" (tensor cores) or "simt" (fp32, heads beyond 128 elements)."""
     if dtype != torch.bfloat16 or dp > 128 or vp > 128 or page < 8 or page > 128 or 128 % page:
         return "simt", 1
     blocks = kv_heads * ((heads // kv_heads + 15) // 16)
-    return "tc", decode_splits_tc(n * blocks, (max_kv_len + 127) // 128, sm_count)
+    return "tc", decode_splits_tc(n * blocks, _key_tiles(max_kv_len, window, keep), sm_count)
 
 
 def grouped_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, meta, heads: int,
                       kv_heads: int, scale: float, slopes: Optional[torch.Tensor], sink: bool, out_scale: float,
-                      sm_count: int = 148, kernel: Optional[str] = None) -> None:
+                      sm_count: int = 148, kernel: Optional[str] = None, window: int = 0, keep: int = 0) -> None:
     """Causal attention of a step's rows over the paged caches; head h's score loses ``slopes[h] * (i - j)``; ``sink``
-    adds one to the denominator; the result is multiplied by ``out_scale``. ``kernel``: force "simt" (tests)."""
+    adds one to the denominator; the result is multiplied by ``out_scale``; ``window`` > 0: a row sees the last ``window``
+    keys, itself among them, and the sequence's first ``keep``. ``kernel``: force "simt" (tests)."""
     if not q.is_cuda:
-        ref.grouped_attention(q, k_cache, v_cache, out, meta, heads, kv_heads, scale, slopes, sink, out_scale)
+        ref.grouped_attention(q, k_cache, v_cache, out, meta, heads, kv_heads, scale, slopes, sink, out_scale, window, keep)
         return
     dt = _dt(q, k_cache, v_cache, out)
     page, dp, vp = k_cache.shape[1], k_cache.shape[-1], v_cache.shape[-1]
@@ -433,16 +491,17 @@ def grouped_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
                      v_cache.data_ptr(), k_cache.shape[0], page, out.data_ptr(), _row_stride(out), meta.cu_q.data_ptr(),
                      meta.kv_lens.data_ptr(), meta.block_table.data_ptr(), meta.block_table.shape[1],
                      meta.tile_seq.data_ptr(), meta.tile_q0.data_ptr(), meta.num_tiles, heads, kv_heads, dp, vp,
-                     float(scale), _p(slopes), int(sink), float(out_scale), status_word(q.device).data_ptr(), _stream())
+                     float(scale), _p(slopes), int(sink), float(out_scale), int(window), int(keep),
+                     status_word(q.device).data_ptr(), _stream())
     n = meta.num_single
     if n == 0:
         return
-    plan, splits = attention_rows_plan(n, heads, kv_heads, dp, vp, page, q.dtype, meta.max_kv_len, sm_count)
+    plan, splits = attention_rows_plan(n, heads, kv_heads, dp, vp, page, q.dtype, meta.max_kv_len, sm_count, window, keep)
     if (kernel or plan) == "simt":
         _native.call("tw_attn_rows", q.data_ptr(), _row_stride(q), k_cache.data_ptr(), v_cache.data_ptr(), page,
                      out.data_ptr(), _row_stride(out), meta.tok_row.data_ptr(), meta.tok_seq.data_ptr(),
                      meta.tok_kvlen.data_ptr(), n, meta.block_table.data_ptr(), meta.block_table.shape[1], heads, kv_heads,
-                     dp, vp, float(scale), _p(slopes), int(sink), float(out_scale), dt, _stream())
+                     dp, vp, float(scale), _p(slopes), int(sink), float(out_scale), int(window), int(keep), dt, _stream())
         return
     po = pm = None
     if splits > 1:
@@ -450,5 +509,5 @@ def grouped_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     _native.call("tw_attn_decode_grouped", q.data_ptr(), _row_stride(q), k_cache.data_ptr(), v_cache.data_ptr(),
                  k_cache.shape[0], page, out.data_ptr(), _row_stride(out), meta.tok_row.data_ptr(), meta.tok_seq.data_ptr(),
                  meta.tok_kvlen.data_ptr(), n, meta.block_table.data_ptr(), meta.block_table.shape[1], heads, kv_heads, dp,
-                 vp, float(scale), _p(slopes), int(sink), float(out_scale), splits, _p(po), _p(pm),
+                 vp, float(scale), _p(slopes), int(sink), float(out_scale), int(window), int(keep), splits, _p(po), _p(pm),
                  status_word(q.device).data_ptr(), _stream())

@@ -380,11 +380,31 @@ def moe_router(x: torch.Tensor, gate_w: torch.Tensor, topk: int, renormalize: bo
     return w, ids.to(torch.int32), logits
 
 
+def moe_route(x: torch.Tensor, w: torch.Tensor, experts: int, topk: int, correction: Optional[torch.Tensor],
+              sum_eps: float):
+    """Softmax scores over all experts, choice by score + correction, weights from the scores of the chosen ones; the rows
+    of ``w`` behind the experts' are gates. Returns (weights, ids, sigmoid gates)."""
+    logits = x.float() @ w.float().t()
+    scores = torch.softmax(logits[:, :experts], dim=-1)
+    choice = scores if correction is None else scores + correction
+    ids = torch.topk(choice, topk, dim=-1).indices
+    chosen = scores.gather(1, ids)
+    return chosen / (chosen.sum(-1, keepdim=True) + sum_eps), ids.to(torch.int32), torch.sigmoid(logits[:, experts:])
+
+
+def gemm_clamped(a: torch.Tensor, w_gate_up: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+    """``g sigmoid(alpha g) (u + 1)`` with ``g = min(a @ Wg.T, limit)``, ``u = a @ Wu.T`` inside ``[-limit, limit]``."""
+    y = a.float() @ w_gate_up.float().t()
+    g, u = y.chunk(2, -1)
+    g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + 1)).to(a.dtype)
+
+
 def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torch.Tensor,
-                topk_ids: torch.Tensor) -> torch.Tensor:
-    """Loop-over-experts MoE MLP: ``sum_k w_k * W2[e_k] (silu(W1[e_k] x) * W3[e_k] x)``.
-    ``w13``: [E, 2*I, H] (gate rows first), ``w2``: [E, H, I]. The activation and the weighted
-    expert output are rounded to the storage dtype, the top-k sum runs in fp32."""
+                topk_ids: torch.Tensor, act="silu") -> torch.Tensor:
+    """Loop-over-experts MoE MLP: ``sum_k w_k * W2[e_k] (silu(W1[e_k] x) * W3[e_k] x)``, or with the clamped gate
+    ``act = ("clamped", limit, alpha)``. ``w13``: [E, 2*I, H] (gate rows first), ``w2``: [E, H, I]. The activation and the
+    weighted expert output are rounded to the storage dtype, the top-k sum runs in fp32."""
     T, H = x.shape
     E = w13.shape[0]
     out = torch.zeros(T, H, dtype=torch.float32, device=x.device)
@@ -394,8 +414,8 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: to
         if tok.numel() == 0:
             continue
         xe = x.index_select(0, tok)
-        act = gemm_swiglu(xe, w13[e])
-        ye = gemm(act, w2[e], row_scale=topk_w[tok, slot])
+        mid = gemm_swiglu(xe, w13[e]) if act == "silu" else gemm_clamped(xe, w13[e], *act[1:])
+        ye = gemm(mid, w2[e], row_scale=topk_w[tok, slot])
         out.index_add_(0, tok, ye.float())
     return out.to(x.dtype)
 

@@ -7,6 +7,8 @@ from typing import Optional
 import torch
 import torch.nn.functional as F
 
+from .reference import gemm_clamped
+
 
 def _unit(x: torch.Tensor, eps: float) -> torch.Tensor:
     return x / torch.sqrt(x.pow(2).mean(-1, keepdim=True) + eps)
@@ -49,6 +51,16 @@ def _rotate(x, cos_sin, positions, rot_dims: int):
     return torch.cat([u * cos - v * sin, v * cos + u * sin, x[..., rot_dims:]], -1)
 
 
+def _rotate_pairs(x, cos_sin, positions):
+    """``x`` [T, heads, D]: the first ``cos_sin.shape[1]`` dimensions rotated, dimensions 2i and 2i + 1 as a pair."""
+    dims = cos_sin.shape[1]
+    cs = cos_sin.index_select(0, positions.long()).unsqueeze(1)
+    cos, sin = cs[..., :dims // 2], cs[..., dims // 2:]
+    u, v = x[..., 0:dims:2], x[..., 1:dims:2]
+    turned = torch.stack([u * cos - v * sin, v * cos + u * sin], -1).flatten(-2)
+    return torch.cat([turned, x[..., dims:]], -1)
+
+
 def latent_prep(p, q_off, q_rank, wq, cq, kv_off, kv_rank, wkv, rot, rot_dims, cos_sin, positions, slots, cache,
                 eps: float) -> None:
     pf = p.float()
@@ -72,7 +84,7 @@ def latent_absorb(q, rows, w_ukt, heads, dim, rot, rot_dims, kv_rank, cos_sin, p
     return out.to(q.dtype)
 
 
-def latent_attention(qa, cache, tok_seq, tok_kvlen, block_table, kv_rank, scale):
+def latent_attention(qa, cache, tok_seq, tok_kvlen, block_table, kv_rank, scale, window: int = 0, sink=None):
     n, heads, _ = qa.shape
     page = cache.shape[1]
     out = torch.empty(n, heads, kv_rank, dtype=qa.dtype)
@@ -83,8 +95,9 @@ def latent_attention(qa, cache, tok_seq, tok_kvlen, block_table, kv_rank, scale)
         blocks = block_table[s, : (top + page - 1) // page].long()
         flat[s] = cache.index_select(0, blocks).reshape(-1, cache.shape[-1]).float()
     for i in range(n):
-        keys = flat[seqs[i]][: lens[i]]
-        w = torch.softmax(qa[i].float() @ keys.t() * scale, -1)
+        keys = flat[seqs[i]][max(0, lens[i] - window) if window else 0: lens[i]]
+        s = qa[i].float() @ keys.t() * scale
+        w = torch.softmax(s if sink is None else torch.cat([s, sink[:, None]], -1), -1)[:, :keys.shape[0]]
         out[i] = (w @ keys[:, :kv_rank]).to(qa.dtype)
     return out
 
@@ -149,6 +162,26 @@ def decay_scan(p, decay, state, y, seqs, cu_q, kv_lens, slots) -> None:
     _recurrence(r[:, :inner].reshape(T, heads, vdim), k, q, one * decay, one, None, state, y, seqs, cu_q, kv_lens, slots)
 
 
+# ---- hyper-connections -------------------------------------------------------------------------------------------
+def embed_streams(ids, table, x, hc_in, weight, offset: float, eps: float, xa) -> None:
+    h = weight.numel()
+    ok = (ids >= 0) & (ids < table.shape[0])
+    rows = table.index_select(0, torch.where(ok, ids, torch.zeros_like(ids)).long())[:, :h].float() * ok.unsqueeze(-1)
+    x[:, :, :h] = rows.unsqueeze(1)
+    xa[:, :h] = _unit(rows * hc_in.sum(), eps) * (offset + weight.float())
+
+
+def streams_step(y, x, hc, mult: float, next_in, weight, offset: float, eps: float, xa) -> None:
+    h = weight.numel()
+    new = torch.einsum("nsw,st->ntw", x[:, :, :h], hc["mix"]) + mult * hc["out"][:, None] * y[:, None, :h].float()
+    if next_in is None:
+        u = new.sum(1)
+    else:
+        x[:, :, :h] = new
+        u = torch.einsum("nsw,s->nw", new, next_in)
+    xa[:, :h] = _unit(u, eps) * (offset + weight.float())
+
+
 # ---- blocks whose sublayers read one norm of the stream ---------------------------------------------------------
 def pair_rows(ids, row_seq, cu_q, prev_token, spec):
     """Row of the pair table for every token; its last row for a token without one before it."""
@@ -184,7 +217,10 @@ def add_prenorm_(y, x32, first, weight, eps: float, xa) -> None:
     xa[:, :h] = _unit(x, eps) * weight.float()
 
 
-def gated_product(x, w, act: str, out) -> None:
+def gated_product(x, w, act, out) -> None:
+    if not isinstance(act, str):
+        out.copy_(gemm_clamped(x, w, *act[1:]))
+        return
     d = w.shape[0] // 2
     z = x.float() @ w.float().t()
     g = F.silu(z[:, :d]) if act == "silu" else F.gelu(z[:, :d], approximate="tanh")
@@ -198,7 +234,7 @@ def norm_gate(y, gate, weight, count: int, eps: float, scale: float, out) -> Non
 
 
 def qkv_prep(p, heads: int, kv_heads: int, dim: int, vdim: int, q, k_cache, v_cache, meta, conv_w, conv_state, qk_norm,
-             wq, wk, eps: float, temp_coef: float, temp_every: int) -> None:
+             wq, wk, eps: float, temp_coef: float, temp_every: int, cos_sin=None) -> None:
     dp, vp, T = k_cache.shape[-1], v_cache.shape[-1], p.shape[0]
     x = p.float()
     if conv_w is not None:
@@ -223,6 +259,9 @@ def qkv_prep(p, heads: int, kv_heads: int, dim: int, vdim: int, q, k_cache, v_ca
         return t.reshape(T, -1)
     if qk_norm:
         qs, ks = normed(qs, wq, heads), normed(ks, wk, kv_heads)
+    if cos_sin is not None:
+        qs, ks = (_rotate_pairs(t.reshape(T, n, dp), cos_sin, meta.positions).reshape(T, -1)
+                  for t, n in ((qs, heads), (ks, kv_heads)))
     if temp_coef:
         turn = torch.div(meta.positions.long() + 1, temp_every, rounding_mode="floor")
         qs = qs * (1 + temp_coef * torch.log(turn.float() + 1)).unsqueeze(-1)
@@ -234,7 +273,7 @@ def qkv_prep(p, heads: int, kv_heads: int, dim: int, vdim: int, q, k_cache, v_ca
 
 
 def grouped_attention(q, k_cache, v_cache, out, meta, heads: int, kv_heads: int, scale: float, slopes, sink: bool,
-                      out_scale: float) -> None:
+                      out_scale: float, window: int = 0, keep: int = 0) -> None:
     page, dp, vp, rep = k_cache.shape[1], k_cache.shape[-1], v_cache.shape[-1], heads // kv_heads
     for b, kv_len in enumerate(meta.kv_lens_cpu):
         t0, t1 = meta.cu_q_cpu[b], meta.cu_q_cpu[b + 1]
@@ -245,7 +284,10 @@ def grouped_attention(q, k_cache, v_cache, out, meta, heads: int, kv_heads: int,
         dist = torch.arange(kv_len - (t1 - t0), kv_len).unsqueeze(-1) - torch.arange(kv_len)
         if slopes is not None:
             s = s - slopes[:, None, None] * dist
-        s = s.masked_fill(dist < 0, float("-inf"))
+        hidden = dist < 0
+        if window:
+            hidden = hidden | ((dist >= window) & (torch.arange(kv_len) >= keep))
+        s = s.masked_fill(hidden, float("-inf"))
         if sink:
             s = torch.cat([s, torch.zeros(heads, t1 - t0, 1)], -1)
         w = torch.softmax(s, -1)[..., :kv_len]
