@@ -121,7 +121,8 @@ def unequal_requests(oracle, cfg, w, path, where):
                 logits = logits[len(part):]
             for rid in end:
                 del live[rid]
-        assert r.core.kv.states.num_free == 3 and r.core.kv.pool.num_free == 19
+        states = r.core.kv.states                      # None in models without recurrent state
+        assert (states is None or states.num_free == 3) and r.core.kv.pool.num_free == 19
     for rid, t in todo:
         check(torch.cat(got[rid]), oracle.logits(cfg, w, t), where, rid)
 

@@ -228,6 +228,23 @@ def _kebopel(vocab, width, ff, layers, attn, left, right, decay, loop, bigram) -
                         "mlp": {"kind": "dense", "ff": ff}} for i in range(layers)]}
 
 
+def _netezen(vocab, width, layers, streams, attn, latent, dense, moe, shared, windows) -> dict:
+    """``config.json`` of a Netezen model: a latent attention with a dense feed-forward first, then attentions and latent
+    attentions in turn with mixtures of experts. attn: (heads, kv_heads, dim, vdim, rotated), latent: (heads, dim, rot_dim,
+    vdim, kv_rank, q_rank), moe: (experts, top, ff, limit), shared: (ff, limit), windows: (attention, kept first, latent)."""
+    sizes = lambda names, v: dict(zip(names.split(), v))
+    a = {**sizes("heads kv_heads dim vdim", attn), "scale": attn[2] ** -0.5,
+         "rot": {"base": 500000.0, "dims": attn[4], "scaling": dict(factor=16.0, original=8192, fast=32.0, slow=1.0)},
+         "mask": {"size": windows[0], "keep_first": windows[1]}}
+    l = {**sizes("heads dim rot_dim vdim kv_rank q_rank", latent), "scale": (latent[1] + latent[2]) ** -0.5,
+         "rot": {"base": 10000.0, "dims": latent[2]}, "mask": {"size": windows[2]}}
+    ff = {"kind": "moe", "router": sizes("experts top", moe), "expert": sizes("ff limit", moe[2:]),
+          "shared": sizes("ff limit", shared)}
+    return {"architecture": "Netezen", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "streams": streams,
+            "residual_mult": 0.5, "layers": [{"type": "attention" if i % 2 else "latent_attention", "mixer": a if i % 2 else l,
+                                              "mlp": ff if i else {"kind": "dense", "ff": dense}} for i in range(layers)]}
+
+
 def _decays(n: int) -> list:
     """Memories from a few tokens to a few thousand, evenly spaced in the logarithm."""
     return [1.0 - 2.0 ** (-2.0 - 9.0 * i / max(1, n - 1)) for i in range(n)]
@@ -276,6 +293,10 @@ MODEL_PRESETS: dict[str, dict[str, Any]] = {
                                          dict(start=1, stop=3, times=2), 1000)),
     "kebopel-9b": dict(config=_kebopel(128256, 4096, 14336, 27, (32, 8, 128, 128), (32, 8, 128, 128), (32, 128, 128),
                                        _decays(32), dict(start=9, stop=18, times=2), 262144)),
+    "tiny-netezen": dict(config=_netezen(512, 160, 3, 2, (6, 2, 40, 32, 24), (4, 40, 16, 32, 72, 48), 256, (8, 2, 64, 3.0),
+                                         (96, 3.0), (100, 2, 70))),
+    "netezen-30b": dict(config=_netezen(128256, 4096, 36, 4, (32, 8, 128, 128, 64), (32, 128, 64, 128, 512, 1536), 14336,
+                                        (32, 4, 1792, 7.0), (3584, 7.0), (4096, 4, 1024))),
     "llama-3.3-70b": dict(architecture="llama", hidden_size=8192, num_layers=80, num_q_heads=64, num_kv_heads=8,
                           head_dim=128, intermediate_size=28672, vocab_size=128256, rms_norm_eps=1e-5,
                           rope_theta=500000.0, max_model_len=131072,

@@ -55,6 +55,15 @@ __device__ __forceinline__ float2 fadd2(float2 a, float2 b) {
   return d;
 }
 
+// e to 16 bits of mantissa in two bf16 terms: the leading one cut off (no conversion), the rest rounded
+__device__ __forceinline__ void split_weights(float2 e, uint32_t& hi, uint32_t& lo) {
+  const uint32_t x = __float_as_uint(e.x), y = __float_as_uint(e.y);
+  hi = __byte_perm(x, y, 0x7632);
+  const float2 l = fma2(make_float2(__uint_as_float(x & 0xffff0000u), __uint_as_float(y & 0xffff0000u)),
+                        make_float2(-1.f, -1.f), e);
+  lo = pack_bf16x2(l.x, l.y);
+}
+
 // Items of CTA `c` of `G`: round r takes the c-th item of the r-th block of G items, counted from the
 // front in even rounds and from the back in odd ones (heavy items meet light ones).
 __device__ __forceinline__ int split_item_index(int round, int c, int G) {

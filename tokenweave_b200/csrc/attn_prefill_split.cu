@@ -64,15 +64,6 @@ __device__ __forceinline__ float fast_tanh(float x) {
   return y;
 }
 
-// e to 16 bits of mantissa in two bf16 terms: the leading one cut off (no conversion), the rest rounded
-__device__ __forceinline__ void split_weights(float2 e, uint32_t& hi, uint32_t& lo) {
-  const uint32_t x = __float_as_uint(e.x), y = __float_as_uint(e.y);
-  hi = __byte_perm(x, y, 0x7632);
-  const float2 l = fma2(make_float2(__uint_as_float(x & 0xffff0000u), __uint_as_float(y & 0xffff0000u)),
-                        make_float2(-1.f, -1.f), e);
-  lo = pack_bf16x2(l.x, l.y);
-}
-
 // One work item: a 128-query tile of one head.
 struct SplitItem {
   // key tiles [0, n_pre) and [j_lo, j_lo + n_tiles - n_pre) are needed (j_lo > 0 only under a sliding window, n_pre > 0 only

@@ -10,7 +10,8 @@
 // room for one tile in shared memory (two tiles of 64 keys were 40 % slower: an MMA of this shape takes about 60 cycles
 // whether it has 64 or 128 rows). Rows of up to 640 elements, latents of up to 512. The keys of a
 // row can be cut into splits, whose fp32 partial results a second kernel merges. Under a sliding window only the tiles that
-// hold visible keys are visited; a sink per head joins the denominator at the end.
+// hold visible keys are visited; a sink per head joins the denominator at the end. EXACT: the softmax weights reach the
+// product with the latents as two bf16 terms, which keeps 16 bits of them.
 //
 // Roles (192 threads): warp 0 TMA producer, warp 1 MMA issuer, warps 2..5 softmax (one thread per key of the tile),
 // rescaling and epilogue (one thread per latent column). Waits are bounded; after a timeout the roles keep their trip
@@ -51,12 +52,12 @@ __device__ __forceinline__ void tmem_st_cols(uint32_t addr, const uint32_t (&r)[
 __device__ __forceinline__ void tmem_st_cols(uint32_t addr, const uint32_t (&r)[32]) { tmem_st_32x32(addr, r); }
 
 // Shared memory behind the tiles: Q, P, barriers, exchange.
-template <int NC>
+template <int NC, bool EXACT>
 __host__ __device__ constexpr int ld_fixed_bytes(int chunks) {
-  return chunks * NC * 128 + 2 * NC * 128 + 512 + 2 * 4 * NC * 4 + 1024;
+  return chunks * NC * 128 + (EXACT ? 4 : 2) * NC * 128 + 512 + 2 * 4 * NC * 4 + 1024;
 }
 
-template <int NC>
+template <int NC, bool EXACT>
 __global__ void __launch_bounds__(LD_THREADS, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmQ,
                      const LatentDecodeParams p) {
@@ -75,7 +76,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
   const int tile_bytes = pairs * 2 * CHUNK;
   uint8_t* s_q = smem + p.stages * tile_bytes;
   uint8_t* s_p = s_q + p.chunks * NC * 128;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(s_p + 2 * NC * 128);
+  constexpr int P_LO = 2 * NC * 128;                          // second terms of the weights behind the first ones
+  uint64_t* bars = reinterpret_cast<uint64_t*>(s_p + (EXACT ? 2 : 1) * P_LO);
   uint64_t* full = bars;                                      // [stages][LD_MAX_PAIRS]
   uint64_t* empty = bars + LD_MAX_STAGES * LD_MAX_PAIRS;
   uint64_t* s_full = bars + 2 * LD_MAX_STAGES * LD_MAX_PAIRS;  // [2]
@@ -236,6 +238,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
           for (int k = 0; k < LD_BN / 16; ++k)
             umma_ss_e(d, da + k * (16 * 128 / 16), desc_p + ((k >> 2) * (NC * 128) + (k & 3) * 32) / 16, IDESC_O,
                     (j | k) != 0 ? 1u : 0u);
+          if (EXACT) {
+#pragma unroll
+            for (int k = 0; k < LD_BN / 16; ++k)
+              umma_ss_e(d, da + k * (16 * 128 / 16), desc_p + (P_LO + (k >> 2) * (NC * 128) + (k & 3) * 32) / 16, IDESC_O, 1u);
+          }
           umma_commit_e(&empty[st * LD_MAX_PAIRS + m]);
         }
         umma_commit_e(o_done);
@@ -329,7 +336,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmC, const __grid_const
       for (int g = 0; g < NC; ++g) {
         const float pv = ld_exp2(fmaf(__uint_as_float(sv[g]), p.scale_log2, -m_ref[g]));
         l_part[g] += pv;
-        *reinterpret_cast<__nv_bfloat16*>(p_buf + g * 128 + ((kc ^ (g & 7)) * 16) + ke * 2) = __float2bfloat16(pv);
+        uint8_t* at = p_buf + g * 128 + ((kc ^ (g & 7)) * 16) + ke * 2;
+        const __nv_bfloat16 hi = __float2bfloat16(pv);
+        *reinterpret_cast<__nv_bfloat16*>(at) = hi;
+        if (EXACT) *reinterpret_cast<__nv_bfloat16*>(at + P_LO) = __float2bfloat16(pv - __bfloat162float(hi));
       }
       if (rescale) {
 #pragma unroll 1
@@ -456,7 +466,7 @@ latent_decode_merge_kernel(const float* __restrict__ part_o, const float* __rest
   }
 }
 
-template <int NC>
+template <int NC, bool EXACT>
 static int launch_latent_decode(const void* cache, int num_blocks, LatentDecodeParams& p, int n, cudaStream_t stream) {
   CUtensorMap tm;
   {
@@ -472,7 +482,7 @@ static int launch_latent_decode(const void* cache, int num_blocks, LatentDecodeP
     uint32_t box[2] = {64, NC};
     if (!make_tensor_map_bf16(&tmQ, p.q, 2, dims, strides, box)) return 1;
   }
-  const int tile_bytes = (p.chunks + 1) / 2 * 2 * LD_BN * 128, fixed = ld_fixed_bytes<NC>(p.chunks);
+  const int tile_bytes = (p.chunks + 1) / 2 * 2 * LD_BN * 128, fixed = ld_fixed_bytes<NC, EXACT>(p.chunks);
   p.stages = (LD_SMEM_LIMIT - fixed) / tile_bytes;
   if (p.stages > LD_MAX_STAGES) p.stages = LD_MAX_STAGES;
   if (p.stages < 1) {
@@ -485,14 +495,14 @@ static int launch_latent_decode(const void* cache, int num_blocks, LatentDecodeP
   cudaGetDevice(&dev);
   if (configured_dev != dev) {
     const cudaError_t e =
-        cudaFuncSetAttribute(latent_decode_kernel<NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, LD_SMEM_LIMIT);
+        cudaFuncSetAttribute(latent_decode_kernel<NC, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, LD_SMEM_LIMIT);
     if (e != cudaSuccess) {
       set_last_error("latent_decode: cudaFuncSetAttribute failed: %s", cudaGetErrorString(e));
       return 1;
     }
     configured_dev = dev;
   }
-  latent_decode_kernel<NC><<<dim3(n, (p.heads + NC - 1) / NC, p.splits), LD_THREADS, bytes, stream>>>(tm, tmQ, p);
+  latent_decode_kernel<NC, EXACT><<<dim3(n, (p.heads + NC - 1) / NC, p.splits), LD_THREADS, bytes, stream>>>(tm, tmQ, p);
   cudaError_t e = cudaGetLastError();
   if (e == cudaSuccess && p.splits > 1) {
     latent_decode_merge_kernel<<<n * p.heads, 128, 0, stream>>>(p.part_o, p.part_ml, p.splits, p.kv_rank, p.sink,
@@ -514,7 +524,7 @@ using namespace tw;
 // [n, heads, kv_rank]; part_o [n, heads, splits, kv_rank] and part_ml [n, heads, splits, 2] when splits > 1.
 extern "C" int tw_latent_decode(const void* qa, const void* cache, int num_blocks, int page, const int* tok_seq,
                                 const int* tok_kvlen, int n, const int* block_table, int max_blocks, void* out, int heads,
-                                int row, int kv_rank, float scale, int window, const float* sink, int splits,
+                                int row, int kv_rank, float scale, int window, const float* sink, int exact, int splits,
                                 float* part_o, float* part_ml, uint32_t* status, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (row % 8 != 0 || row > 64 * 2 * LD_MAX_PAIRS || kv_rank > 512 || kv_rank > row || page < 8 || page > 128 || 128 % page != 0) {
@@ -530,6 +540,9 @@ extern "C" int tw_latent_decode(const void* qa, const void* cache, int num_block
                        reinterpret_cast<const __nv_bfloat16*>(cache), tok_seq, tok_kvlen,
                        block_table, max_blocks, page, heads, row, kv_rank, splits, (row + 63) / 64, 1,
                        scale * 1.4426950408889634f, part_o, part_ml, status, window, sink};
-  return heads <= 16 ? launch_latent_decode<16>(cache, num_blocks, p, n, stream)
-                     : launch_latent_decode<32>(cache, num_blocks, p, n, stream);
+  if (exact)
+    return heads <= 16 ? launch_latent_decode<16, true>(cache, num_blocks, p, n, stream)
+                       : launch_latent_decode<32, true>(cache, num_blocks, p, n, stream);
+  return heads <= 16 ? launch_latent_decode<16, false>(cache, num_blocks, p, n, stream)
+                     : launch_latent_decode<32, false>(cache, num_blocks, p, n, stream);
 }

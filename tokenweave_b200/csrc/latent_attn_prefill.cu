@@ -8,8 +8,11 @@
 // of P V. What differs: a key tile is KC chunks of 64 columns, the first ones from the head's unrotated keys and the
 // others from the shared rotated part (chunks are zero-filled behind each part's end by the tensor maps, so widths need
 // not be multiples of 64); values are VC chunks; K and V have separate buffers because their sizes differ; the epilogue
-// multiplies the output by sigmoid(gate), the output gate of the layer; a sink per head may join the denominator; and with a
-// sliding window (an instantiation of its own) an item visits the tiles that hold visible keys only.
+// multiplies the output by sigmoid(gate), the output gate of the layer; and a sink per head may join the denominator.
+//
+// The windowed form (an instantiation of its own): an item visits the tiles that hold visible keys only, and the softmax
+// weights reach the product with V as two bf16 terms, which keeps 16 bits of them (the leading terms in the upper half of
+// the S columns, the others in the lower half); that product starts when the weights of a tile's first 64 keys are there.
 //
 // Roles (320 threads): warp 0 TMA producer, warp 1 MMA issuer, warps 2..5 softmax group A (one thread per query row),
 // warps 6..9 group B. Every mbarrier wait is bounded; after a timeout the roles keep their trip counts, report
@@ -102,7 +105,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   uint64_t* p_ready = bars + 20;      // [2]
   uint64_t* o_done = bars + 22;       // [2]
   uint64_t* epi_done = bars + 24;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 25);
+  uint64_t* p_half = bars + 25;       // [2], windowed form: weights of the first 64 keys
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 27);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5;
@@ -122,6 +126,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     for (int g = 0; g < 2; ++g) {
       mbar_init(&s_full[g], 1);
       mbar_init(&p_ready[g], 128);
+      mbar_init(&p_half[g], 128);
       mbar_init(&o_done[g], 1);
     }
     mbar_init(epi_done, ATT_SOFTMAX_THREADS);
@@ -233,16 +238,24 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
           return true;
         };
         auto issue_pv = [&](int g, bool first) {
-          if (!mbar_wait(&p_ready[g], cnt[g] & 1)) return false;
+          if (!mbar_wait(WINDOW ? &p_half[g] : &p_ready[g], cnt[g] & 1)) return false;
           const int slot = cnt[g] % S::VS;
           if (!mbar_wait(&v_full[g * LP_MAX_SLOTS + slot], (cnt[g] / S::VS) & 1)) return false;
           tc_fence_after_sync();
           const uint32_t v_addr = smem_u32(smem + S::OFF_V + (g * S::VS + slot) * S::V_BYTES);
+          auto pv = [&](int k, uint32_t col, bool init) {
+            umma_ts(tmem_base + COL_O + g * 128, tmem_base + COL_S + g * 128 + col + k * 8,
+                    make_smem_desc_sw128(v_addr + k * 16 * 128, ATT_HALF_BYTES, 1024), IDESC_PV, init ? 0u : 1u);
+          };
 #pragma unroll
-          for (int k = 0; k < ATT_BN / 16; ++k)
-            umma_ts(tmem_base + COL_O + g * 128, tmem_base + COL_S + g * 128 + COL_P + k * 8,
-                    make_smem_desc_sw128(v_addr + k * 16 * 128, ATT_HALF_BYTES, 1024), IDESC_PV,
-                    (first && k == 0) ? 0u : 1u);
+          for (int k = 0; k < ATT_BN / 16; ++k) {
+            if (WINDOW && k == 4) {
+              if (!mbar_wait(&p_ready[g], cnt[g] & 1)) return false;
+              tc_fence_after_sync();
+            }
+            pv(k, COL_P, first && k == 0);
+            if (WINDOW) pv(k, 0, false);
+          }
           umma_commit(&v_empty[g * LP_MAX_SLOTS + slot]);
           umma_commit(&o_done[g]);
           ++cnt[g];
@@ -337,20 +350,25 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         const float2 sc2 = make_float2(p.scale_log2, p.scale_log2);
         const float2 nm2 = make_float2(-m_use, -m_use);
         float2 sum2[2] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
-        uint32_t pk[16];
+        uint32_t pk[16], lo[16];
         auto exp_chunk = [&](const uint32_t (&buf)[32]) {
 #pragma unroll
           for (int i = 0; i < 16; ++i) {
             const float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc2, nm2);
             const float2 e = make_float2(fast_exp2(x.x), fast_exp2(x.y));
             sum2[i & 1] = fadd2(sum2[i & 1], e);
-            pk[i] = pack_bf16x2(e.x, e.y);
+            if (WINDOW) split_weights(e, pk[i], lo[i]);
+            else pk[i] = pack_bf16x2(e.x, e.y);
           }
         };
+        auto store_chunk = [&](int chunk) {
+          tmem_st_32x16(t_p + chunk * 16, pk);
+          if (WINDOW) tmem_st_32x16(t_s + chunk * 16, lo);
+        };
         exp_chunk(s0);
-        tmem_st_32x16(t_p, pk);
+        store_chunk(0);
         exp_chunk(s1);
-        tmem_st_32x16(t_p + 16, pk);
+        store_chunk(1);
         if (t > 0 && __any_sync(0xffffffffu, rescale)) {
           // O_g may be touched once P V of the previous tile has completed
           if (ok) ok = mbar_wait(&o_done[g], (cnt - 1) & 1);
@@ -366,10 +384,15 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
             tmem_st_32x32(t_o + c * 32, v);
           }
         }
+        if (WINDOW) {
+          tmem_wait_st();
+          tc_fence_before_sync();
+          mbar_arrive(&p_half[g]);      // (O_g is scaled by then: the product may go on)
+        }
         exp_chunk(s2);
-        tmem_st_32x16(t_p + 32, pk);
+        store_chunk(2);
         exp_chunk(s3);
-        tmem_st_32x16(t_p + 48, pk);
+        store_chunk(3);
         l_sum = l_sum * alpha + ((sum2[0].x + sum2[0].y) + (sum2[1].x + sum2[1].y));
         tmem_wait_st();
         tc_fence_before_sync();

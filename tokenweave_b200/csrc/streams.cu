@@ -7,8 +7,8 @@
 //   tw_streams_step    what lies between two sublayers, in one pass: the streams behind a sublayer's output and the next
 //                      sublayer's normed input (behind the last one: the norm of the plain sum, the streams are not stored)
 //
-// One CTA per row; the weighted sum stays in registers between the two passes. All arithmetic is fp32; y, w and xa are bf16
-// or fp32. S = 1 with coefficients of one is a pre-norm residual stream.
+// One CTA per row; the weighted sum stays in registers between the two passes (in shared memory beyond four streams). All
+// arithmetic is fp32; y, w and xa are bf16 or fp32. S = 1 with coefficients of one is a pre-norm residual stream.
 #include "tw_host.h"
 #include "tw_kernels.h"
 #include "tw_typed.cuh"
@@ -97,6 +97,67 @@ streams_step_kernel(const StreamsArgs a) {
   }
 }
 
+// More streams than a thread can hold eight elements of: four elements at a time.
+template <typename T>
+__global__ void __launch_bounds__(512)
+streams_step_wide_kernel(const StreamsArgs a) {
+  extern __shared__ float u_s[];                                     // [H rounded up to eight]
+  __shared__ float scratch[32];
+  __shared__ float mix_s[STREAMS_MAX * STREAMS_MAX], out_s[STREAMS_MAX], in_s[STREAMS_MAX];
+  for (int i = threadIdx.x; i < STREAMS_MAX * STREAMS_MAX; i += blockDim.x) {
+    const int to = i / STREAMS_MAX, from = i % STREAMS_MAX;
+    mix_s[i] = to < a.S && from < a.S ? a.mix[from * a.S + to] : 0.f;
+  }
+  if (threadIdx.x < a.S) {
+    out_s[threadIdx.x] = a.mult * a.out[threadIdx.x];
+    in_s[threadIdx.x] = a.in != nullptr ? a.in[threadIdx.x] : 1.f;
+  }
+  __syncthreads();
+  const T* yr = reinterpret_cast<const T*>(a.y);
+  const T* w = reinterpret_cast<const T*>(a.w);
+  T* xa = reinterpret_cast<T*>(a.xa);
+  for (int t = blockIdx.x; t < a.rows; t += gridDim.x) {
+    float ss[1] = {0.f};
+    for (int i = threadIdx.x * 4; i < a.H; i += blockDim.x * 4) {    // (a row's pad holds zeros and may be read)
+      float* x = a.x + t * a.ldx + i;
+      float4 old[STREAMS_MAX];
+#pragma unroll
+      for (int s = 0; s < STREAMS_MAX; ++s)
+        old[s] = s < a.S ? *reinterpret_cast<const float4*>(x + s * a.lds) : make_float4(0.f, 0.f, 0.f, 0.f);
+      float y[4], u[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+      for (int j = 0; j < 4; ++j) y[j] = i + j < a.H ? ld1(yr + t * a.ldy + i + j) : 0.f;
+#pragma unroll 1
+      for (int to = 0; to < a.S; ++to) {
+        const float o = out_s[to], in = in_s[to];
+        float4 v = make_float4(o * y[0], o * y[1], o * y[2], o * y[3]);
+#pragma unroll
+        for (int s = 0; s < STREAMS_MAX; ++s) {
+          const float m = mix_s[to * STREAMS_MAX + s];
+          v.x = fmaf(m, old[s].x, v.x);
+          v.y = fmaf(m, old[s].y, v.y);
+          v.z = fmaf(m, old[s].z, v.z);
+          v.w = fmaf(m, old[s].w, v.w);
+        }
+        if (a.store) *reinterpret_cast<float4*>(x + to * a.lds) = v;
+        u[0] = fmaf(in, v.x, u[0]);
+        u[1] = fmaf(in, v.y, u[1]);
+        u[2] = fmaf(in, v.z, u[2]);
+        u[3] = fmaf(in, v.w, u[3]);
+      }
+      *reinterpret_cast<float4*>(u_s + i) = make_float4(u[0], u[1], u[2], u[3]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ss[0] += u[j] * u[j];
+    }
+    block_sum<1>(ss, scratch);
+    const float r = 1.f / sqrtf(ss[0] / static_cast<float>(a.H) + a.eps);
+    for (int i = threadIdx.x * 4; i < a.H; i += blockDim.x * 4)      // each thread reads back what it wrote
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+        if (i + j < a.H) st1(xa + t * a.lda + i + j, u_s[i + j] * r * (a.offset + ld1(w + i + j)));
+  }
+}
+
 template <typename T, int VPT>
 __global__ void __launch_bounds__(512)
 embed_streams_kernel(const StreamsArgs a) {
@@ -133,8 +194,11 @@ static void launch_streams(const StreamsArgs& a, int grid, int threads, cudaStre
   if (a.ids != nullptr) embed_streams_kernel<T, VPT><<<grid, threads, 0, stream>>>(a);
   else if (a.S <= 2) streams_step_kernel<T, VPT, 2><<<grid, threads, 0, stream>>>(a);
   else if (a.S <= 4) streams_step_kernel<T, VPT, 4><<<grid, threads, 0, stream>>>(a);
-  else if (a.S <= 8) streams_step_kernel<T, VPT, 8><<<grid, threads, 0, stream>>>(a);
-  else streams_step_kernel<T, VPT, STREAMS_MAX><<<grid, threads, 0, stream>>>(a);
+  else {
+    const int smem = (a.H + 7) / 8 * 8 * 4;
+    cudaFuncSetAttribute(streams_step_wide_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    streams_step_wide_kernel<T><<<grid, threads, smem, stream>>>(a);
+  }
 }
 
 static int run_streams(const StreamsArgs& a, int dtype, const char* what, cudaStream_t stream) {

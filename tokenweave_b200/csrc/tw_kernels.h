@@ -230,7 +230,7 @@ int tw_latent_attn(const void* qa, const void* cache, const int* tok_seq, const 
 // tensor-core forms (latent_attn_decode.cu, latent_attn_prefill.cu), bf16
 int tw_latent_decode(const void* qa, const void* cache, int num_blocks, int page, const int* tok_seq,
                      const int* tok_kvlen, int n, const int* block_table, int max_blocks, void* out, int heads, int row,
-                     int kv_rank, float scale, int window, const float* sink, int splits, float* part_o, float* part_ml,
+                     int kv_rank, float scale, int window, const float* sink, int exact, int splits, float* part_o, float* part_ml,
                      uint32_t* status, cudaStream_t stream);
 int tw_latent_prefill(const void* q, long long ldq, int T, const void* kv, long long ldkv, const void* kr, long long ldr,
                       int ctx_rows, const int* ctx_begin, void* out, long long ldo, const void* gate, long long ldg,

@@ -55,14 +55,15 @@ def read(cfg: dict) -> dict:
     """Fields of :class:`ModelConfig` from a ``config.json`` of this design."""
     layers = cfg["layers"]
     m = layers[0]["mixer"]
-    ff = [l["mlp"]["ff"] if l["mlp"]["kind"] == "dense" else l["mlp"]["expert"]["ff"] for l in layers if l.get("mlp")]
+    specs = [layer_spec(l) for l in layers]
+    ff = [s["mlp"]["ff"] for s in specs if s["mlp"]]
     # the configuration names no longest context: what the rotary scaling was made for, else the engine's default
     scalings = [s for s in (l["mixer"]["rot"].get("scaling") for l in layers) if s]
     return dict(
         architecture="netezen", block="streams", streams=int(cfg["streams"]), residual_mult=float(cfg["residual_mult"]),
         norm_offset=1.0, tie_word_embeddings=True, hidden_size=cfg["width"], num_layers=len(layers),
         num_q_heads=m["heads"], num_kv_heads=m.get("kv_heads", 1), head_dim=m["dim"], intermediate_size=max(ff, default=0),
-        vocab_size=cfg["vocab"], rms_norm_eps=float(cfg["norm"]["eps"]), layers=[layer_spec(l) for l in layers],
+        vocab_size=cfg["vocab"], rms_norm_eps=float(cfg["norm"]["eps"]), layers=specs,
         max_model_len=max([8192] + [int(s["original"] * s["factor"]) for s in scalings]))
 
 

@@ -91,7 +91,7 @@ _SIGNATURES = {
     "tw_latent_query": [vp, ll, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, vp],
     "tw_head_gemm": [vp, ll, i32, vp, vp, ll, i32, vp, ll, i32, vp, vp, ll, i32, i32, i32, i32, i32, i32, vp],
     "tw_latent_attn": [vp, vp, vp, vp, i32, vp, i32, i32, vp, i32, i32, i32, f32, i32, vp, i32, vp],
-    "tw_latent_decode": [vp, vp, i32, i32, vp, vp, i32, vp, i32, vp, i32, i32, i32, f32, i32, vp, i32, vp, vp, vp, vp],
+    "tw_latent_decode": [vp, vp, i32, i32, vp, vp, i32, vp, i32, vp, i32, i32, i32, f32, i32, vp, i32, i32, vp, vp, vp, vp],
     "tw_latent_prefill": [vp, ll, i32, vp, ll, vp, ll, i32, vp, vp, ll, vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, i32,
                           f32, i32, vp, vp, vp],
     "tw_latent_gather": [vp, vp, vp, vp, vp, i32, i32, vp, i32, i32, i32, vp],

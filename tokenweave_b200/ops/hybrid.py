@@ -184,7 +184,8 @@ def latent_attention(qa: torch.Tensor, cache: torch.Tensor, tok_seq: torch.Tenso
                      sm_count: int = 148, kernel: Optional[str] = None, window: int = 0,
                      sink: Optional[torch.Tensor] = None) -> None:
     """Causal attention of ``n`` absorbed query rows over the paged latent cache; ``out`` [n, heads, kv_rank].
-    ``window`` > 0: a row sees the last ``window`` keys, itself among them; ``sink`` (fp32 [heads]): exp(sink) joins the
+    ``window`` > 0: a row sees the last ``window`` keys, itself among them (and the tensor-core kernels keep 16 bits of the
+    softmax weights, 8 without it); ``sink`` (fp32 [heads]): exp(sink) joins the
     denominator. ``kernel``: force one of :func:`latent_decode_plan`'s kernels (tests)."""
     if n == 0:
         return
@@ -201,7 +202,7 @@ def latent_attention(qa: torch.Tensor, cache: torch.Tensor, tok_seq: torch.Tenso
             po, pm = _partial_buffers(qa.device, n * heads * splits, kv_rank)
         _native.call("tw_latent_decode", qa.data_ptr(), cache.data_ptr(), cache.shape[0], page, tok_seq.data_ptr(),
                      tok_kvlen.data_ptr(), n, block_table.data_ptr(), block_table.shape[1], out.data_ptr(), heads, row,
-                     kv_rank, float(scale), int(window), _p(sink), splits, _p(po), _p(pm),
+                     kv_rank, float(scale), int(window), _p(sink), int(window > 0), splits, _p(po), _p(pm),
                      status_word(qa.device).data_ptr(), _stream())
         return
     _native.call("tw_latent_attn", qa.data_ptr(), cache.data_ptr(), tok_seq.data_ptr(), tok_kvlen.data_ptr(), n,
