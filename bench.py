@@ -51,10 +51,11 @@ def parse_args():
                     choices=["overlap", "fuse_only", "fused_gemm", "baseline_nccl", "baseline_custom_ar", "baseline_multimem",
                              "no_ar"])
     ap.add_argument("--layers", type=int, default=None, help="debug only: fewer layers (marks the result invalid)")
-    ap.add_argument("--workload", default="prefill", choices=["prefill", "hybrid", "kebopel"],
+    ap.add_argument("--workload", default="prefill", choices=["prefill", "hybrid", "kebopel", "netezen"],
                     help="hybrid: the hybrid decoder (latent attention + Mamba-2) beside the Llama layout at equal size, "
                          "prefill, decode and every kernel (artifact/hybrid_bench.py); kebopel: the same for Kebopel "
-                         "(artifact/kebopel_bench.py); one GPU")
+                         "(artifact/kebopel_bench.py); netezen: Netezen beside the Mixtral layout (artifact/netezen_bench.py); "
+                         "one GPU")
     ap.add_argument("--cuda-graphs", dest="cuda_graphs", action="store_true", default=None,
                     help="replay the step from a CUDA graph (captured during warm-up; the default when --warmup >= 3)")
     ap.add_argument("--no-cuda-graphs", dest="cuda_graphs", action="store_false",
@@ -185,11 +186,11 @@ def run_reference(args) -> None:
         "clocks": clocks, "e2e": {"value": value, "unit": "tokens/s"}, "impl": "reference"}), flush=True)
 
 
-def run_beside_llama(args) -> None:
-    """Throughput of a hybrid decoder (``--workload``) and of the Llama layout at the same widths, one JSON line; ``value``
+def run_beside_closest(args) -> None:
+    """Throughput of a hybrid decoder (``--workload``) and of its closest uniform layout at the same widths, one JSON line; ``value``
     is the hybrid model's prefill at the largest width."""
     import importlib
-    name, model = args.workload, {"hybrid": "sidisun", "kebopel": "kebopel"}[args.workload]
+    name, model = args.workload, {"hybrid": "sidisun"}.get(args.workload, args.workload)
     if args.gpus != 1:
         raise SystemExit(f"--workload {name} runs on one GPU")
     run = importlib.import_module(f"artifact.{name}_bench").run
@@ -209,7 +210,7 @@ def run_beside_llama(args) -> None:
 def main() -> None:
     args = parse_args()
     if args.workload != "prefill":
-        run_beside_llama(args)
+        run_beside_closest(args)
         return
     if args.cuda_graphs is None:
         # eager on the first sight of a step shape, capture on the second, replay from the third on

@@ -490,12 +490,16 @@ def test_hyper_connections(streams):
     new = oracle.connect(old, wide, lambda u: (seen.append(oracle.unit(u, eps) * (1 + w)), y[:, :W].double())[1], 0.7)
     assert (xa[:, :W] - seen[0]).abs().max() < 1e-5
     last = x.clone()
-    hops.streams_step(y, last, hc, 0.7, None, w, 1.0, eps, xa)
+    hops.streams_step(y, last, hc, 0.7, None, w, 1.0, eps, xa, first=True)
     assert (xa[:, :W] - oracle.unit(new.sum(0), eps) * (1 + w)).abs().max() < 1e-4
-    hops.streams_step(y, x, hc, 0.7, nxt, w, 1.0, eps, xa)
+    hops.streams_step(y, x, hc, 0.7, nxt, w, 1.0, eps, xa, first=True)
     assert (x.transpose(0, 1)[..., :W] - new).abs().max() < 1e-5
     u = sum(nxt[s].double() * new[s] for s in range(streams))
     assert (xa[:, :W] - oracle.unit(u, eps) * (1 + w)).abs().max() < 1e-4
+    # and once more, from streams that differ
+    again = oracle.connect(new, wide, lambda _: y[:, :W].double(), 0.7)
+    hops.streams_step(y, x, hc, 0.7, nxt, w, 1.0, eps, xa)
+    assert (x.transpose(0, 1)[..., :W] - again).abs().max() < 1e-4
 
 
 @pytest.mark.parametrize("experts,top", [(6, 2), (6, 6), (40, 9), (1, 1)])

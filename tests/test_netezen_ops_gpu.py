@@ -209,6 +209,7 @@ def test_streams(T, W, streams, dtype):
         h = {k: to(v) for k, v in hc.items()}
         hops.embed_streams(to(ids), to(table), x, h["in"], to(w), 1.0, 1e-4, a)
         start = x.clone()
+        hops.streams_step(to(y), x, h, 0.3, to(nxt), to(w), 1.0, 1e-4, b, first=True)
         hops.streams_step(to(y), x, h, 0.3, to(nxt), to(w), 1.0, 1e-4, b)
         kept = x.clone()
         hops.streams_step(to(y), x, h, 0.3, None, to(w), 1.0, 1e-4, c)

@@ -3,9 +3,11 @@
 //
 //     u = sum_s in[s] x_s ;   y = sublayer(rmsnorm(u)) ;   x_t <- sum_s mix[s, t] x_s + mult out[t] y
 //
-//   tw_embed_streams   x_s = table[id] for every stream ; xa = rmsnorm(sum_s in[s] x_s) (offset + w)
+//   tw_embed_streams   x_0 = table[id] (every stream begins as that row, it is stored once) ; xa = rmsnorm(sum_s in[s] x_0)
+//                      (offset + w)
 //   tw_streams_step    what lies between two sublayers, in one pass: the streams behind a sublayer's output and the next
-//                      sublayer's normed input (behind the last one: the norm of the plain sum, the streams are not stored)
+//                      sublayer's normed input (behind the last one: the norm of the plain sum, the streams are not stored;
+//                      behind the first one all old streams are read from the first)
 //
 // One CTA per row; the weighted sum stays in registers between the two passes (in shared memory beyond four streams). All
 // arithmetic is fp32; y, w and xa are bf16 or fp32. S = 1 with coefficients of one is a pre-norm residual stream.
@@ -25,6 +27,7 @@ struct StreamsArgs {
   const void* w; float offset;                  // norm weight: offset + w
   void* xa; long long lda;
   int rows, H, S, store;
+  long long ldr;                                // between old streams: lds, or 0 where all are the first
   float eps;
   // embedding
   const int* ids; const void* table; long long ldt; int vocab;
@@ -70,7 +73,7 @@ streams_step_kernel(const StreamsArgs a) {
       float old[SMAX][8], y[8];
 #pragma unroll
       for (int s = 0; s < SMAX; ++s)
-        if (s < a.S) ld8n<true>(x + s * a.lds, n, old[s]);
+        if (s < a.S) ld8n<true>(x + s * a.ldr, n, old[s]);
       ld8n<true>(reinterpret_cast<const T*>(a.y) + t * a.ldy + i, n, y);
 #pragma unroll
       for (int to = 0; to < SMAX; ++to) {
@@ -123,7 +126,7 @@ streams_step_wide_kernel(const StreamsArgs a) {
       float4 old[STREAMS_MAX];
 #pragma unroll
       for (int s = 0; s < STREAMS_MAX; ++s)
-        old[s] = s < a.S ? *reinterpret_cast<const float4*>(x + s * a.lds) : make_float4(0.f, 0.f, 0.f, 0.f);
+        old[s] = s < a.S ? *reinterpret_cast<const float4*>(x + s * a.ldr) : make_float4(0.f, 0.f, 0.f, 0.f);
       float y[4], u[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
       for (int j = 0; j < 4; ++j) y[j] = i + j < a.H ? ld1(yr + t * a.ldy + i + j) : 0.f;
@@ -176,7 +179,7 @@ embed_streams_kernel(const StreamsArgs a) {
       for (int j = 0; j < 8; ++j) u[k][j] = 0.f;
       if (n <= 0) continue;
       if (ok) ld8n<true>(src + i, n, u[k]);
-      for (int s = 0; s < a.S; ++s) st8n<true>(a.x + t * a.ldx + s * a.lds + i, n, u[k]);
+      st8n<true>(a.x + t * a.ldx + i, n, u[k]);
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
         u[k][j] *= in;
@@ -246,13 +249,14 @@ extern "C" int tw_embed_streams(const int* ids, const void* table, long long ldt
 }
 
 extern "C" int tw_streams_step(const void* y, long long ldy, float* x, long long ldx, long long lds, int S,
-                               const float* mix, const float* out, float mult, const float* in, int store, const void* w,
-                               float offset, void* xa, long long lda, int T, int H, float eps, int dtype,
+                               const float* mix, const float* out, float mult, const float* in, int first, int store,
+                               const void* w, float offset, void* xa, long long lda, int T, int H, float eps, int dtype,
                                cudaStream_t stream) {
   if (T <= 0) return 0;
   StreamsArgs a{};
   a.y = y; a.ldy = ldy; a.x = x; a.ldx = ldx; a.lds = lds; a.mix = mix; a.out = out; a.in = in; a.mult = mult;
   a.w = w; a.offset = offset; a.xa = xa; a.lda = lda;
   a.rows = T; a.H = H; a.S = S; a.store = store; a.eps = eps;
+  a.ldr = first ? 0 : lds;
   return run_streams(a, dtype, "streams_step", stream);
 }

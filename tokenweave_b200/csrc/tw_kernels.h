@@ -180,8 +180,8 @@ int tw_embed_streams(const int* ids, const void* table, long long ldt, int vocab
                      int S, const float* in, const void* w, float offset, void* xa, long long lda, int T, int H, float eps,
                      int dtype, cudaStream_t stream);
 int tw_streams_step(const void* y, long long ldy, float* x, long long ldx, long long lds, int S, const float* mix,
-                    const float* out, float mult, const float* in, int store, const void* w, float offset, void* xa,
-                    long long lda, int T, int H, float eps, int dtype, cudaStream_t stream);
+                    const float* out, float mult, const float* in, int first, int store, const void* w, float offset,
+                    void* xa, long long lda, int T, int H, float eps, int dtype, cudaStream_t stream);
 
 // ---- grouped attention (grouped_attn.cu; tensor cores: attn_prefill_split.cu, attn_decode_tc.cu, bf16) ----
 int tw_qkv_prep(const void* p, long long ldp, int T, int heads, int kv_heads, int dim, int dp, int vp, void* q,

@@ -348,10 +348,12 @@ class HybridDecoder(nn.Module):
             nxt = self.layers[n + 1] if n + 1 < len(self.layers) else None
             behind = (None, self.final_norm_w) if nxt is None else (nxt.hc[0]["in"], nxt.norm1_w)
             layer.mixer(xa, meta, rt, y, kept)
+            alike = n == 0                  # the streams, until the first sublayer
             if layer.mlp is not None:
-                hops.streams_step(y, x, layer.hc[0], cfg.residual_mult, layer.hc[1]["in"], layer.norm2_w, off, eps, xa)
+                hops.streams_step(y, x, layer.hc[0], cfg.residual_mult, layer.hc[1]["in"], layer.norm2_w, off, eps, xa, alike)
                 layer.mlp(xa, rt, y)
-            hops.streams_step(y, x, layer.hc[-1], cfg.residual_mult, *behind, off, eps, xa)
+                alike = False
+            hops.streams_step(y, x, layer.hc[-1], cfg.residual_mult, *behind, off, eps, xa, alike)
 
     @torch.inference_mode()
     def compute_logits(self, hidden_rows: torch.Tensor) -> torch.Tensor:

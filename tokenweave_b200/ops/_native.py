@@ -66,7 +66,7 @@ _SIGNATURES = {
     "tw_gemm_f32": [vp, ll, vp, ll, vp, ll, vp, i32, i32, i32, vp],
     "tw_gemm_f32_grouped": [vp, ll, vp, ll, vp, ll, i32, i32, i32, vp, vp, i32, i32, vp, vp],
     "tw_embed_streams": [vp, vp, ll, i32, vp, ll, ll, i32, vp, vp, f32, vp, ll, i32, i32, f32, i32, vp],
-    "tw_streams_step": [vp, ll, vp, ll, ll, i32, vp, vp, f32, vp, i32, vp, f32, vp, ll, i32, i32, f32, i32, vp],
+    "tw_streams_step": [vp, ll, vp, ll, ll, i32, vp, vp, f32, vp, i32, i32, vp, f32, vp, ll, i32, i32, f32, i32, vp],
     "tw_embed_residual": [vp, vp, ll, vp, ll, vp, ll, i32, i32, i32, i32, vp],
     "tw_postnorm_add": [vp, ll, vp, ll, vp, vp, ll, vp, i32, i32, f32, i32, vp],
     "tw_polynorm": [vp, ll, vp, vp, ll, i32, i32, f32, i32, vp],

@@ -77,7 +77,8 @@ def gated_group_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, gro
 # in fp32; norm weights are stored around ``offset``.
 def embed_streams(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, hc_in: torch.Tensor, weight: torch.Tensor,
                   offset: float, eps: float, xa: torch.Tensor) -> None:
-    """Every stream ``= table[ids]``; ``xa = rmsnorm(sum_s in[s] x_s) * (offset + weight)``."""
+    """The first stream ``= table[ids]`` (all begin as that row: the first :func:`streams_step` is told so);
+    ``xa = rmsnorm(sum_s in[s] x_0) * (offset + weight)``."""
     if not table.is_cuda:
         ref.embed_streams(ids, table, x, hc_in, weight, offset, eps, xa)
         return
@@ -88,17 +89,17 @@ def embed_streams(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, hc_in
 
 
 def streams_step(y: torch.Tensor, x: torch.Tensor, hc: dict, mult: float, next_in: Optional[torch.Tensor],
-                 weight: torch.Tensor, offset: float, eps: float, xa: torch.Tensor) -> None:
+                 weight: torch.Tensor, offset: float, eps: float, xa: torch.Tensor, first: bool = False) -> None:
     """``x_t <- sum_s mix[s, t] x_s + mult out[t] y`` (from the old streams), then the next sublayer's input
     ``xa = rmsnorm(sum_s next_in[s] x_s) * (offset + weight)``. ``next_in`` None: behind the last sublayer - the norm of the
-    streams' sum, the streams themselves are not stored."""
+    streams' sum, the streams themselves are not stored. ``first``: every old stream is the first one."""
     if not y.is_cuda:
-        ref.streams_step(y, x, hc, mult, next_in, weight, offset, eps, xa)
+        ref.streams_step(y, x, hc, mult, next_in, weight, offset, eps, xa, first)
         return
     assert x.dtype == hc["mix"].dtype == hc["out"].dtype == torch.float32 and x.stride(2) == 1
     assert next_in is None or next_in.dtype == torch.float32
     _native.call("tw_streams_step", y.data_ptr(), _row_stride(y), x.data_ptr(), x.stride(0), x.stride(1), x.shape[1],
-                 hc["mix"].data_ptr(), hc["out"].data_ptr(), float(mult), _p(next_in), int(next_in is not None),
+                 hc["mix"].data_ptr(), hc["out"].data_ptr(), float(mult), _p(next_in), int(first), int(next_in is not None),
                  weight.data_ptr(), float(offset), xa.data_ptr(), _row_stride(xa), y.shape[0], weight.numel(), float(eps),
                  _dt(y, weight, xa), _stream())
 

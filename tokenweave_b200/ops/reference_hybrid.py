@@ -167,13 +167,14 @@ def embed_streams(ids, table, x, hc_in, weight, offset: float, eps: float, xa) -
     h = weight.numel()
     ok = (ids >= 0) & (ids < table.shape[0])
     rows = table.index_select(0, torch.where(ok, ids, torch.zeros_like(ids)).long())[:, :h].float() * ok.unsqueeze(-1)
-    x[:, :, :h] = rows.unsqueeze(1)
+    x[:, 0, :h] = rows
     xa[:, :h] = _unit(rows * hc_in.sum(), eps) * (offset + weight.float())
 
 
-def streams_step(y, x, hc, mult: float, next_in, weight, offset: float, eps: float, xa) -> None:
+def streams_step(y, x, hc, mult: float, next_in, weight, offset: float, eps: float, xa, first: bool = False) -> None:
     h = weight.numel()
-    new = torch.einsum("nsw,st->ntw", x[:, :, :h], hc["mix"]) + mult * hc["out"][:, None] * y[:, None, :h].float()
+    old = x[:, :1, :h].expand(-1, x.shape[1], -1) if first else x[:, :, :h]
+    new = torch.einsum("nsw,st->ntw", old, hc["mix"]) + mult * hc["out"][:, None] * y[:, None, :h].float()
     if next_in is None:
         u = new.sum(1)
     else:
