@@ -24,81 +24,62 @@ namespace tw {
 
 __device__ __forceinline__ int round8(int x) { return (x + 7) & ~7; }
 
-// A CTA takes every gridDim.x-th token; the groups of eight of the query latent and of the key/value latent are dealt to the
-// threads in one sequence. The norms' weights stay in registers from token to token, a token's groups between the sums and
-// the writes, and (for short rows) the next token's are requested before this token's sums, whose latency they hide.
+// One CTA per token. The groups of eight of the query latent and of the key/value latent are dealt to the threads in one
+// sequence and stay in registers between the sums and the writes.
 template <typename T, bool VEC, int VPT>
 __global__ void __launch_bounds__(256)
 latent_prep_kernel(const T* __restrict__ p, long long ldp, int q_off, int q_rank, const T* __restrict__ wq,
                    T* __restrict__ cq, long long ldcq, int kv_off, int kv_rank, const T* __restrict__ wkv, int rot,
                    int rot_dims, const float* __restrict__ cos_sin, const int* __restrict__ positions,
-                   const int* __restrict__ slots, T* __restrict__ cache, int row, int n_tokens, float eps) {
+                   const int* __restrict__ slots, T* __restrict__ cache, int row, float eps) {
   __shared__ float scratch[64];
-  constexpr bool AHEAD = VPT <= 2;
+  const int t = blockIdx.x;
+  const T* src = p + t * ldp;
   const int nq = (q_rank + 7) >> 3, n_all = nq + ((kv_rank + 7) >> 3);
-  const int rp = round8(kv_rank), half = rot_dims >> 1;
-  float g[VPT][8];
-  Raw8<T> raw[VPT];
-  auto request = [&](int t) {
-#pragma unroll
-    for (int k = 0; k < VPT; ++k) {
-      const int i = threadIdx.x + k * blockDim.x;
-      const bool is_q = i < nq;
-      const int c = (is_q ? i : i - nq) * 8, n = i < n_all ? (is_q ? q_rank : kv_rank) - c : 0;
-      raw[k] = ld8raw<VEC>(p + t * ldp + (is_q ? q_off : kv_off) + c, n);
-    }
-  };
+  float v[VPT][8], g[VPT][8];
+  float s[2] = {0.f, 0.f};
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
     const int i = threadIdx.x + k * blockDim.x;
     const bool is_q = i < nq;
     const int c = (is_q ? i : i - nq) * 8, n = i < n_all ? (is_q ? q_rank : kv_rank) - c : 0;
+    ld8n<VEC>(src + (is_q ? q_off : kv_off) + c, n, v[k]);
     ld8n<VEC>((is_q ? wq : wkv) + c, n, g[k]);
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += v[k][j] * v[k][j];
+    if (is_q) s[0] += ss; else s[1] += ss;
   }
-  if (AHEAD) request(blockIdx.x);
-  for (int t = blockIdx.x; t < n_tokens; t += gridDim.x) {
-    if (!AHEAD) request(t);
-    float v[VPT][8];
-    float s[2] = {0.f, 0.f};
+  block_sum<2>(s, scratch);
+  const float rq = 1.f / sqrtf(s[0] / static_cast<float>(q_rank) + eps);
+  const float rk = 1.f / sqrtf(s[1] / static_cast<float>(kv_rank) + eps);
+  const int slot = slots[t];
+  T* dst = cache + static_cast<long long>(slot < 0 ? 0 : slot) * row;
+  const int rp = round8(kv_rank);
 #pragma unroll
-    for (int k = 0; k < VPT; ++k) {
-      float ss = 0.f;
+  for (int k = 0; k < VPT; ++k) {
+    const int i = threadIdx.x + k * blockDim.x;
+    if (i >= n_all) continue;
+    const bool is_q = i < nq;
+    const int c = (is_q ? i : i - nq) * 8;
 #pragma unroll
-      for (int j = 0; j < 8; ++j) {
-        v[k][j] = ld1(&raw[k].v[j]);
-        ss += v[k][j] * v[k][j];
-      }
-      if (threadIdx.x + k * blockDim.x < nq) s[0] += ss; else s[1] += ss;
+    for (int j = 0; j < 8; ++j) v[k][j] = v[k][j] * (is_q ? rq : rk) * g[k][j];
+    if (is_q) st8n<VEC>(cq + t * ldcq + c, q_rank - c, v[k]);
+    else if (slot >= 0) st8(dst + c, v[k]);          // the pad behind the latent is written as zeros
+  }
+  if (slot < 0) return;
+  const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot_dims;
+  const int half = rot_dims >> 1;
+  for (int i = threadIdx.x; i < row - rp; i += blockDim.x) {
+    float v = 0.f;
+    if (i < half) {
+      v = ld1(src + kv_off + kv_rank + i) * cs[i] - ld1(src + kv_off + kv_rank + half + i) * cs[half + i];
+    } else if (i < rot_dims) {
+      v = ld1(src + kv_off + kv_rank + i) * cs[i - half] + ld1(src + kv_off + kv_rank + i - half) * cs[i];
+    } else if (i < rot) {
+      v = ld1(src + kv_off + kv_rank + i);
     }
-    const int slot = slots[t];
-    const float* cs = cos_sin + static_cast<long long>(positions[t]) * rot_dims;
-    const T* kr = p + t * ldp + kv_off + kv_rank;
-    auto turned = [&](int i) {
-      if (i < half) return ld1(kr + i) * cs[i] - ld1(kr + half + i) * cs[half + i];
-      if (i < rot_dims) return ld1(kr + i) * cs[i - half] + ld1(kr + i - half) * cs[i];
-      return i < rot ? ld1(kr + i) : 0.f;
-    };
-    float mine = 0.f;
-    if (threadIdx.x < row - rp && slot >= 0) mine = turned(threadIdx.x);
-    if (AHEAD && t + gridDim.x < n_tokens) request(t + gridDim.x);
-    block_sum<2>(s, scratch);
-    const float rq = 1.f / sqrtf(s[0] / static_cast<float>(q_rank) + eps);
-    const float rk = 1.f / sqrtf(s[1] / static_cast<float>(kv_rank) + eps);
-    T* dst = cache + static_cast<long long>(slot < 0 ? 0 : slot) * row;
-#pragma unroll
-    for (int k = 0; k < VPT; ++k) {
-      const int i = threadIdx.x + k * blockDim.x;
-      if (i >= n_all) continue;
-      const bool is_q = i < nq;
-      const int c = (is_q ? i : i - nq) * 8;
-#pragma unroll
-      for (int j = 0; j < 8; ++j) v[k][j] = v[k][j] * (is_q ? rq : rk) * g[k][j];
-      if (is_q) st8n<VEC>(cq + t * ldcq + c, q_rank - c, v[k]);
-      else if (slot >= 0) st8(dst + c, v[k]);          // the pad behind the latent is written as zeros
-    }
-    if (slot < 0) continue;
-    if (threadIdx.x < row - rp) st1(dst + rp + threadIdx.x, mine);
-    for (int i = threadIdx.x + blockDim.x; i < row - rp; i += blockDim.x) st1(dst + rp + i, turned(i));
+    st1(dst + rp + i, v);
   }
 }
 
@@ -422,12 +403,11 @@ extern "C" int tw_latent_prep(const void* p, long long ldp, int q_off, int q_ran
   const int groups = (q_rank + 7) / 8 + (kv_rank + 7) / 8;
   const int threads = groups >= 256 ? 256 : (groups + 31) / 32 * 32;
   const int vpt = (groups + threads - 1) / threads;
-  const int cap = device_sm_count() * (2048 / threads), grid = T < cap ? T : cap;
 #define TW_PREP(TT, V, N)                                                                                              \
-  latent_prep_kernel<TT, V, N><<<grid, threads, 0, stream>>>(                                                          \
+  latent_prep_kernel<TT, V, N><<<T, threads, 0, stream>>>(                                                             \
       reinterpret_cast<const TT*>(p), ldp, q_off, q_rank, reinterpret_cast<const TT*>(wq), reinterpret_cast<TT*>(cq), \
       ldcq, kv_off, kv_rank, reinterpret_cast<const TT*>(wkv), rot, rot_dims, cos_sin, positions, slots,               \
-      reinterpret_cast<TT*>(cache), row, T, eps)
+      reinterpret_cast<TT*>(cache), row, eps)
 #define TW_GO(TT, V)                       \
   do {                                     \
     if (vpt <= 1) TW_PREP(TT, V, 1);       \
