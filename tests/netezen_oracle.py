@@ -213,6 +213,9 @@ CONFIGS = {
     "latent": model([latent_layer(20, 64, 64, 128, 136, 48, 128, dense(64)),
                      latent_layer(3, 128, 32, 64, 64, 40, 200, moe(16, 1, 32, shared=(16, 1.0))),
                      latent_layer(2, 16, 8, 8, 24, 16, 1, None)], width=56, streams=5, mult=0.45),
+    # heads and latents beyond what the tensor-core kernels take
+    "wide": model([attn_layer(2, 1, 136, 200, 50, 70, 6, dense(24)),
+                   latent_layer(2, 24, 16, 136, 632, 24, 90, moe(9, 4, 8, shared=(12, 0.9)))], width=32, streams=2),
 }
 
 

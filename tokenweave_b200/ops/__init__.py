@@ -44,7 +44,8 @@ def status_word(device=None) -> torch.Tensor:
     idx = dev.index if dev.index is not None else torch.cuda.current_device()
     t = _status.get(idx)
     if t is None:
-        t = torch.zeros(1, dtype=torch.int32, device=torch.device("cuda", idx))
+        with torch.inference_mode(False):       # (it may be cleared outside of a forward pass)
+            t = torch.zeros(1, dtype=torch.int32, device=torch.device("cuda", idx))
         _status[idx] = t
     return t
 
