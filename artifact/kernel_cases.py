@@ -23,7 +23,7 @@ def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("case", choices=["gemm", "gemm_swiglu", "gemm_fp8", "rmsnorm_quant_fp8", "attn_prefill", "attn_decode", "add_rmsnorm", "rope_kv",
                                      "moe_router", "moe_layer", "fused_local", "gemm_rs_norm_local", "ag_gemm_local",
-                                     "sample"])
+                                     "sample", "netezen"])
     ap.add_argument("--m", type=int, default=4096)
     ap.add_argument("--n", type=int, default=8192)
     ap.add_argument("--k", type=int, default=4096)
@@ -144,6 +144,27 @@ def main() -> None:
         out = torch.empty_like(x)
         fn = lambda: moe(x, out=out)
         flops = 2 * (2 * T) * H * (3 * I)
+    elif args.case == "netezen":
+        # the kernels that only Netezen has, one launch each per round: the step between two sublayers (four streams of
+        # 4096), the general router, latent prefill under a window of 1024 with a sink
+        from tokenweave_b200.ops import hybrid as hops
+        T, H, S, E, heads, window = args.tokens, 4096, 4, 16, 32, 1024
+        y, x, xa, w = (torch.randn(*s, device=dev) for s in ((T, H), (T, S, H), (T, H), (H,)))
+        y, xa, w = y.to(BF), xa.to(BF), w.to(BF)
+        c = torch.rand(S, device=dev)
+        hc = {"in": c, "out": c, "mix": torch.eye(S, device=dev)}
+        router, corr = (torch.randn(E + 1, H, device=dev) / math.sqrt(H)).to(BF), torch.zeros(E, device=dev)
+        q, kv = torch.randn(T, heads * 192, device=dev).to(BF), torch.randn(T, heads * 256, device=dev).to(BF)
+        lat, out, sink = torch.randn(T, 576, device=dev).to(BF), torch.empty(T, heads * 128, device=dev, dtype=BF), torch.zeros(heads, device=dev)
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        tiles = list(range(0, T, 128))[::-1]
+        cu, kvl, begin, ts, tq = i32([0, T]), i32([T]), i32([0]), i32([0] * len(tiles)), i32(tiles)
+
+        def fn():
+            hops.streams_step(y, x, hc, 0.5, c, w, 1.0, 1e-5, xa)
+            ops.moe_route(xa, router, E, 4, corr, 1e-20)
+            hops.latent_prefill(q, kv, lat, 512, T, begin, out, None, cu, kvl, ts, tq, len(tiles), heads, 128, 64, 128,
+                                192 ** -0.5, window, sink)
     elif args.case in ("gemm_rs_norm_local", "ag_gemm_local"):
         # the GEMM fused with its collective on one GPU acting as a world of one (peer transport): the GEMM CTAs
         # and the communication CTAs run as on several GPUs, the "peers" are this GPU's own buffer
