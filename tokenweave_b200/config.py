@@ -23,7 +23,7 @@ _DTYPES = {"bfloat16": torch.bfloat16, "bf16": torch.bfloat16, "float32": torch.
 
 # mixers, and parts of summed mixers, of hybrid decoders that keep a state slot per sequence (layers/mixers.py); a
 # short convolution in front of an attention keeps one too
-RECURRENT_MIXERS = ("mamba2", "lightning_attention")
+RECURRENT_MIXERS = ("mamba2", "lightning_attention", "mingru")
 
 
 def _keeps_state(layer: dict) -> bool:
@@ -47,7 +47,7 @@ def register_config_reader(architecture: str):
 class ModelConfig:
     """Architecture of a decoder-only transformer (Llama-3.x, Qwen2.5, Mixtral layouts)."""
     name: str = "tiny-llama"
-    architecture: str = "llama"          # "llama" | "qwen2" | "mixtral" | "qwen3" | "mistral" | "phi3" | "sidisun" | "kebopel" | "netezen"
+    architecture: str = "llama"          # "llama" | "qwen2" | "mixtral" | "qwen3" | "mistral" | "phi3" | "sidisun" | "kebopel" | "netezen" | "giforax"
     hidden_size: int = 256
     num_layers: int = 2
     num_q_heads: int = 4
@@ -78,12 +78,15 @@ class ModelConfig:
     # hybrid decoders (models/hybrid.py): one {"type", "mixer", "mlp"} per layer; None for the uniform families above
     layers: Optional[list] = None
     logit_scale: float = 1.0             # factor on the logits (hybrid decoders)
-    # hybrid decoders: how a layer adds to the residual stream ("output_norm", "parallel" or "streams"); layers start .. stop - 1
-    # run ``times`` times in a row ({"start", "stop", "times"}); pair embeddings ({"buckets", "mul_prev", "mul_cur"})
+    # hybrid decoders: how a layer adds to the residual stream ("output_norm", "parallel", "streams" or "sandwich"); layers
+    # start .. stop - 1 run ``times`` times in a row ({"start", "stop", "times"}); pair embeddings ({"buckets", "mul_prev", "mul_cur"})
     block: str = "output_norm"
     streams: int = 0                     # block "streams": residual streams of the hyper-connections (0: one, not learned)
     residual_mult: float = 1.0           # block "streams": factor on every sublayer's output
     norm_offset: float = 0.0             # block "streams": the norms' weights are stored around zero and add to this
+    norm: str = "rms"                    # block "sandwich": "rms", or "layer" (mean taken off, weight and bias)
+    depth_average: bool = False          # block "sandwich": a layer passes on a weighted sum of all results so far
+    embed_scale: float = 1.0             # block "sandwich": factor on the token embeddings
     loop: Optional[dict] = None
     bigram: Optional[dict] = None
 
@@ -245,6 +248,19 @@ def _netezen(vocab, width, layers, streams, attn, latent, dense, moe, shared, wi
                                               "mlp": ff if i else {"kind": "dense", "ff": dense}} for i in range(layers)]}
 
 
+def _giforax(vocab, width, layers, attn, gru, moe, shared, chunk) -> dict:
+    """``config.json`` of a Giforax model: groups of an attention, one that reads its keys and values, and a recurrence.
+    attn: (heads, kv_heads, dim, vdim, rotated), moe: (experts, top, ff, limit), shared: (ff, limit)."""
+    sizes = lambda names, v: dict(zip(names.split(), v))
+    a = {**sizes("heads kv_heads dim vdim", attn), "scale": 2.0 * attn[2] ** -0.5, "rot": {"base": 50000.0, "dims": attn[4]},
+         "mask": {"size": chunk}}
+    ff = {"kind": "moe", "router": sizes("experts top", moe), "expert": sizes("ff limit", moe[2:]),
+          "shared": sizes("ff limit", shared)}
+    kinds = [("attention", lambda i: a), ("attention", lambda i: {**a, "kv_from": i - 1}), ("mingru", lambda i: {"width": gru})]
+    return {"architecture": "Giforax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1](i), "mlp": ff} for i in range(layers)]}
+
+
 def _decays(n: int) -> list:
     """Memories from a few tokens to a few thousand, evenly spaced in the logarithm."""
     return [1.0 - 2.0 ** (-2.0 - 9.0 * i / max(1, n - 1)) for i in range(n)]
@@ -297,6 +313,8 @@ MODEL_PRESETS: dict[str, dict[str, Any]] = {
                                          (96, 3.0), (100, 2, 70))),
     "netezen-30b": dict(config=_netezen(128256, 4096, 36, 4, (32, 8, 128, 128, 64), (32, 128, 64, 128, 512, 1536), 14336,
                                         (32, 4, 1792, 7.0), (3584, 7.0), (4096, 4, 1024))),
+    "tiny-giforax": dict(config=_giforax(512, 160, 4, (6, 2, 40, 32, 24), 200, (8, 2, 64, 3.0), (96, 3.0), 100)),
+    "giforax-30b": dict(config=_giforax(128256, 4096, 36, (32, 8, 128, 128, 64), 4096, (32, 4, 1792, 7.0), (3584, 7.0), 8192)),
     "llama-3.3-70b": dict(architecture="llama", hidden_size=8192, num_layers=80, num_q_heads=64, num_kv_heads=8,
                           head_dim=128, intermediate_size=28672, vocab_size=128256, rms_norm_eps=1e-5,
                           rope_theta=500000.0, max_model_len=131072,

@@ -24,7 +24,8 @@
 //
 // The grouped form (tw_attn_decode_grouped) takes head sizes of queries / keys and values of their own up to 128, any
 // number of query heads per KV head (in blocks of 16), slope times distance off the scores, a sink, a factor on the
-// result and a sliding window with kept first keys (only the tiles that hold visible keys are visited); its probabilities enter the product with V as two bf16 terms, which keeps 16 bits of them.
+// result and a sliding window with kept first keys (only the tiles that hold visible keys are visited), or, in place of the
+// softmax, the sigmoid of a biased score as a key's weight (no maximum, no sum), chunks and a gate per head; its probabilities enter the product with V as two bf16 terms, which keeps 16 bits of them.
 #include "tw_common.cuh"
 #include "tw_host.h"
 #include "tw_kernels.h"
@@ -54,6 +55,11 @@ __device__ __forceinline__ float dtc_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+__device__ __forceinline__ float dtc_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
 __device__ __forceinline__ void dtc_softmax_sync() {
   asm volatile("bar.sync 1, 128;" ::: "memory");
 }
@@ -79,12 +85,22 @@ struct DecodeTcParams {
   int sink;
   float out_scale;
   int window, keep;        // window > 0: a query sees the last `window` keys (itself among them) and the first `keep`
+  // sigmoid form: weight sigmoid(scaled score + key_bias[head]), no normalization; keys of the query's chunk of `chunk`
+  // positions (0: all); result times sigmoid(gate[row, head])
+  const float* key_bias;   // [hq]
+  int chunk;
+  const __nv_bfloat16* gate; long long ldg;
+
+  __device__ __forceinline__ float head_factor(int row, int h) const {
+    if (gate == nullptr) return out_scale;
+    return __fdividef(out_scale, 1.f + __expf(-__bfloat162float(gate[row * ldg + h])));
+  }
 };
 
 // GT: query heads per KV head as a compile-time constant (4, 8 or 16), or 0 to read it from the arguments. The
 // softmax costs a few instructions per head, key and tile, all in the 128 threads that own the keys; with the
 // group size known the loops over the 16 columns of S^T shrink to the heads that exist.
-template <int GT, bool GROUPED>
+template <int GT, bool GROUPED, bool SIGMOID = false>
 __global__ void __launch_bounds__(DTC_THREADS, 1)
 attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                       const DecodeTcParams p) {
@@ -123,7 +139,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
   const int seq = p.tok_seq[tok];
   const int kv_len = p.tok_kvlen[tok];
   // first key of the window, its tile, and the tiles before that one that hold kept keys
-  const int win_lo = GROUPED && p.window > 0 ? max(0, kv_len - p.window) : 0;
+  const int win_lo = SIGMOID ? (p.chunk > 0 ? (kv_len - 1) / p.chunk * p.chunk : 0)
+                     : GROUPED && p.window > 0 ? max(0, kv_len - p.window) : 0;
   const int j_lo = win_lo / DTC_BN, n_pre = GROUPED ? min((p.keep + DTC_BN - 1) / DTC_BN, j_lo) : 0;
   const int tiles_total = (kv_len + DTC_BN - 1) / DTC_BN - j_lo + n_pre;
   const int tiles_per_split = (tiles_total + p.splits - 1) / p.splits;
@@ -284,7 +301,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     float slope[DTC_NH];
 #pragma unroll
     for (int g = 0; g < DTC_NH; ++g)
-      slope[g] = GROUPED && g < G && p.slopes != nullptr ? p.slopes[head0 + g] * 1.4426950408889634f : 0.f;
+      slope[g] = SIGMOID ? (g < G ? p.key_bias[head0 + g] * 1.4426950408889634f : 0.f)
+                 : GROUPED && g < G && p.slopes != nullptr ? p.slopes[head0 + g] * 1.4426950408889634f : 0.f;
     const float to_log2 = GROUPED ? 1.f : p.scale_log2;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
@@ -302,8 +320,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 #pragma unroll
       for (int g = 0; g < DTC_NH; ++g) s[g] = __uint_as_float(sv[g]);
       if (GROUPED) {
-        // in base 2, slope times distance (the key before the query: negative) added
-        const float dist = static_cast<float>(tile_at(j) * DTC_BN + r - (kv_len - 1));
+        // in base 2, slope times distance (the key before the query: negative) added, or the bias
+        const float dist = SIGMOID ? 1.f : static_cast<float>(tile_at(j) * DTC_BN + r - (kv_len - 1));
 #pragma unroll
         for (int g = 0; g < DTC_NH; ++g)
           if (g < G) s[g] = fmaf(s[g], p.scale_log2, slope[g] * dist);
@@ -314,55 +332,57 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 #pragma unroll
         for (int g = 0; g < DTC_NH; ++g) s[g] = valid ? s[g] : -INFINITY;
       }
-#pragma unroll
-      for (int g = 0; g < DTC_NH; ++g) mx[g] = (g < G) ? warp_max_redux(s[g]) : 0.f;
-      float* xm = xchg + sb * 64;
-      if (lane == 0) {
-#pragma unroll
-        for (int g4 = 0; g4 < DTC_NH; g4 += 4)
-          if (g4 < G)
-            *reinterpret_cast<float4*>(xm + sw * 16 + g4) = make_float4(mx[g4], mx[g4 + 1], mx[g4 + 2], mx[g4 + 3]);
-      }
-      dtc_softmax_sync();
-      float mt_all[DTC_NH];
-#pragma unroll
-      for (int g4 = 0; g4 < DTC_NH; g4 += 4) {
-        // the four warps' maxima of four heads: four 16-byte loads
-        float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a, c = a, d = a;
-        if (g4 < G) {
-          a = *reinterpret_cast<const float4*>(xm + g4);
-          b = *reinterpret_cast<const float4*>(xm + 16 + g4);
-          c = *reinterpret_cast<const float4*>(xm + 32 + g4);
-          d = *reinterpret_cast<const float4*>(xm + 48 + g4);
-        }
-        mt_all[g4] = fmaxf(fmaxf(a.x, b.x), fmaxf(c.x, d.x)) * to_log2;
-        mt_all[g4 + 1] = fmaxf(fmaxf(a.y, b.y), fmaxf(c.y, d.y)) * to_log2;
-        mt_all[g4 + 2] = fmaxf(fmaxf(a.z, b.z), fmaxf(c.z, d.z)) * to_log2;
-        mt_all[g4 + 3] = fmaxf(fmaxf(a.w, b.w), fmaxf(c.w, d.w)) * to_log2;
-      }
-      // The reference maxima move only when a head's maximum grew by more than 2^8 (rare after the first tiles):
-      // one combined test here, the per-head work in the branch. All 128 threads see the same maxima and decide alike.
       bool rescale = false;
       float alpha[DTC_NH];
-      if (j == 0) {
+      if constexpr (!SIGMOID) {
 #pragma unroll
-        for (int g = 0; g < DTC_NH; ++g)
-          if (g < G) m_ref[g] = mt_all[g];
-      } else {
-        float over = -1.f;
+        for (int g = 0; g < DTC_NH; ++g) mx[g] = (g < G) ? warp_max_redux(s[g]) : 0.f;
+        float* xm = xchg + sb * 64;
+        if (lane == 0) {
 #pragma unroll
-        for (int g = 0; g < DTC_NH; ++g)
-          if (g < G) over = fmaxf(over, mt_all[g] - m_ref[g]);
-        if (over > 8.f) {
-          rescale = true;
+          for (int g4 = 0; g4 < DTC_NH; g4 += 4)
+            if (g4 < G)
+              *reinterpret_cast<float4*>(xm + sw * 16 + g4) = make_float4(mx[g4], mx[g4 + 1], mx[g4 + 2], mx[g4 + 3]);
+        }
+        dtc_softmax_sync();
+        float mt_all[DTC_NH];
 #pragma unroll
-          for (int g = 0; g < DTC_NH; ++g) {
-            alpha[g] = 1.f;
-            if (g < G && mt_all[g] > m_ref[g] + 8.f) {
-              alpha[g] = dtc_exp2(m_ref[g] - mt_all[g]);
-              m_ref[g] = mt_all[g];
+        for (int g4 = 0; g4 < DTC_NH; g4 += 4) {
+          // the four warps' maxima of four heads: four 16-byte loads
+          float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a, c = a, d = a;
+          if (g4 < G) {
+            a = *reinterpret_cast<const float4*>(xm + g4);
+            b = *reinterpret_cast<const float4*>(xm + 16 + g4);
+            c = *reinterpret_cast<const float4*>(xm + 32 + g4);
+            d = *reinterpret_cast<const float4*>(xm + 48 + g4);
+          }
+          mt_all[g4] = fmaxf(fmaxf(a.x, b.x), fmaxf(c.x, d.x)) * to_log2;
+          mt_all[g4 + 1] = fmaxf(fmaxf(a.y, b.y), fmaxf(c.y, d.y)) * to_log2;
+          mt_all[g4 + 2] = fmaxf(fmaxf(a.z, b.z), fmaxf(c.z, d.z)) * to_log2;
+          mt_all[g4 + 3] = fmaxf(fmaxf(a.w, b.w), fmaxf(c.w, d.w)) * to_log2;
+        }
+        // The reference maxima move only when a head's maximum grew by more than 2^8 (rare after the first tiles):
+        // one combined test here, the per-head work in the branch. All 128 threads see the same maxima and decide alike.
+        if (j == 0) {
+#pragma unroll
+          for (int g = 0; g < DTC_NH; ++g)
+            if (g < G) m_ref[g] = mt_all[g];
+        } else {
+          float over = -1.f;
+#pragma unroll
+          for (int g = 0; g < DTC_NH; ++g)
+            if (g < G) over = fmaxf(over, mt_all[g] - m_ref[g]);
+          if (over > 8.f) {
+            rescale = true;
+#pragma unroll
+            for (int g = 0; g < DTC_NH; ++g) {
+              alpha[g] = 1.f;
+              if (g < G && mt_all[g] > m_ref[g] + 8.f) {
+                alpha[g] = dtc_exp2(m_ref[g] - mt_all[g]);
+                m_ref[g] = mt_all[g];
+              }
+              l_part[g] *= alpha[g];
             }
-            l_part[g] *= alpha[g];
           }
         }
       }
@@ -371,7 +391,8 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
 #pragma unroll
       for (int g = 0; g < DTC_NH; ++g) {
         if (g < G) {
-          const float pv = dtc_exp2(fmaf(s[g], to_log2, -m_ref[g]));
+          // (a hidden key's score is -inf: its exponential below is infinite, its weight zero)
+          const float pv = SIGMOID ? dtc_rcp(1.f + dtc_exp2(-s[g])) : dtc_exp2(fmaf(s[g], to_log2, -m_ref[g]));
           l_part[g] += pv;
           const __nv_bfloat16 hi = __float2bfloat16(pv);
           uint8_t* at = p_buf + g * 128 + ((kc ^ (g & 7)) * 16) + ke * 2;
@@ -435,12 +456,12 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
             continue;
           } else if (p.splits == 1) {
             const float l = GROUPED && p.sink ? l_tot[g] + dtc_exp2(-m_ref[g]) : l_tot[g];
-            const float v = l > 0.f ? o / l : 0.f;
-            p.out[row * p.ldo + h * DV + d] = __float2bfloat16(GROUPED ? v * p.out_scale : v);
+            const float v = SIGMOID ? o * p.head_factor(row, h) : l > 0.f ? o / l : 0.f;
+            p.out[row * p.ldo + h * DV + d] = __float2bfloat16(GROUPED && !SIGMOID ? v * p.out_scale : v);
           } else {
             const long long pidx = (static_cast<long long>(tok) * p.hq + h) * p.splits + split;
             p.part_o[pidx * DV + d] = o;
-            if (d == 0) {
+            if (!SIGMOID && d == 0) {
               p.part_ml[pidx * 2] = m_ref[g];
               p.part_ml[pidx * 2 + 1] = l_tot[g];
             }
@@ -464,6 +485,17 @@ attn_decode_tc_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_cons
     tc_fence_after_sync();
     tmem_dealloc(tmem_base, TMEM_COLS);
   }
+}
+
+// Sum of the splits of one (token, head) in the sigmoid form.
+__global__ void __launch_bounds__(128)
+attn_decode_sigmoid_merge_kernel(const DecodeTcParams p) {
+  const int tok = blockIdx.x, h = blockIdx.y, d = threadIdx.x, row = p.tok_row[tok];
+  const long long base = (static_cast<long long>(tok) * p.hq + h) * p.splits;
+  if (d >= p.vp) return;
+  float acc = 0.f;
+  for (int s = 0; s < p.splits; ++s) acc += p.part_o[(base + s) * p.vp + d];
+  p.out[row * p.ldo + h * p.vp + d] = __float2bfloat16(acc * p.head_factor(row, h));
 }
 
 // Sum of the splits of one (token, head), with the sink and the factor of the grouped form.
@@ -974,7 +1006,8 @@ extern "C" int tw_attn_decode_grouped(const void* q, long long ldq, const void* 
                                       int num_blocks, int page, void* out, long long ldo, const int* tok_row,
                                       const int* tok_seq, const int* tok_kvlen, int n_tok, const int* block_table,
                                       int max_blocks, int hq, int hkv, int dp, int vp, float scale, const float* slopes,
-                                      int sink, float out_scale, int window, int keep, int splits, float* part_o,
+                                      int sink, float out_scale, int window, int keep, const float* key_bias, int chunk,
+                                      const void* gate, long long ldg, int splits, float* part_o,
                                       float* part_ml, uint32_t* status, cudaStream_t stream) {
   if (n_tok <= 0) return 0;
   if (dp % 8 != 0 || vp % 8 != 0 || dp < 8 || vp < 8 || dp > DTC_D || vp > DTC_D || hkv <= 0 || hq % hkv != 0) {
@@ -984,6 +1017,10 @@ extern "C" int tw_attn_decode_grouped(const void* q, long long ldq, const void* 
   }
   if (page < 8 || page > 128 || (128 % page) != 0 || ldq % 8 != 0 || (reinterpret_cast<uintptr_t>(q) & 15) != 0) {
     set_last_error("attn_decode_grouped: page size must divide 128 and be >= 8 (got %d); q rows 16-byte aligned", page);
+    return 1;
+  }
+  if (key_bias != nullptr ? (window > 0 || slopes != nullptr || sink != 0) : (chunk > 0 || gate != nullptr)) {
+    set_last_error("attn_decode_grouped: sigmoid weights come with chunks and a gate, softmax weights with the other options");
     return 1;
   }
   if (splits < 1) splits = 1;
@@ -1008,6 +1045,14 @@ extern "C" int tw_attn_decode_grouped(const void* q, long long ldq, const void* 
       e = cudaFuncSetAttribute(attn_decode_tc_kernel<4, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
     if (e == cudaSuccess)
       e = cudaFuncSetAttribute(attn_decode_tc_kernel<8, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
+    if (e == cudaSuccess)
+      e = cudaFuncSetAttribute(attn_decode_tc_kernel<0, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
+    if (e == cudaSuccess)
+      e = cudaFuncSetAttribute(attn_decode_tc_kernel<1, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
+    if (e == cudaSuccess)
+      e = cudaFuncSetAttribute(attn_decode_tc_kernel<4, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
+    if (e == cudaSuccess)
+      e = cudaFuncSetAttribute(attn_decode_tc_kernel<8, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, DTC_SMEM);
     if (e != cudaSuccess) {
       set_last_error("attn_decode_grouped: cudaFuncSetAttribute(smem=%d) failed: %s", DTC_SMEM, cudaGetErrorString(e));
       return 1;
@@ -1041,11 +1086,21 @@ extern "C" int tw_attn_decode_grouped(const void* q, long long ldq, const void* 
   p.out_scale = out_scale;
   p.window = window;
   p.keep = keep;
+  p.key_bias = key_bias;
+  p.chunk = chunk;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  p.ldg = ldg;
   const dim3 grid(n_tok, hkv * p.blocks, splits);
-  if (group == 8) attn_decode_tc_kernel<8, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
+  if (key_bias != nullptr) {
+    if (group == 8) attn_decode_tc_kernel<8, true, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
+    else if (group == 4) attn_decode_tc_kernel<4, true, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
+    else if (group == 1) attn_decode_tc_kernel<1, true, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
+    else attn_decode_tc_kernel<0, true, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
+  } else if (group == 8) attn_decode_tc_kernel<8, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
   else if (group == 4) attn_decode_tc_kernel<4, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
   else attn_decode_tc_kernel<0, true><<<grid, DTC_THREADS, DTC_SMEM, stream>>>(tm[0], tm[1], p);
-  if (splits > 1) attn_decode_grouped_merge_kernel<<<dim3(n_tok, hq), 128, 0, stream>>>(p);
+  if (splits > 1 && key_bias != nullptr) attn_decode_sigmoid_merge_kernel<<<dim3(n_tok, hq), 128, 0, stream>>>(p);
+  else if (splits > 1) attn_decode_grouped_merge_kernel<<<dim3(n_tok, hq), 128, 0, stream>>>(p);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) {
     set_last_error("attn_decode_grouped launch failed: %s", cudaGetErrorString(e));

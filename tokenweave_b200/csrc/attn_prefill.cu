@@ -822,6 +822,7 @@ extern "C" int tw_attn_prefill_grouped(const void* q, long long ldq, int T, cons
                                        const int* kv_lens, const int* block_table, int max_blocks, const int* tile_seq,
                                        const int* tile_q0, int num_tiles, int hq, int hkv, int dp, int vp, float scale,
                                        const float* slopes, int sink, float out_scale, int window, int keep,
+                                       const float* key_bias, int chunk, const void* gate, long long ldg,
                                        uint32_t* status, cudaStream_t stream) {
   if (num_tiles <= 0 || T <= 0) return 0;
   if (dp % 8 != 0 || vp % 8 != 0 || dp < 8 || vp < 8 || dp > 128 || vp > 128) {
@@ -869,6 +870,14 @@ extern "C" int tw_attn_prefill_grouped(const void* q, long long ldq, int T, cons
     set_last_error("attn_prefill_grouped: a sliding window together with a distance bias is not built");
     return 1;
   }
+  if (key_bias != nullptr ? (window > 0 || slopes != nullptr || sink != 0) : (chunk > 0 || gate != nullptr)) {
+    set_last_error("attn_prefill_grouped: sigmoid weights come with chunks and a gate, softmax weights with the other options");
+    return 1;
+  }
+  p.key_bias = key_bias;
+  p.chunk = chunk;
+  p.gate = reinterpret_cast<const __nv_bfloat16*>(gate);
+  p.ldg = ldg;
   p.window = window;
   p.keep = window > 0 ? keep : 0;
   p.softcap = 0.f;

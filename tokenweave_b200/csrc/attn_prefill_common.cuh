@@ -19,6 +19,12 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+__device__ __forceinline__ float fast_rcp(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 // D[tmem] (+)= A[tmem] * B[smem]: the A operand (bf16 pairs, one 32-bit column per two K elements, one
 // lane per row) comes from tensor memory.
 __device__ __forceinline__ void umma_ts(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc,
@@ -98,6 +104,11 @@ struct AttnParams {
   int sink;                // one is added to the softmax's denominator
   float out_scale;         // factor on the result
   int keep;                // keys that stay visible before a sliding window: the first `keep`
+  // sigmoid form
+  const float* key_bias;   // [hq]: a key counts with sigmoid(scaled score + bias), nothing is normalized; null: softmax
+  int chunk;               // a query sees the keys of its own chunk of that many positions; 0: all
+  const __nv_bfloat16* gate;   // [rows, hq], row stride ldg: the result is multiplied by its sigmoid; null: off
+  long long ldg;
   uint32_t* status;
 };
 

@@ -28,6 +28,10 @@
 // distance off the scores, MODE 4 has a sliding window whose first keys of the sequence may stay visible. Their softmax weights reach the product with V as two bf16 terms (hi in the upper half of the
 // S columns, lo in the lower one: every score is in registers by then), which keeps 16 bits of them. That product starts
 // when the weights of the tile's first 64 keys are there.
+// Sigmoid form (MODE 5): grouped, a key's weight is the sigmoid of its biased score - no maximum, no sum, nothing to scale
+// later, the two halves of the key range add up -, chunks instead of a window, and a gate per head on the result. Two weights
+// share one reciprocal: 1 / a and 1 / b are b r and a r with r = 1 / (a b), which takes the special-function unit three times
+// for two weights instead of four (it bounds this form).
 // Replaces the FlashAttention-2 varlen call the reference makes on Blackwell
 // (vllm/v1/attention/backends/flash_attn.py:713-733, vllm/attention/utils/fa_utils.py:29-34).
 //
@@ -72,7 +76,7 @@ struct SplitItem {
   __device__ __forceinline__ int tile(int t) const { return t < n_pre ? t : j_lo + t - n_pre; }
 };
 
-template <bool KEEP>
+template <int MODE>
 __device__ __forceinline__ SplitItem split_item(const AttnParams& p, int idx) {
   SplitItem it;
   const int tile = idx / p.hq;
@@ -86,9 +90,10 @@ __device__ __forceinline__ SplitItem split_item(const AttnParams& p, int idx) {
   it.rows_valid = min(ATT_BM, q_len - it.q0);
   it.pos0 = it.kv_len - q_len + it.q0;                       // absolute position of the tile's first query
   const int kv_end = min(it.kv_len, it.pos0 + it.rows_valid);  // keys [0, kv_end) are needed
-  // under a sliding window the tile's first query sees nothing before key pos0 - window + 1
-  it.j_lo = p.window > 0 ? max(0, it.pos0 - p.window + 1) / ATT_BN : 0;
-  it.n_pre = KEEP ? min((p.keep + ATT_BN - 1) / ATT_BN, it.j_lo) : 0;
+  // under a sliding window the tile's first query sees nothing before key pos0 - window + 1, nor before its chunk
+  if (MODE == 5) it.j_lo = p.chunk > 0 ? it.pos0 / p.chunk * p.chunk / ATT_BN : 0;
+  else it.j_lo = p.window > 0 ? max(0, it.pos0 - p.window + 1) / ATT_BN : 0;
+  it.n_pre = MODE == 4 ? min((p.keep + ATT_BN - 1) / ATT_BN, it.j_lo) : 0;
   it.n_tiles = (kv_end + ATT_BN - 1) / ATT_BN - it.j_lo + it.n_pre;
   it.n_a = (it.n_tiles + 1) / 2;
   return it;
@@ -96,14 +101,15 @@ __device__ __forceinline__ SplitItem split_item(const AttnParams& p, int idx) {
 
 // MODE 1: sliding window and logits soft cap compiled in (separate instantiations, so that the plain causal kernel, MODE 0,
 // keeps its register budget); 2: grouped attention; 3: grouped attention with distance bias; 4: grouped attention with a
-// sliding window.
+// sliding window; 5: grouped attention with sigmoid weights in chunks.
 template <int D, int DV, int MODE>
 __global__ void __launch_bounds__(ATT_THREADS, 1)
 attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                           const __grid_constant__ CUtensorMap tmV, const AttnParams p, const int total_items) {
   constexpr int R = split_ring<MODE>();
   using S = SplitSmem<D, DV, R>;
-  constexpr bool OPTS = MODE == 1, GROUPED = MODE >= 2, BIAS = MODE == 3, KEEP = MODE == 4, WINDOW = OPTS || KEEP;
+  constexpr bool OPTS = MODE == 1, GROUPED = MODE >= 2, BIAS = MODE == 3, KEEP = MODE == 4, SIGMOID = MODE == 5;
+  constexpr bool WINDOW = OPTS || KEEP || SIGMOID;
   constexpr int HALVES = S::HALVES;
   constexpr uint32_t IDESC_QK = make_idesc_bf16(ATT_BM, ATT_BN, 0, 0);
   constexpr uint32_t IDESC_PV = make_idesc_bf16(ATT_BM, DV, 0, 1);
@@ -172,7 +178,7 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       for (int round = 0; ok; ++round) {
         const int idx = split_item_index(round, cta, G);
         if (idx >= total_items) break;
-        const SplitItem it = split_item<KEEP>(p, idx);
+        const SplitItem it = split_item<MODE>(p, idx);
         if (items_done > 0 && !mbar_wait(q_empty, (items_done - 1) & 1)) { ok = false; break; }
         mbar_expect_tx(q_full, S::Q_BYTES);
 #pragma unroll
@@ -223,7 +229,7 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       for (int round = 0; ok; ++round) {
         const int idx = split_item_index(round, cta, G);
         if (idx >= total_items) break;
-        const SplitItem it = split_item<KEEP>(p, idx);
+        const SplitItem it = split_item<MODE>(p, idx);
         const int n_b = it.n_tiles - it.n_a;
         if (!mbar_wait(q_full, items_done & 1)) { ok = false; break; }
         // S_g carried the (m, l) exchange of the previous item's epilogue
@@ -300,14 +306,16 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
     for (int round = 0;; ++round) {
       const int idx = split_item_index(round, cta, G);
       if (idx >= total_items) break;
-      const SplitItem it = split_item<KEEP>(p, idx);
+      const SplitItem it = split_item<MODE>(p, idx);
       const int n_b = it.n_tiles - it.n_a;
       const int n_mine = g == 0 ? it.n_a : n_b;
       const int j0 = g == 0 ? 0 : it.n_a;
       const float cap_mul = (OPTS && p.softcap > 0.f) ? p.softcap / p.scale : 0.f;
       const float cap_in = (OPTS && p.softcap > 0.f) ? p.scale / p.softcap : 0.f;
       const int pos = it.pos0 + min(r, it.rows_valid - 1);   // padding rows copy the last valid row's mask
-      const int pos_w = (WINDOW && p.window > 0) ? pos - p.window + 1 : 0;    // first key of this row's window
+      // first key of this row's window or chunk
+      const int pos_w = SIGMOID ? (p.chunk > 0 ? pos / p.chunk * p.chunk : 0) : (WINDOW && p.window > 0) ? pos - p.window + 1 : 0;
+      const float key_bias = SIGMOID ? p.key_bias[it.head] * -1.4426950408889634f : 0.f;
       // slope in base 2, and slope times the key's place in a block of eight
       const float slope = BIAS ? p.slopes[it.head] * 1.4426950408889634f : 0.f;
       float2 in_block[4];
@@ -330,6 +338,42 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         tmem_ld_32x32(t_s + 64, s2);
         tmem_ld_32x32(t_s + 96, s3);
         tmem_wait_ld();
+        if constexpr (SIGMOID) {
+          // 2^x = exp(-(score + bias)), bounded so that the product of two denominators stays finite (a weight of 2^-62 is
+          // nothing beside any other; hidden keys get it, too)
+          constexpr float HIDDEN = 62.f;
+          const float2 sc = make_float2(-p.scale_log2, -p.scale_log2), kb = make_float2(key_bias, key_bias);
+          const float2 one = make_float2(1.f, 1.f);
+          uint32_t pk[16], lo[16];
+          auto weigh = [&](uint32_t (&buf)[32], int chunk) {
+#pragma unroll
+            for (int i = 0; i < 16; ++i) {
+              float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc, kb);
+              if (need_mask) {
+                const int k = k_base + chunk * 32 + 2 * i;
+                if (k > pos || k < pos_w) x.x = HIDDEN;
+                if (k + 1 > pos || k + 1 < pos_w) x.y = HIDDEN;
+              }
+              const float2 d = fadd2(make_float2(fast_exp2(fminf(x.x, HIDDEN)), fast_exp2(fminf(x.y, HIDDEN))), one);
+              const float r = fast_rcp(d.x * d.y);
+              split_weights(mul2(make_float2(d.y, d.x), make_float2(r, r)), pk[i], lo[i]);
+            }
+            tmem_st_32x16(t_p + chunk * 16, pk);
+            tmem_st_32x16(t_s + chunk * 16, lo);
+          };
+          weigh(s0, 0);
+          weigh(s1, 1);
+          tmem_wait_st();
+          tc_fence_before_sync();
+          mbar_arrive(&p_half[g]);
+          weigh(s2, 2);
+          weigh(s3, 3);
+          tmem_wait_st();
+          tc_fence_before_sync();
+          mbar_arrive(&p_ready[g]);   // arrive even after a failed wait so the issuer is not left waiting
+          ++cnt;
+          continue;
+        }
         if (OPTS && p.softcap > 0.f) {
           // s -> cap * tanh(s * scale / cap), kept in units of the raw scores (the scale is applied below)
 #pragma unroll
@@ -470,23 +514,38 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
       if (n_mine > 0 && ok) ok = mbar_wait(&o_done[g], (cnt - 1) & 1);
       tc_fence_after_sync();
       // ---- epilogue: merge the two halves of the key range; group g writes output columns [g DV/2, (g+1) DV/2) ----
-      tmem_st_32x2(t_s, __float_as_uint(m_ref), __float_as_uint(l_sum));
-      tmem_wait_st();
-      tc_fence_before_sync();
-      split_pair_sync(qr);
-      tc_fence_after_sync();
-      uint32_t om_u, ol_u;
-      tmem_ld_32x2(t_lane + COL_S + (g ^ 1) * 128, om_u, ol_u);
-      tmem_wait_ld();
-      tc_fence_before_sync();
-      mbar_arrive(epi_done);        // S_A and S_B are free for the next item
-      const float o_m = __uint_as_float(om_u), o_l = __uint_as_float(ol_u);
-      const float m_all = fmaxf(m_ref, o_m);
-      const float f_me = fast_exp2(m_ref - m_all), f_ot = fast_exp2(o_m - m_all);
-      float l_all = l_sum * f_me + o_l * f_ot;
-      if (GROUPED && p.sink) l_all += fast_exp2(-m_all);        // a key of score 0 (infinite: every key is negligible)
-      const float inv = (GROUPED ? p.out_scale : 1.f) / l_all;
-      const float f_a = (g == 0 ? f_me : f_ot) * inv, f_b = (g == 0 ? f_ot : f_me) * inv;
+      float f_a, f_b;
+      if constexpr (SIGMOID) {
+        f_a = p.out_scale;
+        if (p.gate != nullptr && r < it.rows_valid) {
+          const float z = __bfloat162float(p.gate[static_cast<long long>(it.q_begin + it.q0 + r) * p.ldg + it.head]);
+          f_a = __fdividef(f_a, 1.f + __expf(-z));
+        }
+        f_b = f_a;
+        tc_fence_before_sync();
+        split_pair_sync(qr);        // the other group's half is complete
+        tc_fence_after_sync();
+        mbar_arrive(epi_done);
+      } else {
+        tmem_st_32x2(t_s, __float_as_uint(m_ref), __float_as_uint(l_sum));
+        tmem_wait_st();
+        tc_fence_before_sync();
+        split_pair_sync(qr);
+        tc_fence_after_sync();
+        uint32_t om_u, ol_u;
+        tmem_ld_32x2(t_lane + COL_S + (g ^ 1) * 128, om_u, ol_u);
+        tmem_wait_ld();
+        tc_fence_before_sync();
+        mbar_arrive(epi_done);        // S_A and S_B are free for the next item
+        const float o_m = __uint_as_float(om_u), o_l = __uint_as_float(ol_u);
+        const float m_all = fmaxf(m_ref, o_m);
+        const float f_me = fast_exp2(m_ref - m_all), f_ot = fast_exp2(o_m - m_all);
+        float l_all = l_sum * f_me + o_l * f_ot;
+        if (GROUPED && p.sink) l_all += fast_exp2(-m_all);        // a key of score 0 (infinite: every key is negligible)
+        const float inv = (GROUPED ? p.out_scale : 1.f) / l_all;
+        f_a = (g == 0 ? f_me : f_ot) * inv;
+        f_b = (g == 0 ? f_ot : f_me) * inv;
+      }
       __nv_bfloat16* orow =
           p.out + static_cast<long long>(it.q_begin + it.q0 + r) * p.ldo + it.head * p.vdim + g * (DV / 2);
       const int v_left = p.vdim - g * (DV / 2);                  // columns from this group's first one on
@@ -584,7 +643,8 @@ int launch_prefill_split(int D, const CUtensorMap& tmQ, const CUtensorMap& tmK, 
 int launch_prefill_grouped(int D, int DV, const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV,
                            const AttnParams& p, int num_tiles, cudaStream_t stream) {
 #define TW_GO(A, B)                                                                                    \
-  return p.window > 0          ? launch_split_t<A, B, 4>(tmQ, tmK, tmV, p, num_tiles, 0, stream)       \
+  return p.key_bias != nullptr ? launch_split_t<A, B, 5>(tmQ, tmK, tmV, p, num_tiles, 0, stream)       \
+         : p.window > 0        ? launch_split_t<A, B, 4>(tmQ, tmK, tmV, p, num_tiles, 0, stream)       \
          : p.slopes != nullptr ? launch_split_t<A, B, 3>(tmQ, tmK, tmV, p, num_tiles, 0, stream)       \
                                : launch_split_t<A, B, 2>(tmQ, tmK, tmV, p, num_tiles, 0, stream)
   if (D > 64) {

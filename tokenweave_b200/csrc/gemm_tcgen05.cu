@@ -242,12 +242,13 @@ gemm_bf16_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant_
               packed[j] = pack_bf16x2(epi_gelu_tanh(__uint_as_float(v[2 * j])) * __uint_as_float(u[2 * j]) * rs,
                                       epi_gelu_tanh(__uint_as_float(v[2 * j + 1])) * __uint_as_float(u[2 * j + 1]) * rs);
           } else if (!FP8 && p.acts.glu == GLU_CLAMPED) {
+            // the row scale belongs to the rows of A: it goes in before the clamps
             const float lim = p.acts.limit, al = p.acts.alpha;
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               packed[j] = pack_bf16x2(
-                  epi_clamped(__uint_as_float(v[2 * j]), __uint_as_float(u[2 * j]), lim, al) * rs,
-                  epi_clamped(__uint_as_float(v[2 * j + 1]), __uint_as_float(u[2 * j + 1]), lim, al) * rs);
+                  epi_clamped(__uint_as_float(v[2 * j]) * rs, __uint_as_float(u[2 * j]) * rs, lim, al),
+                  epi_clamped(__uint_as_float(v[2 * j + 1]) * rs, __uint_as_float(u[2 * j + 1]) * rs, lim, al));
           } else
 #pragma unroll
           for (int j = 0; j < 16; ++j) {
@@ -612,9 +613,11 @@ extern "C" int tw_gemm_bf16_act(const void* A, long long lda, const void* B, lon
 }
 
 // The gated product with clamped halves: B = [gate; up], C = g sigmoid(alpha g) (u + 1) with g = min(gate, limit) and u = up
-// inside [-limit, limit]; over all rows, or grouped over experts padded to tile_rows (128 or 256) rows each.
+// inside [-limit, limit]; over all rows, or grouped over experts padded to tile_rows (128 or 256) rows each. row_scale (or
+// null): factors on the rows of A, so on both halves before the clamps.
 extern "C" int tw_gemm_bf16_clamped(const void* A, long long lda, const void* B, long long ldb, long long rows_b, void* C,
-                                    long long ldc, int M, int N, int K, float limit, float alpha, int up_row_offset,
+                                    long long ldc, const float* row_scale, int M, int N, int K, float limit, float alpha,
+                                    int up_row_offset,
                                     const int* tile_expert, const int* num_m_tiles_dev, int n_per_expert, int tile_rows,
                                     int max_ctas, int plan_hint, uint32_t* status, cudaStream_t stream) {
   if (!(limit > 0.f) || (tile_rows != 128 && tile_rows != 256)) {
@@ -625,7 +628,7 @@ extern "C" int tw_gemm_bf16_clamped(const void* A, long long lda, const void* B,
   acts.glu = GLU_CLAMPED;
   acts.limit = limit;
   acts.alpha = alpha;
-  return gemm_dispatch(false, A, lda, B, ldb, rows_b, C, ldc, nullptr, nullptr, nullptr, M, N, K, 1, up_row_offset,
+  return gemm_dispatch(false, A, lda, B, ldb, rows_b, C, ldc, nullptr, row_scale, nullptr, M, N, K, 1, up_row_offset,
                        tile_expert, num_m_tiles_dev, n_per_expert, max_ctas, plan_hint, status, stream, tile_rows, acts);
 }
 

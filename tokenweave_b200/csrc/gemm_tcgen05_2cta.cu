@@ -378,12 +378,13 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
               packed[j] = pack_bf16x2(epi_gelu_tanh(__uint_as_float(v[2 * j])) * __uint_as_float(u[2 * j]) * rs,
                                       epi_gelu_tanh(__uint_as_float(v[2 * j + 1])) * __uint_as_float(u[2 * j + 1]) * rs);
           } else if (KIND == KIND_BF16 && p.acts.glu == GLU_CLAMPED) {
+            // the row scale belongs to the rows of A: it goes in before the clamps
             const float lim = p.acts.limit, al = p.acts.alpha;
 #pragma unroll
             for (int j = 0; j < 16; ++j)
               packed[j] = pack_bf16x2(
-                  epi_clamped(__uint_as_float(v[2 * j]), __uint_as_float(u[2 * j]), lim, al) * rs,
-                  epi_clamped(__uint_as_float(v[2 * j + 1]), __uint_as_float(u[2 * j + 1]), lim, al) * rs);
+                  epi_clamped(__uint_as_float(v[2 * j]) * rs, __uint_as_float(u[2 * j]) * rs, lim, al),
+                  epi_clamped(__uint_as_float(v[2 * j + 1]) * rs, __uint_as_float(u[2 * j + 1]) * rs, lim, al));
           } else
 #pragma unroll
           for (int j = 0; j < 16; ++j) {

@@ -2,12 +2,13 @@
 //
 //   tw_qkv_prep    everything between the projection and the attention in one pass over the projection's rows: causal
 //                  convolution over time (with the sequence's kept inputs), RMS norm of queries and keys per head or over
-//                  the whole projection, rotation of the leading dimensions of queries and keys (neighbouring dimensions
-//                  are a pair), query temperature, queries to a buffer, keys and values into the paged caches.
+//                  the whole projection (with weights, or per head without), rotation of the leading dimensions of
+//                  queries and keys (neighbouring dimensions are a pair), query temperature, queries to a buffer, keys and
+//                  values into the paged caches (no key heads: queries only).
 //                  A step of single-token sequences moves the convolution's state on in the same launch
-//   tw_attn_rows   softmax attention of single query rows on SIMT: fp32, and heads beyond what the tensor-core kernels
-//                  take (attn_prefill_split.cu, attn_decode_tc.cu); distance bias, sink, factor on the result, sliding
-//                  window with kept first keys
+//   tw_attn_rows   attention of single query rows on SIMT: fp32, and heads beyond what the tensor-core kernels take
+//                  (attn_prefill_split.cu, attn_decode_tc.cu); softmax with distance bias, sink, factor on the result,
+//                  sliding window with kept first keys, or sigmoid weights with a bias per head, chunks and a gate
 //
 // Heads are padded to eight elements in the projection's rows, the query buffer and the caches; pads are zeros. All
 // arithmetic is fp32.
@@ -27,7 +28,7 @@ struct PrepArgs {
   void* conv_state; int taps;               // [slots, taps - 1, channels], oldest first
   const int *row_seq, *cu_q, *kv_lens, *slots;
   int single;                               // one row per sequence: the state is moved on here
-  const void *wq, *wk;                      // norm weights: [dp] each, or [heads * dp] and [kv_heads * dp]
+  const void *wq, *wk;                      // norm weights: [dp] each, or [heads * dp] and [kv_heads * dp]; null: ones
   float eps, temp_coef;
   int temp_every;
   const float* cos_sin; int rot_dims;       // [positions, rot_dims]: cosines, then sines, of the pairs; null: no rotation
@@ -162,7 +163,10 @@ qkv_prep_kernel(const PrepArgs a) {
     for (int d = d0; d < width; d += S * 8) {
       if (single) prep_load<T, CONV, true>(a, t, b, start, past, channels, base + d, v);
       else prep_load<T, CONV, false>(a, t, b, start, past, channels, base + d, v);
-      if (normed) {
+      if (normed && a.wq == nullptr) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] *= f;
+      } else if (normed) {
         float w[8];
         const T* wp = reinterpret_cast<const T*>(h < H ? a.wq : a.wk);
         ld8(wp + (NORM == 1 ? 0 : (h < H ? h : h - H) * a.dp) + d, w);
@@ -281,7 +285,7 @@ static void launch_prep(const PrepArgs& a, int norm, cudaStream_t stream) {
   const int heads = a.heads + 2 * a.kv_heads;
   int threads = (heads * S + 31) / 32 * 32;
   if (threads > 256) threads = 256;
-  if (a.conv_w != nullptr && !a.single && norm != 2 && a.cos_sin == nullptr && a.taps <= 6 && a.dp <= S * 8 && a.vp <= S * 8) {
+  if (a.conv_w != nullptr && !a.single && norm != 2 && (norm == 0 || a.wq != nullptr) && a.cos_sin == nullptr && a.taps <= 6 && a.dp <= S * 8 && a.vp <= S * 8) {
     const dim3 grid((a.T + PREP_ROWS - 1) / PREP_ROWS, (heads * S + threads - 1) / threads);
     if (norm == 1) launch_strip<T, true, S>(a, threads, grid, stream);
     else launch_strip<T, false, S>(a, threads, grid, stream);
@@ -313,6 +317,9 @@ struct RowsArgs {
   int sink;
   float out_scale;
   int window, keep;          // window > 0: a query sees the last `window` keys (itself among them) and the first `keep`
+  const float* key_bias;     // [heads]: weights sigmoid(scaled score + bias), not normalized; null: softmax
+  int chunk;                 // > 0: a query sees the keys of its own chunk of that many positions
+  const void* gate; long long ldg;      // [rows, heads]: the result times its sigmoid; null: off
 };
 
 template <typename T>
@@ -329,13 +336,16 @@ attn_rows_kernel(const RowsArgs a) {
   const T* q = reinterpret_cast<const T*>(a.q) + row * a.ldq + h * a.dp;
   for (int i = threadIdx.x; i < a.dp; i += ROWS_THREADS) q_s[i] = ld1(q + i);
   const float slope = a.slopes != nullptr ? a.slopes[h] : 0.f;
+  const bool sigmoid = a.key_bias != nullptr;
+  const float key_bias = sigmoid ? a.key_bias[h] : 0.f;
   const T* kc = reinterpret_cast<const T*>(a.k_cache);
   const T* vc = reinterpret_cast<const T*>(a.v_cache);
   float m = -INFINITY, l = 0.f, acc[ROWS_VPT];
 #pragma unroll
   for (int c = 0; c < ROWS_VPT; ++c) acc[c] = 0.f;
   // the visible keys: `kept` first ones, then those from `from` on
-  const int from = a.window > 0 ? max(0, kv_len - a.window) : 0, kept = min(a.keep, from);
+  const int from = a.chunk > 0 ? (kv_len - 1) / a.chunk * a.chunk : a.window > 0 ? max(0, kv_len - a.window) : 0;
+  const int kept = min(a.keep, from);
   const int visible = kept + kv_len - from;
   __syncthreads();
   for (int j0 = 0; j0 < visible; j0 += ROWS_THREADS) {
@@ -355,14 +365,20 @@ attn_rows_kernel(const RowsArgs a) {
       }
       s = dot * a.scale - slope * static_cast<float>(kv_len - 1 - j);
     }
-    float mx = warp_max(s);
-    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = mx;
-    __syncthreads();
-    mx = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
-    const float m_new = fmaxf(m, mx), alpha = expf(m - m_new);        // 0 in the first round
-    m = m_new;
-    const float p = i0 < visible ? expf(s - m_new) : 0.f;
-    l = l * alpha + p;
+    float p, alpha = 1.f;
+    if (sigmoid) {
+      p = i0 < visible ? sigmoid_f(s + key_bias) : 0.f;
+    } else {
+      float mx = warp_max(s);
+      if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = mx;
+      __syncthreads();
+      mx = fmaxf(fmaxf(red[0], red[1]), fmaxf(red[2], red[3]));
+      const float m_new = fmaxf(m, mx);
+      alpha = expf(m - m_new);        // 0 in the first round
+      m = m_new;
+      p = i0 < visible ? expf(s - m_new) : 0.f;
+      l = l * alpha + p;
+    }
     p_s[threadIdx.x] = p;
     __syncthreads();
 #pragma unroll
@@ -376,10 +392,14 @@ attn_rows_kernel(const RowsArgs a) {
     }
     __syncthreads();
   }
-  float tot[1] = {l};
-  block_sum<1>(tot, red);
-  if (a.sink) tot[0] += expf(-m);
-  const float inv = a.out_scale / tot[0];
+  float inv = a.out_scale;
+  if (!sigmoid) {
+    float tot[1] = {l};
+    block_sum<1>(tot, red);
+    if (a.sink) tot[0] += expf(-m);
+    inv /= tot[0];
+  }
+  if (a.gate != nullptr) inv *= sigmoid_f(ld1(reinterpret_cast<const T*>(a.gate) + row * a.ldg + h));
   T* o = reinterpret_cast<T*>(a.out) + row * a.ldo + h * a.vp;
 #pragma unroll
   for (int c = 0; c < ROWS_VPT; ++c) {
@@ -417,7 +437,8 @@ extern "C" int tw_qkv_prep(const void* p, long long ldp, int T, int heads, int k
     set_last_error("qkv_prep: %d rotated dimensions of %d", rot_dims, dim);
     return 1;
   }
-  if (heads <= 0 || kv_heads <= 0 || norm < 0 || norm > 2 || (norm != 0 && (wq == nullptr || wk == nullptr)) ||
+  if (heads <= 0 || kv_heads < 0 || (kv_heads > 0 && (k_cache == nullptr || v_cache == nullptr)) || norm < 0 || norm > 2 ||
+      (wq == nullptr) != (wk == nullptr) || (norm == 2 && wq == nullptr) ||
       temp_every <= 0 || (conv_w != nullptr && (row_seq == nullptr || taps < 1)) ||
       (conv_w != nullptr && taps > 1 && (conv_state == nullptr || slots == nullptr))) {
     set_last_error("qkv_prep: bad arguments (heads=%d, kv_heads=%d, norm=%d, taps=%d)", heads, kv_heads, norm, taps);
@@ -446,8 +467,8 @@ extern "C" int tw_qkv_prep(const void* p, long long ldp, int T, int heads, int k
 extern "C" int tw_attn_rows(const void* q, long long ldq, const void* k_cache, const void* v_cache, int page, void* out,
                             long long ldo, const int* tok_row, const int* tok_seq, const int* tok_kvlen, int n,
                             const int* block_table, int max_blocks, int heads, int kv_heads, int dp, int vp, float scale,
-                            const float* slopes, int sink, float out_scale, int window, int keep, int dtype,
-                            cudaStream_t stream) {
+                            const float* slopes, int sink, float out_scale, int window, int keep, const float* key_bias,
+                            int chunk, const void* gate, long long ldg, int dtype, cudaStream_t stream) {
   if (n <= 0) return 0;
   if (dp % 8 != 0 || dp > 4096 || vp > ROWS_VPT * ROWS_THREADS || kv_heads <= 0 || heads % kv_heads != 0 ||
       !aligned16(k_cache)) {
@@ -456,7 +477,7 @@ extern "C" int tw_attn_rows(const void* q, long long ldq, const void* k_cache, c
     return 1;
   }
   const RowsArgs a{q, ldq, k_cache, v_cache, page, out, ldo, tok_row, tok_seq, tok_kvlen, block_table, max_blocks, heads,
-                   kv_heads, dp, vp, scale, slopes, sink, out_scale, window, keep};
+                   kv_heads, dp, vp, scale, slopes, sink, out_scale, window, keep, key_bias, chunk, gate, ldg};
   const dim3 grid(n, heads);
   if (dtype == TW_BF16) attn_rows_kernel<__nv_bfloat16><<<grid, ROWS_THREADS, dp * 4, stream>>>(a);
   else attn_rows_kernel<float><<<grid, ROWS_THREADS, dp * 4, stream>>>(a);

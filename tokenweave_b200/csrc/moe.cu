@@ -4,16 +4,17 @@
 //                      Reference: replicated gate linear, then csrc/moe/topk_softmax_kernels.cu
 //                      and the renormalisation in fused_moe.py:831-844.
 //   tw_moe_route       the general router, any number of experts up to 256, bf16 and fp32: scores are the softmax over all
-//                      experts, the top ones are chosen by score + correction, their weights are the scores over the
-//                      scores' sum; further rows of the same matrix give sigmoid gates (of a shared expert)
+//                      experts or the sigmoid of each logit, the top ones are chosen by score + correction, their weights
+//                      are the scores, or those over their sum; further rows of the same matrix give sigmoid gates (of a
+//                      shared expert)
 //   tw_moe_align       counting sort of (token, k) pairs by expert with every expert's segment
 //                      padded to the GEMM's 128-row tile; emits the expert of each row tile, the
 //                      number of tiles, the sorted position of every pair.
 //                      Reference: csrc/moe/moe_align_sum_kernels.cu:24-112.
 //   tw_moe_scatter     copies token rows into expert-sorted order (the A operand of the grouped
 //                      GEMM) and the routing weight of each sorted row.
-//   tw_moe_combine     out[t] = sum_k y_sorted[pos[t,k]] (+ gate[t] * shared[t]) (weights were applied by the second
-//                      grouped GEMM's epilogue). Reference: moe_sum_kernel,
+//   tw_moe_combine     out[t] = sum_k y_sorted[pos[t,k]] (+ gate[t] * shared[t], or + shared[t]) (weights were applied by
+//                      a grouped GEMM's epilogue). Reference: moe_sum_kernel,
 //                      moe_align_sum_kernels.cu:277-293.
 #include "tw_common.cuh"
 #include "tw_host.h"
@@ -149,6 +150,7 @@ struct RouteArgs {
   float* topk_w; int* topk_ids;             // [T, topk]
   float* gate;                              // [T, gates]
   int T, H, E, gates, topk;
+  int sigmoid, normalize;                   // scores: sigmoid or softmax of the logits; weights over their sum, or as they are
   float sum_eps;
 };
 
@@ -162,18 +164,29 @@ __device__ __forceinline__ void route_select(const RouteArgs& a, const float* lo
     s[j] = e < a.E ? logits[e] : -INFINITY;
     mx = fmaxf(mx, s[j]);
   }
-  mx = warp_max(mx);
+  if (a.sigmoid) {
+    // without corrections the order of the logits is that of their scores, also where these have rounded to one
 #pragma unroll
-  for (int j = 0; j < MOE_MAX_EXPERTS / 32; ++j) {
-    s[j] = expf(s[j] - mx);
-    sum += s[j];
-  }
-  const float inv = 1.f / warp_sum(sum);
+    for (int j = 0; j < MOE_MAX_EXPERTS / 32; ++j) {
+      const int e = lane + 32 * j;
+      const float z = s[j];
+      s[j] = sigmoid_f(z);
+      c[j] = e >= a.E ? -INFINITY : a.correction != nullptr ? s[j] + a.correction[e] : z;
+    }
+  } else {
+    mx = warp_max(mx);
 #pragma unroll
-  for (int j = 0; j < MOE_MAX_EXPERTS / 32; ++j) {
-    const int e = lane + 32 * j;
-    s[j] *= inv;
-    c[j] = e < a.E ? s[j] + (a.correction != nullptr ? a.correction[e] : 0.f) : -INFINITY;
+    for (int j = 0; j < MOE_MAX_EXPERTS / 32; ++j) {
+      s[j] = expf(s[j] - mx);
+      sum += s[j];
+    }
+    const float inv = 1.f / warp_sum(sum);
+#pragma unroll
+    for (int j = 0; j < MOE_MAX_EXPERTS / 32; ++j) {
+      const int e = lane + 32 * j;
+      s[j] *= inv;
+      c[j] = e < a.E ? s[j] + (a.correction != nullptr ? a.correction[e] : 0.f) : -INFINITY;
+    }
   }
   float total = 0.f, my_w = 0.f;
   int my_id = 0;
@@ -197,7 +210,7 @@ __device__ __forceinline__ void route_select(const RouteArgs& a, const float* lo
     if (lane == k) { my_w = score; my_id = id; }
   }
   if (lane < a.topk) {
-    a.topk_w[static_cast<long long>(t) * a.topk + lane] = my_w / (total + a.sum_eps);
+    a.topk_w[static_cast<long long>(t) * a.topk + lane] = a.normalize ? my_w / (total + a.sum_eps) : my_w;
     a.topk_ids[static_cast<long long>(t) * a.topk + lane] = my_id;
   }
   if (lane < a.gates) a.gate[static_cast<long long>(t) * a.gates + lane] = sigmoid_f(logits[a.E + lane]);
@@ -356,7 +369,7 @@ moe_scatter_kernel(const uint4* __restrict__ x, long long ldx, const int* __rest
   }
 }
 
-// out[t] = sum_k y[pos[t,k]] (+ gate[t] shared[t]) in fp32, rounded once.
+// out[t] = sum_k y[pos[t,k]] (+ gate[t] shared[t]; no gate: one) in fp32, rounded once.
 template <typename T_>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const T_* __restrict__ y, const int* __restrict__ sorted_pos, const T_* __restrict__ shared_y,
@@ -376,7 +389,7 @@ moe_combine_kernel(const T_* __restrict__ y, const int* __restrict__ sorted_pos,
         for (int j = 0; j < 8; ++j) acc[j] += f[j];
       }
       if (shared_y != nullptr) {
-        const float g = gate[t];
+        const float g = gate != nullptr ? gate[t] : 1.f;
         ld8(shared_y + t * lds + v * 8, f);
 #pragma unroll
         for (int j = 0; j < 8; ++j) acc[j] = fmaf(g, f[j], acc[j]);
@@ -441,14 +454,14 @@ extern "C" int tw_moe_router(const void* x, long long ldx, const void* wg, float
 
 extern "C" int tw_moe_route(const void* x, long long ldx, const void* w, long long ldw, const float* correction,
                             float* topk_w, int* topk_ids, float* gate, int T, int H, int E, int gates, int topk,
-                            float sum_eps, int dtype, cudaStream_t stream) {
+                            int sigmoid, int normalize, float sum_eps, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (E < 1 || E > MOE_MAX_EXPERTS || topk < 1 || topk > E || topk > ROUTE_MAX_TOPK || gates < 0 ||
       gates > ROUTE_MAX_GATES || (gates > 0 && gate == nullptr)) {
     set_last_error("moe_route: unsupported sizes (%d experts, top %d, %d gates)", E, topk, gates);
     return 1;
   }
-  const RouteArgs a{x, ldx, w, ldw, correction, topk_w, topk_ids, gate, T, H, E, gates, topk, sum_eps};
+  const RouteArgs a{x, ldx, w, ldw, correction, topk_w, topk_ids, gate, T, H, E, gates, topk, sigmoid, normalize, sum_eps};
   if (dtype != TW_BF16) {
     moe_route_f32_kernel<<<T, 256, 0, stream>>>(a);
     return moe_check("moe_route");
@@ -506,12 +519,12 @@ extern "C" int tw_moe_scatter(const void* x, long long ldx, const int* topk_ids,
   return moe_check("moe_scatter");
 }
 
-// shared_y (or null): [T, H] with row stride lds, times gate [T].
+// shared_y (or null): [T, H] with row stride lds, times gate [T] (or null: one).
 extern "C" int tw_moe_combine(const void* y, const int* sorted_pos, const void* shared_y, long long lds, const float* gate,
                               void* out, long long ldo, int T, int topk, int H, int dtype, cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (H % 8 != 0 || ldo % 8 != 0 || lds % 8 != 0 || (shared_y != nullptr && gate == nullptr)) {
-    set_last_error("moe_combine: rows of %d elements (multiples of eight are needed), or a shared row without its gate", H);
+  if (H % 8 != 0 || ldo % 8 != 0 || lds % 8 != 0) {
+    set_last_error("moe_combine: rows of %d elements (multiples of eight are needed)", H);
     return 1;
   }
   int grid = T;

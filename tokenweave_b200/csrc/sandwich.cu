@@ -1,0 +1,228 @@
+// Residual blocks with a norm in front of a sublayer and one behind it, and averages over the depth of the network:
+//
+//     x <- x + N_post(sublayer(N_pre(x)))                       after every sublayer
+//     X_n = x ;  x <- sum_{j <= n} coef[j] X_j                  after every layer (X_0: the embedding output)
+//
+//   tw_embed_sandwich  x = X_0 = scale * table[id] ; xa = N(x) (the first sublayer's input)
+//   tw_sandwich_step   what lies between two sublayers, in one pass: norm of the sublayer's output, sum, (the layer's result
+//                      kept, the average over all results so far,) and the next sublayer's norm (or the final one)
+//
+// N is a layer norm (mean taken off, weight and bias) or an RMS norm (weight alone). The stream and the kept results are
+// fp32, y, xa and the norms' weights bf16 or fp32, all arithmetic is fp32; deviations are summed from the mean, not as a
+// difference of squares. One CTA per row; the row stays in registers between the passes.
+#include "tw_host.h"
+#include "tw_kernels.h"
+#include "tw_typed.cuh"
+
+namespace tw {
+
+struct SandwichArgs {
+  const void* y; long long ldy;                  // [rows, H] sublayer output
+  float* x; long long ldx;                       // [rows, H] stream
+  int store;                                     // the new stream is written back
+  const void *w_post, *b_post;                   // norm of the output
+  const float* past; long long ldp, lds;         // X_j of row t: past + j * lds + t * ldp
+  int n_past;
+  const float* coef;                             // [n_past + 1]; null: no average
+  float* result;                                 // X_n (row stride ldp); null: not kept
+  const void *w_next, *b_next;                   // the next norm
+  void* xa; long long lda;
+  int rows, H, center;
+  float eps;
+  const int* ids; const void* table; long long ldt; int vocab; float scale;        // embedding
+};
+
+// Replaces a row by its norm. Elements outside the row are zeros.
+template <typename T, int VPT>
+__device__ __forceinline__ void norm_row(const SandwichArgs& a, float (&v)[VPT][8], const void* w, const void* b,
+                                         float* scratch) {
+  float s[1], mean = 0.f;
+  if (a.center) {
+    s[0] = 0.f;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k)
+#pragma unroll
+      for (int j = 0; j < 8; ++j) s[0] += v[k][j];
+    block_sum<1>(s, scratch);
+    mean = s[0] / static_cast<float>(a.H);
+  }
+  s[0] = 0.f;
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int n = a.H - (threadIdx.x + k * blockDim.x) * 8;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) {
+      v[k][j] = j < n ? v[k][j] - mean : 0.f;
+      s[0] += v[k][j] * v[k][j];
+    }
+  }
+  block_sum<1>(s, scratch);
+  const float r = 1.f / sqrtf(s[0] / static_cast<float>(a.H) + a.eps);
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
+    if (n <= 0) continue;
+    float g[8], c[8];
+    ld8n<true>(reinterpret_cast<const T*>(w) + i, n, g);
+    if (b != nullptr) {
+      ld8n<true>(reinterpret_cast<const T*>(b) + i, n, c);
+    } else {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) c[j] = 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[k][j] = fmaf(v[k][j] * r, g[j], c[j]);
+  }
+}
+
+template <typename T, int VPT>
+__device__ __forceinline__ void next_input(const SandwichArgs& a, int t, float (&v)[VPT][8], float* scratch) {
+  norm_row<T, VPT>(a, v, a.w_next, a.b_next, scratch);
+#pragma unroll
+  for (int k = 0; k < VPT; ++k) {
+    const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
+    if (n > 0) st8n<true>(reinterpret_cast<T*>(a.xa) + t * a.lda + i, n, v[k]);
+  }
+}
+
+template <typename T, int VPT>
+__global__ void __launch_bounds__(512)
+sandwich_step_kernel(const SandwichArgs a) {
+  __shared__ float scratch[32];
+  for (int t = blockIdx.x; t < a.rows; t += gridDim.x) {
+    float v[VPT][8], x[VPT][8];
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[k][j] = x[k][j] = 0.f;
+      if (n <= 0) continue;
+      ld8n<true>(reinterpret_cast<const T*>(a.y) + t * a.ldy + i, n, v[k]);
+      ld8n<true>(a.x + t * a.ldx + i, n, x[k]);
+    }
+    norm_row<T, VPT>(a, v, a.w_post, a.b_post, scratch);
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
+      if (n <= 0) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[k][j] = 0.f;
+        continue;
+      }
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[k][j] += x[k][j];
+      if (a.coef != nullptr) {
+        if (a.result != nullptr) st8n<true>(a.result + t * a.ldp + i, n, v[k]);
+        const float mine = a.coef[a.n_past];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[k][j] *= mine;
+        const float* p = a.past + t * a.ldp + i;
+#pragma unroll 4
+        for (int q = 0; q < a.n_past; ++q) {
+          const float c = a.coef[q];
+          float u[8];
+          ld8n<true>(p + q * a.lds, n, u);
+#pragma unroll
+          for (int j = 0; j < 8; ++j) v[k][j] = fmaf(c, u[j], v[k][j]);
+        }
+      }
+      if (a.store) st8n<true>(a.x + t * a.ldx + i, n, v[k]);
+    }
+    next_input<T, VPT>(a, t, v, scratch);
+  }
+}
+
+template <typename T, int VPT>
+__global__ void __launch_bounds__(512)
+embed_sandwich_kernel(const SandwichArgs a) {
+  __shared__ float scratch[32];
+  for (int t = blockIdx.x; t < a.rows; t += gridDim.x) {
+    const int id = a.ids[t];
+    const bool ok = id >= 0 && id < a.vocab;
+    const T* src = reinterpret_cast<const T*>(a.table) + (ok ? id : 0) * a.ldt;
+    float v[VPT][8];
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+      const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[k][j] = 0.f;
+      if (n <= 0) continue;
+      if (ok) ld8n<true>(src + i, n, v[k]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[k][j] *= a.scale;
+      st8n<true>(a.x + t * a.ldx + i, n, v[k]);
+      if (a.result != nullptr) st8n<true>(a.result + t * a.ldp + i, n, v[k]);
+    }
+    next_input<T, VPT>(a, t, v, scratch);
+  }
+}
+
+static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
+
+template <typename T, int VPT>
+static void launch_sandwich(const SandwichArgs& a, int grid, int threads, cudaStream_t stream) {
+  if (a.ids != nullptr) embed_sandwich_kernel<T, VPT><<<grid, threads, 0, stream>>>(a);
+  else sandwich_step_kernel<T, VPT><<<grid, threads, 0, stream>>>(a);
+}
+
+static int run_sandwich(const SandwichArgs& a, int dtype, const char* what, cudaStream_t stream) {
+  const int nvec = (a.H + 7) / 8, vpt = nvec <= 512 ? 1 : nvec <= 1024 ? 2 : 4;
+  const int threads = ((nvec + vpt - 1) / vpt + 31) / 32 * 32;
+  if (a.H <= 0 || threads > 512) {
+    set_last_error("%s: rows of %d elements (up to 16384)", what, a.H);
+    return 1;
+  }
+  if (a.ldy % 8 != 0 || a.ldx % 8 != 0 || a.lda % 8 != 0 || a.ldt % 8 != 0 || a.ldp % 8 != 0 || a.lds % 8 != 0 ||
+      !aligned16(a.y) || !aligned16(a.x) || !aligned16(a.xa) || !aligned16(a.table) || !aligned16(a.past) ||
+      !aligned16(a.result) || !aligned16(a.w_post) || !aligned16(a.b_post) || !aligned16(a.w_next) || !aligned16(a.b_next)) {
+    set_last_error("%s: rows on 16-byte boundaries are needed", what);
+    return 1;
+  }
+  const int cap = device_sm_count() * (threads <= 128 ? 16 : threads <= 256 ? 8 : 4);
+  const int grid = a.rows < cap ? a.rows : cap;
+#define TW_GO(TT)                                                       \
+  do {                                                                  \
+    if (vpt == 1) launch_sandwich<TT, 1>(a, grid, threads, stream);     \
+    else if (vpt == 2) launch_sandwich<TT, 2>(a, grid, threads, stream); \
+    else launch_sandwich<TT, 4>(a, grid, threads, stream);              \
+  } while (0)
+  if (dtype == TW_BF16) TW_GO(__nv_bfloat16);
+  else TW_GO(float);
+#undef TW_GO
+  const cudaError_t e = cudaGetLastError();
+  if (e == cudaSuccess) return 0;
+  set_last_error("%s launch failed: %s", what, cudaGetErrorString(e));
+  return 1;
+}
+
+}  // namespace tw
+
+using namespace tw;
+
+extern "C" int tw_embed_sandwich(const int* ids, const void* table, long long ldt, int vocab, float scale, float* x,
+                                 long long ldx, float* first, long long ldp, const void* w, const void* b, int center,
+                                 void* xa, long long lda, int T, int H, float eps, int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  SandwichArgs a{};
+  a.ids = ids; a.table = table; a.ldt = ldt; a.vocab = vocab; a.scale = scale;
+  a.x = x; a.ldx = ldx; a.result = first; a.ldp = ldp; a.w_next = w; a.b_next = b; a.center = center;
+  a.xa = xa; a.lda = lda; a.rows = T; a.H = H; a.eps = eps;
+  return run_sandwich(a, dtype, "embed_sandwich", stream);
+}
+
+extern "C" int tw_sandwich_step(const void* y, long long ldy, float* x, long long ldx, int store, const void* w_post,
+                                const void* b_post, const float* past, long long ldp, long long lds, int n_past,
+                                const float* coef, float* result, const void* w_next, const void* b_next, int center,
+                                void* xa, long long lda, int T, int H, float eps, int dtype, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (n_past < 0 || (coef != nullptr && n_past > 0 && past == nullptr)) {
+    set_last_error("sandwich_step: an average over %d earlier results that are not there", n_past);
+    return 1;
+  }
+  SandwichArgs a{};
+  a.y = y; a.ldy = ldy; a.x = x; a.ldx = ldx; a.store = store; a.w_post = w_post; a.b_post = b_post;
+  a.past = past; a.ldp = ldp; a.lds = lds; a.n_past = n_past; a.coef = coef; a.result = result;
+  a.w_next = w_next; a.b_next = b_next; a.center = center;
+  a.xa = xa; a.lda = lda; a.rows = T; a.H = H; a.eps = eps;
+  return run_sandwich(a, dtype, "sandwich_step", stream);
+}

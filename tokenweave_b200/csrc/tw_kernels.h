@@ -124,8 +124,8 @@ int tw_moe_scatter(const void* x, long long ldx, const int* topk_ids, const floa
 int tw_moe_combine(const void* y, const int* sorted_pos, const void* shared_y, long long lds, const float* gate, void* out,
                    long long ldo, int T, int topk, int H, int dtype, cudaStream_t stream);
 int tw_moe_route(const void* x, long long ldx, const void* w, long long ldw, const float* correction, float* topk_w,
-                 int* topk_ids, float* gate, int T, int H, int E, int gates, int topk, float sum_eps, int dtype,
-                 cudaStream_t stream);
+                 int* topk_ids, float* gate, int T, int H, int E, int gates, int topk, int sigmoid, int normalize,
+                 float sum_eps, int dtype, cudaStream_t stream);
 
 // ---- in-kernel collectives (comm_fused.cu) ----
 // mc_base: multicast address of the symmetric buffer or NULL (peer transport). peer_bases /
@@ -183,6 +183,20 @@ int tw_streams_step(const void* y, long long ldy, float* x, long long ldx, long 
                     const float* out, float mult, const float* in, int first, int store, const void* w, float offset,
                     void* xa, long long lda, int T, int H, float eps, int dtype, cudaStream_t stream);
 
+// ---- norms on both sides of a sublayer, averages over the depth (sandwich.cu) ----
+int tw_embed_sandwich(const int* ids, const void* table, long long ldt, int vocab, float scale, float* x, long long ldx,
+                      float* first, long long ldp, const void* w, const void* b, int center, void* xa, long long lda, int T,
+                      int H, float eps, int dtype, cudaStream_t stream);
+int tw_sandwich_step(const void* y, long long ldy, float* x, long long ldx, int store, const void* w_post,
+                     const void* b_post, const float* past, long long ldp, long long lds, int n_past, const float* coef,
+                     float* result, const void* w_next, const void* b_next, int center, void* xa, long long lda, int T, int H,
+                     float eps, int dtype, cudaStream_t stream);
+
+// ---- minGRU (min_gru.cu) ----
+int tw_min_gru(const void* p, long long ldp, const float* bz, const float* bx, float* state, void* out, long long ldo,
+               const int* seqs, int n_seqs, const int* cu_q, const int* kv_lens, const int* slots, int n, int chunked,
+               int dtype, cudaStream_t stream);
+
 // ---- grouped attention (grouped_attn.cu; tensor cores: attn_prefill_split.cu, attn_decode_tc.cu, bf16) ----
 int tw_qkv_prep(const void* p, long long ldp, int T, int heads, int kv_heads, int dim, int dp, int vp, void* q,
                 long long ldq, void* k_cache, void* v_cache, const int* positions, const int* cache_slots,
@@ -192,22 +206,25 @@ int tw_qkv_prep(const void* p, long long ldp, int T, int heads, int kv_heads, in
 int tw_attn_rows(const void* q, long long ldq, const void* k_cache, const void* v_cache, int page, void* out,
                  long long ldo, const int* tok_row, const int* tok_seq, const int* tok_kvlen, int n,
                  const int* block_table, int max_blocks, int heads, int kv_heads, int dp, int vp, float scale,
-                 const float* slopes, int sink, float out_scale, int window, int keep, int dtype, cudaStream_t stream);
+                 const float* slopes, int sink, float out_scale, int window, int keep, const float* key_bias, int chunk,
+                 const void* gate, long long ldg, int dtype, cudaStream_t stream);
 int tw_attn_prefill_grouped(const void* q, long long ldq, int T, const void* k_cache, const void* v_cache,
                             int num_blocks, int page, void* out, long long ldo, const int* cu_q, const int* kv_lens,
                             const int* block_table, int max_blocks, const int* tile_seq, const int* tile_q0,
                             int num_tiles, int hq, int hkv, int dp, int vp, float scale, const float* slopes, int sink,
-                            float out_scale, int window, int keep, uint32_t* status, cudaStream_t stream);
+                            float out_scale, int window, int keep, const float* key_bias, int chunk, const void* gate,
+                            long long ldg, uint32_t* status, cudaStream_t stream);
 int tw_attn_decode_grouped(const void* q, long long ldq, const void* k_cache, const void* v_cache, int num_blocks,
                            int page, void* out, long long ldo, const int* tok_row, const int* tok_seq,
                            const int* tok_kvlen, int n_tok, const int* block_table, int max_blocks, int hq, int hkv,
                            int dp, int vp, float scale, const float* slopes, int sink, float out_scale, int window,
-                           int keep, int splits, float* part_o, float* part_ml, uint32_t* status, cudaStream_t stream);
+                           int keep, const float* key_bias, int chunk, const void* gate, long long ldg, int splits,
+                           float* part_o, float* part_ml, uint32_t* status, cudaStream_t stream);
 int tw_gemm_bf16_act(const void* A, long long lda, const void* B, long long ldb, void* C, long long ldc,
                      const void* bias, int M, int N, int K, int act, int act_begin, int act_end, int max_ctas, int plan_hint,
                      uint32_t* status, cudaStream_t stream);
 int tw_gemm_bf16_clamped(const void* A, long long lda, const void* B, long long ldb, long long rows_b, void* C,
-                         long long ldc, int M, int N, int K, float limit, float alpha, int up_row_offset,
+                         long long ldc, const float* row_scale, int M, int N, int K, float limit, float alpha, int up_row_offset,
                          const int* tile_expert, const int* num_m_tiles_dev, int n_per_expert, int tile_rows, int max_ctas,
                          int plan_hint, uint32_t* status, cudaStream_t stream);
 

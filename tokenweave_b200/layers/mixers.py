@@ -36,10 +36,13 @@ def _vec(n: int, dtype, device, fill: float = 1.0) -> nn.Parameter:
 
 # ---- rotation ---------------------------------------------------------------------------------------------------------
 # ``rot`` = {"base", "dims", "scaling": None or YaRN's {"factor", "original", "fast", "slow"}}
+def rotation_key(rot: dict) -> tuple:
+    return int(rot["dims"]), float(rot["base"]), tuple(sorted((rot.get("scaling") or {}).items()))
+
+
 def rope_table(rt, rot: dict) -> torch.Tensor:
     """Cosines and sines by position ([positions, dims]: cosines, then sines), one table per kind of rotation in a model."""
-    s = rot.get("scaling")
-    key = (int(rot["dims"]), float(rot["base"]), tuple(sorted((s or {}).items())))
+    s, key = rot.get("scaling"), rotation_key(rot)
     if key not in rt.rope_tables:
         scaling = None
         if s:
@@ -322,6 +325,45 @@ class Mamba2Mixer(Mixer):
         self.o_proj(g, out=out)
 
 
+class MinGRUMixer(Mixer):
+    """minGRU: a recurrence per channel whose gates read the current token alone. ``z = sigmoid(W_z x + b_z)``,
+    ``u = W_x x + b_x``, ``S <- (1 - z) S + z (u + 1/2 if u >= 0 else sigmoid(u))`` with an fp32 state, output projection of
+    ``S silu(W_g x)``. One product makes z, u and the gate; their biases are added in fp32 behind it."""
+    recurrent = True
+
+    def __init__(self, sizes: dict, width: int, eps: float, *, dtype, device):
+        super().__init__()
+        self.inner, self.width = int(sizes["width"]), width
+        self.padded = pad8(self.inner)
+        self.in_proj = PaddedLinear(width, 3 * self.padded, dtype=dtype, device=device)
+        self.z_bias, self.x_bias = (_vec(self.padded, torch.float32, device, 0.0) for _ in range(2))
+        self.o_proj = PaddedLinear(self.inner, width, dtype=dtype, device=device)
+
+    def workspaces(self) -> list[tuple[str, int]]:
+        return [("proj", self.in_proj.out_padded), ("mixed", self.o_proj.in_padded)]
+
+    def state_bytes_per_slot(self) -> int:
+        return 4 * self.padded
+
+    def init_state(self, kept: dict, num_slots: int) -> None:
+        kept["state"] = torch.zeros(num_slots, self.padded, dtype=torch.float32, device=self.z_bias.device)
+
+    def tensor_targets(self) -> dict:
+        I, W, P = self.inner, self.width, self.padded
+        out = {name: ((I, W), lambda t, row=row: self.in_proj.load_rows(t, row)) for name, row in (("z", 0), ("x", P), ("g", 2 * P))}
+        out.update({name: ((I,), b.data[:I].copy_) for name, b in (("z.b", self.z_bias), ("x.b", self.x_bias))})
+        out["o"] = ((W, I), lambda t: self.o_proj.load_rows(t, 0))
+        return out
+
+    def forward(self, x: torch.Tensor, meta: AttentionMetadata, rt, out: torch.Tensor, kept: dict) -> None:
+        n, e = x.shape[0], meta.extra
+        p = self.in_proj(x, out=rt.buffer("proj", n, self.in_proj.out_padded))
+        y = rt.buffer("mixed", n, self.o_proj.in_padded)
+        for seqs, chunked in ((e["scan_seqs"], False), (e["chunk_seqs"], True)):
+            hops.min_gru(p, self.z_bias, self.x_bias, kept["state"], y, seqs, meta.cu_q, meta.kv_lens, e["state_slots"], chunked)
+        self.o_proj(y, out=out)
+
+
 class FeedForward(nn.Module):
     """A sublayer without state: ``forward(x, rt, out)``."""
 
@@ -387,10 +429,12 @@ class ActMLP(FeedForward):
 
 
 class RoutedMLP(FeedForward):
-    """Mixture of experts: every token takes ``top`` of ``experts`` gated feed-forwards, chosen by the softmax over all
-    experts plus a correction per expert; their outputs are weighted with the scores (without it) over the scores' sum +
-    ``sum_eps``. ``act``: as for ``ops.gemm``. ``shared`` = {"ff", "act"} or None: one more gated feed-forward that every
-    token takes, times the sigmoid of a projection to one number.
+    """Mixture of experts: every token takes ``top`` of ``experts`` gated feed-forwards, chosen by their scores: the softmax
+    over all experts, or (``scores`` "sigmoid") each logit's sigmoid; with ``correction`` a number per expert joins the scores
+    for the choice. Their weights are the scores (without it), with ``normalize`` over the scores' sum + ``sum_eps``; a weight
+    is on the expert's output or (``weigh`` "input") on its input. ``act``: as for ``ops.gemm``. ``shared`` = {"ff", "act",
+    "gated"} or None: one more gated feed-forward that every token takes, with "gated" (the default) times the sigmoid of a
+    projection to one number.
 
     The router's rows and the shared feed-forward's gate are one product; the pipeline behind it is ``layers/moe.py``."""
 
@@ -400,11 +444,16 @@ class RoutedMLP(FeedForward):
         if not 0 < self.top <= self.experts:
             raise ValueError(f"{self.top} of {self.experts} experts")
         self.act, self.sum_eps = self._act(sizes["act"]), float(sizes.get("sum_eps", 0.0))
+        self.scores, self.normalize = str(sizes.get("scores", "softmax")), bool(sizes.get("normalize", True))
+        if self.scores not in ("softmax", "sigmoid") or sizes.get("weigh", "output") not in ("output", "input"):
+            raise ValueError(f"unknown scores {self.scores!r} or place of the weights {sizes.get('weigh')!r}")
+        self.weigh_input = sizes.get("weigh") == "input"
         w8, self.f8 = pad8(width), pad8(self.ff)
         par = lambda *s, dt=dtype: nn.Parameter(torch.zeros(*s, dtype=dt, device=device), requires_grad=False)
         shared = sizes.get("shared")
-        self.router_w = par(self.experts + (1 if shared else 0), w8)
-        self.correction = par(self.experts, dt=torch.float32)
+        self.shared_gate = bool(shared) and bool(shared.get("gated", True))
+        self.router_w = par(self.experts + int(self.shared_gate), w8)
+        self.correction = par(self.experts, dt=torch.float32) if sizes.get("correction", True) else None
         self.w13, self.w2 = par(self.experts, 2 * self.f8, w8), par(self.experts, w8, self.f8)
         self.shared_up = self.shared_down = None
         if shared:
@@ -440,8 +489,9 @@ class RoutedMLP(FeedForward):
     # ---- weights -------------------------------------------------------------------------------------------
     def tensor_targets(self) -> dict:
         W, F, f8 = self.width, self.ff, self.f8
-        out = {"router": ((self.experts, W), lambda t: self.router_w.data[:self.experts, :W].copy_(t)),
-               "correction": ((self.experts,), self.correction.data.copy_)}
+        out = {"router": ((self.experts, W), lambda t: self.router_w.data[:self.experts, :W].copy_(t))}
+        if self.correction is not None:
+            out["correction"] = ((self.experts,), self.correction.data.copy_)
         for e in range(self.experts):
             out[f"e{e}.gate"] = ((F, W), lambda t, e=e: self.w13.data[e, :F, :W].copy_(t))
             out[f"e{e}.up"] = ((F, W), lambda t, e=e: self.w13.data[e, f8:f8 + F, :W].copy_(t))
@@ -451,27 +501,29 @@ class RoutedMLP(FeedForward):
             out["shared.gate"] = ((S, W), lambda t: self.shared_up.load_rows(t, 0))
             out["shared.up"] = ((S, W), lambda t: self.shared_up.load_rows(t, pad8(S)))
             out["shared.down"] = ((W, S), lambda t: self.shared_down.load_rows(t, 0))
+        if self.shared_gate:
             out["shared.sg"] = ((1, W), lambda t: self.router_w.data[self.experts:, :W].copy_(t))
         return out
 
     # ---- forward -------------------------------------------------------------------------------------------
     def forward(self, x: torch.Tensor, rt, out: torch.Tensor) -> None:
         n, shared, gate = x.shape[0], None, None
-        weights, ids, gates = ops.moe_route(x, self.router_w, self.experts, self.top, self.correction, self.sum_eps)
+        weights, ids, gates = ops.moe_route(x, self.router_w, self.experts, self.top, self.correction, self.sum_eps,
+                                            self.scores, self.normalize)
         if self.shared_up is not None:
             a = rt.buffer("shared_act", n, self.shared_down.in_padded)
             tmp = rt.buffer("shared_gate_up", n, self.shared_up.out_padded) if x.dtype == torch.float32 else None
             hops.gated_product(x, self.shared_up.weight, self.shared_act, a, tmp)
             shared = self.shared_down(a, out=rt.buffer("shared_out", n, self.shared_down.out_padded))
-            gate = gates[:, 0]
+            gate = gates[:, 0] if self.shared_gate else None
         if not x.is_cuda:
-            y = reference.moe_experts(x, self.w13, self.w2, weights, ids, self.act)
-            out.copy_(y if shared is None else y + gate[:, None] * shared)
+            y = reference.moe_experts(x, self.w13, self.w2, weights, ids, self.act, self.weigh_input)
+            out.copy_(y if shared is None else y + (shared if gate is None else gate[:, None] * shared))
             return
         ws = dict(rt.tables[("experts", self.experts, self.top)])
         rows = max_expert_rows(n, self.top, self.experts)
         ws.update((name, rt.buffer("experts." + name, rows, cols)) for name, cols in self._sorted_rows())
-        run_experts(x, weights, ids, self.w13, self.w2, ws, out, self.act, shared, gate)
+        run_experts(x, weights, ids, self.w13, self.w2, ws, out, self.act, shared, gate, weigh_input=self.weigh_input)
 
 
 # ---- several parts side by side --------------------------------------------------------------------------------------
@@ -525,8 +577,8 @@ class GroupedAttention(Part):
     * ``bias``: biases of the three projections;
     * ``conv``: a causal convolution of that many taps over time on every channel of q, k and v, right behind the
       projection (no bias, no activation); the last ``conv - 1`` projected rows of a sequence are part of its state;
-    * ``qk_norm``: "head" (RMS norm of every query and key head, one weight for all), "whole" (RMS norm of all queries,
-      and of all keys, of a token at once) or None;
+    * ``qk_norm``: "head" (RMS norm of every query and key head, one weight for all), "unit" (the same without a weight),
+      "whole" (RMS norm of all queries, and of all keys, of a token at once) or None;
     * ``q_temp`` = {"coef", "every"}: queries times ``1 + coef * ln(floor((p + 1) / every) + 1)`` at position p;
     * ``distance_bias``: ``2^(-8 (h + 1) / heads) * (i - j)`` is taken off the score of head h;
     * ``sink``: one is added to the softmax's denominator (a key of score 0 without a value);
@@ -534,32 +586,51 @@ class GroupedAttention(Part):
     * ``rot``: rotation of the first ``rot["dims"]`` dimensions of queries and keys, behind the norm;
       ``neighbour_pairs``: dimensions 2i and 2i + 1 turn together (else i and i + dims / 2);
     * ``window`` > 0: a position sees the last ``window`` positions, itself among them, and the sequence's first
-      ``keep_first``.
+      ``keep_first``;
+    * ``weights``: "softmax", or "sigmoid": a key counts with the sigmoid of its score plus a learned number per head, and
+      nothing is normalized (no sink, window or distance bias then); with it ``chunk`` > 0: a position sees the positions of
+      its own chunk of that many, counted from the sequence's start; ``head_gate``: each head's result times the sigmoid of a
+      projection of the input to one number per head;
+    * ``kv_from``: the layer whose keys and values this one reads, as that layer's cache holds them: no projections and no
+      cache of its own for them.
     """
     attends = True
 
     def __init__(self, sizes: dict, eps: float, *, dtype, device, bias: bool = False, conv: Optional[int] = None,
                  qk_norm: Optional[str] = None, q_temp: Optional[dict] = None, distance_bias: bool = False,
                  sink: bool = False, out_scale: float = 1.0, rot: Optional[dict] = None, neighbour_pairs: bool = False,
-                 window: int = 0, keep_first: int = 0):
+                 window: int = 0, keep_first: int = 0, weights: str = "softmax", chunk: int = 0, head_gate: bool = False,
+                 kv_from: Optional[int] = None):
         super().__init__()
         self.heads, self.kv_heads, self.dim, self.vdim = (int(sizes[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
         if self.heads % self.kv_heads:
             raise ValueError(f"{self.heads} query heads do not divide into {self.kv_heads} groups")
-        if qk_norm not in (None, "head", "whole"):
+        if qk_norm not in hops.QK_NORMS:
             raise ValueError(f"unknown query and key norm {qk_norm!r}")
+        if weights not in ("softmax", "sigmoid"):
+            raise ValueError(f"unknown attention weights {weights!r}")
+        if (window or sink or distance_bias) if weights == "sigmoid" else (chunk or head_gate):
+            raise ValueError("chunks and head gates go with sigmoid weights; windows, sinks and distance biases with a softmax")
+        if kv_from is not None and (conv or bias):
+            raise ValueError("a layer that reads another's keys and values has no convolution or biases of its own")
         self.scale, self.eps, self.dtype, self.taps = float(sizes["scale"]), eps, dtype, int(conv or 0)
         self.qk_norm, self.distance_bias, self.sink, self.out_scale = qk_norm, distance_bias, sink, float(out_scale)
         self.temp_coef, self.temp_every = (float(q_temp["coef"]), int(q_temp["every"])) if q_temp else (0.0, 1)
         self.biased, self.recurrent = bias, self.taps > 1
         self.dp, self.vp = pad8(self.dim), pad8(self.vdim)
         self.k_off = self.heads * self.dp
-        self.v_off = self.k_off + self.kv_heads * self.dp
-        self.in_cols, self.out_cols = self.v_off + self.kv_heads * self.vp, self.heads * self.vp
+        self.kv_from = kv_from
+        self.own_kv = 0 if kv_from is not None else self.kv_heads        # key heads that it projects and keeps
+        self.v_off = self.k_off + self.own_kv * self.dp
+        self.g_off = self.v_off + self.own_kv * self.vp
+        self.in_cols, self.out_cols = self.g_off + (pad8(self.heads) if head_gate else 0), self.heads * self.vp
+        self.chunk, self.head_gate = int(chunk), head_gate
+        self.key_bias = (nn.Parameter(torch.zeros(self.heads, dtype=torch.float32, device=device), requires_grad=False)
+                         if weights == "sigmoid" else None)
         self.conv_w = self.q_norm_w = self.k_norm_w = None
         if self.taps:
             self.conv_w = nn.Parameter(torch.zeros(self.taps, self.in_cols, dtype=dtype, device=device), requires_grad=False)
-        if qk_norm:
+        if qk_norm in ("head", "whole"):
             n = (1, 1) if qk_norm == "head" else (self.heads, self.kv_heads)
             self.q_norm_w, self.k_norm_w = (_vec(i * self.dp, dtype, device, 0.0) for i in n)
         self.device = torch.device(device)
@@ -584,11 +655,18 @@ class GroupedAttention(Part):
 
     # ---- cache and state ---------------------------------------------------------------------------------
     def cache_bytes_per_block(self, block_size: int) -> int:
-        return block_size * self.kv_heads * (self.dp + self.vp) * self.dtype.itemsize
+        return block_size * self.own_kv * (self.dp + self.vp) * self.dtype.itemsize
 
     def init_cache(self, kept: dict, num_blocks: int, block_size: int) -> None:
+        if self.kv_from is not None:
+            return                           # :meth:`SumMixer.share_cache`
         for name, n in (("k", self.dp), ("v", self.vp)):
             kept[name] = torch.zeros(num_blocks, block_size, self.kv_heads, n, dtype=self.dtype, device=self.device)
+
+    def reads(self, other: "GroupedAttention") -> bool:
+        """Whether ``other``'s cache holds keys and values as this part would have made them."""
+        alike = lambda p: (p.kv_heads, p.dim, p.vdim, p.dtype, p.rot and rotation_key(p.rot), p.rot_order is None)
+        return isinstance(other, GroupedAttention) and other.kv_from is None and alike(self) == alike(other)
 
     def state_bytes_per_slot(self) -> int:
         return max(0, self.taps - 1) * self.in_cols * self.dtype.itemsize
@@ -605,7 +683,7 @@ class GroupedAttention(Part):
 
     def launch_key(self, meta: AttentionMetadata, block_size: int, sm_count: int) -> tuple:
         return hops.attention_rows_plan(meta.num_single, self.heads, self.kv_heads, self.dp, self.vp, block_size, self.dtype,
-                                        meta.max_kv_len, sm_count, self.window, self.keep)
+                                        meta.max_kv_len, sm_count, self.window or self.chunk, self.keep)
 
     # ---- weights -------------------------------------------------------------------------------------------
     def _reordered(self, t: torch.Tensor) -> torch.Tensor:
@@ -616,7 +694,9 @@ class GroupedAttention(Part):
 
     def tensor_targets(self, width: int, load_in, load_bias, load_out) -> dict:
         H, G, D, V = self.heads, self.kv_heads, self.dim, self.vdim
-        spans = {"q": (H, D, self.dp, 0), "k": (G, D, self.dp, self.k_off), "v": (G, V, self.vp, self.v_off)}
+        spans = {"q": (H, D, self.dp, 0)}
+        if self.kv_from is None:
+            spans.update(k=(G, D, self.dp, self.k_off), v=(G, V, self.vp, self.v_off))
         out = {"o": ((width, H * V), lambda t: _by_head(lambda r, i: load_out(r.t(), i), V, self.vp, 0)(t.t()))}
         for name, (n, d, padded, base) in spans.items():
             out[name] = ((n * d, width), _by_head(load_in, d, padded, base))
@@ -625,7 +705,7 @@ class GroupedAttention(Part):
             if self.taps:
                 put = _pad_heads(self.conv_w[:, base:base + n * padded], n, d, padded)
                 out[name + ".conv"] = ((n * d, self.taps), lambda t, put=put: put(t.t()))
-        if self.qk_norm:
+        if self.q_norm_w is not None:
             for name, w, n in (("q", self.q_norm_w, H), ("k", self.k_norm_w, G)):
                 n = n if self.qk_norm == "whole" else 1
                 out[name + ".norm"] = ((n * D,), _pad_heads(w, n, D, self.dp))
@@ -633,16 +713,21 @@ class GroupedAttention(Part):
             for name, (shape, put) in list(out.items()):
                 if name[0] in "qk":
                     out[name] = (shape, lambda t, put=put: put(self._reordered(t)))
+        if self.key_bias is not None:
+            out["pb"] = ((H,), self.key_bias.data.copy_)
+        if self.head_gate:
+            out["g"] = ((H, width), lambda t: load_in(t, self.g_off))
         return out
 
     # ---- forward -------------------------------------------------------------------------------------------
     def mix(self, p: torch.Tensor, meta: AttentionMetadata, rt, out: torch.Tensor, kept: dict) -> None:
         q = rt.buffer("query", p.shape[0], self.k_off)
-        hops.qkv_prep(p, self.heads, self.kv_heads, self.dim, self.vdim, q, kept["k"], kept["v"], meta, self.conv_w,
-                      kept.get("conv"), self.qk_norm, self.q_norm_w, self.k_norm_w, self.eps, self.temp_coef,
+        own = (kept["k"], kept["v"]) if self.kv_from is None else (None, None)
+        hops.qkv_prep(p, self.heads, self.own_kv, self.dim, self.vdim, q, *own, meta, self.conv_w, kept.get("conv"), self.qk_norm, self.q_norm_w, self.k_norm_w, self.eps, self.temp_coef,
                       self.temp_every, self.cos_sin)
         hops.grouped_attention(q, kept["k"], kept["v"], out, meta, self.heads, self.kv_heads, self.scale, self.slopes,
-                               self.sink, self.out_scale, rt.sm_count, window=self.window, keep=self.keep)
+                               self.sink, self.out_scale, rt.sm_count, window=self.window, keep=self.keep,
+                               key_bias=self.key_bias, chunk=self.chunk, gate=p[:, self.g_off:] if self.head_gate else None)
 
 
 class LightningAttention(Part):
@@ -782,6 +867,13 @@ class SumMixer(Mixer):
         for name, part in self.parts.items():
             part.init_cache(kept[name], num_blocks, block_size)
 
+    def kv_sources(self) -> dict:
+        """part -> the layer whose part of that name keeps its keys and values"""
+        return {n: p.kv_from for n, p in self.parts.items() if getattr(p, "kv_from", None) is not None}
+
+    def share_cache(self, name: str, kept: dict, source_kept: dict) -> None:
+        kept[name].update((k, source_kept[name][k]) for k in ("k", "v"))
+
     def init_state(self, kept: dict, num_slots: int) -> None:
         for name, part in self.parts.items():
             part.init_state(kept[name], num_slots)
@@ -822,5 +914,5 @@ class SumMixer(Mixer):
         self.out_proj(mixed, out=out)
 
 
-MIXERS = {"latent_attention": LatentAttention, "mamba2": Mamba2Mixer, "sum": SumMixer}
+MIXERS = {"latent_attention": LatentAttention, "mamba2": Mamba2Mixer, "mingru": MinGRUMixer, "sum": SumMixer}
 FEED_FORWARDS = {"dense": PolyNormMLP, "activated": ActMLP, "routed": RoutedMLP}

@@ -43,9 +43,10 @@ def expert_index(tokens: int, top_k: int, experts: int, device) -> dict:
 
 def run_experts(x: torch.Tensor, topk_w: torch.Tensor, topk_ids: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, ws: dict,
                 out: torch.Tensor, act="silu", shared: Optional[torch.Tensor] = None,
-                gate: Optional[torch.Tensor] = None, pair_tiles: bool = True, max_ctas: int = 0) -> None:
-    """``out = sum_k w_k W2[e_k] act(W13[e_k] x) (+ gate * shared)`` (CUDA). ``ws``: the buffers of :func:`expert_index` and
-    the expert-sorted rows ``a_sorted``, ``act`` and ``y`` (in fp32 also ``gate_up``: that product has no gated form)."""
+                gate: Optional[torch.Tensor] = None, pair_tiles: bool = True, max_ctas: int = 0,
+                weigh_input: bool = False) -> None:
+    """``out = sum_k w_k W2[e_k] act(W13[e_k] x) (+ gate * shared, no gate: one)`` (CUDA); ``weigh_input``: the weight is on
+    the expert's input, ``W2[e_k] act(W13[e_k] (w_k x))``. ``ws``: the buffers of :func:`expert_index` and the expert-sorted rows ``a_sorted``, ``act`` and ``y`` (in fp32 also ``gate_up``: that product has no gated form)."""
     T, top_k = topk_ids.shape
     E, I2, H = w13.shape
     tile_rows = TILE_ROWS_PAIR if T * top_k >= 512 * E and pair_tiles else TILE_ROWS
@@ -57,11 +58,14 @@ def run_experts(x: torch.Tensor, topk_w: torch.Tensor, topk_ids: torch.Tensor, w
     a, mid = ws["a_sorted"][:n_rows], ws["act"][:n_rows]
     groups = dict(tile_expert=tile_expert, num_m_tiles=ws["meta"][:1], max_ctas=max_ctas, tile_rows=tile_rows)
     if x.dtype == torch.float32:
-        z = ops.gemm(a, w13.view(E * I2, H), out=ws["gate_up"][:n_rows], n_per_expert=I2, **groups)
+        z = ops.gemm(a, w13.view(E * I2, H), out=ws["gate_up"][:n_rows], n_per_expert=I2,
+                     row_scale=ws["row_scale"] if weigh_input else None, **groups)
         hops.glu(z, act, mid)
     else:
-        ops.gemm(a, w13.view(E * I2, H), out=mid, swiglu=True, act=act, n_per_expert=I2, **groups)
-    y = ops.gemm(mid, w2.view(E * H, I2 // 2), out=ws["y"][:n_rows], row_scale=ws["row_scale"], n_per_expert=H, **groups)
+        ops.gemm(a, w13.view(E * I2, H), out=mid, swiglu=True, act=act, n_per_expert=I2,
+                 in_scale=ws["row_scale"] if weigh_input else None, **groups)
+    y = ops.gemm(mid, w2.view(E * H, I2 // 2), out=ws["y"][:n_rows], row_scale=None if weigh_input else ws["row_scale"],
+                 n_per_expert=H, **groups)
     ops.moe_combine(y, sorted_pos, out, top_k, shared, gate)
 
 

@@ -13,6 +13,10 @@ runner this class shares:
   "streams": hyper-connections - several residual streams, every sublayer reads the norm of a weighted sum of them and all
   streams are rebuilt from the old ones and the sublayer's output; that and the next sublayer's norm are one kernel (one
   stream with weights of one is the usual pre-norm block);
+  "sandwich": a norm in front of every sublayer and one behind it, ``x += post(f(pre(x)))``; with ``depth_average`` a layer
+  passes on a weighted sum of the embedding output and all layers' results so far, which are kept for the step; norm, sum,
+  average and the next sublayer's norm are one kernel;
+* a layer may read the keys and values that an earlier one keeps (``GroupedAttention``'s ``kv_from``);
 * layers may be run several times in a row with the same weights (``ModelConfig.loop``); every pass keeps its own cache
   and state, and before each pass but the first the embedding output is added to the stream;
 * a table of embeddings of token pairs may be added to the token embeddings (``ModelConfig.bigram``);
@@ -53,6 +57,9 @@ class HybridRuntime:
         self.hidden.zero_()
         self.residual = torch.zeros(max_tokens, max(1, cfg.streams) * w8, dtype=torch.float32, device=device)
         self.sublayer = torch.zeros(max_tokens, w8, dtype=cfg.dtype, device=device)
+        # the embedding output and the results of the layers but the last, for averages over the depth
+        self.results = (torch.zeros(cfg.num_layers, max_tokens, w8, dtype=torch.float32, device=device)
+                        if cfg.depth_average else None)
         # the embedding output, for layers that run again
         self.first = torch.zeros(max_tokens, w8, dtype=torch.float32, device=device) if cfg.loop else None
         self.comm = TPCommunicator(self.staging, tp, tw_cfg.wait_budget_ms, tw_cfg.transport)
@@ -148,7 +155,54 @@ class StreamLayer(HybridLayer):
         return out
 
 
-BLOCKS = {"output_norm": HybridLayer, "parallel": ParallelLayer, "streams": StreamLayer}
+class Norm(nn.Module):
+    """Weights of a layer norm ("layer": weight and bias) or an RMS norm ("rms": weight alone)."""
+
+    def __init__(self, kind: str, width: int, dtype, device):
+        super().__init__()
+        if kind not in ("rms", "layer"):
+            raise ValueError(f"unknown norm {kind!r}")
+        vec = lambda fill: nn.Parameter(torch.full((width,), fill, dtype=dtype, device=device), requires_grad=False)
+        self.w, self.b = vec(1.0), vec(0.0) if kind == "layer" else None
+
+    @property
+    def pair(self) -> tuple:
+        return self.w, self.b
+
+    def tensor_targets(self, name: str) -> dict:
+        out = {name: ((self.w.numel(),), self.w.data.copy_)}
+        if self.b is not None:
+            out[name + ".b"] = ((self.b.numel(),), self.b.data.copy_)
+        return out
+
+
+class SandwichLayer(HybridLayer):
+    """``x += norm1b(mixer(norm1(x)))``, ``x += norm2b(ff(norm2(x)))``; ``dwa[j]``: weight of result j (0: the embedding
+    output, the last one: this layer's own) in what the layer passes on."""
+
+    def __init__(self, spec: dict, cfg: ModelConfig, *, device, index: int):
+        super().__init__(spec, cfg, device=device)
+        self.norm1_w = self.norm2_w = None          # in ``norms``
+        names = ("norm1", "norm1b") + (() if self.mlp is None else ("norm2", "norm2b"))
+        self.norms = nn.ModuleDict({n: Norm(cfg.norm, cfg.hidden_size, cfg.dtype, device) for n in names})
+        self.dwa = None
+        if cfg.depth_average:
+            own = torch.zeros(index + 2, dtype=torch.float32, device=device)
+            own[-1] = 1.0
+            self.dwa = nn.Parameter(own, requires_grad=False)
+
+    def tensor_targets(self) -> dict:
+        out = {f"mix.{k}": v for k, v in self.mixer.tensor_targets().items()}
+        if self.mlp is not None:
+            out.update({f"mlp.{k}": v for k, v in self.mlp.tensor_targets().items()})
+        for name, norm in self.norms.items():
+            out.update(norm.tensor_targets(name))
+        if self.dwa is not None:
+            out["dwa"] = (tuple(self.dwa.shape), self.dwa.data.copy_)
+        return out
+
+
+BLOCKS = {"output_norm": HybridLayer, "parallel": ParallelLayer, "streams": StreamLayer, "sandwich": SandwichLayer}
 
 
 def layer_runs(num_layers: int, loop: Optional[dict]) -> list[tuple[int, bool]]:
@@ -191,12 +245,19 @@ class HybridDecoder(nn.Module):
         if cfg.bigram:                      # one row per bucket, and one for tokens without a token before them
             self.bigram_w = nn.Parameter(torch.zeros(int(cfg.bigram["buckets"]) + 1, pad8(W), dtype=dt, device=device),
                                          requires_grad=False)
-        self.layers = nn.ModuleList([BLOCKS[cfg.block](s, cfg, device=device) for s in cfg.layers])
+        sandwich = cfg.block == "sandwich"
+        if not sandwich and (cfg.norm != "rms" or cfg.depth_average or cfg.embed_scale != 1.0):
+            raise ValueError("layer norms, depth averages and an embedding scale are built for sandwich blocks")
+        self.layers = nn.ModuleList([BLOCKS[cfg.block](s, cfg, device=device, **({"index": i} if sandwich else {}))
+                                     for i, s in enumerate(cfg.layers)])
         self.runs = layer_runs(len(self.layers), cfg.loop)
         if cfg.block != "parallel" and (cfg.loop or cfg.bigram):
             raise ValueError("loops and pair embeddings are built for parallel blocks")
         self.kept = [self.layers[i].mixer.new_kept() for i, _ in self.runs]
         self.final_norm_w = nn.Parameter(torch.ones(W, dtype=dt, device=device), requires_grad=False)
+        self.final_norm_b = (nn.Parameter(torch.zeros(W, dtype=dt, device=device), requires_grad=False)
+                             if cfg.norm == "layer" else None)
+        self._check_kv_sources()
         self.rt: Optional[HybridRuntime] = None
         mixers = [l.mixer for l in self.layers]
         latent = [m for m in mixers if isinstance(m, LatentAttention)]
@@ -208,6 +269,21 @@ class HybridDecoder(nn.Module):
         self.expand_window = 0 if any(not m.window for m in latent) else max((m.window for m in latent), default=0)
         self.tiles = (bool(latent or grouped) and all(m.expandable for m in latent) and all(m.tileable for m in grouped))
         self.recurrent = any(m.recurrent for m in mixers)
+
+    def _kv_sources(self):
+        """(layer, part, the layer whose keys and values it reads)"""
+        return [(i, part, j) for i, l in enumerate(self.layers) if isinstance(l.mixer, SumMixer)
+                for part, j in l.mixer.kv_sources().items()]
+
+    def _check_kv_sources(self) -> None:
+        for i, part, j in self._kv_sources():
+            if self.cfg.loop:
+                raise ValueError("layers that read another's keys and values do not run in loops")
+            source = self.layers[j].mixer if 0 <= j < i else None
+            if not isinstance(source, SumMixer) or part not in source.parts or not self.layers[i].mixer.parts[part].reads(
+                    source.parts[part]):
+                raise ValueError(f"layer {i} reads the keys and values of layer {j}: an earlier layer with projections of its "
+                                 "own, the same sizes and rotation is needed")
 
     # ---- runtime ---------------------------------------------------------------------------------------
     def setup_runtime(self, max_tokens: int, tw_cfg, provider: Optional[str] = None,
@@ -235,13 +311,15 @@ class HybridDecoder(nn.Module):
     def init_kv_cache(self, num_blocks: int, block_size: int) -> None:
         for (i, _), kept in zip(self.runs, self.kept):
             self.layers[i].mixer.init_cache(kept, num_blocks, block_size)
+        for i, part, j in self._kv_sources():
+            self.layers[i].mixer.share_cache(part, self.kept[i], self.kept[j])
 
     def init_state(self, num_slots: int) -> None:
         for (i, _), kept in zip(self.runs, self.kept):
             self.layers[i].mixer.init_state(kept, num_slots)
 
     def cache_tensors(self) -> list[torch.Tensor]:
-        return [t for kept in self.kept for t in _tensors(kept)]
+        return list({id(t): t for kept in self.kept for t in _tensors(kept)}.values())      # (some are shared)
 
     def drop_caches(self) -> None:
         self.kept = [self.layers[i].mixer.new_kept() for i, _ in self.runs]
@@ -318,6 +396,9 @@ class HybridDecoder(nn.Module):
         if cfg.block == "streams":
             self._forward_streams(step, x32.view(T, max(1, cfg.streams), -1), xa, y)
             return xa
+        if cfg.block == "sandwich":
+            self._forward_sandwich(step, x32, xa, y)
+            return xa
         if cfg.block == "parallel":
             first = rt.first[:T] if rt.first is not None else None
             hops.embed_norm(step.input_ids, self.embed_w, self.bigram_w, cfg.bigram, meta, x32, first,
@@ -355,6 +436,23 @@ class HybridDecoder(nn.Module):
                 alike = False
             hops.streams_step(y, x, layer.hc[-1], cfg.residual_mult, *behind, off, eps, xa, alike)
 
+    def _forward_sandwich(self, step, x32: torch.Tensor, xa: torch.Tensor, y: torch.Tensor) -> None:
+        rt, cfg, meta, eps = self.rt, self.cfg, step.meta, self.cfg.rms_norm_eps
+        results = rt.results[:, :x32.shape[0]] if rt.results is not None else None
+        hops.embed_sandwich(step.input_ids, self.embed_w, cfg.embed_scale, x32, results[0] if results is not None else None,
+                            self.layers[0].norms["norm1"].pair, eps, xa)
+        for i, (layer, kept) in enumerate(zip(self.layers, self.kept)):
+            last = i + 1 == len(self.layers)
+            nxt = (self.final_norm_w, self.final_norm_b) if last else self.layers[i + 1].norms["norm1"].pair
+            norms = layer.norms
+            layer.mixer(xa, meta, rt, y, kept)
+            behind = norms["norm1b"]
+            if layer.mlp is not None:
+                hops.sandwich_step(y, x32, behind.pair, norms["norm2"].pair, eps, xa)
+                layer.mlp(xa, rt, y)
+                behind = norms["norm2b"]
+            hops.sandwich_step(y, x32, behind.pair, nxt, eps, xa, layer.dwa, results, last)
+
     @torch.inference_mode()
     def compute_logits(self, hidden_rows: torch.Tensor) -> torch.Tensor:
         """fp32 logits ``[rows, vocab]``."""
@@ -365,6 +463,8 @@ class HybridDecoder(nn.Module):
         V, W = self.cfg.vocab_size, self.cfg.hidden_size
         out = {"embed": ((V, W), lambda t: self.embed_w.data[:, :W].copy_(t)),
                "final.norm": ((W,), self.final_norm_w.data.copy_)}
+        if self.final_norm_b is not None:
+            out["final.norm.b"] = ((W,), self.final_norm_b.data.copy_)
         if not self.cfg.tie_word_embeddings:
             out["head"] = ((V, W), lambda t: self.head.load_rows(t, 0))
         if self.bigram_w is not None:
@@ -405,7 +505,7 @@ class HybridDecoder(nn.Module):
         def fill(name, shape):
             t = torch.empty(shape, dtype=torch.float32, device=dev)
             leaf = name.split(".mix.")[-1]
-            if name.endswith(("norm1", "norm2", "final.norm")):
+            if name.endswith(("norm1", "norm2", "norm1b", "norm2b", "final.norm")):
                 return t.fill_(1.0 - self.cfg.norm_offset)
             if name.endswith("norm") or leaf == "D":
                 return t.fill_(1.0)
@@ -413,6 +513,14 @@ class HybridDecoder(nn.Module):
                 return t.copy_(torch.eye(shape[0]) if leaf.endswith("mix") else torch.full(shape, 1.0 / shape[0]))
             if leaf == "sink" or name.endswith(".correction"):
                 return t.zero_()
+            if leaf == "pb":                    # keys count about one in a few tens
+                return t.fill_(-3.0)
+            if leaf == "z.b":                   # memories of a few to a few hundred tokens
+                return t.uniform_(-6.0, -1.0, generator=g)
+            if name.endswith(".dwa"):
+                t.fill_(0.2 / max(1, shape[0] - 1))
+                t[-1] = 0.8
+                return t
             if leaf == "A_log":
                 return t.uniform_(1.0, 16.0, generator=g).log_()
             if leaf == "dt_bias":

@@ -7,6 +7,7 @@ from ..config import EngineConfig
 
 
 def get_model_class(architecture: str):
+    from .giforax import GiforaxForCausalLM
     from .kebopel import KebopelForCausalLM
     from .llama import LlamaForCausalLM
     from .mistral import MistralForCausalLM
@@ -18,7 +19,8 @@ def get_model_class(architecture: str):
     from .sidisun import SidisunForCausalLM
     table = {"llama": LlamaForCausalLM, "qwen2": Qwen2ForCausalLM, "mixtral": MixtralForCausalLM,
              "qwen3": Qwen3ForCausalLM, "mistral": MistralForCausalLM, "phi3": Phi3ForCausalLM,
-             "sidisun": SidisunForCausalLM, "kebopel": KebopelForCausalLM, "netezen": NetezenForCausalLM}
+             "sidisun": SidisunForCausalLM, "kebopel": KebopelForCausalLM, "netezen": NetezenForCausalLM,
+             "giforax": GiforaxForCausalLM}
     if architecture not in table:
         raise ValueError(f"unsupported architecture {architecture!r} (supported: {sorted(table)})")
     return table[architecture]
@@ -26,7 +28,7 @@ def get_model_class(architecture: str):
 
 def load_config_readers() -> None:
     """Imports the modules that register a reader for their own ``config.json`` layout."""
-    from . import kebopel, netezen, sidisun  # noqa: F401
+    from . import giforax, kebopel, netezen, sidisun  # noqa: F401
 
 
 def build_model(config: EngineConfig, device: torch.device, embedding_parallel: bool = False):

@@ -88,11 +88,13 @@ COL_ACTS = {"silu": 1, "relu2": 2}
 def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *,
          bias: Optional[torch.Tensor] = None, row_scale: Optional[torch.Tensor] = None, swiglu: bool = False,
          act: "str | tuple" = "silu", col_act: Optional[tuple[str, int, int]] = None, max_ctas: int = 0,
+         in_scale: Optional[torch.Tensor] = None,
          tile_expert: Optional[torch.Tensor] = None,
          num_m_tiles: Optional[torch.Tensor] = None, n_per_expert: int = 0, tile_rows: int = 128) -> torch.Tensor:
     """``out = a @ w.T`` (+bias, *row_scale); with ``swiglu`` the weight is ``[gate; up]`` and the
     output is ``act(a@gate.T) * (a@up.T)``, ``act`` "silu", "gelu_tanh" or ("clamped", limit, alpha):
-    ``g sigmoid(alpha g) (u + 1)`` with ``g = min(a@gate.T, limit)`` and ``u = a@up.T`` inside ``[-limit, limit]``.
+    ``g sigmoid(alpha g) (u + 1)`` with ``g = min(a@gate.T, limit)`` and ``u = a@up.T`` inside ``[-limit, limit]``;
+    ``in_scale`` (fp32, with the clamped form): factors on the rows of ``a``, so on both halves before the clamps.
     ``col_act`` = ("silu" or "relu2", begin, end): that activation on these columns of a plain product (behind the bias;
     relu2: the square of relu). Grouped mode (``tile_expert`` given): every ``tile_rows``-row
     tile of ``a`` multiplies the weight block of its expert, ``w`` being ``[E * n_per_expert, K]``;
@@ -103,6 +105,8 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
     N = per_expert // 2 if swiglu else per_expert
     if out is None:
         out = torch.empty(M, N, dtype=a.dtype, device=a.device)
+    if in_scale is not None and (not swiglu or isinstance(act, str)):
+        raise ValueError("factors on the input's rows go with the clamped gated product")
     if not a.is_cuda:
         if act != "silu" or col_act is not None:
             raise NotImplementedError("these epilogues on CPU go through ops.reference_hybrid")
@@ -139,7 +143,8 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out: Optional[torch.Tensor] = None, *
             raise ValueError(f"unknown gated product {act!r}, or a bias or row scales with it")
         grouped = tile_expert is not None
         _native.call("tw_gemm_bf16_clamped", a.data_ptr(), _row_stride(a), w.data_ptr(), _row_stride(w), rows_b,
-                     out.data_ptr(), _row_stride(out), M, N, K, float(limit), float(alpha), per_expert // 2, _p(tile_expert),
+                     out.data_ptr(), _row_stride(out), _p(in_scale), M, N, K, float(limit), float(alpha), per_expert // 2,
+                     _p(tile_expert),
                      _p(num_m_tiles), per_expert, tile_rows, max_ctas,
                      0 if grouped else gemm_table.lookup(M, N, K, True, max_ctas), status_word(a.device).data_ptr(),
                      _stream(), tag=f"[{'grouped ' if grouped else ''}{M}x{N}x{K}+clamped]" if _native._timing is not None else "")
@@ -704,13 +709,14 @@ def moe_router(x: torch.Tensor, gate_w: torch.Tensor, topk: int, renormalize: bo
 
 
 def moe_route(x: torch.Tensor, w: torch.Tensor, experts: int, topk: int, correction: Optional[torch.Tensor] = None,
-              sum_eps: float = 0.0):
+              sum_eps: float = 0.0, scores: str = "softmax", normalize: bool = True):
     """The general router, bf16 or fp32. ``w`` [experts + gates, >= width]: a row per expert, then a row per gate. Scores
-    are the softmax over all experts; the ``topk`` with the largest score + ``correction`` (fp32 [experts]) are chosen, their
-    weights are the scores without it over (their sum + ``sum_eps``). Returns (weights fp32 [T, k], ids int32 [T, k],
+    are the softmax over all experts or (``scores`` "sigmoid") each logit's sigmoid; the ``topk`` with the largest score +
+    ``correction`` (fp32 [experts]) are chosen, their weights are the scores without it, with ``normalize`` over (their sum +
+    ``sum_eps``). Returns (weights fp32 [T, k], ids int32 [T, k],
     sigmoid of the gate rows fp32 [T, gates])."""
     if not x.is_cuda:
-        return reference.moe_route(x, w, experts, topk, correction, sum_eps)
+        return reference.moe_route(x, w, experts, topk, correction, sum_eps, scores, normalize)
     if x.dtype != w.dtype or x.dtype not in (torch.bfloat16, torch.float32):
         raise TypeError(f"expected rows and router of one type, bfloat16 or float32, got {x.dtype} and {w.dtype}")
     T, H = x.shape
@@ -718,7 +724,8 @@ def moe_route(x: torch.Tensor, w: torch.Tensor, experts: int, topk: int, correct
     ids = torch.empty(T, topk, dtype=torch.int32, device=x.device)
     wts, gate = (torch.empty(T, n, dtype=torch.float32, device=x.device) for n in (topk, gates))
     _native.call("tw_moe_route", x.data_ptr(), _row_stride(x), w.data_ptr(), _row_stride(w), _p(correction), wts.data_ptr(),
-                 ids.data_ptr(), gate.data_ptr() if gates else None, T, H, experts, gates, topk, float(sum_eps),
+                 ids.data_ptr(), gate.data_ptr() if gates else None, T, H, experts, gates, topk,
+                 {"softmax": 0, "sigmoid": 1}[scores], int(normalize), float(sum_eps),
                  0 if x.dtype == torch.bfloat16 else 1, _stream())
     return wts, ids, gate
 
@@ -743,7 +750,7 @@ def moe_scatter(x: torch.Tensor, topk_ids: torch.Tensor, topk_w: torch.Tensor, e
 
 def moe_combine(y_sorted: torch.Tensor, sorted_pos: torch.Tensor, out: torch.Tensor, topk: int,
                 shared: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
-    """``out = sum over a token's experts`` of their weighted rows, ``+ gate * shared`` (one gate per token)."""
+    """``out = sum over a token's experts`` of their rows, ``+ gate * shared`` (one gate per token, or none)."""
     T, H = out.shape
     _native.call("tw_moe_combine", y_sorted.data_ptr(), sorted_pos.data_ptr(), _p(shared),
                  _row_stride(shared) if shared is not None else 0, _p(gate), out.data_ptr(), _row_stride(out),

@@ -53,7 +53,7 @@ _SIGNATURES = {
     "tw_moe_align": [vp, i32, i32, i32, vp, vp, vp, i32, vp, vp],
     "tw_moe_scatter": [vp, ll, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, vp],
     "tw_moe_combine": [vp, vp, vp, ll, vp, vp, ll, i32, i32, i32, i32, vp],
-    "tw_moe_route": [vp, ll, vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, i32, f32, i32, vp],
+    "tw_moe_route": [vp, ll, vp, ll, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp],
     "tw_fused_rs_norm_ag": [vp, vp, vp, i32, i32, i32, u64, vp, ll, vp, ll, vp, i32, i32, f32, i32, i32, i32,
                             vp],
     "tw_collective": [vp, vp, vp, i32, i32, i32, u64, vp, ll, ll, i32, i32, vp],
@@ -67,6 +67,9 @@ _SIGNATURES = {
     "tw_gemm_f32_grouped": [vp, ll, vp, ll, vp, ll, i32, i32, i32, vp, vp, i32, i32, vp, vp],
     "tw_embed_streams": [vp, vp, ll, i32, vp, ll, ll, i32, vp, vp, f32, vp, ll, i32, i32, f32, i32, vp],
     "tw_streams_step": [vp, ll, vp, ll, ll, i32, vp, vp, f32, vp, i32, i32, vp, f32, vp, ll, i32, i32, f32, i32, vp],
+    "tw_embed_sandwich": [vp, vp, ll, i32, f32, vp, ll, vp, ll, vp, vp, i32, vp, ll, i32, i32, f32, i32, vp],
+    "tw_sandwich_step": [vp, ll, vp, ll, i32, vp, vp, vp, ll, ll, i32, vp, vp, vp, vp, i32, vp, ll, i32, i32, f32, i32, vp],
+    "tw_min_gru": [vp, ll, vp, vp, vp, vp, ll, vp, i32, vp, vp, vp, i32, i32, i32, vp],
     "tw_embed_residual": [vp, vp, ll, vp, ll, vp, ll, i32, i32, i32, i32, vp],
     "tw_postnorm_add": [vp, ll, vp, ll, vp, vp, ll, vp, i32, i32, f32, i32, vp],
     "tw_polynorm": [vp, ll, vp, vp, ll, i32, i32, f32, i32, vp],
@@ -79,13 +82,13 @@ _SIGNATURES = {
     "tw_qkv_prep": [vp, ll, i32, i32, i32, i32, i32, i32, vp, ll, vp, vp, vp, vp, vp, vp, i32, vp, vp, vp, vp, i32, i32,
                     i32, vp, vp, f32, f32, i32, vp, i32, i32, vp],
     "tw_attn_rows": [vp, ll, vp, vp, i32, vp, ll, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, f32, vp, i32, f32, i32, i32,
-                     i32, vp],
+                     vp, i32, vp, ll, i32, vp],
     "tw_attn_prefill_grouped": [vp, ll, i32, vp, vp, i32, i32, vp, ll, vp, vp, vp, i32, vp, vp, i32, i32, i32, i32, i32,
-                                f32, vp, i32, f32, i32, i32, vp, vp],
+                                f32, vp, i32, f32, i32, i32, vp, i32, vp, ll, vp, vp],
     "tw_attn_decode_grouped": [vp, ll, vp, vp, i32, i32, vp, ll, vp, vp, vp, i32, vp, i32, i32, i32, i32, i32, f32, vp, i32,
-                               f32, i32, i32, i32, vp, vp, vp, vp],
+                               f32, i32, i32, vp, i32, vp, ll, i32, vp, vp, vp, vp],
     "tw_gemm_bf16_act": [vp, ll, vp, ll, vp, ll, vp, i32, i32, i32, i32, i32, i32, i32, i32, vp, vp],
-    "tw_gemm_bf16_clamped": [vp, ll, vp, ll, ll, vp, ll, i32, i32, i32, f32, f32, i32, vp, vp, i32, i32, i32, i32, vp, vp],
+    "tw_gemm_bf16_clamped": [vp, ll, vp, ll, ll, vp, ll, vp, i32, i32, i32, f32, f32, i32, vp, vp, i32, i32, i32, i32, vp, vp],
     "tw_latent_prep": [vp, ll, i32, i32, vp, vp, ll, i32, i32, vp, i32, i32, vp, vp, vp, vp, i32, i32, f32, i32, vp],
     "tw_rope_tail": [vp, ll, i32, i32, i32, i32, i32, vp, vp, i32, vp],
     "tw_latent_query": [vp, ll, vp, i32, vp, i32, i32, i32, i32, i32, i32, i32, vp, vp, i32, vp],

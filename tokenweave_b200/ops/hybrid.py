@@ -2,7 +2,8 @@
 over a paged latent cache, the state-space (Mamba-2) recurrence with its convolution, the norm of a sublayer's output
 added to the residual, and the polynomial-norm activation; for blocks whose sublayers read one norm of the stream,
 grouped attention with its options (query and key norms, short convolution, rotation, query temperature, distance bias,
-sink, sliding window), lightning attention, embeddings with token pairs, and the fused projections; hyper-connections.
+sink, sliding window, sigmoid weights in chunks), lightning attention, embeddings with token pairs, and the fused projections;
+hyper-connections; norms on both sides of a sublayer with averages over the depth; the minGRU recurrence.
 
 Like the other operators, CUDA tensors (bf16 or fp32) go to the kernels of ``_C.so`` and CPU tensors to plain PyTorch
 (:mod:`.reference_hybrid`). ``meta`` below is the step's :class:`~tokenweave_b200.layers.attention.AttentionMetadata`.
@@ -104,6 +105,62 @@ def streams_step(y: torch.Tensor, x: torch.Tensor, hc: dict, mult: float, next_i
                  _dt(y, weight, xa), _stream())
 
 
+# ---- norms on both sides of a sublayer, averages over the depth -------------------------------------------------
+# A norm is a pair (weight, bias): a layer norm, or (weight, None): an RMS norm. ``results``: fp32 [layers, T, padded width],
+# the embedding output and the layers' results in order.
+def embed_sandwich(ids: torch.Tensor, table: torch.Tensor, scale: float, x32: torch.Tensor, first: Optional[torch.Tensor],
+                   norm: tuple, eps: float, xa: torch.Tensor) -> None:
+    """``x32 = scale * table[ids]``; ``first``: a copy of it; ``xa`` its norm."""
+    w, b = norm
+    if not table.is_cuda:
+        ref.embed_sandwich(ids, table, scale, x32, first, norm, eps, xa)
+        return
+    assert ids.dtype == torch.int32 and x32.dtype == torch.float32 and (first is None or first.dtype == torch.float32)
+    _native.call("tw_embed_sandwich", ids.data_ptr(), table.data_ptr(), _row_stride(table), table.shape[0], float(scale),
+                 x32.data_ptr(), _row_stride(x32), _p(first), _row_stride(first) if first is not None else 0, w.data_ptr(),
+                 _p(b), int(b is not None), xa.data_ptr(), _row_stride(xa), ids.shape[0], w.numel(), float(eps),
+                 _dt(table, w, b, xa), _stream())
+
+
+def sandwich_step(y: torch.Tensor, x32: torch.Tensor, post: tuple, nxt: tuple, eps: float, xa: torch.Tensor,
+                  coef: Optional[torch.Tensor] = None, results: Optional[torch.Tensor] = None, last: bool = False) -> None:
+    """``x32 += norm_post(y)``; behind a layer, with ``coef`` (fp32 [n + 1]): the sum is result n (kept in ``results[n]``,
+    unless ``last``) and ``x32 = sum_j coef[j] results[j]``; then ``xa = norm_next(x32)``. ``last``: behind the last sublayer,
+    the stream itself is not stored."""
+    (w, b), (wn, bn) = post, nxt
+    if (b is None) != (bn is None):
+        raise ValueError("norms of one kind are needed")
+    n = coef.numel() - 1 if coef is not None else 0
+    if not y.is_cuda:
+        ref.sandwich_step(y, x32, post, nxt, eps, xa, coef, results, last)
+        return
+    assert x32.dtype == torch.float32 and (coef is None or (coef.dtype == results.dtype == torch.float32
+                                                            and results.stride(2) == 1 and results.shape[0] >= n + (not last)))
+    keep = results[n] if coef is not None and not last else None
+    ldp, lds = (results.stride(1), results.stride(0)) if coef is not None else (0, 0)
+    _native.call("tw_sandwich_step", y.data_ptr(), _row_stride(y), x32.data_ptr(), _row_stride(x32), int(not last),
+                 w.data_ptr(), _p(b), _p(results) if coef is not None else None, ldp, lds, n, _p(coef), _p(keep),
+                 wn.data_ptr(), _p(bn), int(b is not None), xa.data_ptr(), _row_stride(xa), y.shape[0], w.numel(), float(eps),
+                 _dt(y, w, b, wn, bn, xa), _stream())
+
+
+# ---- minGRU -----------------------------------------------------------------------------------------------------
+def min_gru(p: torch.Tensor, bz: torch.Tensor, bx: torch.Tensor, state: torch.Tensor, out: torch.Tensor, seqs: torch.Tensor,
+            cu_q: torch.Tensor, kv_lens: torch.Tensor, slots: torch.Tensor, chunked: bool = False) -> None:
+    """Per channel ``z = sigmoid(pz + bz)``, ``u = px + bx``, ``S <- (1 - z) S + z (u + 1/2 if u >= 0 else sigmoid(u))``,
+    ``out = S silu(pg)`` of the listed sequences; ``p`` rows are [pz | px | pg], each as wide as ``state`` (fp32 [slots,
+    channels, a multiple of eight]). ``chunked``: many tokens at a time (long runs)."""
+    if seqs.shape[0] == 0:
+        return
+    if not p.is_cuda:
+        ref.min_gru(p, bz, bx, state, out, seqs, cu_q, kv_lens, slots)
+        return
+    assert state.dtype == bz.dtype == bx.dtype == torch.float32
+    _native.call("tw_min_gru", p.data_ptr(), _row_stride(p), bz.data_ptr(), bx.data_ptr(), state.data_ptr(), out.data_ptr(),
+                 _row_stride(out), seqs.data_ptr(), seqs.shape[0], cu_q.data_ptr(), kv_lens.data_ptr(), slots.data_ptr(),
+                 state.shape[1], int(chunked), _dt(p, out), _stream())
+
+
 # ---- latent attention -----------------------------------------------------------------------------------------
 def latent_row(kv_rank: int, rot: int) -> int:
     """Elements of a latent cache row: the latent and the rotated key part, each padded to eight."""
@@ -150,7 +207,7 @@ def latent_absorb(q: torch.Tensor, rows: torch.Tensor, w_ukt: torch.Tensor, head
 
 
 def _key_tiles(max_kv_len: int, window: int = 0, keep: int = 0) -> int:
-    """Most 128-key tiles that hold visible keys of one row."""
+    """Most 128-key tiles that hold visible keys of one row (``window``: of a window or a chunk)."""
     tiles = (max_kv_len + 127) // 128
     return min(tiles, (window + 126) // 128 + 1 + (keep + 127) // 128) if window else tiles
 
@@ -434,27 +491,29 @@ def gated_product(x: torch.Tensor, w: torch.Tensor, act: "str | tuple", out: tor
 
 
 # ---- grouped attention ------------------------------------------------------------------------------------------------
-QK_NORMS = {None: 0, "head": 1, "whole": 2}
+QK_NORMS = {None: 0, "head": 1, "whole": 2, "unit": 1}       # "unit": per head, without weights
 
 
-def qkv_prep(p: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, q: torch.Tensor, k_cache: torch.Tensor,
-             v_cache: torch.Tensor, meta, conv_w: Optional[torch.Tensor], conv_state: Optional[torch.Tensor],
+def qkv_prep(p: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int, q: torch.Tensor,
+             k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], meta, conv_w: Optional[torch.Tensor], conv_state: Optional[torch.Tensor],
              qk_norm: Optional[str], wq: Optional[torch.Tensor], wk: Optional[torch.Tensor], eps: float, temp_coef: float,
              temp_every: int, cos_sin: Optional[torch.Tensor] = None) -> None:
     """Everything between the projection and the attention. ``p`` rows are [queries | keys | values], heads padded to
     the caches' last dimension; ``conv_w`` [taps, columns] and ``conv_state`` [slots, taps - 1, columns]: causal
-    convolution over time, the state moved on; norm of queries and keys per head or whole; rotation of the first
+    convolution over time, the state moved on; norm of queries and keys per head (with weights, or "unit") or whole; rotation of the first
     ``cos_sin.shape[1]`` dimensions of every query and key head (dimensions 2i and 2i + 1 are a pair; the table's rows are
     cosines, then sines, by position); queries times ``1 + temp_coef * ln(floor((position + 1) / temp_every) + 1)``; ``q`` [T, heads * padded], keys and values into the
-    caches [blocks, page, kv_heads, padded]."""
+    caches [blocks, page, kv_heads, padded]. Without key heads (and caches) the rows hold queries only."""
     if not p.is_cuda:
         ref.qkv_prep(p, heads, kv_heads, dim, vdim, q, k_cache, v_cache, meta, conv_w, conv_state, qk_norm, wq, wk, eps,
                      temp_coef, temp_every, cos_sin)
         return
     e = meta.extra
     assert cos_sin is None or (cos_sin.dtype == torch.float32 and cos_sin.is_contiguous())
-    _native.call("tw_qkv_prep", p.data_ptr(), _row_stride(p), p.shape[0], heads, kv_heads, dim, k_cache.shape[-1],
-                 v_cache.shape[-1], q.data_ptr(), _row_stride(q), k_cache.data_ptr(), v_cache.data_ptr(),
+    dp = q.shape[1] // heads
+    assert kv_heads == 0 or k_cache.shape[-1] == dp
+    _native.call("tw_qkv_prep", p.data_ptr(), _row_stride(p), p.shape[0], heads, kv_heads, dim, dp,
+                 v_cache.shape[-1] if v_cache is not None else dp, q.data_ptr(), _row_stride(q), _p(k_cache), _p(v_cache),
                  meta.positions.data_ptr(), meta.slot_mapping.data_ptr(), _p(conv_w), _p(conv_state),
                  conv_w.shape[0] if conv_w is not None else 1, _p(e.get("row_seq")), meta.cu_q.data_ptr(),
                  meta.kv_lens.data_ptr(), _p(e.get("state_slots")), meta.num_seqs, int(meta.all_single),
@@ -479,31 +538,42 @@ def attention_rows_plan(n: int, heads: int, kv_heads: int, dp: int, vp: int, pag
 
 def grouped_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, out: torch.Tensor, meta, heads: int,
                       kv_heads: int, scale: float, slopes: Optional[torch.Tensor], sink: bool, out_scale: float,
-                      sm_count: int = 148, kernel: Optional[str] = None, window: int = 0, keep: int = 0) -> None:
+                      sm_count: int = 148, kernel: Optional[str] = None, window: int = 0, keep: int = 0,
+                      key_bias: Optional[torch.Tensor] = None, chunk: int = 0, gate: Optional[torch.Tensor] = None) -> None:
     """Causal attention of a step's rows over the paged caches; head h's score loses ``slopes[h] * (i - j)``; ``sink``
     adds one to the denominator; the result is multiplied by ``out_scale``; ``window`` > 0: a row sees the last ``window``
-    keys, itself among them, and the sequence's first ``keep``. ``kernel``: force "simt" (tests)."""
+    keys, itself among them, and the sequence's first ``keep``. With ``key_bias`` (fp32 [heads]) there is no softmax: a key
+    counts with the sigmoid of its score + ``key_bias[h]``; ``chunk`` > 0: a row sees the keys of its own chunk of that many
+    positions, counted from the sequence's start; ``gate`` [T, >= heads]: head h's result times ``sigmoid(gate[:, h])``
+    (these options go together, without those of the softmax). ``kernel``: force "simt" (tests)."""
+    if key_bias is None and (chunk or gate is not None) or key_bias is not None and (window or sink or slopes is not None):
+        raise ValueError("chunks and gates go with sigmoid weights; windows, sinks and distance biases with a softmax")
     if not q.is_cuda:
-        ref.grouped_attention(q, k_cache, v_cache, out, meta, heads, kv_heads, scale, slopes, sink, out_scale, window, keep)
+        ref.grouped_attention(q, k_cache, v_cache, out, meta, heads, kv_heads, scale, slopes, sink, out_scale, window, keep,
+                              key_bias, chunk, gate)
         return
-    dt = _dt(q, k_cache, v_cache, out)
+    dt = _dt(q, k_cache, v_cache, out, gate)
+    assert key_bias is None or key_bias.dtype == torch.float32
+    sigmoid = (_p(key_bias), int(chunk), _p(gate), _row_stride(gate) if gate is not None else 0)
     page, dp, vp = k_cache.shape[1], k_cache.shape[-1], v_cache.shape[-1]
     if meta.num_tiles:
         _native.call("tw_attn_prefill_grouped", q.data_ptr(), _row_stride(q), q.shape[0], k_cache.data_ptr(),
                      v_cache.data_ptr(), k_cache.shape[0], page, out.data_ptr(), _row_stride(out), meta.cu_q.data_ptr(),
                      meta.kv_lens.data_ptr(), meta.block_table.data_ptr(), meta.block_table.shape[1],
                      meta.tile_seq.data_ptr(), meta.tile_q0.data_ptr(), meta.num_tiles, heads, kv_heads, dp, vp,
-                     float(scale), _p(slopes), int(sink), float(out_scale), int(window), int(keep),
+                     float(scale), _p(slopes), int(sink), float(out_scale), int(window), int(keep), *sigmoid,
                      status_word(q.device).data_ptr(), _stream())
     n = meta.num_single
     if n == 0:
         return
-    plan, splits = attention_rows_plan(n, heads, kv_heads, dp, vp, page, q.dtype, meta.max_kv_len, sm_count, window, keep)
+    plan, splits = attention_rows_plan(n, heads, kv_heads, dp, vp, page, q.dtype, meta.max_kv_len, sm_count, window or chunk,
+                                       keep)
     if (kernel or plan) == "simt":
         _native.call("tw_attn_rows", q.data_ptr(), _row_stride(q), k_cache.data_ptr(), v_cache.data_ptr(), page,
                      out.data_ptr(), _row_stride(out), meta.tok_row.data_ptr(), meta.tok_seq.data_ptr(),
                      meta.tok_kvlen.data_ptr(), n, meta.block_table.data_ptr(), meta.block_table.shape[1], heads, kv_heads,
-                     dp, vp, float(scale), _p(slopes), int(sink), float(out_scale), int(window), int(keep), dt, _stream())
+                     dp, vp, float(scale), _p(slopes), int(sink), float(out_scale), int(window), int(keep), *sigmoid, dt,
+                     _stream())
         return
     po = pm = None
     if splits > 1:
@@ -511,5 +581,6 @@ def grouped_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Ten
     _native.call("tw_attn_decode_grouped", q.data_ptr(), _row_stride(q), k_cache.data_ptr(), v_cache.data_ptr(),
                  k_cache.shape[0], page, out.data_ptr(), _row_stride(out), meta.tok_row.data_ptr(), meta.tok_seq.data_ptr(),
                  meta.tok_kvlen.data_ptr(), n, meta.block_table.data_ptr(), meta.block_table.shape[1], heads, kv_heads, dp,
-                 vp, float(scale), _p(slopes), int(sink), float(out_scale), int(window), int(keep), splits, _p(po), _p(pm),
+                 vp, float(scale), _p(slopes), int(sink), float(out_scale), int(window), int(keep), *sigmoid, splits, _p(po),
+                 _p(pm),
                  status_word(q.device).data_ptr(), _stream())

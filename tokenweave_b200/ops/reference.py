@@ -381,30 +381,35 @@ def moe_router(x: torch.Tensor, gate_w: torch.Tensor, topk: int, renormalize: bo
 
 
 def moe_route(x: torch.Tensor, w: torch.Tensor, experts: int, topk: int, correction: Optional[torch.Tensor],
-              sum_eps: float):
-    """Softmax scores over all experts, choice by score + correction, weights from the scores of the chosen ones; the rows
-    of ``w`` behind the experts' are gates. Returns (weights, ids, sigmoid gates)."""
+              sum_eps: float, scores: str = "softmax", normalize: bool = True):
+    """Softmax scores over all experts (or sigmoid scores), choice by score + correction, weights from the scores of the
+    chosen ones; the rows of ``w`` behind the experts' are gates. Returns (weights, ids, sigmoid gates)."""
     logits = x.float() @ w.float().t()
-    scores = torch.softmax(logits[:, :experts], dim=-1)
-    choice = scores if correction is None else scores + correction
+    s = torch.softmax(logits[:, :experts], dim=-1) if scores == "softmax" else torch.sigmoid(logits[:, :experts])
+    choice = s + correction if correction is not None else logits[:, :experts]
     ids = torch.topk(choice, topk, dim=-1).indices
-    chosen = scores.gather(1, ids)
-    return chosen / (chosen.sum(-1, keepdim=True) + sum_eps), ids.to(torch.int32), torch.sigmoid(logits[:, experts:])
+    chosen = s.gather(1, ids)
+    return chosen / (chosen.sum(-1, keepdim=True) + sum_eps) if normalize else chosen, ids.to(torch.int32), torch.sigmoid(logits[:, experts:])
 
 
-def gemm_clamped(a: torch.Tensor, w_gate_up: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
-    """``g sigmoid(alpha g) (u + 1)`` with ``g = min(a @ Wg.T, limit)``, ``u = a @ Wu.T`` inside ``[-limit, limit]``."""
+def gemm_clamped(a: torch.Tensor, w_gate_up: torch.Tensor, limit: float, alpha: float,
+                 in_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``g sigmoid(alpha g) (u + 1)`` with ``g = min(a @ Wg.T, limit)``, ``u = a @ Wu.T`` inside ``[-limit, limit]``;
+    ``in_scale``: factors on the rows of ``a``."""
     y = a.float() @ w_gate_up.float().t()
+    if in_scale is not None:
+        y = y * in_scale[:, None]
     g, u = y.chunk(2, -1)
     g, u = g.clamp(max=limit), u.clamp(-limit, limit)
     return (g * torch.sigmoid(alpha * g) * (u + 1)).to(a.dtype)
 
 
 def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: torch.Tensor,
-                topk_ids: torch.Tensor, act="silu") -> torch.Tensor:
+                topk_ids: torch.Tensor, act="silu", weigh_input: bool = False) -> torch.Tensor:
     """Loop-over-experts MoE MLP: ``sum_k w_k * W2[e_k] (silu(W1[e_k] x) * W3[e_k] x)``, or with the clamped gate
     ``act = ("clamped", limit, alpha)``. ``w13``: [E, 2*I, H] (gate rows first), ``w2``: [E, H, I]. The activation and the
-    weighted expert output are rounded to the storage dtype, the top-k sum runs in fp32."""
+    weighted expert output are rounded to the storage dtype, the top-k sum runs in fp32. ``weigh_input``: the weight is on
+    the expert's input, before its activation (clamped gate)."""
     T, H = x.shape
     E = w13.shape[0]
     out = torch.zeros(T, H, dtype=torch.float32, device=x.device)
@@ -414,8 +419,10 @@ def moe_experts(x: torch.Tensor, w13: torch.Tensor, w2: torch.Tensor, topk_w: to
         if tok.numel() == 0:
             continue
         xe = x.index_select(0, tok)
-        mid = gemm_swiglu(xe, w13[e]) if act == "silu" else gemm_clamped(xe, w13[e], *act[1:])
-        ye = gemm(mid, w2[e], row_scale=topk_w[tok, slot])
+        wt = topk_w[tok, slot]
+        mid = (gemm_swiglu(xe, w13[e]) if act == "silu"
+               else gemm_clamped(xe, w13[e], *act[1:], in_scale=wt if weigh_input else None))
+        ye = gemm(mid, w2[e], row_scale=None if weigh_input else wt)
         out.index_add_(0, tok, ye.float())
     return out.to(x.dtype)
 

@@ -162,6 +162,51 @@ def decay_scan(p, decay, state, y, seqs, cu_q, kv_lens, slots) -> None:
     _recurrence(r[:, :inner].reshape(T, heads, vdim), k, q, one * decay, one, None, state, y, seqs, cu_q, kv_lens, slots)
 
 
+# ---- norms on both sides of a sublayer, averages over the depth -----------------------------------------------------
+def _norm(x, norm, eps: float):
+    w, b = norm
+    if b is None:
+        return _unit(x, eps) * w.float()
+    return _unit(x - x.mean(-1, keepdim=True), eps) * w.float() + b.float()
+
+
+def embed_sandwich(ids, table, scale: float, x32, first, norm, eps: float, xa) -> None:
+    h = norm[0].numel()
+    ok = (ids >= 0) & (ids < table.shape[0])
+    x = table.index_select(0, torch.where(ok, ids, torch.zeros_like(ids)).long())[:, :h].float() * ok.unsqueeze(-1) * scale
+    x32[:, :h] = x
+    if first is not None:
+        first[:, :h] = x
+    xa[:, :h] = _norm(x, norm, eps)
+
+
+def sandwich_step(y, x32, post, nxt, eps: float, xa, coef, results, last: bool) -> None:
+    h = post[0].numel()
+    x = x32[:, :h] + _norm(y[:, :h].float(), post, eps)
+    if coef is not None:
+        n = coef.numel() - 1
+        if not last:
+            results[n, :, :h] = x
+        x = coef[n] * x
+        for j in range(n):
+            x = x + coef[j] * results[j, :, :h]
+    x32[:, :h] = x
+    xa[:, :h] = _norm(x, nxt, eps)
+
+
+def min_gru(p, bz, bx, state, out, seqs, cu_q, kv_lens, slots) -> None:
+    n, r = state.shape[1], p.float()
+    z, u, g = torch.sigmoid(r[:, :n] + bz), r[:, n:2 * n] + bx, F.silu(r[:, 2 * n:3 * n])
+    add = z * torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+    cu, kv, sl = cu_q.tolist(), kv_lens.tolist(), slots.tolist()
+    for b in seqs.tolist():
+        s = state[sl[b]].clone() if kv[b] > cu[b + 1] - cu[b] else torch.zeros(n)
+        for t in range(cu[b], cu[b + 1]):
+            s = (1 - z[t]) * s + add[t]
+            out[t, :n] = (s * g[t]).to(out.dtype)
+        state[sl[b]] = s
+
+
 # ---- hyper-connections -------------------------------------------------------------------------------------------
 def embed_streams(ids, table, x, hc_in, weight, offset: float, eps: float, xa) -> None:
     h = weight.numel()
@@ -236,7 +281,7 @@ def norm_gate(y, gate, weight, count: int, eps: float, scale: float, out) -> Non
 
 def qkv_prep(p, heads: int, kv_heads: int, dim: int, vdim: int, q, k_cache, v_cache, meta, conv_w, conv_state, qk_norm,
              wq, wk, eps: float, temp_coef: float, temp_every: int, cos_sin=None) -> None:
-    dp, vp, T = k_cache.shape[-1], v_cache.shape[-1], p.shape[0]
+    dp, T = q.shape[1] // heads, p.shape[0]
     x = p.float()
     if conv_w is not None:
         taps, w = conv_w.shape[0], conv_w.float()
@@ -250,23 +295,26 @@ def qkv_prep(p, heads: int, kv_heads: int, dim: int, vdim: int, q, k_cache, v_ca
                 conv_state[sl[b]] = keep.to(conv_state.dtype)
         x = mixed
     nq, nk = heads * dp, kv_heads * dp
-    qs, ks, vs = x[:, :nq], x[:, nq:nq + nk], x[:, nq + nk:]
+    vp = v_cache.shape[-1] if kv_heads else 0
+    qs, ks, vs = x[:, :nq], x[:, nq:nq + nk], x[:, nq + nk:nq + nk + kv_heads * vp]
 
     def normed(t, weight, n):
-        parts = n if qk_norm == "head" else 1
+        parts = 1 if qk_norm == "whole" else n
         t = t.reshape(T, parts, -1)
         count = dim * n // parts
-        t = t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / count + eps) * weight.float()
-        return t.reshape(T, -1)
+        t = t * torch.rsqrt(t.pow(2).sum(-1, keepdim=True) / count + eps)
+        return (t * weight.float() if weight is not None else t).reshape(T, -1)
     if qk_norm:
-        qs, ks = normed(qs, wq, heads), normed(ks, wk, kv_heads)
+        qs, ks = normed(qs, wq, heads), normed(ks, wk, kv_heads) if kv_heads else ks
     if cos_sin is not None:
-        qs, ks = (_rotate_pairs(t.reshape(T, n, dp), cos_sin, meta.positions).reshape(T, -1)
+        qs, ks = (_rotate_pairs(t.reshape(T, n, dp), cos_sin, meta.positions).reshape(T, n * dp)
                   for t, n in ((qs, heads), (ks, kv_heads)))
     if temp_coef:
         turn = torch.div(meta.positions.long() + 1, temp_every, rounding_mode="floor")
         qs = qs * (1 + temp_coef * torch.log(turn.float() + 1)).unsqueeze(-1)
     q.copy_(qs)
+    if not kv_heads:
+        return
     slots = meta.slot_mapping.long()
     ok = slots >= 0
     k_cache.view(-1, nk)[slots[ok]] = ks[ok].to(k_cache.dtype)
@@ -274,7 +322,7 @@ def qkv_prep(p, heads: int, kv_heads: int, dim: int, vdim: int, q, k_cache, v_ca
 
 
 def grouped_attention(q, k_cache, v_cache, out, meta, heads: int, kv_heads: int, scale: float, slopes, sink: bool,
-                      out_scale: float, window: int = 0, keep: int = 0) -> None:
+                      out_scale: float, window: int = 0, keep: int = 0, key_bias=None, chunk: int = 0, gate=None) -> None:
     page, dp, vp, rep = k_cache.shape[1], k_cache.shape[-1], v_cache.shape[-1], heads // kv_heads
     for b, kv_len in enumerate(meta.kv_lens_cpu):
         t0, t1 = meta.cu_q_cpu[b], meta.cu_q_cpu[b + 1]
@@ -288,8 +336,16 @@ def grouped_attention(q, k_cache, v_cache, out, meta, heads: int, kv_heads: int,
         hidden = dist < 0
         if window:
             hidden = hidden | ((dist >= window) & (torch.arange(kv_len) >= keep))
-        s = s.masked_fill(hidden, float("-inf"))
-        if sink:
-            s = torch.cat([s, torch.zeros(heads, t1 - t0, 1)], -1)
-        w = torch.softmax(s, -1)[..., :kv_len]
-        out[t0:t1] = (torch.einsum("hqk,khd->qhd", w, v) * out_scale).reshape(t1 - t0, -1).to(out.dtype)
+        if chunk:
+            hidden = hidden | (torch.arange(kv_len - (t1 - t0), kv_len).unsqueeze(-1) // chunk != torch.arange(kv_len) // chunk)
+        if key_bias is not None:
+            w = torch.sigmoid(s + key_bias[:, None, None]).masked_fill(hidden, 0.0)
+        else:
+            s = s.masked_fill(hidden, float("-inf"))
+            if sink:
+                s = torch.cat([s, torch.zeros(heads, t1 - t0, 1)], -1)
+            w = torch.softmax(s, -1)[..., :kv_len]
+        o = torch.einsum("hqk,khd->qhd", w, v) * out_scale
+        if gate is not None:
+            o = o * torch.sigmoid(gate[t0:t1, :heads].float()).unsqueeze(-1)
+        out[t0:t1] = o.reshape(t1 - t0, -1).to(out.dtype)
