@@ -219,8 +219,8 @@ def tensor_shapes(cfg):
 def random_weights(cfg, seed=0, decided=False):
     """bf16 weights under which faults show: a key bias that makes most weights small, so that single keys stand out, update
     gates between short and long memories, depth averages in which every layer's result counts, no unit or zero constant.
-    ``decided``: the constant part of a router's input ranks the experts, what depends on the token moves neighbours past one
-    another, so that hardly a choice hangs on the rounding of that input (which may be bf16)."""
+    ``decided``: the constant part of a router's input ranks the experts, what depends on the token changes the weights and
+    hardly the ranks: no choice hangs on the rounding of that input (which may be bf16)."""
     g = torch.Generator().manual_seed(seed)
     out = {}
     for name, shape in tensor_shapes(cfg).items():
@@ -249,9 +249,11 @@ def random_weights(cfg, seed=0, decided=False):
         out[name] = t.to(torch.bfloat16)
     for i, layer in enumerate(cfg["layers"] if decided else ()):
         if layer["mlp"] is not None:
+            out[f"l{i}.norm2.b"] *= 5
             r, b = (out[f"l{i}.{k}"].float() for k in ("mlp.router", "norm2.b"))
-            rank = torch.randperm(r.shape[0], generator=g).float()
-            out[f"l{i}.mlp.router"] = (0.15 * r + torch.outer(0.8 - 0.6 * rank, b / (b @ b))).to(torch.bfloat16)
+            rank, along = torch.randperm(r.shape[0], generator=g).float(), b / (b @ b)
+            r = 0.02 * (r - torch.outer(r @ b, along)) + torch.outer(0.8 - 0.6 * rank, along)
+            out[f"l{i}.mlp.router"] = r.to(torch.bfloat16)
     return out
 
 
