@@ -51,10 +51,10 @@ def parse_args():
                     choices=["overlap", "fuse_only", "fused_gemm", "baseline_nccl", "baseline_custom_ar", "baseline_multimem",
                              "no_ar"])
     ap.add_argument("--layers", type=int, default=None, help="debug only: fewer layers (marks the result invalid)")
-    ap.add_argument("--workload", default="prefill", choices=["prefill", "hybrid", "kebopel", "netezen"],
+    ap.add_argument("--workload", default="prefill", choices=["prefill", "hybrid", "kebopel", "netezen", "giforax"],
                     help="hybrid: the hybrid decoder (latent attention + Mamba-2) beside the Llama layout at equal size, "
                          "prefill, decode and every kernel (artifact/hybrid_bench.py); kebopel: the same for Kebopel "
-                         "(artifact/kebopel_bench.py); netezen: Netezen beside the Mixtral layout (artifact/netezen_bench.py); "
+                         "(artifact/kebopel_bench.py); netezen, giforax: these beside the Mixtral layout (artifact/netezen_bench.py, giforax_bench.py); "
                          "one GPU")
     ap.add_argument("--cuda-graphs", dest="cuda_graphs", action="store_true", default=None,
                     help="replay the step from a CUDA graph (captured during warm-up; the default when --warmup >= 3)")

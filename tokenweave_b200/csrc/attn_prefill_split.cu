@@ -31,7 +31,9 @@
 // Sigmoid form (MODE 5): grouped, a key's weight is the sigmoid of its biased score - no maximum, no sum, nothing to scale
 // later, the two halves of the key range add up -, chunks instead of a window, and a gate per head on the result. Two weights
 // share one reciprocal: 1 / a and 1 / b are b r and a r with r = 1 / (a b), which takes the special-function unit three times
-// for two weights instead of four (it bounds this form).
+// for two weights instead of four. Without a maximum over the row there is no need to hold all of it: scores are read 32 at a
+// time, and the two terms of their weights take the place of these scores (all 128 in registers, as above: 1.29 ms for 8192
+// tokens of 32 heads).
 // Replaces the FlashAttention-2 varlen call the reference makes on Blackwell
 // (vllm/v1/attention/backends/flash_attn.py:713-733, vllm/attention/utils/fa_utils.py:29-34).
 //
@@ -49,7 +51,7 @@ namespace tw {
 // K/V tile slots per softmax group. The grouped forms spill registers in the softmax, and beside three slots per group there
 // is hardly an L1 cache left for them (head size 128: 776 us with two slots, 808 with three; with bias 928 and 1143).
 template <int MODE>
-constexpr int split_ring() { return MODE >= 2 ? 2 : 3; }
+constexpr int split_ring() { return MODE >= 2 && MODE < 5 ? 2 : 3; }
 
 template <int D, int DV, int RING>
 struct SplitSmem {
@@ -269,8 +271,9 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
               if (!mbar_wait(&p_ready[g], cnt[g] & 1)) return false;
               tc_fence_after_sync();
             }
-            pv(k, COL_P, first && k == 0);
-            if (GROUPED) pv(k, 0, false);
+            // (sigmoid form: both terms of 32 keys where their scores were)
+            pv(k, SIGMOID ? (k >> 1) * 16 : COL_P, first && k == 0);
+            if (GROUPED) pv(k, SIGMOID ? (k >> 1) * 16 + 16 : 0, false);
           }
           umma_commit(&ring_empty[g * R + slot]);
           umma_commit(&o_done[g]);
@@ -330,22 +333,14 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         // warp-uniform: lane 0 holds the warp's smallest position, lane 31 its largest
         bool need_mask = (k_base + ATT_BN - 1) > __shfl_sync(0xffffffffu, pos, 0);
         if (WINDOW) need_mask = need_mask || k_base < __shfl_sync(0xffffffffu, pos_w, 31);
-        // The row's 128 scores come to registers in one go (four loads in flight, one wait): the latency of
-        // tensor-memory loads is paid once per tile, and everything below runs from registers.
-        uint32_t s0[32], s1[32], s2[32], s3[32];
-        tmem_ld_32x32(t_s, s0);
-        tmem_ld_32x32(t_s + 32, s1);
-        tmem_ld_32x32(t_s + 64, s2);
-        tmem_ld_32x32(t_s + 96, s3);
-        tmem_wait_ld();
         if constexpr (SIGMOID) {
           // 2^x = exp(-(score + bias)), bounded so that the product of two denominators stays finite (a weight of 2^-62 is
           // nothing beside any other; hidden keys get it, too)
           constexpr float HIDDEN = 62.f;
           const float2 sc = make_float2(-p.scale_log2, -p.scale_log2), kb = make_float2(key_bias, key_bias);
           const float2 one = make_float2(1.f, 1.f);
-          uint32_t pk[16], lo[16];
-          auto weigh = [&](uint32_t (&buf)[32], int chunk) {
+          auto weigh = [&](const uint32_t (&buf)[32], int chunk) {
+            uint32_t pk[16], lo[16];
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
               float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc, kb);
@@ -358,22 +353,40 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
               const float r = fast_rcp(d.x * d.y);
               split_weights(mul2(make_float2(d.y, d.x), make_float2(r, r)), pk[i], lo[i]);
             }
-            tmem_st_32x16(t_p + chunk * 16, pk);
-            tmem_st_32x16(t_s + chunk * 16, lo);
+            tmem_st_32x16(t_s + chunk * 32, pk);
+            tmem_st_32x16(t_s + chunk * 32 + 16, lo);
           };
+          // 32 keys at a time, the next ones on their way; their weights take their scores' place
+          uint32_t s0[32], s1[32];
+          tmem_ld_32x32(t_s, s0);
+          tmem_wait_ld_of(s0);
+          tmem_ld_32x32(t_s + 32, s1);
           weigh(s0, 0);
+          tmem_wait_ld_of(s1);
+          tmem_ld_32x32(t_s + 64, s0);
           weigh(s1, 1);
           tmem_wait_st();
           tc_fence_before_sync();
           mbar_arrive(&p_half[g]);
-          weigh(s2, 2);
-          weigh(s3, 3);
+          tmem_wait_ld_of(s0);
+          tmem_ld_32x32(t_s + 96, s1);
+          weigh(s0, 2);
+          tmem_wait_ld_of(s1);
+          weigh(s1, 3);
           tmem_wait_st();
           tc_fence_before_sync();
           mbar_arrive(&p_ready[g]);   // arrive even after a failed wait so the issuer is not left waiting
           ++cnt;
           continue;
         }
+        // The row's 128 scores come to registers in one go (four loads in flight, one wait): the latency of
+        // tensor-memory loads is paid once per tile, and everything below runs from registers.
+        uint32_t s0[32], s1[32], s2[32], s3[32];
+        tmem_ld_32x32(t_s, s0);
+        tmem_ld_32x32(t_s + 32, s1);
+        tmem_ld_32x32(t_s + 64, s2);
+        tmem_ld_32x32(t_s + 96, s3);
+        tmem_wait_ld();
         if (OPTS && p.softcap > 0.f) {
           // s -> cap * tanh(s * scale / cap), kept in units of the raw scores (the scale is applied below)
 #pragma unroll

@@ -32,32 +32,64 @@ struct SandwichArgs {
   const int* ids; const void* table; long long ldt; int vocab; float scale;        // embedding
 };
 
-// Replaces a row by its norm. Elements outside the row are zeros.
-template <typename T, int VPT>
-__device__ __forceinline__ void norm_row(const SandwichArgs& a, float (&v)[VPT][8], const void* w, const void* b,
-                                         float* scratch) {
-  float s[1], mean = 0.f;
+// Block-wide mean and sum of squared deviations of a row in one exchange: every warp takes the deviations from its own mean, and
+// the warps' results are put together with the distances between their means. Without `center` the mean is zero.
+template <int VPT>
+__device__ __forceinline__ void row_moments(const SandwichArgs& a, const float (&v)[VPT][8], float* scratch, float& mean,
+                                            float& dev) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  // elements of the row that a warp holds
+  auto held = [&](int w) {
+    int n = 0;
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) n += max(0, min(256, a.H - (w * 32 + k * static_cast<int>(blockDim.x)) * 8));
+    return static_cast<float>(n);
+  };
+  float s = 0.f, m = 0.f;
   if (a.center) {
-    s[0] = 0.f;
 #pragma unroll
     for (int k = 0; k < VPT; ++k)
 #pragma unroll
-      for (int j = 0; j < 8; ++j) s[0] += v[k][j];
-    block_sum<1>(s, scratch);
-    mean = s[0] / static_cast<float>(a.H);
+      for (int j = 0; j < 8; ++j) s += v[k][j];
+    s = warp_sum(s);
+    const float n = held(warp);
+    m = n > 0.f ? s / n : 0.f;
   }
-  s[0] = 0.f;
+  float d = 0.f;
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
     const int n = a.H - (threadIdx.x + k * blockDim.x) * 8;
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      v[k][j] = j < n ? v[k][j] - mean : 0.f;
-      s[0] += v[k][j] * v[k][j];
+      const float e = j < n ? v[k][j] - m : 0.f;
+      d = fmaf(e, e, d);
     }
   }
-  block_sum<1>(s, scratch);
-  const float r = 1.f / sqrtf(s[0] / static_cast<float>(a.H) + a.eps);
+  d = warp_sum(d);
+  if (lane == 0) {
+    scratch[warp] = s;
+    scratch[32 + warp] = d;
+  }
+  __syncthreads();
+  s = lane < warps ? scratch[lane] : 0.f;
+  d = lane < warps ? scratch[32 + lane] : 0.f;
+  mean = 0.f;
+  if (a.center) {
+    const float n = lane < warps ? held(lane) : 0.f;
+    mean = warp_sum(s) / static_cast<float>(a.H);
+    const float e = n > 0.f ? s / n - mean : 0.f;
+    d = fmaf(n * e, e, d);
+  }
+  dev = warp_sum(d);
+}
+
+// Replaces a row by its norm. Elements outside the row are zeros. (Consecutive calls take different scratch.)
+template <typename T, int VPT>
+__device__ __forceinline__ void norm_row(const SandwichArgs& a, float (&v)[VPT][8], const void* w, const void* b,
+                                         float* scratch) {
+  float mean, dev;
+  row_moments<VPT>(a, v, scratch, mean, dev);
+  const float r = 1.f / sqrtf(dev / static_cast<float>(a.H) + a.eps);
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
     const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
@@ -71,7 +103,7 @@ __device__ __forceinline__ void norm_row(const SandwichArgs& a, float (&v)[VPT][
       for (int j = 0; j < 8; ++j) c[j] = 0.f;
     }
 #pragma unroll
-    for (int j = 0; j < 8; ++j) v[k][j] = fmaf(v[k][j] * r, g[j], c[j]);
+    for (int j = 0; j < 8; ++j) v[k][j] = fmaf((v[k][j] - mean) * r, g[j], c[j]);
   }
 }
 
@@ -85,22 +117,45 @@ __device__ __forceinline__ void next_input(const SandwichArgs& a, int t, float (
   }
 }
 
-template <typename T, int VPT>
+template <typename T, int VPT, bool AVERAGE>
 __global__ void __launch_bounds__(512)
 sandwich_step_kernel(const SandwichArgs a) {
-  __shared__ float scratch[32];
-  for (int t = blockIdx.x; t < a.rows; t += gridDim.x) {
-    float v[VPT][8], x[VPT][8];
+  __shared__ float scratch[2][64];
+  const float own = AVERAGE ? a.coef[a.n_past] : 1.f;
+  Raw8<T> y[VPT];
+  float x[VPT][8];
+  auto request = [&](int t) {
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
       const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
-#pragma unroll
-      for (int j = 0; j < 8; ++j) v[k][j] = x[k][j] = 0.f;
-      if (n <= 0) continue;
-      ld8n<true>(reinterpret_cast<const T*>(a.y) + t * a.ldy + i, n, v[k]);
-      ld8n<true>(a.x + t * a.ldx + i, n, x[k]);
+      y[k] = ld8raw<true>(reinterpret_cast<const T*>(a.y) + t * a.ldy + (n > 0 ? i : 0), n);
+      if (n > 0) ld8n<true>(a.x + t * a.ldx + i, n, x[k]);
     }
-    norm_row<T, VPT>(a, v, a.w_post, a.b_post, scratch);
+  };
+  if (static_cast<int>(blockIdx.x) < a.rows) request(blockIdx.x);
+  for (int t = blockIdx.x; t < a.rows; t += gridDim.x) {
+    float v[VPT][8], sum[VPT][8];
+#pragma unroll
+    for (int k = 0; k < VPT; ++k) {
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        v[k][j] = ld1(&y[k].v[j]);
+        sum[k][j] = 0.f;
+      }
+      if (!AVERAGE) continue;
+      const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
+      if (n <= 0) continue;
+      const float* p = a.past + t * a.ldp + i;
+#pragma unroll 4
+      for (int q = 0; q < a.n_past; ++q) {
+        const float c = a.coef[q];
+        float u[8];
+        ld8n<true>(p + q * a.lds, n, u);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) sum[k][j] = fmaf(c, u[j], sum[k][j]);
+      }
+    }
+    norm_row<T, VPT>(a, v, a.w_post, a.b_post, scratch[0]);
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
       const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
@@ -111,32 +166,24 @@ sandwich_step_kernel(const SandwichArgs a) {
       }
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[k][j] += x[k][j];
-      if (a.coef != nullptr) {
+      if (AVERAGE) {
         if (a.result != nullptr) st8n<true>(a.result + t * a.ldp + i, n, v[k]);
-        const float mine = a.coef[a.n_past];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) v[k][j] *= mine;
-        const float* p = a.past + t * a.ldp + i;
-#pragma unroll 4
-        for (int q = 0; q < a.n_past; ++q) {
-          const float c = a.coef[q];
-          float u[8];
-          ld8n<true>(p + q * a.lds, n, u);
-#pragma unroll
-          for (int j = 0; j < 8; ++j) v[k][j] = fmaf(c, u[j], v[k][j]);
-        }
+        for (int j = 0; j < 8; ++j) v[k][j] = fmaf(own, v[k][j], sum[k][j]);
       }
       if (a.store) st8n<true>(a.x + t * a.ldx + i, n, v[k]);
     }
-    next_input<T, VPT>(a, t, v, scratch);
+    // the next row is on its way while this one's second norm is formed
+    if (t + static_cast<int>(gridDim.x) < a.rows) request(t + gridDim.x);
+    next_input<T, VPT>(a, t, v, scratch[1]);
   }
 }
 
 template <typename T, int VPT>
 __global__ void __launch_bounds__(512)
 embed_sandwich_kernel(const SandwichArgs a) {
-  __shared__ float scratch[32];
-  for (int t = blockIdx.x; t < a.rows; t += gridDim.x) {
+  __shared__ float scratch[2][64];
+  for (int t = blockIdx.x, turn = 0; t < a.rows; t += gridDim.x, turn ^= 1) {
     const int id = a.ids[t];
     const bool ok = id >= 0 && id < a.vocab;
     const T* src = reinterpret_cast<const T*>(a.table) + (ok ? id : 0) * a.ldt;
@@ -153,7 +200,7 @@ embed_sandwich_kernel(const SandwichArgs a) {
       st8n<true>(a.x + t * a.ldx + i, n, v[k]);
       if (a.result != nullptr) st8n<true>(a.result + t * a.ldp + i, n, v[k]);
     }
-    next_input<T, VPT>(a, t, v, scratch);
+    next_input<T, VPT>(a, t, v, scratch[turn]);
   }
 }
 
@@ -162,7 +209,8 @@ static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 
 template <typename T, int VPT>
 static void launch_sandwich(const SandwichArgs& a, int grid, int threads, cudaStream_t stream) {
   if (a.ids != nullptr) embed_sandwich_kernel<T, VPT><<<grid, threads, 0, stream>>>(a);
-  else sandwich_step_kernel<T, VPT><<<grid, threads, 0, stream>>>(a);
+  else if (a.coef != nullptr) sandwich_step_kernel<T, VPT, true><<<grid, threads, 0, stream>>>(a);
+  else sandwich_step_kernel<T, VPT, false><<<grid, threads, 0, stream>>>(a);
 }
 
 static int run_sandwich(const SandwichArgs& a, int dtype, const char* what, cudaStream_t stream) {
