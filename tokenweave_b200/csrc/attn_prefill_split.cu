@@ -337,18 +337,20 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
           // 2^x = exp(-(score + bias)), bounded so that the product of two denominators stays finite (a weight of 2^-62 is
           // nothing beside any other; hidden keys get it, too)
           constexpr float HIDDEN = 62.f;
+          const uint32_t hide = p.scale_log2 > 0.f ? 0xff800000u : 0x7f800000u;      // x infinite (or nothing: the bound)
           const float2 sc = make_float2(-p.scale_log2, -p.scale_log2), kb = make_float2(key_bias, key_bias);
           const float2 one = make_float2(1.f, 1.f);
-          auto weigh = [&](const uint32_t (&buf)[32], int chunk) {
+          auto weigh = [&](uint32_t (&buf)[32], int chunk) {
+            if (need_mask) {
+              const int from = pos_w - k_base - chunk * 32, to = pos - k_base - chunk * 32;
+#pragma unroll
+              for (int i = 0; i < 32; ++i)
+                if (i > to || i < from) buf[i] = hide;
+            }
             uint32_t pk[16], lo[16];
 #pragma unroll
             for (int i = 0; i < 16; ++i) {
-              float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc, kb);
-              if (need_mask) {
-                const int k = k_base + chunk * 32 + 2 * i;
-                if (k > pos || k < pos_w) x.x = HIDDEN;
-                if (k + 1 > pos || k + 1 < pos_w) x.y = HIDDEN;
-              }
+              const float2 x = fma2(make_float2(__uint_as_float(buf[2 * i]), __uint_as_float(buf[2 * i + 1])), sc, kb);
               const float2 d = fadd2(make_float2(fast_exp2(fminf(x.x, HIDDEN)), fast_exp2(fminf(x.y, HIDDEN))), one);
               const float r = fast_rcp(d.x * d.y);
               split_weights(mul2(make_float2(d.y, d.x), make_float2(r, r)), pk[i], lo[i]);
@@ -356,26 +358,22 @@ attn_prefill_split_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
             tmem_st_32x16(t_s + chunk * 32, pk);
             tmem_st_32x16(t_s + chunk * 32 + 16, lo);
           };
-          // 32 keys at a time, the next ones on their way; their weights take their scores' place
+          // 32 keys at a time, the next ones on their way; their weights take their scores' place. (A loop: four copies of
+          // it wait for instructions.)
           uint32_t s0[32], s1[32];
           tmem_ld_32x32(t_s, s0);
-          tmem_wait_ld_of(s0);
-          tmem_ld_32x32(t_s + 32, s1);
-          weigh(s0, 0);
-          tmem_wait_ld_of(s1);
-          tmem_ld_32x32(t_s + 64, s0);
-          weigh(s1, 1);
-          tmem_wait_st();
-          tc_fence_before_sync();
-          mbar_arrive(&p_half[g]);
-          tmem_wait_ld_of(s0);
-          tmem_ld_32x32(t_s + 96, s1);
-          weigh(s0, 2);
-          tmem_wait_ld_of(s1);
-          weigh(s1, 3);
-          tmem_wait_st();
-          tc_fence_before_sync();
-          mbar_arrive(&p_ready[g]);   // arrive even after a failed wait so the issuer is not left waiting
+#pragma unroll 1
+          for (int half = 0; half < 2; ++half) {
+            tmem_wait_ld_of(s0);
+            tmem_ld_32x32(t_s + half * 64 + 32, s1);
+            weigh(s0, 2 * half);
+            tmem_wait_ld_of(s1);
+            if (half == 0) tmem_ld_32x32(t_s + 64, s0);
+            weigh(s1, 2 * half + 1);
+            tmem_wait_st();
+            tc_fence_before_sync();
+            mbar_arrive(half == 0 ? &p_half[g] : &p_ready[g]);   // also after a failed wait: the issuer is not left waiting
+          }
           ++cnt;
           continue;
         }

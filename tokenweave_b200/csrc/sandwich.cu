@@ -32,14 +32,27 @@ struct SandwichArgs {
   const int* ids; const void* table; long long ldt; int vocab; float scale;        // embedding
 };
 
+// Eight elements of a row from i on of which n are inside it. FULL: every thread's groups are (the row is as long as the CTA).
+template <bool FULL, typename T>
+__device__ __forceinline__ void ldg8(const T* p, int n, float (&v)[8]) {
+  if (FULL) ld8(p, v);
+  else ld8n<true>(p, n, v);
+}
+template <bool FULL, typename T>
+__device__ __forceinline__ void stg8(T* p, int n, const float (&v)[8]) {
+  if (FULL) st8(p, v);
+  else st8n<true>(p, n, v);
+}
+
 // Block-wide mean and sum of squared deviations of a row in one exchange: every warp takes the deviations from its own mean, and
 // the warps' results are put together with the distances between their means. Without `center` the mean is zero.
-template <int VPT>
+template <int VPT, bool FULL>
 __device__ __forceinline__ void row_moments(const SandwichArgs& a, const float (&v)[VPT][8], float* scratch, float& mean,
                                             float& dev) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   // elements of the row that a warp holds
   auto held = [&](int w) {
+    if (FULL) return 256.f * VPT;
     int n = 0;
 #pragma unroll
     for (int k = 0; k < VPT; ++k) n += max(0, min(256, a.H - (w * 32 + k * static_cast<int>(blockDim.x)) * 8));
@@ -61,7 +74,7 @@ __device__ __forceinline__ void row_moments(const SandwichArgs& a, const float (
     const int n = a.H - (threadIdx.x + k * blockDim.x) * 8;
 #pragma unroll
     for (int j = 0; j < 8; ++j) {
-      const float e = j < n ? v[k][j] - m : 0.f;
+      const float e = FULL || j < n ? v[k][j] - m : 0.f;
       d = fmaf(e, e, d);
     }
   }
@@ -84,20 +97,20 @@ __device__ __forceinline__ void row_moments(const SandwichArgs& a, const float (
 }
 
 // Replaces a row by its norm. Elements outside the row are zeros. (Consecutive calls take different scratch.)
-template <typename T, int VPT>
+template <typename T, int VPT, bool FULL>
 __device__ __forceinline__ void norm_row(const SandwichArgs& a, float (&v)[VPT][8], const void* w, const void* b,
                                          float* scratch) {
   float mean, dev;
-  row_moments<VPT>(a, v, scratch, mean, dev);
+  row_moments<VPT, FULL>(a, v, scratch, mean, dev);
   const float r = 1.f / sqrtf(dev / static_cast<float>(a.H) + a.eps);
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
     const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
-    if (n <= 0) continue;
+    if (!FULL && n <= 0) continue;
     float g[8], c[8];
-    ld8n<true>(reinterpret_cast<const T*>(w) + i, n, g);
+    ldg8<FULL>(reinterpret_cast<const T*>(w) + i, n, g);
     if (b != nullptr) {
-      ld8n<true>(reinterpret_cast<const T*>(b) + i, n, c);
+      ldg8<FULL>(reinterpret_cast<const T*>(b) + i, n, c);
     } else {
 #pragma unroll
       for (int j = 0; j < 8; ++j) c[j] = 0.f;
@@ -107,17 +120,17 @@ __device__ __forceinline__ void norm_row(const SandwichArgs& a, float (&v)[VPT][
   }
 }
 
-template <typename T, int VPT>
+template <typename T, int VPT, bool FULL>
 __device__ __forceinline__ void next_input(const SandwichArgs& a, int t, float (&v)[VPT][8], float* scratch) {
-  norm_row<T, VPT>(a, v, a.w_next, a.b_next, scratch);
+  norm_row<T, VPT, FULL>(a, v, a.w_next, a.b_next, scratch);
 #pragma unroll
   for (int k = 0; k < VPT; ++k) {
     const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
-    if (n > 0) st8n<true>(reinterpret_cast<T*>(a.xa) + t * a.lda + i, n, v[k]);
+    if (FULL || n > 0) stg8<FULL>(reinterpret_cast<T*>(a.xa) + t * a.lda + i, n, v[k]);
   }
 }
 
-template <typename T, int VPT, bool AVERAGE>
+template <typename T, int VPT, bool FULL, bool AVERAGE>
 __global__ void __launch_bounds__(512)
 sandwich_step_kernel(const SandwichArgs a) {
   __shared__ float scratch[2][64];
@@ -128,8 +141,8 @@ sandwich_step_kernel(const SandwichArgs a) {
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
       const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
-      y[k] = ld8raw<true>(reinterpret_cast<const T*>(a.y) + t * a.ldy + (n > 0 ? i : 0), n);
-      if (n > 0) ld8n<true>(a.x + t * a.ldx + i, n, x[k]);
+      y[k] = ld8raw<true>(reinterpret_cast<const T*>(a.y) + t * a.ldy + (FULL || n > 0 ? i : 0), FULL ? 8 : n);
+      if (FULL || n > 0) ldg8<FULL>(a.x + t * a.ldx + i, n, x[k]);
     }
   };
   if (static_cast<int>(blockIdx.x) < a.rows) request(blockIdx.x);
@@ -144,22 +157,22 @@ sandwich_step_kernel(const SandwichArgs a) {
       }
       if (!AVERAGE) continue;
       const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
-      if (n <= 0) continue;
+      if (!FULL && n <= 0) continue;
       const float* p = a.past + t * a.ldp + i;
 #pragma unroll 4
       for (int q = 0; q < a.n_past; ++q) {
         const float c = a.coef[q];
         float u[8];
-        ld8n<true>(p + q * a.lds, n, u);
+        ldg8<FULL>(p + q * a.lds, n, u);
 #pragma unroll
         for (int j = 0; j < 8; ++j) sum[k][j] = fmaf(c, u[j], sum[k][j]);
       }
     }
-    norm_row<T, VPT>(a, v, a.w_post, a.b_post, scratch[0]);
+    norm_row<T, VPT, FULL>(a, v, a.w_post, a.b_post, scratch[0]);
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
       const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
-      if (n <= 0) {
+      if (!FULL && n <= 0) {
 #pragma unroll
         for (int j = 0; j < 8; ++j) v[k][j] = 0.f;
         continue;
@@ -167,19 +180,19 @@ sandwich_step_kernel(const SandwichArgs a) {
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[k][j] += x[k][j];
       if (AVERAGE) {
-        if (a.result != nullptr) st8n<true>(a.result + t * a.ldp + i, n, v[k]);
+        if (a.result != nullptr) stg8<FULL>(a.result + t * a.ldp + i, n, v[k]);
 #pragma unroll
         for (int j = 0; j < 8; ++j) v[k][j] = fmaf(own, v[k][j], sum[k][j]);
       }
-      if (a.store) st8n<true>(a.x + t * a.ldx + i, n, v[k]);
+      if (a.store) stg8<FULL>(a.x + t * a.ldx + i, n, v[k]);
     }
     // the next row is on its way while this one's second norm is formed
     if (t + static_cast<int>(gridDim.x) < a.rows) request(t + gridDim.x);
-    next_input<T, VPT>(a, t, v, scratch[1]);
+    next_input<T, VPT, FULL>(a, t, v, scratch[1]);
   }
 }
 
-template <typename T, int VPT>
+template <typename T, int VPT, bool FULL>
 __global__ void __launch_bounds__(512)
 embed_sandwich_kernel(const SandwichArgs a) {
   __shared__ float scratch[2][64];
@@ -193,24 +206,24 @@ embed_sandwich_kernel(const SandwichArgs a) {
       const int i = (threadIdx.x + k * blockDim.x) * 8, n = a.H - i;
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[k][j] = 0.f;
-      if (n <= 0) continue;
-      if (ok) ld8n<true>(src + i, n, v[k]);
+      if (!FULL && n <= 0) continue;
+      if (ok) ldg8<FULL>(src + i, n, v[k]);
 #pragma unroll
       for (int j = 0; j < 8; ++j) v[k][j] *= a.scale;
-      st8n<true>(a.x + t * a.ldx + i, n, v[k]);
-      if (a.result != nullptr) st8n<true>(a.result + t * a.ldp + i, n, v[k]);
+      stg8<FULL>(a.x + t * a.ldx + i, n, v[k]);
+      if (a.result != nullptr) stg8<FULL>(a.result + t * a.ldp + i, n, v[k]);
     }
-    next_input<T, VPT>(a, t, v, scratch[turn]);
+    next_input<T, VPT, FULL>(a, t, v, scratch[turn]);
   }
 }
 
 static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
-template <typename T, int VPT>
+template <typename T, int VPT, bool FULL>
 static void launch_sandwich(const SandwichArgs& a, int grid, int threads, cudaStream_t stream) {
-  if (a.ids != nullptr) embed_sandwich_kernel<T, VPT><<<grid, threads, 0, stream>>>(a);
-  else if (a.coef != nullptr) sandwich_step_kernel<T, VPT, true><<<grid, threads, 0, stream>>>(a);
-  else sandwich_step_kernel<T, VPT, false><<<grid, threads, 0, stream>>>(a);
+  if (a.ids != nullptr) embed_sandwich_kernel<T, VPT, FULL><<<grid, threads, 0, stream>>>(a);
+  else if (a.coef != nullptr) sandwich_step_kernel<T, VPT, FULL, true><<<grid, threads, 0, stream>>>(a);
+  else sandwich_step_kernel<T, VPT, FULL, false><<<grid, threads, 0, stream>>>(a);
 }
 
 static int run_sandwich(const SandwichArgs& a, int dtype, const char* what, cudaStream_t stream) {
@@ -228,11 +241,14 @@ static int run_sandwich(const SandwichArgs& a, int dtype, const char* what, cuda
   }
   const int cap = device_sm_count() * (threads <= 128 ? 16 : threads <= 256 ? 8 : 4);
   const int grid = a.rows < cap ? a.rows : cap;
-#define TW_GO(TT)                                                       \
-  do {                                                                  \
-    if (vpt == 1) launch_sandwich<TT, 1>(a, grid, threads, stream);     \
-    else if (vpt == 2) launch_sandwich<TT, 2>(a, grid, threads, stream); \
-    else launch_sandwich<TT, 4>(a, grid, threads, stream);              \
+  const bool full = a.H == threads * vpt * 8;
+#define TW_GO(TT)                                                                              \
+  do {                                                                                         \
+    if (vpt == 1 && full) launch_sandwich<TT, 1, true>(a, grid, threads, stream);              \
+    else if (vpt == 1) launch_sandwich<TT, 1, false>(a, grid, threads, stream);                \
+    else if (vpt == 2 && full) launch_sandwich<TT, 2, true>(a, grid, threads, stream);         \
+    else if (vpt == 2) launch_sandwich<TT, 2, false>(a, grid, threads, stream);                \
+    else launch_sandwich<TT, 4, false>(a, grid, threads, stream);                              \
   } while (0)
   if (dtype == TW_BF16) TW_GO(__nv_bfloat16);
   else TW_GO(float);
