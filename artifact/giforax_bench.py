@@ -107,7 +107,7 @@ def kernels(width: int, T: int = 8192, batch: int = 128, context: int = 2048) ->
         if single:
             t("ssd_scan [decode]", "", lambda: hops.ssd_scan(xbc, dt, A, A, A, ss, ys, seqs, cu, kvl, seqs, 1),
               m * (chan + gru) * 2 + state)
-            t("min_gru [decode]", "ssd_scan [decode]", lambda: run(False), m * gru * 16)
+            t("min_gru [decode]", "add_rmsnorm [decode]", lambda: run(False), m * gru * 16)
         else:
             t("ssd_chunk [prefill]", "", lambda: hops.ssd_chunk(xbc, dt, A, A, A, ss, ys, seqs, cu, kvl, seqs, 1),
               m * (chan + gru) * 2 + state, 2.0 * m * (mh * 64 * 64 / 2 + 2 * mh * 128 * 64))

@@ -220,7 +220,10 @@ embed_sandwich_kernel(const SandwichArgs a) {
 static bool aligned16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
 
 template <typename T, int VPT, bool FULL>
-static void launch_sandwich(const SandwichArgs& a, int grid, int threads, cudaStream_t stream) {
+static void launch_sandwich(const SandwichArgs& a, int threads, cudaStream_t stream) {
+  // as many CTAs as fit at a time, so that each one's next row is on its way
+  const int cap = device_sm_count() * (a.ids != nullptr ? 3 : 2) * (threads <= 128 ? 4 : threads <= 256 ? 2 : 1);
+  const int grid = a.rows < cap ? a.rows : cap;
   if (a.ids != nullptr) embed_sandwich_kernel<T, VPT, FULL><<<grid, threads, 0, stream>>>(a);
   else if (a.coef != nullptr) sandwich_step_kernel<T, VPT, FULL, true><<<grid, threads, 0, stream>>>(a);
   else sandwich_step_kernel<T, VPT, FULL, false><<<grid, threads, 0, stream>>>(a);
@@ -239,16 +242,14 @@ static int run_sandwich(const SandwichArgs& a, int dtype, const char* what, cuda
     set_last_error("%s: rows on 16-byte boundaries are needed", what);
     return 1;
   }
-  const int cap = device_sm_count() * (threads <= 128 ? 16 : threads <= 256 ? 8 : 4);
-  const int grid = a.rows < cap ? a.rows : cap;
   const bool full = a.H == threads * vpt * 8;
 #define TW_GO(TT)                                                                              \
   do {                                                                                         \
-    if (vpt == 1 && full) launch_sandwich<TT, 1, true>(a, grid, threads, stream);              \
-    else if (vpt == 1) launch_sandwich<TT, 1, false>(a, grid, threads, stream);                \
-    else if (vpt == 2 && full) launch_sandwich<TT, 2, true>(a, grid, threads, stream);         \
-    else if (vpt == 2) launch_sandwich<TT, 2, false>(a, grid, threads, stream);                \
-    else launch_sandwich<TT, 4, false>(a, grid, threads, stream);                              \
+    if (vpt == 1 && full) launch_sandwich<TT, 1, true>(a, threads, stream);              \
+    else if (vpt == 1) launch_sandwich<TT, 1, false>(a, threads, stream);                \
+    else if (vpt == 2 && full) launch_sandwich<TT, 2, true>(a, threads, stream);         \
+    else if (vpt == 2) launch_sandwich<TT, 2, false>(a, threads, stream);                \
+    else launch_sandwich<TT, 4, false>(a, threads, stream);                              \
   } while (0)
   if (dtype == TW_BF16) TW_GO(__nv_bfloat16);
   else TW_GO(float);
