@@ -1,8 +1,8 @@
 """Giforax (``models/giforax.py``) beside the framework's closest models at equal size: throughput of prefill and decode,
 and every kernel against its roofline and beside the like kernel's distance.
 
-* ``throughput``: four layers (attention, attention on the first one's keys and values, minGRU, attention, each with a mixture
-  of experts) and a Mixtral layout of the same width, heads and parameters, random weights and token ids, as in
+* ``throughput``: four layers (minGRU, attention, attention on the keys and values of the one before it, minGRU, each with a
+  mixture of experts) and a Mixtral layout of the same width, heads and parameters, random weights and token ids, as in
   ``hybrid_bench.py``.
 * ``kernels``: as there; the like kernels are those of the Mixtral layout (attention, router, grouped products, norms), of
   Netezen's routed layer and of Sidisun's recurrence.

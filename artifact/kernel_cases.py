@@ -12,6 +12,7 @@ import argparse
 import math
 import os
 import sys
+from types import SimpleNamespace
 
 sys.path.insert(0, os.path.dirname(os.path.abspath(__file__)))
 from common import measured_peaks  # noqa: E402
@@ -23,7 +24,7 @@ def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("case", choices=["gemm", "gemm_swiglu", "gemm_fp8", "rmsnorm_quant_fp8", "attn_prefill", "attn_decode", "add_rmsnorm", "rope_kv",
                                      "moe_router", "moe_layer", "fused_local", "gemm_rs_norm_local", "ag_gemm_local",
-                                     "sample", "netezen"])
+                                     "sample", "netezen", "giforax"])
     ap.add_argument("--m", type=int, default=4096)
     ap.add_argument("--n", type=int, default=8192)
     ap.add_argument("--k", type=int, default=4096)
@@ -165,6 +166,25 @@ def main() -> None:
             ops.moe_route(xa, router, E, 4, corr, 1e-20)
             hops.latent_prefill(q, kv, lat, 512, T, begin, out, None, cu, kvl, ts, tq, len(tiles), heads, 128, 64, 128,
                                 192 ** -0.5, window, sink)
+    elif args.case == "giforax":
+        # the kernels that only Giforax has, one launch each per round: the step behind a layer (the average of five results
+        # of 4096), minGRU, attention with sigmoid weights
+        from tokenweave_b200.ops import hybrid as hops
+        T, H, heads, hkv, past, page = args.tokens, 4096, 32, 8, 4, 128
+        y, xa, w, b, p, out = (torch.randn(*s, device=dev).to(BF) for s in ((T, H), (T, H), (H,), (H,), (T, 3 * H), (T, H)))
+        x, results, coef = (torch.randn(*s, device=dev) for s in ((T, H), (past + 1, T, H), (past + 1,)))
+        bz, bx, state = torch.randn(H, device=dev) - 3, torch.randn(H, device=dev), torch.zeros(1, H, device=dev)
+        q, o, pg = (torch.randn(T, n, device=dev).to(BF) for n in (heads * 128, heads * 128, heads))
+        kc, vc = (torch.randn(T // page + 1, page, hkv, 128, device=dev).to(BF) for _ in range(2))
+        i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+        tiles, one, cu, kvl, bias = list(range(0, T, 128))[::-1], i32([0]), i32([0, T]), i32([T]), torch.full((heads,), -3.0, device=dev)
+        meta = SimpleNamespace(num_tiles=len(tiles), num_single=0, cu_q=cu, kv_lens=kvl, max_kv_len=T, tile_seq=i32([0] * len(tiles)),
+                               tile_q0=i32(tiles), block_table=i32(list(range(1, T // page + 1))).view(1, -1))
+
+        def fn():
+            hops.sandwich_step(y, x, (w, b), (w, b), 1e-5, xa, coef, results)
+            hops.min_gru(p, bz, bx, state, out, one, cu, kvl, one, True)
+            hops.grouped_attention(q, kc, vc, o, meta, heads, hkv, 128 ** -0.5, None, False, 1.0, key_bias=bias, gate=pg)
     elif args.case in ("gemm_rs_norm_local", "ag_gemm_local"):
         # the GEMM fused with its collective on one GPU acting as a world of one (peer transport): the GEMM CTAs
         # and the communication CTAs run as on several GPUs, the "peers" are this GPU's own buffer

@@ -249,14 +249,14 @@ def _netezen(vocab, width, layers, streams, attn, latent, dense, moe, shared, wi
 
 
 def _giforax(vocab, width, layers, attn, gru, moe, shared, chunk) -> dict:
-    """``config.json`` of a Giforax model: groups of an attention, one that reads its keys and values, and a recurrence.
+    """``config.json`` of a Giforax model: groups of a recurrence, an attention, and one that reads its keys and values.
     attn: (heads, kv_heads, dim, vdim, rotated), moe: (experts, top, ff, limit), shared: (ff, limit)."""
     sizes = lambda names, v: dict(zip(names.split(), v))
-    a = {**sizes("heads kv_heads dim vdim", attn), "scale": 2.0 * attn[2] ** -0.5, "rot": {"base": 50000.0, "dims": attn[4]},
+    a = {**sizes("heads kv_heads dim vdim", attn), "scale": 2.0 * attn[2] ** -0.5, "rot": {"base": 500000.0, "dims": attn[4]},
          "mask": {"size": chunk}}
     ff = {"kind": "moe", "router": sizes("experts top", moe), "expert": sizes("ff limit", moe[2:]),
           "shared": sizes("ff limit", shared)}
-    kinds = [("attention", lambda i: a), ("attention", lambda i: {**a, "kv_from": i - 1}), ("mingru", lambda i: {"width": gru})]
+    kinds = [("mingru", lambda i: {"width": gru}), ("attention", lambda i: a), ("attention", lambda i: {**a, "kv_from": i - 1})]
     return {"architecture": "Giforax", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
             "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1](i), "mlp": ff} for i in range(layers)]}
 
