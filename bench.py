@@ -54,7 +54,8 @@ def parse_args():
     ap.add_argument("--workload", default="prefill", choices=["prefill", "hybrid", "kebopel", "netezen", "giforax"],
                     help="hybrid: the hybrid decoder (latent attention + Mamba-2) beside the Llama layout at equal size, "
                          "prefill, decode and every kernel (artifact/hybrid_bench.py); kebopel: the same for Kebopel "
-                         "(artifact/kebopel_bench.py); netezen, giforax: these beside the Mixtral layout (artifact/netezen_bench.py, giforax_bench.py); "
+                         "(artifact/kebopel_bench.py); netezen, giforax: these beside the Mixtral layout "
+                         "(artifact/netezen_bench.py, artifact/giforax_bench.py); "
                          "one GPU")
     ap.add_argument("--cuda-graphs", dest="cuda_graphs", action="store_true", default=None,
                     help="replay the step from a CUDA graph (captured during warm-up; the default when --warmup >= 3)")

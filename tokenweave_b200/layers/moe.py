@@ -46,7 +46,8 @@ def run_experts(x: torch.Tensor, topk_w: torch.Tensor, topk_ids: torch.Tensor, w
                 gate: Optional[torch.Tensor] = None, pair_tiles: bool = True, max_ctas: int = 0,
                 weigh_input: bool = False) -> None:
     """``out = sum_k w_k W2[e_k] act(W13[e_k] x) (+ gate * shared, no gate: one)`` (CUDA); ``weigh_input``: the weight is on
-    the expert's input, ``W2[e_k] act(W13[e_k] (w_k x))``. ``ws``: the buffers of :func:`expert_index` and the expert-sorted rows ``a_sorted``, ``act`` and ``y`` (in fp32 also ``gate_up``: that product has no gated form)."""
+    the expert's input, ``W2[e_k] act(W13[e_k] (w_k x))``. ``ws``: the buffers of :func:`expert_index` and the expert-sorted rows
+    ``a_sorted``, ``act`` and ``y`` (in fp32 also ``gate_up``: that product has no gated form)."""
     T, top_k = topk_ids.shape
     E, I2, H = w13.shape
     tile_rows = TILE_ROWS_PAIR if T * top_k >= 512 * E and pair_tiles else TILE_ROWS
